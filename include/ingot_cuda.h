@@ -267,6 +267,100 @@ int ingot_attn_layers_host(ingot_kv* kv, int layer_begin, int layer_count, const
                            int n_tok, void* stream);
 int ingot_stream_sync(void* stream);
 
+/* ---- Recurrent mixers and shared-row attention over a ragged batch ---------------------------------
+ * No counterpart in the reference, whose models are attention-only with one sequence per call. A step carries, for each of
+ * n_seq sequences, its next len tokens; the tokens are rows 0..n_tok-1 of every activation matrix, sequence after sequence.
+ * All arrays are device memory (the struct itself is host memory, read during the call). */
+typedef struct ingot_step {
+    int n_tok, n_seq;
+    int max_len;               /* host-side upper bound of len[] (sizes the launch grids) */
+    const int32_t* row_seq;    /* [n_tok] sequence (index within the step) of each row */
+    const int32_t* row_start;  /* [n_seq] first row */
+    const int32_t* len;        /* [n_seq] */
+    const int32_t* pos0;       /* [n_seq] position of the first token; 0 starts from the zero state whatever the slot holds */
+    const int32_t* slot;       /* [n_seq] state slot */
+} ingot_step;
+
+/* Time chunks of a step for the recurrences: every sequence's len tokens cut into runs, sequence after sequence. */
+typedef struct ingot_scan_plan {
+    int n_chunks;
+    int max_chunks;             /* most chunks any one sequence has: 1 = no chunk needs another's end state */
+    const int32_t* chunk_seq;   /* [n_chunks] */
+    const int32_t* chunk_t0;    /* [n_chunks] first token, counted from the sequence's first in this step */
+    const int32_t* chunk_len;   /* [n_chunks] */
+    const int32_t* seq_chunk0;  /* [n_seq + 1] */
+    float* scratch_dev;         /* partial states; see the entry points for its size. May be null if max_chunks is 1 */
+    size_t scratch_floats;
+} ingot_scan_plan;
+
+/* Where a kernel leaves an activation matrix [n_tok][ld]: f32 rows, and / or a bf16 plane, or a bf16 hi + lo pair (the
+ * operands of the projection kernels). Null pointers are skipped. */
+typedef struct ingot_act_out {
+    float* f32;
+    void *hi, *lo;
+    int ld;
+} ingot_act_out;
+
+/* Per-channel causal convolution with carried history:
+ *   out[t][c] = act(bias[c] + sum_j w[c][j] (in[t - (taps-1) + j][c] + in_bias[c])), zeros before position 0; act: silu or none.
+ * state_dev [slot][taps-1][channels]: the last taps-1 inputs (in + in_bias), oldest first; read and replaced. 1 <= taps <= 16.
+ * in rows are in_ld floats apart; in_bias and bias may be null. */
+int ingot_causal_conv(const ingot_step* step, const float* in_dev, int in_ld, const float* in_bias_dev, const float* w_dev,
+                      const float* bias_dev, int taps, int channels, int silu, float* state_dev, const ingot_act_out* out,
+                      void* stream);
+
+/* States per channel as stored: n_state rounded up (at least to a multiple of 8); 0 if n_state is not supported (1..256). */
+int ingot_scan_state_pad(int n_state);
+/* Selective scan: with dt = softplus(dt_dev + dt_bias), per channel c and state n
+ *   S[c][n] <- exp(dt A[c][n]) S[c][n] + dt x[c] B[n];  y[c] = sum_n S[c][n] C[n] + D[c] x[c];  out[c] = y[c] * silu(z[c]).
+ * a_log2e_dev [inner][pad] = A * log2(e), zeros in the padding; B and C are the n_state columns at b_off / c_off of the rows of
+ * bc_dev (pad columns are read, the ones beyond n_state must be finite). state_dev [slot][inner][pad] f32, read and replaced.
+ * exact: decays through expm1 instead of the hardware 2^x (see csrc/recurrent.cu).
+ * Scratch: n_chunks * inner * (pad + 1) floats. inner, row lengths and offsets are multiples of 4. */
+int ingot_selective_scan(const ingot_step* step, const ingot_scan_plan* plan, const float* x_dev, int x_ld, const float* dt_dev,
+                         int dt_ld, const float* dt_bias_dev, const float* bc_dev, int bc_ld, int b_off, int c_off,
+                         const float* z_dev, int z_ld, const float* a_log2e_dev, const float* d_dev, float* state_dev, int inner,
+                         int n_state, int exact, const ingot_act_out* out, void* stream);
+
+/* Real-gated linear recurrent unit with its output gate:
+ *   r = sigmoid(g_r + r_bias), i = sigmoid(g_i + i_bias), log a = -8 r softplus(lam),
+ *   S <- a S + sqrt(1 - a^2) i u;  out = out_scale * S * gelu_tanh(y + y_bias).
+ * gates_dev rows hold, for each block of `block` channels, its g_r and then its g_i. state_dev [slot][width] f32, read and
+ * replaced. Scratch: 2 * n_chunks * width floats. */
+int ingot_gated_lru(const ingot_step* step, const ingot_scan_plan* plan, const float* u_dev, int u_ld, const float* gates_dev,
+                    int gates_ld, int block, const float* r_bias_dev, const float* i_bias_dev, const float* softplus_lam_dev,
+                    const float* y_dev, int y_ld, const float* y_bias_dev, float* state_dev, int width, float out_scale,
+                    const ingot_act_out* out, void* stream);
+
+/* Shared-row cache: one row per token and KV head is key and value at once (the value is the projection itself, the key the
+ * projection normalised over all KV heads), paged in 16-position blocks, with causal or chunk-local visibility.
+ * chunk > 0: position i sees j <= i of its own run of `chunk` positions counted from position 0; page of position p =
+ * (p / chunk) * ceil(chunk / 16) + (p % chunk) / 16. chunk 0: plain causal, page p / 16. Rows [page][n_head_kv][16][head_dim]
+ * f32 or f16 (head_dim even, <= 512, zero-padded heads allowed). Allocates on the current device; synchronous. */
+typedef struct ingot_skv ingot_skv;
+int ingot_skv_create(ingot_skv** out, int n_layer, int n_head_kv, int head_dim, int dtype, int chunk, int n_blocks);
+void ingot_skv_destroy(ingot_skv* kv);
+/* Pages that positions 0..n_positions-1 of one sequence span. */
+int ingot_skv_pages(int chunk, int n_positions);
+/* Row length to create an f16 cache with for heads of this size (the layout the tensor-core kernels take). */
+int ingot_skv_row_length(int head_size);
+/* The device status word itself, for callers that read several of them with their own copies. */
+int* ingot_skv_status_dev(ingot_skv* kv);
+/* Reads and clears the device status word (bit 2: a block-table entry outside the pool; the access was skipped). */
+int ingot_skv_status(ingot_skv* kv, void* stream, int* status_out);
+/* Query / key normalisation and append: columns q_off.. (n_head * head_dim) and k_off.. (n_head_kv * head_dim) of proj_dev's rows
+ * (f32, proj_ld apart) are the projections, heads padded to head_dim with zeros, head_size their true size. Writes the cache rows
+ * of the step's positions, and q_out_dev [n_tok][n_head][head_dim] in the cache's type: q / rms(q) * q_norm * k_norm, the key norm
+ * weight folded in. q_norm_dev [n_head * head_dim], k_norm_dev [n_head_kv * head_dim], zero in the padding.
+ * tables_dev [n_seq][max_blocks]: blocks of the step's sequences, entry 0 of a row being page first_page_dev[seq] (null: page 0). */
+int ingot_skv_append(ingot_skv* kv, int layer, const ingot_step* step, const float* proj_dev, int proj_ld, int q_off, int k_off,
+                     int n_head, int head_size, const float* q_norm_dev, const float* k_norm_dev, float eps, void* q_out_dev,
+                     const int32_t* tables_dev, const int32_t* first_page_dev, int max_blocks, void* stream);
+/* Softmax over the visible keys of every row (appended before), scores = q . k_row / rms(k) * scale; out[t][h * out_dim + d] =
+ * out_scale * result for d < out_dim. impl: 0 = library's choice, 1 = the plain f32-arithmetic kernel. */
+int ingot_skv_attend(ingot_skv* kv, int layer, const ingot_step* step, const void* q_dev, int n_head, int out_dim, float scale,
+                     float out_scale, const ingot_act_out* out, const int32_t* tables_dev, const int32_t* first_page_dev, int max_blocks, int impl, void* stream);
+
 /* ---- Diagnostics ----------------------------------------------------------------------------------
  * HBM read-bandwidth probe: what the reference's `bwtest` verb measures (src/main.cpp:450-455,
  * MetalBackend::bandwidth_test src/metal_backend.mm:533-592 with the bw_fill / bw_sum kernels,

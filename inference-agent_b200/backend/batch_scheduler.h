@@ -2,9 +2,10 @@
 //
 // The reference serves one request at a time: tokenise, prefill, then sample / forward until a stop token or the
 // token limit (src/server.cpp:139-140, 164-184). This scheduler runs that same per-request loop for up to
-// max_seqs() requests at once. Every step() makes ONE forward_multi call that carries one token of each running
-// request - the next token of its prompt while it is still being read in, afterwards the token it sampled last -
-// so requests that arrive at different times and are at different phases ride in the same launches. A finished
+// max_seqs() requests at once. Every step() makes ONE backend call that carries tokens of each running request - the next
+// token of its prompt, or on a backend that takes portions (max_portion() > 1) the next run of prompt tokens, while it is
+// still being read in, afterwards the token it sampled last - so requests that arrive at different times and are at
+// different phases ride in the same launches. Decoded tokens go first; prompts share what is left of max_step_tokens(). A finished
 // request gives its cache blocks back (release_sequence) and its slot goes to the next queued request.
 //
 // Per request the observable behaviour is the reference loop's: the same Sampler (src/sampler.h) over the
@@ -23,14 +24,15 @@
 #include <vector>
 
 #include "batched_backend.h"
-#include "sampler.h"
 
-class BatchScheduler {
+// SamplerT: sample(logits, history) and a constructor from (ParamsT, n_vocab), as the reference's src/sampler.h has them.
+template <class SamplerT, class ParamsT>
+class BasicBatchScheduler {
 public:
     struct Request {
         std::vector<int32_t> prompt;
         int max_tokens = 128;
-        SamplerParams sampling;                  // temperature 0 = greedy (the default)
+        ParamsT sampling;                        // temperature 0 = greedy (the default)
         std::function<bool(int32_t)> is_stop;    // empty: the reply only ends on the token limit
         std::function<void(int32_t)> on_token;   // empty, or called for every token as it joins the reply
     };
@@ -39,7 +41,7 @@ public:
         const char* finish = nullptr;            // nullptr while queued or running, then "stop", "length" or "cancelled"
     };
 
-    BatchScheduler(BatchedBackend& backend, int n_vocab)
+    BasicBatchScheduler(BatchedBackend& backend, int n_vocab)
         : backend_(backend), n_vocab_(n_vocab), slots_(size_t(backend.max_seqs())) {
         if (n_vocab < 1) throw std::runtime_error("scheduler: vocabulary size must be positive");
     }
@@ -73,29 +75,55 @@ public:
             queue_.pop_front();
             const Request& r = requests_[size_t(slot.request)];
             slot.history = r.prompt;
-            slot.sampler = std::make_unique<Sampler>(r.sampling, n_vocab_);
+            slot.sampler = std::make_unique<SamplerT>(r.sampling, n_vocab_);
         }
-        tok_.clear(); seq_.clear(); pos_.clear();
+        entries_.clear(); want_.clear(); carried_.clear();
+        want_.resize(slots_.size());
+        int budget = std::max(backend_.max_step_tokens(), int(slots_.size()));
+        int reading = 0;  // requests still inside their prompt; each is sure of one token
+        for (const Slot& slot : slots_)
+            if (slot.request >= 0) {
+                if (slot.fed < int(requests_[size_t(slot.request)].prompt.size())) reading++;
+                else budget--;
+            }
         for (size_t s = 0; s < slots_.size(); s++) {
             const Slot& slot = slots_[s];
             if (slot.request < 0) continue;
             const Request& r = requests_[size_t(slot.request)];
-            tok_.push_back(slot.fed < int(r.prompt.size()) ? r.prompt[size_t(slot.fed)] : slot.next);
-            seq_.push_back(int32_t(s));
-            pos_.push_back(slot.fed);
+            StepEntry e;
+            e.seq_id = int32_t(s);
+            e.pos0 = slot.fed;
+            const int left = int(r.prompt.size()) - slot.fed;
+            if (left > 0) {
+                e.tokens = r.prompt.data() + slot.fed;
+                e.n_tokens = std::max(1, std::min({left, backend_.max_portion(), budget - (reading - 1)}));
+                budget -= e.n_tokens;
+                reading--;
+            } else {
+                e.tokens = &slot.next;
+                e.n_tokens = 1;
+            }
+            if (e.n_tokens >= left) {  // the portion reaches the end of the prompt (or is a decoded token): sample from its last row
+                want_[s] = e.n_tokens - 1;
+                e.want = &want_[s];
+                e.n_want = 1;
+            }
+            entries_.push_back(e);
+            carried_.push_back(e.n_tokens);
         }
-        if (tok_.empty()) return false;
-        const float* logits = backend_.forward_multi(tok_.data(), seq_.data(), pos_.data(), int(tok_.size()));
+        if (entries_.empty()) return false;
+        const float* logits = backend_.forward_step(entries_.data(), int(entries_.size()), n_vocab_);
         steps_++;
-        rows_ += tok_.size();
-        for (size_t i = 0; i < seq_.size(); i++) {
-            Slot& slot = slots_[size_t(seq_[i])];
+        size_t row_i = 0;
+        for (size_t i = 0; i < entries_.size(); i++) {
+            Slot& slot = slots_[size_t(entries_[i].seq_id)];
             const Request& r = requests_[size_t(slot.request)];
             Result& out = results_[size_t(slot.request)];
-            slot.fed++;
-            if (slot.fed < int(r.prompt.size())) continue;  // still inside the prompt: these logits are not sampled
+            rows_ += carried_[i];
+            slot.fed += carried_[i];
+            if (!entries_[i].n_want) continue;  // still inside the prompt: nothing to sample
             // the backend's logits are writable host memory (the sampler edits them in place, as in the reference)
-            float* row = const_cast<float*>(logits) + i * size_t(n_vocab_);
+            float* row = const_cast<float*>(logits) + (row_i++) * size_t(n_vocab_);
             const int32_t next = slot.sampler->sample(row, slot.history);
             if (r.is_stop && r.is_stop(next)) {
                 finish(slot, out, "stop");
@@ -130,7 +158,7 @@ public:
         for (const Slot& s : slots_) n += s.request >= 0;
         return n;
     }
-    long long steps() const { return steps_; }   // forward_multi calls so far
+    long long steps() const { return steps_; }   // backend calls so far
     long long rows() const { return rows_; }     // tokens those calls carried
 
 private:
@@ -139,7 +167,7 @@ private:
         int fed = 0;                  // tokens of this request the backend has seen = position of the next one
         int32_t next = 0;             // sampled and not yet fed
         std::vector<int32_t> history; // prompt + reply, what the sampler's repetition penalty looks at
-        std::unique_ptr<Sampler> sampler;
+        std::unique_ptr<SamplerT> sampler;
     };
 
     void finish(Slot& slot, Result& out, const char* why) {
@@ -155,6 +183,8 @@ private:
     std::deque<Request> requests_;   // deques: references stay valid when a callback submits a new request
     std::deque<Result> results_;
     std::deque<int> queue_;
-    std::vector<int32_t> tok_, seq_, pos_;
+    std::vector<StepEntry> entries_;
+    std::vector<int32_t> want_;
+    std::vector<int> carried_;
     long long steps_ = 0, rows_ = 0;
 };

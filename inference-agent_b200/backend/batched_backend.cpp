@@ -1,5 +1,5 @@
-// make_batched_backend: the batched interface over a named backend (see batched_backend.h).
-#include "batched_backend.h"
+// make_batched_backend: the batched interface over a named backend (see gguf_batched_backend.h).
+#include "gguf_batched_backend.h"
 
 #include <cstring>
 #include <stdexcept>

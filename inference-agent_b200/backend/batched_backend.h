@@ -12,11 +12,18 @@
 #pragma once
 
 #include <cstdint>
-#include <memory>
-#include <string>
+#include <stdexcept>
+#include <vector>
 
-#include "gguf.h"
-#include "model.h"
+// The next tokens of one sequence in a step, and the places among them whose logits are asked for.
+struct StepEntry {
+    int32_t seq_id = 0;
+    int32_t pos0 = 0;                  // position of tokens[0]
+    const int32_t* tokens = nullptr;
+    int32_t n_tokens = 0;
+    const int32_t* want = nullptr;     // indices into tokens, ascending
+    int32_t n_want = 0;
+};
 
 class BatchedBackend {
 public:
@@ -27,19 +34,48 @@ public:
     // messages for a bad token id ("token id out of range") or position ("context window exceeded"), and for a
     // repeated or out-of-range sequence id.
     virtual const float* forward_multi(const int32_t* tokens, const int32_t* seq_ids, const int32_t* positions, int n) = 0;
+    // The general step: one batch of portions of n DIFFERENT sequences, of one or more tokens each (portions of prompts beside
+    // single decoded tokens). Returns the wanted rows of n_vocab logits in the order of the entries and of their `want` (writable
+    // host memory, valid until the next call), or null if nothing is wanted. This default feeds a backend that takes one token
+    // of a sequence per call; such a backend needs no portions, so max_portion() tells callers not to make any.
+    virtual const float* forward_step(const StepEntry* entries, int n, int n_vocab) {
+        int longest = 0;
+        for (int i = 0; i < n; i++) longest = entries[i].n_tokens > longest ? entries[i].n_tokens : longest;
+        size_t total = 0;
+        std::vector<size_t> first(static_cast<size_t>(n));
+        for (int i = 0; i < n; i++) { first[size_t(i)] = total; total += size_t(entries[i].n_want); }
+        step_logits_.resize(total * size_t(n_vocab));
+        for (int t = 0; t < longest; t++) {
+            std::vector<int32_t> tok, seq, pos;
+            std::vector<int> src;
+            for (int i = 0; i < n; i++) {
+                if (t >= entries[i].n_tokens) continue;
+                tok.push_back(entries[i].tokens[t]);
+                seq.push_back(entries[i].seq_id);
+                pos.push_back(entries[i].pos0 + t);
+                src.push_back(i);
+            }
+            const float* rows = forward_multi(tok.data(), seq.data(), pos.data(), int(tok.size()));
+            for (size_t r = 0; r < src.size(); r++) {
+                const StepEntry& e = entries[src[r]];
+                for (int w = 0; w < e.n_want; w++)
+                    if (e.want[w] == t) {
+                        const float* from = rows + r * size_t(n_vocab);
+                        float* to = step_logits_.data() + (first[size_t(src[r])] + size_t(w)) * size_t(n_vocab);
+                        for (int v = 0; v < n_vocab; v++) to[v] = from[v];
+                    }
+            }
+        }
+        return total ? step_logits_.data() : nullptr;
+    }
+    // Most tokens of one sequence that a step may carry with profit (1: single tokens only), and most tokens of a step.
+    virtual int max_portion() const { return 1; }
+    virtual int max_step_tokens() const { return max_seqs(); }
     // Gives a sequence's cache blocks back to the pool (its id can then serve a new request).
     virtual void release_sequence(int seq_id) = 0;
     virtual int max_seqs() const = 0;
     virtual int n_ctx_per_seq() const = 0;
+
+private:
+    std::vector<float> step_logits_;  // of the default forward_step
 };
-
-// max_seqs sequences of up to n_ctx_per_seq positions each share one paged cache (16-token blocks handed out on
-// demand). Throws like make_cuda_backend.
-std::unique_ptr<BatchedBackend> make_cuda_batched_backend(const gguf::File& file, const Model& model, int n_ctx_per_seq, int max_seqs);
-
-// The batched interface over a named backend. "cuda" (or "metal", the name the reference's engine knows its GPU
-// backend by) is make_cuda_batched_backend. Any other name the reference's make_backend accepts ("cpu") gets one
-// single-sequence backend instance per sequence slot, stepped one after another: no sharing of launches, but the
-// same interface and the same results, e.g. to run a serving loop written against forward_multi without a GPU.
-std::unique_ptr<BatchedBackend> make_batched_backend(const std::string& name, const gguf::File& file, const Model& model,
-                                                     int n_ctx_per_seq, int max_seqs);

@@ -17,7 +17,7 @@
 // This file also defines make_metal_backend and the four metal_* diagnostics, so that the reference's
 // engine.cpp / main.cpp link against this backend without a source edit.
 #include "cuda_backend.h"
-#include "batched_backend.h"
+#include "gguf_batched_backend.h"
 
 #include <cuda_fp16.h>
 #include <cuda_runtime.h>
@@ -32,9 +32,12 @@
 #include <algorithm>
 #include <vector>
 
+#include "block_pool.h"
+#include "cuda_util.h"
 #include "ingot_cuda.h"
 #include "metal_backend.h"
 #include "ops.h"
+#include "weight_streamer.h"
 
 extern "C" {
 cudaError_t ingot_support_rmsnorm(float* out, const float* x, const float* w, int n_rows, int n, float eps, cudaStream_t s);
@@ -75,13 +78,6 @@ int ingot_linear_ws_status(ingot_linear_ws* ws);
 
 namespace {
 
-void cuda_check(cudaError_t e, const char* what) {
-    if (e != cudaSuccess) throw std::runtime_error(std::string("cuda: ") + what + ": " + cudaGetErrorString(e));
-}
-void ingot_check(int rc) {
-    if (rc != INGOT_OK) throw std::runtime_error(ingot_last_error()[0] ? ingot_last_error() : ingot_status_string(rc));
-}
-
 struct DevWeight {
     void* data = nullptr;  // f32 / f16 rows, or the repacked planes of a block-quantised matrix (quant_kernels.cu)
     int is_f16 = 0;
@@ -91,51 +87,6 @@ struct DevWeight {
     // format code of the weight-streaming single-token kernel (support_kernels.cu): 0 f16, 1 Q8_0, 2 Q4_0, -1 none
     int stream_fmt() const { return is_f16 ? 0 : qtype == 8 ? 1 : qtype == 2 ? 2 : -1; }
     int n_in = 0, n_out = 0;
-};
-
-// Streams weights from the memory-mapped model file to the device through a small ring of pinned staging buffers:
-// the CPU copy of chunk i+1 out of the page cache (where the page faults and disk reads happen) overlaps the DMA
-// of chunk i, and no call blocks on a pageable copy. The Metal backend wraps the mmap without copying
-// (src/metal_backend.mm:213-246); a discrete GPU has to move the bytes once, so they move as a stream.
-class WeightStreamer {
-public:
-    WeightStreamer() {
-        cuda_check(cudaStreamCreateWithFlags(&stream_, cudaStreamNonBlocking), "cudaStreamCreate(load)");
-        for (int i = 0; i < kBufs; i++) {
-            cuda_check(cudaMallocHost(&buf_[i], kChunk), "cudaMallocHost(load staging)");
-            cuda_check(cudaEventCreateWithFlags(&done_[i], cudaEventDisableTiming), "cudaEventCreate");
-        }
-    }
-    ~WeightStreamer() {
-        cudaStreamSynchronize(stream_);
-        for (int i = 0; i < kBufs; i++) { cudaFreeHost(buf_[i]); cudaEventDestroy(done_[i]); }
-        cudaStreamDestroy(stream_);
-    }
-    void copy(void* dst_dev, const void* src_host, size_t bytes) {
-        const char* src = static_cast<const char*>(src_host);
-        char* dst = static_cast<char*>(dst_dev);
-        for (size_t off = 0; off < bytes; off += kChunk) {
-            const size_t n = std::min(kChunk, bytes - off);
-            const int b = next_++ % kBufs;
-            cuda_check(cudaEventSynchronize(done_[b]), "load staging");  // the DMA that last read this buffer is over
-            memcpy(buf_[b], src + off, n);
-            cuda_check(cudaMemcpyAsync(dst + off, buf_[b], n, cudaMemcpyHostToDevice, stream_), "cudaMemcpyAsync(weight)");
-            cuda_check(cudaEventRecord(done_[b], stream_), "cudaEventRecord");
-            bytes_ += n;
-        }
-    }
-    cudaStream_t stream() const { return stream_; }
-    void finish() { cuda_check(cudaStreamSynchronize(stream_), "weight upload"); }
-    size_t bytes() const { return bytes_; }
-
-private:
-    static constexpr int kBufs = 4;
-    static constexpr size_t kChunk = size_t(32) << 20;
-    cudaStream_t stream_ = nullptr;
-    void* buf_[kBufs] = {};
-    cudaEvent_t done_[kBufs] = {};
-    unsigned next_ = 0;
-    size_t bytes_ = 0;
 };
 
 class CudaBackend : public Backend, public BatchedBackend {
@@ -158,9 +109,7 @@ public:
             blocks_per_seq_ = (n_ctx + INGOT_BLOCK_TOKENS - 1) / INGOT_BLOCK_TOKENS;
             const int n_blocks = blocks_per_seq_ * max_seqs_;
             ingot_check(ingot_kv_create(&kv_, INGOT_KV_PAGED, c.n_layer, c.n_head_kv, c.head_dim, n_blocks, max_seqs_));
-            block_table_.assign(size_t(max_seqs_) * blocks_per_seq_, -1);
-            // Blocks are handed out in arrival order, so the sequences' blocks interleave in the pool.
-            for (int b = n_blocks - 1; b >= 0; b--) free_blocks_.push_back(b);
+            pool_ = BlockPool(n_blocks, max_seqs_, blocks_per_seq_);
         } else {
             ingot_check(ingot_kv_create(&kv_, INGOT_KV_CONTIGUOUS, c.n_layer, c.n_head_kv, c.head_dim, n_ctx, 1));
         }
@@ -476,14 +425,9 @@ public:
         }
         for (int i = 0; i < n; i++) {
             // the block that holds this position is taken from the pool when the sequence first reaches it
-            int32_t* row = block_table_.data() + size_t(seq_ids[i]) * blocks_per_seq_;
-            const int blk = positions[i] / INGOT_BLOCK_TOKENS;
-            for (int b = 0; b <= blk; b++) {  // a sequence may start beyond position 0 only over blocks it owns
-                if (row[b] >= 0) continue;
-                if (free_blocks_.empty()) throw std::runtime_error("context window exceeded");
-                row[b] = free_blocks_.back();
-                free_blocks_.pop_back();
-            }
+            // (a sequence may start beyond position 0 only over blocks it owns)
+            pool_.ensure(seq_ids[i], 0, positions[i] / INGOT_BLOCK_TOKENS);
+            const int32_t* row = pool_.row(seq_ids[i]);
             tok_host_[i] = tokens[i];
             pos_h[i] = positions[i];
             len_h[i] = positions[i] + 1;
@@ -504,9 +448,7 @@ public:
     }
     void release_sequence(int seq_id) override {
         if (seq_id < 0 || seq_id >= max_seqs_) throw std::runtime_error("cuda: sequence id out of range");
-        int32_t* row = block_table_.data() + size_t(seq_id) * blocks_per_seq_;
-        for (int b = 0; b < blocks_per_seq_; b++)
-            if (row[b] >= 0) { free_blocks_.push_back(row[b]); row[b] = -1; }
+        pool_.release(seq_id);
     }
     int max_seqs() const override { return max_seqs_; }
     int n_ctx_per_seq() const override { return n_ctx_; }
@@ -673,8 +615,7 @@ private:
     const Model& m_;
     int n_ctx_, n_batch_;
     int max_seqs_ = 0, blocks_per_seq_ = 0;       // batched form: paged cache shared by max_seqs_ sequences
-    std::vector<int32_t> block_table_;            // [max_seqs_][blocks_per_seq_], -1 = not allocated
-    std::vector<int32_t> free_blocks_;
+    BlockPool pool_;
     int32_t *multi_dev_ = nullptr, *multi_host_ = nullptr;  // per step: positions, key counts, row ids [max_seqs_ each], block-table rows
     cudaStream_t stream_ = nullptr;
     ingot_kv* kv_ = nullptr;

@@ -10,8 +10,8 @@
 #include <string>
 #include <vector>
 
-#include "batch_scheduler.h"
-#include "batched_backend.h"
+#include "gguf_scheduler.h"
+#include "gguf_batched_backend.h"
 #include "engine.h"
 #include "metal_backend.h"
 #include "gguf.h"

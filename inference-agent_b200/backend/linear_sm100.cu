@@ -13,6 +13,12 @@
 // near 1e-3). The weights are used as stored, the products are exact, the accumulation is f32: the result
 // differs from the reference only by summation order and that truncation of x.
 //
+// bf16 models (ingot_linear_ws_create_bf16). The same kernel on bf16 weights with the activations as one bf16 plane (plain
+// bf16 products) or as a hi + lo pair (16 significant bits, for products that feed a recurrence's gates); the number of
+// planes is chosen per product. Rows of any length that is a multiple of 8 are accepted (the last k-step is zero-filled
+// by TMA), and a matrix may be block-diagonal: output tiles of block b then read the k_block activation columns that
+// start at b * k_block.
+//
 // Kernel. One CTA = 128 tokens x 128 outputs over a slice of k (split-k fills the GPU when there are few
 // output tiles; slices go to a scratch and are summed in slice order, by a small kernel or by the kernel
 // that consumes the product, so results are reproducible). 6 warps: warp 0 streams [128 rows][64 k] boxes of hi, lo and W (128-byte swizzle, 48 KB per
@@ -22,6 +28,7 @@
 // Every mbarrier wait is bounded; on expiry the CTA raises the workspace's status word and leaves.
 #include "../csrc/sm100_ptx.cuh"
 
+#include <cuda_bf16.h>
 #include <cuda_fp16.h>
 
 #include <algorithm>
@@ -38,15 +45,21 @@ using namespace ingot_sm100;
 #endif
 constexpr int kBM = 128, kBN = INGOT_GEMM_BN, kBK = 64;  // outputs per CTA: 128, or 256 (a third less L2 traffic per output)
 static_assert(kBN == 128 || kBN == 256, "128 or 256 outputs per CTA");
-constexpr int kStages = kBN == 256 ? 3 : 4;
+constexpr int kMaxStages = 6;
 constexpr int kBoxBytes = 128 * kBK * 2;        // 16 KB: 128 rows x 64 f16
 constexpr int kWBytes = kBN * kBK * 2;          // the W box: kBN rows
-constexpr int kStageBytes = 2 * kBoxBytes + kWBytes;  // hi, lo, W
 constexpr int kThreads = 192;
-constexpr int kOffBar = kStages * kStageBytes;
-constexpr int kSmemBytes = kOffBar + 128 + 1024;  // barriers + alignment slack
+template <int kPlanes>
+struct Ring {
+    static constexpr int kStageBytes = kPlanes * kBoxBytes + kWBytes;  // hi(, lo), W
+    static constexpr int kStages = 196608 / kStageBytes;               // 192 KB ring: 4 stages of 48 KB or 6 of 32 KB
+    static constexpr int kOffBar = kStages * kStageBytes;
+    static constexpr int kSmemBytes = kOffBar + 256 + 1024;            // barriers + alignment slack
+    static_assert(kStages <= kMaxStages, "barrier arrays");
+};
 constexpr uint32_t kTmemCols = kBN;
-constexpr uint32_t kIdesc = (1u << 4) | ((uint32_t)(kBN >> 3) << 17) | ((uint32_t)(kBM >> 4) << 24);  // f16 x f16 -> f32, both K-major
+constexpr uint32_t kIdescF16 = (1u << 4) | ((uint32_t)(kBN >> 3) << 17) | ((uint32_t)(kBM >> 4) << 24);  // f16 x f16 -> f32, both K-major
+constexpr uint32_t kIdescBF16 = kIdescF16 | (1u << 7) | (1u << 10);                                        // bf16 x bf16 -> f32
 constexpr unsigned long long kWaitLimitNs = 2000000000ull;
 
 __device__ __forceinline__ uint32_t smem_u32(const void* p) { return (uint32_t)__cvta_generic_to_shared(p); }
@@ -73,8 +86,8 @@ static cudaError_t launch_pdl(void (*kernel)(KArgs...), dim3 grid, dim3 block, s
 }
 
 struct Bars {
-    uint64_t full[kStages];
-    uint64_t empty[kStages];
+    uint64_t full[kMaxStages];
+    uint64_t empty[kMaxStages];
     uint64_t done;
     uint32_t tmem_base;
     uint32_t abort_flag;
@@ -88,13 +101,18 @@ struct GemmParams {
     int* status;
     int n_tok, k_steps, n_split, accumulate;
     int n_out[3], tile_end[3];
+    uint32_t idesc;
+    int rows_per_block, k_block, tiles_per_block;  // block-diagonal matrix (rows_per_block > 0, count == 1)
     int to_partial;  // write the slice(s) to `partial` even when there is only one (a consumer kernel sums them)
 };
 
+template <int kPlanes>
 __global__ void __launch_bounds__(kThreads, 1)
 linear_sm100_kernel(const __grid_constant__ CUtensorMap map_hi, const __grid_constant__ CUtensorMap map_lo,
                     const __grid_constant__ CUtensorMap map_w0, const __grid_constant__ CUtensorMap map_w1,
                     const __grid_constant__ CUtensorMap map_w2, const GemmParams p) {
+    constexpr int kStages = Ring<kPlanes>::kStages, kStageBytes = Ring<kPlanes>::kStageBytes, kOffBar = Ring<kPlanes>::kOffBar;
+    constexpr int kOffW = kPlanes * kBoxBytes;
     extern __shared__ unsigned char smem_dyn[];
     LINEAR_PDL_TRIGGER();
     const uint32_t smem_base = (smem_u32(smem_dyn) + 1023u) & ~1023u;
@@ -106,8 +124,12 @@ linear_sm100_kernel(const __grid_constant__ CUtensorMap map_hi, const __grid_con
     const int mat = ((int)blockIdx.x >= p.tile_end[0]) + ((int)blockIdx.x >= p.tile_end[1]);  // warp-uniform
     const CUtensorMap* const map_w_p = mat == 0 ? &map_w0 : mat == 1 ? &map_w1 : &map_w2;
     const int mat_n_out = mat == 0 ? p.n_out[0] : mat == 1 ? p.n_out[1] : p.n_out[2];
+    const int blk = p.tiles_per_block > 0 ? (int)blockIdx.x / p.tiles_per_block : 0;
+    const int col_end = p.tiles_per_block > 0 ? (blk + 1) * p.rows_per_block : mat_n_out;
+    const int a_k0 = blk * p.k_block;  // first activation column of this tile's products
     float* const mat_partial = mat == 0 ? p.partial[0] : mat == 1 ? p.partial[1] : p.partial[2];
-    const int n0 = ((int)blockIdx.x - (mat == 0 ? 0 : mat == 1 ? p.tile_end[0] : p.tile_end[1])) * kBN;
+    const int n0 = p.tiles_per_block > 0 ? blk * p.rows_per_block + ((int)blockIdx.x - blk * p.tiles_per_block) * kBN
+                                         : ((int)blockIdx.x - (mat == 0 ? 0 : mat == 1 ? p.tile_end[0] : p.tile_end[1])) * kBN;
     const int m0 = blockIdx.y * kBM, split = blockIdx.z;
     const int ks_begin = (int)((long long)p.k_steps * split / p.n_split);
     const int ks_end = (int)((long long)p.k_steps * (split + 1) / p.n_split);
@@ -135,7 +157,7 @@ linear_sm100_kernel(const __grid_constant__ CUtensorMap map_hi, const __grid_con
         for (int it = 0; it < n_pre; it++) {
             const uint32_t full = smem_u32(&bars->full[it]);
             mbar_expect_tx(full, kStageBytes);
-            tma_load_2d(smem_base + it * kStageBytes + 2 * kBoxBytes, map_w_p, (ks_begin + it) * kBK, n0, full);
+            tma_load_2d(smem_base + it * kStageBytes + kOffW, map_w_p, (ks_begin + it) * kBK, n0, full);
         }
     }
     LINEAR_PDL_WAIT();
@@ -151,15 +173,15 @@ linear_sm100_kernel(const __grid_constant__ CUtensorMap map_hi, const __grid_con
                 const uint32_t dst = smem_base + s * kStageBytes;
                 const int k = (ks_begin + it) * kBK;
                 if (it < n_pre) {  // first use of the slot: armed and its W box requested before the wait above
-                    tma_load_2d(dst, &map_hi, k, m0, full);
-                    tma_load_2d(dst + kBoxBytes, &map_lo, k, m0, full);
+                    tma_load_2d(dst, &map_hi, a_k0 + k, m0, full);
+                    if (kPlanes > 1) tma_load_2d(dst + kBoxBytes, &map_lo, a_k0 + k, m0, full);
                 } else {
                     ok = mbar_wait(smem_u32(&bars->empty[s]), (uint32_t)(((it / kStages) & 1) ^ 1), abort_flag, kWaitLimitNs);
                     if (ok) {
                         mbar_expect_tx(full, kStageBytes);
-                        tma_load_2d(dst, &map_hi, k, m0, full);
-                        tma_load_2d(dst + kBoxBytes, &map_lo, k, m0, full);
-                        tma_load_2d(dst + 2 * kBoxBytes, map_w_p, k, n0, full);
+                        tma_load_2d(dst, &map_hi, a_k0 + k, m0, full);
+                        if (kPlanes > 1) tma_load_2d(dst + kBoxBytes, &map_lo, a_k0 + k, m0, full);
+                        tma_load_2d(dst + kOffW, map_w_p, k, n0, full);
                     }
                 }
             }
@@ -183,13 +205,15 @@ linear_sm100_kernel(const __grid_constant__ CUtensorMap map_hi, const __grid_con
             if (!ok) break;
             tc_fence_after();
             if (elect_one()) {
-                const uint32_t a_hi = smem_base + s * kStageBytes, a_lo = a_hi + kBoxBytes, b = a_hi + 2 * kBoxBytes;
+                const uint32_t a_hi = smem_base + s * kStageBytes, a_lo = a_hi + kBoxBytes, b = a_hi + kOffW;
 #pragma unroll
                 for (int ks = 0; ks < kBK / 16; ks++)
-                    tc_mma_ss(tmem, make_desc(a_hi + ks * 32, 16, 1024), make_desc(b + ks * 32, 16, 1024), kIdesc, (it > 0 || ks > 0) ? 1u : 0u);
+                    tc_mma_ss(tmem, make_desc(a_hi + ks * 32, 16, 1024), make_desc(b + ks * 32, 16, 1024), p.idesc, (it > 0 || ks > 0) ? 1u : 0u);
+                if (kPlanes > 1) {
 #pragma unroll
-                for (int ks = 0; ks < kBK / 16; ks++)
-                    tc_mma_ss(tmem, make_desc(a_lo + ks * 32, 16, 1024), make_desc(b + ks * 32, 16, 1024), kIdesc, 1u);
+                    for (int ks = 0; ks < kBK / 16; ks++)
+                        tc_mma_ss(tmem, make_desc(a_lo + ks * 32, 16, 1024), make_desc(b + ks * 32, 16, 1024), p.idesc, 1u);
+                }
                 tc_commit(smem_u32(&bars->empty[s]));
                 if (it == n_it - 1) tc_commit(smem_u32(&bars->done));
             }
@@ -215,14 +239,14 @@ linear_sm100_kernel(const __grid_constant__ CUtensorMap map_hi, const __grid_con
 #pragma unroll
                     for (int i = 0; i < 32; i += 4) {
                         const int col = n0 + c * 32 + i;
-                        if (col + 3 < mat_n_out) {
+                        if (col + 3 < col_end) {
                             float4* d4 = reinterpret_cast<float4*>(dst + c * 32 + i);
                             float4 o = make_float4(v[i], v[i + 1], v[i + 2], v[i + 3]);
                             if (add) { const float4 old = *d4; o.x += old.x; o.y += old.y; o.z += old.z; o.w += old.w; }
                             *d4 = o;
                         } else {
                             for (int e = 0; e < 4; e++)
-                                if (col + e < mat_n_out) dst[c * 32 + i + e] = add ? dst[c * 32 + i + e] + v[i + e] : v[i + e];
+                                if (col + e < col_end) dst[c * 32 + i + e] = add ? dst[c * 32 + i + e] + v[i + e] : v[i + e];
                         }
                     }
                 }
@@ -253,38 +277,48 @@ __global__ void splitk_reduce_kernel(float* out, const float* partial, int n_spl
     *reinterpret_cast<float4*>(out + i) = acc;
 }
 
-// hi = f16(x), lo = f16(x - hi)
-__global__ void split_f16_kernel(__half* hi, __half* lo, const float* x, size_t n) {
-    LINEAR_PDL_TRIGGER();
-    LINEAR_PDL_WAIT();
-    const size_t i = ((size_t)blockIdx.x * blockDim.x + threadIdx.x) * 4;
-    if (i >= n) return;
-    const float4 v = *reinterpret_cast<const float4*>(x + i);
-    const float f[4] = {v.x, v.y, v.z, v.w};
-    __half h[4], l[4];
+// How f32 activations become MMA operands: an f16 pair hi = f16(x), lo = f16(x - hi), one bf16 plane, or a bf16 pair.
+enum : int { kActF16Pair = 0, kActBF16 = 1, kActBF16Pair = 2 };
+template <int kAct>
+__device__ __forceinline__ void store_split4(__half* hi, __half* lo, size_t i, const float (&f)[4]) {
+    if (kAct == kActF16Pair) {
+        __half h[4], l[4];
 #pragma unroll
-    for (int e = 0; e < 4; e++) {
-        h[e] = __float2half_rn(f[e]);
-        l[e] = __float2half_rn(f[e] - __half2float(h[e]));
+        for (int e = 0; e < 4; e++) {
+            h[e] = __float2half_rn(f[e]);
+            l[e] = __float2half_rn(f[e] - __half2float(h[e]));
+        }
+        *reinterpret_cast<uint2*>(hi + i) = *reinterpret_cast<const uint2*>(h);
+        *reinterpret_cast<uint2*>(lo + i) = *reinterpret_cast<const uint2*>(l);
+    } else {
+        __nv_bfloat16 h[4], l[4];
+#pragma unroll
+        for (int e = 0; e < 4; e++) {
+            h[e] = __float2bfloat16_rn(f[e]);
+            l[e] = __float2bfloat16_rn(f[e] - __bfloat162float(h[e]));
+        }
+        *reinterpret_cast<uint2*>(hi + i) = *reinterpret_cast<const uint2*>(h);
+        if (kAct == kActBF16Pair) *reinterpret_cast<uint2*>(lo + i) = *reinterpret_cast<const uint2*>(l);
     }
-    *reinterpret_cast<uint2*>(hi + i) = *reinterpret_cast<const uint2*>(h);
-    *reinterpret_cast<uint2*>(lo + i) = *reinterpret_cast<const uint2*>(l);
 }
 
-__device__ __forceinline__ void store_split4(__half* hi, __half* lo, size_t i, const float (&f)[4]) {
-    __half h[4], l[4];
-#pragma unroll
-    for (int e = 0; e < 4; e++) {
-        h[e] = __float2half_rn(f[e]);
-        l[e] = __float2half_rn(f[e] - __half2float(h[e]));
-    }
-    *reinterpret_cast<uint2*>(hi + i) = *reinterpret_cast<const uint2*>(h);
-    *reinterpret_cast<uint2*>(lo + i) = *reinterpret_cast<const uint2*>(l);
+// x rows are x_ld floats apart, the planes' rows n; grid.y = row
+template <int kAct>
+__global__ void split_act_kernel(__half* hi, __half* lo, const float* x, int x_ld, int n) {
+    LINEAR_PDL_TRIGGER();
+    LINEAR_PDL_WAIT();
+    const int i = (blockIdx.x * blockDim.x + threadIdx.x) * 4;
+    if (i >= n) return;
+    const float4 v = *reinterpret_cast<const float4*>(x + (size_t)blockIdx.y * x_ld + i);
+    const float f[4] = {v.x, v.y, v.z, v.w};
+    store_split4<kAct>(hi, lo, (size_t)blockIdx.y * n + i, f);
 }
 
 // hi/lo of rmsnorm(x) = x * rsqrt(mean(x^2) + eps) * w, one CTA per token row (ops::rmsnorm, src/ops.cpp:227-232,
 // with the same expression order as the standalone norm kernel, so the split sees the same f32 values).
-__global__ void rmsnorm_split_kernel(__half* hi, __half* lo, const float* x, const float* w, int n, float eps) {
+// The mean is taken over n_mean of the row's n floats (rows zero-padded to an aligned length).
+template <int kAct>
+__global__ void rmsnorm_split_kernel(__half* hi, __half* lo, const float* x, const float* w, int n, int n_mean, float eps) {
     LINEAR_PDL_TRIGGER();
     LINEAR_PDL_WAIT();
     __shared__ float red[32];
@@ -299,14 +333,14 @@ __global__ void rmsnorm_split_kernel(__half* hi, __half* lo, const float* x, con
         float v = threadIdx.x < (blockDim.x >> 5) ? red[threadIdx.x] : 0.f;
 #pragma unroll
         for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
-        if (threadIdx.x == 0) red[0] = 1.0f / sqrtf(v / float(n) + eps);
+        if (threadIdx.x == 0) red[0] = 1.0f / sqrtf(v / float(n_mean) + eps);
     }
     __syncthreads();
     const float scale = red[0];
     for (int i = threadIdx.x * 4; i < n; i += blockDim.x * 4) {
         const float4 v = *reinterpret_cast<const float4*>(xr + i), g = *reinterpret_cast<const float4*>(w + i);
         const float f[4] = {v.x * scale * g.x, v.y * scale * g.y, v.z * scale * g.z, v.w * scale * g.w};
-        store_split4(hi, lo, (size_t)blockIdx.x * n + i, f);
+        store_split4<kAct>(hi, lo, (size_t)blockIdx.x * n + i, f);
     }
 }
 
@@ -344,7 +378,8 @@ __global__ void finish_group_kernel(const FinishGroup g, int n_tok) {
 
 // x[t][:] += sum of slices (the residual add of wo / down), then, if norm_w is given, hi/lo of rmsnorm(x[t]) for the
 // next projections. One CTA per token.
-__global__ void finish_residual_norm_kernel(float* x, const Slices in, __half* hi, __half* lo, const float* norm_w, int n, int n_tok,
+template <int kAct>
+__global__ void finish_residual_norm_kernel(float* x, const Slices in, __half* hi, __half* lo, const float* norm_w, int n, int n_mean, int n_tok,
                                             float eps) {
     __shared__ float red[32];
     LINEAR_PDL_TRIGGER();
@@ -366,14 +401,14 @@ __global__ void finish_residual_norm_kernel(float* x, const Slices in, __half* h
         float v = threadIdx.x < (blockDim.x >> 5) ? red[threadIdx.x] : 0.f;
 #pragma unroll
         for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
-        if (threadIdx.x == 0) red[0] = 1.0f / sqrtf(v / float(n) + eps);
+        if (threadIdx.x == 0) red[0] = 1.0f / sqrtf(v / float(n_mean) + eps);
     }
     __syncthreads();
     const float scale = red[0];
     for (int i = threadIdx.x * 4; i < n; i += blockDim.x * 4) {
         const float4 v = *reinterpret_cast<const float4*>(x + row + i), g = *reinterpret_cast<const float4*>(norm_w + i);
         const float f[4] = {v.x * scale * g.x, v.y * scale * g.y, v.z * scale * g.z, v.w * scale * g.w};
-        store_split4(hi, lo, row + i, f);
+        store_split4<kAct>(hi, lo, row + i, f);
     }
 }
 
@@ -387,7 +422,27 @@ __global__ void finish_swiglu_kernel(__half* hi, __half* lo, const Slices gate, 
     const float4 g = sum_slices(gate, i, n, z), u = sum_slices(up, i, n, z);
     const float f[4] = {g.x / (1.0f + expf(-g.x)) * u.x, g.y / (1.0f + expf(-g.y)) * u.y, g.z / (1.0f + expf(-g.z)) * u.z,
                         g.w / (1.0f + expf(-g.w)) * u.w};
-    store_split4(hi, lo, i, f);
+    store_split4<kActF16Pair>(hi, lo, i, f);
+}
+
+// One bf16 plane of act(gate) * up, where one product of width 2 n holds both: gate = columns 0..n-1, up = columns n..2n-1.
+// act: 0 silu, 1 the tanh form of gelu. grid.y = row.
+__global__ void finish_gated_kernel(__half* hi, const Slices in, int n, size_t slice, int act) {
+    LINEAR_PDL_TRIGGER();
+    LINEAR_PDL_WAIT();
+    const int i = (blockIdx.x * blockDim.x + threadIdx.x) * 4;
+    if (i >= n) return;
+    const size_t row = (size_t)blockIdx.y * 2 * n;
+    const float4 z = make_float4(0.f, 0.f, 0.f, 0.f);
+    const float4 g = sum_slices(in, row + i, slice, z), u = sum_slices(in, row + n + i, slice, z);
+    const float gv[4] = {g.x, g.y, g.z, g.w}, uv[4] = {u.x, u.y, u.z, u.w};
+    float f[4];
+#pragma unroll
+    for (int e = 0; e < 4; e++) {
+        const float t = gv[e];
+        f[e] = (act == 0 ? t / (1.0f + expf(-t)) : 0.5f * t * (1.0f + tanhf(0.7978845608028654f * (t + 0.044715f * t * t * t)))) * uv[e];
+    }
+    store_split4<kActBF16>(hi, nullptr, (size_t)blockIdx.y * n + i, f);
 }
 
 typedef CUresult (*EncodeTiledFn)(CUtensorMap*, CUtensorMapDataType, cuuint32_t, void*, const cuuint64_t*, const cuuint64_t*,
@@ -407,15 +462,15 @@ EncodeTiledFn encode_fn() {
     return fn;
 }
 
-// f16 matrix [rows][cols] row-major, boxes of box_rows rows x 64 columns, 128-byte swizzle, zero fill outside
-bool make_map(CUtensorMap* map, const void* base, int rows, int cols, int box_rows = 128) {
+// f16 or bf16 matrix [rows][cols] row-major, boxes of box_rows rows x 64 columns, 128-byte swizzle, zero fill outside
+bool make_map(CUtensorMap* map, const void* base, int rows, int cols, int box_rows = 128, bool bf16 = false) {
     EncodeTiledFn fn = encode_fn();
     if (!fn) return false;
     const cuuint64_t dims[2] = {(cuuint64_t)cols, (cuuint64_t)rows};
     const cuuint64_t strides[1] = {(cuuint64_t)cols * 2};
     const cuuint32_t box[2] = {(cuuint32_t)kBK, (cuuint32_t)box_rows};
     const cuuint32_t elem[2] = {1, 1};
-    return fn(map, CU_TENSOR_MAP_DATA_TYPE_FLOAT16, 2, const_cast<void*>(base), dims, strides, box, elem, CU_TENSOR_MAP_INTERLEAVE_NONE,
+    return fn(map, bf16 ? CU_TENSOR_MAP_DATA_TYPE_BFLOAT16 : CU_TENSOR_MAP_DATA_TYPE_FLOAT16, 2, const_cast<void*>(base), dims, strides, box, elem, CU_TENSOR_MAP_INTERLEAVE_NONE,
               CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_128B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) == CUDA_SUCCESS;
 }
 
@@ -430,6 +485,9 @@ struct ingot_linear_ws {
     int slot_split[3] = {0, 0, 0};             // slices the last GEMM into each slot produced
     int slot_out[3] = {0, 0, 0};               // and its output width
     int num_sms = 0;
+    bool bf16 = false;
+    int n_slots = 3;
+    int planes = 2;                            // of the prepared activations
     int prepared_tok = 0, prepared_in = 0;
     CUtensorMap map_hi, map_lo;
     std::map<std::tuple<const void*, int, int>, CUtensorMap> w_maps;  // one per weight matrix
@@ -438,7 +496,8 @@ struct ingot_linear_ws {
 // (Re)builds the activation tensor maps when the prepared shape changes.
 static cudaError_t set_prepared(ingot_linear_ws* ws, int n_in, int n_tok) {
     if (ws->prepared_tok != n_tok || ws->prepared_in != n_in) {
-        if (!make_map(&ws->map_hi, ws->hi, n_tok, n_in) || !make_map(&ws->map_lo, ws->lo, n_tok, n_in)) return cudaErrorUnknown;
+        if (!make_map(&ws->map_hi, ws->hi, n_tok, n_in, 128, ws->bf16) || !make_map(&ws->map_lo, ws->lo, n_tok, n_in, 128, ws->bf16))
+            return cudaErrorUnknown;
         ws->prepared_tok = n_tok;
         ws->prepared_in = n_in;
     }
@@ -447,28 +506,44 @@ static cudaError_t set_prepared(ingot_linear_ws* ws, int n_in, int n_tok) {
 
 extern "C" {
 
-// max_tok x max_in: the largest activation matrix that will be prepared; also the largest output (tokens x width).
-cudaError_t ingot_linear_ws_create(ingot_linear_ws** out, int max_tok, int max_in) {
+static cudaError_t ws_create(ingot_linear_ws** out, size_t act_elems, size_t partial_floats, int n_slots, bool bf16) {
     *out = nullptr;
     ingot_linear_ws* ws = new ingot_linear_ws();
-    ws->act_elems = (size_t)max_tok * max_in;
-    // k-slice partials: three slots, each at least two full-width slices of the largest batch (the hi-plane and the
-    // lo-plane product of a quantised matrix), 24 MB or more
-    ws->partial_floats = std::max((size_t)6 << 20, 2 * ws->act_elems);
+    ws->act_elems = act_elems;
+    ws->partial_floats = partial_floats;
+    ws->n_slots = n_slots;
+    ws->bf16 = bf16;
+    ws->planes = bf16 ? 1 : 2;
     int dev = 0;
     cudaError_t e;
     if ((e = cudaGetDevice(&dev)) != cudaSuccess ||
         (e = cudaDeviceGetAttribute(&ws->num_sms, cudaDevAttrMultiProcessorCount, dev)) != cudaSuccess ||
         (e = cudaMalloc(&ws->hi, ws->act_elems * 2)) != cudaSuccess || (e = cudaMalloc(&ws->lo, ws->act_elems * 2)) != cudaSuccess ||
-        (e = cudaMalloc(&ws->partial, 3 * ws->partial_floats * 4)) != cudaSuccess || (e = cudaMalloc(&ws->status, sizeof(int))) != cudaSuccess ||
+        // zero-filled: padding columns that no producer writes must be finite, they meet zero weights
+        (e = cudaMemset(ws->hi, 0, ws->act_elems * 2)) != cudaSuccess || (e = cudaMemset(ws->lo, 0, ws->act_elems * 2)) != cudaSuccess ||
+        (e = cudaMalloc(&ws->partial, n_slots * ws->partial_floats * 4)) != cudaSuccess || (e = cudaMalloc(&ws->status, sizeof(int))) != cudaSuccess ||
         (e = cudaMemset(ws->status, 0, sizeof(int))) != cudaSuccess ||
-        (e = cudaFuncSetAttribute(linear_sm100_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, kSmemBytes)) != cudaSuccess) {
+        (e = cudaFuncSetAttribute(linear_sm100_kernel<2>, cudaFuncAttributeMaxDynamicSharedMemorySize, Ring<2>::kSmemBytes)) != cudaSuccess ||
+        (e = cudaFuncSetAttribute(linear_sm100_kernel<1>, cudaFuncAttributeMaxDynamicSharedMemorySize, Ring<1>::kSmemBytes)) != cudaSuccess) {
         cudaFree(ws->hi); cudaFree(ws->lo); cudaFree(ws->partial); cudaFree(ws->status);
         delete ws;
         return e;
     }
     *out = ws;
     return cudaSuccess;
+}
+
+// max_tok x max_in: the largest activation matrix that will be prepared; also the largest output (tokens x width).
+cudaError_t ingot_linear_ws_create(ingot_linear_ws** out, int max_tok, int max_in) {
+    // k-slice partials: three slots, each at least two full-width slices of the largest batch (the hi-plane and the
+    // lo-plane product of a quantised matrix), 24 MB or more
+    const size_t act = (size_t)max_tok * max_in;
+    return ws_create(out, act, std::max((size_t)6 << 20, 2 * act), 3, false);
+}
+
+// bf16 weights: one partial slot that holds at least one slice of max_tok x max_out.
+cudaError_t ingot_linear_ws_create_bf16(ingot_linear_ws** out, int max_tok, int max_in, int max_out) {
+    return ws_create(out, (size_t)max_tok * max_in, std::max((size_t)6 << 20, (size_t)max_tok * max_out), 1, true);
 }
 
 void ingot_linear_ws_destroy(ingot_linear_ws* ws) {
@@ -479,24 +554,57 @@ void ingot_linear_ws_destroy(ingot_linear_ws* ws) {
 
 // Whether a projection of this shape can take the tensor-core path.
 int ingot_linear_tc_supported(const ingot_linear_ws* ws, int w_is_f16, int n_in, int n_out, int n_tok) {
-    return ws && encode_fn() && w_is_f16 && n_tok >= 16 && n_in % kBK == 0 && n_out % 4 == 0 && (size_t)n_tok * n_in <= ws->act_elems;
+    if (!ws || !encode_fn() || n_tok < 16 || n_out % 4 != 0 || (size_t)n_tok * n_in > ws->act_elems) return 0;
+    return ws->bf16 ? n_in % 8 == 0 : w_is_f16 && n_in % kBK == 0;
+}
+
+// Row length the planes may have: whole k-steps of f16, any multiple of 8 of bf16.
+static bool act_shape_ok(const ingot_linear_ws* ws, int n_in, int n_tok) {
+    return (size_t)n_tok * n_in <= ws->act_elems && n_in % (ws->bf16 ? 8 : kBK) == 0;
 }
 
 // Splits x [n_tok][n_in] f32 into the workspace's hi/lo f16 matrices; the following ingot_linear_tc_run calls use them.
 cudaError_t ingot_linear_tc_prepare(ingot_linear_ws* ws, const float* x, int n_in, int n_tok, cudaStream_t s) {
-    const size_t n = (size_t)n_tok * n_in;
-    if (n > ws->act_elems || n_in % kBK != 0) return cudaErrorInvalidValue;
-    cudaError_t le = launch_pdl(split_f16_kernel, dim3((unsigned)((n / 4 + 255) / 256)), dim3(256), 0, s, ws->hi, ws->lo, x, n);
+    if (!act_shape_ok(ws, n_in, n_tok) || ws->bf16) return cudaErrorInvalidValue;
+    cudaError_t le = launch_pdl(split_act_kernel<kActF16Pair>, dim3((unsigned)((n_in / 4 + 255) / 256), n_tok), dim3(256), 0, s, ws->hi, ws->lo, x, n_in, n_in);
     if (le != cudaSuccess) return le;
+    return set_prepared(ws, n_in, n_tok);
+}
+
+// bf16 workspace: rows of x are x_ld floats apart; planes 1 or 2.
+cudaError_t ingot_linear_tc_prepare_bf16(ingot_linear_ws* ws, const float* x, int x_ld, int n_in, int n_tok, int planes, cudaStream_t s) {
+    if (!act_shape_ok(ws, n_in, n_tok) || !ws->bf16 || x_ld % 4 != 0) return cudaErrorInvalidValue;
+    const dim3 grid((unsigned)((n_in / 4 + 255) / 256), n_tok);
+    cudaError_t le = planes > 1 ? launch_pdl(split_act_kernel<kActBF16Pair>, grid, dim3(256), 0, s, ws->hi, ws->lo, x, x_ld, n_in)
+                                : launch_pdl(split_act_kernel<kActBF16>, grid, dim3(256), 0, s, ws->hi, ws->lo, x, x_ld, n_in);
+    if (le != cudaSuccess) return le;
+    ws->planes = planes > 1 ? 2 : 1;
+    return set_prepared(ws, n_in, n_tok);
+}
+
+// The planes themselves ([n_tok][n_in] bf16, row-contiguous) for kernels that write their output as the next product's
+// operand, and the declaration that they have been (or, in stream order, will have been) written.
+void ingot_linear_ws_planes(ingot_linear_ws* ws, void** hi, void** lo) { *hi = ws->hi; *lo = ws->lo; }
+cudaError_t ingot_linear_tc_prepared(ingot_linear_ws* ws, int n_in, int n_tok, int planes) {
+    if (!act_shape_ok(ws, n_in, n_tok) || !ws->bf16) return cudaErrorInvalidValue;
+    ws->planes = planes > 1 ? 2 : 1;
     return set_prepared(ws, n_in, n_tok);
 }
 
 // The same with the producer of the activations folded in: rmsnorm(x; norm_w, eps).
 cudaError_t ingot_linear_tc_prepare_norm(ingot_linear_ws* ws, const float* x, const float* norm_w, float eps, int n_in, int n_tok,
                                          cudaStream_t s) {
-    if ((size_t)n_tok * n_in > ws->act_elems || n_in % kBK != 0) return cudaErrorInvalidValue;
-    cudaError_t le = launch_pdl(rmsnorm_split_kernel, dim3(n_tok), dim3(256), 0, s, ws->hi, ws->lo, x, norm_w, n_in, eps);
+    if (!act_shape_ok(ws, n_in, n_tok) || ws->bf16) return cudaErrorInvalidValue;
+    cudaError_t le = launch_pdl(rmsnorm_split_kernel<kActF16Pair>, dim3(n_tok), dim3(256), 0, s, ws->hi, ws->lo, x, norm_w, n_in, n_in, eps);
     if (le != cudaSuccess) return le;
+    return set_prepared(ws, n_in, n_tok);
+}
+cudaError_t ingot_linear_tc_prepare_norm_bf16(ingot_linear_ws* ws, const float* x, const float* norm_w, float eps, int n_in, int n_mean, int n_tok,
+                                              cudaStream_t s) {
+    if (!act_shape_ok(ws, n_in, n_tok) || !ws->bf16) return cudaErrorInvalidValue;
+    cudaError_t le = launch_pdl(rmsnorm_split_kernel<kActBF16>, dim3(n_tok), dim3(256), 0, s, ws->hi, ws->lo, x, norm_w, n_in, n_mean, eps);
+    if (le != cudaSuccess) return le;
+    ws->planes = 1;
     return set_prepared(ws, n_in, n_tok);
 }
 
@@ -505,10 +613,14 @@ cudaError_t ingot_linear_tc_prepare_norm(ingot_linear_ws* ws, const float* x, co
 // append: the slices are written behind the ones the slots already hold (all slots of the group must hold the same
 // number), so that a second product - the lo plane of a quantised matrix after its hi plane - simply adds k slices
 // for the consumer kernel to sum.
+// rows_per_block > 0 (count == 1): block-diagonal; n_in is then the row length of one block and the prepared activations hold
+// n_out / rows_per_block such blocks side by side.
 static cudaError_t launch_gemm(ingot_linear_ws* ws, float* out, const void* const* w, int n_in, const int* n_out, int count,
-                               int accumulate, int first_slot, bool to_partial, bool append, cudaStream_t s) {
+                               int accumulate, int first_slot, bool to_partial, bool append, cudaStream_t s, int rows_per_block = 0) {
     const int n_tok = ws->prepared_tok;
-    if (n_in != ws->prepared_in || n_tok < 1 || count < 1 || first_slot < 0 || first_slot + count > 3 || (count > 1 && !to_partial) ||
+    if (rows_per_block > 0 && (count != 1 || n_out[0] % rows_per_block != 0 || rows_per_block % 4 != 0 || n_in % 8 != 0)) return cudaErrorInvalidValue;
+    const int act_in = rows_per_block > 0 ? n_in * (n_out[0] / rows_per_block) : n_in;
+    if (act_in != ws->prepared_in || n_tok < 1 || count < 1 || first_slot < 0 || first_slot + count > ws->n_slots || (count > 1 && !to_partial) ||
         (append && !to_partial))
         return cudaErrorInvalidValue;
     const int held = append ? ws->slot_split[first_slot] : 0;
@@ -522,11 +634,11 @@ static cudaError_t launch_gemm(ingot_linear_ws* ws, float* out, const void* cons
         auto it = ws->w_maps.find(key);
         if (it == ws->w_maps.end()) {
             CUtensorMap tm;
-            if (!make_map(&tm, w[m], n_out[m], n_in, kBN)) return cudaErrorUnknown;
+            if (!make_map(&tm, w[m], n_out[m], n_in, kBN, ws->bf16)) return cudaErrorUnknown;
             it = ws->w_maps.emplace(key, tm).first;
         }
         maps[m] = &it->second;
-        tiles_n += (n_out[m] + kBN - 1) / kBN;
+        tiles_n += rows_per_block > 0 ? n_out[m] / rows_per_block * ((rows_per_block + kBN - 1) / kBN) : (n_out[m] + kBN - 1) / kBN;
         p.tile_end[m] = tiles_n;
         p.n_out[m] = n_out[m];
         p.partial[m] = ws->partial + (size_t)(first_slot + m) * ws->partial_floats + (size_t)held * n_tok * n_out[m];
@@ -534,16 +646,21 @@ static cudaError_t launch_gemm(ingot_linear_ws* ws, float* out, const void* cons
     }
     for (int m = count; m < 3; m++) { maps[m] = maps[count - 1]; p.tile_end[m] = tiles_n; p.n_out[m] = n_out[count - 1]; p.partial[m] = p.partial[count - 1]; }
     const int tiles = tiles_n * ((n_tok + kBM - 1) / kBM);
-    const int k_steps = n_in / kBK;
+    const int k_steps = (n_in + kBK - 1) / kBK;
     // enough k slices to give every SM a CTA, at least 4 k-steps each, and no more than the slots hold
     if (to_partial && fit < 1) return cudaErrorInvalidValue;
     const int n_split = std::max(1, std::min({ws->num_sms / tiles, k_steps / 4, fit}));
     p.out = out; p.status = ws->status;
     p.n_tok = n_tok; p.k_steps = k_steps; p.n_split = n_split; p.accumulate = accumulate;
     p.to_partial = to_partial ? 1 : 0;
+    p.idesc = ws->bf16 ? kIdescBF16 : kIdescF16;
+    p.rows_per_block = rows_per_block;
+    p.k_block = rows_per_block > 0 ? n_in : 0;
+    p.tiles_per_block = rows_per_block > 0 ? (rows_per_block + kBN - 1) / kBN : 0;
     dim3 grid(tiles_n, (n_tok + kBM - 1) / kBM, n_split);
-    cudaError_t le = launch_pdl(linear_sm100_kernel, grid, dim3(kThreads), (size_t)kSmemBytes, s, ws->map_hi, ws->map_lo, *maps[0], *maps[1],
-                                *maps[2], p);
+    cudaError_t le = ws->planes > 1
+        ? launch_pdl(linear_sm100_kernel<2>, grid, dim3(kThreads), (size_t)Ring<2>::kSmemBytes, s, ws->map_hi, ws->map_lo, *maps[0], *maps[1], *maps[2], p)
+        : launch_pdl(linear_sm100_kernel<1>, grid, dim3(kThreads), (size_t)Ring<1>::kSmemBytes, s, ws->map_hi, ws->map_lo, *maps[0], *maps[1], *maps[2], p);
     if (le != cudaSuccess) return le;
     for (int m = 0; m < count; m++) {
         ws->slot_split[first_slot + m] = held + n_split;
@@ -561,6 +678,12 @@ static cudaError_t launch_gemm(ingot_linear_ws* ws, float* out, const void* cons
 // out [n_tok][n_out] (+)= prepared activations x W^T, W f16 [n_out][n_in] on the device.
 cudaError_t ingot_linear_tc_run(ingot_linear_ws* ws, float* out, const void* w, int n_in, int n_out, int accumulate, cudaStream_t s) {
     return launch_gemm(ws, out, &w, n_in, &n_out, 1, accumulate, 0, false, false, s);
+}
+
+// Block-diagonal product: W [n_out][k_block], output rows of block b = row / rows_per_block times the prepared columns
+// b * k_block .. (b + 1) * k_block - 1.
+cudaError_t ingot_linear_tc_run_blocks(ingot_linear_ws* ws, float* out, const void* w, int k_block, int n_out, int rows_per_block, cudaStream_t s) {
+    return launch_gemm(ws, out, &w, k_block, &n_out, 1, 0, 0, false, false, s, rows_per_block);
 }
 
 // The same product left as k slices in scratch slot 0..2 for one of the ingot_linear_tc_finish_* calls below.
@@ -601,10 +724,29 @@ cudaError_t ingot_linear_tc_finish_group(ingot_linear_ws* ws, float* const* outs
 // become the prepared input of the next projections (n_in = the product's width).
 cudaError_t ingot_linear_tc_finish_residual_norm(ingot_linear_ws* ws, float* x, const float* norm_w, float eps, int slot, cudaStream_t s) {
     const int n = ws->slot_out[slot], n_tok = ws->prepared_tok;
-    if (n % 4 != 0 || (norm_w && ((size_t)n_tok * n > ws->act_elems || n % kBK != 0))) return cudaErrorInvalidValue;
-    cudaError_t le = launch_pdl(finish_residual_norm_kernel, dim3(n_tok), dim3(256), 0, s, x, slices_of(ws, slot), ws->hi, ws->lo, norm_w, n, n_tok, eps);
+    if (n % 4 != 0 || (norm_w && !act_shape_ok(ws, n, n_tok)) || ws->bf16) return cudaErrorInvalidValue;
+    cudaError_t le = launch_pdl(finish_residual_norm_kernel<kActF16Pair>, dim3(n_tok), dim3(256), 0, s, x, slices_of(ws, slot), ws->hi, ws->lo, norm_w, n, n, n_tok, eps);
     if (le != cudaSuccess) return le;
     return norm_w ? set_prepared(ws, n, n_tok) : cudaGetLastError();
+}
+cudaError_t ingot_linear_tc_finish_residual_norm_bf16(ingot_linear_ws* ws, float* x, const float* norm_w, float eps, int n_mean, cudaStream_t s) {
+    const int n = ws->slot_out[0], n_tok = ws->prepared_tok;
+    if (n % 4 != 0 || (norm_w && !act_shape_ok(ws, n, n_tok)) || !ws->bf16) return cudaErrorInvalidValue;
+    cudaError_t le = launch_pdl(finish_residual_norm_kernel<kActBF16>, dim3(n_tok), dim3(256), 0, s, x, slices_of(ws, 0), ws->hi, ws->lo, norm_w, n, n_mean, n_tok, eps);
+    if (le != cudaSuccess) return le;
+    ws->planes = 1;
+    return norm_w ? set_prepared(ws, n, n_tok) : cudaGetLastError();
+}
+
+// The product in slot 0 (width 2 n: gate half, up half) becomes the bf16 operand act(gate) * up of the next product.
+cudaError_t ingot_linear_tc_finish_gated_bf16(ingot_linear_ws* ws, int act, cudaStream_t s) {
+    const int n = ws->slot_out[0] / 2, n_tok = ws->prepared_tok;
+    if (!ws->bf16 || n % 8 != 0 || !act_shape_ok(ws, n, n_tok)) return cudaErrorInvalidValue;
+    cudaError_t le = launch_pdl(finish_gated_kernel, dim3((unsigned)((n / 4 + 255) / 256), n_tok), dim3(256), 0, s, ws->hi, slices_of(ws, 0), n,
+                                (size_t)n_tok * 2 * n, act);
+    if (le != cudaSuccess) return le;
+    ws->planes = 1;
+    return set_prepared(ws, n, n_tok);
 }
 
 // hi/lo of silu(slot_gate) .* slot_up become the prepared input of the next projection.
@@ -616,6 +758,8 @@ cudaError_t ingot_linear_tc_finish_swiglu(ingot_linear_ws* ws, int slot_gate, in
     if (le != cudaSuccess) return le;
     return set_prepared(ws, n_in, n_tok);
 }
+
+int* ingot_linear_ws_status_dev(ingot_linear_ws* ws) { return ws->status; }
 
 // The status word: non-zero after a bounded wait expired in some launch since the last call. Synchronises the device.
 int ingot_linear_ws_status(ingot_linear_ws* ws) {

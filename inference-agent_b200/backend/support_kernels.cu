@@ -3,8 +3,11 @@
 // shaders/kernels.metal:129-252, 706-710). Activations stay f32 everywhere, weights are read in their
 // stored type (f16 or f32) and widened, products accumulate in f32 — the arithmetic of ops::dot_row
 // (src/ops.cpp:127-141) up to summation order — so that greedy decoding follows the CPU reference.
+// bf16 weights (models loaded from safetensors folders) are read the same way: widened, never rounded further.
 // Single-token steps with f16 weights use the weight-streaming kernel (gemv_stream_kernel); batches use the
 // tensor-core kernel of linear_sm100.cu; the plain kernels here cover f32 weights and odd shapes.
+#include <algorithm>
+#include <cuda_bf16.h>
 #include <cuda_fp16.h>
 #include <type_traits>
 #include <cuda_runtime.h>
@@ -43,6 +46,38 @@ __global__ void rmsnorm_kernel(float* out, const float* x, const float* w, int n
     for (int i = threadIdx.x; i < n; i += blockDim.x) orow[i] = xr[i] * scale * w[i];
 }
 
+// The same with a row gather, and with the mean over n_mean of the row's n floats (rows zero-padded to an aligned length).
+__global__ void rmsnorm_rows_kernel(float* out, const float* x, const float* w, const int32_t* rows, int n, int n_mean, float eps) {
+    asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
+    asm volatile("griddepcontrol.wait;" ::: "memory");
+    __shared__ float red[32];
+    const float* xr = x + (size_t)(rows ? rows[blockIdx.x] : (int)blockIdx.x) * n;
+    float* orow = out + (size_t)blockIdx.x * n;
+    float ss = 0.f;
+    for (int i = threadIdx.x; i < n; i += blockDim.x) ss += xr[i] * xr[i];
+    ss = warp_sum(ss);
+    if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = ss;
+    __syncthreads();
+    float t = 0.f;
+    for (int i = 0; i < (int)(blockDim.x >> 5); i++) t += red[i];
+    const float scale = 1.0f / sqrtf(t / float(n_mean) + eps);
+    for (int i = threadIdx.x; i < n; i += blockDim.x) orow[i] = xr[i] * scale * w[i];
+}
+
+// Activation of gated feed-forwards: 0 silu, 1 the tanh form of gelu.
+__device__ __forceinline__ float gate_act(float g, int act) {
+    if (act == 0) return g / (1.0f + expf(-g));
+    return 0.5f * g * (1.0f + tanhf(0.7978845608028654f * (g + 0.044715f * g * g * g)));
+}
+__global__ void gated_act_kernel(float* out, const float* in, int n, size_t total, int act) {
+    asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
+    asm volatile("griddepcontrol.wait;" ::: "memory");
+    const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
+    if (i >= total) return;
+    const size_t r = i / n, c = i - r * n;
+    out[i] = gate_act(in[r * 2 * n + c], act) * in[r * 2 * n + n + c];
+}
+
 // gate[i] = silu(gate[i]) * up[i]      (src/cpu_backend.cpp:79, ops::silu src/ops.h:35)
 __global__ void silu_mul_kernel(float* gate, const float* up, size_t n) {
     const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
@@ -66,20 +101,40 @@ __device__ __forceinline__ void load8<__half>(const __half* p, float (&w)[8]) {
     }
 }
 template <>
+__device__ __forceinline__ void load8<__nv_bfloat16>(const __nv_bfloat16* p, float (&w)[8]) {
+    const uint4 raw = *reinterpret_cast<const uint4*>(p);
+    const uint32_t u[4] = {raw.x, raw.y, raw.z, raw.w};
+#pragma unroll
+    for (int i = 0; i < 4; i++) {  // a bf16 value is the high half of the f32 with the same bits
+        w[2 * i] = __uint_as_float(u[i] << 16);
+        w[2 * i + 1] = __uint_as_float(u[i] & 0xffff0000u);
+    }
+}
+template <>
 __device__ __forceinline__ void load8<float>(const float* p, float (&w)[8]) {
     const float4 a = *reinterpret_cast<const float4*>(p), b = *reinterpret_cast<const float4*>(p + 4);
     w[0] = a.x; w[1] = a.y; w[2] = a.z; w[3] = a.w; w[4] = b.x; w[5] = b.y; w[6] = b.z; w[7] = b.w;
 }
 
+// Activation rows may be longer than n_in (x_ld apart), and the matrix may be block-diagonal: with rows_per_block > 0,
+// output row r reads the n_in columns that start at (r / rows_per_block) * n_in.
+struct XLayout {
+    int ld, rows_per_block;
+    __device__ __forceinline__ int col0(int row, int n_in) const { return rows_per_block > 0 ? (row / rows_per_block) * n_in : 0; }
+};
+
 // out[t][r] (+)= dot(W[r][:], x[t][:]) for a tile of TT tokens; one warp per output row.
 // W is [n_out][n_in] row-major (ggml ne = [n_in, n_out]); n_in is a multiple of 8.
 template <typename W, int TT>
-__global__ void linear_kernel(float* out, const W* w, const float* x, int n_in, int n_out, int n_tok, int accumulate) {
+__global__ void linear_kernel(float* out, const W* w, const float* x, int n_in, int n_out, int n_tok, int accumulate, XLayout xl) {
+    asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
+    asm volatile("griddepcontrol.wait;" ::: "memory");
     const int row = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
     const int lane = threadIdx.x & 31;
     const int t0 = blockIdx.y * TT;
     if (row >= n_out) return;
     const W* wr = w + (size_t)row * n_in;
+    const float* x0 = x + xl.col0(row, n_in);
     float acc[TT];
 #pragma unroll
     for (int t = 0; t < TT; t++) acc[t] = 0.f;
@@ -89,7 +144,7 @@ __global__ void linear_kernel(float* out, const W* w, const float* x, int n_in, 
 #pragma unroll
         for (int t = 0; t < TT; t++) {
             if (t0 + t < n_tok) {
-                const float* xr = x + (size_t)(t0 + t) * n_in + i;
+                const float* xr = x0 + (size_t)(t0 + t) * xl.ld + i;
                 const float4 a = *reinterpret_cast<const float4*>(xr), b = *reinterpret_cast<const float4*>(xr + 4);
                 acc[t] = fmaf(wv[0], a.x, acc[t]); acc[t] = fmaf(wv[1], a.y, acc[t]);
                 acc[t] = fmaf(wv[2], a.z, acc[t]); acc[t] = fmaf(wv[3], a.w, acc[t]);
@@ -114,13 +169,15 @@ __global__ void linear_kernel(float* out, const W* w, const float* x, int n_in, 
 // out[r] (+)= dot(W[r][:], x).
 template <typename W>
 __global__ void __launch_bounds__(256) gemv_kernel(float* out, const W* w, const float* x, int n_in, int n_out, int accumulate) {
+    asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
+    asm volatile("griddepcontrol.wait;" ::: "memory");
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int row = blockIdx.x * (blockDim.x >> 5) + warp;
     if (row >= n_out) return;
     const W* wr = w + (size_t)row * n_in;
     float acc0 = 0.f, acc1 = 0.f, acc2 = 0.f, acc3 = 0.f;
     auto fma8 = [&](float& acc, const float (&wv)[8], const float* xs) {
-        const float4 xa = __ldg(reinterpret_cast<const float4*>(xs)), xb = __ldg(reinterpret_cast<const float4*>(xs + 4));
+        const float4 xa = *reinterpret_cast<const float4*>(xs), xb = *reinterpret_cast<const float4*>(xs + 4);
         acc = fmaf(wv[0], xa.x, acc); acc = fmaf(wv[1], xa.y, acc); acc = fmaf(wv[2], xa.z, acc); acc = fmaf(wv[3], xa.w, acc);
         acc = fmaf(wv[4], xb.x, acc); acc = fmaf(wv[5], xb.y, acc); acc = fmaf(wv[6], xb.z, acc); acc = fmaf(wv[7], xb.w, acc);
     };
@@ -177,12 +234,25 @@ __device__ __forceinline__ float dot8(const uint4& raw, const float4* x4) {
     return acc;
 }
 
+__device__ __forceinline__ float dot8_bf16(const uint4& raw, const float4* x4) {
+    const float4 xa = x4[0], xb = x4[32];
+    float acc = __uint_as_float(raw.x << 16) * xa.x;
+    acc = fmaf(__uint_as_float(raw.x & 0xffff0000u), xa.y, acc);
+    acc = fmaf(__uint_as_float(raw.y << 16), xa.z, acc); acc = fmaf(__uint_as_float(raw.y & 0xffff0000u), xa.w, acc);
+    acc = fmaf(__uint_as_float(raw.z << 16), xb.x, acc); acc = fmaf(__uint_as_float(raw.z & 0xffff0000u), xb.y, acc);
+    acc = fmaf(__uint_as_float(raw.w << 16), xb.z, acc); acc = fmaf(__uint_as_float(raw.w & 0xffff0000u), xb.w, acc);
+    return acc;
+}
+
 // Weight formats of the streaming kernel. A lane's 16-byte load covers kElems weights: 8 f16 values, 16 Q8_0
 // quants (half a block) or the 32 nibbles of one Q4_0 block; the 32 lanes of a warp therefore cover 512 bytes =
 // 256 / 512 / 1024 consecutive weights per load. Quantised rows come from the repacked planes of
 // quant_kernels.cu: quants contiguous per row, one f16 scale per 32 weights in a plane of its own.
-enum : int { kFmtF16 = 0, kFmtQ8_0 = 1, kFmtQ4_0 = 2 };
-template <int kFmt> struct FmtTraits { static constexpr int kElems = kFmt == kFmtF16 ? 8 : kFmt == kFmtQ8_0 ? 16 : 32; };
+enum : int { kFmtF16 = 0, kFmtQ8_0 = 1, kFmtQ4_0 = 2, kFmtBF16 = 3 };
+template <int kFmt> struct FmtTraits {
+    static constexpr int kElems = kFmt == kFmtQ8_0 ? 16 : kFmt == kFmtQ4_0 ? 32 : 8;
+    static constexpr bool kPlain = kFmt == kFmtF16 || kFmt == kFmtBF16;  // no block scales
+};
 
 __device__ __forceinline__ uint32_t prmt_b(uint32_t a, uint32_t b, uint32_t sel) {
     uint32_t r;
@@ -197,6 +267,7 @@ __device__ __forceinline__ float byte_f(uint32_t word, int k, float bias) {
 template <int kFmt>
 __device__ __forceinline__ float dot_load(const uint4& raw, const float4* x4, unsigned short scale_bits) {
     if (kFmt == kFmtF16) return dot8(raw, x4);
+    if (kFmt == kFmtBF16) return dot8_bf16(raw, x4);
     const float d = __half2float(__ushort_as_half(scale_bits));
     const uint32_t w[4] = {raw.x, raw.y, raw.z, raw.w};
     float s0 = 0.f, s1 = 0.f, s2 = 0.f, s3 = 0.f;
@@ -236,11 +307,11 @@ __device__ __forceinline__ float dot_load(const uint4& raw, const float4* x4, un
 // the quantised formats need up to 122 and stay at 256 threads, two or three CTAs per SM (512-thread CTAs measured:
 // Q8_0 tg32 561 -> 536 tok/s, Q4_0 539 -> 544).
 template <int kFmt>
-struct StreamThreads { static constexpr int value = kFmt == 0 ? 768 : 256; };
+struct StreamThreads { static constexpr int value = FmtTraits<kFmt>::kPlain ? 768 : 256; };
 
 template <bool kNorm, bool kSwiGLU, int kLoads, int kFmt>
 __global__ void __launch_bounds__(StreamThreads<kFmt>::value) gemv_stream_kernel(const GemvGroup g, const float* x, const float* norm_w, float eps, int n_in,
-                                                          int total_rows, int accumulate, int use_pdl) {
+                                                          int total_rows, int accumulate, int use_pdl, int n_mean, int act) {
     extern __shared__ float xs[];  // x', n_in floats
     __shared__ float red[25];
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -260,13 +331,13 @@ __global__ void __launch_bounds__(StreamThreads<kFmt>::value) gemv_stream_kernel
         if (kSwiGLU) {
             wa = static_cast<const char*>(g.w[0]) + (size_t)r * row_bytes;
             wb = static_cast<const char*>(g.w[1]) + (size_t)r * row_bytes;
-            da = kFmt == kFmtF16 ? nullptr : g.d[0] + (size_t)r * row_scales;
-            db = kFmt == kFmtF16 ? nullptr : g.d[1] + (size_t)r * row_scales;
+            da = FmtTraits<kFmt>::kPlain ? nullptr : g.d[0] + (size_t)r * row_scales;
+            db = FmtTraits<kFmt>::kPlain ? nullptr : g.d[1] + (size_t)r * row_scales;
         } else {
             const int m = (r >= g.row_end[0]) + (r >= g.row_end[1] && g.n_mat > 2);
             const int local = m == 0 ? r : r - (m == 1 ? g.row_end[0] : g.row_end[1]);
             wa = static_cast<const char*>(m == 0 ? g.w[0] : m == 1 ? g.w[1] : g.w[2]) + (size_t)local * row_bytes;
-            da = kFmt == kFmtF16 ? nullptr : (m == 0 ? g.d[0] : m == 1 ? g.d[1] : g.d[2]) + (size_t)local * row_scales;
+            da = FmtTraits<kFmt>::kPlain ? nullptr : (m == 0 ? g.d[0] : m == 1 ? g.d[1] : g.d[2]) + (size_t)local * row_scales;
             wb = nullptr;
             db = nullptr;
         }
@@ -282,7 +353,7 @@ __global__ void __launch_bounds__(StreamThreads<kFmt>::value) gemv_stream_kernel
             if (c < n_chunks) {
                 A[h] = ld_stream_u4(wa + (size_t)c * 512 + lane * 16);
                 if (kSwiGLU) B[h] = ld_stream_u4(wb + (size_t)c * 512 + lane * 16);
-                if (kFmt != kFmtF16) {
+                if (!FmtTraits<kFmt>::kPlain) {
                     const int blk = ((c * 32 + lane) * kElems) >> 5;
                     SA[h] = __ldg(reinterpret_cast<const unsigned short*>(da) + blk);
                     if (kSwiGLU) SB[h] = __ldg(reinterpret_cast<const unsigned short*>(db) + blk);
@@ -319,7 +390,7 @@ __global__ void __launch_bounds__(StreamThreads<kFmt>::value) gemv_stream_kernel
     if (kNorm) {
         float t = 0.f;
         for (int w = 0; w < (int)(blockDim.x >> 5); w++) t += red[w];
-        scale = 1.0f / sqrtf(t / float(n_in) + eps);
+        scale = 1.0f / sqrtf(t / float(n_mean) + eps);
     }
 
     float acc_a = 0.f, acc_b = 0.f;
@@ -343,7 +414,7 @@ __global__ void __launch_bounds__(StreamThreads<kFmt>::value) gemv_stream_kernel
             if (lane == 0) {
                 if (kSwiGLU) {
                     const float gt = acc_a * scale, up = acc_b * scale;
-                    g.out[0][r] = gt / (1.0f + expf(-gt)) * up;
+                    g.out[0][r] = gate_act(gt, act) * up;
                 } else {
                     const int m = (r >= g.row_end[0]) + (r >= g.row_end[1] && g.n_mat > 2);
                     const int local = m == 0 ? r : r - (m == 1 ? g.row_end[0] : g.row_end[1]);
@@ -367,10 +438,18 @@ __global__ void __launch_bounds__(StreamThreads<kFmt>::value) gemv_stream_kernel
 // weight matrix is read once per 128 tokens.
 constexpr int kGM = 128, kGN = 64, kGK = 16;
 template <typename W>
-__global__ void __launch_bounds__(256) gemm_kernel(float* out, const W* w, const float* x, int n_in, int n_out, int n_tok, int accumulate) {
+__global__ void __launch_bounds__(256) gemm_kernel(float* out, const W* w, const float* x, int n_in, int n_out, int n_tok, int accumulate, XLayout xl) {
+    asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
+    asm volatile("griddepcontrol.wait;" ::: "memory");
     __shared__ __align__(16) float xs[kGK][kGM + 4];
     __shared__ __align__(16) float ws[kGK][kGN + 4];
-    const int t0 = blockIdx.y * kGM, r0 = blockIdx.x * kGN;
+    const int t0 = blockIdx.y * kGM;
+    // block-diagonal matrices: the output tiles of a block never straddle into the next one
+    const int tiles_per_block = xl.rows_per_block > 0 ? (xl.rows_per_block + kGN - 1) / kGN : 0;
+    const int blk = tiles_per_block ? blockIdx.x / tiles_per_block : 0;
+    const int r0 = tiles_per_block ? blk * xl.rows_per_block + (blockIdx.x - blk * tiles_per_block) * kGN : blockIdx.x * kGN;
+    const int r_end = tiles_per_block ? (blk + 1) * xl.rows_per_block : n_out;
+    const float* x0 = x + (tiles_per_block ? blk * n_in : 0);
     const int tid = threadIdx.x;
     const int tm = (tid >> 4) * 8, tn = (tid & 15) * 4;  // this thread's 8 tokens x 4 outputs
     float acc[8][4];
@@ -385,13 +464,13 @@ __global__ void __launch_bounds__(256) gemm_kernel(float* out, const W* w, const
             const int idx = it * 256 + tid;
             const int row = idx >> 2, c4 = (idx & 3) * 4;
             float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
-            if (t0 + row < n_tok) v = *reinterpret_cast<const float4*>(x + (size_t)(t0 + row) * n_in + k0 + c4);
+            if (t0 + row < n_tok && k0 + c4 < n_in) v = *reinterpret_cast<const float4*>(x0 + (size_t)(t0 + row) * xl.ld + k0 + c4);
             xs[c4 + 0][row] = v.x; xs[c4 + 1][row] = v.y; xs[c4 + 2][row] = v.z; xs[c4 + 3][row] = v.w;
         }
         if (tid < 128) {
             const int row = tid >> 1, c8 = (tid & 1) * 8;
             float wv[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
-            if (r0 + row < n_out) load8<W>(w + (size_t)(r0 + row) * n_in + k0 + c8, wv);
+            if (r0 + row < r_end && k0 + c8 < n_in) load8<W>(w + (size_t)(r0 + row) * n_in + k0 + c8, wv);
 #pragma unroll
             for (int i = 0; i < 8; i++) ws[c8 + i][row] = wv[i];
         }
@@ -414,7 +493,7 @@ __global__ void __launch_bounds__(256) gemm_kernel(float* out, const W* w, const
         const int t = t0 + tm + i;
         if (t >= n_tok) continue;
         float* o = out + (size_t)t * n_out + r0 + tn;
-        if (r0 + tn + 3 < n_out) {
+        if (r0 + tn + 3 < r_end) {
             float4 v = make_float4(acc[i][0], acc[i][1], acc[i][2], acc[i][3]);
             if (accumulate) {
                 const float4 old = *reinterpret_cast<const float4*>(o);
@@ -423,13 +502,14 @@ __global__ void __launch_bounds__(256) gemm_kernel(float* out, const W* w, const
             *reinterpret_cast<float4*>(o) = v;
         } else {
             for (int j = 0; j < 4; j++)
-                if (r0 + tn + j < n_out) o[j] = accumulate ? o[j] + acc[i][j] : acc[i][j];
+                if (r0 + tn + j < r_end) o[j] = accumulate ? o[j] + acc[i][j] : acc[i][j];
         }
     }
 }
 
 __device__ __forceinline__ float embed_to_f32(float v) { return v; }
 __device__ __forceinline__ float embed_to_f32(__half v) { return __half2float(v); }
+__device__ __forceinline__ float embed_to_f32(__nv_bfloat16 v) { return __bfloat162float(v); }
 
 // Embedding gather: out[r][:] = table[rows[r]][:] widened to f32 (src/cpu_backend.cpp:33 does this with
 // ops::dequant_row on the host). A row index outside the table gives zeros and raises *status.
@@ -474,18 +554,20 @@ cudaError_t ingot_support_silu_mul(float* gate, const float* up, size_t n, cudaS
 // matrix repacked by ingot_quant_repack). norm_w != nullptr folds the RMS norm in; swiglu != 0 takes exactly two
 // matrices of equal height (gate, up) and outs[0] receives silu(gate) * up. n_in must be a multiple of 256 (f16),
 // 512 (Q8_0) or 1024 (Q4_0).
-cudaError_t ingot_support_gemv_group(float* const* outs, const void* const* ws, const void* const* scales, int fmt, const int* n_out, int n_mat,
-                                     int swiglu, const float* x, const float* norm_w, float eps, int n_in, int accumulate, cudaStream_t s) {
-    const int chunk = fmt == kFmtF16 ? 256 : fmt == kFmtQ8_0 ? 512 : 1024;
-    if (fmt < 0 || fmt > 2 || n_mat < 1 || n_mat > 3 || n_in % chunk != 0 || n_in > kGemvMaxIn ||
-        (swiglu && (n_mat != 2 || n_out[0] != n_out[1] || !norm_w)) || (fmt != kFmtF16 && !scales))
+static cudaError_t gemv_group(float* const* outs, const void* const* ws, const void* const* scales, int fmt, const int* n_out, int n_mat,
+                              int swiglu, int act, const float* x, const float* norm_w, float eps, int n_in, int n_mean, int accumulate,
+                              cudaStream_t s) {
+    const bool plain = fmt == kFmtF16 || fmt == kFmtBF16;
+    const int chunk = plain ? 256 : fmt == kFmtQ8_0 ? 512 : 1024;
+    if (fmt < 0 || fmt > 3 || n_mat < 1 || n_mat > 3 || n_in % chunk != 0 || n_in > kGemvMaxIn ||
+        (swiglu && (n_mat != 2 || n_out[0] != n_out[1] || !norm_w)) || (!plain && !scales))
         return cudaErrorInvalidValue;
     GemvGroup g = {};
     int total = 0;
     for (int m = 0; m < 3; m++) {
         const int mm = m < n_mat ? m : n_mat - 1;
         g.w[m] = ws[mm];
-        g.d[m] = fmt == kFmtF16 ? nullptr : static_cast<const __half*>(scales[mm]);
+        g.d[m] = plain ? nullptr : static_cast<const __half*>(scales[mm]);
         g.out[m] = outs[mm];
         if (m < n_mat) total += n_out[m];
         g.row_end[m] = swiglu ? n_out[0] : total;
@@ -495,13 +577,13 @@ cudaError_t ingot_support_gemv_group(float* const* outs, const void* const* ws, 
     const size_t smem = (size_t)n_in * sizeof(float);
     // kLoads = 6 for short rows: with the current and the next step in flight the whole row is requested at once
     const bool short_rows = n_in / chunk <= 12;  // current and next step together cover the row
-    typedef void (*Kernel)(GemvGroup, const float*, const float*, float, int, int, int, int);
+    typedef void (*Kernel)(GemvGroup, const float*, const float*, float, int, int, int, int, int, int);
     auto pick = [&](auto fmt_tag) -> Kernel {
         constexpr int F = decltype(fmt_tag)::value;
         return short_rows ? (swiglu ? gemv_stream_kernel<true, true, 6, F> : norm_w ? gemv_stream_kernel<true, false, 6, F> : gemv_stream_kernel<false, false, 6, F>)
                           : (swiglu ? gemv_stream_kernel<true, true, 4, F> : norm_w ? gemv_stream_kernel<true, false, 4, F> : gemv_stream_kernel<false, false, 4, F>);
     };
-    Kernel kernel = fmt == kFmtF16 ? pick(std::integral_constant<int, kFmtF16>()) : fmt == kFmtQ8_0 ? pick(std::integral_constant<int, kFmtQ8_0>())
+    Kernel kernel = fmt == kFmtBF16 ? pick(std::integral_constant<int, kFmtBF16>()) : fmt == kFmtF16 ? pick(std::integral_constant<int, kFmtF16>()) : fmt == kFmtQ8_0 ? pick(std::integral_constant<int, kFmtQ8_0>())
                                                                                                : pick(std::integral_constant<int, kFmtQ4_0>());
     // Environment knobs are process-wide and read once; the SM count belongs to the current device and is looked up
     // on every call (a cached attribute read), so that one process may drive several GPUs.
@@ -514,7 +596,7 @@ cudaError_t ingot_support_gemv_group(float* const* outs, const void* const* ws, 
     if (e == cudaSuccess) e = cudaDeviceGetAttribute(&num_sms, cudaDevAttrMultiProcessorCount, dev);
     if (e != cudaSuccess) return e;
     int occ = 0;
-    const int threads = fmt == kFmtF16 ? StreamThreads<kFmtF16>::value : StreamThreads<kFmtQ8_0>::value, cta_warps = threads / 32;
+    const int threads = plain ? StreamThreads<kFmtF16>::value : StreamThreads<kFmtQ8_0>::value, cta_warps = threads / 32;
     e = cudaOccupancyMaxActiveBlocksPerMultiprocessor(&occ, kernel, threads, smem);
     if (e != cudaSuccess) return e;
     if (occ < 1) occ = 1;
@@ -524,7 +606,7 @@ cudaError_t ingot_support_gemv_group(float* const* outs, const void* const* ws, 
     // leaves some SMs without a CTA but has no uneven tail - measured tg32 589 against 578 tok/s with the full grid,
     // while the quantised formats gain from it (Q8_0 561 -> 565, Q4_0 540 -> 554).
     int ctas;
-    if (fmt == kFmtF16) {
+    if (plain) {
         const int capacity = num_sms * occ * cta_warps;
         const int rows_per_warp = (rows + capacity - 1) / capacity;
         ctas = ((rows + rows_per_warp - 1) / rows_per_warp + cta_warps - 1) / cta_warps;
@@ -541,27 +623,104 @@ cudaError_t ingot_support_gemv_group(float* const* outs, const void* const* ws, 
     attr[0].val.programmaticStreamSerializationAllowed = 1;
     cfg.attrs = attr;
     cfg.numAttrs = use_pdl ? 1 : 0;
-    return cudaLaunchKernelEx(&cfg, kernel, g, x, norm_w, eps, n_in, rows, accumulate, use_pdl ? 1 : 0);
+    return cudaLaunchKernelEx(&cfg, kernel, g, x, norm_w, eps, n_in, rows, accumulate, use_pdl ? 1 : 0, n_mean, act);
 }
+
+cudaError_t ingot_support_gemv_group(float* const* outs, const void* const* ws, const void* const* scales, int fmt, const int* n_out, int n_mat,
+                                     int swiglu, const float* x, const float* norm_w, float eps, int n_in, int accumulate, cudaStream_t s) {
+    if (fmt > 2) return cudaErrorInvalidValue;
+    return gemv_group(outs, ws, scales, fmt, n_out, n_mat, swiglu, 0, x, norm_w, eps, n_in, n_in, accumulate, s);
+}
+
+// The same streaming kernel for one bf16 matrix [n_out][n_in] (n_in a multiple of 256): out (+)= W x', x' = rmsnorm(x) with the mean
+// over n_mean floats if norm_w is given. gated: W holds a gate and an up half of n_out rows each, out = act(gate) * up.
+cudaError_t ingot_support_gemv_bf16(float* out, const void* w, int n_out, int n_in, const float* x, const float* norm_w, float eps, int n_mean,
+                                    int gated, int act, int accumulate, cudaStream_t s) {
+    float* outs[2] = {out, out};
+    const void* ws[2] = {w, static_cast<const char*>(w) + (size_t)n_out * n_in * 2};
+    const int rows[2] = {n_out, n_out};
+    return gemv_group(outs, ws, nullptr, kFmtBF16, rows, gated ? 2 : 1, gated, act, x, norm_w, eps, n_in, n_mean, accumulate, s);
+}
+
+}  // extern "C"
+
+namespace {
+template <typename... KArgs, typename... Args>
+cudaError_t support_launch(void (*kernel)(KArgs...), dim3 grid, dim3 block, size_t smem, cudaStream_t s, Args&&... args) {
+    static const bool use_pdl = getenv("INGOT_NO_PDL") == nullptr;
+    cudaLaunchConfig_t cfg = {};
+    cfg.gridDim = grid;
+    cfg.blockDim = block;
+    cfg.dynamicSmemBytes = smem;
+    cfg.stream = s;
+    cudaLaunchAttribute attr[1];
+    attr[0].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+    attr[0].val.programmaticStreamSerializationAllowed = 1;
+    cfg.attrs = attr;
+    cfg.numAttrs = use_pdl ? 1 : 0;
+    return cudaLaunchKernelEx(&cfg, kernel, KArgs(args)...);
+}
+
+template <typename W>
+cudaError_t launch_linear(float* out, const void* w, const float* x, int x_ld, int n_in, int n_out, int rows_per_block, int n_tok,
+                          int accumulate, cudaStream_t s) {
+    const int warps = 8;
+    const W* wt = static_cast<const W*>(w);
+    const XLayout xl = {x_ld, rows_per_block};
+    if (n_tok == 1 && rows_per_block == 0) {
+        const unsigned grid = (n_out + warps - 1) / warps;
+        return support_launch(gemv_kernel<W>, dim3(grid), dim3(warps * 32), 0, s, out, wt, x, n_in, n_out, accumulate);
+    }
+    if (n_tok >= 16 && n_out % 4 == 0 && (rows_per_block == 0 || rows_per_block % 4 == 0)) {
+        const int per = rows_per_block > 0 ? rows_per_block : n_out;
+        dim3 grid((n_out / per) * ((per + kGN - 1) / kGN), (n_tok + kGM - 1) / kGM);
+        return support_launch(gemm_kernel<W>, grid, dim3(256), 0, s, out, wt, x, n_in, n_out, n_tok, accumulate, xl);
+    }
+    if (n_tok == 1) {
+        dim3 grid((n_out + warps - 1) / warps, 1);
+        return support_launch(linear_kernel<W, 1>, grid, dim3(warps * 32), 0, s, out, wt, x, n_in, n_out, n_tok, accumulate, xl);
+    }
+    dim3 grid((n_out + warps - 1) / warps, (n_tok + 7) / 8);
+    return support_launch(linear_kernel<W, 8>, grid, dim3(warps * 32), 0, s, out, wt, x, n_in, n_out, n_tok, accumulate, xl);
+}
+}  // namespace
+
+extern "C" {
 
 // w_is_f16: 1 = __half weights, 0 = float weights.
 cudaError_t ingot_support_linear(float* out, const void* w, int w_is_f16, const float* x, int n_in, int n_out, int n_tok,
                                  int accumulate, cudaStream_t s) {
-    const int warps = 8;
-    if (n_tok == 1) {
-        const unsigned grid = (n_out + warps - 1) / warps;
-        if (w_is_f16) gemv_kernel<__half><<<grid, warps * 32, 0, s>>>(out, static_cast<const __half*>(w), x, n_in, n_out, accumulate);
-        else gemv_kernel<float><<<grid, warps * 32, 0, s>>>(out, static_cast<const float*>(w), x, n_in, n_out, accumulate);
-    } else if (n_tok >= 16 && n_in % kGK == 0 && n_out % 4 == 0) {
-        dim3 grid((n_out + kGN - 1) / kGN, (n_tok + kGM - 1) / kGM);
-        if (w_is_f16) gemm_kernel<__half><<<grid, 256, 0, s>>>(out, static_cast<const __half*>(w), x, n_in, n_out, n_tok, accumulate);
-        else gemm_kernel<float><<<grid, 256, 0, s>>>(out, static_cast<const float*>(w), x, n_in, n_out, n_tok, accumulate);
-    } else {
-        dim3 grid((n_out + warps - 1) / warps, (n_tok + 7) / 8);
-        if (w_is_f16) linear_kernel<__half, 8><<<grid, warps * 32, 0, s>>>(out, static_cast<const __half*>(w), x, n_in, n_out, n_tok, accumulate);
-        else linear_kernel<float, 8><<<grid, warps * 32, 0, s>>>(out, static_cast<const float*>(w), x, n_in, n_out, n_tok, accumulate);
-    }
+    return w_is_f16 ? launch_linear<__half>(out, w, x, n_in, n_in, n_out, 0, n_tok, accumulate, s)
+                    : launch_linear<float>(out, w, x, n_in, n_in, n_out, 0, n_tok, accumulate, s);
+}
+
+// bf16 weights, f32 activations whose rows are x_ld floats apart (a multiple of 4, as is the offset of x), f32 products.
+// rows_per_block > 0: block-diagonal (see XLayout). n_in a multiple of 8.
+cudaError_t ingot_support_linear_bf16(float* out, const void* w, const float* x, int x_ld, int n_in, int n_out, int rows_per_block,
+                                      int n_tok, int accumulate, cudaStream_t s) {
+    if (n_in % 8 != 0 || x_ld % 4 != 0 || (rows_per_block > 0 && n_out % rows_per_block != 0)) return cudaErrorInvalidValue;
+    return launch_linear<__nv_bfloat16>(out, w, x, x_ld, n_in, n_out, rows_per_block, n_tok, accumulate, s);
+}
+
+// Embedding rows of a bf16 table, widened to f32 (table rows n_in apart).
+cudaError_t ingot_support_embed_rows_bf16(float* out, const void* table, int n_in, int n_rows_table, const int32_t* rows_dev, int n_rows,
+                                          int* status_dev, cudaStream_t s) {
+    if (n_rows < 1 || n_in < 1) return cudaErrorInvalidValue;
+    embed_rows_kernel<__nv_bfloat16><<<n_rows, 256, 0, s>>>(out, static_cast<const __nv_bfloat16*>(table), n_in, n_rows_table, rows_dev, status_dev);
     return cudaGetLastError();
+}
+
+// out[r][:] = rmsnorm(x[rows ? rows[r] : r]) over rows of n floats whose mean is taken over n_mean of them (rows padded with
+// zeros up to n). rows may be null.
+cudaError_t ingot_support_rmsnorm_rows(float* out, const float* x, const float* w, const int32_t* rows_dev, int n_rows, int n, int n_mean,
+                                       float eps, cudaStream_t s) {
+    return support_launch(rmsnorm_rows_kernel, dim3(n_rows), dim3(256), 0, s, out, x, w, rows_dev, n, n_mean, eps);
+}
+
+// out[r][i] = act(gate) * up with gate = in[r][i], up = in[r][n + i] (one product holds both halves); act: 0 silu, 1 gelu (tanh form)
+cudaError_t ingot_support_gated_act(float* out, const float* in, int n_rows, int n, int act, cudaStream_t s) {
+    const size_t total = (size_t)n_rows * n;
+    return support_launch(gated_act_kernel, dim3(unsigned((total + 255) / 256)), dim3(256), 0, s, out, in, n, total, act);
 }
 
 }  // extern "C"

@@ -1,4 +1,4 @@
-// KV-cache handle, error reporting and the host-buffer convenience entry point of libingot_cuda.so.
+// KV-cache handle and the host-buffer convenience entry point of libingot_cuda.so.
 //
 // The cache replaces the one each reference backend owns (src/backend.h:1): f32
 // [n_layer][n_ctx][n_head_kv*head_dim] on the CPU (src/cpu_backend.h:23) and f16 with the same
@@ -13,45 +13,7 @@
 #include "ingot_internal.cuh"
 #include "attn_decode_params.cuh"
 
-static thread_local std::string g_last_error;
-
-void ingot_set_error(const std::string& msg) { g_last_error = msg; }
-
-int ingot_cuda_fail(cudaError_t e, const char* what) {
-    g_last_error = std::string(what) + ": " + cudaGetErrorString(e);
-    return e == cudaErrorMemoryAllocation ? INGOT_ERR_NOMEM : INGOT_ERR_CUDA;
-}
-
-bool ingot_use_pdl() {
-    static const bool v = getenv("INGOT_NO_PDL") == nullptr;
-    return v;
-}
-
 extern "C" {
-
-const char* ingot_status_string(int status) {
-    switch (status) {
-        case INGOT_OK: return "ok";
-        case INGOT_ERR_INVALID: return "invalid argument";
-        case INGOT_ERR_CUDA: return "CUDA call failed";
-        case INGOT_ERR_UNSUPPORTED: return "unsupported shape or dtype";
-        case INGOT_ERR_NOMEM: return "out of device memory";
-        case INGOT_ERR_DEVICE: return "a kernel reported an error";
-        default: return "unknown status";
-    }
-}
-
-const char* ingot_last_error(void) { return g_last_error.c_str(); }
-
-const char* ingot_build_arch(void) { return "sm_100a"; }
-
-const char* ingot_build_flags(void) {
-#ifdef INGOT_BOUNDS_CHECK
-    return "bounds-check";
-#else
-    return "";
-#endif
-}
 
 int ingot_kv_create(ingot_kv** out, int layout, int n_layer, int n_head_kv, int head_dim, int capacity,
                     int max_seqs) {

@@ -1,0 +1,493 @@
+// Recurrent sequence mixers over a ragged batch: per-channel causal convolution, the selective scan (state-space models
+// with input-dependent step size) and the real-gated linear recurrent unit. No counterpart in the reference, which only
+// has attention layers.
+//
+// A step carries tokens of several sequences (ingot_step). Each sequence owns one slot of every layer's state; a sequence
+// whose first token of the step is at position 0 starts from the zero state whatever its slot holds, so a slot needs no
+// clearing when it is handed to the next sequence. All recurrences run in f32.
+//
+// Time parallelism. A recurrence S_t = a_t S_(t-1) + b_t is cut into time chunks (ingot_scan_plan, made on the host):
+//   pass 1  every chunk runs from the zero state (a sequence's first chunk from its slot) and leaves its end state and the
+//           total decay of the chunk - for the selective scan exp(A * sum dt), for the gated unit exp(sum log a), so only
+//           one sum per channel is kept;
+//   pass 2  one thread per state element walks a sequence's chunks in order and turns end states into start states;
+//   pass 3  every chunk runs again from its start state and writes the outputs; the last chunk writes the slot.
+// A sequence that is a single chunk (every decoded token) takes pass 3 alone, straight from and to its slot.
+//
+// Decays. A slow channel multiplies its state by a = exp(x), x near 0, at every token, so an error of a that is always of
+// the same sign adds up over the memory of the channel (the 2^x unit is good to about 2^-22). Where that matters - the gated
+// unit, and the selective scan in its exact form - the state moves by S + S expm1(x), whose error is relative to 1 - a.
+#include "ingot_internal.cuh"
+
+#include <cuda_bf16.h>
+
+namespace {
+
+__device__ __forceinline__ float ex2f(float x) {
+    float y;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+    return y;
+}
+__device__ __forceinline__ float sigmoidf(float z) { return 1.0f / (1.0f + expf(-z)); }
+__device__ __forceinline__ float siluf(float z) { return z / (1.0f + expf(-z)); }
+__device__ __forceinline__ float softplusf(float z) { return z > 20.0f ? z + log1pf(expf(-z)) : log1pf(expf(z)); }
+__device__ __forceinline__ float gelu_tanhf(float z) { return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z))); }
+
+// An f32 result as the next product's operand: f32 rows, and / or one bf16 plane, or a bf16 hi + lo pair.
+struct ActOut {
+    float* f32;
+    __nv_bfloat16 *hi, *lo;
+    int ld;  // row length of every destination
+    __device__ __forceinline__ void store(size_t row, int c, float v) const {
+        const size_t i = row * ld + c;
+        if (f32) f32[i] = v;
+        if (hi) {
+            const __nv_bfloat16 h = __float2bfloat16_rn(v);
+            hi[i] = h;
+            if (lo) lo[i] = __float2bfloat16_rn(v - __bfloat162float(h));
+        }
+    }
+};
+
+// ---- causal convolution -------------------------------------------------------------------------------------------
+// out[t][c] = act(bias[c] + sum_j w[c][j] * in[t - (taps-1) + j][c]), in = raw + in_bias, zeros before position 0.
+// state [slot][taps-1][channels]: the sequence's last taps-1 inputs, oldest first. A CTA owns 128 channels and one run
+// of kConvRun tokens of one sequence; the run that starts at the sequence's first token reads the slot, computes, and
+// afterwards writes it, so no other CTA touches the slot and a run is never shorter than the history it replaces.
+constexpr int kConvRun = 16;
+constexpr int kMaxTaps = 16;
+struct ConvParams {
+    ingot_step st;
+    const float* raw;
+    int raw_ld;
+    const float *in_bias, *w, *bias;
+    int taps, channels, silu;
+    float* state;
+    ActOut out;
+};
+template <int kTaps>  // 0: run-time tap count
+__global__ void __launch_bounds__(128) causal_conv_kernel(const ConvParams p) {
+    INGOT_PDL_TRIGGER();
+    INGOT_PDL_WAIT();
+    const int taps = kTaps ? kTaps : p.taps;
+    const int seq = blockIdx.z, c = blockIdx.x * 128 + threadIdx.x;
+    const int len = p.st.len[seq], t0 = blockIdx.y * kConvRun;
+    if (c >= p.channels || t0 >= len) return;
+    const int pos0 = p.st.pos0[seq];
+    const float* in = p.raw + (size_t)p.st.row_start[seq] * p.raw_ld + c;
+    const size_t row0 = p.st.row_start[seq];
+    float* slot = p.state + (size_t)p.st.slot[seq] * (taps - 1) * p.channels + c;
+    const float ib = p.in_bias ? p.in_bias[c] : 0.f, b = p.bias ? p.bias[c] : 0.f;
+    constexpr int kH = kTaps ? kTaps : kMaxTaps;
+    float w[kH], h[kH];  // h: the last taps inputs, newest at taps-1
+#pragma unroll
+    for (int j = 0; j < kH; j++) w[j] = j < taps ? p.w[(size_t)c * taps + j] : 0.f;
+    // input at position t of this step (t < 0: from the slot, or zero before the sequence's start)
+    auto input = [&](int t) -> float {
+        if (t >= 0) return in[(size_t)t * p.raw_ld] + ib;
+        return pos0 + t >= 0 ? slot[(size_t)(taps - 1 + t) * p.channels] : 0.f;
+    };
+#pragma unroll
+    for (int j = 0; j < kH; j++) h[j] = j < taps - 1 ? input(t0 - (taps - 1) + j) : 0.f;
+    const int t_end = min(len, t0 + kConvRun);
+    for (int t = t0; t < t_end; t++) {
+        const float x = in[(size_t)t * p.raw_ld] + ib;
+        float acc = b;
+#pragma unroll
+        for (int j = 0; j < kH; j++)
+            if (j < taps - 1) acc = fmaf(w[j], h[j], acc);
+#pragma unroll
+        for (int j = 0; j < kH; j++)
+            if (j == taps - 1) acc = fmaf(w[j], x, acc);
+        p.out.store(row0 + t, c, p.silu ? siluf(acc) : acc);
+#pragma unroll
+        for (int j = 0; j + 1 < kH; j++) h[j] = j < taps - 2 ? h[j + 1] : x;
+    }
+    if (t0 == 0) {
+        // the slot's new contents: inputs len-(taps-1) .. len-1; the ones that are older than this step move down
+        float n[kH];
+#pragma unroll
+        for (int j = 0; j < kH; j++) n[j] = j < taps - 1 ? input(len - (taps - 1) + j) : 0.f;
+#pragma unroll
+        for (int j = 0; j < kH; j++)
+            if (j < taps - 1) slot[(size_t)j * p.channels] = n[j];
+    }
+}
+
+// ---- selective scan -------------------------------------------------------------------------------------------------
+// Per channel c and state n: S <- exp(dt A) S + dt x B, y = sum_n S C + D x, out = y * silu(z); dt = softplus(raw + bias).
+// kLanes lanes share a channel, each holding kS of its states in registers. A CTA of 128 threads owns 128 / lanes channels
+// over one time chunk; inputs are staged 16 tokens at a time in shared memory, the next 16 requested (cp.async) while the
+// current ones are computed.
+constexpr int kScanTile = 16;
+struct ScanParams {
+    ingot_step st;
+    const int32_t *chunk_seq, *chunk_t0, *chunk_len, *seq_chunk0;
+    int n_chunks;
+    const float* x; int x_ld;
+    const float* dt; int dt_ld;
+    const float* dt_bias;
+    const float* bc; int bc_ld, b_off, c_off;
+    const float* z; int z_ld;
+    const float* a2;     // [inner][n_pad]: -exp(A_log) * log2(e), 0 in the padding
+    const float* d;
+    float* state;        // [slot][inner][n_pad]
+    float* part;         // [chunk][inner][n_pad] end states, then start states
+    float* part_sum;     // [chunk][inner] sum of dt
+    int inner, n_pad, lanes_log2;
+    ActOut out;
+};
+__device__ __forceinline__ void cp_async16(void* dst, const void* src, bool on) {
+    const uint32_t d = (uint32_t)__cvta_generic_to_shared(dst);
+    asm volatile("cp.async.ca.shared.global [%0], [%1], 16, %2;" ::"r"(d), "l"(src), "r"(on ? 16 : 0) : "memory");
+}
+__device__ __forceinline__ void cp_async_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
+template <int N>
+__device__ __forceinline__ void cp_async_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
+
+// kLg: log2 of the lanes per channel, or -1 for p.lanes_log2
+template <int kS, bool kOutput, int kLg, bool kExact>
+__global__ void __launch_bounds__(128) selective_scan_kernel(const ScanParams p) {
+    extern __shared__ __align__(16) float smem[];
+    INGOT_PDL_TRIGGER();
+    INGOT_PDL_WAIT();
+    const int chunk = blockIdx.y;
+    const int seq = p.chunk_seq[chunk], t0 = p.chunk_t0[chunk], len = p.chunk_len[chunk];
+    const bool first = t0 == 0, last = t0 + len == p.st.len[seq];
+    if (!kOutput && first && last) return;  // a single chunk needs no partial state
+    const int lg = kLg >= 0 ? kLg : p.lanes_log2;
+    const int lanes = 1 << lg, n_ch = 128 >> lg;
+    const int ch = threadIdx.x >> lg, part = threadIdx.x & (lanes - 1);
+    const int c_base = blockIdx.x * n_ch, c = c_base + ch;
+    const bool live = c < p.inner;
+    const size_t row0 = (size_t)p.st.row_start[seq] + t0;
+    const int np = p.n_pad;
+
+    // [2 buffers][16 tokens]: x, dt [n_ch], B, C [np]; then dt * x of the current tile and y
+    const int tile_floats = kScanTile * (2 * n_ch + 2 * np);
+    float* const s_dtx = smem + 2 * tile_floats;
+    float* const s_y = s_dtx + kScanTile * n_ch;
+
+    auto stage = [&](int tile) {
+        float* sx = smem + (tile & 1) * tile_floats;
+        float* sdt = sx + kScanTile * n_ch;
+        float* sb = sdt + kScanTile * n_ch;
+        float* sc = sb + kScanTile * np;
+        const int t_base = tile * kScanTile;
+        const int ch4 = n_ch >> 2;
+        for (int i = threadIdx.x; i < kScanTile * ch4; i += 128) {
+            const int t = i / ch4, q = (i - t * ch4) * 4;
+            const bool on = t_base + t < len && c_base + q < p.inner;
+            const size_t row = row0 + min(t_base + t, len - 1);
+            const int cc = min(c_base + q, p.inner - 4);
+            cp_async16(sx + t * n_ch + q, p.x + row * p.x_ld + cc, on);
+            cp_async16(sdt + t * n_ch + q, p.dt + row * p.dt_ld + cc, on);
+        }
+        const int np4 = np >> 2;
+        for (int i = threadIdx.x; i < kScanTile * np4; i += 128) {
+            const int t = i / np4, q = (i - t * np4) * 4;
+            const bool on = t_base + t < len;
+            const size_t row = row0 + min(t_base + t, len - 1);
+            cp_async16(sb + t * np + q, p.bc + row * p.bc_ld + p.b_off + q, on);
+            if (kOutput) cp_async16(sc + t * np + q, p.bc + row * p.bc_ld + p.c_off + q, on);
+        }
+        cp_async_commit();
+    };
+
+    const int n_tiles = (len + kScanTile - 1) / kScanTile;
+    stage(0);
+
+    float a[kS], s[kS];
+    const size_t sidx = (size_t)(live ? c : 0) * np + part * kS;
+#pragma unroll
+    for (int i = 0; i < kS; i++) {
+        a[i] = live ? p.a2[sidx + i] : 0.f;
+        s[i] = 0.f;
+    }
+    const size_t slot_base = (size_t)p.st.slot[seq] * p.inner * np;
+    if (live) {
+        if (first) {
+            // pass 3 of a multi-chunk sequence reads its start state from the scratch too: the last chunk's CTA may write
+            // the slot before this CTA gets to read it
+            if (kOutput && !last) {
+#pragma unroll
+                for (int i = 0; i < kS; i++) s[i] = p.part[(size_t)chunk * p.inner * np + sidx + i];
+            } else if (p.st.pos0[seq] > 0) {
+#pragma unroll
+                for (int i = 0; i < kS; i++) s[i] = p.state[slot_base + sidx + i];
+            }
+        } else if (kOutput) {
+#pragma unroll
+            for (int i = 0; i < kS; i++) s[i] = p.part[(size_t)chunk * p.inner * np + sidx + i];
+        }
+    }
+    const int my_ch = threadIdx.x % n_ch;  // the channel this thread prepares and writes (n_ch divides 128)
+    const bool my_live = c_base + my_ch < p.inner;
+    const float my_bias = my_live ? p.dt_bias[c_base + my_ch] : 0.f;
+    const float my_d = kOutput && my_live ? p.d[c_base + my_ch] : 0.f;
+    float sum_dt = 0.f;
+
+    for (int tile = 0; tile < n_tiles; tile++) {
+        if (tile + 1 < n_tiles) { stage(tile + 1); cp_async_wait<1>(); } else { cp_async_wait<0>(); }
+        __syncthreads();
+        float* sx = smem + (tile & 1) * tile_floats;
+        float* sdt = sx + kScanTile * n_ch;
+        const float* sb = sdt + kScanTile * n_ch;
+        const float* sc = sb + kScanTile * np;
+        const int n_t = min(kScanTile, len - tile * kScanTile);
+        for (int i = threadIdx.x; i < kScanTile * n_ch; i += 128) {
+            const int t = i / n_ch;
+            const float dt = t < n_t ? softplusf(sdt[i] + my_bias) : 0.f;
+            sdt[i] = dt;
+            s_dtx[i] = dt * sx[i];
+        }
+        __syncthreads();
+#pragma unroll 4
+        for (int t = 0; t < n_t; t++) {
+            const float dt = sdt[t * n_ch + ch], dtx = s_dtx[t * n_ch + ch];
+            const float* b = sb + t * np + part * kS;
+            const float* cc = sc + t * np + part * kS;
+            float y = 0.f;
+#pragma unroll
+            for (int i = 0; i < kS; i++) {
+                if (kExact) s[i] += fmaf(expm1f(dt * a[i] * 0.69314718f), s[i], dtx * b[i]);
+                else s[i] = fmaf(ex2f(dt * a[i]), s[i], dtx * b[i]);
+                if (kOutput) y = fmaf(s[i], cc[i], y);
+            }
+            if (kOutput) {
+                for (int o = lanes >> 1; o > 0; o >>= 1) y += __shfl_xor_sync(0xffffffffu, y, o);
+                if (part == 0) s_y[t * n_ch + ch] = y;
+            } else {
+                sum_dt += dt;
+            }
+        }
+        if (kOutput) {
+            __syncthreads();
+            if (my_live) {
+                for (int i = threadIdx.x; i < n_t * n_ch; i += 128) {
+                    const size_t row = row0 + tile * kScanTile + i / n_ch;
+                    const float y = fmaf(my_d, sx[i], s_y[i]);
+                    p.out.store(row, c_base + my_ch, y * siluf(p.z[row * p.z_ld + c_base + my_ch]));
+                }
+            }
+        }
+        __syncthreads();  // the tile's buffers are staged over two tiles from now, s_dtx / s_y in the next one
+    }
+    if (!live) return;
+    if (!kOutput) {
+#pragma unroll
+        for (int i = 0; i < kS; i++) p.part[(size_t)chunk * p.inner * np + sidx + i] = s[i];
+        if (part == 0) p.part_sum[(size_t)chunk * p.inner + c] = sum_dt;
+    } else if (last) {
+#pragma unroll
+        for (int i = 0; i < kS; i++) p.state[slot_base + sidx + i] = s[i];
+    }
+}
+
+// Pass 2: end states -> start states, sequence by sequence. The first chunk ran from the slot, so its end state is exact.
+__global__ void __launch_bounds__(256) selective_scan_link_kernel(const ScanParams p) {
+    INGOT_PDL_TRIGGER();
+    INGOT_PDL_WAIT();
+    const int seq = blockIdx.y;
+    const int k0 = p.seq_chunk0[seq], k1 = p.seq_chunk0[seq + 1];
+    const size_t per = (size_t)p.inner * p.n_pad;
+    const size_t i = (size_t)blockIdx.x * 256 + threadIdx.x;
+    if (k1 - k0 < 2 || i >= per) return;
+    const int c = int(i / p.n_pad);
+    const float a = p.a2[i];
+    float s = p.st.pos0[seq] > 0 ? p.state[(size_t)p.st.slot[seq] * per + i] : 0.f;
+    float end = p.part[(size_t)k0 * per + i];
+    p.part[(size_t)k0 * per + i] = s;
+    s = end;
+    for (int k = k0 + 1; k < k1; k++) {
+        end = p.part[(size_t)k * per + i];
+        p.part[(size_t)k * per + i] = s;
+        s = fmaf(ex2f(a * p.part_sum[(size_t)k * p.inner + c]), s, end);
+    }
+}
+
+// ---- real-gated linear recurrent unit -------------------------------------------------------------------------------
+// r = sigmoid(gr + br), i = sigmoid(gi + bi), log a = -8 r softplus(lam), S <- a S + sqrt(1 - a^2) i u;
+// out = out_scale * S * gelu(y + y_bias). gates [rows][...]: the products of the two block-diagonal gate matrices, block b's
+// m recurrence gates followed by its m input gates.
+struct LruParams {
+    ingot_step st;
+    const int32_t *chunk_seq, *chunk_t0, *chunk_len, *seq_chunk0;
+    int n_chunks;
+    const float* u; int u_ld;
+    const float* gates; int gates_ld, block;
+    const float *br, *bi, *sp;  // gate biases, softplus(lam)
+    const float* y; int y_ld;
+    const float* y_bias;
+    float* state;     // [slot][width]
+    float *part, *part_sum;  // [chunk][width]
+    int width;
+    float out_scale;
+    ActOut out;
+};
+template <bool kOutput>
+__global__ void __launch_bounds__(128) gated_lru_kernel(const LruParams p) {
+    INGOT_PDL_TRIGGER();
+    INGOT_PDL_WAIT();
+    const int chunk = blockIdx.y, c = blockIdx.x * 128 + threadIdx.x;
+    const int seq = p.chunk_seq[chunk], t0 = p.chunk_t0[chunk], len = p.chunk_len[chunk];
+    const bool first = t0 == 0, last = t0 + len == p.st.len[seq];
+    if ((!kOutput && first && last) || c >= p.width) return;
+    const size_t row0 = (size_t)p.st.row_start[seq] + t0;
+    const int gcol = (c / p.block) * 2 * p.block + c % p.block;
+    const float br = p.br[c], bi = p.bi[c], k = -8.0f * p.sp[c], yb = kOutput ? p.y_bias[c] : 0.f;
+    float* slot = p.state + (size_t)p.st.slot[seq] * p.width + c;
+    float s = 0.f;
+    if (kOutput && !(first && last)) s = p.part[(size_t)chunk * p.width + c];
+    else if (first && p.st.pos0[seq] > 0) s = *slot;
+    float sum = 0.f;
+    const float* u = p.u + row0 * p.u_ld + c;
+    const float* g = p.gates + row0 * p.gates_ld + gcol;
+    const float* y = kOutput ? p.y + row0 * p.y_ld + c : nullptr;
+#pragma unroll 4
+    for (int t = 0; t < len; t++) {
+        const float log_a = k * sigmoidf(g[(size_t)t * p.gates_ld] + br);
+        const float in = sigmoidf(g[(size_t)t * p.gates_ld + p.block] + bi) * u[(size_t)t * p.u_ld];
+        const float e = expm1f(log_a);  // a - 1; 1 - a^2 = -e (2 + e)
+        s += fmaf(e, s, sqrtf(-e * (2.0f + e)) * in);
+        if (kOutput) p.out.store(row0 + t, c, p.out_scale * s * gelu_tanhf(y[(size_t)t * p.y_ld] + yb));
+        else sum += log_a;
+    }
+    if (!kOutput) {
+        p.part[(size_t)chunk * p.width + c] = s;
+        p.part_sum[(size_t)chunk * p.width + c] = sum;
+    } else if (last) {
+        *slot = s;
+    }
+}
+__global__ void __launch_bounds__(128) gated_lru_link_kernel(const LruParams p) {
+    INGOT_PDL_TRIGGER();
+    INGOT_PDL_WAIT();
+    const int seq = blockIdx.y, c = blockIdx.x * 128 + threadIdx.x;
+    const int k0 = p.seq_chunk0[seq], k1 = p.seq_chunk0[seq + 1];
+    if (k1 - k0 < 2 || c >= p.width) return;
+    float s = p.st.pos0[seq] > 0 ? p.state[(size_t)p.st.slot[seq] * p.width + c] : 0.f;
+    float end = p.part[(size_t)k0 * p.width + c];
+    p.part[(size_t)k0 * p.width + c] = s;
+    s = end;
+    for (int k = k0 + 1; k < k1; k++) {
+        end = p.part[(size_t)k * p.width + c];
+        p.part[(size_t)k * p.width + c] = s;
+        s = fmaf(expf(p.part_sum[(size_t)k * p.width + c]), s, end);
+    }
+}
+
+bool step_ok(const ingot_step* st) {
+    return st && st->n_tok >= 1 && st->n_seq >= 1 && st->n_seq <= 65535 && st->max_len >= 1 && st->row_start && st->len && st->pos0 && st->slot;
+}
+bool plan_ok(const ingot_scan_plan* pl) {
+    return pl && pl->n_chunks >= 1 && pl->n_chunks <= 65535 && pl->chunk_seq && pl->chunk_t0 && pl->chunk_len && pl->seq_chunk0;
+}
+ActOut act_out(const ingot_act_out* o) {
+    return ActOut{o->f32, static_cast<__nv_bfloat16*>(o->hi), static_cast<__nv_bfloat16*>(o->lo), o->ld};
+}
+
+int scan_lanes_log2(int n_state) {
+    int l = 2;  // 4 lanes per channel up to 32 states, then as many as keep 8 states per lane
+    while ((8 << l) < n_state) l++;
+    return l;
+}
+
+}  // namespace
+
+extern "C" {
+
+int ingot_causal_conv(const ingot_step* step, const float* in_dev, int in_ld, const float* in_bias_dev, const float* w_dev,
+                      const float* bias_dev, int taps, int channels, int silu, float* state_dev, const ingot_act_out* out,
+                      void* stream) {
+    INGOT_REQUIRE(step_ok(step) && in_dev && w_dev && state_dev && out, "ingot_causal_conv: null argument or empty step");
+    INGOT_REQUIRE(channels >= 1 && taps >= 1 && taps <= kMaxTaps, "ingot_causal_conv: between 1 and 16 taps");
+    ConvParams p = {*step, in_dev, in_ld, in_bias_dev, w_dev, bias_dev, taps, channels, silu, state_dev, act_out(out)};
+    const dim3 grid((channels + 127) / 128, (step->max_len + kConvRun - 1) / kConvRun, step->n_seq);
+    INGOT_REQUIRE(grid.y <= 65535, "ingot_causal_conv: too many tokens of one sequence in one step");
+    auto kernel = taps == 2 ? causal_conv_kernel<2> : taps == 3 ? causal_conv_kernel<3> : taps == 4 ? causal_conv_kernel<4> : causal_conv_kernel<0>;
+    INGOT_CUDA_TRY(ingot_launch_pdl(kernel, grid, dim3(128), 0, static_cast<cudaStream_t>(stream), p));
+    return INGOT_OK;
+}
+
+int ingot_scan_state_pad(int n_state) {
+    if (n_state < 1 || n_state > 256) return 0;
+    const int lanes = 1 << scan_lanes_log2(n_state);
+    const int q = lanes > 8 ? lanes : 8;
+    return (n_state + q - 1) / q * q;
+}
+
+int ingot_selective_scan(const ingot_step* step, const ingot_scan_plan* plan, const float* x_dev, int x_ld, const float* dt_dev,
+                         int dt_ld, const float* dt_bias_dev, const float* bc_dev, int bc_ld, int b_off, int c_off,
+                         const float* z_dev, int z_ld, const float* a_log2e_dev, const float* d_dev, float* state_dev, int inner,
+                         int n_state, int exact, const ingot_act_out* out, void* stream) {
+    INGOT_REQUIRE(step_ok(step) && plan_ok(plan), "ingot_selective_scan: bad step or plan");
+    INGOT_REQUIRE(x_dev && dt_dev && dt_bias_dev && bc_dev && z_dev && a_log2e_dev && d_dev && state_dev && out, "ingot_selective_scan: null argument");
+    INGOT_REQUIRE(inner >= 4 && inner % 4 == 0 && x_ld % 4 == 0 && dt_ld % 4 == 0 && bc_ld % 4 == 0 && b_off % 4 == 0 && c_off % 4 == 0,
+                  "ingot_selective_scan: rows and offsets must be multiples of 4 floats");
+    const int n_pad = ingot_scan_state_pad(n_state);
+    INGOT_REQUIRE(n_pad > 0, "ingot_selective_scan: between 1 and 256 states");
+    const bool multi = plan->max_chunks > 1;
+    INGOT_REQUIRE(!multi || (plan->scratch_dev && plan->scratch_floats >= (size_t)plan->n_chunks * inner * (n_pad + 1)),
+                  "ingot_selective_scan: scratch too small");
+    const int lg = scan_lanes_log2(n_state), lanes = 1 << lg, n_ch = 128 >> lg;
+    const int per_lane = (n_state + lanes - 1) / lanes;
+    ScanParams p = {*step, plan->chunk_seq, plan->chunk_t0, plan->chunk_len, plan->seq_chunk0, plan->n_chunks,
+                    x_dev, x_ld, dt_dev, dt_ld, dt_bias_dev, bc_dev, bc_ld, b_off, c_off, z_dev, z_ld, a_log2e_dev, d_dev,
+                    state_dev, plan->scratch_dev, plan->scratch_dev ? plan->scratch_dev + (size_t)plan->n_chunks * inner * n_pad : nullptr,
+                    inner, n_pad, lg, act_out(out)};
+    const size_t smem = (size_t)kScanTile * (2 * (2 * n_ch + 2 * n_pad) + 2 * n_ch) * sizeof(float);
+    typedef void (*Kernel)(ScanParams);
+    Kernel k_end, k_out;
+#define INGOT_SCAN_PICK(S, OUT)                                                                                                     \
+    (exact ? (lg == 2 ? selective_scan_kernel<S, OUT, 2, true> : selective_scan_kernel<(S < 5 ? 5 : S), OUT, -1, true>)             \
+           : (lg == 2 ? selective_scan_kernel<S, OUT, 2, false> : selective_scan_kernel<(S < 5 ? 5 : S), OUT, -1, false>))
+#define INGOT_SCAN_CASE(S)                 \
+    case S:                                \
+        k_end = INGOT_SCAN_PICK(S, false); \
+        k_out = INGOT_SCAN_PICK(S, true);  \
+        break
+    switch (per_lane) {  // more than 4 lanes: always 5 to 8 states per lane
+        INGOT_SCAN_CASE(1); INGOT_SCAN_CASE(2); INGOT_SCAN_CASE(3); INGOT_SCAN_CASE(4);
+        INGOT_SCAN_CASE(5); INGOT_SCAN_CASE(6); INGOT_SCAN_CASE(7); INGOT_SCAN_CASE(8);
+        default: ingot_set_error("ingot_selective_scan: unsupported state count"); return INGOT_ERR_UNSUPPORTED;
+    }
+#undef INGOT_SCAN_CASE
+#undef INGOT_SCAN_PICK
+    cudaStream_t s = static_cast<cudaStream_t>(stream);
+    const dim3 grid((inner + n_ch - 1) / n_ch, plan->n_chunks);
+    if (smem > 48 * 1024) {
+        INGOT_CUDA_TRY(cudaFuncSetAttribute(k_end, cudaFuncAttributeMaxDynamicSharedMemorySize, int(smem)));
+        INGOT_CUDA_TRY(cudaFuncSetAttribute(k_out, cudaFuncAttributeMaxDynamicSharedMemorySize, int(smem)));
+    }
+    if (multi) {
+        INGOT_CUDA_TRY(ingot_launch_pdl(k_end, grid, dim3(128), smem, s, p));
+        INGOT_CUDA_TRY(ingot_launch_pdl(selective_scan_link_kernel, dim3(unsigned(((size_t)inner * n_pad + 255) / 256), step->n_seq), dim3(256), 0, s, p));
+    }
+    INGOT_CUDA_TRY(ingot_launch_pdl(k_out, grid, dim3(128), smem, s, p));
+    return INGOT_OK;
+}
+
+int ingot_gated_lru(const ingot_step* step, const ingot_scan_plan* plan, const float* u_dev, int u_ld, const float* gates_dev,
+                    int gates_ld, int block, const float* r_bias_dev, const float* i_bias_dev, const float* softplus_lam_dev,
+                    const float* y_dev, int y_ld, const float* y_bias_dev, float* state_dev, int width, float out_scale,
+                    const ingot_act_out* out, void* stream) {
+    INGOT_REQUIRE(step_ok(step) && plan_ok(plan), "ingot_gated_lru: bad step or plan");
+    INGOT_REQUIRE(u_dev && gates_dev && r_bias_dev && i_bias_dev && softplus_lam_dev && y_dev && y_bias_dev && state_dev && out, "ingot_gated_lru: null argument");
+    INGOT_REQUIRE(width >= 1 && block >= 1 && width % block == 0, "ingot_gated_lru: the width must be a multiple of the block size");
+    const bool multi = plan->max_chunks > 1;
+    INGOT_REQUIRE(!multi || (plan->scratch_dev && plan->scratch_floats >= (size_t)plan->n_chunks * width * 2), "ingot_gated_lru: scratch too small");
+    LruParams p = {*step, plan->chunk_seq, plan->chunk_t0, plan->chunk_len, plan->seq_chunk0, plan->n_chunks, u_dev, u_ld, gates_dev, gates_ld,
+                   block, r_bias_dev, i_bias_dev, softplus_lam_dev, y_dev, y_ld, y_bias_dev, state_dev, plan->scratch_dev,
+                   plan->scratch_dev ? plan->scratch_dev + (size_t)plan->n_chunks * width : nullptr, width, out_scale, act_out(out)};
+    cudaStream_t s = static_cast<cudaStream_t>(stream);
+    const dim3 grid((width + 127) / 128, plan->n_chunks);
+    if (multi) {
+        INGOT_CUDA_TRY(ingot_launch_pdl(gated_lru_kernel<false>, grid, dim3(128), 0, s, p));
+        INGOT_CUDA_TRY(ingot_launch_pdl(gated_lru_link_kernel, dim3((width + 127) / 128, step->n_seq), dim3(128), 0, s, p));
+    }
+    INGOT_CUDA_TRY(ingot_launch_pdl(gated_lru_kernel<true>, grid, dim3(128), 0, s, p));
+    return INGOT_OK;
+}
+
+}  // extern "C"
