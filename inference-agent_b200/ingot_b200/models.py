@@ -1,0 +1,143 @@
+"""ctypes binding of libingot_models.so: model folders (config.json + model.safetensors), the ragged step and the scheduler.
+
+Build it with `make -C inference-agent_b200/backend models`. Tokens are ids; logits come back as numpy arrays.
+"""
+import ctypes as C
+import os
+
+import numpy as np
+
+_HERE = os.path.dirname(os.path.abspath(__file__))
+LIB_PATH = os.path.join(os.path.dirname(_HERE), "backend", "_build", "libingot_models.so")
+_i32 = np.ctypeslib.ndpointer(np.int32, flags="C_CONTIGUOUS")
+_lib = None
+
+
+def lib():
+    global _lib
+    if _lib is None:
+        if not os.path.exists(LIB_PATH):
+            raise FileNotFoundError(f"{LIB_PATH} not found: build it with `make -C inference-agent_b200/backend models`")
+        l = C.CDLL(LIB_PATH)
+        l.ingot_models_last_error.restype = C.c_char_p
+        l.ingot_model_open.restype = C.c_void_p
+        l.ingot_model_open.argtypes = [C.c_char_p, C.c_int, C.c_int, C.c_int, C.c_int]
+        l.ingot_model_close.argtypes = [C.c_void_p]
+        l.ingot_model_vocab.argtypes = [C.c_void_p]
+        l.ingot_model_weight_bytes.argtypes = [C.c_void_p]
+        l.ingot_model_weight_bytes.restype = C.c_longlong
+        l.ingot_model_last_step_ms.argtypes = [C.c_void_p]
+        l.ingot_model_last_step_ms.restype = C.c_float
+        l.ingot_model_step.argtypes = [C.c_void_p, C.c_int, _i32, _i32, _i32, _i32, _i32, _i32, C.c_void_p]
+        l.ingot_model_release.argtypes = [C.c_void_p, C.c_int]
+        l.ingot_model_tap.argtypes = [C.c_void_p, C.c_int]
+        l.ingot_model_residuals.argtypes = [C.c_void_p, C.c_void_p, C.c_longlong]
+        l.ingot_model_residuals.restype = C.c_longlong
+        l.ingot_model_generate.argtypes = [C.c_void_p, _i32, _i32, _i32, C.c_void_p, C.c_int, C.c_int, C.c_void_p, _i32, C.c_int, _i32,
+                                           C.c_void_p]
+        _lib = l
+    return _lib
+
+
+class ModelError(RuntimeError):
+    pass
+
+
+def _a(x):
+    return np.ascontiguousarray(np.asarray(x, dtype=np.int32).reshape(-1))
+
+
+class Model:
+    """An opened model folder. max_tokens: tokens the live sequences hold together; max_seqs: sequences alive at a time."""
+
+    def __init__(self, path, f32=False, max_tokens=4096, max_seqs=4, max_step_tokens=0):
+        self.handle = lib().ingot_model_open(os.fsencode(path), int(f32), max_tokens, max_seqs, max_step_tokens)
+        if not self.handle:
+            raise ModelError(lib().ingot_models_last_error().decode())
+        self.n_vocab = lib().ingot_model_vocab(self.handle)
+
+    def close(self):
+        if self.handle:
+            lib().ingot_model_close(self.handle)
+            self.handle = None
+
+    def __enter__(self):
+        return self
+
+    def __exit__(self, *exc):
+        self.close()
+
+    def _check(self, rc):
+        if rc != 0:
+            raise ModelError(lib().ingot_models_last_error().decode())
+
+    def step(self, portions):
+        """portions: [(seq_id, pos0, tokens, want)]: one batch. Returns the wanted logits rows, in order, [n, vocab]."""
+        n_want = sum(len(p[3]) for p in portions)
+        out = np.empty((n_want, self.n_vocab), dtype=np.float32)
+        cat = lambda k: _a(np.concatenate([np.asarray(p[k], dtype=np.int32).reshape(-1) for p in portions]))
+        self._check(lib().ingot_model_step(self.handle, len(portions), _a([p[0] for p in portions]), _a([p[1] for p in portions]),
+                                           _a([len(p[2]) for p in portions]), cat(2), _a([len(p[3]) for p in portions]), cat(3),
+                                           out.ctypes.data if n_want else None))
+        return out
+
+    def release(self, seq_id):
+        self._check(lib().ingot_model_release(self.handle, seq_id))
+
+    def tap(self, on=True):
+        lib().ingot_model_tap(self.handle, int(on))
+
+    def residuals(self):
+        n = lib().ingot_model_residuals
+        buf = np.empty(1 << 24, dtype=np.float32)
+        total = n(self.handle, buf.ctypes.data, buf.size)
+        return buf[:total].copy()
+
+    def generate(self, prompts, max_new, arrival=None, stop_token=-1, sampling=None):
+        """prompts: lists of ids; max_new: int or list. Returns ([ids], steps, rows) after running all through the scheduler."""
+        n = len(prompts)
+        lim = _a(max_new if np.ndim(max_new) else [max_new] * n)
+        out = np.zeros((n, max(1, int(lim.max()))), dtype=np.int32)
+        counts = np.zeros(n, dtype=np.int32)
+        stats = (C.c_longlong * 2)()
+        sp = None if sampling is None else np.asarray(sampling, dtype=np.float64)
+        arr = None if arrival is None else _a(arrival)
+        self._check(lib().ingot_model_generate(self.handle, _a(np.concatenate([np.asarray(p, dtype=np.int32) for p in prompts])),
+                                               _a([len(p) for p in prompts]), lim, None if arr is None else arr.ctypes.data, n, stop_token,
+                                               None if sp is None else sp.ctypes.data, out, out.shape[1], counts, stats))
+        return [out[i, :counts[i]].tolist() for i in range(n)], stats[0], stats[1]
+
+    @property
+    def weight_bytes(self):
+        return lib().ingot_model_weight_bytes(self.handle)
+
+    @property
+    def last_step_ms(self):
+        return lib().ingot_model_last_step_ms(self.handle)
+
+
+def write_safetensors(path, tensors):
+    """tensors: name -> (dtype name, numpy array holding the raw bits: uint16 for BF16). Streams to `path`."""
+    import json
+    import struct
+    header, at = {}, 0
+    for name, (dtype, arr) in tensors.items():
+        header[name] = {"dtype": dtype, "shape": list(arr.shape), "data_offsets": [at, at + arr.nbytes]}
+        at += arr.nbytes
+    text = json.dumps(header).encode()
+    text += b" " * (-len(text) % 8)
+    with open(path, "wb") as f:
+        f.write(struct.pack("<Q", len(text)))
+        f.write(text)
+        for _, arr in tensors.values():
+            f.write(np.ascontiguousarray(arr).tobytes())
+
+
+def to_bf16(x):
+    """float array -> bf16 bits (uint16), round to nearest even."""
+    u = np.ascontiguousarray(x, dtype=np.float32).view(np.uint32)
+    return ((u + 0x7FFF + ((u >> 16) & 1)) >> 16).astype(np.uint16)
+
+
+def from_bf16(bits):
+    return (bits.astype(np.uint32) << 16).view(np.float32)

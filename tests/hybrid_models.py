@@ -1,0 +1,99 @@
+"""Small random models of the hybrid design for the tests: configurations, weights, folders, and the checker's logits."""
+import json
+import os
+
+import numpy as np
+
+import hybrid_reference as R
+from ingot_b200 import models as M
+
+
+def mamba(inner, state, dt_rank, conv, ff=None):
+    return {"type": "mamba1", "mixer": {"inner": inner, "state": state, "dt_rank": dt_rank, "conv": conv},
+            "mlp": None if ff is None else {"kind": "dense", "ff": ff}}
+
+
+def parallel(heads, kv_heads, dim, size, width, blocks, conv, ff=None, scale=0.2, left_scale=0.7, right_scale=0.9):
+    return {"type": "parallel",
+            "mixer": {"left": {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": dim, "scale": scale, "mask": {"size": size}},
+                      "right": {"width": width, "blocks": blocks, "conv": conv}, "left_scale": left_scale, "right_scale": right_scale},
+            "mlp": None if ff is None else {"kind": "dense", "ff": ff}}
+
+
+def config(layers, vocab=96, width=48, eps=1e-5):
+    return {"architecture": "Besudra", "layers": layers, "norm": {"eps": eps}, "vocab": vocab, "width": width}
+
+
+def shapes(cfg):
+    d, v = cfg["width"], cfg["vocab"]
+    out = {"embed": (v, d), "head": (v, d), "final.norm": (d,)}
+    for i, layer in enumerate(cfg["layers"]):
+        p, m = f"l{i}.", layer["mixer"]
+        out[p + "norm1"] = (d,)
+        if layer["type"] == "mamba1":
+            n, s, r = m["inner"], m["state"], m["dt_rank"]
+            out.update({p + "mix.in": (2 * n, d), p + "mix.conv": (n, m["conv"]), p + "mix.conv.b": (n,), p + "mix.x": (r + 2 * s, n),
+                        p + "mix.dt": (n, r), p + "mix.dt.b": (n,), p + "mix.A_log": (n, s), p + "mix.D": (n,), p + "mix.o": (d, n)})
+        else:
+            a, b, q = m["left"], m["right"], p + "mix."
+            hq, hk, w = a["heads"] * a["dim"], a["kv_heads"] * a["dim"], b["width"]
+            k = w // b["blocks"]
+            out.update({q + "left.q": (hq, d), q + "left.k": (hk, d), q + "left.q.norm": (hq,), q + "left.k.norm": (hk,), q + "left.o": (d, hq),
+                        q + "right.y": (w, d), q + "right.y.b": (w,), q + "right.x": (w, d), q + "right.x.b": (w,),
+                        q + "right.conv": (w, b["conv"]), q + "right.conv.b": (w,), q + "right.ra": (b["blocks"], k, k),
+                        q + "right.ra.b": (b["blocks"], k), q + "right.ri": (b["blocks"], k, k), q + "right.ri.b": (b["blocks"], k),
+                        q + "right.lam": (w,), q + "right.o": (d, w)})
+        if layer["mlp"] is not None:
+            f = layer["mlp"]["ff"]
+            out.update({p + "norm2": (d,), p + "mlp.gate": (f, d), p + "mlp.up": (f, d), p + "mlp.down": (d, f)})
+    return out
+
+
+def random_weights(cfg, seed=0, qk_gain=2.5):
+    """bf16-representable float32 weights. Decays are slow (long memory) and the scores are sharp, so that a lost state or a
+    key on the wrong side of an edge moves the logits."""
+    rng = np.random.default_rng(seed)
+    w = {}
+    for name, shape in shapes(cfg).items():
+        leaf = name.split(".", 1)[1] if name.startswith("l") and "." in name else name
+        if name == "embed":
+            x = rng.standard_normal(shape)
+        elif leaf.endswith("norm") or leaf.endswith("norm1") or leaf.endswith("norm2"):
+            x = 1.0 + 0.25 * rng.standard_normal(shape)
+            if leaf.endswith("q.norm") or leaf.endswith("k.norm"):
+                x = x * qk_gain
+        elif leaf.endswith("dt.b"):
+            x = rng.uniform(-4.5, -2.0, shape)
+        elif leaf.endswith("A_log"):
+            x = rng.uniform(-1.0, 2.0, shape)
+        elif leaf.endswith("lam"):
+            x = rng.uniform(-5.0, 0.0, shape)
+        elif leaf.endswith(".D"):
+            x = rng.standard_normal(shape)
+        elif leaf.endswith("conv"):
+            x = rng.standard_normal(shape) / np.sqrt(shape[1])
+        elif leaf.endswith(".b"):
+            x = 0.3 * rng.standard_normal(shape)
+        else:
+            x = rng.standard_normal(shape) / np.sqrt(shape[-1])
+        w[name] = M.from_bf16(M.to_bf16(x))
+    return w
+
+
+def write(folder, cfg, weights):
+    os.makedirs(folder, exist_ok=True)
+    with open(os.path.join(folder, "config.json"), "w") as f:
+        json.dump(cfg, f)
+    M.write_safetensors(os.path.join(folder, "model.safetensors"), {k: ("BF16", M.to_bf16(v)) for k, v in weights.items()})
+    return str(folder)
+
+
+def reference_logits(cfg, weights, tokens):
+    return R.forward(tokens, {k: v.astype(np.float64) for k, v in weights.items()}, cfg)
+
+
+def error(got, want):
+    """Root mean square over the vocabulary of the mean-free difference, relative to the spread of the logits, per row."""
+    d = np.asarray(got, dtype=np.float64) - want
+    d -= d.mean(axis=1, keepdims=True)
+    return np.sqrt((d * d).mean(axis=1)) / want.std()

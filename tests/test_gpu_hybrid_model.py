@@ -1,0 +1,205 @@
+"""Whole models of the hybrid design through the framework's step function, scheduler and command line, against the plain
+implementation in hybrid_reference.py. Sizes are deliberately uneven; none needs to be a multiple of anything."""
+import json
+import os
+import subprocess
+
+import numpy as np
+import pytest
+
+import hybrid_models as H
+from ingot_b200 import models as M
+
+pytestmark = pytest.mark.gpu
+ROOT = os.path.dirname(os.path.dirname(os.path.abspath(__file__)))
+
+CONFIGS = {
+    # widths that need padding everywhere, a chunk that is no multiple of a page, two attention layers with different chunks
+    "odd": H.config([H.mamba(44, 10, 6, 3), H.parallel(6, 2, 20, 37, 36, 3, 4, ff=52), H.mamba(44, 10, 6, 3, ff=28),
+                     H.parallel(4, 4, 16, 64, 50, 5, 2)], vocab=101, width=42),
+    # one KV head, long chunk, wide state, two-tap convolution, several mixers of one kind in a row
+    "wide": H.config([H.parallel(8, 1, 64, 200, 128, 2, 4, ff=192), H.mamba(256, 40, 16, 4), H.mamba(256, 40, 16, 4)], vocab=160, width=256),
+    # single block, single-tap and many-tap convolutions, chunk of one page, state of one
+    "edge": H.config([H.parallel(3, 3, 8, 16, 16, 1, 1, left_scale=1.0, right_scale=1.0, scale=1.0), H.mamba(32, 1, 1, 6), H.parallel(2, 1, 80, 5, 64, 8, 3, ff=8)],
+                     vocab=50, width=64),
+}
+TOL = {True: 3e-5, False: 4e-2}
+
+
+@pytest.fixture(scope="module", params=CONFIGS)
+def case(request, tmp_path_factory):
+    cfg = CONFIGS[request.param]
+    w = H.random_weights(cfg, seed=len(request.param))
+    folder = H.write(tmp_path_factory.mktemp(request.param), cfg, w)
+    rng = np.random.default_rng(9)
+    tokens = [rng.integers(0, cfg["vocab"], n).tolist() for n in (231, 90, 41, 3, 130)]
+    want = [H.reference_logits(cfg, w, t) for t in tokens]
+    return cfg, folder, tokens, want
+
+
+def feed(model, seq, tokens, cuts, start=0):
+    """Runs one sequence alone in portions (cut lengths repeated), every logit wanted."""
+    out, at, k = [], start, 0
+    while at < len(tokens):
+        n = min(cuts[k % len(cuts)], len(tokens) - at)
+        out.append(model.step([(seq, at, tokens[at:at + n], list(range(n)))]))
+        at += n
+        k += 1
+    return np.concatenate(out)
+
+
+@pytest.mark.parametrize("f32", [True, False])
+def test_whole_prompts(case, f32):
+    cfg, folder, tokens, want = case
+    with M.Model(folder, f32=f32, max_tokens=512) as m:
+        for t, w in zip(tokens, want):
+            got = m.step([(0, 0, t, list(range(len(t))))])
+            assert H.error(got, w).max() < TOL[f32]
+
+
+@pytest.mark.parametrize("f32", [True, False])
+@pytest.mark.parametrize("cuts", [[1], [2], [64, 2, 17, 3, 33], [16], [100]], ids=str)
+def test_portions_and_token_by_token(case, f32, cuts):
+    cfg, folder, tokens, want = case
+    with M.Model(folder, f32=f32, max_tokens=512) as m:
+        for t, w in ((tokens[0], want[0]), (tokens[3], want[3])):  # both on slot 0: state and pages of the first are used again
+            got = feed(m, 0, t, cuts)
+            m.release(0)
+            assert H.error(got, w).max() < TOL[f32]
+
+
+@pytest.mark.parametrize("f32", [True, False])
+def test_mixed_batches_equal_each_sequence_alone(case, f32):
+    """Unequal sequences in one batch - portions beside single tokens, sequences that pause, end and give their slot and pages to
+    the next - in a pool that only just holds the live ones."""
+    cfg, folder, tokens, want = case
+    rng = np.random.default_rng(3)
+    with M.Model(folder, f32=f32, max_tokens=64 * 9, max_seqs=3) as m:
+        waiting, live, got = list(range(5)) + [1, 3], {}, {}
+        held = lambda n: (len(tokens[n]) + 63) // 64 * 64
+        run = 0
+        while waiting or live:
+            while waiting and len(live) < 3 and held(waiting[0]) + sum(held(v[0]) for v in live.values()) <= 64 * 9:
+                slot = next(s for s in (2, 0, 1) if s not in live)
+                live[slot] = [waiting.pop(0), 0, run]
+                got[run] = []
+                run += 1
+            step = []
+            for s, (i, at, _) in live.items():
+                if len(live) > 1 and rng.random() < 0.2:
+                    continue  # pauses
+                n = min(int(rng.choice([1, 1, 2, 5, 23, 64])), len(tokens[i]) - at)
+                step.append((s, at, tokens[i][at:at + n], list(range(n))))
+            if not step:
+                continue
+            rows = m.step(step)
+            r = 0
+            for s, at, t, _ in step:
+                got[live[s][2]].append(rows[r:r + len(t)])
+                r += len(t)
+                live[s][1] += len(t)
+                if live[s][1] == len(tokens[live[s][0]]):
+                    m.release(s)
+                    del live[s]
+        for k, i in enumerate(list(range(5)) + [1, 3]):
+            assert H.error(np.concatenate(got[k]), want[i]).max() < TOL[f32]
+
+
+def test_the_batch_does_not_change_a_sequence(case):
+    """Single tokens of three sequences in one batch against the same tokens alone: equal up to summation order."""
+    cfg, folder, tokens, _ = case
+    with M.Model(folder, max_tokens=1024, max_seqs=4) as m:
+        for s in range(3):
+            m.step([(s, 0, tokens[s][:30], [])])
+        together = [m.step([(s, 30 + k, tokens[s][30 + k:31 + k], [0]) for s in range(3)]) for k in range(8)]
+        for s in range(3):
+            m.release(s)
+        for s in range(3):
+            m.step([(3, 0, tokens[s][:30], [])])
+            for k in range(8):
+                alone = m.step([(3, 30 + k, tokens[s][30 + k:31 + k], [0])])
+                assert H.error(alone, together[k][s:s + 1].astype(np.float64)).max() < 1e-4
+            m.release(3)
+
+
+def test_long_decoding(case):
+    """Hundreds of decoded tokens after a short prompt, across many chunk and page borders (the replayed decode graph)."""
+    cfg, folder, _, _ = case
+    rng = np.random.default_rng(17)
+    t = rng.integers(0, cfg["vocab"], 420).tolist()
+    w = H.random_weights(cfg, seed=[len(k) for k, v in CONFIGS.items() if v is cfg][0])
+    want = H.reference_logits(cfg, w, t)
+    for f32 in (True, False):
+        with M.Model(folder, f32=f32, max_tokens=448, max_seqs=2) as m:
+            first = m.step([(1, 0, t[:9], list(range(9)))])
+            rest = [m.step([(1, p, t[p:p + 1], [0])]) for p in range(9, len(t))]
+            assert H.error(np.concatenate([first] + rest), want).max() < TOL[f32]
+
+
+def test_greedy_generation_through_the_scheduler(case):
+    """Requests that arrive at different times share the steps; in 32-bit every reply is the plain implementation's."""
+    cfg, folder, tokens, _ = case
+    w = H.random_weights(cfg, seed=[len(k) for k, v in CONFIGS.items() if v is cfg][0])
+    prompts = [tokens[1][:40], tokens[2], tokens[3], tokens[4][:71]]
+    new = [10, 6, 12, 8]
+    want = []
+    for p, n in zip(prompts, new):
+        ids = list(p)
+        for _ in range(n):
+            ids.append(int(np.argmax(H.reference_logits(cfg, w, ids)[-1])))
+        want.append(ids[len(p):])
+    with M.Model(folder, f32=True, max_tokens=512, max_seqs=2, max_step_tokens=48) as m:
+        got, steps, rows = m.generate(prompts, new, arrival=[0, 0, 1, 4])
+        assert got == want
+        assert rows == sum(len(p) + n - 1 for p, n in zip(prompts, new)) and steps < rows
+        # sampling is seeded per request
+        a = m.generate(prompts[:2], 8, sampling=[0.8, 20, 0.9, 1.1, 32, 7])[0]
+        b = m.generate(prompts[:2], 8, sampling=[0.8, 20, 0.9, 1.1, 32, 7])[0]
+        assert a == b
+        # a stop token ends a reply and is not part of it
+        stop = want[0][3]
+        cut = m.generate([prompts[0]], 10, stop_token=stop)[0][0]
+        assert cut == want[0][:want[0].index(stop)]
+    cmd = [os.path.join(ROOT, "bin", "ingot_models"), "generate", "--model", folder, "--dtype", "float32", "--max-new", "6", "--max-tokens", "512"]
+    for p in prompts[:2]:
+        cmd += ["--prompt-ids", ",".join(map(str, p))]
+    out = subprocess.run(cmd, capture_output=True, text=True, timeout=1200, check=True).stdout.strip().splitlines()
+    assert [[int(x) for x in line.split("#")[0].split(",")] for line in out] == [want[0][:6], want[1][:6]]
+
+
+def test_trace_replay(case, tmp_path):
+    cfg, folder, tokens, want = case
+    steps = [{"step": 0, "entries": [{"id": "a", "tokens": tokens[1][:50], "want": [3, 49]}], "end": []},
+             {"step": 1, "entries": [{"id": "a", "tokens": tokens[1][50:], "want": []}, {"id": "b", "tokens": tokens[2][:1], "want": [0]}], "end": ["a"]},
+             {"step": 2, "entries": [{"id": "c", "tokens": tokens[3], "want": [2]}, {"id": "b", "tokens": tokens[2][1:], "want": [0, 39]}], "end": ["b", "c"]}]
+    r = subprocess.run([os.path.join(ROOT, "bin", "trace_run"), "--model", folder, "--dtype", "float32", "--out", str(tmp_path), "--max-tokens", "192"],
+                       input="".join(json.dumps(s) + "\n" for s in steps), capture_output=True, text=True, timeout=1200)
+    assert r.returncode == 0, r.stderr
+    assert r.stdout.split("\n")[:3] == ["done 0", "done 1", "done 2"]
+    rows = lambda n: np.fromfile(tmp_path / f"{n}.f32", "<f4").reshape(-1, cfg["vocab"])
+    assert H.error(rows(0), want[1][[3, 49]]).max() < TOL[True]
+    assert H.error(rows(1), want[2][[0]]).max() < TOL[True]
+    assert H.error(rows(2), np.concatenate([want[3][[2]], want[2][[1, 40]]])).max() < TOL[True]
+
+
+def test_refusals(case, tmp_path):
+    cfg, folder, tokens, _ = case
+    with M.Model(folder, max_tokens=128, max_seqs=2) as m:
+        bad = [([(0, 0, [cfg["vocab"]], [0])], "token id"), ([(2, 0, [1], [0])], "sequence id"), ([(0, 0, [1], [0]), (0, 1, [1], [0])], "twice"),
+               ([(0, 5, [1], [0])], "continue"), ([(0, 0, [1] * 129, [])], "context window"), ([(0, 0, [1, 2], [2])], "wanted place")]
+        for step, text in bad:
+            with pytest.raises(M.ModelError, match=text):
+                m.step(step)
+        m.step([(0, 0, [1, 2, 3], [2])])  # still in working order
+    w = H.random_weights(cfg)
+    broken = json.loads(json.dumps(cfg))
+    broken["layers"][0]["type"] = "nothing"
+    with pytest.raises(M.ModelError, match="unknown layer type"):
+        M.Model(H.write(tmp_path / "a", broken, w))
+    broken = json.loads(json.dumps(cfg))
+    broken["width"] += 1
+    with pytest.raises(M.ModelError, match="shape"):
+        M.Model(H.write(tmp_path / "b", broken, w))
+    del w["final.norm"]
+    with pytest.raises(M.ModelError, match="final.norm is missing"):
+        M.Model(H.write(tmp_path / "c", cfg, w))
