@@ -336,7 +336,7 @@ int ingot_gated_lru(const ingot_step* step, const ingot_scan_plan* plan, const f
  * projection normalised over all KV heads), paged in 16-position blocks, with causal or chunk-local visibility.
  * chunk > 0: position i sees j <= i of its own run of `chunk` positions counted from position 0; page of position p =
  * (p / chunk) * ceil(chunk / 16) + (p % chunk) / 16. chunk 0: plain causal, page p / 16. Rows [page][n_head_kv][16][head_dim]
- * f32 or f16 (head_dim even, <= 512, zero-padded heads allowed). Allocates on the current device; synchronous. */
+ * f32 or f16 (head_dim a multiple of 4, <= 512, zero-padded heads allowed). Allocates on the current device; synchronous. */
 typedef struct ingot_skv ingot_skv;
 int ingot_skv_create(ingot_skv** out, int n_layer, int n_head_kv, int head_dim, int dtype, int chunk, int n_blocks);
 void ingot_skv_destroy(ingot_skv* kv);
@@ -357,7 +357,8 @@ int ingot_skv_append(ingot_skv* kv, int layer, const ingot_step* step, const flo
                      int n_head, int head_size, const float* q_norm_dev, const float* k_norm_dev, float eps, void* q_out_dev,
                      const int32_t* tables_dev, const int32_t* first_page_dev, int max_blocks, void* stream);
 /* Softmax over the visible keys of every row (appended before), scores = q . k_row / rms(k) * scale; out[t][h * out_dim + d] =
- * out_scale * result for d < out_dim. impl: 0 = library's choice, 1 = the plain f32-arithmetic kernel. */
+ * out_scale * result for d < out_dim. impl: 0 = library's choice (tensor cores for f16 rows of the lengths
+ * ingot_skv_row_length returns up to 256), 1 = the plain f32-arithmetic kernel. */
 int ingot_skv_attend(ingot_skv* kv, int layer, const ingot_step* step, const void* q_dev, int n_head, int out_dim, float scale,
                      float out_scale, const ingot_act_out* out, const int32_t* tables_dev, const int32_t* first_page_dev, int max_blocks, int impl, void* stream);
 

@@ -6,11 +6,11 @@
 //                   here plus a line in make_mixer().
 //   LayerOps        what every mixer is written in: projections (with the RMS norm of their input or the residual add of
 //                   their output folded in), scratch activations, weight upload. It picks the kernel by the number of
-//                   tokens: weight-streaming GEMV for one token, f32 kernels for a few, tcgen05 GEMM from 16 on.
+//                   tokens: weight-streaming GEMV for one token, tcgen05 GEMM for more (f32 kernels in the 32-bit form).
 //   HybridBackend   the step: one ragged batch of portions of several sequences, state slots and cache pages, logits.
 //
 // Precision. Weights are bf16. In the 16-bit form the tensor-core products take bf16 activations (a hi + lo pair where the
-// product feeds a recurrence's gates or step sizes) and accumulate in f32; everything between products - residual stream,
+// product feeds a recurrence's gates or step sizes, and in small batches) and accumulate in f32; everything between products - residual stream,
 // norms, scores and softmax, gates, recurrent states - is f32, and single tokens multiply f32 activations. In the f32 form
 // every product is f32 FMA on widened weights and the attention cache is f32.
 //
@@ -52,17 +52,22 @@ void ingot_linear_ws_planes(ingot_linear_ws* ws, void** hi, void** lo);
 cudaError_t ingot_linear_tc_prepared(ingot_linear_ws* ws, int n_in, int n_tok, int planes);
 cudaError_t ingot_linear_tc_prepare_bf16(ingot_linear_ws* ws, const float* x, int x_ld, int n_in, int n_tok, int planes, cudaStream_t s);
 cudaError_t ingot_linear_tc_prepare_norm_bf16(ingot_linear_ws* ws, const float* x, const float* norm_w, float eps, int n_in, int n_mean, int n_tok,
-                                              cudaStream_t s);
+                                              int planes, cudaStream_t s);
 cudaError_t ingot_linear_tc_run(ingot_linear_ws* ws, float* out, const void* w, int n_in, int n_out, int accumulate, cudaStream_t s);
 cudaError_t ingot_linear_tc_run_blocks(ingot_linear_ws* ws, float* out, const void* w, int k_block, int n_out, int rows_per_block, cudaStream_t s);
 cudaError_t ingot_linear_tc_run_partial(ingot_linear_ws* ws, const void* w, int n_in, int n_out, int slot, cudaStream_t s);
-cudaError_t ingot_linear_tc_finish_residual_norm_bf16(ingot_linear_ws* ws, float* x, const float* norm_w, float eps, int n_mean, cudaStream_t s);
-cudaError_t ingot_linear_tc_finish_gated_bf16(ingot_linear_ws* ws, int act, cudaStream_t s);
+cudaError_t ingot_linear_tc_finish_residual_norm_bf16(ingot_linear_ws* ws, float* x, const float* norm_w, float eps, int n_mean, int planes,
+                                                      cudaStream_t s);
+cudaError_t ingot_linear_tc_finish_gated_bf16(ingot_linear_ws* ws, int act, int planes, cudaStream_t s);
 }
 
 namespace {
 
-constexpr int kMinTcTokens = 16;  // fewest tokens the tensor-core GEMM takes
+constexpr int kMinTcTokens = 2;  // from two tokens on, a 128-token tile that is mostly padding still only streams the weights once
+
+// Up to this many tokens a product is bound by streaming the weights, so the activations go in as a hi + lo pair at no cost: a
+// decoded token's logits then hardly depend on whether it is alone (f32 activations) or in a batch.
+constexpr int kPairTokens = 64;
 
 int round_up(int v, int q) { return (v + q - 1) / q * q; }
 
@@ -102,7 +107,8 @@ enum Buf { kProj, kConv, kStateIn, kDt, kGates, kMix, kGateUp, kMid, kNormed, kQ
 struct StepCtx {
     ingot_step st = {};
     ingot_scan_plan scan = {}, lru = {};
-    bool tc = false;  // products on the tensor cores (16-bit form, enough tokens)
+    bool tc = false;  // products on the tensor cores (16-bit form, more than one token)
+    int planes = 1;   // bf16 planes an activation is given as there
 };
 
 // Shared-row attention caches of equal shape live in one handle with one page pool.
@@ -191,18 +197,18 @@ public:
     // ---- the step ----
     float* buf(Buf b) const { return bufs_[b]; }
     // Output of a kernel that feeds a product: the operand planes on the tensor-core path (and f32 rows if `keep`), else f32.
-    ingot_act_out operand(const StepCtx& s, float* f32, int ld, bool keep, int planes = 1) const {
+    ingot_act_out operand(const StepCtx& s, float* f32, int ld, bool keep, int planes = 0) const {
         ingot_act_out o = {};
         o.ld = ld;
         if (!s.tc || keep) o.f32 = f32;
         if (s.tc) {
             ingot_linear_ws_planes(ws, &o.hi, &o.lo);
-            if (planes < 2) o.lo = nullptr;
+            if (std::max(planes, s.planes) < 2) o.lo = nullptr;
         }
         return o;
     }
-    void operand_ready(const StepCtx& s, int n_in, int planes = 1) const {
-        if (s.tc) cuda_check(ingot_linear_tc_prepared(ws, n_in, s.st.n_tok, planes), "operand");
+    void operand_ready(const StepCtx& s, int n_in, int planes = 0) const {
+        if (s.tc) cuda_check(ingot_linear_tc_prepared(ws, n_in, s.st.n_tok, std::max(planes, s.planes)), "operand");
     }
     static bool streams(const Matrix& w) { return w.n_in % 256 == 0 && w.n_in <= 12032 && w.rows_per_block == 0; }
 
@@ -239,7 +245,7 @@ public:
         norm_ready_ = nullptr;
         if (s.tc) {
             cuda_check(ingot_linear_tc_run_partial(ws, w.data, w.n_in, w.n_out, 0, stream), "output projection");
-            cuda_check(ingot_linear_tc_finish_residual_norm_bf16(ws, x, next_norm, eps, width, stream), "residual");
+            cuda_check(ingot_linear_tc_finish_residual_norm_bf16(ws, x, next_norm, eps, width, s.planes, stream), "residual");
             norm_ready_ = next_norm;
         } else if (s.st.n_tok == 1 && streams(w)) {
             cuda_check(ingot_support_gemv_bf16(x, w.data, w.n_out, w.n_in, in, nullptr, 0.f, w.n_in, 0, 0, 1, stream), "output projection");
@@ -253,7 +259,7 @@ public:
         if (s.tc) {
             prepare_norm(s, w, norm);
             cuda_check(ingot_linear_tc_run_partial(ws, w.data, w.n_in, w.n_out, 0, stream), "gate / up");
-            cuda_check(ingot_linear_tc_finish_gated_bf16(ws, 1, stream), "gate");
+            cuda_check(ingot_linear_tc_finish_gated_bf16(ws, 1, s.planes, stream), "gate");
         } else if (s.st.n_tok == 1 && streams(w)) {
             cuda_check(ingot_support_gemv_bf16(buf(kMid), w.data, ff, w.n_in, x, norm, eps, width, 1, 1, 0, stream), "gate / up");
         } else {
@@ -291,7 +297,7 @@ private:
     }
     void prepare_norm(const StepCtx& s, const Matrix& w, const float* norm) {
         if (norm_ready_ == norm && norm) return;  // the kernel that finished x already normalised it for this product
-        cuda_check(ingot_linear_tc_prepare_norm_bf16(ws, x, norm, eps, w.n_in, width, s.st.n_tok, stream), "rmsnorm");
+        cuda_check(ingot_linear_tc_prepare_norm_bf16(ws, x, norm, eps, w.n_in, width, s.st.n_tok, s.planes, stream), "rmsnorm");
     }
     WeightStreamer loader_;
     std::vector<void*> allocs_;
@@ -464,6 +470,7 @@ public:
         ingot_act_out right = left;
         if (right.f32) right.f32 += attn_cols_;
         if (right.hi) right.hi = static_cast<char*>(right.hi) + size_t(attn_cols_) * 2;
+        if (right.lo) right.lo = static_cast<char*>(right.lo) + size_t(attn_cols_) * 2;
         ingot_check(ingot_gated_lru(&s.st, &s.lru, u, wp_, gates, 2 * wp_, block_, r_b_, i_b_, softplus_lam_, proj + y_off_, proj_ld_, y_b_, state_, wp_,
                                     right_scale_, &right, ops.stream));
         ops.operand_ready(s, mix_ld_);
@@ -719,9 +726,10 @@ private:
             }
     }
 
+    // INGOT_SCAN_THREADS: threads per SM the chunks of a recurrence aim for (tuning).
     // Length of the time chunks of a recurrence one token-chunk of which occupies `threads` threads: as few chunks as fill the GPU.
     int chunk_tokens(int n_tok, int threads) const {
-        const int chunks = std::max(1, num_sms_ * 1024 / std::max(threads, 1));
+        const int chunks = std::max(1, num_sms_ * scan_threads_per_sm_ / std::max(threads, 1));
         return std::max(32, round_up((n_tok + chunks - 1) / chunks, 16));
     }
 
@@ -837,6 +845,7 @@ private:
             ops_.caches[i]->tables = meta_dev_ + table_at[i].second;
         }
         s.tc = ops_.ws != nullptr && step.n_tok >= kMinTcTokens;
+        s.planes = s.tc && step.n_tok <= kPairTokens ? 2 : 1;
         return s;
     }
 
@@ -882,7 +891,7 @@ private:
         }
         cuda_check(ingot_support_rmsnorm_rows(ops_.buf(kNormed), ops_.x, final_norm_, step.want_rows, step.n_want, ld, ops_.width, ops_.eps, ops_.stream), "final norm");
         if (ops_.ws && step.n_want >= kMinTcTokens) {
-            cuda_check(ingot_linear_tc_prepare_bf16(ops_.ws, ops_.buf(kNormed), ld, ld, step.n_want, 1, ops_.stream), "final norm");
+            cuda_check(ingot_linear_tc_prepare_bf16(ops_.ws, ops_.buf(kNormed), ld, ld, step.n_want, step.n_want <= kPairTokens ? 2 : 1, ops_.stream), "final norm");
             cuda_check(ingot_linear_tc_run(ops_.ws, logits_dev_, head_.data, head_.n_in, head_.n_out, 0, ops_.stream), "logits");
         } else {
             cuda_check(ingot_support_linear_bf16(logits_dev_, head_.data, ops_.buf(kNormed), ld, ld, head_.n_out, 0, step.n_want, 0, ops_.stream), "logits");
@@ -918,6 +927,7 @@ private:
     int* status_host_ = nullptr;
     std::map<int, Graph> graphs_;      // by batch size
     const bool use_graphs_ = !(getenv("INGOT_DECODE_GRAPH") && atoi(getenv("INGOT_DECODE_GRAPH")) == 0);
+    const int scan_threads_per_sm_ = getenv("INGOT_SCAN_THREADS") ? std::max(1, atoi(getenv("INGOT_SCAN_THREADS"))) : 1024;
     std::vector<float>* tap_ = nullptr;
     cudaEvent_t ev0_ = nullptr, ev1_ = nullptr;
     float last_ms_ = 0.f;

@@ -40,26 +40,22 @@ namespace {
 
 using namespace ingot_sm100;
 
-#ifndef INGOT_GEMM_BN
-#define INGOT_GEMM_BN 128
-#endif
-constexpr int kBM = 128, kBN = INGOT_GEMM_BN, kBK = 64;  // outputs per CTA: 128, or 256 (a third less L2 traffic per output)
-static_assert(kBN == 128 || kBN == 256, "128 or 256 outputs per CTA");
+constexpr int kBM = 128, kBK = 64;  // outputs per CTA (kBN): 128, or 256 (a quarter less L2 traffic per output with one plane)
+constexpr int kGroupM = 16;         // token tiles that sweep the weight matrix together (see the tile order in the kernel)
 constexpr int kMaxStages = 6;
 constexpr int kBoxBytes = 128 * kBK * 2;        // 16 KB: 128 rows x 64 f16
-constexpr int kWBytes = kBN * kBK * 2;          // the W box: kBN rows
 constexpr int kThreads = 192;
-template <int kPlanes>
+template <int kPlanes, int kBN>
 struct Ring {
+    static constexpr int kWBytes = kBN * kBK * 2;                      // the W box: kBN rows
     static constexpr int kStageBytes = kPlanes * kBoxBytes + kWBytes;  // hi(, lo), W
     static constexpr int kStages = 196608 / kStageBytes;               // 192 KB ring: 4 stages of 48 KB or 6 of 32 KB
     static constexpr int kOffBar = kStages * kStageBytes;
     static constexpr int kSmemBytes = kOffBar + 256 + 1024;            // barriers + alignment slack
     static_assert(kStages <= kMaxStages, "barrier arrays");
 };
-constexpr uint32_t kTmemCols = kBN;
-constexpr uint32_t kIdescF16 = (1u << 4) | ((uint32_t)(kBN >> 3) << 17) | ((uint32_t)(kBM >> 4) << 24);  // f16 x f16 -> f32, both K-major
-constexpr uint32_t kIdescBF16 = kIdescF16 | (1u << 7) | (1u << 10);                                        // bf16 x bf16 -> f32
+constexpr uint32_t idesc_f16(int kBN) { return (1u << 4) | ((uint32_t)(kBN >> 3) << 17) | ((uint32_t)(kBM >> 4) << 24); }  // f16 x f16 -> f32, both K-major
+constexpr uint32_t kIdescBF16 = (1u << 7) | (1u << 10);  // bf16 x bf16 -> f32
 constexpr unsigned long long kWaitLimitNs = 2000000000ull;
 
 __device__ __forceinline__ uint32_t smem_u32(const void* p) { return (uint32_t)__cvta_generic_to_shared(p); }
@@ -94,24 +90,27 @@ struct Bars {
 };
 
 // One launch covers up to three weight matrices that read the same activations (q/k/v, gate/up): grid.x runs over
-// the output tiles of all of them, tile_end[m] being the running total of tiles up to and including matrix m.
+// the token tiles and the output tiles of all of them, tile_end[m] being the running total of tiles up to and including matrix m.
 struct GemmParams {
     float* out;           // [n_tok][n_out] (single matrix only)
     float* partial[3];    // per matrix: [n_split][n_tok][n_out] when n_split > 1 or to_partial
     int* status;
     int n_tok, k_steps, n_split, accumulate;
     int n_out[3], tile_end[3];
+    int tiles_n, tiles_m;
     uint32_t idesc;
     int rows_per_block, k_block, tiles_per_block;  // block-diagonal matrix (rows_per_block > 0, count == 1)
     int to_partial;  // write the slice(s) to `partial` even when there is only one (a consumer kernel sums them)
 };
 
-template <int kPlanes>
+template <int kPlanes, int kBN>
 __global__ void __launch_bounds__(kThreads, 1)
 linear_sm100_kernel(const __grid_constant__ CUtensorMap map_hi, const __grid_constant__ CUtensorMap map_lo,
                     const __grid_constant__ CUtensorMap map_w0, const __grid_constant__ CUtensorMap map_w1,
                     const __grid_constant__ CUtensorMap map_w2, const GemmParams p) {
-    constexpr int kStages = Ring<kPlanes>::kStages, kStageBytes = Ring<kPlanes>::kStageBytes, kOffBar = Ring<kPlanes>::kOffBar;
+    using R = Ring<kPlanes, kBN>;
+    constexpr int kStages = R::kStages, kStageBytes = R::kStageBytes, kOffBar = R::kOffBar;
+    constexpr uint32_t kTmemCols = kBN;
     constexpr int kOffW = kPlanes * kBoxBytes;
     extern __shared__ unsigned char smem_dyn[];
     LINEAR_PDL_TRIGGER();
@@ -121,16 +120,21 @@ linear_sm100_kernel(const __grid_constant__ CUtensorMap map_hi, const __grid_con
     volatile uint32_t* abort_flag = &bars->abort_flag;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int warp_u = __shfl_sync(0xffffffffu, warp, 0);
-    const int mat = ((int)blockIdx.x >= p.tile_end[0]) + ((int)blockIdx.x >= p.tile_end[1]);  // warp-uniform
+    // Tile order: kGroupM token tiles walk the output tiles together, so that CTAs that run at the same time share weight
+    // boxes and the weight matrix comes out of HBM once per kGroupM * 128 tokens instead of once per 128.
+    const int group_tiles = kGroupM * p.tiles_n, grp = (int)blockIdx.x / group_tiles, in_grp = (int)blockIdx.x - grp * group_tiles;
+    const int group_m = min(kGroupM, p.tiles_m - grp * kGroupM);
+    const int tile_n = in_grp / group_m, tile_m = grp * kGroupM + in_grp - tile_n * group_m;
+    const int mat = (tile_n >= p.tile_end[0]) + (tile_n >= p.tile_end[1]);  // warp-uniform
     const CUtensorMap* const map_w_p = mat == 0 ? &map_w0 : mat == 1 ? &map_w1 : &map_w2;
     const int mat_n_out = mat == 0 ? p.n_out[0] : mat == 1 ? p.n_out[1] : p.n_out[2];
-    const int blk = p.tiles_per_block > 0 ? (int)blockIdx.x / p.tiles_per_block : 0;
+    const int blk = p.tiles_per_block > 0 ? tile_n / p.tiles_per_block : 0;
     const int col_end = p.tiles_per_block > 0 ? (blk + 1) * p.rows_per_block : mat_n_out;
     const int a_k0 = blk * p.k_block;  // first activation column of this tile's products
     float* const mat_partial = mat == 0 ? p.partial[0] : mat == 1 ? p.partial[1] : p.partial[2];
-    const int n0 = p.tiles_per_block > 0 ? blk * p.rows_per_block + ((int)blockIdx.x - blk * p.tiles_per_block) * kBN
-                                         : ((int)blockIdx.x - (mat == 0 ? 0 : mat == 1 ? p.tile_end[0] : p.tile_end[1])) * kBN;
-    const int m0 = blockIdx.y * kBM, split = blockIdx.z;
+    const int n0 = p.tiles_per_block > 0 ? blk * p.rows_per_block + (tile_n - blk * p.tiles_per_block) * kBN
+                                         : (tile_n - (mat == 0 ? 0 : mat == 1 ? p.tile_end[0] : p.tile_end[1])) * kBN;
+    const int m0 = tile_m * kBM, split = blockIdx.z;
     const int ks_begin = (int)((long long)p.k_steps * split / p.n_split);
     const int ks_end = (int)((long long)p.k_steps * (split + 1) / p.n_split);
     const int n_it = ks_end - ks_begin;
@@ -425,9 +429,10 @@ __global__ void finish_swiglu_kernel(__half* hi, __half* lo, const Slices gate, 
     store_split4<kActF16Pair>(hi, lo, i, f);
 }
 
-// One bf16 plane of act(gate) * up, where one product of width 2 n holds both: gate = columns 0..n-1, up = columns n..2n-1.
+// One or two bf16 planes of act(gate) * up, where one product of width 2 n holds both: gate = columns 0..n-1, up = columns n..2n-1.
 // act: 0 silu, 1 the tanh form of gelu. grid.y = row.
-__global__ void finish_gated_kernel(__half* hi, const Slices in, int n, size_t slice, int act) {
+template <int kAct>
+__global__ void finish_gated_kernel(__half* hi, __half* lo, const Slices in, int n, size_t slice, int act) {
     LINEAR_PDL_TRIGGER();
     LINEAR_PDL_WAIT();
     const int i = (blockIdx.x * blockDim.x + threadIdx.x) * 4;
@@ -442,7 +447,7 @@ __global__ void finish_gated_kernel(__half* hi, const Slices in, int n, size_t s
         const float t = gv[e];
         f[e] = (act == 0 ? t / (1.0f + expf(-t)) : 0.5f * t * (1.0f + tanhf(0.7978845608028654f * (t + 0.044715f * t * t * t)))) * uv[e];
     }
-    store_split4<kActBF16>(hi, nullptr, (size_t)blockIdx.y * n + i, f);
+    store_split4<kAct>(hi, lo, (size_t)blockIdx.y * n + i, f);
 }
 
 typedef CUresult (*EncodeTiledFn)(CUtensorMap*, CUtensorMapDataType, cuuint32_t, void*, const cuuint64_t*, const cuuint64_t*,
@@ -490,7 +495,7 @@ struct ingot_linear_ws {
     int planes = 2;                            // of the prepared activations
     int prepared_tok = 0, prepared_in = 0;
     CUtensorMap map_hi, map_lo;
-    std::map<std::tuple<const void*, int, int>, CUtensorMap> w_maps;  // one per weight matrix
+    std::map<std::tuple<const void*, int, int, int>, CUtensorMap> w_maps;  // one per weight matrix
 };
 
 // (Re)builds the activation tensor maps when the prepared shape changes.
@@ -523,8 +528,9 @@ static cudaError_t ws_create(ingot_linear_ws** out, size_t act_elems, size_t par
         (e = cudaMemset(ws->hi, 0, ws->act_elems * 2)) != cudaSuccess || (e = cudaMemset(ws->lo, 0, ws->act_elems * 2)) != cudaSuccess ||
         (e = cudaMalloc(&ws->partial, n_slots * ws->partial_floats * 4)) != cudaSuccess || (e = cudaMalloc(&ws->status, sizeof(int))) != cudaSuccess ||
         (e = cudaMemset(ws->status, 0, sizeof(int))) != cudaSuccess ||
-        (e = cudaFuncSetAttribute(linear_sm100_kernel<2>, cudaFuncAttributeMaxDynamicSharedMemorySize, Ring<2>::kSmemBytes)) != cudaSuccess ||
-        (e = cudaFuncSetAttribute(linear_sm100_kernel<1>, cudaFuncAttributeMaxDynamicSharedMemorySize, Ring<1>::kSmemBytes)) != cudaSuccess) {
+        (e = cudaFuncSetAttribute(linear_sm100_kernel<2, 128>, cudaFuncAttributeMaxDynamicSharedMemorySize, Ring<2, 128>::kSmemBytes)) != cudaSuccess ||
+        (e = cudaFuncSetAttribute(linear_sm100_kernel<1, 128>, cudaFuncAttributeMaxDynamicSharedMemorySize, Ring<1, 128>::kSmemBytes)) != cudaSuccess ||
+        (e = cudaFuncSetAttribute(linear_sm100_kernel<1, 256>, cudaFuncAttributeMaxDynamicSharedMemorySize, Ring<1, 256>::kSmemBytes)) != cudaSuccess) {
         cudaFree(ws->hi); cudaFree(ws->lo); cudaFree(ws->partial); cudaFree(ws->status);
         delete ws;
         return e;
@@ -554,7 +560,7 @@ void ingot_linear_ws_destroy(ingot_linear_ws* ws) {
 
 // Whether a projection of this shape can take the tensor-core path.
 int ingot_linear_tc_supported(const ingot_linear_ws* ws, int w_is_f16, int n_in, int n_out, int n_tok) {
-    if (!ws || !encode_fn() || n_tok < 16 || n_out % 4 != 0 || (size_t)n_tok * n_in > ws->act_elems) return 0;
+    if (!ws || !encode_fn() || n_tok < (ws->bf16 ? 2 : 16) || n_out % 4 != 0 || (size_t)n_tok * n_in > ws->act_elems) return 0;
     return ws->bf16 ? n_in % 8 == 0 : w_is_f16 && n_in % kBK == 0;
 }
 
@@ -600,11 +606,13 @@ cudaError_t ingot_linear_tc_prepare_norm(ingot_linear_ws* ws, const float* x, co
     return set_prepared(ws, n_in, n_tok);
 }
 cudaError_t ingot_linear_tc_prepare_norm_bf16(ingot_linear_ws* ws, const float* x, const float* norm_w, float eps, int n_in, int n_mean, int n_tok,
-                                              cudaStream_t s) {
+                                              int planes, cudaStream_t s) {
     if (!act_shape_ok(ws, n_in, n_tok) || !ws->bf16) return cudaErrorInvalidValue;
-    cudaError_t le = launch_pdl(rmsnorm_split_kernel<kActBF16>, dim3(n_tok), dim3(256), 0, s, ws->hi, ws->lo, x, norm_w, n_in, n_mean, eps);
+    cudaError_t le = planes > 1
+        ? launch_pdl(rmsnorm_split_kernel<kActBF16Pair>, dim3(n_tok), dim3(256), 0, s, ws->hi, ws->lo, x, norm_w, n_in, n_mean, eps)
+        : launch_pdl(rmsnorm_split_kernel<kActBF16>, dim3(n_tok), dim3(256), 0, s, ws->hi, ws->lo, x, norm_w, n_in, n_mean, eps);
     if (le != cudaSuccess) return le;
-    ws->planes = 1;
+    ws->planes = planes > 1 ? 2 : 1;
     return set_prepared(ws, n_in, n_tok);
 }
 
@@ -628,9 +636,19 @@ static cudaError_t launch_gemm(ingot_linear_ws* ws, float* out, const void* cons
         if (ws->slot_split[first_slot + m] != held || ws->slot_out[first_slot + m] != n_out[m]) return cudaErrorInvalidValue;
     const CUtensorMap* maps[3] = {nullptr, nullptr, nullptr};
     GemmParams p = {};
+    const int tiles_m = (n_tok + kBM - 1) / kBM;
+    // 256 outputs per CTA where the operand traffic bounds the kernel (one plane, whole waves of tiles): a 256-wide tile takes
+    // about 1.5 times as long as a 128-wide one
+    int kBN = 128;
+    if (ws->planes == 1 && count == 1 && rows_per_block == 0) {
+        const long long waves128 = ((long long)((n_out[0] + 127) / 128) * tiles_m + ws->num_sms - 1) / ws->num_sms;
+        const long long waves256 = ((long long)((n_out[0] + 255) / 256) * tiles_m + ws->num_sms - 1) / ws->num_sms;
+        if (waves128 > 1 && 3 * waves256 < 2 * waves128) kBN = 256;
+        if (const char* e = getenv("INGOT_GEMM_BN")) kBN = atoi(e) == 256 ? 256 : 128;
+    }
     int tiles_n = 0, fit = 1 << 30;
     for (int m = 0; m < count; m++) {
-        const auto key = std::make_tuple(w[m], n_out[m], n_in);
+        const auto key = std::make_tuple(w[m], n_out[m], n_in, kBN);
         auto it = ws->w_maps.find(key);
         if (it == ws->w_maps.end()) {
             CUtensorMap tm;
@@ -645,7 +663,9 @@ static cudaError_t launch_gemm(ingot_linear_ws* ws, float* out, const void* cons
         fit = std::min(fit, (int)(ws->partial_floats / ((size_t)n_tok * n_out[m])) - held);
     }
     for (int m = count; m < 3; m++) { maps[m] = maps[count - 1]; p.tile_end[m] = tiles_n; p.n_out[m] = n_out[count - 1]; p.partial[m] = p.partial[count - 1]; }
-    const int tiles = tiles_n * ((n_tok + kBM - 1) / kBM);
+    const int tiles = tiles_n * tiles_m;
+    p.tiles_n = tiles_n;
+    p.tiles_m = tiles_m;
     const int k_steps = (n_in + kBK - 1) / kBK;
     // enough k slices to give every SM a CTA, at least 4 k-steps each, and no more than the slots hold
     if (to_partial && fit < 1) return cudaErrorInvalidValue;
@@ -653,14 +673,17 @@ static cudaError_t launch_gemm(ingot_linear_ws* ws, float* out, const void* cons
     p.out = out; p.status = ws->status;
     p.n_tok = n_tok; p.k_steps = k_steps; p.n_split = n_split; p.accumulate = accumulate;
     p.to_partial = to_partial ? 1 : 0;
-    p.idesc = ws->bf16 ? kIdescBF16 : kIdescF16;
+    p.idesc = idesc_f16(kBN) | (ws->bf16 ? kIdescBF16 : 0u);
     p.rows_per_block = rows_per_block;
     p.k_block = rows_per_block > 0 ? n_in : 0;
     p.tiles_per_block = rows_per_block > 0 ? (rows_per_block + kBN - 1) / kBN : 0;
-    dim3 grid(tiles_n, (n_tok + kBM - 1) / kBM, n_split);
-    cudaError_t le = ws->planes > 1
-        ? launch_pdl(linear_sm100_kernel<2>, grid, dim3(kThreads), (size_t)Ring<2>::kSmemBytes, s, ws->map_hi, ws->map_lo, *maps[0], *maps[1], *maps[2], p)
-        : launch_pdl(linear_sm100_kernel<1>, grid, dim3(kThreads), (size_t)Ring<1>::kSmemBytes, s, ws->map_hi, ws->map_lo, *maps[0], *maps[1], *maps[2], p);
+    dim3 grid(tiles, 1, n_split);
+    auto run = [&](auto kernel, int smem) {
+        return launch_pdl(kernel, grid, dim3(kThreads), (size_t)smem, s, ws->map_hi, ws->map_lo, *maps[0], *maps[1], *maps[2], p);
+    };
+    cudaError_t le = ws->planes > 1 ? run(linear_sm100_kernel<2, 128>, Ring<2, 128>::kSmemBytes)
+                   : kBN == 256     ? run(linear_sm100_kernel<1, 256>, Ring<1, 256>::kSmemBytes)
+                                    : run(linear_sm100_kernel<1, 128>, Ring<1, 128>::kSmemBytes);
     if (le != cudaSuccess) return le;
     for (int m = 0; m < count; m++) {
         ws->slot_split[first_slot + m] = held + n_split;
@@ -729,23 +752,28 @@ cudaError_t ingot_linear_tc_finish_residual_norm(ingot_linear_ws* ws, float* x, 
     if (le != cudaSuccess) return le;
     return norm_w ? set_prepared(ws, n, n_tok) : cudaGetLastError();
 }
-cudaError_t ingot_linear_tc_finish_residual_norm_bf16(ingot_linear_ws* ws, float* x, const float* norm_w, float eps, int n_mean, cudaStream_t s) {
+cudaError_t ingot_linear_tc_finish_residual_norm_bf16(ingot_linear_ws* ws, float* x, const float* norm_w, float eps, int n_mean, int planes,
+                                                      cudaStream_t s) {
     const int n = ws->slot_out[0], n_tok = ws->prepared_tok;
     if (n % 4 != 0 || (norm_w && !act_shape_ok(ws, n, n_tok)) || !ws->bf16) return cudaErrorInvalidValue;
-    cudaError_t le = launch_pdl(finish_residual_norm_kernel<kActBF16>, dim3(n_tok), dim3(256), 0, s, x, slices_of(ws, 0), ws->hi, ws->lo, norm_w, n, n_mean, n_tok, eps);
+    cudaError_t le = planes > 1
+        ? launch_pdl(finish_residual_norm_kernel<kActBF16Pair>, dim3(n_tok), dim3(256), 0, s, x, slices_of(ws, 0), ws->hi, ws->lo, norm_w, n, n_mean, n_tok, eps)
+        : launch_pdl(finish_residual_norm_kernel<kActBF16>, dim3(n_tok), dim3(256), 0, s, x, slices_of(ws, 0), ws->hi, ws->lo, norm_w, n, n_mean, n_tok, eps);
     if (le != cudaSuccess) return le;
-    ws->planes = 1;
+    ws->planes = planes > 1 ? 2 : 1;
     return norm_w ? set_prepared(ws, n, n_tok) : cudaGetLastError();
 }
 
 // The product in slot 0 (width 2 n: gate half, up half) becomes the bf16 operand act(gate) * up of the next product.
-cudaError_t ingot_linear_tc_finish_gated_bf16(ingot_linear_ws* ws, int act, cudaStream_t s) {
+cudaError_t ingot_linear_tc_finish_gated_bf16(ingot_linear_ws* ws, int act, int planes, cudaStream_t s) {
     const int n = ws->slot_out[0] / 2, n_tok = ws->prepared_tok;
     if (!ws->bf16 || n % 8 != 0 || !act_shape_ok(ws, n, n_tok)) return cudaErrorInvalidValue;
-    cudaError_t le = launch_pdl(finish_gated_kernel, dim3((unsigned)((n / 4 + 255) / 256), n_tok), dim3(256), 0, s, ws->hi, slices_of(ws, 0), n,
-                                (size_t)n_tok * 2 * n, act);
+    const dim3 grid((unsigned)((n / 4 + 255) / 256), n_tok);
+    cudaError_t le = planes > 1
+        ? launch_pdl(finish_gated_kernel<kActBF16Pair>, grid, dim3(256), 0, s, ws->hi, ws->lo, slices_of(ws, 0), n, (size_t)n_tok * 2 * n, act)
+        : launch_pdl(finish_gated_kernel<kActBF16>, grid, dim3(256), 0, s, ws->hi, ws->lo, slices_of(ws, 0), n, (size_t)n_tok * 2 * n, act);
     if (le != cudaSuccess) return le;
-    ws->planes = 1;
+    ws->planes = planes > 1 ? 2 : 1;
     return set_prepared(ws, n, n_tok);
 }
 

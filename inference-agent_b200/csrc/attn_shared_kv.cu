@@ -16,6 +16,7 @@
 #include <algorithm>
 #include <new>
 
+#include "attn_common.cuh"
 #include "ingot_internal.cuh"
 
 #include <cuda_bf16.h>
@@ -28,6 +29,9 @@ struct ingot_skv {
     void* rows = nullptr;
     float* inv_rms = nullptr;  // [layer][block][16]
     int* status_dev = nullptr;
+    float* part = nullptr;  // split-key partials of decoded tokens, grown on demand
+    size_t part_floats = 0;
+    std::vector<void*> retired;
 };
 
 namespace {
@@ -41,13 +45,17 @@ struct PageMap {
 
 struct SharedOut {
     float* f32;
-    __nv_bfloat16* hi;
+    __nv_bfloat16 *hi, *lo;
     int ld;
     float scale;
     __device__ __forceinline__ void store(size_t row, int c, float v) const {
         const size_t i = row * ld + c;
         if (f32) f32[i] = v * scale;
-        if (hi) hi[i] = __float2bfloat16_rn(v * scale);
+        if (hi) {
+            const __nv_bfloat16 h = __float2bfloat16_rn(v * scale);
+            hi[i] = h;
+            if (lo) lo[i] = __float2bfloat16_rn(v * scale - __bfloat162float(h));
+        }
     }
 };
 
@@ -63,8 +71,14 @@ __device__ __forceinline__ float warp_max(float v) {
 }
 __device__ __forceinline__ float widen(float v) { return v; }
 __device__ __forceinline__ float widen(__half v) { return __half2float(v); }
-__device__ __forceinline__ void narrow(float* p, float v) { *p = v; }
 __device__ __forceinline__ void narrow(__half* p, float v) { *p = __float2half_rn(fminf(fmaxf(v, -65504.f), 65504.f)); }
+
+__device__ __forceinline__ void narrow4(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
+__device__ __forceinline__ void narrow4(__half* p, float4 v) {
+    __half h[4];
+    narrow(h, v.x); narrow(h + 1, v.y); narrow(h + 2, v.z); narrow(h + 3, v.w);
+    *reinterpret_cast<uint2*>(p) = *reinterpret_cast<const uint2*>(h);
+}
 
 // One CTA per token: RMS of q and k over their whole projections, the folded query (rows [token][head][dim]), and the
 // token's cache rows. q_cols / k_cols are n_head * dim and n_head_kv * dim columns of the projection row; the padding
@@ -91,37 +105,52 @@ __device__ __forceinline__ int table_block(const int32_t* tables, const int32_t*
     atomicOr(status, kDevErrBlockRange);
     return -1;
 }
+constexpr int kAppendThreads = 256;
 template <typename T>
-__global__ void __launch_bounds__(128) shared_kv_append_kernel(const AppendParams p) {
+__global__ void __launch_bounds__(kAppendThreads) shared_kv_append_kernel(const AppendParams p) {
     INGOT_PDL_TRIGGER();
     INGOT_PDL_WAIT();
-    __shared__ float red[8];
+    __shared__ float red[2 * kAppendThreads / 32];
     const int row = blockIdx.x, seq = p.st.row_seq[row];
     const int pos = p.st.pos0[seq] + row - p.st.row_start[seq];
     const float* q = p.proj + (size_t)row * p.proj_ld + p.q_off;
     const float* k = p.proj + (size_t)row * p.proj_ld + p.k_off;
     const int nq = p.n_head * p.dim, nk = p.n_head_kv * p.dim;
     float sq = 0.f, sk = 0.f;
-    for (int i = threadIdx.x; i < nq; i += 128) sq = fmaf(q[i], q[i], sq);
-    for (int i = threadIdx.x; i < nk; i += 128) sk = fmaf(k[i], k[i], sk);
+    for (int i = threadIdx.x * 4; i < nq; i += kAppendThreads * 4) {
+        const float4 v = *reinterpret_cast<const float4*>(q + i);
+        sq = fmaf(v.x, v.x, sq); sq = fmaf(v.y, v.y, sq); sq = fmaf(v.z, v.z, sq); sq = fmaf(v.w, v.w, sq);
+    }
+    for (int i = threadIdx.x * 4; i < nk; i += kAppendThreads * 4) {
+        const float4 v = *reinterpret_cast<const float4*>(k + i);
+        sk = fmaf(v.x, v.x, sk); sk = fmaf(v.y, v.y, sk); sk = fmaf(v.z, v.z, sk); sk = fmaf(v.w, v.w, sk);
+    }
     sq = warp_sum(sq);
     sk = warp_sum(sk);
-    if ((threadIdx.x & 31) == 0) { red[threadIdx.x >> 5] = sq; red[4 + (threadIdx.x >> 5)] = sk; }
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    if (lane == 0) { red[warp] = sq; red[kAppendThreads / 32 + warp] = sk; }
     __syncthreads();
-    const float iq = 1.0f / sqrtf((red[0] + red[1] + red[2] + red[3]) / float(p.q_mean) + p.eps);
-    const float ik = 1.0f / sqrtf((red[4] + red[5] + red[6] + red[7]) / float(p.k_mean) + p.eps);
+    sq = sk = 0.f;
+#pragma unroll
+    for (int w = 0; w < kAppendThreads / 32; w++) { sq += red[w]; sk += red[kAppendThreads / 32 + w]; }
+    const float iq = 1.0f / sqrtf(sq / float(p.q_mean) + p.eps);
+    const float ik = 1.0f / sqrtf(sk / float(p.k_mean) + p.eps);
     T* qo = static_cast<T*>(p.q_out) + (size_t)row * nq;
     const int group = p.n_head / p.n_head_kv;
-    for (int i = threadIdx.x; i < nq; i += 128) {
-        const int h = i / p.dim, d = i - h * p.dim;
-        narrow(qo + i, q[i] * iq * p.wq[i] * p.wk[(h / group) * p.dim + d]);
+    for (int h = warp; h < p.n_head; h += kAppendThreads / 32) {
+        const float* wk = p.wk + (h / group) * p.dim;
+        for (int d = lane * 4; d < p.dim; d += 128) {
+            const int i = h * p.dim + d;
+            const float4 v = *reinterpret_cast<const float4*>(q + i), a = *reinterpret_cast<const float4*>(p.wq + i), b = *reinterpret_cast<const float4*>(wk + d);
+            narrow4(qo + i, make_float4(v.x * iq * a.x * b.x, v.y * iq * a.y * b.y, v.z * iq * a.z * b.z, v.w * iq * a.w * b.w));
+        }
     }
     const int page = p.map.page(pos), slot = p.map.slot(pos);
     const int blk = table_block(p.tables, p.first_page, p.max_blocks, p.n_blocks, seq, page, p.status);
     if (blk < 0) return;
-    for (int i = threadIdx.x; i < nk; i += 128) {
-        const int h = i / p.dim, d = i - h * p.dim;
-        narrow(static_cast<T*>(p.rows) + (((size_t)blk * p.n_head_kv + h) * kBlockTokens + slot) * p.dim + d, k[i]);
+    for (int h = warp; h < p.n_head_kv; h += kAppendThreads / 32) {
+        T* dst = static_cast<T*>(p.rows) + (((size_t)blk * p.n_head_kv + h) * kBlockTokens + slot) * p.dim;
+        for (int d = lane * 4; d < p.dim; d += 128) narrow4(dst + d, *reinterpret_cast<const float4*>(k + h * p.dim + d));
     }
     if (threadIdx.x == 0) p.inv_rms[(size_t)blk * kBlockTokens + slot] = ik;
 }
@@ -137,6 +166,8 @@ struct AttendParams {
     float scale;
     SharedOut out;
     int* status;
+    int n_splits;   // decoding: CTAs per (token, KV head) over the keys
+    float* part;    // [token][head][split][dim + 2]
 };
 
 // ---- plain form: f32 arithmetic on the FMA pipes, any row length up to 512, f32 or f16 rows -------------------------
@@ -252,6 +283,319 @@ int launch_plain(const AttendParams& p, cudaStream_t s) {
     return INGOT_OK;
 }
 
+// ---- tensor-core form: f16 rows, m16n8k16 MMAs, one shared-memory tile for both products ------------------------------
+// Because a cached row is key and value at once, a staged tile serves S = Q K^T (plain ldmatrix) and O += P V (transposing
+// ldmatrix): half the copies and half the shared memory of a K + V kernel. Tiles are 64 keys = 4 pages, fetched page by page
+// with cp.async; the key's scale (1/rms * score scale) and its position travel with the tile, and the scale multiplies the
+// f32 score.
+//   prompts  (kDecode false): 8 warps of 16 (token, head) rows each share every tile.
+//   decoding (kDecode true):  the 4 warps of a CTA share one 16-row tile (the heads of one token that read this KV head) and
+//            take one page of every tile each; their states are merged through shared memory, and the keys of a sequence may
+//            be split over CTAs whose partial results (o, m, l) a second launch merges.
+constexpr int kTileKeys = 64;
+constexpr int kSplitKeysMin = 128;
+template <int kDim> struct MmaTile {
+    static constexpr int kStride = kDim + 8;  // halves; rows start 4 banks apart (mod 32 a permutation), so ldmatrix is conflict-free
+    static constexpr int kBytes = kTileKeys * kStride * 2;
+};
+__device__ __forceinline__ void ldmatrix4(uint32_t (&r)[4], uint32_t addr) {
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
+}
+__device__ __forceinline__ void ldmatrix4_trans(uint32_t (&r)[4], uint32_t addr) {
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
+}
+__device__ __forceinline__ void cp16(uint32_t dst, const void* src, bool on) {
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(on ? 16 : 0) : "memory");
+}
+
+template <int kDim, bool kDecode>
+__global__ void __launch_bounds__(kDecode ? 128 : 256) shared_kv_mma_kernel(const AttendParams p) {
+    constexpr int kThreads = kDecode ? 128 : 256, kWarps = kThreads / 32, kStages = kDecode ? 4 : 2;
+    constexpr int kStride = MmaTile<kDim>::kStride, kK = kDim / 16, kNt = kDecode ? 2 : 8;  // kNt: 8-key groups a warp scores per tile
+    extern __shared__ __align__(16) unsigned char smem_raw[];
+    INGOT_PDL_TRIGGER();
+    INGOT_PDL_WAIT();
+    const int seq = blockIdx.z, group = p.n_head / p.n_head_kv;
+    const int split = kDecode ? blockIdx.x % p.n_splits : 0;
+    const int kvh = blockIdx.y, len = p.st.len[seq], n_rows = len * group;
+    // prompts: later tiles see more keys, they go first
+    const int tile_rows = kDecode ? 16 : kWarps * 16;
+    const int row0 = (kDecode ? blockIdx.x / p.n_splits : (int)gridDim.x - 1 - (int)blockIdx.x) * tile_rows;
+    if (row0 >= n_rows) return;
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, j = lane & 3;
+    const int pos0 = p.st.pos0[seq];
+    const size_t tok0 = p.st.row_start[seq];
+    const __half* rows = static_cast<const __half*>(p.rows);
+
+    const int pos_first = pos0 + row0 / group, pos_last = pos0 + (min(row0 + tile_rows, n_rows) - 1) / group;
+    const int page_a = p.map.page(p.map.first_visible(pos_first)), page_b = p.map.page(pos_last);
+    int t_begin = 0, t_end = (page_b - page_a) / 4 + 1;
+    if (kDecode) {
+        const int per = (t_end + p.n_splits - 1) / p.n_splits;
+        t_begin = split * per;
+        t_end = min(t_end, t_begin + per);
+    }
+
+    // this thread's two rows
+    const int r_lo = row0 + (kDecode ? 0 : warp * 16) + g, r_hi = r_lo + 8;
+    const int pos_lo = pos0 + min(r_lo, n_rows - 1) / group, pos_hi = pos0 + min(r_hi, n_rows - 1) / group;
+    const int vis_lo = p.map.first_visible(pos_lo), vis_hi = p.map.first_visible(pos_hi);
+    uint32_t qf[kK][4];
+    {
+        const __half* q = static_cast<const __half*>(p.q);
+        const __half* a = q + ((tok0 + r_lo / group) * p.n_head + kvh * group + r_lo % group) * kDim;
+        const __half* b = q + ((tok0 + r_hi / group) * p.n_head + kvh * group + r_hi % group) * kDim;
+#pragma unroll
+        for (int k = 0; k < kK; k++) {
+            qf[k][0] = r_lo < n_rows ? *reinterpret_cast<const uint32_t*>(a + k * 16 + 2 * j) : 0u;
+            qf[k][1] = r_hi < n_rows ? *reinterpret_cast<const uint32_t*>(b + k * 16 + 2 * j) : 0u;
+            qf[k][2] = r_lo < n_rows ? *reinterpret_cast<const uint32_t*>(a + k * 16 + 8 + 2 * j) : 0u;
+            qf[k][3] = r_hi < n_rows ? *reinterpret_cast<const uint32_t*>(b + k * 16 + 8 + 2 * j) : 0u;
+        }
+    }
+
+    const uint32_t s_tile = (uint32_t)__cvta_generic_to_shared(smem_raw);
+    float* s_scale = reinterpret_cast<float*>(smem_raw + kStages * MmaTile<kDim>::kBytes);  // [stage][64]
+    int* s_pos = reinterpret_cast<int*>(s_scale + kStages * kTileKeys);                      // [stage][64]: position, or INT_MAX
+
+    auto stage = [&](int t, int buf) {
+        constexpr int kPieces = kDim / 8;
+        for (int i = threadIdx.x; i < kTileKeys * kPieces; i += kThreads) {
+            const int key = i / kPieces, c = i - key * kPieces;
+            const int page = page_a + t * 4 + (key >> 4);
+            const int blk = page <= page_b ? table_block(p.tables, p.first_page, p.max_blocks, p.n_blocks, seq, page, p.status) : -1;
+            const __half* src = rows + (((size_t)max(blk, 0) * p.n_head_kv + kvh) * kBlockTokens + (key & 15)) * kDim + c * 8;
+            cp16(s_tile + buf * MmaTile<kDim>::kBytes + (key * kStride + c * 8) * 2, src, blk >= 0);
+        }
+        asm volatile("cp.async.commit_group;" ::: "memory");
+        if (threadIdx.x < kTileKeys) {
+            const int key = threadIdx.x, page = page_a + t * 4 + (key >> 4);
+            const int blk = page <= page_b ? table_block(p.tables, p.first_page, p.max_blocks, p.n_blocks, seq, page, p.status) : -1;
+            int pos = 0x7fffffff;
+            if (blk >= 0) {
+                if (p.map.chunk > 0) {
+                    const int c = page / p.map.pages_per_chunk, rel = (page - c * p.map.pages_per_chunk) * kBlockTokens + (key & 15);
+                    if (rel < p.map.chunk) pos = c * p.map.chunk + rel;
+                } else {
+                    pos = page * kBlockTokens + (key & 15);
+                }
+            }
+            s_pos[buf * kTileKeys + key] = pos;
+            s_scale[buf * kTileKeys + key] = blk >= 0 ? p.inv_rms[(size_t)blk * kBlockTokens + (key & 15)] * p.scale * 1.44269504f : 0.f;
+        }
+    };
+
+    float m_lo = -INFINITY, m_hi = -INFINITY, l_lo = 0.f, l_hi = 0.f;
+    float o[kDim / 8][4];
+#pragma unroll
+    for (int i = 0; i < kDim / 8; i++) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
+
+#pragma unroll
+    for (int i = 0; i < kStages - 1; i++) {
+        if (t_begin + i < t_end) stage(t_begin + i, i);
+        else asm volatile("cp.async.commit_group;" ::: "memory");
+    }
+    for (int t = t_begin; t < t_end; t++) {
+        const int buf = (t - t_begin) % kStages;
+        asm volatile("cp.async.wait_group %0;" ::"n"(kStages - 2) : "memory");
+        __syncthreads();  // tile t is in, and every warp is done with the buffer that is staged next
+        if (t + kStages - 1 < t_end) stage(t + kStages - 1, (t - t_begin + kStages - 1) % kStages);
+        else asm volatile("cp.async.commit_group;" ::: "memory");
+        const uint32_t tile = s_tile + buf * MmaTile<kDim>::kBytes;
+        const int key_base = kDecode ? warp * 16 : 0;
+        const float* sc = s_scale + buf * kTileKeys + key_base;
+        const int* kp = s_pos + buf * kTileKeys + key_base;
+
+        float s[kNt][4];
+#pragma unroll
+        for (int nt = 0; nt < kNt; nt += 2) {
+#pragma unroll
+            for (int e = 0; e < 4; e++) s[nt][e] = s[nt + 1][e] = 0.f;
+            // matrices: keys nt*8.. dims 0-7, same keys dims 8-15, keys (nt+1)*8.. dims 0-7, dims 8-15
+            const uint32_t a = tile + ((key_base + nt * 8 + (lane & 7) + ((lane >> 4) & 1) * 8) * kStride + ((lane >> 3) & 1) * 8) * 2;
+#pragma unroll
+            for (int k = 0; k < kK; k++) {
+                uint32_t b[4];
+                ldmatrix4(b, a + k * 32);
+                mma_16816(s[nt], qf[k][0], qf[k][1], qf[k][2], qf[k][3], b[0], b[1]);
+                mma_16816(s[nt + 1], qf[k][0], qf[k][1], qf[k][2], qf[k][3], b[2], b[3]);
+            }
+        }
+        // scale and mask; a tile all of whose keys every row of the CTA sees needs no mask
+        const bool masked = kDecode || s_pos[buf * kTileKeys] < p.map.first_visible(pos_last) || s_pos[buf * kTileKeys + kTileKeys - 1] > pos_first ||
+                            (p.map.chunk > 0 && p.map.chunk % kBlockTokens != 0);
+        float mx_lo = -INFINITY, mx_hi = -INFINITY;
+#pragma unroll
+        for (int nt = 0; nt < kNt; nt++) {
+            const float2 ks = *reinterpret_cast<const float2*>(sc + nt * 8 + 2 * j);
+            s[nt][0] *= ks.x; s[nt][1] *= ks.y; s[nt][2] *= ks.x; s[nt][3] *= ks.y;
+            if (masked) {
+                const int2 kpos = *reinterpret_cast<const int2*>(kp + nt * 8 + 2 * j);
+                if (kpos.x < vis_lo || kpos.x > pos_lo) s[nt][0] = -INFINITY;
+                if (kpos.y < vis_lo || kpos.y > pos_lo) s[nt][1] = -INFINITY;
+                if (kpos.x < vis_hi || kpos.x > pos_hi) s[nt][2] = -INFINITY;
+                if (kpos.y < vis_hi || kpos.y > pos_hi) s[nt][3] = -INFINITY;
+            }
+            mx_lo = fmaxf(mx_lo, fmaxf(s[nt][0], s[nt][1]));
+            mx_hi = fmaxf(mx_hi, fmaxf(s[nt][2], s[nt][3]));
+        }
+        mx_lo = fmaxf(mx_lo, __shfl_xor_sync(0xffffffffu, mx_lo, 1));
+        mx_lo = fmaxf(mx_lo, __shfl_xor_sync(0xffffffffu, mx_lo, 2));
+        mx_hi = fmaxf(mx_hi, __shfl_xor_sync(0xffffffffu, mx_hi, 1));
+        mx_hi = fmaxf(mx_hi, __shfl_xor_sync(0xffffffffu, mx_hi, 2));
+        const float mn_lo = fmaxf(m_lo, mx_lo), mn_hi = fmaxf(m_hi, mx_hi);
+        // a row that has not seen a key yet keeps -inf; 0 stands in for it in the exponents
+        const float rf_lo = mn_lo == -INFINITY ? 0.f : mn_lo, rf_hi = mn_hi == -INFINITY ? 0.f : mn_hi;
+        const float a_lo = exp2f(m_lo - rf_lo), a_hi = exp2f(m_hi - rf_hi);
+        m_lo = mn_lo;
+        m_hi = mn_hi;
+        float sum_lo = 0.f, sum_hi = 0.f;
+        uint32_t pa[kNt][2];
+#pragma unroll
+        for (int nt = 0; nt < kNt; nt++) {
+            const float p0 = exp2f(s[nt][0] - rf_lo), p1 = exp2f(s[nt][1] - rf_lo), p2 = exp2f(s[nt][2] - rf_hi), p3 = exp2f(s[nt][3] - rf_hi);
+            sum_lo += p0 + p1;
+            sum_hi += p2 + p3;
+            pa[nt][0] = pack_half2_rn(p0, p1);
+            pa[nt][1] = pack_half2_rn(p2, p3);
+        }
+        l_lo = l_lo * a_lo + sum_lo;
+        l_hi = l_hi * a_hi + sum_hi;
+        if (a_lo != 1.f || a_hi != 1.f) {
+#pragma unroll
+            for (int i = 0; i < kDim / 8; i++) { o[i][0] *= a_lo; o[i][1] *= a_lo; o[i][2] *= a_hi; o[i][3] *= a_hi; }
+        }
+        // O += P V; transposed 8x8 matrices: keys 0-7 dims d.., keys 8-15 dims d.., keys 0-7 dims d+8.., keys 8-15 dims d+8..
+#pragma unroll
+        for (int kk = 0; kk < kNt / 2; kk++) {
+            const uint32_t a = tile + ((key_base + kk * 16 + (lane & 15)) * kStride + (lane >> 4) * 8) * 2;
+#pragma unroll
+            for (int d = 0; d < kDim / 16; d++) {
+                uint32_t b[4];
+                ldmatrix4_trans(b, a + d * 32);
+                mma_16816(o[2 * d], pa[2 * kk][0], pa[2 * kk][1], pa[2 * kk + 1][0], pa[2 * kk + 1][1], b[0], b[1]);
+                mma_16816(o[2 * d + 1], pa[2 * kk][0], pa[2 * kk][1], pa[2 * kk + 1][0], pa[2 * kk + 1][1], b[2], b[3]);
+            }
+        }
+    }
+    l_lo += __shfl_xor_sync(0xffffffffu, l_lo, 1);
+    l_lo += __shfl_xor_sync(0xffffffffu, l_lo, 2);
+    l_hi += __shfl_xor_sync(0xffffffffu, l_hi, 1);
+    l_hi += __shfl_xor_sync(0xffffffffu, l_hi, 2);
+
+    if (!kDecode) {
+        const float i_lo = 1.0f / l_lo, i_hi = 1.0f / l_hi;
+#pragma unroll
+        for (int half = 0; half < 2; half++) {
+            const int r = half ? r_hi : r_lo;
+            if (r >= n_rows) continue;
+            const size_t row = tok0 + r / group;
+            const int c0 = (kvh * group + r % group) * p.out_dim;
+            const float inv = half ? i_hi : i_lo;
+#pragma unroll
+            for (int i = 0; i < kDim / 8; i++)
+#pragma unroll
+                for (int e = 0; e < 2; e++) {
+                    const int d = i * 8 + 2 * j + e;
+                    if (d < p.out_dim) p.out.store(row, c0 + d, o[i][half * 2 + e] * inv);
+                }
+        }
+        return;
+    }
+    // merge the warps' states: [warp][16 rows][kDim] and (m, l)
+    __syncthreads();
+    float* so = reinterpret_cast<float*>(smem_raw);
+    float* sml = so + kWarps * 16 * kDim;
+#pragma unroll
+    for (int i = 0; i < kDim / 8; i++) {
+        *reinterpret_cast<float2*>(so + (warp * 16 + g) * kDim + i * 8 + 2 * j) = make_float2(o[i][0], o[i][1]);
+        *reinterpret_cast<float2*>(so + (warp * 16 + g + 8) * kDim + i * 8 + 2 * j) = make_float2(o[i][2], o[i][3]);
+    }
+    if (j == 0) {
+        sml[(warp * 16 + g) * 2] = m_lo; sml[(warp * 16 + g) * 2 + 1] = l_lo;
+        sml[(warp * 16 + g + 8) * 2] = m_hi; sml[(warp * 16 + g + 8) * 2 + 1] = l_hi;
+    }
+    __syncthreads();
+    const int rows_here = min(16, n_rows - row0);
+    for (int i = threadIdx.x; i < rows_here * kDim; i += kThreads) {
+        const int r = i / kDim, d = i - r * kDim;
+        float m = -INFINITY;
+#pragma unroll
+        for (int w = 0; w < kWarps; w++) m = fmaxf(m, sml[(w * 16 + r) * 2]);
+        const float rf = m == -INFINITY ? 0.f : m;
+        float l = 0.f, acc = 0.f;
+#pragma unroll
+        for (int w = 0; w < kWarps; w++) {
+            const float f = exp2f(sml[(w * 16 + r) * 2] - rf);
+            l = fmaf(f, sml[(w * 16 + r) * 2 + 1], l);
+            acc = fmaf(f, so[(w * 16 + r) * kDim + d], acc);
+        }
+        const int rr = row0 + r, h = kvh * group + rr % group;
+        const size_t row = tok0 + rr / group;
+        if (p.n_splits == 1) {
+            if (d < p.out_dim) p.out.store(row, h * p.out_dim + d, acc / l);
+        } else {
+            float* part = p.part + ((row * p.n_head + h) * p.n_splits + split) * (kDim + 2);
+            part[d] = acc;
+            if (d == 0) { part[kDim] = m; part[kDim + 1] = l; }
+        }
+    }
+}
+
+// out = sum_s o_s 2^(m_s - M) / sum_s l_s 2^(m_s - M) over the splits of one (token, head)
+__global__ void __launch_bounds__(128) shared_kv_merge_kernel(const AttendParams p) {
+    INGOT_PDL_TRIGGER();
+    INGOT_PDL_WAIT();
+    const int h = blockIdx.x;
+    const size_t row = blockIdx.y;
+    const float* part = p.part + (row * p.n_head + h) * p.n_splits * (p.dim + 2);
+    float m = -INFINITY;
+    for (int s = 0; s < p.n_splits; s++) m = fmaxf(m, part[s * (p.dim + 2) + p.dim]);
+    for (int d = threadIdx.x; d < p.out_dim; d += 128) {
+        float l = 0.f, acc = 0.f;
+        for (int s = 0; s < p.n_splits; s++) {
+            const float f = exp2f(part[s * (p.dim + 2) + p.dim] - m);  // every query sees itself: the overall maximum is finite
+            l = fmaf(f, part[s * (p.dim + 2) + p.dim + 1], l);
+            acc = fmaf(f, part[s * (p.dim + 2) + d], acc);
+        }
+        p.out.store(row, h * p.out_dim + d, acc / l);
+    }
+}
+
+template <int kDim>
+int launch_mma(ingot_skv* kv, AttendParams p, cudaStream_t s) {
+    const int group = p.n_head / p.n_head_kv;
+    if (p.st.max_len > 1) {
+        constexpr int kSmem = 2 * (MmaTile<kDim>::kBytes + kTileKeys * 8);
+        const dim3 grid((unsigned)(((size_t)p.st.max_len * group + 127) / 128), p.n_head_kv, p.st.n_seq);
+        p.n_splits = 1;
+        INGOT_CUDA_TRY(cudaFuncSetAttribute(shared_kv_mma_kernel<kDim, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, kSmem));
+        INGOT_CUDA_TRY(ingot_launch_pdl(shared_kv_mma_kernel<kDim, false>, grid, dim3(256), kSmem, s, p));
+        return INGOT_OK;
+    }
+    const int row_tiles = (group + 15) / 16, keys = p.max_blocks * kBlockTokens;
+    // enough CTAs for two per SM, at least kSplitKeysMin keys each
+    p.n_splits = std::max(1, std::min({(keys + kSplitKeysMin - 1) / kSplitKeysMin, 2 * kv->num_sms / (row_tiles * p.n_head_kv * p.st.n_seq), 32}));
+    if (p.n_splits > 1) {
+        const size_t need = (size_t)p.st.n_tok * p.n_head * p.n_splits * (kDim + 2);
+        if (need > kv->part_floats) {
+            float* fresh = nullptr;
+            INGOT_CUDA_TRY(cudaMalloc(&fresh, need * sizeof(float)));
+            if (kv->part) kv->retired.push_back(kv->part);  // a captured graph may still point into it
+            kv->part = fresh;
+            kv->part_floats = need;
+        }
+        p.part = kv->part;
+    }
+    constexpr int kRing = 4 * (MmaTile<kDim>::kBytes + kTileKeys * 8), kMerge = 4 * 16 * (kDim + 2) * 4;
+    constexpr int kSmem = kRing > kMerge ? kRing : kMerge;
+    INGOT_CUDA_TRY(cudaFuncSetAttribute(shared_kv_mma_kernel<kDim, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, kSmem));
+    const dim3 grid(row_tiles * p.n_splits, p.n_head_kv, p.st.n_seq);
+    INGOT_CUDA_TRY(ingot_launch_pdl(shared_kv_mma_kernel<kDim, true>, grid, dim3(128), kSmem, s, p));
+    if (p.n_splits > 1) INGOT_CUDA_TRY(ingot_launch_pdl(shared_kv_merge_kernel, dim3(p.n_head, p.st.n_tok), dim3(128), 0, s, p));
+    return INGOT_OK;
+}
+
 bool step_ok(const ingot_step* st) {
     return st && st->n_tok >= 1 && st->n_seq >= 1 && st->n_seq <= 65535 && st->max_len >= 1 && st->row_seq && st->row_start && st->len && st->pos0;
 }
@@ -265,8 +609,8 @@ int ingot_skv_create(ingot_skv** out, int n_layer, int n_head_kv, int head_dim, 
     *out = nullptr;
     INGOT_REQUIRE(n_layer >= 1 && n_head_kv >= 1 && n_blocks >= 1 && chunk >= 0, "ingot_skv_create: bad sizes");
     INGOT_REQUIRE(dtype == INGOT_F32 || dtype == INGOT_F16, "ingot_skv_create: rows are f32 or f16");
-    if (head_dim < 2 || head_dim > 512 || head_dim % 2 != 0) {
-        ingot_set_error("ingot_skv_create: row length must be even and at most 512");
+    if (head_dim < 4 || head_dim > 512 || head_dim % 4 != 0) {
+        ingot_set_error("ingot_skv_create: row length must be a multiple of 4 and at most 512");
         return INGOT_ERR_UNSUPPORTED;
     }
     ingot_skv* kv = new (std::nothrow) ingot_skv();
@@ -294,6 +638,8 @@ void ingot_skv_destroy(ingot_skv* kv) {
     cudaFree(kv->rows);
     cudaFree(kv->inv_rms);
     cudaFree(kv->status_dev);
+    cudaFree(kv->part);
+    for (void* p : kv->retired) cudaFree(p);
     delete kv;
 }
 
@@ -305,7 +651,12 @@ int ingot_skv_pages(int chunk, int n_positions) {
 
 int* ingot_skv_status_dev(ingot_skv* kv) { return kv ? kv->status_dev : nullptr; }
 
-int ingot_skv_row_length(int head_size) { return head_size < 1 ? 0 : (head_size + 15) / 16 * 16; }
+int ingot_skv_row_length(int head_size) {
+    if (head_size < 1) return 0;
+    for (int d : {32, 64, 96, 128, 192, 256})
+        if (head_size <= d) return d;
+    return (head_size + 15) / 16 * 16;
+}
 
 int ingot_skv_status(ingot_skv* kv, void* stream, int* status_out) {
     INGOT_REQUIRE(kv && status_out, "ingot_skv_status: null argument");
@@ -323,6 +674,7 @@ int ingot_skv_append(ingot_skv* kv, int layer, const ingot_step* step, const flo
     INGOT_REQUIRE_DEVICE(kv);
     INGOT_REQUIRE(layer >= 0 && layer < kv->n_layer, "ingot_skv_append: layer out of range");
     INGOT_REQUIRE(proj_dev && q_norm_dev && k_norm_dev && q_out_dev && tables_dev && max_blocks >= 1, "ingot_skv_append: null argument");
+    INGOT_REQUIRE(proj_ld % 4 == 0 && q_off % 4 == 0 && k_off % 4 == 0, "ingot_skv_append: rows and offsets must be multiples of 4 floats");
     INGOT_REQUIRE(n_head >= kv->n_head_kv && n_head % kv->n_head_kv == 0, "ingot_skv_append: n_head must be a multiple of n_head_kv");
     INGOT_REQUIRE(head_size >= 1 && head_size <= kv->dim, "ingot_skv_append: head size beyond the row length");
     const size_t esz = kv->dtype == INGOT_F32 ? 4 : 2;
@@ -331,7 +683,7 @@ int ingot_skv_append(ingot_skv* kv, int layer, const ingot_step* step, const flo
                       kv->inv_rms + (size_t)layer * kv->n_blocks * kBlockTokens, tables_dev, first_page_dev, max_blocks, kv->n_blocks,
                       PageMap{kv->chunk, (kv->chunk + kBlockTokens - 1) / kBlockTokens}, kv->status_dev};
     auto kernel = kv->dtype == INGOT_F32 ? shared_kv_append_kernel<float> : shared_kv_append_kernel<__half>;
-    INGOT_CUDA_TRY(ingot_launch_pdl(kernel, dim3(step->n_tok), dim3(128), 0, static_cast<cudaStream_t>(stream), p));
+    INGOT_CUDA_TRY(ingot_launch_pdl(kernel, dim3(step->n_tok), dim3(kAppendThreads), 0, static_cast<cudaStream_t>(stream), p));
     return INGOT_OK;
 }
 
@@ -342,15 +694,24 @@ int ingot_skv_attend(ingot_skv* kv, int layer, const ingot_step* step, const voi
     INGOT_REQUIRE(layer >= 0 && layer < kv->n_layer, "ingot_skv_attend: layer out of range");
     INGOT_REQUIRE(q_dev && out && tables_dev && max_blocks >= 1, "ingot_skv_attend: null argument");
     INGOT_REQUIRE(n_head >= kv->n_head_kv && n_head % kv->n_head_kv == 0, "ingot_skv_attend: n_head must be a multiple of n_head_kv");
-    INGOT_REQUIRE(out_dim >= 1 && out_dim <= kv->dim && !out->lo, "ingot_skv_attend: bad output");
-    (void)impl;
+    INGOT_REQUIRE(out_dim >= 1 && out_dim <= kv->dim, "ingot_skv_attend: bad output");
     const size_t esz = kv->dtype == INGOT_F32 ? 4 : 2;
     AttendParams p = {*step, q_dev, static_cast<const char*>(kv->rows) + kv->layer_elems * layer * esz,
                       kv->inv_rms + (size_t)layer * kv->n_blocks * kBlockTokens, tables_dev, first_page_dev, max_blocks, kv->n_blocks, n_head, kv->n_head_kv,
                       kv->dim, out_dim, PageMap{kv->chunk, (kv->chunk + kBlockTokens - 1) / kBlockTokens}, scale,
-                      SharedOut{out->f32, static_cast<__nv_bfloat16*>(out->hi), out->ld, out_scale}, kv->status_dev};
+                      SharedOut{out->f32, static_cast<__nv_bfloat16*>(out->hi), static_cast<__nv_bfloat16*>(out->lo), out->ld, out_scale}, kv->status_dev, 1, nullptr};
     cudaStream_t s = static_cast<cudaStream_t>(stream);
-    return kv->dtype == INGOT_F32 ? launch_plain<float>(p, s) : launch_plain<__half>(p, s);
+    if (kv->dtype == INGOT_F32) return launch_plain<float>(p, s);
+    if (impl != 1) switch (kv->dim) {
+        case 32: return launch_mma<32>(kv, p, s);
+        case 64: return launch_mma<64>(kv, p, s);
+        case 96: return launch_mma<96>(kv, p, s);
+        case 128: return launch_mma<128>(kv, p, s);
+        case 192: return launch_mma<192>(kv, p, s);
+        case 256: return launch_mma<256>(kv, p, s);
+        default: break;
+    }
+    return launch_plain<__half>(p, s);
 }
 
 }  // extern "C"

@@ -47,6 +47,25 @@ struct ActOut {
             if (lo) lo[i] = __float2bfloat16_rn(v - __bfloat162float(h));
         }
     }
+    // four consecutive columns, c and ld multiples of 4
+    __device__ __forceinline__ void store4(size_t row, int c, float4 v) const {
+        const size_t i = row * ld + c;
+        if (f32) *reinterpret_cast<float4*>(f32 + i) = v;
+        if (hi) {
+            const __nv_bfloat162 a = __floats2bfloat162_rn(v.x, v.y), b = __floats2bfloat162_rn(v.z, v.w);
+            uint2 w;
+            w.x = *reinterpret_cast<const uint32_t*>(&a);
+            w.y = *reinterpret_cast<const uint32_t*>(&b);
+            *reinterpret_cast<uint2*>(hi + i) = w;
+            if (lo) {
+                const float2 af = __bfloat1622float2(a), bf = __bfloat1622float2(b);
+                const __nv_bfloat162 c2 = __floats2bfloat162_rn(v.x - af.x, v.y - af.y), d2 = __floats2bfloat162_rn(v.z - bf.x, v.w - bf.y);
+                w.x = *reinterpret_cast<const uint32_t*>(&c2);
+                w.y = *reinterpret_cast<const uint32_t*>(&d2);
+                *reinterpret_cast<uint2*>(lo + i) = w;
+            }
+        }
+    }
 };
 
 // ---- causal convolution -------------------------------------------------------------------------------------------
@@ -145,6 +164,44 @@ __device__ __forceinline__ void cp_async_commit() { asm volatile("cp.async.commi
 template <int N>
 __device__ __forceinline__ void cp_async_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
 
+// Pairs of f32 in one 64-bit register: two multiply-adds per instruction.
+typedef unsigned long long f32x2;
+__device__ __forceinline__ f32x2 pair(float x, float y) {
+    f32x2 r;
+    asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(x), "f"(y));
+    return r;
+}
+__device__ __forceinline__ float2 unpair(f32x2 v) {
+    float2 r;
+    asm("mov.b64 {%0, %1}, %2;" : "=f"(r.x), "=f"(r.y) : "l"(v));
+    return r;
+}
+__device__ __forceinline__ f32x2 mul2(f32x2 a, f32x2 b) {
+    f32x2 r;
+    asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
+    return r;
+}
+__device__ __forceinline__ f32x2 fma2(f32x2 a, f32x2 b, f32x2 c) {
+    f32x2 r;
+    asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c));
+    return r;
+}
+// kS consecutive floats of shared memory as pairs
+template <int kS>
+__device__ __forceinline__ void load_pairs(const float* p, f32x2 (&v)[kS / 2]) {
+    if (kS % 4 == 0) {
+#pragma unroll
+        for (int i = 0; i < kS / 4; i++) {
+            const ulonglong2 q = *reinterpret_cast<const ulonglong2*>(p + 4 * i);
+            v[2 * i] = q.x;
+            v[2 * i + 1] = q.y;
+        }
+    } else {
+#pragma unroll
+        for (int i = 0; i < kS / 2; i++) v[i] = *reinterpret_cast<const f32x2*>(p + 2 * i);
+    }
+}
+
 // kLg: log2 of the lanes per channel, or -1 for p.lanes_log2
 template <int kS, bool kOutput, int kLg, bool kExact>
 __global__ void __launch_bounds__(128) selective_scan_kernel(const ScanParams p) {
@@ -154,7 +211,7 @@ __global__ void __launch_bounds__(128) selective_scan_kernel(const ScanParams p)
     const int chunk = blockIdx.y;
     const int seq = p.chunk_seq[chunk], t0 = p.chunk_t0[chunk], len = p.chunk_len[chunk];
     const bool first = t0 == 0, last = t0 + len == p.st.len[seq];
-    if (!kOutput && first && last) return;  // a single chunk needs no partial state
+    if (!kOutput && last) return;  // nothing follows a sequence's last chunk
     const int lg = kLg >= 0 ? kLg : p.lanes_log2;
     const int lanes = 1 << lg, n_ch = 128 >> lg;
     const int ch = threadIdx.x >> lg, part = threadIdx.x & (lanes - 1);
@@ -163,18 +220,19 @@ __global__ void __launch_bounds__(128) selective_scan_kernel(const ScanParams p)
     const size_t row0 = (size_t)p.st.row_start[seq] + t0;
     const int np = p.n_pad;
 
-    // [2 buffers][16 tokens]: x, dt [n_ch], B, C [np]; then dt * x of the current tile and y
-    const int tile_floats = kScanTile * (2 * n_ch + 2 * np);
+    // [2 buffers][16 tokens]: x, dt, z [n_ch], B, C [np]; then dt * x of the current tile and y
+    const int tile_floats = kScanTile * (3 * n_ch + 2 * np);
     float* const s_dtx = smem + 2 * tile_floats;
     float* const s_y = s_dtx + kScanTile * n_ch;
+    const int ch4 = n_ch >> 2, np4 = np >> 2;
 
     auto stage = [&](int tile) {
         float* sx = smem + (tile & 1) * tile_floats;
         float* sdt = sx + kScanTile * n_ch;
-        float* sb = sdt + kScanTile * n_ch;
+        float* sz = sdt + kScanTile * n_ch;
+        float* sb = sz + kScanTile * n_ch;
         float* sc = sb + kScanTile * np;
         const int t_base = tile * kScanTile;
-        const int ch4 = n_ch >> 2;
         for (int i = threadIdx.x; i < kScanTile * ch4; i += 128) {
             const int t = i / ch4, q = (i - t * ch4) * 4;
             const bool on = t_base + t < len && c_base + q < p.inner;
@@ -182,8 +240,8 @@ __global__ void __launch_bounds__(128) selective_scan_kernel(const ScanParams p)
             const int cc = min(c_base + q, p.inner - 4);
             cp_async16(sx + t * n_ch + q, p.x + row * p.x_ld + cc, on);
             cp_async16(sdt + t * n_ch + q, p.dt + row * p.dt_ld + cc, on);
+            if (kOutput) cp_async16(sz + t * n_ch + q, p.z + row * p.z_ld + cc, on);
         }
-        const int np4 = np >> 2;
         for (int i = threadIdx.x; i < kScanTile * np4; i += 128) {
             const int t = i / np4, q = (i - t * np4) * 4;
             const bool on = t_base + t < len;
@@ -197,34 +255,27 @@ __global__ void __launch_bounds__(128) selective_scan_kernel(const ScanParams p)
     const int n_tiles = (len + kScanTile - 1) / kScanTile;
     stage(0);
 
-    float a[kS], s[kS];
+    f32x2 a[kS / 2], s[kS / 2];
     const size_t sidx = (size_t)(live ? c : 0) * np + part * kS;
-#pragma unroll
-    for (int i = 0; i < kS; i++) {
-        a[i] = live ? p.a2[sidx + i] : 0.f;
-        s[i] = 0.f;
-    }
     const size_t slot_base = (size_t)p.st.slot[seq] * p.inner * np;
-    if (live) {
-        if (first) {
-            // pass 3 of a multi-chunk sequence reads its start state from the scratch too: the last chunk's CTA may write
-            // the slot before this CTA gets to read it
-            if (kOutput && !last) {
+    {
+        // Start state: the slot for a sequence's first chunk (zero before position 0), else what pass 2 left. Pass 3 of a
+        // multi-chunk sequence takes the first chunk's from there too: the last chunk's CTA may write the slot before this
+        // CTA gets to read it.
+        const float* from = nullptr;
+        if (kOutput && !(first && last)) from = p.part + (size_t)chunk * p.inner * np + sidx;
+        else if (first && p.st.pos0[seq] > 0) from = p.state + slot_base + sidx;
 #pragma unroll
-                for (int i = 0; i < kS; i++) s[i] = p.part[(size_t)chunk * p.inner * np + sidx + i];
-            } else if (p.st.pos0[seq] > 0) {
-#pragma unroll
-                for (int i = 0; i < kS; i++) s[i] = p.state[slot_base + sidx + i];
-            }
-        } else if (kOutput) {
-#pragma unroll
-            for (int i = 0; i < kS; i++) s[i] = p.part[(size_t)chunk * p.inner * np + sidx + i];
+        for (int i = 0; i < kS / 2; i++) {
+            a[i] = live ? *reinterpret_cast<const f32x2*>(p.a2 + sidx + 2 * i) : 0;
+            s[i] = live && from ? *reinterpret_cast<const f32x2*>(from + 2 * i) : 0;
         }
     }
-    const int my_ch = threadIdx.x % n_ch;  // the channel this thread prepares and writes (n_ch divides 128)
-    const bool my_live = c_base + my_ch < p.inner;
-    const float my_bias = my_live ? p.dt_bias[c_base + my_ch] : 0.f;
-    const float my_d = kOutput && my_live ? p.d[c_base + my_ch] : 0.f;
+    const int my_q = (threadIdx.x % ch4) * 4;  // the four channels this thread prepares and writes (ch4 divides 128)
+    const bool my_live = c_base + my_q < p.inner;
+    const float4 zero4 = make_float4(0.f, 0.f, 0.f, 0.f);
+    const float4 my_bias = my_live ? *reinterpret_cast<const float4*>(p.dt_bias + c_base + my_q) : zero4;
+    const float4 my_d = kOutput && my_live ? *reinterpret_cast<const float4*>(p.d + c_base + my_q) : zero4;
     float sum_dt = 0.f;
 
     for (int tile = 0; tile < n_tiles; tile++) {
@@ -232,42 +283,65 @@ __global__ void __launch_bounds__(128) selective_scan_kernel(const ScanParams p)
         __syncthreads();
         float* sx = smem + (tile & 1) * tile_floats;
         float* sdt = sx + kScanTile * n_ch;
-        const float* sb = sdt + kScanTile * n_ch;
+        const float* sz = sdt + kScanTile * n_ch;
+        const float* sb = sz + kScanTile * n_ch;
         const float* sc = sb + kScanTile * np;
         const int n_t = min(kScanTile, len - tile * kScanTile);
-        for (int i = threadIdx.x; i < kScanTile * n_ch; i += 128) {
-            const int t = i / n_ch;
-            const float dt = t < n_t ? softplusf(sdt[i] + my_bias) : 0.f;
-            sdt[i] = dt;
-            s_dtx[i] = dt * sx[i];
+        for (int i = threadIdx.x; i < n_t * ch4; i += 128) {
+            const float4 raw = reinterpret_cast<const float4*>(sdt)[i], xv = reinterpret_cast<const float4*>(sx)[i];
+            const float4 dt = make_float4(softplusf(raw.x + my_bias.x), softplusf(raw.y + my_bias.y), softplusf(raw.z + my_bias.z), softplusf(raw.w + my_bias.w));
+            reinterpret_cast<float4*>(sdt)[i] = dt;
+            reinterpret_cast<float4*>(s_dtx)[i] = make_float4(dt.x * xv.x, dt.y * xv.y, dt.z * xv.z, dt.w * xv.w);
         }
         __syncthreads();
-#pragma unroll 4
-        for (int t = 0; t < n_t; t++) {
+        auto token = [&](int t) {
             const float dt = sdt[t * n_ch + ch], dtx = s_dtx[t * n_ch + ch];
-            const float* b = sb + t * np + part * kS;
-            const float* cc = sc + t * np + part * kS;
-            float y = 0.f;
+            f32x2 b[kS / 2], cc[kS / 2];
+            load_pairs<kS>(sb + t * np + part * kS, b);
+            if (kOutput) load_pairs<kS>(sc + t * np + part * kS, cc);
+            const f32x2 dt2 = kExact ? pair(dt * 0.69314718f, dt * 0.69314718f) : pair(dt, dt), dtx2 = pair(dtx, dtx);
+            f32x2 y2 = 0;
 #pragma unroll
-            for (int i = 0; i < kS; i++) {
-                if (kExact) s[i] += fmaf(expm1f(dt * a[i] * 0.69314718f), s[i], dtx * b[i]);
-                else s[i] = fmaf(ex2f(dt * a[i]), s[i], dtx * b[i]);
-                if (kOutput) y = fmaf(s[i], cc[i], y);
+            for (int i = 0; i < kS / 2; i++) {
+                const float2 x = unpair(mul2(dt2, a[i]));
+                const f32x2 in = mul2(dtx2, b[i]);
+                if (kExact) {
+                    const float2 sv = unpair(s[i]), iv = unpair(in);
+                    s[i] = pair(sv.x + fmaf(expm1f(x.x), sv.x, iv.x), sv.y + fmaf(expm1f(x.y), sv.y, iv.y));
+                } else {
+                    s[i] = fma2(pair(ex2f(x.x), ex2f(x.y)), s[i], in);
+                }
+                if (kOutput) y2 = fma2(s[i], cc[i], y2);
             }
             if (kOutput) {
-                for (int o = lanes >> 1; o > 0; o >>= 1) y += __shfl_xor_sync(0xffffffffu, y, o);
+                const float2 yv = unpair(y2);
+                float y = yv.x + yv.y;
+                if (kLg == 2) {
+                    y += __shfl_xor_sync(0xffffffffu, y, 2);
+                    y += __shfl_xor_sync(0xffffffffu, y, 1);
+                } else {
+                    for (int o = lanes >> 1; o > 0; o >>= 1) y += __shfl_xor_sync(0xffffffffu, y, o);
+                }
                 if (part == 0) s_y[t * n_ch + ch] = y;
             } else {
                 sum_dt += dt;
             }
+        };
+        if (n_t == kScanTile) {
+#pragma unroll 8
+            for (int t = 0; t < kScanTile; t++) token(t);
+        } else {
+            for (int t = 0; t < n_t; t++) token(t);
         }
         if (kOutput) {
             __syncthreads();
             if (my_live) {
-                for (int i = threadIdx.x; i < n_t * n_ch; i += 128) {
-                    const size_t row = row0 + tile * kScanTile + i / n_ch;
-                    const float y = fmaf(my_d, sx[i], s_y[i]);
-                    p.out.store(row, c_base + my_ch, y * siluf(p.z[row * p.z_ld + c_base + my_ch]));
+                for (int i = threadIdx.x; i < n_t * ch4; i += 128) {
+                    const size_t row = row0 + tile * kScanTile + i / ch4;
+                    const float4 xv = reinterpret_cast<const float4*>(sx)[i], yv = reinterpret_cast<const float4*>(s_y)[i],
+                                 zv = reinterpret_cast<const float4*>(sz)[i];
+                    p.out.store4(row, c_base + my_q, make_float4(fmaf(my_d.x, xv.x, yv.x) * siluf(zv.x), fmaf(my_d.y, xv.y, yv.y) * siluf(zv.y),
+                                                                 fmaf(my_d.z, xv.z, yv.z) * siluf(zv.z), fmaf(my_d.w, xv.w, yv.w) * siluf(zv.w)));
                 }
             }
         }
@@ -276,11 +350,11 @@ __global__ void __launch_bounds__(128) selective_scan_kernel(const ScanParams p)
     if (!live) return;
     if (!kOutput) {
 #pragma unroll
-        for (int i = 0; i < kS; i++) p.part[(size_t)chunk * p.inner * np + sidx + i] = s[i];
+        for (int i = 0; i < kS / 2; i++) *reinterpret_cast<f32x2*>(p.part + (size_t)chunk * p.inner * np + sidx + 2 * i) = s[i];
         if (part == 0) p.part_sum[(size_t)chunk * p.inner + c] = sum_dt;
     } else if (last) {
 #pragma unroll
-        for (int i = 0; i < kS; i++) p.state[slot_base + sidx + i] = s[i];
+        for (int i = 0; i < kS / 2; i++) *reinterpret_cast<f32x2*>(p.state + slot_base + sidx + 2 * i) = s[i];
     }
 }
 
@@ -293,7 +367,7 @@ __global__ void __launch_bounds__(256) selective_scan_link_kernel(const ScanPara
     const size_t per = (size_t)p.inner * p.n_pad;
     const size_t i = (size_t)blockIdx.x * 256 + threadIdx.x;
     if (k1 - k0 < 2 || i >= per) return;
-    const int c = int(i / p.n_pad);
+    const int c = int(i / p.n_pad);  // the last chunk leaves no end state; what is read in its place goes nowhere
     const float a = p.a2[i];
     float s = p.st.pos0[seq] > 0 ? p.state[(size_t)p.st.slot[seq] * per + i] : 0.f;
     float end = p.part[(size_t)k0 * per + i];
@@ -332,7 +406,7 @@ __global__ void __launch_bounds__(128) gated_lru_kernel(const LruParams p) {
     const int chunk = blockIdx.y, c = blockIdx.x * 128 + threadIdx.x;
     const int seq = p.chunk_seq[chunk], t0 = p.chunk_t0[chunk], len = p.chunk_len[chunk];
     const bool first = t0 == 0, last = t0 + len == p.st.len[seq];
-    if ((!kOutput && first && last) || c >= p.width) return;
+    if ((!kOutput && last) || c >= p.width) return;
     const size_t row0 = (size_t)p.st.row_start[seq] + t0;
     const int gcol = (c / p.block) * 2 * p.block + c % p.block;
     const float br = p.br[c], bi = p.bi[c], k = -8.0f * p.sp[c], yb = kOutput ? p.y_bias[c] : 0.f;
@@ -393,6 +467,12 @@ int scan_lanes_log2(int n_state) {
     return l;
 }
 
+// States a lane holds: an even number, so that pairs fill 64-bit registers.
+int scan_states_per_lane(int n_state) {
+    const int lg = scan_lanes_log2(n_state), per = ((n_state + (1 << lg) - 1) >> lg) + 1 & ~1;
+    return lg > 2 && per < 6 ? 6 : per;
+}
+
 }  // namespace
 
 extern "C" {
@@ -412,9 +492,7 @@ int ingot_causal_conv(const ingot_step* step, const float* in_dev, int in_ld, co
 
 int ingot_scan_state_pad(int n_state) {
     if (n_state < 1 || n_state > 256) return 0;
-    const int lanes = 1 << scan_lanes_log2(n_state);
-    const int q = lanes > 8 ? lanes : 8;
-    return (n_state + q - 1) / q * q;
+    return scan_states_per_lane(n_state) << scan_lanes_log2(n_state);
 }
 
 int ingot_selective_scan(const ingot_step* step, const ingot_scan_plan* plan, const float* x_dev, int x_ld, const float* dt_dev,
@@ -423,33 +501,32 @@ int ingot_selective_scan(const ingot_step* step, const ingot_scan_plan* plan, co
                          int n_state, int exact, const ingot_act_out* out, void* stream) {
     INGOT_REQUIRE(step_ok(step) && plan_ok(plan), "ingot_selective_scan: bad step or plan");
     INGOT_REQUIRE(x_dev && dt_dev && dt_bias_dev && bc_dev && z_dev && a_log2e_dev && d_dev && state_dev && out, "ingot_selective_scan: null argument");
-    INGOT_REQUIRE(inner >= 4 && inner % 4 == 0 && x_ld % 4 == 0 && dt_ld % 4 == 0 && bc_ld % 4 == 0 && b_off % 4 == 0 && c_off % 4 == 0,
+    INGOT_REQUIRE(inner >= 4 && inner % 4 == 0 && x_ld % 4 == 0 && dt_ld % 4 == 0 && z_ld % 4 == 0 && out->ld % 4 == 0 && bc_ld % 4 == 0 && b_off % 4 == 0 && c_off % 4 == 0,
                   "ingot_selective_scan: rows and offsets must be multiples of 4 floats");
     const int n_pad = ingot_scan_state_pad(n_state);
     INGOT_REQUIRE(n_pad > 0, "ingot_selective_scan: between 1 and 256 states");
     const bool multi = plan->max_chunks > 1;
     INGOT_REQUIRE(!multi || (plan->scratch_dev && plan->scratch_floats >= (size_t)plan->n_chunks * inner * (n_pad + 1)),
                   "ingot_selective_scan: scratch too small");
-    const int lg = scan_lanes_log2(n_state), lanes = 1 << lg, n_ch = 128 >> lg;
-    const int per_lane = (n_state + lanes - 1) / lanes;
+    const int lg = scan_lanes_log2(n_state), n_ch = 128 >> lg;
+    const int per_lane = scan_states_per_lane(n_state);
     ScanParams p = {*step, plan->chunk_seq, plan->chunk_t0, plan->chunk_len, plan->seq_chunk0, plan->n_chunks,
                     x_dev, x_ld, dt_dev, dt_ld, dt_bias_dev, bc_dev, bc_ld, b_off, c_off, z_dev, z_ld, a_log2e_dev, d_dev,
                     state_dev, plan->scratch_dev, plan->scratch_dev ? plan->scratch_dev + (size_t)plan->n_chunks * inner * n_pad : nullptr,
                     inner, n_pad, lg, act_out(out)};
-    const size_t smem = (size_t)kScanTile * (2 * (2 * n_ch + 2 * n_pad) + 2 * n_ch) * sizeof(float);
+    const size_t smem = (size_t)kScanTile * (2 * (3 * n_ch + 2 * n_pad) + 2 * n_ch) * sizeof(float);
     typedef void (*Kernel)(ScanParams);
     Kernel k_end, k_out;
 #define INGOT_SCAN_PICK(S, OUT)                                                                                                     \
-    (exact ? (lg == 2 ? selective_scan_kernel<S, OUT, 2, true> : selective_scan_kernel<(S < 5 ? 5 : S), OUT, -1, true>)             \
-           : (lg == 2 ? selective_scan_kernel<S, OUT, 2, false> : selective_scan_kernel<(S < 5 ? 5 : S), OUT, -1, false>))
+    (exact ? (lg == 2 ? selective_scan_kernel<S, OUT, 2, true> : selective_scan_kernel<(S < 6 ? 6 : S), OUT, -1, true>)             \
+           : (lg == 2 ? selective_scan_kernel<S, OUT, 2, false> : selective_scan_kernel<(S < 6 ? 6 : S), OUT, -1, false>))
 #define INGOT_SCAN_CASE(S)                 \
     case S:                                \
         k_end = INGOT_SCAN_PICK(S, false); \
         k_out = INGOT_SCAN_PICK(S, true);  \
         break
-    switch (per_lane) {  // more than 4 lanes: always 5 to 8 states per lane
-        INGOT_SCAN_CASE(1); INGOT_SCAN_CASE(2); INGOT_SCAN_CASE(3); INGOT_SCAN_CASE(4);
-        INGOT_SCAN_CASE(5); INGOT_SCAN_CASE(6); INGOT_SCAN_CASE(7); INGOT_SCAN_CASE(8);
+    switch (per_lane) {  // more than 4 lanes: always 6 or 8 states per lane
+        INGOT_SCAN_CASE(2); INGOT_SCAN_CASE(4); INGOT_SCAN_CASE(6); INGOT_SCAN_CASE(8);
         default: ingot_set_error("ingot_selective_scan: unsupported state count"); return INGOT_ERR_UNSUPPORTED;
     }
 #undef INGOT_SCAN_CASE

@@ -105,10 +105,12 @@ def test_mixed_batches_equal_each_sequence_alone(case, f32):
             assert H.error(np.concatenate(got[k]), want[i]).max() < TOL[f32]
 
 
-def test_the_batch_does_not_change_a_sequence(case):
-    """Single tokens of three sequences in one batch against the same tokens alone: equal up to summation order."""
+@pytest.mark.parametrize("f32,tol", [(True, 1e-5), (False, 1e-3)])
+def test_the_batch_does_not_change_a_sequence(case, f32, tol):
+    """Single tokens of three sequences in one batch against the same tokens alone. In 32-bit only summation orders differ; in the
+    16-bit form a batch multiplies bf16 hi + lo pairs where a single token multiplies f32, and the cache rounds to f16."""
     cfg, folder, tokens, _ = case
-    with M.Model(folder, max_tokens=1024, max_seqs=4) as m:
+    with M.Model(folder, f32=f32, max_tokens=1024, max_seqs=4) as m:
         for s in range(3):
             m.step([(s, 0, tokens[s][:30], [])])
         together = [m.step([(s, 30 + k, tokens[s][30 + k:31 + k], [0]) for s in range(3)]) for k in range(8)]
@@ -118,7 +120,7 @@ def test_the_batch_does_not_change_a_sequence(case):
             m.step([(3, 0, tokens[s][:30], [])])
             for k in range(8):
                 alone = m.step([(3, 30 + k, tokens[s][30 + k:31 + k], [0])])
-                assert H.error(alone, together[k][s:s + 1].astype(np.float64)).max() < 1e-4
+                assert H.error(alone, together[k][s:s + 1].astype(np.float64)).max() < tol
             m.release(3)
 
 
