@@ -358,7 +358,8 @@ int ingot_skv_append(ingot_skv* kv, int layer, const ingot_step* step, const flo
                      const int32_t* tables_dev, const int32_t* first_page_dev, int max_blocks, void* stream);
 /* Softmax over the visible keys of every row (appended before), scores = q . k_row / rms(k) * scale; out[t][h * out_dim + d] =
  * out_scale * result for d < out_dim. impl: 0 = library's choice (tensor cores for f16 rows of the lengths
- * ingot_skv_row_length returns up to 256), 1 = the plain f32-arithmetic kernel. */
+ * ingot_skv_row_length returns up to 256), 1 = the plain f32-arithmetic kernel, 2 = the warp-level tensor-core
+ * kernel, 3 = the tcgen05 kernel (rows of 128 values). */
 int ingot_skv_attend(ingot_skv* kv, int layer, const ingot_step* step, const void* q_dev, int n_head, int out_dim, float scale,
                      float out_scale, const ingot_act_out* out, const int32_t* tables_dev, const int32_t* first_page_dev, int max_blocks, int impl, void* stream);
 

@@ -16,48 +16,9 @@
 #include <algorithm>
 #include <new>
 
-#include "attn_common.cuh"
-#include "ingot_internal.cuh"
-
-#include <cuda_bf16.h>
-
-struct ingot_skv {
-    int device = 0, num_sms = 0;
-    int n_layer = 0, n_head_kv = 0, dim = 0;  // dim: row length (padded head size)
-    int dtype = INGOT_F32, chunk = 0, n_blocks = 0;
-    size_t layer_elems = 0;
-    void* rows = nullptr;
-    float* inv_rms = nullptr;  // [layer][block][16]
-    int* status_dev = nullptr;
-    float* part = nullptr;  // split-key partials of decoded tokens, grown on demand
-    size_t part_floats = 0;
-    std::vector<void*> retired;
-};
+#include "attn_shared_kv.cuh"
 
 namespace {
-
-struct PageMap {
-    int chunk, pages_per_chunk;  // chunk 0: one chunk of unlimited length
-    __host__ __device__ __forceinline__ int page(int pos) const { return chunk > 0 ? (pos / chunk) * pages_per_chunk + (pos % chunk) / kBlockTokens : pos / kBlockTokens; }
-    __host__ __device__ __forceinline__ int slot(int pos) const { return (chunk > 0 ? pos % chunk : pos) % kBlockTokens; }
-    __host__ __device__ __forceinline__ int first_visible(int pos) const { return chunk > 0 ? pos / chunk * chunk : 0; }
-};
-
-struct SharedOut {
-    float* f32;
-    __nv_bfloat16 *hi, *lo;
-    int ld;
-    float scale;
-    __device__ __forceinline__ void store(size_t row, int c, float v) const {
-        const size_t i = row * ld + c;
-        if (f32) f32[i] = v * scale;
-        if (hi) {
-            const __nv_bfloat16 h = __float2bfloat16_rn(v * scale);
-            hi[i] = h;
-            if (lo) lo[i] = __float2bfloat16_rn(v * scale - __bfloat162float(h));
-        }
-    }
-};
 
 __device__ __forceinline__ float warp_sum(float v) {
 #pragma unroll
@@ -97,14 +58,6 @@ struct AppendParams {
     PageMap map;
     int* status;
 };
-// Block of a page of sequence `seq` (index within the step), or -1 with the status bit raised if the table has none.
-__device__ __forceinline__ int table_block(const int32_t* tables, const int32_t* first_page, int max_blocks, int n_blocks, int seq, int page, int* status) {
-    const int i = page - (first_page ? first_page[seq] : 0);
-    const int blk = i >= 0 && i < max_blocks ? tables[(size_t)seq * max_blocks + i] : -1;
-    if (blk >= 0 && blk < n_blocks) return blk;
-    atomicOr(status, kDevErrBlockRange);
-    return -1;
-}
 constexpr int kAppendThreads = 256;
 template <typename T>
 __global__ void __launch_bounds__(kAppendThreads) shared_kv_append_kernel(const AppendParams p) {
@@ -154,21 +107,6 @@ __global__ void __launch_bounds__(kAppendThreads) shared_kv_append_kernel(const 
     }
     if (threadIdx.x == 0) p.inv_rms[(size_t)blk * kBlockTokens + slot] = ik;
 }
-
-struct AttendParams {
-    ingot_step st;
-    const void* q;
-    const void* rows;
-    const float* inv_rms;
-    const int32_t *tables, *first_page;
-    int max_blocks, n_blocks, n_head, n_head_kv, dim, out_dim;
-    PageMap map;
-    float scale;
-    SharedOut out;
-    int* status;
-    int n_splits;   // decoding: CTAs per (token, KV head) over the keys
-    float* part;    // [token][head][split][dim + 2]
-};
 
 // ---- plain form: f32 arithmetic on the FMA pipes, any row length up to 512, f32 or f16 rows -------------------------
 // A CTA owns 16 (token, head) rows of one KV head - 4 per warp - and walks the visible keys 32 at a time through shared
@@ -702,6 +640,11 @@ int ingot_skv_attend(ingot_skv* kv, int layer, const ingot_step* step, const voi
                       SharedOut{out->f32, static_cast<__nv_bfloat16*>(out->hi), static_cast<__nv_bfloat16*>(out->lo), out->ld, out_scale}, kv->status_dev, 1, nullptr};
     cudaStream_t s = static_cast<cudaStream_t>(stream);
     if (kv->dtype == INGOT_F32) return launch_plain<float>(p, s);
+    // portions of prompts over rows of 128 values: the tcgen05 kernel, from 256 (token, head) rows per KV head on
+    if (kv->dim == 128 && (impl == 3 || (impl == 0 && (long long)step->max_len * (n_head / kv->n_head_kv) >= 256))) {
+        const int rc = launch_shared_kv_sm100(kv, layer, p, s);
+        if (rc != INGOT_ERR_UNSUPPORTED || impl == 3) return rc;
+    }
     if (impl != 1) switch (kv->dim) {
         case 32: return launch_mma<32>(kv, p, s);
         case 64: return launch_mma<64>(kv, p, s);

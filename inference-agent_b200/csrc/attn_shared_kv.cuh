@@ -1,0 +1,73 @@
+// Shared by the kernels of the shared-row attention (attn_shared_kv.cu, attn_shared_kv_sm100.cu): the cache handle, the
+// page arithmetic and the launch parameters.
+#pragma once
+
+#include <cuda_bf16.h>
+
+#include "attn_common.cuh"
+#include "ingot_internal.cuh"
+
+struct ingot_skv {
+    int device = 0, num_sms = 0;
+    int n_layer = 0, n_head_kv = 0, dim = 0;  // dim: row length (padded head size)
+    int dtype = INGOT_F32, chunk = 0, n_blocks = 0;
+    size_t layer_elems = 0;
+    void* rows = nullptr;
+    float* inv_rms = nullptr;  // [layer][block][16]
+    int* status_dev = nullptr;
+    float* part = nullptr;  // split-key partials of decoded tokens, grown on demand
+    size_t part_floats = 0;
+    std::vector<void*> retired;
+    std::vector<CUtensorMap> tmaps;  // per layer, 128-value f16 rows only: [page * kv head][16][128] in boxes of 16 x 64
+};
+
+struct PageMap {
+    int chunk, pages_per_chunk;  // chunk 0: one chunk of unlimited length
+    __host__ __device__ __forceinline__ int page(int pos) const { return chunk > 0 ? (pos / chunk) * pages_per_chunk + (pos % chunk) / kBlockTokens : pos / kBlockTokens; }
+    __host__ __device__ __forceinline__ int slot(int pos) const { return (chunk > 0 ? pos % chunk : pos) % kBlockTokens; }
+    __host__ __device__ __forceinline__ int first_visible(int pos) const { return chunk > 0 ? pos / chunk * chunk : 0; }
+};
+
+struct SharedOut {
+    float* f32;
+    __nv_bfloat16 *hi, *lo;
+    int ld;
+    float scale;
+    __device__ __forceinline__ void store(size_t row, int c, float v) const {
+        const size_t i = row * ld + c;
+        if (f32) f32[i] = v * scale;
+        if (hi) {
+            const __nv_bfloat16 h = __float2bfloat16_rn(v * scale);
+            hi[i] = h;
+            if (lo) lo[i] = __float2bfloat16_rn(v * scale - __bfloat162float(h));
+        }
+    }
+};
+
+// Block of a page of sequence `seq` (index within the step), or -1 with the status bit raised if the table has none.
+__device__ __forceinline__ int table_block(const int32_t* tables, const int32_t* first_page, int max_blocks, int n_blocks, int seq, int page, int* status) {
+    const int i = page - (first_page ? first_page[seq] : 0);
+    const int blk = i >= 0 && i < max_blocks ? tables[(size_t)seq * max_blocks + i] : -1;
+    if (blk >= 0 && blk < n_blocks) return blk;
+    atomicOr(status, kDevErrBlockRange);
+    return -1;
+}
+
+struct AttendParams {
+    ingot_step st;
+    const void* q;
+    const void* rows;
+    const float* inv_rms;
+    const int32_t *tables, *first_page;
+    int max_blocks, n_blocks, n_head, n_head_kv, dim, out_dim;
+    PageMap map;
+    float scale;  // of the scores
+    SharedOut out;
+    int* status;
+    int n_splits;   // decoding: CTAs per (token, KV head) over the keys
+    float* part;    // [token][head][split][dim + 2]
+};
+
+// tcgen05 form for portions of prompts over rows of 128 values (attn_shared_kv_sm100.cu); INGOT_ERR_UNSUPPORTED if the driver
+// cannot encode its tensor map.
+int launch_shared_kv_sm100(ingot_skv* kv, int layer, const AttendParams& p, cudaStream_t stream);

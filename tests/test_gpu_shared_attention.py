@@ -93,7 +93,7 @@ SHAPES = [(6, 1, 64, 48), (4, 4, 24, 40), (8, 2, 128, 0), (12, 3, 20, 33), (16, 
 
 @pytest.mark.parametrize("cut", CUTS)
 @pytest.mark.parametrize("heads,kv_heads,dim,chunk", SHAPES)
-@pytest.mark.parametrize("dtype,impl", [(F32, 0), (F16, 1), (F16, 0)])
+@pytest.mark.parametrize("dtype,impl", [(F32, 0), (F16, 1), (F16, 2), (F16, 0)])
 def test_against_plain_attention(heads, kv_heads, dim, chunk, cut, dtype, impl):
     rng = np.random.default_rng(heads * dim)
     wq, wk = 1 + 0.3 * rng.standard_normal(heads * dim), 1 + 0.3 * rng.standard_normal(kv_heads * dim)
@@ -105,7 +105,7 @@ def test_against_plain_attention(heads, kv_heads, dim, chunk, cut, dtype, impl):
 
 
 @pytest.mark.parametrize("decoded", [False, True])
-@pytest.mark.parametrize("dtype,impl", [(F32, 0), (F16, 1), (F16, 0)])
+@pytest.mark.parametrize("dtype,impl", [(F32, 0), (F16, 1), (F16, 2), (F16, 0)])
 def test_a_key_that_stands_out_is_seen_up_to_the_chunks_edge_and_not_beyond(dtype, impl, decoded):
     """One query matches one key so strongly that it takes all the weight if it is visible; the key sits at the first and at the
     last place of a chunk, at page borders, and the query just inside and just outside."""
@@ -123,6 +123,20 @@ def test_a_key_that_stands_out_is_seen_up_to_the_chunks_edge_and_not_beyond(dtyp
         seen = key // chunk == query // chunk
         assert (got[query, 0] > 0.9 * OUT_SCALE * 6) == seen, (key, query)
         assert np.abs(got - want).max() < (2e-5 if dtype == F32 else 2e-2)
+
+
+@pytest.mark.parametrize("heads,kv_heads,dim,chunk", [(8, 2, 128, 0), (4, 4, 112, 96), (6, 1, 128, 200), (16, 2, 100, 33), (3, 1, 126, 1000)])
+def test_tcgen05_kernel(heads, kv_heads, dim, chunk):
+    """Rows of 128 values on the tcgen05 kernel: several row tiles, unequal sequences, portions that start inside chunks and
+    pages, single tokens beside long portions."""
+    rng = np.random.default_rng(heads + dim)
+    wq, wk = 1 + 0.3 * rng.standard_normal(heads * dim), 1 + 0.3 * rng.standard_normal(kv_heads * dim)
+    seqs = [(rng.standard_normal((n, heads * dim)), 2 * rng.standard_normal((n, kv_heads * dim))) for n in (700, 300, 5)]
+    for cuts in ([[10 ** 9]] * 3, [[133, 1, 300], [7, 90, 1], [1]]):
+        got = run(seqs, cuts, heads, kv_heads, dim, chunk, F16, wq, wk, 3)
+        for (q, kv), g in zip(seqs, got):
+            want = reference(q, kv, wq, wk, heads, kv_heads, dim, chunk)
+            assert np.abs(g - want).max() < 8e-3, np.abs(g - want).max()
 
 
 def test_a_table_entry_outside_the_pool_is_reported():
