@@ -302,7 +302,8 @@ typedef struct ingot_act_out {
 } ingot_act_out;
 
 /* Per-channel causal convolution with carried history:
- *   out[t][c] = act(bias[c] + sum_j w[c][j] (in[t - (taps-1) + j][c] + in_bias[c])), zeros before position 0; act: silu or none.
+ *   out[t][c] = act(bias[c] + sum_j w[c][j] (in[t - (taps-1) + j][c] + in_bias[c])), zeros before position 0; act: none (silu 0), silu (1), or
+ * silu from the hardware 2^x unit (2).
  * state_dev [slot][taps-1][channels]: the last taps-1 inputs (in + in_bias), oldest first; read and replaced. 1 <= taps <= 16.
  * in rows are in_ld floats apart; in_bias and bias may be null. */
 int ingot_causal_conv(const ingot_step* step, const float* in_dev, int in_ld, const float* in_bias_dev, const float* w_dev,
@@ -315,7 +316,7 @@ int ingot_scan_state_pad(int n_state);
  *   S[c][n] <- exp(dt A[c][n]) S[c][n] + dt x[c] B[n];  y[c] = sum_n S[c][n] C[n] + D[c] x[c];  out[c] = y[c] * silu(z[c]).
  * a_log2e_dev [inner][pad] = A * log2(e), zeros in the padding; B and C are the n_state columns at b_off / c_off of the rows of
  * bc_dev (pad columns are read, the ones beyond n_state must be finite). state_dev [slot][inner][pad] f32, read and replaced.
- * exact: decays through expm1 instead of the hardware 2^x (see csrc/recurrent.cu).
+ * exact: decays through expm1, softplus and silu from expf / log1pf, instead of the hardware 2^x (see csrc/recurrent.cu).
  * Scratch: n_chunks * inner * (pad + 1) floats. inner, row lengths and offsets are multiples of 4. */
 int ingot_selective_scan(const ingot_step* step, const ingot_scan_plan* plan, const float* x_dev, int x_ld, const float* dt_dev,
                          int dt_ld, const float* dt_bias_dev, const float* bc_dev, int bc_ld, int b_off, int c_off,
@@ -326,11 +327,11 @@ int ingot_selective_scan(const ingot_step* step, const ingot_scan_plan* plan, co
  *   r = sigmoid(g_r + r_bias), i = sigmoid(g_i + i_bias), log a = -8 r softplus(lam),
  *   S <- a S + sqrt(1 - a^2) i u;  out = out_scale * S * gelu_tanh(y + y_bias).
  * gates_dev rows hold, for each block of `block` channels, its g_r and then its g_i. state_dev [slot][width] f32, read and
- * replaced. Scratch: 2 * n_chunks * width floats. */
+ * replaced. exact: activations from expf / tanhf instead of the hardware 2^x unit. Scratch: 2 * n_chunks * width floats. */
 int ingot_gated_lru(const ingot_step* step, const ingot_scan_plan* plan, const float* u_dev, int u_ld, const float* gates_dev,
                     int gates_ld, int block, const float* r_bias_dev, const float* i_bias_dev, const float* softplus_lam_dev,
                     const float* y_dev, int y_ld, const float* y_bias_dev, float* state_dev, int width, float out_scale,
-                    const ingot_act_out* out, void* stream);
+                    int exact, const ingot_act_out* out, void* stream);
 
 /* Shared-row cache: one row per token and KV head is key and value at once (the value is the projection itself, the key the
  * projection normalised over all KV heads), paged in 16-position blocks, with causal or chunk-local visibility.

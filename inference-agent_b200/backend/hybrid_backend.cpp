@@ -367,7 +367,7 @@ public:
         const int ld_bc = rank_p_ + 2 * np_;
         ops.norm_project(s, xz, w_in_, norm);
         const ingot_act_out conv = ops.operand(s, xc, ip_, true);
-        ingot_check(ingot_causal_conv(&s.st, xz, 2 * ip_, nullptr, conv_w_, conv_b_, taps_, ip_, 1, conv_state_, &conv, ops.stream));
+        ingot_check(ingot_causal_conv(&s.st, xz, 2 * ip_, nullptr, conv_w_, conv_b_, taps_, ip_, ops.opt.f32 ? 1 : 2, conv_state_, &conv, ops.stream));
         ops.operand_ready(s, ip_);
         ops.project(s, dbc, w_x_, xc, ip_);
         ops.project_rows(s, dt, w_dt_, dbc, ld_bc, 2);
@@ -377,7 +377,7 @@ public:
         ops.operand_ready(s, ip_);
         ops.project_residual(s, w_o_, ops.buf(kMix), next_norm);
     }
-    int scan_threads() const override { return ip_ * 4; }
+    int scan_threads() const override { return ip_ * 2; }
     size_t scan_scratch_per_chunk() const override { return size_t(ip_) * (np_ + 1); }
 
 private:
@@ -472,7 +472,7 @@ public:
         if (right.hi) right.hi = static_cast<char*>(right.hi) + size_t(attn_cols_) * 2;
         if (right.lo) right.lo = static_cast<char*>(right.lo) + size_t(attn_cols_) * 2;
         ingot_check(ingot_gated_lru(&s.st, &s.lru, u, wp_, gates, 2 * wp_, block_, r_b_, i_b_, softplus_lam_, proj + y_off_, proj_ld_, y_b_, state_, wp_,
-                                    right_scale_, &right, ops.stream));
+                                    right_scale_, ops.opt.f32 ? 1 : 0, &right, ops.stream));
         ops.operand_ready(s, mix_ld_);
         ops.project_residual(s, w_o_, mix, next_norm);
     }

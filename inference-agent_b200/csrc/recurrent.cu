@@ -31,6 +31,18 @@ __device__ __forceinline__ float ex2f(float x) {
 __device__ __forceinline__ float sigmoidf(float z) { return 1.0f / (1.0f + expf(-z)); }
 __device__ __forceinline__ float siluf(float z) { return z / (1.0f + expf(-z)); }
 __device__ __forceinline__ float softplusf(float z) { return z > 20.0f ? z + log1pf(expf(-z)) : log1pf(expf(z)); }
+// The same from the hardware 2^x, lg2 and reciprocal units: about 1e-6 relative, for the 16-bit form.
+__device__ __forceinline__ float fast_sigmoid(float z) { return __fdividef(1.0f, 1.0f + ex2f(-1.44269504f * z)); }
+__device__ __forceinline__ float fast_silu(float z) { return __fdividef(z, 1.0f + ex2f(-1.44269504f * z)); }
+// max(z, 0) + log(1 + t) with t = exp(-|z|); for small t the series t - t^2/2 + t^3/3 - ..., where 1 + t would round t away
+__device__ __forceinline__ float fast_softplus(float z) {
+    const float t = ex2f(-1.44269504f * fabsf(z));
+    const float series = t * fmaf(t, fmaf(t, fmaf(t, fmaf(t, fmaf(t, fmaf(t, 1.f / 7.f, -1.f / 6.f), 0.2f), -0.25f), 1.f / 3.f), -0.5f), 1.f);
+    return fmaxf(z, 0.f) + (t < 0.125f ? series : __logf(1.0f + t));
+}
+__device__ __forceinline__ float fast_gelu_tanh(float z) {  // 0.5 (1 + tanh(v)) = sigmoid(2 v)
+    return z * fast_sigmoid(1.5957691216f * (z + 0.044715f * z * z * z));
+}
 __device__ __forceinline__ float gelu_tanhf(float z) { return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z))); }
 
 // An f32 result as the next product's operand: f32 rows, and / or one bf16 plane, or a bf16 hi + lo pair.
@@ -118,7 +130,7 @@ __global__ void __launch_bounds__(128) causal_conv_kernel(const ConvParams p) {
 #pragma unroll
         for (int j = 0; j < kH; j++)
             if (j == taps - 1) acc = fmaf(w[j], x, acc);
-        p.out.store(row0 + t, c, p.silu ? siluf(acc) : acc);
+        p.out.store(row0 + t, c, p.silu == 0 ? acc : p.silu == 1 ? siluf(acc) : fast_silu(acc));
 #pragma unroll
         for (int j = 0; j + 1 < kH; j++) h[j] = j < taps - 2 ? h[j + 1] : x;
     }
@@ -133,9 +145,68 @@ __global__ void __launch_bounds__(128) causal_conv_kernel(const ConvParams p) {
     }
 }
 
+// The same for 2 to 4 taps and four channels per thread (channels and row lengths multiples of 4): inputs of four tokens are
+// requested together.
+template <int kTaps>
+__global__ void __launch_bounds__(128) causal_conv4_kernel(const ConvParams p) {
+    INGOT_PDL_TRIGGER();
+    INGOT_PDL_WAIT();
+    const int seq = blockIdx.z, c = (blockIdx.x * 128 + threadIdx.x) * 4;
+    const int len = p.st.len[seq], t0 = blockIdx.y * kConvRun;
+    if (c >= p.channels || t0 >= len) return;
+    const int pos0 = p.st.pos0[seq];
+    const size_t row0 = p.st.row_start[seq];
+    const float* in = p.raw + row0 * p.raw_ld + c;
+    float* slot = p.state + (size_t)p.st.slot[seq] * (kTaps - 1) * p.channels + c;
+    const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
+    const float4 ib = p.in_bias ? *reinterpret_cast<const float4*>(p.in_bias + c) : zero, b = p.bias ? *reinterpret_cast<const float4*>(p.bias + c) : zero;
+    auto add = [](float4 a, float4 v) { return make_float4(a.x + v.x, a.y + v.y, a.z + v.z, a.w + v.w); };
+    auto input = [&](int t) -> float4 {
+        if (t >= 0) return add(*reinterpret_cast<const float4*>(in + (size_t)t * p.raw_ld), ib);
+        return pos0 + t >= 0 ? *reinterpret_cast<const float4*>(slot + (size_t)(kTaps - 1 + t) * p.channels) : zero;
+    };
+    float w[4][kTaps];
+#pragma unroll
+    for (int e = 0; e < 4; e++)
+#pragma unroll
+        for (int j = 0; j < kTaps; j++) w[e][j] = p.w[(size_t)(c + e) * kTaps + j];
+    float4 h[kTaps + 3];  // inputs t - (taps-1) .. t + 3
+#pragma unroll
+    for (int j = 0; j < kTaps - 1; j++) h[j] = input(t0 - (kTaps - 1) + j);
+    const int t_end = min(len, t0 + kConvRun);
+    for (int t = t0; t < t_end; t += 4) {
+#pragma unroll
+        for (int i = 0; i < 4; i++) h[kTaps - 1 + i] = t + i < t_end ? input(t + i) : zero;
+#pragma unroll
+        for (int i = 0; i < 4; i++) {
+            if (t + i >= t_end) break;
+            float4 a = b;
+#pragma unroll
+            for (int j = 0; j < kTaps; j++) {
+                a.x = fmaf(w[0][j], h[i + j].x, a.x);
+                a.y = fmaf(w[1][j], h[i + j].y, a.y);
+                a.z = fmaf(w[2][j], h[i + j].z, a.z);
+                a.w = fmaf(w[3][j], h[i + j].w, a.w);
+            }
+            if (p.silu == 1) a = make_float4(siluf(a.x), siluf(a.y), siluf(a.z), siluf(a.w));
+            else if (p.silu == 2) a = make_float4(fast_silu(a.x), fast_silu(a.y), fast_silu(a.z), fast_silu(a.w));
+            p.out.store4(row0 + t + i, c, a);
+        }
+#pragma unroll
+        for (int j = 0; j < kTaps - 1; j++) h[j] = h[j + 4];
+    }
+    if (t0 == 0) {
+        float4 n[kTaps - 1];
+#pragma unroll
+        for (int j = 0; j < kTaps - 1; j++) n[j] = input(len - (kTaps - 1) + j);
+#pragma unroll
+        for (int j = 0; j < kTaps - 1; j++) *reinterpret_cast<float4*>(slot + (size_t)j * p.channels) = n[j];
+    }
+}
+
 // ---- selective scan -------------------------------------------------------------------------------------------------
 // Per channel c and state n: S <- exp(dt A) S + dt x B, y = sum_n S C + D x, out = y * silu(z); dt = softplus(raw + bias).
-// kLanes lanes share a channel, each holding kS of its states in registers. A CTA of 128 threads owns 128 / lanes channels
+// 4 or more lanes share two channels, each holding kS of their states in registers. A CTA of 128 threads owns 256 / lanes channels
 // over one time chunk; inputs are staged 16 tokens at a time in shared memory, the next 16 requested (cp.async) while the
 // current ones are computed.
 constexpr int kScanTile = 16;
@@ -202,7 +273,8 @@ __device__ __forceinline__ void load_pairs(const float* p, f32x2 (&v)[kS / 2]) {
     }
 }
 
-// kLg: log2 of the lanes per channel, or -1 for p.lanes_log2
+// kLg: log2 of the lanes per pair of channels, or -1 for p.lanes_log2. A thread holds the same kS states of two neighbouring
+// channels, so that every B and C value it fetches from shared memory is used twice.
 template <int kS, bool kOutput, int kLg, bool kExact>
 __global__ void __launch_bounds__(128) selective_scan_kernel(const ScanParams p) {
     extern __shared__ __align__(16) float smem[];
@@ -213,10 +285,10 @@ __global__ void __launch_bounds__(128) selective_scan_kernel(const ScanParams p)
     const bool first = t0 == 0, last = t0 + len == p.st.len[seq];
     if (!kOutput && last) return;  // nothing follows a sequence's last chunk
     const int lg = kLg >= 0 ? kLg : p.lanes_log2;
-    const int lanes = 1 << lg, n_ch = 128 >> lg;
+    const int lanes = 1 << lg, n_ch = 256 >> lg;
     const int ch = threadIdx.x >> lg, part = threadIdx.x & (lanes - 1);
-    const int c_base = blockIdx.x * n_ch, c = c_base + ch;
-    const bool live = c < p.inner;
+    const int c_base = blockIdx.x * n_ch, c = c_base + 2 * ch;
+    const bool live = c < p.inner;  // the channel count is even
     const size_t row0 = (size_t)p.st.row_start[seq] + t0;
     const int np = p.n_pad;
 
@@ -255,7 +327,7 @@ __global__ void __launch_bounds__(128) selective_scan_kernel(const ScanParams p)
     const int n_tiles = (len + kScanTile - 1) / kScanTile;
     stage(0);
 
-    f32x2 a[kS / 2], s[kS / 2];
+    f32x2 a[2][kS / 2], s[2][kS / 2];
     const size_t sidx = (size_t)(live ? c : 0) * np + part * kS;
     const size_t slot_base = (size_t)p.st.slot[seq] * p.inner * np;
     {
@@ -266,17 +338,19 @@ __global__ void __launch_bounds__(128) selective_scan_kernel(const ScanParams p)
         if (kOutput && !(first && last)) from = p.part + (size_t)chunk * p.inner * np + sidx;
         else if (first && p.st.pos0[seq] > 0) from = p.state + slot_base + sidx;
 #pragma unroll
-        for (int i = 0; i < kS / 2; i++) {
-            a[i] = live ? *reinterpret_cast<const f32x2*>(p.a2 + sidx + 2 * i) : 0;
-            s[i] = live && from ? *reinterpret_cast<const f32x2*>(from + 2 * i) : 0;
-        }
+        for (int e = 0; e < 2; e++)
+#pragma unroll
+            for (int i = 0; i < kS / 2; i++) {
+                a[e][i] = live ? *reinterpret_cast<const f32x2*>(p.a2 + sidx + e * np + 2 * i) : 0;
+                s[e][i] = live && from ? *reinterpret_cast<const f32x2*>(from + e * np + 2 * i) : 0;
+            }
     }
     const int my_q = (threadIdx.x % ch4) * 4;  // the four channels this thread prepares and writes (ch4 divides 128)
     const bool my_live = c_base + my_q < p.inner;
     const float4 zero4 = make_float4(0.f, 0.f, 0.f, 0.f);
     const float4 my_bias = my_live ? *reinterpret_cast<const float4*>(p.dt_bias + c_base + my_q) : zero4;
     const float4 my_d = kOutput && my_live ? *reinterpret_cast<const float4*>(p.d + c_base + my_q) : zero4;
-    float sum_dt = 0.f;
+    float sum_dt[2] = {0.f, 0.f};
 
     for (int tile = 0; tile < n_tiles; tile++) {
         if (tile + 1 < n_tiles) { stage(tile + 1); cp_async_wait<1>(); } else { cp_async_wait<0>(); }
@@ -289,46 +363,53 @@ __global__ void __launch_bounds__(128) selective_scan_kernel(const ScanParams p)
         const int n_t = min(kScanTile, len - tile * kScanTile);
         for (int i = threadIdx.x; i < n_t * ch4; i += 128) {
             const float4 raw = reinterpret_cast<const float4*>(sdt)[i], xv = reinterpret_cast<const float4*>(sx)[i];
-            const float4 dt = make_float4(softplusf(raw.x + my_bias.x), softplusf(raw.y + my_bias.y), softplusf(raw.z + my_bias.z), softplusf(raw.w + my_bias.w));
+            auto sp = [](float v) { return kExact ? softplusf(v) : fast_softplus(v); };
+            const float4 dt = make_float4(sp(raw.x + my_bias.x), sp(raw.y + my_bias.y), sp(raw.z + my_bias.z), sp(raw.w + my_bias.w));
             reinterpret_cast<float4*>(sdt)[i] = dt;
             reinterpret_cast<float4*>(s_dtx)[i] = make_float4(dt.x * xv.x, dt.y * xv.y, dt.z * xv.z, dt.w * xv.w);
         }
         __syncthreads();
         auto token = [&](int t) {
-            const float dt = sdt[t * n_ch + ch], dtx = s_dtx[t * n_ch + ch];
+            const float2 dt = *reinterpret_cast<const float2*>(sdt + t * n_ch + 2 * ch), dtx = *reinterpret_cast<const float2*>(s_dtx + t * n_ch + 2 * ch);
             f32x2 b[kS / 2], cc[kS / 2];
             load_pairs<kS>(sb + t * np + part * kS, b);
             if (kOutput) load_pairs<kS>(sc + t * np + part * kS, cc);
-            const f32x2 dt2 = kExact ? pair(dt * 0.69314718f, dt * 0.69314718f) : pair(dt, dt), dtx2 = pair(dtx, dtx);
-            f32x2 y2 = 0;
+            float y[2];
 #pragma unroll
-            for (int i = 0; i < kS / 2; i++) {
-                const float2 x = unpair(mul2(dt2, a[i]));
-                const f32x2 in = mul2(dtx2, b[i]);
-                if (kExact) {
-                    const float2 sv = unpair(s[i]), iv = unpair(in);
-                    s[i] = pair(sv.x + fmaf(expm1f(x.x), sv.x, iv.x), sv.y + fmaf(expm1f(x.y), sv.y, iv.y));
-                } else {
-                    s[i] = fma2(pair(ex2f(x.x), ex2f(x.y)), s[i], in);
+            for (int e = 0; e < 2; e++) {
+                const float d = kExact ? (e ? dt.y : dt.x) * 0.69314718f : (e ? dt.y : dt.x);
+                const f32x2 dt2 = pair(d, d), dtx2 = e ? pair(dtx.y, dtx.y) : pair(dtx.x, dtx.x);
+                f32x2 y2 = 0;
+#pragma unroll
+                for (int i = 0; i < kS / 2; i++) {
+                    const float2 x = unpair(mul2(dt2, a[e][i]));
+                    const f32x2 in = mul2(dtx2, b[i]);
+                    if (kExact) {
+                        const float2 sv = unpair(s[e][i]), iv = unpair(in);
+                        s[e][i] = pair(sv.x + fmaf(expm1f(x.x), sv.x, iv.x), sv.y + fmaf(expm1f(x.y), sv.y, iv.y));
+                    } else {
+                        s[e][i] = fma2(pair(ex2f(x.x), ex2f(x.y)), s[e][i], in);
+                    }
+                    if (kOutput) y2 = fma2(s[e][i], cc[i], y2);
                 }
-                if (kOutput) y2 = fma2(s[i], cc[i], y2);
+                const float2 yv = unpair(y2);
+                y[e] = yv.x + yv.y;
             }
             if (kOutput) {
-                const float2 yv = unpair(y2);
-                float y = yv.x + yv.y;
-                if (kLg == 2) {
-                    y += __shfl_xor_sync(0xffffffffu, y, 2);
-                    y += __shfl_xor_sync(0xffffffffu, y, 1);
-                } else {
-                    for (int o = lanes >> 1; o > 0; o >>= 1) y += __shfl_xor_sync(0xffffffffu, y, o);
-                }
-                if (part == 0) s_y[t * n_ch + ch] = y;
+                // the first exchange halves the work: the upper lanes of a group go on with the second channel only
+                const bool upper = part & (lanes >> 1);
+                float v = upper ? y[1] : y[0];
+                v += __shfl_xor_sync(0xffffffffu, upper ? y[0] : y[1], lanes >> 1);
+                if (kLg == 2) v += __shfl_xor_sync(0xffffffffu, v, 1);
+                else for (int o = lanes >> 2; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
+                if ((part & ((lanes >> 1) - 1)) == 0) s_y[t * n_ch + 2 * ch + (upper ? 1 : 0)] = v;
             } else {
-                sum_dt += dt;
+                sum_dt[0] += dt.x;
+                sum_dt[1] += dt.y;
             }
         };
         if (n_t == kScanTile) {
-#pragma unroll 8
+#pragma unroll 4
             for (int t = 0; t < kScanTile; t++) token(t);
         } else {
             for (int t = 0; t < n_t; t++) token(t);
@@ -340,21 +421,25 @@ __global__ void __launch_bounds__(128) selective_scan_kernel(const ScanParams p)
                     const size_t row = row0 + tile * kScanTile + i / ch4;
                     const float4 xv = reinterpret_cast<const float4*>(sx)[i], yv = reinterpret_cast<const float4*>(s_y)[i],
                                  zv = reinterpret_cast<const float4*>(sz)[i];
-                    p.out.store4(row, c_base + my_q, make_float4(fmaf(my_d.x, xv.x, yv.x) * siluf(zv.x), fmaf(my_d.y, xv.y, yv.y) * siluf(zv.y),
-                                                                 fmaf(my_d.z, xv.z, yv.z) * siluf(zv.z), fmaf(my_d.w, xv.w, yv.w) * siluf(zv.w)));
+                    auto act = [](float v) { return kExact ? siluf(v) : fast_silu(v); };
+                    p.out.store4(row, c_base + my_q, make_float4(fmaf(my_d.x, xv.x, yv.x) * act(zv.x), fmaf(my_d.y, xv.y, yv.y) * act(zv.y),
+                                                                 fmaf(my_d.z, xv.z, yv.z) * act(zv.z), fmaf(my_d.w, xv.w, yv.w) * act(zv.w)));
                 }
             }
         }
         __syncthreads();  // the tile's buffers are staged over two tiles from now, s_dtx / s_y in the next one
     }
     if (!live) return;
-    if (!kOutput) {
 #pragma unroll
-        for (int i = 0; i < kS / 2; i++) *reinterpret_cast<f32x2*>(p.part + (size_t)chunk * p.inner * np + sidx + 2 * i) = s[i];
-        if (part == 0) p.part_sum[(size_t)chunk * p.inner + c] = sum_dt;
-    } else if (last) {
+    for (int e = 0; e < 2; e++) {
+        if (!kOutput) {
 #pragma unroll
-        for (int i = 0; i < kS / 2; i++) *reinterpret_cast<f32x2*>(p.state + slot_base + sidx + 2 * i) = s[i];
+            for (int i = 0; i < kS / 2; i++) *reinterpret_cast<f32x2*>(p.part + (size_t)chunk * p.inner * np + sidx + e * np + 2 * i) = s[e][i];
+            if (part == 0) p.part_sum[(size_t)chunk * p.inner + c + e] = sum_dt[e];
+        } else if (last) {
+#pragma unroll
+            for (int i = 0; i < kS / 2; i++) *reinterpret_cast<f32x2*>(p.state + slot_base + sidx + e * np + 2 * i) = s[e][i];
+        }
     }
 }
 
@@ -399,7 +484,7 @@ struct LruParams {
     float out_scale;
     ActOut out;
 };
-template <bool kOutput>
+template <bool kOutput, bool kExact>
 __global__ void __launch_bounds__(128) gated_lru_kernel(const LruParams p) {
     INGOT_PDL_TRIGGER();
     INGOT_PDL_WAIT();
@@ -418,14 +503,27 @@ __global__ void __launch_bounds__(128) gated_lru_kernel(const LruParams p) {
     const float* u = p.u + row0 * p.u_ld + c;
     const float* g = p.gates + row0 * p.gates_ld + gcol;
     const float* y = kOutput ? p.y + row0 * p.y_ld + c : nullptr;
-#pragma unroll 4
-    for (int t = 0; t < len; t++) {
-        const float log_a = k * sigmoidf(g[(size_t)t * p.gates_ld] + br);
-        const float in = sigmoidf(g[(size_t)t * p.gates_ld + p.block] + bi) * u[(size_t)t * p.u_ld];
-        const float e = expm1f(log_a);  // a - 1; 1 - a^2 = -e (2 + e)
-        s += fmaf(e, s, sqrtf(-e * (2.0f + e)) * in);
-        if (kOutput) p.out.store(row0 + t, c, p.out_scale * s * gelu_tanhf(y[(size_t)t * p.y_ld] + yb));
-        else sum += log_a;
+    constexpr int kAhead = 8;  // tokens whose inputs are requested together
+    for (int tb = 0; tb < len; tb += kAhead) {
+        float gr[kAhead], gi[kAhead], uv[kAhead], yv[kAhead];
+#pragma unroll
+        for (int i = 0; i < kAhead; i++) {
+            const size_t t = min(tb + i, len - 1);
+            gr[i] = g[t * p.gates_ld];
+            gi[i] = g[t * p.gates_ld + p.block];
+            uv[i] = u[t * p.u_ld];
+            if (kOutput) yv[i] = y[t * p.y_ld];
+        }
+#pragma unroll
+        for (int i = 0; i < kAhead; i++) {
+            if (tb + i >= len) break;
+            const float log_a = k * (kExact ? sigmoidf(gr[i] + br) : fast_sigmoid(gr[i] + br));
+            const float in = (kExact ? sigmoidf(gi[i] + bi) : fast_sigmoid(gi[i] + bi)) * uv[i];
+            const float e = expm1f(log_a);  // a - 1; 1 - a^2 = -e (2 + e)
+            s += fmaf(e, s, sqrtf(-e * (2.0f + e)) * in);
+            if (kOutput) p.out.store(row0 + tb + i, c, p.out_scale * s * (kExact ? gelu_tanhf(yv[i] + yb) : fast_gelu_tanh(yv[i] + yb)));
+            else sum += log_a;
+        }
     }
     if (!kOutput) {
         p.part[(size_t)chunk * p.width + c] = s;
@@ -483,9 +581,11 @@ int ingot_causal_conv(const ingot_step* step, const float* in_dev, int in_ld, co
     INGOT_REQUIRE(step_ok(step) && in_dev && w_dev && state_dev && out, "ingot_causal_conv: null argument or empty step");
     INGOT_REQUIRE(channels >= 1 && taps >= 1 && taps <= kMaxTaps, "ingot_causal_conv: between 1 and 16 taps");
     ConvParams p = {*step, in_dev, in_ld, in_bias_dev, w_dev, bias_dev, taps, channels, silu, state_dev, act_out(out)};
-    const dim3 grid((channels + 127) / 128, (step->max_len + kConvRun - 1) / kConvRun, step->n_seq);
+    const bool four = taps >= 2 && taps <= 4 && channels % 4 == 0 && in_ld % 4 == 0 && out->ld % 4 == 0;
+    const dim3 grid(four ? (channels + 511) / 512 : (channels + 127) / 128, (step->max_len + kConvRun - 1) / kConvRun, step->n_seq);
     INGOT_REQUIRE(grid.y <= 65535, "ingot_causal_conv: too many tokens of one sequence in one step");
-    auto kernel = taps == 2 ? causal_conv_kernel<2> : taps == 3 ? causal_conv_kernel<3> : taps == 4 ? causal_conv_kernel<4> : causal_conv_kernel<0>;
+    auto kernel = four ? (taps == 2 ? causal_conv4_kernel<2> : taps == 3 ? causal_conv4_kernel<3> : causal_conv4_kernel<4>)
+                       : taps == 2 ? causal_conv_kernel<2> : taps == 3 ? causal_conv_kernel<3> : taps == 4 ? causal_conv_kernel<4> : causal_conv_kernel<0>;
     INGOT_CUDA_TRY(ingot_launch_pdl(kernel, grid, dim3(128), 0, static_cast<cudaStream_t>(stream), p));
     return INGOT_OK;
 }
@@ -508,7 +608,7 @@ int ingot_selective_scan(const ingot_step* step, const ingot_scan_plan* plan, co
     const bool multi = plan->max_chunks > 1;
     INGOT_REQUIRE(!multi || (plan->scratch_dev && plan->scratch_floats >= (size_t)plan->n_chunks * inner * (n_pad + 1)),
                   "ingot_selective_scan: scratch too small");
-    const int lg = scan_lanes_log2(n_state), n_ch = 128 >> lg;
+    const int lg = scan_lanes_log2(n_state), n_ch = 256 >> lg;
     const int per_lane = scan_states_per_lane(n_state);
     ScanParams p = {*step, plan->chunk_seq, plan->chunk_t0, plan->chunk_len, plan->seq_chunk0, plan->n_chunks,
                     x_dev, x_ld, dt_dev, dt_ld, dt_bias_dev, bc_dev, bc_ld, b_off, c_off, z_dev, z_ld, a_log2e_dev, d_dev,
@@ -548,7 +648,7 @@ int ingot_selective_scan(const ingot_step* step, const ingot_scan_plan* plan, co
 int ingot_gated_lru(const ingot_step* step, const ingot_scan_plan* plan, const float* u_dev, int u_ld, const float* gates_dev,
                     int gates_ld, int block, const float* r_bias_dev, const float* i_bias_dev, const float* softplus_lam_dev,
                     const float* y_dev, int y_ld, const float* y_bias_dev, float* state_dev, int width, float out_scale,
-                    const ingot_act_out* out, void* stream) {
+                    int exact, const ingot_act_out* out, void* stream) {
     INGOT_REQUIRE(step_ok(step) && plan_ok(plan), "ingot_gated_lru: bad step or plan");
     INGOT_REQUIRE(u_dev && gates_dev && r_bias_dev && i_bias_dev && softplus_lam_dev && y_dev && y_bias_dev && state_dev && out, "ingot_gated_lru: null argument");
     INGOT_REQUIRE(width >= 1 && block >= 1 && width % block == 0, "ingot_gated_lru: the width must be a multiple of the block size");
@@ -560,10 +660,10 @@ int ingot_gated_lru(const ingot_step* step, const ingot_scan_plan* plan, const f
     cudaStream_t s = static_cast<cudaStream_t>(stream);
     const dim3 grid((width + 127) / 128, plan->n_chunks);
     if (multi) {
-        INGOT_CUDA_TRY(ingot_launch_pdl(gated_lru_kernel<false>, grid, dim3(128), 0, s, p));
+        INGOT_CUDA_TRY(ingot_launch_pdl(exact ? gated_lru_kernel<false, true> : gated_lru_kernel<false, false>, grid, dim3(128), 0, s, p));
         INGOT_CUDA_TRY(ingot_launch_pdl(gated_lru_link_kernel, dim3((width + 127) / 128, step->n_seq), dim3(128), 0, s, p));
     }
-    INGOT_CUDA_TRY(ingot_launch_pdl(gated_lru_kernel<true>, grid, dim3(128), 0, s, p));
+    INGOT_CUDA_TRY(ingot_launch_pdl(exact ? gated_lru_kernel<true, true> : gated_lru_kernel<true, false>, grid, dim3(128), 0, s, p));
     return INGOT_OK;
 }
 

@@ -55,7 +55,7 @@ ABI = {
     "ingot_causal_conv": (_I, [_P, _P, _I, _P, _P, _P, _I, _I, _I, _P, _P, _P]),
     "ingot_scan_state_pad": (_I, [_I]),
     "ingot_selective_scan": (_I, [_P, _P, _P, _I, _P, _I, _P, _P, _I, _I, _I, _P, _I, _P, _P, _P, _I, _I, _I, _P, _P]),
-    "ingot_gated_lru": (_I, [_P, _P, _P, _I, _P, _I, _I, _P, _P, _P, _P, _I, _P, _P, _I, C.c_float, _P, _P]),
+    "ingot_gated_lru": (_I, [_P, _P, _P, _I, _P, _I, _I, _P, _P, _P, _P, _I, _P, _P, _I, C.c_float, _I, _P, _P]),
     "ingot_skv_create": (_I, [C.POINTER(_P), _I, _I, _I, _I, _I, _I]),
     "ingot_skv_destroy": (None, [_P]),
     "ingot_skv_pages": (_I, [_I, _I]),

@@ -27,9 +27,10 @@ def run_in_portions(cuts, lens, call):
 CUTS = {"whole": [[10 ** 9]], "portions": [[2, 17, 1, 40], [33, 3], [5]], "single": [[1]]}
 
 
+@pytest.mark.parametrize("act", [1, 2])
 @pytest.mark.parametrize("cut", CUTS)
 @pytest.mark.parametrize("taps,channels", [(4, 200), (2, 64), (3, 130), (1, 24), (7, 40)])
-def test_causal_conv(taps, channels, cut):
+def test_causal_conv(taps, channels, cut, act):
     import torch
     rng = np.random.default_rng(taps)
     lens, slots = [61, 37, 5], [3, 0, 2]
@@ -49,7 +50,7 @@ def test_causal_conv(taps, channels, cut):
         x = dev(rows)
         out, hi, lo = (torch.zeros(st.n_tok, channels, device="cuda", dtype=t) for t in (torch.float32, torch.bfloat16, torch.bfloat16))
         o = act_out(out, hi, lo)
-        lib(lib().ingot_causal_conv(C.byref(st.c), x.data_ptr(), ld, ibd.data_ptr(), wd.data_ptr(), bd.data_ptr(), taps, channels, 1,
+        lib(lib().ingot_causal_conv(C.byref(st.c), x.data_ptr(), ld, ibd.data_ptr(), wd.data_ptr(), bd.data_ptr(), taps, channels, act,
                                     state.data_ptr(), C.byref(o), None))
         torch.cuda.synchronize()
         assert torch.equal(hi, out.bfloat16()) and torch.equal(lo, (out - hi.float()).bfloat16())
@@ -109,9 +110,10 @@ def test_selective_scan(inner, n_state, cut, exact):
         assert np.abs(g - e).max() < 3e-5 * max(1.0, np.abs(e).max())
 
 
+@pytest.mark.parametrize("exact", [0, 1])
 @pytest.mark.parametrize("cut", CUTS)
 @pytest.mark.parametrize("width,block", [(96, 24), (200, 200), (24, 8)])
-def test_gated_lru(width, block, cut):
+def test_gated_lru(width, block, cut, exact):
     import torch
     rng = np.random.default_rng(width)
     lens, slots = [90, 33, 4], [2, 1, 3]
@@ -134,7 +136,7 @@ def test_gated_lru(width, block, cut):
         pl = plan(part, 16, 2 * width)
         lib(lib().ingot_gated_lru(C.byref(st.c), C.byref(pl.c), ud.data_ptr(), width, gd.data_ptr(), 2 * width, block, dv[0].data_ptr(),
                                   dv[1].data_ptr(), dv[2].data_ptr(), yd.data_ptr(), width, dv[3].data_ptr(), state.data_ptr(), width, 0.75,
-                                  C.byref(o), None))
+                                  exact, C.byref(o), None))
         torch.cuda.synchronize()
         r = 0
         for i, p, n in zip(live, pos0, part):
