@@ -458,10 +458,21 @@ __global__ void __launch_bounds__(256) selective_scan_link_kernel(const ScanPara
     float end = p.part[(size_t)k0 * per + i];
     p.part[(size_t)k0 * per + i] = s;
     s = end;
-    for (int k = k0 + 1; k < k1; k++) {
-        end = p.part[(size_t)k * per + i];
-        p.part[(size_t)k * per + i] = s;
-        s = fmaf(ex2f(a * p.part_sum[(size_t)k * p.inner + c]), s, end);
+    constexpr int kAhead = 8;  // chunks whose end states are requested together
+    for (int kb = k0 + 1; kb < k1; kb += kAhead) {
+        float e[kAhead], f[kAhead];
+#pragma unroll
+        for (int j = 0; j < kAhead; j++) {
+            const int k = min(kb + j, k1 - 1);
+            e[j] = p.part[(size_t)k * per + i];
+            f[j] = p.part_sum[(size_t)k * p.inner + c];
+        }
+#pragma unroll
+        for (int j = 0; j < kAhead; j++) {
+            if (kb + j >= k1) break;
+            p.part[(size_t)(kb + j) * per + i] = s;
+            s = fmaf(ex2f(a * f[j]), s, e[j]);
+        }
     }
 }
 
@@ -542,10 +553,21 @@ __global__ void __launch_bounds__(128) gated_lru_link_kernel(const LruParams p) 
     float end = p.part[(size_t)k0 * p.width + c];
     p.part[(size_t)k0 * p.width + c] = s;
     s = end;
-    for (int k = k0 + 1; k < k1; k++) {
-        end = p.part[(size_t)k * p.width + c];
-        p.part[(size_t)k * p.width + c] = s;
-        s = fmaf(expf(p.part_sum[(size_t)k * p.width + c]), s, end);
+    constexpr int kAhead = 8;
+    for (int kb = k0 + 1; kb < k1; kb += kAhead) {
+        float e[kAhead], f[kAhead];
+#pragma unroll
+        for (int j = 0; j < kAhead; j++) {
+            const int k = min(kb + j, k1 - 1);
+            e[j] = p.part[(size_t)k * p.width + c];
+            f[j] = p.part_sum[(size_t)k * p.width + c];
+        }
+#pragma unroll
+        for (int j = 0; j < kAhead; j++) {
+            if (kb + j >= k1) break;
+            p.part[(size_t)(kb + j) * p.width + c] = s;
+            s = fmaf(expf(f[j]), s, e[j]);
+        }
     }
 }
 
