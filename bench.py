@@ -1,7 +1,7 @@
 #!/usr/bin/env python
 """Benchmark of the B200 attention path: decode KV-cache HBM GB/s and causal-prefill TFLOP/s.
 
-    python bench.py --gpus N --steps K --warmup W [--workload decode_c2|prefill_c5|c1_prefill128|c3_chunked|c4_batched|e2e_model]
+    python bench.py --gpus N --steps K --warmup W [--workload decode_c2|prefill_c5|c1_prefill128|c3_chunked|c4_batched|e2e_model|hybrid_layers]
                     [--impl reference]
 
 Headline (`metric`/`value`): single-token decode attention at 4096 keys, 24 query / 8 KV heads,
@@ -827,6 +827,32 @@ def run_e2e_model(args):
                          "note": "single-token steps are bound by reading every weight once per token"},
             "note": "reference README (Apple M5, Metal, F16): pp128 864 tok/s, tg32 15.6 tok/s"}
 
+
+def run_hybrid_layers(args):
+    """Prefill and decode throughput of the hybrid recurrent / attention design (model folders, backend/hybrid_backend.cpp) at
+    sizes of real layers with random weights, beside this framework's Llama-shaped layers of equal width (same projection
+    kernels, f16 weights). Device time per step through the library's own step function; weights exceed the L2."""
+    import torch
+    from ingot_b200 import hybrid_bench as HB
+    torch.cuda.set_device(0)
+    hybrid = HB.run_hybrid(args.hybrid_size, reps=max(args.steps // 5, 5), work=os.environ.get("INGOT_E2E_DIR", "/tmp"))
+    llama = HB.run_llama(args.hybrid_size, reps=max(args.steps // 5, 5))
+    peaks = measured_peaks()
+    top = hybrid["prefill"][2048]
+    return {"metric": "hybrid layers, 2048-token prefill tokens/s", "value": top["tok_s"], "unit": "tok/s", "n_gpus": 1, "steps": max(args.steps // 5, 5),
+            "warmup": 3, "ms_per_step": top["ms"], "higher_is_better": True, "scaling": "weak", "vs_baseline": None,
+            "dtype": "bf16 weights, bf16 products with f32 accumulation, f32 residual, norms and states", "data": "synthetic",
+            "config": {"workload": f"{args.hybrid_size}: {HB.config(args.hybrid_size)['layers'][0]['mixer']} x 3, {HB.config(args.hybrid_size)['layers'][-1]['mixer']} "
+                                   f"with a feed-forward x 1, vocabulary {HB.VOCAB}; decode at 1024 tokens of context",
+                       "l2": "weights of a step exceed the L2"},
+            "hybrid": hybrid, "llama_layers": llama,
+            "roofline": {"bound": "tensor", "unit": "TFLOP/s", "peak": peaks["tflops_burst"], "achieved": top["tflops"],
+                         "frac": round(top["tflops"] / peaks["tflops_burst"], 4),
+                         "decode_weight_stream_frac": round(hybrid["decode"][1]["weight_gb_s"] / peaks["hbm_gbs"], 4),
+                         "llama_prefill_frac": round(llama["prefill"][2048]["tflops"] / peaks["tflops_burst"], 4),
+                         "llama_decode_weight_stream_frac": round(llama["decode"][1]["weight_gb_s"] / peaks["hbm_gbs"], 4)}}
+
+
 # ------------------------------------------------------------------------------------------------
 # CPU reference legs
 # ------------------------------------------------------------------------------------------------
@@ -929,7 +955,8 @@ def main():
     ap.add_argument("--steps", type=int, default=50)
     ap.add_argument("--warmup", type=int, default=5)
     ap.add_argument("--impl", default="ingot", choices=["ingot", "reference"])
-    ap.add_argument("--workload", default="decode_c2", choices=["decode_c2", "prefill_c5", "c1_prefill128", "c3_chunked", "c4_batched", "e2e_model"])
+    ap.add_argument("--workload", default="decode_c2", choices=["decode_c2", "prefill_c5", "c1_prefill128", "c3_chunked", "c4_batched", "e2e_model", "hybrid_layers"])
+    ap.add_argument("--hybrid-size", default="w4096", choices=["w2048", "w4096"], help="hybrid_layers: width of the layers")
     ap.add_argument("--small-model", action="store_true", help="e2e_model: 2 layers and a 32064-token vocabulary")
     ap.add_argument("--wtype", default="F16", choices=["F16", "Q8_0", "Q4_0", "Q4_1", "Q6_K"], help="e2e_model: weight type of the GGUF")
     ap.add_argument("--output-type", default=None, choices=["F16", "Q8_0", "Q4_0", "Q4_1", "Q6_K"],
@@ -959,6 +986,9 @@ def main():
 
     if args.workload == "e2e_model":
         print(json.dumps(run_e2e_model(args)), flush=True)
+        return
+    if args.workload == "hybrid_layers":
+        print(json.dumps(run_hybrid_layers(args)), flush=True)
         return
 
     start_watchdog(int(os.environ.get("WORLD_SIZE", "1")))  # before the process group comes up: its set-up can stall too

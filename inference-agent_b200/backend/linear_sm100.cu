@@ -98,6 +98,7 @@ struct GemmParams {
     int n_tok, k_steps, n_split, accumulate;
     int n_out[3], tile_end[3];
     int tiles_n, tiles_m;
+    int a_bytes;  // of one activation box: 128 rows, or fewer for a single short token tile
     uint32_t idesc;
     int rows_per_block, k_block, tiles_per_block;  // block-diagonal matrix (rows_per_block > 0, count == 1)
     int to_partial;  // write the slice(s) to `partial` even when there is only one (a consumer kernel sums them)
@@ -156,11 +157,12 @@ linear_sm100_kernel(const __grid_constant__ CUtensorMap map_hi, const __grid_con
     // Barriers and tensor memory are this CTA's own and the weights never depend on the kernel before: the W boxes of
     // the first ring stages are requested now, the activation boxes (and, under accumulate, the output) only after the
     // wait for the predecessor. A stage's barrier is armed once for all three boxes.
+    const uint32_t stage_tx = kPlanes * p.a_bytes + R::kWBytes;
     const int n_pre = min(n_it, kStages);
     if (warp_u == 0 && lane == 0) {
         for (int it = 0; it < n_pre; it++) {
             const uint32_t full = smem_u32(&bars->full[it]);
-            mbar_expect_tx(full, kStageBytes);
+            mbar_expect_tx(full, stage_tx);
             tma_load_2d(smem_base + it * kStageBytes + kOffW, map_w_p, (ks_begin + it) * kBK, n0, full);
         }
     }
@@ -182,7 +184,7 @@ linear_sm100_kernel(const __grid_constant__ CUtensorMap map_hi, const __grid_con
                 } else {
                     ok = mbar_wait(smem_u32(&bars->empty[s]), (uint32_t)(((it / kStages) & 1) ^ 1), abort_flag, kWaitLimitNs);
                     if (ok) {
-                        mbar_expect_tx(full, kStageBytes);
+                        mbar_expect_tx(full, stage_tx);
                         tma_load_2d(dst, &map_hi, a_k0 + k, m0, full);
                         if (kPlanes > 1) tma_load_2d(dst + kBoxBytes, &map_lo, a_k0 + k, m0, full);
                         tma_load_2d(dst + kOffW, map_w_p, k, n0, full);
@@ -493,6 +495,7 @@ struct ingot_linear_ws {
     bool bf16 = false;
     int n_slots = 3;
     int planes = 2;                            // of the prepared activations
+    int box_rows = 128;
     int prepared_tok = 0, prepared_in = 0;
     CUtensorMap map_hi, map_lo;
     std::map<std::tuple<const void*, int, int, int>, CUtensorMap> w_maps;  // one per weight matrix
@@ -501,7 +504,10 @@ struct ingot_linear_ws {
 // (Re)builds the activation tensor maps when the prepared shape changes.
 static cudaError_t set_prepared(ingot_linear_ws* ws, int n_in, int n_tok) {
     if (ws->prepared_tok != n_tok || ws->prepared_in != n_in) {
-        if (!make_map(&ws->map_hi, ws->hi, n_tok, n_in, 128, ws->bf16) || !make_map(&ws->map_lo, ws->lo, n_tok, n_in, 128, ws->bf16))
+        // A batch of few tokens fetches only its own rows (whole 8-row swizzle groups) of the 128 a tile has. What the other rows of
+        // the tile hold is multiplied along and never stored: rows of a product do not mix.
+        ws->box_rows = n_tok >= 128 ? 128 : (n_tok + 7) / 8 * 8;
+        if (!make_map(&ws->map_hi, ws->hi, n_tok, n_in, ws->box_rows, ws->bf16) || !make_map(&ws->map_lo, ws->lo, n_tok, n_in, ws->box_rows, ws->bf16))
             return cudaErrorUnknown;
         ws->prepared_tok = n_tok;
         ws->prepared_in = n_in;
@@ -666,6 +672,7 @@ static cudaError_t launch_gemm(ingot_linear_ws* ws, float* out, const void* cons
     const int tiles = tiles_n * tiles_m;
     p.tiles_n = tiles_n;
     p.tiles_m = tiles_m;
+    p.a_bytes = ws->box_rows * kBK * 2;
     const int k_steps = (n_in + kBK - 1) / kBK;
     // enough k slices to give every SM a CTA, at least 4 k-steps each, and no more than the slots hold
     if (to_partial && fit < 1) return cudaErrorInvalidValue;
