@@ -229,7 +229,7 @@ public:
         if (s.tc) {
             if (w.rows_per_block > 0) cuda_check(ingot_linear_tc_run_blocks(ws, out, w.data, w.n_in, w.n_out, w.rows_per_block, stream), "block projection");
             else cuda_check(ingot_linear_tc_run(ws, out, w.data, w.n_in, w.n_out, 0, stream), "projection");
-        } else if (s.st.n_tok == 1 && streams(w)) {
+        } else if (s.st.n_tok == 1 && streams(w) && w.n_out > 2048) {  // few rows: ingot_support_linear_bf16 gives each a CTA
             cuda_check(ingot_support_gemv_bf16(out, w.data, w.n_out, w.n_in, in, nullptr, 0.f, w.n_in, 0, 0, 0, stream), "projection");
         } else {
             cuda_check(ingot_support_linear_bf16(out, w.data, in, in_ld, w.n_in, w.n_out, w.rows_per_block, s.st.n_tok, 0, stream), "projection");

@@ -196,6 +196,42 @@ __global__ void __launch_bounds__(256) gemv_kernel(float* out, const W* w, const
     if (lane == 0) out[row] = accumulate ? out[row] + v : v;
 }
 
+// Few long rows: one CTA per row, all of whose threads request their share of the row (up to four loads each) before the wait
+// for the preceding kernel. A warp per row would leave most SMs without work.
+__global__ void __launch_bounds__(256) gemv_row_kernel(float* out, const __nv_bfloat16* w, const float* x, int n_in, int accumulate) {
+    asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
+    __shared__ float red[8];
+    const __nv_bfloat16* wr = w + (size_t)blockIdx.x * n_in;
+    const int i0 = threadIdx.x * 8;
+    float p[4][8];
+#pragma unroll
+    for (int j = 0; j < 4; j++)
+        if (i0 + j * 2048 < n_in) load8<__nv_bfloat16>(wr + i0 + j * 2048, p[j]);
+    asm volatile("griddepcontrol.wait;" ::: "memory");
+    float acc = 0.f;
+    auto fma8 = [&](const float (&v)[8], const float* xs) {
+        const float4 a = *reinterpret_cast<const float4*>(xs), b = *reinterpret_cast<const float4*>(xs + 4);
+        acc = fmaf(v[0], a.x, acc); acc = fmaf(v[1], a.y, acc); acc = fmaf(v[2], a.z, acc); acc = fmaf(v[3], a.w, acc);
+        acc = fmaf(v[4], b.x, acc); acc = fmaf(v[5], b.y, acc); acc = fmaf(v[6], b.z, acc); acc = fmaf(v[7], b.w, acc);
+    };
+#pragma unroll
+    for (int j = 0; j < 4; j++)
+        if (i0 + j * 2048 < n_in) fma8(p[j], x + i0 + j * 2048);
+    for (int i = i0 + 8192; i < n_in; i += 2048) {
+        float v[8];
+        load8<__nv_bfloat16>(wr + i, v);
+        fma8(v, x + i);
+    }
+    acc = warp_sum(acc);
+    if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = acc;
+    __syncthreads();
+    if (threadIdx.x == 0) {
+        float t = 0.f;
+        for (int i = 0; i < 8; i++) t += red[i];
+        out[blockIdx.x] = accumulate ? out[blockIdx.x] + t : t;
+    }
+}
+
 // Single-token products with f16 weights: a weight-streaming kernel, HBM-bound by design.
 //   out_m[r] (+)= dot(W_m[r][:], x')            x' = x, or x .* norm_w with the result scaled by
 //   rsqrt(mean(x^2) + eps) (the RMS norm of ops::rmsnorm, src/ops.cpp:227-232, folded in; the same product up to
@@ -667,6 +703,8 @@ cudaError_t launch_linear(float* out, const void* w, const float* x, int x_ld, i
     const int warps = 8;
     const W* wt = static_cast<const W*>(w);
     const XLayout xl = {x_ld, rows_per_block};
+    if (std::is_same<W, __nv_bfloat16>::value && n_tok == 1 && rows_per_block == 0 && n_out <= 2048 && n_in >= 1024)
+        return support_launch(gemv_row_kernel, dim3(n_out), dim3(256), 0, s, out, static_cast<const __nv_bfloat16*>(w), x, n_in, accumulate);
     if (n_tok == 1 && rows_per_block == 0) {
         const unsigned grid = (n_out + warps - 1) / warps;
         return support_launch(gemv_kernel<W>, dim3(grid), dim3(warps * 32), 0, s, out, wt, x, n_in, n_out, accumulate);
