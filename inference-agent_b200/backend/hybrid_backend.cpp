@@ -558,8 +558,9 @@ public:
         for (auto& g : ops_.caches) {
             g->pages_per_chunk = g->chunk > 0 ? (g->chunk + INGOT_BLOCK_TOKENS - 1) / INGOT_BLOCK_TOKENS : 0;
             // the pool holds max_tokens tokens of live sequences however they are spread over max_seqs of them
-            const long long blocks = g->chunk > 0 ? (long long)(max_ctx_ / g->chunk + max_seqs_) * g->pages_per_chunk
-                                                  : (long long)max_ctx_ / INGOT_BLOCK_TOKENS + max_seqs_;
+            // (whole chunks, and one begun chunk and one begun page per sequence)
+            const long long whole = g->chunk > 0 ? (long long)(max_ctx_ / g->chunk) * g->pages_per_chunk : 0, pages = (long long)max_ctx_ / INGOT_BLOCK_TOKENS + max_seqs_;
+            const long long blocks = g->chunk > 0 ? whole + std::min(pages, (long long)max_seqs_ * g->pages_per_chunk) : pages;
             if (blocks > (1 << 26)) throw std::runtime_error("engine: cache pool too large");
             ingot_check(ingot_skv_create(&g->kv, g->n_layer, g->kv_heads, g->dim, opt.f32 ? INGOT_F32 : INGOT_F16, g->chunk, int(blocks)));
             g->pool = BlockPool(int(blocks), max_seqs_, ingot_skv_pages(g->chunk, max_ctx_));

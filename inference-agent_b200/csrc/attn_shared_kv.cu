@@ -226,10 +226,7 @@ int launch_plain(const AttendParams& p, cudaStream_t s) {
 // ldmatrix): half the copies and half the shared memory of a K + V kernel. Tiles are 64 keys = 4 pages, fetched page by page
 // with cp.async; the key's scale (1/rms * score scale) and its position travel with the tile, and the scale multiplies the
 // f32 score.
-//   prompts  (kDecode false): 8 warps of 16 (token, head) rows each share every tile.
-//   decoding (kDecode true):  the 4 warps of a CTA share one 16-row tile (the heads of one token that read this KV head) and
-//            take one page of every tile each; their states are merged through shared memory, and the keys of a sequence may
-//            be split over CTAs whose partial results (o, m, l) a second launch merges.
+// 8 warps of 16 (token, head) rows each share every tile.
 constexpr int kTileKeys = 64;
 constexpr int kSplitKeysMin = 128;
 template <int kDim> struct MmaTile {
@@ -246,19 +243,18 @@ __device__ __forceinline__ void cp16(uint32_t dst, const void* src, bool on) {
     asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(on ? 16 : 0) : "memory");
 }
 
-template <int kDim, bool kDecode>
-__global__ void __launch_bounds__(kDecode ? 128 : 256) shared_kv_mma_kernel(const AttendParams p) {
-    constexpr int kThreads = kDecode ? 128 : 256, kWarps = kThreads / 32, kStages = kDecode ? 4 : 2;
-    constexpr int kStride = MmaTile<kDim>::kStride, kK = kDim / 16, kNt = kDecode ? 2 : 8;  // kNt: 8-key groups a warp scores per tile
+template <int kDim>
+__global__ void __launch_bounds__(256) shared_kv_mma_kernel(const AttendParams p) {
+    constexpr int kThreads = 256, kWarps = kThreads / 32, kStages = 2;
+    constexpr int kStride = MmaTile<kDim>::kStride, kK = kDim / 16, kNt = kTileKeys / 8;
     extern __shared__ __align__(16) unsigned char smem_raw[];
     INGOT_PDL_TRIGGER();
     INGOT_PDL_WAIT();
     const int seq = blockIdx.z, group = p.n_head / p.n_head_kv;
-    const int split = kDecode ? blockIdx.x % p.n_splits : 0;
     const int kvh = blockIdx.y, len = p.st.len[seq], n_rows = len * group;
     // prompts: later tiles see more keys, they go first
-    const int tile_rows = kDecode ? 16 : kWarps * 16;
-    const int row0 = (kDecode ? blockIdx.x / p.n_splits : (int)gridDim.x - 1 - (int)blockIdx.x) * tile_rows;
+    constexpr int tile_rows = kWarps * 16;
+    const int row0 = ((int)gridDim.x - 1 - (int)blockIdx.x) * tile_rows;
     if (row0 >= n_rows) return;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, j = lane & 3;
     const int pos0 = p.st.pos0[seq];
@@ -267,15 +263,10 @@ __global__ void __launch_bounds__(kDecode ? 128 : 256) shared_kv_mma_kernel(cons
 
     const int pos_first = pos0 + row0 / group, pos_last = pos0 + (min(row0 + tile_rows, n_rows) - 1) / group;
     const int page_a = p.map.page(p.map.first_visible(pos_first)), page_b = p.map.page(pos_last);
-    int t_begin = 0, t_end = (page_b - page_a) / 4 + 1;
-    if (kDecode) {
-        const int per = (t_end + p.n_splits - 1) / p.n_splits;
-        t_begin = split * per;
-        t_end = min(t_end, t_begin + per);
-    }
+    const int n_tiles = (page_b - page_a) / 4 + 1;
 
     // this thread's two rows
-    const int r_lo = row0 + (kDecode ? 0 : warp * 16) + g, r_hi = r_lo + 8;
+    const int r_lo = row0 + warp * 16 + g, r_hi = r_lo + 8;
     const int pos_lo = pos0 + min(r_lo, n_rows - 1) / group, pos_hi = pos0 + min(r_hi, n_rows - 1) / group;
     const int vis_lo = p.map.first_visible(pos_lo), vis_hi = p.map.first_visible(pos_hi);
     uint32_t qf[kK][4];
@@ -330,19 +321,18 @@ __global__ void __launch_bounds__(kDecode ? 128 : 256) shared_kv_mma_kernel(cons
 
 #pragma unroll
     for (int i = 0; i < kStages - 1; i++) {
-        if (t_begin + i < t_end) stage(t_begin + i, i);
+        if (i < n_tiles) stage(i, i);
         else asm volatile("cp.async.commit_group;" ::: "memory");
     }
-    for (int t = t_begin; t < t_end; t++) {
-        const int buf = (t - t_begin) % kStages;
+    for (int t = 0; t < n_tiles; t++) {
+        const int buf = t % kStages;
         asm volatile("cp.async.wait_group %0;" ::"n"(kStages - 2) : "memory");
         __syncthreads();  // tile t is in, and every warp is done with the buffer that is staged next
-        if (t + kStages - 1 < t_end) stage(t + kStages - 1, (t - t_begin + kStages - 1) % kStages);
+        if (t + kStages - 1 < n_tiles) stage(t + kStages - 1, (t + kStages - 1) % kStages);
         else asm volatile("cp.async.commit_group;" ::: "memory");
         const uint32_t tile = s_tile + buf * MmaTile<kDim>::kBytes;
-        const int key_base = kDecode ? warp * 16 : 0;
-        const float* sc = s_scale + buf * kTileKeys + key_base;
-        const int* kp = s_pos + buf * kTileKeys + key_base;
+        const float* sc = s_scale + buf * kTileKeys;
+        const int* kp = s_pos + buf * kTileKeys;
 
         float s[kNt][4];
 #pragma unroll
@@ -350,7 +340,7 @@ __global__ void __launch_bounds__(kDecode ? 128 : 256) shared_kv_mma_kernel(cons
 #pragma unroll
             for (int e = 0; e < 4; e++) s[nt][e] = s[nt + 1][e] = 0.f;
             // matrices: keys nt*8.. dims 0-7, same keys dims 8-15, keys (nt+1)*8.. dims 0-7, dims 8-15
-            const uint32_t a = tile + ((key_base + nt * 8 + (lane & 7) + ((lane >> 4) & 1) * 8) * kStride + ((lane >> 3) & 1) * 8) * 2;
+            const uint32_t a = tile + ((nt * 8 + (lane & 7) + ((lane >> 4) & 1) * 8) * kStride + ((lane >> 3) & 1) * 8) * 2;
 #pragma unroll
             for (int k = 0; k < kK; k++) {
                 uint32_t b[4];
@@ -360,7 +350,7 @@ __global__ void __launch_bounds__(kDecode ? 128 : 256) shared_kv_mma_kernel(cons
             }
         }
         // scale and mask; a tile all of whose keys every row of the CTA sees needs no mask
-        const bool masked = kDecode || s_pos[buf * kTileKeys] < p.map.first_visible(pos_last) || s_pos[buf * kTileKeys + kTileKeys - 1] > pos_first ||
+        const bool masked = s_pos[buf * kTileKeys] < p.map.first_visible(pos_last) || s_pos[buf * kTileKeys + kTileKeys - 1] > pos_first ||
                             (p.map.chunk > 0 && p.map.chunk % kBlockTokens != 0);
         float mx_lo = -INFINITY, mx_hi = -INFINITY;
 #pragma unroll
@@ -406,7 +396,7 @@ __global__ void __launch_bounds__(kDecode ? 128 : 256) shared_kv_mma_kernel(cons
         // O += P V; transposed 8x8 matrices: keys 0-7 dims d.., keys 8-15 dims d.., keys 0-7 dims d+8.., keys 8-15 dims d+8..
 #pragma unroll
         for (int kk = 0; kk < kNt / 2; kk++) {
-            const uint32_t a = tile + ((key_base + kk * 16 + (lane & 15)) * kStride + (lane >> 4) * 8) * 2;
+            const uint32_t a = tile + ((kk * 16 + (lane & 15)) * kStride + (lane >> 4) * 8) * 2;
 #pragma unroll
             for (int d = 0; d < kDim / 16; d++) {
                 uint32_t b[4];
@@ -421,29 +411,172 @@ __global__ void __launch_bounds__(kDecode ? 128 : 256) shared_kv_mma_kernel(cons
     l_hi += __shfl_xor_sync(0xffffffffu, l_hi, 1);
     l_hi += __shfl_xor_sync(0xffffffffu, l_hi, 2);
 
-    if (!kDecode) {
-        const float i_lo = 1.0f / l_lo, i_hi = 1.0f / l_hi;
+    const float i_lo = 1.0f / l_lo, i_hi = 1.0f / l_hi;
 #pragma unroll
-        for (int half = 0; half < 2; half++) {
-            const int r = half ? r_hi : r_lo;
-            if (r >= n_rows) continue;
-            const size_t row = tok0 + r / group;
-            const int c0 = (kvh * group + r % group) * p.out_dim;
-            const float inv = half ? i_hi : i_lo;
+    for (int half = 0; half < 2; half++) {
+        const int r = half ? r_hi : r_lo;
+        if (r >= n_rows) continue;
+        const size_t row = tok0 + r / group;
+        const int c0 = (kvh * group + r % group) * p.out_dim;
+        const float inv = half ? i_hi : i_lo;
 #pragma unroll
-            for (int i = 0; i < kDim / 8; i++)
+        for (int i = 0; i < kDim / 8; i++)
 #pragma unroll
-                for (int e = 0; e < 2; e++) {
-                    const int d = i * 8 + 2 * j + e;
-                    if (d < p.out_dim) p.out.store(row, c0 + d, o[i][half * 2 + e] * inv);
-                }
-        }
-        return;
+            for (int e = 0; e < 2; e++) {
+                const int d = i * 8 + 2 * j + e;
+                if (d < p.out_dim) p.out.store(row, c0 + d, o[i][half * 2 + e] * inv);
+            }
     }
+}
+
+// ---- decoding: one token of a sequence, split keys -------------------------------------------------------------------
+// A CTA serves the heads of one token that read one KV head (16 rows of the MMAs) over one share of the visible pages. Its four
+// warps take every fourth page each, through a cp.async ring of their own - no barrier in the key loop - with the page's 1/rms
+// travelling along; the block table of the share is read into shared memory first, so that no copy waits for an address. The
+// warps' states are merged through shared memory, and with several shares a second launch merges those.
+constexpr int kDecStages = 4, kDecWarps = 4, kDecMaxPages = 512;
+template <int kDim> struct DecodeSmem {
+    static constexpr int kStride = kDim + 8;
+    static constexpr int kPageBytes = kBlockTokens * kStride * 2;
+    static constexpr int kRing = kDecWarps * kDecStages * kPageBytes, kRms = kDecWarps * kDecStages * kBlockTokens * 4;
+    static constexpr int kMerge = kDecWarps * 16 * (kDim + 2) * 4;
+    static constexpr int kBytes = (kRing + kRms + kDecMaxPages * 4) > kMerge ? (kRing + kRms + kDecMaxPages * 4) : kMerge;
+};
+template <int kDim>
+__global__ void __launch_bounds__(128) shared_kv_decode_kernel(const AttendParams p) {
+    using L = DecodeSmem<kDim>;
+    constexpr int kK = kDim / 16;
+    extern __shared__ __align__(16) unsigned char smem_raw[];
+    INGOT_PDL_TRIGGER();
+    INGOT_PDL_WAIT();
+    const int seq = blockIdx.z, kvh = blockIdx.y, group = p.n_head / p.n_head_kv;
+    const int split = blockIdx.x % p.n_splits, row0 = blockIdx.x / p.n_splits * 16;  // rows: heads of the group
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, j = lane & 3;
+    const int pos = p.st.pos0[seq];
+    const size_t tok = p.st.row_start[seq];
+    const int page_a = p.map.page(p.map.first_visible(pos)), n_pages = p.map.page(pos) - page_a + 1;
+    const int last_key = pos - p.map.first_visible(pos);  // keys 0..last_key of the chunk, 16 per page
+    const int per = (n_pages + p.n_splits - 1) / p.n_splits, first = split * per, count = max(0, min(per, n_pages - first));
+    const __half* rows = static_cast<const __half*>(p.rows);
+
+    const uint32_t s_ring = (uint32_t)__cvta_generic_to_shared(smem_raw) + warp * kDecStages * L::kPageBytes;
+    float* s_rms = reinterpret_cast<float*>(smem_raw + L::kRing) + warp * kDecStages * kBlockTokens;
+    int* s_blk = reinterpret_cast<int*>(smem_raw + L::kRing + L::kRms);
+    for (int i = threadIdx.x; i < count; i += 128)
+        s_blk[i] = table_block(p.tables, p.first_page, p.max_blocks, p.n_blocks, seq, page_a + first + i, p.status);
+    __syncthreads();
+
+    auto stage = [&](int i, int buf) {  // page i of the share
+        if (i < count) {
+            const int blk = s_blk[i];
+            const __half* src = rows + ((size_t)max(blk, 0) * p.n_head_kv + kvh) * kBlockTokens * kDim;
+            constexpr int kPieces = kDim / 8;
+#pragma unroll
+            for (int c = lane; c < kBlockTokens * kPieces; c += 32)
+                cp16(s_ring + buf * L::kPageBytes + (c / kPieces * L::kStride + c % kPieces * 8) * 2, src + c * 8, blk >= 0);
+            if (lane < 4) cp16((uint32_t)__cvta_generic_to_shared(s_rms + buf * kBlockTokens + lane * 4), p.inv_rms + (size_t)max(blk, 0) * kBlockTokens + lane * 4, blk >= 0);
+        }
+        asm volatile("cp.async.commit_group;" ::: "memory");
+    };
+#pragma unroll
+    for (int k = 0; k < kDecStages - 1; k++) stage(warp + k * kDecWarps, k);
+
+    uint32_t qf[kK][4];
+    {
+        const __half* q = static_cast<const __half*>(p.q) + (tok * p.n_head + kvh * group) * kDim;
+        const int lo = row0 + g, hi = lo + 8;
+#pragma unroll
+        for (int k = 0; k < kK; k++) {
+            qf[k][0] = lo < group ? *reinterpret_cast<const uint32_t*>(q + (size_t)lo * kDim + k * 16 + 2 * j) : 0u;
+            qf[k][1] = hi < group ? *reinterpret_cast<const uint32_t*>(q + (size_t)hi * kDim + k * 16 + 2 * j) : 0u;
+            qf[k][2] = lo < group ? *reinterpret_cast<const uint32_t*>(q + (size_t)lo * kDim + k * 16 + 8 + 2 * j) : 0u;
+            qf[k][3] = hi < group ? *reinterpret_cast<const uint32_t*>(q + (size_t)hi * kDim + k * 16 + 8 + 2 * j) : 0u;
+        }
+    }
+    float m_lo = -INFINITY, m_hi = -INFINITY, l_lo = 0.f, l_hi = 0.f;
+    float o[kDim / 8][4];
+#pragma unroll
+    for (int i = 0; i < kDim / 8; i++) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
+    const float scale = p.scale * 1.44269504f;
+
+    int buf = 0;
+    for (int i = warp; i < count; i += kDecWarps) {
+        asm volatile("cp.async.wait_group %0;" ::"n"(kDecStages - 2) : "memory");
+        __syncwarp();  // the page is in, and every lane is done with the buffer that is staged next
+        stage(i + (kDecStages - 1) * kDecWarps, buf == 0 ? kDecStages - 1 : buf - 1);
+        const uint32_t page = s_ring + buf * L::kPageBytes;
+        const float* rms = s_rms + buf * kBlockTokens;
+        float s[2][4];
+#pragma unroll
+        for (int e = 0; e < 4; e++) s[0][e] = s[1][e] = 0.f;
+        const uint32_t a = page + (((lane & 7) + ((lane >> 4) & 1) * 8) * L::kStride + ((lane >> 3) & 1) * 8) * 2;
+#pragma unroll
+        for (int k = 0; k < kK; k++) {
+            uint32_t b[4];
+            ldmatrix4(b, a + k * 32);
+            mma_16816(s[0], qf[k][0], qf[k][1], qf[k][2], qf[k][3], b[0], b[1]);
+            mma_16816(s[1], qf[k][0], qf[k][1], qf[k][2], qf[k][3], b[2], b[3]);
+        }
+        const int left = last_key - (first + i) * kBlockTokens;  // keys of this page up to index `left` exist
+        const bool held = s_blk[i] >= 0;
+        float mx_lo = -INFINITY, mx_hi = -INFINITY;
+#pragma unroll
+        for (int nt = 0; nt < 2; nt++) {
+            const float2 ks = *reinterpret_cast<const float2*>(rms + nt * 8 + 2 * j);
+            const bool on0 = held && nt * 8 + 2 * j <= left, on1 = held && nt * 8 + 2 * j + 1 <= left;
+            s[nt][0] = on0 ? s[nt][0] * (ks.x * scale) : -INFINITY;
+            s[nt][1] = on1 ? s[nt][1] * (ks.y * scale) : -INFINITY;
+            s[nt][2] = on0 ? s[nt][2] * (ks.x * scale) : -INFINITY;
+            s[nt][3] = on1 ? s[nt][3] * (ks.y * scale) : -INFINITY;
+            mx_lo = fmaxf(mx_lo, fmaxf(s[nt][0], s[nt][1]));
+            mx_hi = fmaxf(mx_hi, fmaxf(s[nt][2], s[nt][3]));
+        }
+        mx_lo = fmaxf(mx_lo, __shfl_xor_sync(0xffffffffu, mx_lo, 1));
+        mx_lo = fmaxf(mx_lo, __shfl_xor_sync(0xffffffffu, mx_lo, 2));
+        mx_hi = fmaxf(mx_hi, __shfl_xor_sync(0xffffffffu, mx_hi, 1));
+        mx_hi = fmaxf(mx_hi, __shfl_xor_sync(0xffffffffu, mx_hi, 2));
+        const float mn_lo = fmaxf(m_lo, mx_lo), mn_hi = fmaxf(m_hi, mx_hi);
+        const float rf_lo = mn_lo == -INFINITY ? 0.f : mn_lo, rf_hi = mn_hi == -INFINITY ? 0.f : mn_hi;
+        const float a_lo = exp2f(m_lo - rf_lo), a_hi = exp2f(m_hi - rf_hi);
+        m_lo = mn_lo;
+        m_hi = mn_hi;
+        uint32_t pa[4];
+        float sum_lo = 0.f, sum_hi = 0.f;
+#pragma unroll
+        for (int nt = 0; nt < 2; nt++) {
+            const float p0 = exp2f(s[nt][0] - rf_lo), p1 = exp2f(s[nt][1] - rf_lo), p2 = exp2f(s[nt][2] - rf_hi), p3 = exp2f(s[nt][3] - rf_hi);
+            sum_lo += p0 + p1;
+            sum_hi += p2 + p3;
+            pa[nt * 2] = pack_half2_rn(p0, p1);
+            pa[nt * 2 + 1] = pack_half2_rn(p2, p3);
+        }
+        l_lo = l_lo * a_lo + sum_lo;
+        l_hi = l_hi * a_hi + sum_hi;
+        if (__any_sync(0xffffffffu, a_lo != 1.f || a_hi != 1.f)) {
+#pragma unroll
+            for (int d = 0; d < kDim / 8; d++) { o[d][0] *= a_lo; o[d][1] *= a_lo; o[d][2] *= a_hi; o[d][3] *= a_hi; }
+        }
+        const uint32_t v = page + ((lane & 15) * L::kStride + (lane >> 4) * 8) * 2;
+#pragma unroll
+        for (int d = 0; d < kDim / 16; d++) {
+            uint32_t b[4];
+            ldmatrix4_trans(b, v + d * 32);
+            mma_16816(o[2 * d], pa[0], pa[1], pa[2], pa[3], b[0], b[1]);
+            mma_16816(o[2 * d + 1], pa[0], pa[1], pa[2], pa[3], b[2], b[3]);
+        }
+        buf = buf + 1 == kDecStages ? 0 : buf + 1;
+    }
+
+    l_lo += __shfl_xor_sync(0xffffffffu, l_lo, 1);
+    l_lo += __shfl_xor_sync(0xffffffffu, l_lo, 2);
+    l_hi += __shfl_xor_sync(0xffffffffu, l_hi, 1);
+    l_hi += __shfl_xor_sync(0xffffffffu, l_hi, 2);
+
     // merge the warps' states: [warp][16 rows][kDim] and (m, l)
+    asm volatile("cp.async.wait_group 0;" ::: "memory");
     __syncthreads();
     float* so = reinterpret_cast<float*>(smem_raw);
-    float* sml = so + kWarps * 16 * kDim;
+    float* sml = so + kDecWarps * 16 * kDim;
 #pragma unroll
     for (int i = 0; i < kDim / 8; i++) {
         *reinterpret_cast<float2*>(so + (warp * 16 + g) * kDim + i * 8 + 2 * j) = make_float2(o[i][0], o[i][1]);
@@ -454,22 +587,22 @@ __global__ void __launch_bounds__(kDecode ? 128 : 256) shared_kv_mma_kernel(cons
         sml[(warp * 16 + g + 8) * 2] = m_hi; sml[(warp * 16 + g + 8) * 2 + 1] = l_hi;
     }
     __syncthreads();
-    const int rows_here = min(16, n_rows - row0);
-    for (int i = threadIdx.x; i < rows_here * kDim; i += kThreads) {
+    const int rows_here = min(16, group - row0);
+    for (int i = threadIdx.x; i < rows_here * kDim; i += 128) {
         const int r = i / kDim, d = i - r * kDim;
         float m = -INFINITY;
 #pragma unroll
-        for (int w = 0; w < kWarps; w++) m = fmaxf(m, sml[(w * 16 + r) * 2]);
+        for (int w = 0; w < kDecWarps; w++) m = fmaxf(m, sml[(w * 16 + r) * 2]);
         const float rf = m == -INFINITY ? 0.f : m;
         float l = 0.f, acc = 0.f;
 #pragma unroll
-        for (int w = 0; w < kWarps; w++) {
+        for (int w = 0; w < kDecWarps; w++) {
             const float f = exp2f(sml[(w * 16 + r) * 2] - rf);
             l = fmaf(f, sml[(w * 16 + r) * 2 + 1], l);
             acc = fmaf(f, so[(w * 16 + r) * kDim + d], acc);
         }
-        const int rr = row0 + r, h = kvh * group + rr % group;
-        const size_t row = tok0 + rr / group;
+        const int h = kvh * group + row0 + r;
+        const size_t row = tok;
         if (p.n_splits == 1) {
             if (d < p.out_dim) p.out.store(row, h * p.out_dim + d, acc / l);
         } else {
@@ -507,13 +640,22 @@ int launch_mma(ingot_skv* kv, AttendParams p, cudaStream_t s) {
         constexpr int kSmem = 2 * (MmaTile<kDim>::kBytes + kTileKeys * 8);
         const dim3 grid((unsigned)(((size_t)p.st.max_len * group + 127) / 128), p.n_head_kv, p.st.n_seq);
         p.n_splits = 1;
-        INGOT_CUDA_TRY(cudaFuncSetAttribute(shared_kv_mma_kernel<kDim, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, kSmem));
-        INGOT_CUDA_TRY(ingot_launch_pdl(shared_kv_mma_kernel<kDim, false>, grid, dim3(256), kSmem, s, p));
+        INGOT_CUDA_TRY(cudaFuncSetAttribute(shared_kv_mma_kernel<kDim>, cudaFuncAttributeMaxDynamicSharedMemorySize, kSmem));
+        INGOT_CUDA_TRY(ingot_launch_pdl(shared_kv_mma_kernel<kDim>, grid, dim3(256), kSmem, s, p));
         return INGOT_OK;
     }
+    // Shares of the keys: CTAs run in rounds of as many as fit the GPU, and a share costs about 64 keys' time besides its keys, so
+    // the count that minimises rounds * (share + 64) - and never more pages per share than the kernel's table holds.
     const int row_tiles = (group + 15) / 16, keys = p.max_blocks * kBlockTokens;
-    // enough CTAs for two per SM, at least kSplitKeysMin keys each
-    p.n_splits = std::max(1, std::min({(keys + kSplitKeysMin - 1) / kSplitKeysMin, 2 * kv->num_sms / (row_tiles * p.n_head_kv * p.st.n_seq), 32}));
+    const int ctas = row_tiles * p.n_head_kv * p.st.n_seq, slots = kv->num_sms * std::max(1, std::min(4, 220 * 1024 / DecodeSmem<kDim>::kBytes));
+    long long best = -1;
+    for (int n = 1; n <= 64; n++) {
+        const int share = (keys + n - 1) / n;
+        if (n > 1 && share < kSplitKeysMin) break;
+        const long long cost = ((long long)ctas * n + slots - 1) / slots * (share + 64);
+        if (best < 0 || cost < best) { best = cost; p.n_splits = n; }
+    }
+    p.n_splits = std::max(p.n_splits, (p.max_blocks + kDecMaxPages - 1) / kDecMaxPages);
     if (p.n_splits > 1) {
         const size_t need = (size_t)p.st.n_tok * p.n_head * p.n_splits * (kDim + 2);
         if (need > kv->part_floats) {
@@ -525,11 +667,9 @@ int launch_mma(ingot_skv* kv, AttendParams p, cudaStream_t s) {
         }
         p.part = kv->part;
     }
-    constexpr int kRing = 4 * (MmaTile<kDim>::kBytes + kTileKeys * 8), kMerge = 4 * 16 * (kDim + 2) * 4;
-    constexpr int kSmem = kRing > kMerge ? kRing : kMerge;
-    INGOT_CUDA_TRY(cudaFuncSetAttribute(shared_kv_mma_kernel<kDim, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, kSmem));
+    INGOT_CUDA_TRY(cudaFuncSetAttribute(shared_kv_decode_kernel<kDim>, cudaFuncAttributeMaxDynamicSharedMemorySize, DecodeSmem<kDim>::kBytes));
     const dim3 grid(row_tiles * p.n_splits, p.n_head_kv, p.st.n_seq);
-    INGOT_CUDA_TRY(ingot_launch_pdl(shared_kv_mma_kernel<kDim, true>, grid, dim3(128), kSmem, s, p));
+    INGOT_CUDA_TRY(ingot_launch_pdl(shared_kv_decode_kernel<kDim>, grid, dim3(128), size_t(DecodeSmem<kDim>::kBytes), s, p));
     if (p.n_splits > 1) INGOT_CUDA_TRY(ingot_launch_pdl(shared_kv_merge_kernel, dim3(p.n_head, p.st.n_tok), dim3(128), 0, s, p));
     return INGOT_OK;
 }

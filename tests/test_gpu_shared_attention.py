@@ -139,6 +139,20 @@ def test_tcgen05_kernel(heads, kv_heads, dim, chunk):
             assert np.abs(g - want).max() < 8e-3, np.abs(g - want).max()
 
 
+@pytest.mark.parametrize("heads,kv_heads,dim,chunk,n", [(8, 2, 128, 0, 1500), (6, 1, 64, 900, 2000), (32, 1, 32, 0, 700), (4, 2, 200, 0, 600)])
+def test_decoding_over_many_keys(heads, kv_heads, dim, chunk, n):
+    """Single tokens after long prompts: keys split over several thread blocks, unequal sequences in the batch, more heads than
+    one row tile."""
+    rng = np.random.default_rng(n)
+    wq, wk = 1 + 0.3 * rng.standard_normal(heads * dim), 1 + 0.3 * rng.standard_normal(kv_heads * dim)
+    seqs = [(rng.standard_normal((m, heads * dim)), 2 * rng.standard_normal((m, kv_heads * dim))) for m in (n, n // 3, 9)]
+    cuts = [[n - 3, 1, 1, 1], [n // 3 - 3, 1, 1, 1], [6, 1, 1, 1]]
+    got = run(seqs, cuts, heads, kv_heads, dim, chunk, F16, wq, wk, 0)
+    for (q, kv), g in zip(seqs, got):
+        want = reference(q[:], kv, wq, wk, heads, kv_heads, dim, chunk)
+        assert np.abs(g[-3:] - want[-3:]).max() < 8e-3, np.abs(g - want).max()
+
+
 def test_a_table_entry_outside_the_pool_is_reported():
     import torch
     h = C.c_void_p()
