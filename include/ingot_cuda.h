@@ -364,6 +364,52 @@ int ingot_skv_append(ingot_skv* kv, int layer, const ingot_step* step, const flo
 int ingot_skv_attend(ingot_skv* kv, int layer, const ingot_step* step, const void* q_dev, int n_head, int out_dim, float scale,
                      float out_scale, const ingot_act_out* out, const int32_t* tables_dev, const int32_t* first_page_dev, int max_blocks, int impl, void* stream);
 
+/* The same cache for rows that are keys as they stand (no per-key scale), with a window that slides along: position i sees
+ * i - window + 1 .. i (window 0: the whole past), page of position p = p / 16. row_length a multiple of 4, <= 1024. */
+int ingot_skv_create_window(ingot_skv** out, int n_layer, int n_head_kv, int row_length, int dtype, int window, int n_blocks);
+
+/* ---- Latent attention -------------------------------------------------------------------------------
+ * One row per token for all heads: a normalised latent c (rank columns) and a rotated key part (rot columns), in a window-form
+ * cache with one KV head. Lengths are as stored (padded with zeros); rank_count is the latent's true length. */
+typedef struct ingot_latent_shape {
+    int n_head, dim, rot;      /* per head: unrotated and rotated query columns, stored side by side */
+    int rank, rank_count;
+    int rot_dims;              /* rotated values, even, <= rot: i with i + rot_dims / 2; the rest of the part passes unchanged */
+} ingot_latent_shape;
+/* Columns q_off.. of proj_dev's rows: n_head x [dim | rot]; columns latent_off..: [rank | rot], the latent not yet normalised.
+ * Writes the cache rows of the step's positions, the rotated query parts into q_rows_dev [n_tok][n_head][row length] (cache type;
+ * may be null) and the unrotated query parts to q_plain [n_tok][n_head * dim]. turns_dev [rot_dims / 2]: turns per position
+ * (base^(-2 i / rot_dims) / 2 pi). norm_dev [rank], zero in the padding. Tables as for ingot_skv_append. */
+int ingot_latent_append(ingot_skv* kv, int layer, const ingot_step* step, const float* proj_dev, int proj_ld, int q_off, int latent_off,
+                        const ingot_latent_shape* shape, const float* norm_dev, float eps, const double* turns_dev, const ingot_act_out* q_plain,
+                        void* q_rows_dev, const int32_t* tables_dev, const int32_t* first_page_dev, int max_blocks, void* stream);
+/* Latent queries f32 [n_tok][n_head * rank] into the first rank columns of the query rows. */
+int ingot_latent_queries(const ingot_skv* kv, const float* q_dev, int n_tok, int n_head, int rank, void* q_rows_dev, void* stream);
+/* out [n_tok][n_head * rank]: sum over the visible keys of softmax(q_row . row * scale) times the first rank columns of the row;
+ * sink_dev [n_head] (may be null): the denominator also holds exp(sink). skip_len > 0: sequences of the step with that many tokens
+ * or more are left out. impl: 0 = library's choice, 1 = the plain f32-arithmetic kernel, 2 = the tensor-core kernel (f16 rows, row
+ * length a multiple of 32, rank a multiple of 16 and at most 512). */
+int ingot_latent_attend(ingot_skv* kv, int layer, const ingot_step* step, const void* q_rows_dev, int n_head, int rank, float scale,
+                        const float* sink_dev, const ingot_act_out* out, const int32_t* tables_dev, const int32_t* first_page_dev, int max_blocks,
+                        int skip_len, int impl, void* stream);
+
+/* ---- Mixture of experts -----------------------------------------------------------------------------
+ * Pair p = token * top + k is a token's k-th expert; rows are the pairs sorted by expert, in token order within one. */
+enum { INGOT_ACT_NONE = 0, INGOT_ACT_RELU2 = 1 };  /* RELU2: the square of relu */
+/* The top experts of each token by logit (the lower index of equal ones) with sigmoid(logit) as weight, and their sorting:
+ * expert_of, weight_of, row_of [n_tok * top] by pair, pair_of, row_weight [n_tok * top] by row, group_start [n_expert + 1]. */
+int ingot_moe_route(const float* logits_dev, int ld, int n_tok, int n_expert, int top, int32_t* expert_of_dev, float* weight_of_dev,
+                    int32_t* group_start_dev, int32_t* row_of_dev, int32_t* pair_of_dev, float* row_weight_dev, void* stream);
+/* bf16 planes [n_rows][n] of the rows from planes [n_tok][n] of the tokens (lo may be null). n a multiple of 8. */
+int ingot_moe_gather(void* hi_dev, void* lo_dev, const void* src_hi_dev, const void* src_lo_dev, const int32_t* pair_of_dev, int n_rows,
+                     int top, int n, void* stream);
+/* out[row] = act(row_weight[row] * W_e x), W bf16 [n_expert][n_out][n_in], f32 arithmetic. x row of a row: its token's
+ * (pair_of_dev given) or its own; row_weight_dev may be null. */
+int ingot_moe_linear(float* out_dev, const void* w_dev, const float* x_dev, int x_ld, int n_in, int n_out, int n_expert, int n_rows,
+                     const int32_t* group_start_dev, const int32_t* pair_of_dev, int top, const float* row_weight_dev, int act, void* stream);
+/* x [n_tok][n] += the sum of each token's rows of [n_tok * top][n] (row_of_dev null, top 1: its own). */
+int ingot_moe_add(float* x_dev, const float* rows_dev, const int32_t* row_of_dev, int n_tok, int top, int n, void* stream);
+
 /* ---- Diagnostics ----------------------------------------------------------------------------------
  * HBM read-bandwidth probe: what the reference's `bwtest` verb measures (src/main.cpp:450-455,
  * MetalBackend::bandwidth_test src/metal_backend.mm:533-592 with the bw_fill / bw_sum kernels,

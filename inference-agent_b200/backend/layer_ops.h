@@ -1,0 +1,402 @@
+// What the layers of a model folder are written in: projections (with the RMS norm of their input or the residual add of their
+// output folded in), scratch activations, weight upload, state and cache groups; and the interfaces of a layer's two parts.
+//
+// Precision. Weights are bf16. In the 16-bit form the tensor-core products take bf16 activations (a hi + lo pair where the
+// product feeds a recurrence's gates or step sizes, and in small batches) and accumulate in f32; everything between products - residual stream,
+// norms, scores and softmax, gates, recurrent states, router scores - is f32, and single tokens multiply f32 activations. In the f32 form
+// every product is f32 FMA on widened weights and the attention cache is f32.
+//
+// Padding. Every vector is stored with a length that is a multiple of 8 (heads and gate blocks each padded on their own):
+// padded weight rows and columns are zero, so padded activations are zero and only means need the true count.
+#pragma once
+
+#include <cuda_runtime.h>
+
+#include <algorithm>
+#include <cmath>
+#include <cstring>
+#include <memory>
+#include <string>
+#include <vector>
+
+#include "block_pool.h"
+#include "cuda_util.h"
+#include "grouped_linear.h"
+#include "ingot_cuda.h"
+#include "model_registry.h"
+#include "weight_streamer.h"
+
+extern "C" {
+cudaError_t ingot_support_embed_rows_bf16(float* out, const void* table, int n_in, int n_rows_table, const int32_t* rows_dev, int n_rows,
+                                          int* status_dev, cudaStream_t s);
+cudaError_t ingot_support_embed_sum_bf16(float* out, float* copy, const void* table, int n_rows_table, const int32_t* rows_dev, const void* table2,
+                                         int n_rows_table2, const int32_t* rows2_dev, int n_in, int n_rows, int* status_dev, cudaStream_t s);
+cudaError_t ingot_support_concat_rows(float* f32, void* hi, void* lo, const float* a, const float* b, int n, int n_rows, cudaStream_t s);
+cudaError_t ingot_support_softcap(float* x, size_t n, float cap, cudaStream_t s);
+cudaError_t ingot_support_rmsnorm_rows(float* out, const float* x, const float* w, const int32_t* rows_dev, int n_rows, int n, int n_mean,
+                                       float eps, cudaStream_t s);
+cudaError_t ingot_support_linear_bf16(float* out, const void* w, const float* x, int x_ld, int n_in, int n_out, int rows_per_block,
+                                      int n_tok, int accumulate, cudaStream_t s);
+cudaError_t ingot_support_gemv_bf16(float* out, const void* w, int n_out, int n_in, const float* x, const float* norm_w, float eps, int n_mean,
+                                    int gated, int act, int accumulate, cudaStream_t s);
+cudaError_t ingot_support_gated_act(float* out, const float* in, int n_rows, int n, int act, cudaStream_t s);
+struct ingot_linear_ws;
+cudaError_t ingot_linear_ws_create_bf16(ingot_linear_ws** out, int max_tok, int max_in, int max_out);
+void ingot_linear_ws_destroy(ingot_linear_ws* ws);
+int* ingot_linear_ws_status_dev(ingot_linear_ws* ws);
+void ingot_linear_ws_planes(ingot_linear_ws* ws, void** hi, void** lo);
+cudaError_t ingot_linear_tc_prepared(ingot_linear_ws* ws, int n_in, int n_tok, int planes);
+cudaError_t ingot_linear_tc_prepare_bf16(ingot_linear_ws* ws, const float* x, int x_ld, int n_in, int n_tok, int planes, cudaStream_t s);
+cudaError_t ingot_linear_tc_prepare_norm_bf16(ingot_linear_ws* ws, const float* x, const float* norm_w, float eps, int n_in, int n_mean, int n_tok,
+                                              int planes, cudaStream_t s);
+cudaError_t ingot_linear_tc_run(ingot_linear_ws* ws, float* out, const void* w, int n_in, int n_out, int accumulate, cudaStream_t s);
+cudaError_t ingot_linear_tc_run_blocks(ingot_linear_ws* ws, float* out, const void* w, int k_block, int n_out, int rows_per_block, cudaStream_t s);
+cudaError_t ingot_linear_tc_run_partial(ingot_linear_ws* ws, const void* w, int n_in, int n_out, int slot, cudaStream_t s);
+cudaError_t ingot_linear_tc_run_half(ingot_linear_ws* ws, void* out, int out_ld, int out_block, const void* w, int n_in, int n_out, int rows_per_block,
+                                     cudaStream_t s);
+cudaError_t ingot_linear_tc_finish_residual_norm_bf16(ingot_linear_ws* ws, float* x, const float* norm_w, float eps, int n_mean, int planes,
+                                                      const float* pair_rows, const int32_t* row_of, int top, cudaStream_t s);
+cudaError_t ingot_linear_tc_finish_gated_bf16(ingot_linear_ws* ws, int act, int planes, cudaStream_t s);
+}
+
+inline constexpr int kMinTcTokens = 2;  // from two tokens on, a 128-token tile that is mostly padding still only streams the weights once
+
+// Up to this many tokens a product is bound by streaming the weights, so the activations go in as a hi + lo pair at no cost: a
+// decoded token's logits then hardly depend on whether it is alone (f32 activations) or in a batch.
+inline constexpr int kPairTokens = 64;
+
+inline int round_up(int v, int q) { return (v + q - 1) / q * q; }
+
+inline int get_int(const Json& j, const char* key, int lo = 1, int hi = 1 << 28) {
+    const int64_t v = j.at(key).integer();
+    if (v < lo || v > hi) throw std::runtime_error(std::string("model config: \"") + key + "\" is out of range");
+    return int(v);
+}
+inline float get_float(const Json& j, const char* key) { return float(j.at(key).number()); }
+
+// A dimension of n groups of `size` values, each stored with `padded` places.
+struct Groups {
+    int n, size, padded;
+    int count() const { return n * size; }
+    int width() const { return n * padded; }
+};
+inline Groups flat(int size) { return {1, size, round_up(size, 8)}; }
+
+// A bf16 matrix on the device, [n_out][n_in] row-major, both padded. rows_per_block > 0: block-diagonal, n_in per block.
+struct Matrix {
+    void* data = nullptr;
+    int n_out = 0, n_in = 0, rows_per_block = 0;
+    const void* rows_from(int r) const { return static_cast<const char*>(data) + size_t(r) * n_in * 2; }
+};
+
+// One tensor's place in a matrix: its logical rows (from row src_row0 on; groups src_stride rows apart, 0: side by side) and columns
+// go to r0 + row groups, c0 + column groups.
+struct Part {
+    std::string name;
+    std::vector<int64_t> shape;
+    Groups rows, cols;
+    int r0 = 0, c0 = 0, src_row0 = 0, src_stride = 0;
+};
+
+enum Buf { kProj, kConv, kStateIn, kDt, kGates, kMix, kGateUp, kMid, kNormed, kQuery, kQueryPlain, kLatent, kValue, kRouter, kExpertIn, kExpertMid, kExpertOut,
+           kBranch, kConcat, kBufCount };
+
+// The step as the launches see it.
+struct StepCtx {
+    ingot_step st = {};
+    ingot_scan_plan scan = {}, lru = {};
+    bool tc = false;  // products on the tensor cores (16-bit form, more than one token)
+    int planes = 1;   // bf16 planes an activation is given as there
+};
+
+// Shared-row attention caches of equal shape and visibility live in one handle with one page pool.
+struct CacheGroup {
+    int kv_heads, dim, chunk, window;  // visibility: own chunk, sliding window (one of them 0), or the whole past
+    bool scales;                       // rows with a key scale of their own (ingot_skv_create) or without (ingot_skv_create_window)
+    int n_layer = 0;
+    ingot_skv* kv = nullptr;
+    BlockPool pool;
+    int pages_per_chunk = 0;
+    const int32_t *tables = nullptr, *first_page = nullptr;  // device, of the current step
+    int width = 0;
+    int page(int pos) const { return ingot_skv_pages(chunk, pos + 1) - 1; }
+    int first_visible(int pos) const { return chunk > 0 ? pos / chunk * chunk : window > 0 && pos >= window ? pos - window + 1 : 0; }
+    bool forgets() const { return chunk > 0 || window > 0; }  // pages fall out of sight for good
+    int pages_seen() const { return chunk > 0 ? pages_per_chunk : (window + INGOT_BLOCK_TOKENS - 2) / INGOT_BLOCK_TOKENS + 1; }  // at most, by one token
+};
+
+// What a feed-forward branch leaves for the residual sum: rows of the residual's length, token t's at row_of[t * top + k].
+struct Branch {
+    const float* rows = nullptr;
+    const int32_t* row_of = nullptr;  // null: row t
+    int top = 1;
+};
+
+class LayerOps {
+public:
+    LayerOps(const ModelDir& dir, const EngineOptions& opt, int max_step) : dir(dir), opt(opt), max_step(max_step) {
+        cuda_check(cudaStreamCreateWithFlags(&stream, cudaStreamNonBlocking), "cudaStreamCreate");
+    }
+    ~LayerOps() {
+        cudaStreamSynchronize(stream);
+        ingot_linear_ws_destroy(ws);
+        for (void* p : allocs_) cudaFree(p);
+        cudaStreamDestroy(stream);
+    }
+
+    // ---- construction ----
+    void* alloc(size_t bytes, bool zero = false) {
+        void* p = nullptr;
+        cuda_check(cudaMalloc(&p, std::max<size_t>(bytes, 16)), "cudaMalloc");
+        allocs_.push_back(p);
+        if (zero) cuda_check(cudaMemset(p, 0, std::max<size_t>(bytes, 16)), "cudaMemset");
+        return p;
+    }
+    void need(Buf b, int columns) { columns_[b] = std::max(columns_[b], columns); }
+    void tc_shape(int n_in, int n_out) { tc_in_ = std::max(tc_in_, n_in); tc_out_ = std::max(tc_out_, n_out); }
+    void allocate() {
+        for (int b = 0; b < kBufCount; b++) bufs_[b] = columns_[b] ? static_cast<float*>(alloc(size_t(max_step) * columns_[b] * 4, true)) : nullptr;
+        if (!opt.f32 && max_step >= kMinTcTokens) cuda_check(ingot_linear_ws_create_bf16(&ws, max_step, tc_in_, tc_out_), "linear workspace");
+        loader_.finish();
+        cuda_check(cudaDeviceSynchronize(), "model upload");
+    }
+    float* upload(const std::vector<float>& v) {
+        float* d = static_cast<float*>(alloc(v.size() * 4));
+        cuda_check(cudaMemcpy(d, v.data(), v.size() * 4, cudaMemcpyHostToDevice), "cudaMemcpy");
+        return d;
+    }
+    // A vector tensor with each group padded with zeros.
+    std::vector<float> host_vector(const std::string& name, const std::vector<int64_t>& shape, Groups g) {
+        const std::vector<float> v = tensor_f32(dir.tensor(name, shape));
+        if (int(v.size()) != g.count()) throw std::runtime_error("model: tensor " + name + " does not have " + std::to_string(g.count()) + " values");
+        std::vector<float> out(size_t(g.width()), 0.f);
+        for (int i = 0; i < g.n; i++) std::copy(v.begin() + i * g.size, v.begin() + (i + 1) * g.size, out.begin() + i * g.padded);
+        return out;
+    }
+    float* vector(const std::string& name, const std::vector<int64_t>& shape, Groups g) { return upload(host_vector(name, shape, g)); }
+    float* vector(const std::string& name, int n) { return vector(name, {n}, flat(n)); }
+    // The weight of an RMS norm over the residual stream, as the design stores it (around norm_offset).
+    float* norm_vector(const std::string& name) {
+        std::vector<float> v = host_vector(name, {width}, flat(width));
+        for (int i = 0; i < width; i++) v[size_t(i)] += norm_offset;
+        return upload(v);
+    }
+    const TensorView& bf16(const std::string& name, const std::vector<int64_t>& shape) const {
+        const TensorView& t = dir.tensor(name, shape);
+        if (t.dtype != "BF16") throw std::runtime_error("model: tensor " + name + " has type " + t.dtype + ", expected BF16");
+        return t;
+    }
+    // grouped: a stack of matrices for ingot_grouped_tc_run, whose results do not pass through the workspace
+    Matrix matrix(int n_out, int n_in, const std::vector<Part>& parts, int rows_per_block = 0, bool grouped = false) {
+        std::vector<uint16_t> host(size_t(n_out) * n_in, 0);
+        for (const Part& p : parts) {
+            const TensorView& t = bf16(p.name, p.shape);
+            const int stride = p.src_stride ? p.src_stride : p.rows.size;
+            if (t.elems() < int64_t(p.src_row0 + (p.rows.n - 1) * stride + p.rows.size) * p.cols.count() || t.elems() % p.cols.count() != 0)
+                throw std::runtime_error("model: tensor " + p.name + " has an unexpected size");
+            const int nr = p.rows.count();
+            for (int r = 0; r < nr; r++) {
+                uint16_t* dst = host.data() + size_t(p.r0 + r / p.rows.size * p.rows.padded + r % p.rows.size) * n_in + p.c0;
+                const unsigned char* src = t.data + size_t(p.src_row0 + r / p.rows.size * stride + r % p.rows.size) * p.cols.count() * 2;
+                for (int g = 0; g < p.cols.n; g++) memcpy(dst + g * p.cols.padded, src + size_t(g) * p.cols.size * 2, size_t(p.cols.size) * 2);
+            }
+        }
+        return matrix(host, n_out, n_in, rows_per_block, grouped);
+    }
+    Matrix matrix(const std::vector<uint16_t>& host, int n_out, int n_in, int rows_per_block, bool grouped = false) {
+        Matrix m;
+        m.n_out = n_out;
+        m.n_in = n_in;
+        m.rows_per_block = rows_per_block;
+        m.data = alloc(host.size() * 2);
+        loader_.copy(m.data, host.data(), host.size() * 2);
+        weight_bytes += host.size() * 2;
+        if (!grouped) tc_shape(rows_per_block > 0 ? n_in * (n_out / rows_per_block) : n_in, n_out);
+        return m;
+    }
+    Matrix matrix(const std::string& name, Groups rows, Groups cols) {
+        return matrix(rows.width(), cols.width(), {Part{name, {rows.count(), cols.count()}, rows, cols}});
+    }
+
+    // ---- the step ----
+    float* buf(Buf b) const { return bufs_[b]; }
+    // Output of a kernel that feeds a product: the operand planes on the tensor-core path (and f32 rows if `keep`), else f32.
+    ingot_act_out operand(const StepCtx& s, float* f32, int ld, bool keep, int planes = 0) const {
+        ingot_act_out o = {};
+        o.ld = ld;
+        if (!s.tc || keep) o.f32 = f32;
+        if (s.tc) {
+            ingot_linear_ws_planes(ws, &o.hi, &o.lo);
+            if (std::max(planes, s.planes) < 2) o.lo = nullptr;
+        }
+        return o;
+    }
+    void operand_ready(const StepCtx& s, int n_in, int planes = 0) const {
+        if (s.tc) cuda_check(ingot_linear_tc_prepared(ws, n_in, s.st.n_tok, std::max(planes, s.planes)), "operand");
+    }
+    static bool streams(const Matrix& w) { return w.n_in % 256 == 0 && w.n_in <= 12032 && w.rows_per_block == 0; }
+
+    // out [n_tok][w.n_out] = W rmsnorm(x)
+    void norm_project(const StepCtx& s, float* out, const Matrix& w, const float* norm) {
+        if (s.tc) {
+            prepare_norm(s, w, norm);
+            cuda_check(ingot_linear_tc_run(ws, out, w.data, w.n_in, w.n_out, 0, stream), "projection");
+        } else if (s.st.n_tok == 1 && streams(w)) {
+            cuda_check(ingot_support_gemv_bf16(out, w.data, w.n_out, w.n_in, x, norm, eps, width, 0, 0, 0, stream), "projection");
+        } else {
+            norm_rows(s, norm);
+            cuda_check(ingot_support_linear_bf16(out, w.data, buf(kNormed), w.n_in, w.n_in, w.n_out, 0, s.st.n_tok, 0, stream), "projection");
+        }
+    }
+    // out = W in. Tensor-core path: the operand planes must hold `in` (operand_ready).
+    void project(const StepCtx& s, float* out, const Matrix& w, const float* in, int in_ld) {
+        if (s.tc) {
+            if (w.rows_per_block > 0) cuda_check(ingot_linear_tc_run_blocks(ws, out, w.data, w.n_in, w.n_out, w.rows_per_block, stream), "block projection");
+            else cuda_check(ingot_linear_tc_run(ws, out, w.data, w.n_in, w.n_out, 0, stream), "projection");
+        } else if (s.st.n_tok == 1 && streams(w) && w.n_out > 2048) {  // few rows: ingot_support_linear_bf16 gives each a CTA
+            cuda_check(ingot_support_gemv_bf16(out, w.data, w.n_out, w.n_in, in, nullptr, 0.f, w.n_in, 0, 0, 0, stream), "projection");
+        } else {
+            cuda_check(ingot_support_linear_bf16(out, w.data, in, in_ld, w.n_in, w.n_out, w.rows_per_block, s.st.n_tok, 0, stream), "projection");
+        }
+    }
+    // Tensor-core path: f32 rows become the operand planes.
+    void prepare_rows(const StepCtx& s, const float* in, int in_ld, int n_in, int planes = 0) const {
+        cuda_check(ingot_linear_tc_prepare_bf16(ws, in, in_ld, n_in, s.st.n_tok, std::max(planes, s.planes), stream), "operand");
+    }
+    // The same for f32 rows that are not in the planes yet.
+    void project_rows(const StepCtx& s, float* out, const Matrix& w, const float* in, int in_ld, int planes) {
+        if (s.tc) prepare_rows(s, in, in_ld, w.n_in, planes);
+        project(s, out, w, in, in_ld);
+    }
+    // x += W in; next_norm: the norm that the following product reads x through (null: none), folded into the same kernel.
+    void project_residual(const StepCtx& s, const Matrix& w, const float* in, const float* next_norm) {
+        norm_ready_ = nullptr;
+        if (s.tc) {
+            cuda_check(ingot_linear_tc_run_partial(ws, w.data, w.n_in, w.n_out, 0, stream), "output projection");
+            cuda_check(ingot_linear_tc_finish_residual_norm_bf16(ws, x, next_norm, eps, width, s.planes, branch_.rows, branch_.row_of, branch_.top, stream), "residual");
+            norm_ready_ = next_norm;
+            branch_ = Branch();
+            return;
+        }
+        if (s.st.n_tok == 1 && streams(w)) {
+            cuda_check(ingot_support_gemv_bf16(x, w.data, w.n_out, w.n_in, in, nullptr, 0.f, w.n_in, 0, 0, 1, stream), "output projection");
+        } else {
+            cuda_check(ingot_support_linear_bf16(x, w.data, in, w.n_in, w.n_in, w.n_out, 0, s.st.n_tok, 1, stream), "output projection");
+        }
+        add_branch(s);
+    }
+    // A feed-forward that runs beside the mixer leaves its result here; the mixer's project_residual takes it in.
+    void set_branch(const Branch& b) { branch_ = b; }
+    // The same without a mixer to join: x += branch.
+    void add_branch(const StepCtx& s) {
+        if (!branch_.rows) return;
+        ingot_check(ingot_moe_add(x, branch_.rows, branch_.row_of, s.st.n_tok, branch_.top, round_up(width, 8), stream));
+        branch_ = Branch();
+        norm_ready_ = nullptr;
+    }
+    // x = W [x; x0], two residual-length rows side by side
+    void project_concat(const StepCtx& s, const Matrix& w, const float* x0) {
+        const int n = round_up(width, 8);
+        ingot_act_out o = operand(s, buf(kConcat), 2 * n, false);
+        cuda_check(ingot_support_concat_rows(o.f32, o.hi, o.lo, x, x0, n, s.st.n_tok, stream), "concatenation");
+        operand_ready(s, 2 * n);
+        project(s, x, w, buf(kConcat), 2 * n);
+        norm_ready_ = nullptr;
+    }
+    // kMid (or the operand planes) = gelu(W_gate h) * (W_up h), h = rmsnorm(x); w holds the gate rows and then the up rows
+    void gated_project(const StepCtx& s, const Matrix& w, const float* norm) {
+        const int ff = w.n_out / 2;
+        if (s.tc) {
+            prepare_norm(s, w, norm);
+            cuda_check(ingot_linear_tc_run_partial(ws, w.data, w.n_in, w.n_out, 0, stream), "gate / up");
+            cuda_check(ingot_linear_tc_finish_gated_bf16(ws, 1, s.planes, stream), "gate");
+        } else if (s.st.n_tok == 1 && streams(w)) {
+            cuda_check(ingot_support_gemv_bf16(buf(kMid), w.data, ff, w.n_in, x, norm, eps, width, 1, 1, 0, stream), "gate / up");
+        } else {
+            norm_rows(s, norm);
+            cuda_check(ingot_support_linear_bf16(buf(kGateUp), w.data, buf(kNormed), w.n_in, w.n_in, w.n_out, 0, s.st.n_tok, 0, stream), "gate / up");
+            cuda_check(ingot_support_gated_act(buf(kMid), buf(kGateUp), s.st.n_tok, ff, 1, stream), "gate");
+        }
+    }
+    void begin() { norm_ready_ = nullptr; branch_ = Branch(); }
+    void norm_rows(const StepCtx& s, const float* norm) {
+        cuda_check(ingot_support_rmsnorm_rows(buf(kNormed), x, norm, nullptr, s.st.n_tok, round_up(width, 8), width, eps, stream), "rmsnorm");
+    }
+    // Tensor-core path: the planes hold rmsnorm(x; norm).
+    void prepare_norm(const StepCtx& s, const Matrix& w, const float* norm) {
+        const bool ready = norm_ready_ == norm && norm;  // the kernel that finished x already normalised it for this product
+        norm_ready_ = nullptr;
+        if (!ready) cuda_check(ingot_linear_tc_prepare_norm_bf16(ws, x, norm, eps, w.n_in, width, s.st.n_tok, s.planes, stream), "rmsnorm");
+    }
+
+    const ModelDir& dir;
+    const EngineOptions opt;
+    const int max_step;
+    cudaStream_t stream = nullptr;
+    ingot_linear_ws* ws = nullptr;
+    float* x = nullptr;  // residual stream [n_tok][round_up(width, 8)]
+    int width = 0;
+    float eps = 0.f, norm_offset = 0.f;
+    int passes = 1;  // of the layer under construction: each pass of a loop has a state and a cache of its own
+    int pass = 0;    // the one that runs
+    size_t weight_bytes = 0;
+    std::vector<std::unique_ptr<CacheGroup>> caches;
+
+    // The group a layer's caches belong to; *layer: the first of its `passes` caches there.
+    CacheGroup* cache_group(int kv_heads, int dim, int chunk, int window, bool scales, int* layer) {
+        CacheGroup* g = nullptr;
+        for (auto& c : caches)
+            if (c->kv_heads == kv_heads && c->dim == dim && c->chunk == chunk && c->window == window && c->scales == scales) g = c.get();
+        if (!g) {
+            caches.push_back(std::make_unique<CacheGroup>());
+            g = caches.back().get();
+            g->kv_heads = kv_heads; g->dim = dim; g->chunk = chunk; g->window = window; g->scales = scales;
+        }
+        *layer = g->n_layer;
+        g->n_layer += passes;
+        return g;
+    }
+    // Recurrent state of a layer: `floats` per sequence slot, for every pass; and the running pass's.
+    float* state(size_t floats) { return static_cast<float*>(alloc(size_t(opt.max_seqs) * floats * size_t(passes) * 4, true)); }
+    float* at_pass(float* state, size_t floats) const { return state + size_t(pass) * size_t(opt.max_seqs) * floats; }
+
+private:
+    WeightStreamer loader_;
+    std::vector<void*> allocs_;
+    int columns_[kBufCount] = {};
+    float* bufs_[kBufCount] = {};
+    int tc_in_ = 8, tc_out_ = 8;
+    Branch branch_;
+    const float* norm_ready_ = nullptr;  // the norm weights x has been prepared with
+};
+
+// ---- layers ----------------------------------------------------------------------------------------------------------
+
+class Mixer {
+public:
+    virtual ~Mixer() = default;
+    // x += mixer(rmsnorm(x; norm)) + the branch set beside it; next_norm as in LayerOps::project_residual.
+    virtual void run(LayerOps& ops, const StepCtx& s, const float* norm, const float* next_norm) = 0;
+    // Threads one time chunk of a recurrence of this mixer occupies (0: none); sizes the chunks of a step.
+    virtual int scan_threads() const { return 0; }
+    virtual int lru_threads() const { return 0; }
+    virtual size_t scan_scratch_per_chunk() const { return 0; }
+    virtual size_t lru_scratch_per_chunk() const { return 0; }
+};
+
+class FeedForward {
+public:
+    virtual ~FeedForward() = default;
+    // x += ff(rmsnorm(x; norm)), after the mixer
+    virtual void run(LayerOps& ops, const StepCtx& s, const float* norm, const float* next_norm) = 0;
+    // ff(rmsnorm(x; norm)) as a branch beside the mixer (LayerOps::set_branch); runs before the mixer does
+    virtual void branch(LayerOps& ops, const StepCtx& s, const float* norm) = 0;
+};
+
+// One function per kind; a further kind is a class in a file of its own and a line in make_mixer / make_feed_forward
+// (hybrid_backend.cpp).
+std::unique_ptr<Mixer> make_selective_scan(LayerOps& ops, const Json& config, const std::string& prefix);
+std::unique_ptr<Mixer> make_parallel(LayerOps& ops, const Json& config, const std::string& prefix);
+std::unique_ptr<Mixer> make_latent_attention(LayerOps& ops, const Json& config, const std::string& prefix);
+std::unique_ptr<FeedForward> make_gated_feed_forward(LayerOps& ops, const Json& config, const std::string& prefix);
+std::unique_ptr<FeedForward> make_mixture(LayerOps& ops, const Json& config, const std::string& prefix);

@@ -19,6 +19,11 @@
 // by TMA), and a matrix may be block-diagonal: output tiles of block b then read the k_block activation columns that
 // start at b * k_block.
 //
+// Grouped products (ingot_grouped_tc_run). One matrix per group of rows - the experts of a mixture - in one launch: the rows are
+// sorted by group, group g's rows are a run of the activation matrix that starts anywhere, and its matrix is the g-th of a stack. A
+// CTA finds its group and row tile from the run starts on the device; boxes that reach into the next run are multiplied along and
+// not stored. The activation of an expert is folded into the epilogue, which then writes the bf16 operand of the next product.
+//
 // Kernel. One CTA = 128 tokens x 128 outputs over a slice of k (split-k fills the GPU when there are few
 // output tiles; slices go to a scratch and are summed in slice order, by a small kernel or by the kernel
 // that consumes the product, so results are reproducible). 6 warps: warp 0 streams [128 rows][64 k] boxes of hi, lo and W (128-byte swizzle, 48 KB per
@@ -26,6 +31,7 @@
 // loop, one elected lane issues); warps 2-5 read the 128x128 f32 accumulator out of tensor memory, one
 // thread per token row. Rows past n_tok and outputs past n_out are zero-filled by TMA and not stored.
 // Every mbarrier wait is bounded; on expiry the CTA raises the workspace's status word and leaves.
+#include "grouped_linear.h"
 #include "../csrc/sm100_ptx.cuh"
 
 #include <cuda_bf16.h>
@@ -101,10 +107,18 @@ struct GemmParams {
     int a_bytes;  // of one activation box: 128 rows, or fewer for a single short token tile
     uint32_t idesc;
     int rows_per_block, k_block, tiles_per_block;  // block-diagonal matrix (rows_per_block > 0, count == 1)
+    // grouped: run starts [n_groups + 1] of the rows; out rows are the sorted rows
+    const int32_t* group_start;
+    int n_groups;
+    const float* row_scale;                // epilogue: accumulator * row_scale[row] (null: none), then act
+    int act;                               // 1: square of relu
+    __nv_bfloat16 *out_hi, *out_lo;        // bf16 plane(s) [rows][n_out] instead of f32
+    __half* out_half;                      // f16 instead of f32: row stride half_ld, block b's columns from b * half_block on
+    int half_ld, half_block;
     int to_partial;  // write the slice(s) to `partial` even when there is only one (a consumer kernel sums them)
 };
 
-template <int kPlanes, int kBN>
+template <int kPlanes, int kBN, bool kGrouped>
 __global__ void __launch_bounds__(kThreads, 1)
 linear_sm100_kernel(const __grid_constant__ CUtensorMap map_hi, const __grid_constant__ CUtensorMap map_lo,
                     const __grid_constant__ CUtensorMap map_w0, const __grid_constant__ CUtensorMap map_w1,
@@ -129,13 +143,45 @@ linear_sm100_kernel(const __grid_constant__ CUtensorMap map_hi, const __grid_con
     const int mat = (tile_n >= p.tile_end[0]) + (tile_n >= p.tile_end[1]);  // warp-uniform
     const CUtensorMap* const map_w_p = mat == 0 ? &map_w0 : mat == 1 ? &map_w1 : &map_w2;
     const int mat_n_out = mat == 0 ? p.n_out[0] : mat == 1 ? p.n_out[1] : p.n_out[2];
+    // grouped: which group's which row tile this is, 32 groups at a time
+    int group = 0, group_m0 = 0, group_end = 0;
+    if (kGrouped) {
+        LINEAR_PDL_WAIT();  // the runs come from a kernel before
+        int tile = tile_m;
+        bool found = false;
+        for (int g0 = 0; g0 < p.n_groups && !found; g0 += 32) {
+            const int mine = g0 + lane;
+            const int a = mine < p.n_groups ? p.group_start[mine] : 0, b = mine < p.n_groups ? p.group_start[mine + 1] : 0;
+            const int n = (b - a + kBM - 1) / kBM;
+            int upto = n;
+#pragma unroll
+            for (int o = 1; o < 32; o <<= 1) {
+                const int v = __shfl_up_sync(0xffffffffu, upto, o);
+                if (lane >= o) upto += v;
+            }
+            const unsigned hit = __ballot_sync(0xffffffffu, tile < upto);
+            if (hit) {
+                const int src = __ffs(hit) - 1;
+                const int local = tile - (__shfl_sync(0xffffffffu, upto, src) - __shfl_sync(0xffffffffu, n, src));
+                group = g0 + src;
+                group_m0 = __shfl_sync(0xffffffffu, a, src) + local * kBM;
+                group_end = __shfl_sync(0xffffffffu, b, src);
+                found = true;
+            } else {
+                tile -= __shfl_sync(0xffffffffu, upto, 31);
+            }
+        }
+        if (!found) return;  // the grid covers the most row tiles there can be
+    }
+    const int row_end = kGrouped ? group_end : p.n_tok;
     const int blk = p.tiles_per_block > 0 ? tile_n / p.tiles_per_block : 0;
     const int col_end = p.tiles_per_block > 0 ? (blk + 1) * p.rows_per_block : mat_n_out;
     const int a_k0 = blk * p.k_block;  // first activation column of this tile's products
     float* const mat_partial = mat == 0 ? p.partial[0] : mat == 1 ? p.partial[1] : p.partial[2];
     const int n0 = p.tiles_per_block > 0 ? blk * p.rows_per_block + (tile_n - blk * p.tiles_per_block) * kBN
                                          : (tile_n - (mat == 0 ? 0 : mat == 1 ? p.tile_end[0] : p.tile_end[1])) * kBN;
-    const int m0 = tile_m * kBM, split = blockIdx.z;
+    const int m0 = kGrouped ? group_m0 : tile_m * kBM, split = blockIdx.z;
+    const int w_row0 = kGrouped ? group * mat_n_out + n0 : n0;  // row of the weight matrix, or of the stack of matrices
     const int ks_begin = (int)((long long)p.k_steps * split / p.n_split);
     const int ks_end = (int)((long long)p.k_steps * (split + 1) / p.n_split);
     const int n_it = ks_end - ks_begin;
@@ -163,10 +209,10 @@ linear_sm100_kernel(const __grid_constant__ CUtensorMap map_hi, const __grid_con
         for (int it = 0; it < n_pre; it++) {
             const uint32_t full = smem_u32(&bars->full[it]);
             mbar_expect_tx(full, stage_tx);
-            tma_load_2d(smem_base + it * kStageBytes + kOffW, map_w_p, (ks_begin + it) * kBK, n0, full);
+            tma_load_2d(smem_base + it * kStageBytes + kOffW, map_w_p, (ks_begin + it) * kBK, w_row0, full);
         }
     }
-    LINEAR_PDL_WAIT();
+    if (!kGrouped) LINEAR_PDL_WAIT();
 
     if (warp_u == 0) {
         // ---------------- TMA producer ----------------
@@ -187,7 +233,7 @@ linear_sm100_kernel(const __grid_constant__ CUtensorMap map_hi, const __grid_con
                         mbar_expect_tx(full, stage_tx);
                         tma_load_2d(dst, &map_hi, a_k0 + k, m0, full);
                         if (kPlanes > 1) tma_load_2d(dst + kBoxBytes, &map_lo, a_k0 + k, m0, full);
-                        tma_load_2d(dst + kOffW, map_w_p, k, n0, full);
+                        tma_load_2d(dst + kOffW, map_w_p, k, w_row0, full);
                     }
                 }
             }
@@ -236,23 +282,59 @@ linear_sm100_kernel(const __grid_constant__ CUtensorMap map_hi, const __grid_con
             tc_fence_after();
             float* dst = (split_k ? mat_partial + (size_t)split * p.n_tok * mat_n_out : p.out) + (size_t)row * mat_n_out + n0;
             const bool add = !split_k && p.accumulate;
+            const float scale = p.row_scale && row < row_end ? p.row_scale[row] : 1.0f;
 #pragma unroll
             for (int c = 0; c < kBN / 32; c++) {
                 float v[32];
                 tmem_ld32(tmem + ((uint32_t)(lg * 32) << 16) + c * 32, v);
                 tmem_wait_ld();
-                if (row < p.n_tok) {
+                if (row < row_end) {
+                    if (kGrouped && (p.row_scale || p.act)) {
 #pragma unroll
-                    for (int i = 0; i < 32; i += 4) {
-                        const int col = n0 + c * 32 + i;
-                        if (col + 3 < col_end) {
-                            float4* d4 = reinterpret_cast<float4*>(dst + c * 32 + i);
-                            float4 o = make_float4(v[i], v[i + 1], v[i + 2], v[i + 3]);
-                            if (add) { const float4 old = *d4; o.x += old.x; o.y += old.y; o.z += old.z; o.w += old.w; }
-                            *d4 = o;
-                        } else {
+                        for (int i = 0; i < 32; i++) {
+                            v[i] *= scale;
+                            if (p.act == 1) v[i] = v[i] > 0.f ? v[i] * v[i] : 0.f;
+                        }
+                    }
+                    if (kGrouped && p.out_hi) {  // n_out is a multiple of 8
+#pragma unroll
+                        for (int i = 0; i < 32; i += 8) {
+                            const int col = n0 + c * 32 + i;
+                            if (col >= col_end) break;
+                            const size_t at = (size_t)row * mat_n_out + col;
+                            __nv_bfloat162 h[4], l[4];
+#pragma unroll
+                            for (int e = 0; e < 4; e++) {
+                                h[e] = __floats2bfloat162_rn(v[i + 2 * e], v[i + 2 * e + 1]);
+                                l[e] = __floats2bfloat162_rn(v[i + 2 * e] - __low2float(h[e]), v[i + 2 * e + 1] - __high2float(h[e]));
+                            }
+                            *reinterpret_cast<uint4*>(p.out_hi + at) = *reinterpret_cast<const uint4*>(h);
+                            if (p.out_lo) *reinterpret_cast<uint4*>(p.out_lo + at) = *reinterpret_cast<const uint4*>(l);
+                        }
+                    } else if (!kGrouped && p.out_half) {  // n_out and the blocks are multiples of 8
+#pragma unroll
+                        for (int i = 0; i < 32; i += 8) {
+                            const int col = n0 + c * 32 + i;
+                            if (col >= col_end) break;
+                            __half2 h[4];
+#pragma unroll
                             for (int e = 0; e < 4; e++)
-                                if (col + e < col_end) dst[c * 32 + i + e] = add ? dst[c * 32 + i + e] + v[i + e] : v[i + e];
+                                h[e] = __floats2half2_rn(fminf(fmaxf(v[i + 2 * e], -65504.f), 65504.f), fminf(fmaxf(v[i + 2 * e + 1], -65504.f), 65504.f));
+                            *reinterpret_cast<uint4*>(p.out_half + (size_t)row * p.half_ld + blk * p.half_block + (col - blk * p.rows_per_block)) = *reinterpret_cast<const uint4*>(h);
+                        }
+                    } else {
+#pragma unroll
+                        for (int i = 0; i < 32; i += 4) {
+                            const int col = n0 + c * 32 + i;
+                            if (col + 3 < col_end) {
+                                float4* d4 = reinterpret_cast<float4*>(dst + c * 32 + i);
+                                float4 o = make_float4(v[i], v[i + 1], v[i + 2], v[i + 3]);
+                                if (add) { const float4 old = *d4; o.x += old.x; o.y += old.y; o.z += old.z; o.w += old.w; }
+                                *d4 = o;
+                            } else {
+                                for (int e = 0; e < 4; e++)
+                                    if (col + e < col_end) dst[c * 32 + i + e] = add ? dst[c * 32 + i + e] + v[i + e] : v[i + e];
+                            }
                         }
                     }
                 }
@@ -384,9 +466,10 @@ __global__ void finish_group_kernel(const FinishGroup g, int n_tok) {
 
 // x[t][:] += sum of slices (the residual add of wo / down), then, if norm_w is given, hi/lo of rmsnorm(x[t]) for the
 // next projections. One CTA per token.
+// pair_rows (may be null): rows of another branch that go into the sum, token t's at row_of[t * top + k] (row_of null: t).
 template <int kAct>
 __global__ void finish_residual_norm_kernel(float* x, const Slices in, __half* hi, __half* lo, const float* norm_w, int n, int n_mean, int n_tok,
-                                            float eps) {
+                                            float eps, const float* pair_rows, const int32_t* row_of, int top) {
     __shared__ float red[32];
     LINEAR_PDL_TRIGGER();
     LINEAR_PDL_WAIT();
@@ -394,7 +477,11 @@ __global__ void finish_residual_norm_kernel(float* x, const Slices in, __half* h
     const size_t slice = (size_t)n_tok * n;
     float ss = 0.f;
     for (int i = threadIdx.x * 4; i < n; i += blockDim.x * 4) {
-        const float4 v = sum_slices(in, row + i, slice, *reinterpret_cast<const float4*>(x + row + i));
+        float4 v = sum_slices(in, row + i, slice, *reinterpret_cast<const float4*>(x + row + i));
+        for (int k = 0; k < top; k++) {
+            const float4 a = *reinterpret_cast<const float4*>(pair_rows + (row_of ? (size_t)row_of[blockIdx.x * top + k] : (size_t)blockIdx.x) * n + i);
+            v.x += a.x; v.y += a.y; v.z += a.z; v.w += a.w;
+        }
         *reinterpret_cast<float4*>(x + row + i) = v;
         ss += v.x * v.x; ss += v.y * v.y; ss += v.z * v.z; ss += v.w * v.w;
     }
@@ -498,7 +585,7 @@ struct ingot_linear_ws {
     int box_rows = 128;
     int prepared_tok = 0, prepared_in = 0;
     CUtensorMap map_hi, map_lo;
-    std::map<std::tuple<const void*, int, int, int>, CUtensorMap> w_maps;  // one per weight matrix
+    std::map<std::tuple<const void*, int, int, int>, CUtensorMap> w_maps;  // one per weight matrix (and per row count of grouped activations)
 };
 
 // (Re)builds the activation tensor maps when the prepared shape changes.
@@ -534,9 +621,12 @@ static cudaError_t ws_create(ingot_linear_ws** out, size_t act_elems, size_t par
         (e = cudaMemset(ws->hi, 0, ws->act_elems * 2)) != cudaSuccess || (e = cudaMemset(ws->lo, 0, ws->act_elems * 2)) != cudaSuccess ||
         (e = cudaMalloc(&ws->partial, n_slots * ws->partial_floats * 4)) != cudaSuccess || (e = cudaMalloc(&ws->status, sizeof(int))) != cudaSuccess ||
         (e = cudaMemset(ws->status, 0, sizeof(int))) != cudaSuccess ||
-        (e = cudaFuncSetAttribute(linear_sm100_kernel<2, 128>, cudaFuncAttributeMaxDynamicSharedMemorySize, Ring<2, 128>::kSmemBytes)) != cudaSuccess ||
-        (e = cudaFuncSetAttribute(linear_sm100_kernel<1, 128>, cudaFuncAttributeMaxDynamicSharedMemorySize, Ring<1, 128>::kSmemBytes)) != cudaSuccess ||
-        (e = cudaFuncSetAttribute(linear_sm100_kernel<1, 256>, cudaFuncAttributeMaxDynamicSharedMemorySize, Ring<1, 256>::kSmemBytes)) != cudaSuccess) {
+        (e = cudaFuncSetAttribute(linear_sm100_kernel<2, 128, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, Ring<2, 128>::kSmemBytes)) != cudaSuccess ||
+        (e = cudaFuncSetAttribute(linear_sm100_kernel<1, 128, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, Ring<1, 128>::kSmemBytes)) != cudaSuccess ||
+        (e = cudaFuncSetAttribute(linear_sm100_kernel<1, 256, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, Ring<1, 256>::kSmemBytes)) != cudaSuccess ||
+        (e = cudaFuncSetAttribute(linear_sm100_kernel<2, 128, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, Ring<2, 128>::kSmemBytes)) != cudaSuccess ||
+        (e = cudaFuncSetAttribute(linear_sm100_kernel<1, 128, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, Ring<1, 128>::kSmemBytes)) != cudaSuccess ||
+        (e = cudaFuncSetAttribute(linear_sm100_kernel<1, 256, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, Ring<1, 256>::kSmemBytes)) != cudaSuccess) {
         cudaFree(ws->hi); cudaFree(ws->lo); cudaFree(ws->partial); cudaFree(ws->status);
         delete ws;
         return e;
@@ -630,7 +720,8 @@ cudaError_t ingot_linear_tc_prepare_norm_bf16(ingot_linear_ws* ws, const float* 
 // rows_per_block > 0 (count == 1): block-diagonal; n_in is then the row length of one block and the prepared activations hold
 // n_out / rows_per_block such blocks side by side.
 static cudaError_t launch_gemm(ingot_linear_ws* ws, float* out, const void* const* w, int n_in, const int* n_out, int count,
-                               int accumulate, int first_slot, bool to_partial, bool append, cudaStream_t s, int rows_per_block = 0) {
+                               int accumulate, int first_slot, bool to_partial, bool append, cudaStream_t s, int rows_per_block = 0,
+                               __half* out_half = nullptr, int half_ld = 0, int half_block = 0) {
     const int n_tok = ws->prepared_tok;
     if (rows_per_block > 0 && (count != 1 || n_out[0] % rows_per_block != 0 || rows_per_block % 4 != 0 || n_in % 8 != 0)) return cudaErrorInvalidValue;
     const int act_in = rows_per_block > 0 ? n_in * (n_out[0] / rows_per_block) : n_in;
@@ -676,7 +767,10 @@ static cudaError_t launch_gemm(ingot_linear_ws* ws, float* out, const void* cons
     const int k_steps = (n_in + kBK - 1) / kBK;
     // enough k slices to give every SM a CTA, at least 4 k-steps each, and no more than the slots hold
     if (to_partial && fit < 1) return cudaErrorInvalidValue;
-    const int n_split = std::max(1, std::min({ws->num_sms / tiles, k_steps / 4, fit}));
+    const int n_split = out_half ? 1 : std::max(1, std::min({ws->num_sms / tiles, k_steps / 4, fit}));
+    p.out_half = out_half;
+    p.half_ld = half_ld;
+    p.half_block = half_block;
     p.out = out; p.status = ws->status;
     p.n_tok = n_tok; p.k_steps = k_steps; p.n_split = n_split; p.accumulate = accumulate;
     p.to_partial = to_partial ? 1 : 0;
@@ -688,9 +782,9 @@ static cudaError_t launch_gemm(ingot_linear_ws* ws, float* out, const void* cons
     auto run = [&](auto kernel, int smem) {
         return launch_pdl(kernel, grid, dim3(kThreads), (size_t)smem, s, ws->map_hi, ws->map_lo, *maps[0], *maps[1], *maps[2], p);
     };
-    cudaError_t le = ws->planes > 1 ? run(linear_sm100_kernel<2, 128>, Ring<2, 128>::kSmemBytes)
-                   : kBN == 256     ? run(linear_sm100_kernel<1, 256>, Ring<1, 256>::kSmemBytes)
-                                    : run(linear_sm100_kernel<1, 128>, Ring<1, 128>::kSmemBytes);
+    cudaError_t le = ws->planes > 1 ? run(linear_sm100_kernel<2, 128, false>, Ring<2, 128>::kSmemBytes)
+                   : kBN == 256     ? run(linear_sm100_kernel<1, 256, false>, Ring<1, 256>::kSmemBytes)
+                                    : run(linear_sm100_kernel<1, 128, false>, Ring<1, 128>::kSmemBytes);
     if (le != cudaSuccess) return le;
     for (int m = 0; m < count; m++) {
         ws->slot_split[first_slot + m] = held + n_split;
@@ -714,6 +808,65 @@ cudaError_t ingot_linear_tc_run(ingot_linear_ws* ws, float* out, const void* w, 
 // b * k_block .. (b + 1) * k_block - 1.
 cudaError_t ingot_linear_tc_run_blocks(ingot_linear_ws* ws, float* out, const void* w, int k_block, int n_out, int rows_per_block, cudaStream_t s) {
     return launch_gemm(ws, out, &w, k_block, &n_out, 1, 0, 0, false, false, s, rows_per_block);
+}
+
+// Plain (rows_per_block 0) or block-diagonal product with an f16 result: row t at out + t * out_ld, block b's columns from b * out_block
+// on. Row lengths and blocks are multiples of 8.
+cudaError_t ingot_linear_tc_run_half(ingot_linear_ws* ws, void* out, int out_ld, int out_block, const void* w, int n_in, int n_out, int rows_per_block,
+                                     cudaStream_t s) {
+    if (out_ld % 8 != 0 || out_block % 8 != 0 || n_out % 8 != 0 || rows_per_block % 8 != 0) return cudaErrorInvalidValue;
+    return launch_gemm(ws, nullptr, &w, n_in, &n_out, 1, 0, 0, false, false, s, rows_per_block, static_cast<__half*>(out), out_ld, out_block);
+}
+
+cudaError_t ingot_grouped_tc_run(ingot_linear_ws* ws, const ingot_grouped_gemm* g, cudaStream_t s) {
+    if (!ws->bf16 || g->n_in % 8 != 0 || g->n_out % 8 != 0 || g->n_rows < 1 || g->n_groups < 1 || g->rows_per_group < 1) return cudaErrorInvalidValue;
+    const int planes = g->a_lo ? 2 : 1, box_rows = g->rows_per_group >= 128 ? 128 : (g->rows_per_group + 7) / 8 * 8;
+    GemmParams p = {};
+    p.tiles_m = g->n_rows / kBM + std::min(g->n_rows, g->n_groups);  // at least as many as there can be
+    // as for plain products: 256 outputs per CTA if that saves waves, judged by the row tiles of evenly filled groups
+    const int likely = std::max(1, std::min(g->n_groups, g->n_rows) * ((g->n_rows / std::min(g->n_groups, g->n_rows) + kBM - 1) / kBM));
+    int kBN = 128;
+    if (planes == 1) {
+        const long long waves128 = ((long long)((g->n_out + 127) / 128) * likely + ws->num_sms - 1) / ws->num_sms;
+        const long long waves256 = ((long long)((g->n_out + 255) / 256) * likely + ws->num_sms - 1) / ws->num_sms;
+        if (waves128 > 1 && 3 * waves256 < 2 * waves128) kBN = 256;
+    }
+    auto map_of = [&](const void* base, int rows, int cols, int box) -> const CUtensorMap* {
+        const auto key = std::make_tuple(base, rows, cols, box);
+        auto it = ws->w_maps.find(key);
+        if (it == ws->w_maps.end()) {
+            CUtensorMap tm;
+            if (!make_map(&tm, base, rows, cols, box, true)) return nullptr;
+            if (ws->w_maps.size() > 65536) ws->w_maps.clear();
+            it = ws->w_maps.emplace(key, tm).first;
+        }
+        return &it->second;
+    };
+    const CUtensorMap* hi = map_of(g->a_hi, g->n_rows, g->n_in, box_rows);
+    const CUtensorMap* lo = planes > 1 ? map_of(g->a_lo, g->n_rows, g->n_in, box_rows) : hi;
+    const CUtensorMap* w = map_of(g->w, g->n_groups * g->n_out, g->n_in, kBN);
+    if (!hi || !lo || !w) return cudaErrorUnknown;
+    p.tiles_n = (g->n_out + kBN - 1) / kBN;
+    for (int m = 0; m < 3; m++) { p.n_out[m] = g->n_out; p.tile_end[m] = p.tiles_n; }
+    p.out = g->out;
+    p.status = ws->status;
+    p.n_tok = g->n_rows;
+    p.k_steps = (g->n_in + kBK - 1) / kBK;
+    p.n_split = 1;
+    p.a_bytes = box_rows * kBK * 2;
+    p.idesc = idesc_f16(kBN) | kIdescBF16;
+    p.group_start = g->group_start;
+    p.n_groups = g->n_groups;
+    p.row_scale = g->row_scale;
+    p.act = g->act;
+    p.out_hi = static_cast<__nv_bfloat16*>(g->out_hi);
+    p.out_lo = static_cast<__nv_bfloat16*>(g->out_lo);
+    auto run = [&](auto kernel, int smem) {
+        return launch_pdl(kernel, dim3(p.tiles_n * p.tiles_m), dim3(kThreads), (size_t)smem, s, *hi, *lo, *w, *w, *w, p);
+    };
+    return planes > 1   ? run(linear_sm100_kernel<2, 128, true>, Ring<2, 128>::kSmemBytes)
+           : kBN == 256 ? run(linear_sm100_kernel<1, 256, true>, Ring<1, 256>::kSmemBytes)
+                        : run(linear_sm100_kernel<1, 128, true>, Ring<1, 128>::kSmemBytes);
 }
 
 // The same product left as k slices in scratch slot 0..2 for one of the ingot_linear_tc_finish_* calls below.
@@ -755,17 +908,19 @@ cudaError_t ingot_linear_tc_finish_group(ingot_linear_ws* ws, float* const* outs
 cudaError_t ingot_linear_tc_finish_residual_norm(ingot_linear_ws* ws, float* x, const float* norm_w, float eps, int slot, cudaStream_t s) {
     const int n = ws->slot_out[slot], n_tok = ws->prepared_tok;
     if (n % 4 != 0 || (norm_w && !act_shape_ok(ws, n, n_tok)) || ws->bf16) return cudaErrorInvalidValue;
-    cudaError_t le = launch_pdl(finish_residual_norm_kernel<kActF16Pair>, dim3(n_tok), dim3(256), 0, s, x, slices_of(ws, slot), ws->hi, ws->lo, norm_w, n, n, n_tok, eps);
+    cudaError_t le = launch_pdl(finish_residual_norm_kernel<kActF16Pair>, dim3(n_tok), dim3(256), 0, s, x, slices_of(ws, slot), ws->hi, ws->lo, norm_w, n, n, n_tok, eps, (const float*)nullptr, (const int32_t*)nullptr, 0);
     if (le != cudaSuccess) return le;
     return norm_w ? set_prepared(ws, n, n_tok) : cudaGetLastError();
 }
+// pair_rows (null: none): x[t] also takes in the rows row_of[t * top + k] of it.
 cudaError_t ingot_linear_tc_finish_residual_norm_bf16(ingot_linear_ws* ws, float* x, const float* norm_w, float eps, int n_mean, int planes,
-                                                      cudaStream_t s) {
+                                                      const float* pair_rows, const int32_t* row_of, int top, cudaStream_t s) {
+    if (!pair_rows) top = 0;
     const int n = ws->slot_out[0], n_tok = ws->prepared_tok;
     if (n % 4 != 0 || (norm_w && !act_shape_ok(ws, n, n_tok)) || !ws->bf16) return cudaErrorInvalidValue;
     cudaError_t le = planes > 1
-        ? launch_pdl(finish_residual_norm_kernel<kActBF16Pair>, dim3(n_tok), dim3(256), 0, s, x, slices_of(ws, 0), ws->hi, ws->lo, norm_w, n, n_mean, n_tok, eps)
-        : launch_pdl(finish_residual_norm_kernel<kActBF16>, dim3(n_tok), dim3(256), 0, s, x, slices_of(ws, 0), ws->hi, ws->lo, norm_w, n, n_mean, n_tok, eps);
+        ? launch_pdl(finish_residual_norm_kernel<kActBF16Pair>, dim3(n_tok), dim3(256), 0, s, x, slices_of(ws, 0), ws->hi, ws->lo, norm_w, n, n_mean, n_tok, eps, pair_rows, row_of, top)
+        : launch_pdl(finish_residual_norm_kernel<kActBF16>, dim3(n_tok), dim3(256), 0, s, x, slices_of(ws, 0), ws->hi, ws->lo, norm_w, n, n_mean, n_tok, eps, pair_rows, row_of, top);
     if (le != cudaSuccess) return le;
     ws->planes = planes > 1 ? 2 : 1;
     return norm_w ? set_prepared(ws, n, n_tok) : cudaGetLastError();

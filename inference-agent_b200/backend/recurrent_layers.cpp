@@ -1,0 +1,180 @@
+// Recurrent mixers of the model-folder backend: selective scan, and attention beside a gated linear recurrent unit.
+#include "layer_ops.h"
+
+namespace {
+
+// Selective scan (Mamba): [x | z] = W_in h; x <- silu(conv(x)); [dt | B | C] = W_x x; dt <- W_dt dt; scan; W_o (y silu(z)).
+std::vector<float> pad_rows(const std::vector<float>& v, int rows, int cols, int rows_p, int cols_p) {
+    std::vector<float> out(size_t(rows_p) * cols_p, 0.f);
+    for (int r = 0; r < rows; r++) std::copy(v.begin() + size_t(r) * cols, v.begin() + size_t(r + 1) * cols, out.begin() + size_t(r) * cols_p);
+    return out;
+}
+
+class SelectiveScanMixer : public Mixer {
+public:
+    SelectiveScanMixer(LayerOps& ops, const Json& c, const std::string& p) {
+        inner_ = get_int(c, "inner");
+        states_ = get_int(c, "state", 1, 256);
+        taps_ = get_int(c, "conv", 1, 16);
+        const int rank = get_int(c, "dt_rank"), d = ops.width;
+        const Groups in = flat(inner_), rk = flat(rank);
+        ip_ = in.padded;
+        np_ = ingot_scan_state_pad(states_);
+        rank_p_ = rk.padded;
+        w_in_ = ops.matrix(2 * ip_, flat(d).padded, {Part{p + "in", {2 * inner_, d}, {2, inner_, ip_}, flat(d)}});
+        conv_w_ = ops.upload(pad_rows(tensor_f32(ops.dir.tensor(p + "conv", {inner_, taps_})), inner_, taps_, ip_, taps_));
+        conv_b_ = ops.vector(p + "conv.b", inner_);
+        // rows of W_x: dt, B and C each start on a padded place, so that B and C rows can be fetched 16 bytes at a time
+        const std::vector<int64_t> x_shape = {rank + 2 * states_, inner_};
+        const Groups st = {1, states_, np_};
+        w_x_ = ops.matrix(rank_p_ + 2 * np_, ip_, {Part{p + "x", x_shape, rk, in, 0, 0, 0}, Part{p + "x", x_shape, st, in, rank_p_, 0, rank},
+                                                   Part{p + "x", x_shape, st, in, rank_p_ + np_, 0, rank + states_}});
+        w_dt_ = ops.matrix(ip_, rank_p_, {Part{p + "dt", {inner_, rank}, in, rk}});
+        dt_b_ = ops.vector(p + "dt.b", inner_);
+        std::vector<float> a = tensor_f32(ops.dir.tensor(p + "A_log", {inner_, states_}));
+        for (float& v : a) v = float(-std::exp(double(v)) * 1.4426950408889634);  // exp(dt A) = 2^(dt A log2 e)
+        a2_ = ops.upload(pad_rows(a, inner_, states_, ip_, np_));
+        d_ = ops.vector(p + "D", inner_);
+        w_o_ = ops.matrix(p + "o", flat(d), in);
+        conv_state_ = ops.state(size_t(taps_ - 1) * ip_);
+        state_ = ops.state(size_t(ip_) * np_);
+        ops.need(kProj, 2 * ip_);
+        ops.need(kConv, ip_);
+        ops.need(kStateIn, rank_p_ + 2 * np_);
+        ops.need(kDt, ip_);
+        ops.need(kMix, ip_);
+    }
+    void run(LayerOps& ops, const StepCtx& s, const float* norm, const float* next_norm) override {
+        float *xz = ops.buf(kProj), *xc = ops.buf(kConv), *dbc = ops.buf(kStateIn), *dt = ops.buf(kDt);
+        const int ld_bc = rank_p_ + 2 * np_;
+        ops.norm_project(s, xz, w_in_, norm);
+        const ingot_act_out conv = ops.operand(s, xc, ip_, true);
+        ingot_check(ingot_causal_conv(&s.st, xz, 2 * ip_, nullptr, conv_w_, conv_b_, taps_, ip_, ops.opt.f32 ? 1 : 2, ops.at_pass(conv_state_, size_t(taps_ - 1) * ip_), &conv, ops.stream));
+        ops.operand_ready(s, ip_);
+        ops.project(s, dbc, w_x_, xc, ip_);
+        ops.project_rows(s, dt, w_dt_, dbc, ld_bc, 2);
+        const ingot_act_out y = ops.operand(s, ops.buf(kMix), ip_, false);
+        ingot_check(ingot_selective_scan(&s.st, &s.scan, xc, ip_, dt, ip_, dt_b_, dbc, ld_bc, rank_p_, rank_p_ + np_, xz + ip_, 2 * ip_, a2_, d_,
+                                         ops.at_pass(state_, size_t(ip_) * np_), ip_, states_, ops.opt.f32 ? 1 : 0, &y, ops.stream));
+        ops.operand_ready(s, ip_);
+        ops.project_residual(s, w_o_, ops.buf(kMix), next_norm);
+    }
+    int scan_threads() const override { return ip_ * 2; }
+    size_t scan_scratch_per_chunk() const override { return size_t(ip_) * (np_ + 1); }
+
+private:
+    int inner_, states_, taps_, ip_, np_, rank_p_;
+    Matrix w_in_, w_x_, w_dt_, w_o_;
+    float *conv_w_, *conv_b_, *dt_b_, *a2_, *d_, *conv_state_, *state_;
+};
+
+// Attention beside a gated linear recurrent unit, both reading the same normalised input:
+//   left   chunk-local attention over shared key/value rows (ingot_skv_*)
+//   right  y = gelu(W_y h + b), u = conv(W_x h + b), gates from block-diagonal products of u, S; output S * y
+// x += W_left (left_scale * attention) + W_right (right_scale * recurrence): one input product for the four input matrices
+// and one output product over the two results side by side.
+class ParallelMixer : public Mixer {
+public:
+    ParallelMixer(LayerOps& ops, const Json& c, const std::string& p) {
+        const Json &l = c.at("left"), &r = c.at("right");
+        const int d = ops.width;
+        left_scale_ = get_float(c, "left_scale");
+        right_scale_ = get_float(c, "right_scale");
+        heads_ = get_int(l, "heads");
+        kv_heads_ = get_int(l, "kv_heads");
+        dim_ = get_int(l, "dim");
+        if (heads_ % kv_heads_ != 0) throw std::runtime_error("model config: \"heads\" is not a multiple of \"kv_heads\"");
+        if (l.has("vdim") && get_int(l, "vdim") != dim_) throw std::runtime_error("model config: values that are the keys need \"vdim\" equal to \"dim\"");
+        scale_ = get_float(l, "scale");
+        const int chunk = l.has("mask") && !l.at("mask").is_null() ? get_int(l.at("mask"), "size") : 0;
+        const int row = ops.opt.f32 ? round_up(dim_, 8) : ingot_skv_row_length(dim_);
+        if (row < 2 || row > 512) throw std::runtime_error("model config: heads of more than 512 values are not supported");
+        row_ = row;
+        cache_ = ops.cache_group(kv_heads_, row, chunk, 0, true, &cache_layer_);
+
+        width_ = get_int(r, "width");
+        const int blocks = get_int(r, "blocks");
+        taps_ = get_int(r, "conv", 1, 16);
+        if (width_ % blocks != 0) throw std::runtime_error("model config: \"width\" is not a multiple of \"blocks\"");
+        const int m = width_ / blocks, mp = round_up(m, 8);
+        const Groups q = {heads_, dim_, row}, k = {kv_heads_, dim_, row}, w = {blocks, m, mp}, in = flat(d);
+        wp_ = w.width();
+        block_ = mp;
+        const std::string L = p + "left.", R = p + "right.";
+        k_off_ = q.width();
+        y_off_ = k_off_ + k.width();
+        x_off_ = y_off_ + wp_;
+        proj_ld_ = x_off_ + wp_;
+        w_in_ = ops.matrix(proj_ld_, in.padded, {Part{L + "q", {q.count(), d}, q, in, 0}, Part{L + "k", {k.count(), d}, k, in, k_off_},
+                                                 Part{R + "y", {width_, d}, w, in, y_off_}, Part{R + "x", {width_, d}, w, in, x_off_}});
+        q_norm_ = ops.vector(L + "q.norm", {q.count()}, q);
+        k_norm_ = ops.vector(L + "k.norm", {k.count()}, k);
+        y_b_ = ops.vector(R + "y.b", {width_}, w);
+        x_b_ = ops.vector(R + "x.b", {width_}, w);
+        std::vector<float> cw = tensor_f32(ops.dir.tensor(R + "conv", {width_, taps_})), cw_p(size_t(wp_) * taps_, 0.f);
+        for (int i = 0; i < width_; i++) std::copy(cw.begin() + size_t(i) * taps_, cw.begin() + size_t(i + 1) * taps_, cw_p.begin() + size_t(i / m * mp + i % m) * taps_);
+        conv_w_ = ops.upload(cw_p);
+        conv_b_ = ops.vector(R + "conv.b", {width_}, w);
+        // block b: m rows of the recurrence gate, then m rows of the input gate
+        const Groups gate_rows = {blocks, m, 2 * mp}, gate_cols = {1, m, mp};
+        w_gates_ = ops.matrix(2 * wp_, mp, {Part{R + "ra", {blocks, m, m}, gate_rows, gate_cols, 0}, Part{R + "ri", {blocks, m, m}, gate_rows, gate_cols, mp}}, 2 * mp);
+        r_b_ = ops.vector(R + "ra.b", {blocks, m}, w);
+        i_b_ = ops.vector(R + "ri.b", {blocks, m}, w);
+        std::vector<float> lam = ops.host_vector(R + "lam", {width_}, w);
+        for (float& v : lam) v = float(double(v) > 30 ? double(v) : std::log1p(std::exp(double(v))));
+        softplus_lam_ = ops.upload(lam);
+        const Groups heads_out = flat(q.count());
+        attn_cols_ = heads_out.padded;
+        mix_ld_ = attn_cols_ + wp_;
+        w_o_ = ops.matrix(in.padded, mix_ld_, {Part{L + "o", {d, q.count()}, in, heads_out, 0, 0}, Part{R + "o", {d, width_}, in, w, 0, attn_cols_}});
+        conv_state_ = ops.state(size_t(taps_ - 1) * wp_);
+        state_ = ops.state(size_t(wp_));
+        ops.need(kProj, proj_ld_);
+        ops.need(kConv, wp_);
+        ops.need(kGates, 2 * wp_);
+        ops.need(kMix, mix_ld_);
+        ops.need(kQuery, q.width());
+    }
+    void run(LayerOps& ops, const StepCtx& s, const float* norm, const float* next_norm) override {
+        float *proj = ops.buf(kProj), *u = ops.buf(kConv), *gates = ops.buf(kGates), *mix = ops.buf(kMix);
+        const CacheGroup& g = *cache_;
+        ops.norm_project(s, proj, w_in_, norm);
+        const ingot_act_out conv = ops.operand(s, u, wp_, true, 2);
+        ingot_check(ingot_causal_conv(&s.st, proj + x_off_, proj_ld_, x_b_, conv_w_, conv_b_, taps_, wp_, 0, ops.at_pass(conv_state_, size_t(taps_ - 1) * wp_), &conv, ops.stream));
+        ops.operand_ready(s, wp_, 2);
+        ops.project(s, gates, w_gates_, u, wp_);
+        ingot_check(ingot_skv_append(g.kv, cache_layer_ + ops.pass, &s.st, proj, proj_ld_, 0, k_off_, heads_, dim_, q_norm_, k_norm_, ops.eps, ops.buf(kQuery),
+                                     g.tables, g.first_page, g.width, ops.stream));
+        // the two results side by side are the operand of the output product
+        const ingot_act_out left = ops.operand(s, mix, mix_ld_, false);
+        ingot_check(ingot_skv_attend(g.kv, cache_layer_ + ops.pass, &s.st, ops.buf(kQuery), heads_, dim_, scale_, left_scale_, &left, g.tables, g.first_page, g.width,
+                                     0, ops.stream));
+        ingot_act_out right = left;
+        if (right.f32) right.f32 += attn_cols_;
+        if (right.hi) right.hi = static_cast<char*>(right.hi) + size_t(attn_cols_) * 2;
+        if (right.lo) right.lo = static_cast<char*>(right.lo) + size_t(attn_cols_) * 2;
+        ingot_check(ingot_gated_lru(&s.st, &s.lru, u, wp_, gates, 2 * wp_, block_, r_b_, i_b_, softplus_lam_, proj + y_off_, proj_ld_, y_b_, ops.at_pass(state_, size_t(wp_)), wp_,
+                                    right_scale_, ops.opt.f32 ? 1 : 0, &right, ops.stream));
+        ops.operand_ready(s, mix_ld_);
+        ops.project_residual(s, w_o_, mix, next_norm);
+    }
+    int lru_threads() const override { return wp_; }
+    size_t lru_scratch_per_chunk() const override { return 2 * size_t(wp_); }
+
+private:
+    int heads_, kv_heads_, dim_, row_, width_, wp_, block_, taps_, cache_layer_ = 0;
+    int k_off_, y_off_, x_off_, proj_ld_, attn_cols_, mix_ld_;
+    float scale_, left_scale_, right_scale_;
+    CacheGroup* cache_;
+    Matrix w_in_, w_gates_, w_o_;
+    float *q_norm_, *k_norm_, *y_b_, *x_b_, *conv_w_, *conv_b_, *r_b_, *i_b_, *softplus_lam_, *conv_state_, *state_;
+};
+
+}  // namespace
+
+std::unique_ptr<Mixer> make_selective_scan(LayerOps& ops, const Json& config, const std::string& prefix) {
+    return std::make_unique<SelectiveScanMixer>(ops, config, prefix);
+}
+std::unique_ptr<Mixer> make_parallel(LayerOps& ops, const Json& config, const std::string& prefix) {
+    return std::make_unique<ParallelMixer>(ops, config, prefix);
+}

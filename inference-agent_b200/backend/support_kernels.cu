@@ -563,6 +563,49 @@ __global__ void embed_rows_kernel(float* out, const W* __restrict__ table, int n
     for (int i = threadIdx.x; i < n_in; i += blockDim.x) o[i] = embed_to_f32(src[i]);
 }
 
+// The same from two tables, added; `copy` (may be null) receives the rows too. A row index outside its table gives zeros and raises *status.
+__global__ void embed_sum_kernel(float* out, float* copy, const __nv_bfloat16* __restrict__ table, int n_table, const int32_t* __restrict__ rows,
+                                 const __nv_bfloat16* __restrict__ table2, int n_table2, const int32_t* __restrict__ rows2, int n, int* status) {
+    const int a = rows[blockIdx.x], b = table2 ? rows2[blockIdx.x] : 0;
+    const bool ok = a >= 0 && a < n_table && (!table2 || (b >= 0 && b < n_table2));
+    if (!ok && threadIdx.x == 0) atomicOr(status, 1);
+    for (int i = threadIdx.x; i < n; i += blockDim.x) {
+        float v = ok ? __bfloat162float(table[(size_t)a * n + i]) : 0.f;
+        if (ok && table2) v += __bfloat162float(table2[(size_t)b * n + i]);
+        out[(size_t)blockIdx.x * n + i] = v;
+        if (copy) copy[(size_t)blockIdx.x * n + i] = v;
+    }
+}
+
+// [a | b] row by row, as f32 and / or as bf16 planes (lo may be null)
+__global__ void concat_rows_kernel(float* f32, __nv_bfloat16* hi, __nv_bfloat16* lo, const float* a, const float* b, int n) {
+    asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
+    asm volatile("griddepcontrol.wait;" ::: "memory");
+    const int i = (blockIdx.x * blockDim.x + threadIdx.x) * 4;
+    if (i >= 2 * n) return;
+    const size_t row = blockIdx.y;
+    const float4 v = i < n ? *reinterpret_cast<const float4*>(a + row * n + i) : *reinterpret_cast<const float4*>(b + row * n + i - n);
+    const size_t at = row * 2 * n + i;
+    if (f32) *reinterpret_cast<float4*>(f32 + at) = v;
+    if (hi) {
+        const __nv_bfloat162 h[2] = {__floats2bfloat162_rn(v.x, v.y), __floats2bfloat162_rn(v.z, v.w)};
+        reinterpret_cast<__nv_bfloat162*>(hi + at)[0] = h[0];
+        reinterpret_cast<__nv_bfloat162*>(hi + at)[1] = h[1];
+        if (lo) {
+            reinterpret_cast<__nv_bfloat162*>(lo + at)[0] = __floats2bfloat162_rn(v.x - __low2float(h[0]), v.y - __high2float(h[0]));
+            reinterpret_cast<__nv_bfloat162*>(lo + at)[1] = __floats2bfloat162_rn(v.z - __low2float(h[1]), v.w - __high2float(h[1]));
+        }
+    }
+}
+
+// x = cap * tanh(x / cap)
+__global__ void softcap_kernel(float* x, size_t n, float cap) {
+    asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
+    asm volatile("griddepcontrol.wait;" ::: "memory");
+    const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
+    if (i < n) x[i] = cap * tanhf(x[i] / cap);
+}
+
 }  // namespace
 
 extern "C" {
@@ -759,6 +802,26 @@ cudaError_t ingot_support_rmsnorm_rows(float* out, const float* x, const float* 
 cudaError_t ingot_support_gated_act(float* out, const float* in, int n_rows, int n, int act, cudaStream_t s) {
     const size_t total = (size_t)n_rows * n;
     return support_launch(gated_act_kernel, dim3(unsigned((total + 255) / 256)), dim3(256), 0, s, out, in, n, total, act);
+}
+
+// out[r] (and copy[r], may be null) = table[rows[r]] + table2[rows2[r]] (table2 may be null); rows of n_in values.
+cudaError_t ingot_support_embed_sum_bf16(float* out, float* copy, const void* table, int n_rows_table, const int32_t* rows_dev, const void* table2,
+                                         int n_rows_table2, const int32_t* rows2_dev, int n_in, int n_rows, int* status_dev, cudaStream_t s) {
+    if (n_rows < 1 || n_in < 1 || (table2 && !rows2_dev) || !status_dev) return cudaErrorInvalidValue;
+    embed_sum_kernel<<<n_rows, 256, 0, s>>>(out, copy, static_cast<const __nv_bfloat16*>(table), n_rows_table, rows_dev,
+                                            static_cast<const __nv_bfloat16*>(table2), n_rows_table2, rows2_dev, n_in, status_dev);
+    return cudaGetLastError();
+}
+
+// [a | b] of rows of n values (a multiple of 4) as f32 rows and / or bf16 planes; null pointers are skipped.
+cudaError_t ingot_support_concat_rows(float* f32, void* hi, void* lo, const float* a, const float* b, int n, int n_rows, cudaStream_t s) {
+    if (n < 4 || n % 4 != 0 || n_rows < 1) return cudaErrorInvalidValue;
+    return support_launch(concat_rows_kernel, dim3(unsigned((2 * n / 4 + 255) / 256), n_rows), dim3(256), 0, s, f32, static_cast<__nv_bfloat16*>(hi),
+                          static_cast<__nv_bfloat16*>(lo), a, b, n);
+}
+
+cudaError_t ingot_support_softcap(float* x, size_t n, float cap, cudaStream_t s) {
+    return support_launch(softcap_kernel, dim3(unsigned((n + 255) / 256)), dim3(256), 0, s, x, n, cap);
 }
 
 }  // extern "C"

@@ -1,0 +1,526 @@
+// Latent attention: what a token leaves behind is one row shared by all heads - a normalised latent c and a rotated key part -
+// and each head's keys and values are linear images of c. No counterpart in the reference (its layers cache K and V per head).
+//
+// The mechanism, per head h:
+//     score(i, j) = (q_i . U_h c_j + rot(q_i') . rot(k_j')) * scale,      output_i = sum_j a_ij V_h c_j
+// with a_ij the softmax over the visible keys whose denominator may hold one more term exp(sink_h). Two equal ways to compute it:
+//   on the rows       q_i . U_h c_j = (U_h^T q_i) . c_j and sum_j a_ij V_h c_j = V_h (sum_j a_ij c_j): the query is taken into the
+//                     latent space once, the cached row [c | rot] is the key and its first part the value of every head, V_h
+//                     follows once per token. Reads each cached row once for all heads: decoded tokens and short portions.
+//   on the expansion  U_h c_j and V_h c_j are computed for the keys a portion sees, and heads attend over K and V of their own
+//                     (attn_latent_sm100.cu). Fewer operations per pair of tokens: long portions.
+//
+// Rows are those of the shared-row cache (attn_shared_kv.cuh) with one KV head and no key scales: [rank | rot | zeros], the latent
+// padded to `rank` columns, the whole to the row length. Visibility: causal, or a window that slides along (PageMap).
+// Rotation: value i of the rotated part with value i + rot_dims / 2, by position * base^(-2 i / rot_dims). The angle is reduced to
+// a fraction of a turn in double precision before its sine and cosine are taken in single precision.
+#include <algorithm>
+
+#include "attn_shared_kv.cuh"
+
+namespace {
+
+__device__ __forceinline__ float warp_sum(float v) {
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
+    return v;
+}
+__device__ __forceinline__ void put(float* p, float v) { *p = v; }
+__device__ __forceinline__ void put(__half* p, float v) { *p = __float2half_rn(fminf(fmaxf(v, -65504.f), 65504.f)); }
+
+constexpr int kMaxRot = 512;  // rotated values per head
+
+// One CTA per token: the token's cache row, the rotated part of its query rows, and the unrotated query as operand of the
+// product that takes it into the latent space.
+struct AppendParams {
+    ingot_step st;
+    const float* proj;
+    int proj_ld, q_off, latent_off;
+    ingot_latent_shape sh;
+    const float* norm_w;
+    float eps;
+    const double* turns;  // [rot_dims / 2] turns per position
+    SharedOut plain;      // [n_tok][n_head * dim]
+    void* q_rows;         // [n_tok][n_head][row]; the rotated part is written
+    void* rows;
+    int row;
+    const int32_t *tables, *first_page;
+    int max_blocks, n_blocks;
+    PageMap map;
+    int* status;
+};
+constexpr int kAppendThreads = 256;
+template <typename T>
+__global__ void __launch_bounds__(kAppendThreads) latent_append_kernel(const AppendParams p) {
+    INGOT_PDL_TRIGGER();
+    __shared__ float red[kAppendThreads / 32], s_cos[kMaxRot / 2], s_sin[kMaxRot / 2];
+    const int tok = blockIdx.x, seq = p.st.row_seq[tok];
+    const int pos = p.st.pos0[seq] + tok - p.st.row_start[seq];
+    const int half = p.sh.rot_dims / 2;
+    for (int i = threadIdx.x; i < half; i += kAppendThreads) {
+        double t = double(pos) * p.turns[i];
+        t -= rint(t);
+        sincospif(2.0f * float(t), &s_sin[i], &s_cos[i]);
+    }
+    INGOT_PDL_WAIT();
+    const float* q = p.proj + (size_t)tok * p.proj_ld + p.q_off;
+    const float* c = p.proj + (size_t)tok * p.proj_ld + p.latent_off;
+    float ss = 0.f;
+    for (int i = threadIdx.x; i < p.sh.rank; i += kAppendThreads) ss = fmaf(c[i], c[i], ss);
+    ss = warp_sum(ss);
+    const int warp = threadIdx.x >> 5;
+    if ((threadIdx.x & 31) == 0) red[warp] = ss;
+    __syncthreads();
+    ss = 0.f;
+#pragma unroll
+    for (int w = 0; w < kAppendThreads / 32; w++) ss += red[w];
+    const float inv = 1.0f / sqrtf(ss / float(p.sh.rank_count) + p.eps);
+    // value i of a rotated part that starts at v
+    auto rotated = [&](const float* v, int i) {
+        if (i < half) return v[i] * s_cos[i] - v[i + half] * s_sin[i];
+        if (i < 2 * half) return v[i] * s_cos[i - half] + v[i - half] * s_sin[i - half];
+        return v[i];
+    };
+    const int blk = table_block(p.tables, p.first_page, p.max_blocks, p.n_blocks, seq, p.map.page(pos), p.status);
+    if (blk >= 0) {
+        T* dst = static_cast<T*>(p.rows) + ((size_t)blk * kBlockTokens + p.map.slot(pos)) * p.row;
+        for (int i = threadIdx.x; i < p.sh.rank; i += kAppendThreads) put(dst + i, c[i] * inv * p.norm_w[i]);
+        for (int i = threadIdx.x; i < p.sh.rot; i += kAppendThreads) put(dst + p.sh.rank + i, rotated(c + p.sh.rank, i));
+    }
+    const int per = p.sh.dim + p.sh.rot;
+    if (p.plain.f32 || p.plain.hi) {
+        const int n4 = p.sh.n_head * p.sh.dim / 4, d4 = p.sh.dim / 4;
+        for (int i = threadIdx.x; i < n4; i += kAppendThreads) {
+            const int h = i / d4, d = (i - h * d4) * 4;
+            const float4 v = *reinterpret_cast<const float4*>(q + h * per + d);
+            p.plain.store2(tok, h * p.sh.dim + d, v.x, v.y);
+            p.plain.store2(tok, h * p.sh.dim + d + 2, v.z, v.w);
+        }
+    }
+    if (p.q_rows)
+        for (int i = threadIdx.x; i < p.sh.n_head * p.sh.rot; i += kAppendThreads) {
+            const int h = i / p.sh.rot, d = i - h * p.sh.rot;
+            put(static_cast<T*>(p.q_rows) + ((size_t)tok * p.sh.n_head + h) * p.row + p.sh.rank + d, rotated(q + h * per + p.sh.dim, d));
+        }
+}
+
+// Latent queries f32 [n_tok][n_head * rank] into the query rows.
+template <typename T>
+__global__ void latent_queries_kernel(T* q_rows, const float* q, int rank, int row, size_t n4) {
+    INGOT_PDL_TRIGGER();
+    INGOT_PDL_WAIT();
+    const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
+    if (i >= n4) return;
+    const int r4 = rank / 4;
+    const size_t head = i / r4;
+    const int d = int(i - head * r4) * 4;
+    const float4 v = *reinterpret_cast<const float4*>(q + i * 4);
+    T* o = q_rows + head * row + d;
+    put(o, v.x); put(o + 1, v.y); put(o + 2, v.z); put(o + 3, v.w);
+}
+
+// ---- tensor-core form on the rows: f16, m16n8k16 MMAs -------------------------------------------------------------------
+// A CTA owns 16 kMT rows - (token, head) pairs, token-major - of one sequence and one share of the keys they see, in tiles of 64
+// keys = 4 pages. The rows are long (a latent and a rotated part), so neither the queries nor the result of a tile of rows fits one
+// warp's registers; the 8 warps therefore share the work in two ways:
+//   scores   warp (row tile, key group): kMT row tiles x 8 / kMT key groups, operands from shared memory by ldmatrix
+//   values   warp = 8 kNV columns of the latent for all rows; the weights travel through shared memory as f16
+// with the row maxima exchanged in between. Key tiles are double-buffered with cp.async.
+constexpr int kTileKeys = 64, kLatThreads = 256, kLatWarps = 8, kMaxSharePages = 1024, kPStride = kTileKeys + 8;
+struct LatentSmem {
+    int q, k, p, stats, blocks, bytes;  // offsets
+    __host__ __device__ LatentSmem(int mt, int dim) {
+        const int stride = (dim + 8) * 2;
+        q = 0;
+        k = q + 16 * mt * stride;
+        p = k + 2 * kTileKeys * stride;
+        stats = p + 16 * mt * kPStride * 2;
+        blocks = stats + 8 * 16 * 4;  // [8 / mt key groups][16 mt rows]
+        bytes = blocks + kMaxSharePages * 4;
+    }
+};
+__device__ __forceinline__ void ldmatrix4(uint32_t (&r)[4], uint32_t addr) {
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
+}
+__device__ __forceinline__ void ldmatrix4_trans(uint32_t (&r)[4], uint32_t addr) {
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
+}
+__device__ __forceinline__ void cp16(uint32_t dst, const void* src, bool on) {
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(on ? 16 : 0) : "memory");
+}
+
+template <int kMT, int kNV>
+__global__ void __launch_bounds__(kLatThreads) latent_mma_kernel(const AttendParams p) {
+    constexpr int kKG = kLatWarps / kMT;  // key groups
+    extern __shared__ __align__(16) unsigned char smem[];
+    INGOT_PDL_TRIGGER();
+    INGOT_PDL_WAIT();
+    const int seq = blockIdx.z, len = p.st.len[seq], H = p.n_head, n_rows = len * H;
+    const int split = blockIdx.y, row0 = ((int)gridDim.x - 1 - (int)blockIdx.x) * 16 * kMT;  // later rows see more keys, they go first
+    if (row0 >= n_rows || len >= p.skip_len) return;
+    const LatentSmem L(kMT, p.dim);
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, j = lane & 3;
+    const int mi = warp % kMT, kg = warp / kMT;
+    const int stride = (p.dim + 8) * 2;
+    const int pos0 = p.st.pos0[seq];
+    const size_t tok0 = p.st.row_start[seq];
+    const int pos_first = pos0 + row0 / H, pos_last = pos0 + (min(row0 + 16 * kMT, n_rows) - 1) / H;
+    const int page_a = p.map.page(p.map.first_visible(pos_first)), page_b = p.map.page(pos_last);
+    const int tiles = (page_b - page_a) / 4 + 1, per = (tiles + p.n_splits - 1) / p.n_splits;
+    const int first = split * per, count = max(0, min(per, tiles - first)), page0 = page_a + first * 4;
+    const uint32_t s_base = (uint32_t)__cvta_generic_to_shared(smem);
+    __half* sp = reinterpret_cast<__half*>(smem + L.p);
+    float* s_stat = reinterpret_cast<float*>(smem + L.stats);
+    int* s_blk = reinterpret_cast<int*>(smem + L.blocks);
+
+    for (int i = threadIdx.x; i < count * 4; i += kLatThreads)
+        s_blk[i] = page0 + i <= page_b ? table_block(p.tables, p.first_page, p.max_blocks, p.n_blocks, seq, page0 + i, p.status) : -1;
+    const int pieces = p.dim / 8;
+    {
+        const __half* q = static_cast<const __half*>(p.q) + (tok0 * H + row0) * p.dim;
+        for (int i = threadIdx.x; i < 16 * kMT * pieces; i += kLatThreads) {
+            const int r = i / pieces, c = i - r * pieces;
+            const bool on = row0 + r < n_rows;
+            cp16(s_base + L.q + r * stride + c * 16, q + (on ? (size_t)r * p.dim + c * 8 : 0), on);
+        }
+    }
+    __syncthreads();
+    auto stage = [&](int t) {
+        const uint32_t dst = s_base + L.k + (t & 1) * kTileKeys * stride;
+        for (int i = threadIdx.x; i < kTileKeys * pieces; i += kLatThreads) {
+            const int key = i / pieces, c = i - key * pieces, blk = s_blk[t * 4 + (key >> 4)];
+            cp16(dst + key * stride + c * 16, static_cast<const __half*>(p.rows) + ((size_t)max(blk, 0) * kBlockTokens + (key & 15)) * p.dim + c * 8, blk >= 0);
+        }
+        asm volatile("cp.async.commit_group;" ::: "memory");
+    };
+    if (count > 0) stage(0);
+
+    // positions of this thread's rows in its score tile, and their first visible keys
+    const int r_lo = row0 + mi * 16 + g, r_hi = r_lo + 8;
+    const int pos_lo = pos0 + min(r_lo, n_rows - 1) / H, pos_hi = pos0 + min(r_hi, n_rows - 1) / H;
+    const int vis_lo = p.map.first_visible(pos_lo), vis_hi = p.map.first_visible(pos_hi);
+    const float scale = p.scale * 1.44269504f;
+    const int dv = p.out_dim;
+    float m[kMT][2], l_lo = 0.f, l_hi = 0.f, o[kMT][kNV][4];
+#pragma unroll
+    for (int mt = 0; mt < kMT; mt++) {
+        m[mt][0] = m[mt][1] = -INFINITY;
+#pragma unroll
+        for (int n = 0; n < kNV; n++) o[mt][n][0] = o[mt][n][1] = o[mt][n][2] = o[mt][n][3] = 0.f;
+    }
+
+    for (int t = 0; t < count; t++) {
+        asm volatile("cp.async.wait_group 0;" ::: "memory");
+        __syncthreads();  // the tile is in, and every warp is done with the other buffer
+        if (t + 1 < count) stage(t + 1);
+        const uint32_t tile = s_base + L.k + (t & 1) * kTileKeys * stride;
+
+        float s[kMT][4];
+#pragma unroll
+        for (int n = 0; n < kMT; n++) s[n][0] = s[n][1] = s[n][2] = s[n][3] = 0.f;
+        {
+            const uint32_t a_addr = s_base + L.q + (mi * 16 + (lane & 15)) * stride + (lane >> 4) * 16;
+            if (kMT == 1) {  // one 8-key tile: a load covers two k-steps
+                const uint32_t b_addr = tile + (kg * 8 + (lane & 7)) * stride + (lane >> 3) * 16;
+                for (int ks = 0; ks < p.dim / 16; ks += 2) {
+                    uint32_t a0[4], a1[4], b[4];
+                    ldmatrix4(a0, a_addr + ks * 32);
+                    ldmatrix4(a1, a_addr + ks * 32 + 32);
+                    ldmatrix4(b, b_addr + ks * 32);
+                    mma_16816(s[0], a0[0], a0[1], a0[2], a0[3], b[0], b[1]);
+                    mma_16816(s[0], a1[0], a1[1], a1[2], a1[3], b[2], b[3]);
+                }
+            } else {
+                const uint32_t b_addr = tile + (kg * 8 * kMT + (lane & 7) + ((lane >> 4) & 1) * 8) * stride + ((lane >> 3) & 1) * 16;
+                for (int ks = 0; ks < p.dim / 16; ks++) {
+                    uint32_t a[4];
+                    ldmatrix4(a, a_addr + ks * 32);
+#pragma unroll
+                    for (int n = 0; n + 1 < kMT; n += 2) {
+                        uint32_t b[4];
+                        ldmatrix4(b, b_addr + n * 8 * stride + ks * 32);
+                        mma_16816(s[n], a[0], a[1], a[2], a[3], b[0], b[1]);
+                        mma_16816(s[n + 1], a[0], a[1], a[2], a[3], b[2], b[3]);
+                    }
+                }
+            }
+        }
+        float mx_lo = -INFINITY, mx_hi = -INFINITY;
+        const int key0 = (page0 + t * 4) * kBlockTokens + kg * 8 * kMT + 2 * j;
+#pragma unroll
+        for (int n = 0; n < kMT; n++) {
+            const bool held = s_blk[t * 4 + ((kg * kMT + n) >> 1)] >= 0;
+#pragma unroll
+            for (int e = 0; e < 2; e++) {
+                const int key = key0 + n * 8 + e;
+                s[n][e] = held && key >= vis_lo && key <= pos_lo ? s[n][e] * scale : -INFINITY;
+                s[n][2 + e] = held && key >= vis_hi && key <= pos_hi ? s[n][2 + e] * scale : -INFINITY;
+            }
+            mx_lo = fmaxf(mx_lo, fmaxf(s[n][0], s[n][1]));
+            mx_hi = fmaxf(mx_hi, fmaxf(s[n][2], s[n][3]));
+        }
+        mx_lo = fmaxf(mx_lo, __shfl_xor_sync(0xffffffffu, mx_lo, 1));
+        mx_lo = fmaxf(mx_lo, __shfl_xor_sync(0xffffffffu, mx_lo, 2));
+        mx_hi = fmaxf(mx_hi, __shfl_xor_sync(0xffffffffu, mx_hi, 1));
+        mx_hi = fmaxf(mx_hi, __shfl_xor_sync(0xffffffffu, mx_hi, 2));
+        if (j == 0) {
+            s_stat[kg * 16 * kMT + mi * 16 + g] = mx_lo;
+            s_stat[kg * 16 * kMT + mi * 16 + g + 8] = mx_hi;
+        }
+        __syncthreads();
+        float alpha[kMT][2];
+        bool rescale = false;
+        float ref_lo = 0.f, ref_hi = 0.f, a_lo = 1.f, a_hi = 1.f;
+#pragma unroll
+        for (int mt = 0; mt < kMT; mt++)
+#pragma unroll
+            for (int e = 0; e < 2; e++) {
+                float top = m[mt][e];
+#pragma unroll
+                for (int k = 0; k < kKG; k++) top = fmaxf(top, s_stat[k * 16 * kMT + mt * 16 + g + 8 * e]);
+                const float ref = top == -INFINITY ? 0.f : top;  // a row that has not seen a key yet keeps -inf
+                alpha[mt][e] = exp2f(m[mt][e] - ref);
+                rescale = rescale || alpha[mt][e] != 1.f;
+                m[mt][e] = top;
+                if (mt == mi) {
+                    if (e == 0) { ref_lo = ref; a_lo = alpha[mt][e]; }
+                    else { ref_hi = ref; a_hi = alpha[mt][e]; }
+                }
+            }
+        float sum_lo = 0.f, sum_hi = 0.f;
+#pragma unroll
+        for (int n = 0; n < kMT; n++) {
+            const float p0 = exp2f(s[n][0] - ref_lo), p1 = exp2f(s[n][1] - ref_lo), p2 = exp2f(s[n][2] - ref_hi), p3 = exp2f(s[n][3] - ref_hi);
+            sum_lo += p0 + p1;
+            sum_hi += p2 + p3;
+            const int c = kg * 8 * kMT + n * 8 + 2 * j;
+            *reinterpret_cast<uint32_t*>(sp + (mi * 16 + g) * kPStride + c) = pack_half2_rn(p0, p1);
+            *reinterpret_cast<uint32_t*>(sp + (mi * 16 + g + 8) * kPStride + c) = pack_half2_rn(p2, p3);
+        }
+        l_lo = l_lo * a_lo + sum_lo;
+        l_hi = l_hi * a_hi + sum_hi;
+        if (__any_sync(0xffffffffu, rescale)) {
+#pragma unroll
+            for (int mt = 0; mt < kMT; mt++)
+#pragma unroll
+                for (int n = 0; n < kNV; n++) {
+                    o[mt][n][0] *= alpha[mt][0]; o[mt][n][1] *= alpha[mt][0];
+                    o[mt][n][2] *= alpha[mt][1]; o[mt][n][3] *= alpha[mt][1];
+                }
+        }
+        __syncthreads();  // the weights are in
+        if (warp * 8 * kNV < dv) {
+#pragma unroll
+            for (int kk = 0; kk < kTileKeys / 16; kk++) {
+                uint32_t a[kMT][4];
+#pragma unroll
+                for (int mt = 0; mt < kMT; mt++) ldmatrix4(a[mt], s_base + L.p + ((mt * 16 + (lane & 15)) * kPStride + kk * 16 + (lane >> 4) * 8) * 2);
+                const uint32_t v_addr = tile + (kk * 16 + (lane & 15)) * stride + (warp * 8 * kNV + (lane >> 4) * 8) * 2;
+#pragma unroll
+                for (int n = 0; n < kNV; n += 2) {
+                    if (warp * 8 * kNV + n * 8 < dv) {
+                        uint32_t b[4];
+                        ldmatrix4_trans(b, v_addr + n * 16);
+#pragma unroll
+                        for (int mt = 0; mt < kMT; mt++) {
+                            mma_16816(o[mt][n], a[mt][0], a[mt][1], a[mt][2], a[mt][3], b[0], b[1]);
+                            mma_16816(o[mt][n + 1], a[mt][0], a[mt][1], a[mt][2], a[mt][3], b[2], b[3]);
+                        }
+                    }
+                }
+            }
+        }
+    }
+    asm volatile("cp.async.wait_group 0;" ::: "memory");
+    l_lo += __shfl_xor_sync(0xffffffffu, l_lo, 1);
+    l_lo += __shfl_xor_sync(0xffffffffu, l_lo, 2);
+    l_hi += __shfl_xor_sync(0xffffffffu, l_hi, 1);
+    l_hi += __shfl_xor_sync(0xffffffffu, l_hi, 2);
+    __syncthreads();
+    if (j == 0) {
+        s_stat[kg * 16 * kMT + mi * 16 + g] = l_lo;
+        s_stat[kg * 16 * kMT + mi * 16 + g + 8] = l_hi;
+    }
+    __syncthreads();
+#pragma unroll
+    for (int mt = 0; mt < kMT; mt++)
+#pragma unroll
+        for (int e = 0; e < 2; e++) {
+            const int r = row0 + mt * 16 + g + 8 * e;
+            if (r >= n_rows) continue;
+            float l = 0.f;
+#pragma unroll
+            for (int k = 0; k < kKG; k++) l += s_stat[k * 16 * kMT + mt * 16 + g + 8 * e];
+            const int h = r % H;
+            if (p.n_splits == 1) {
+                float f = 1.0f;
+                if (p.sink) {
+                    const float sink = p.sink[h] * 1.44269504f, top = fmaxf(m[mt][e], sink);
+                    f = exp2f(m[mt][e] - top);
+                    l = l * f + exp2f(sink - top);
+                }
+                f /= l;
+#pragma unroll
+                for (int n = 0; n < kNV; n++) {
+                    const int d = warp * 8 * kNV + n * 8 + 2 * j;
+                    if (d < dv) p.out.store2(tok0 + r / H, h * dv + d, o[mt][n][2 * e] * f, o[mt][n][2 * e + 1] * f);
+                }
+            } else {
+                float* part = p.part + ((tok0 * H + r) * p.n_splits + split) * (dv + 2);
+#pragma unroll
+                for (int n = 0; n < kNV; n++) {
+                    const int d = warp * 8 * kNV + n * 8 + 2 * j;
+                    if (d < dv) *reinterpret_cast<float2*>(part + d) = make_float2(o[mt][n][2 * e], o[mt][n][2 * e + 1]);
+                }
+                if (warp == 0 && j == 0) { part[dv] = m[mt][e]; part[dv + 1] = l; }
+            }
+        }
+}
+
+// out = sum_s o_s 2^(m_s - M) / (sum_s l_s 2^(m_s - M) + 2^(sink - M)) over the splits of one (token, head)
+constexpr int kMergeThreads = 128, kMaxSplits = 64;
+__global__ void __launch_bounds__(kMergeThreads) latent_merge_kernel(const AttendParams p) {
+    INGOT_PDL_TRIGGER();
+    INGOT_PDL_WAIT();
+    __shared__ float s_f[kMaxSplits];
+    const int h = blockIdx.x, seq = p.st.row_seq[blockIdx.y];
+    if (p.st.len[seq] >= p.skip_len) return;
+    const size_t tok = blockIdx.y;
+    const int ld = p.out_dim + 2;
+    const float* part = p.part + (tok * p.n_head + h) * p.n_splits * ld;
+    float top = p.sink ? p.sink[h] * 1.44269504f : -INFINITY;
+    const float sink = top;
+    for (int s = 0; s < p.n_splits; s++) top = fmaxf(top, part[s * ld + p.out_dim]);
+    float l = p.sink ? exp2f(sink - top) : 0.f;
+    for (int s = 0; s < p.n_splits; s++) {
+        const float f = exp2f(part[s * ld + p.out_dim] - top);
+        l = fmaf(f, part[s * ld + p.out_dim + 1], l);
+        if (threadIdx.x == 0) s_f[s] = f;
+    }
+    __syncthreads();
+    const float inv = 1.0f / l;
+    for (int d = threadIdx.x * 2; d < p.out_dim; d += kMergeThreads * 2) {
+        float a = 0.f, b = 0.f;
+        for (int s = 0; s < p.n_splits; s++) {
+            const float2 v = *reinterpret_cast<const float2*>(part + s * ld + d);
+            a = fmaf(s_f[s], v.x, a);
+            b = fmaf(s_f[s], v.y, b);
+        }
+        p.out.store2(tok, h * p.out_dim + d, a * inv, b * inv);
+    }
+}
+
+template <int kMT>
+void (*pick_mma(int dv))(const AttendParams) {
+    return dv <= 128 ? latent_mma_kernel<kMT, 2> : dv <= 256 ? latent_mma_kernel<kMT, 4> : latent_mma_kernel<kMT, 8>;
+}
+
+constexpr int kSmemLimit = 227 * 1024;
+
+bool mma_takes(int dim, int dv) { return dim % 32 == 0 && dv % 16 == 0 && dv <= 512 && LatentSmem(1, dim).bytes <= kSmemLimit; }
+
+int launch_mma(ingot_skv* kv, AttendParams p, cudaStream_t s) {
+    const int rows = std::min(p.st.max_len, p.skip_len) * p.n_head;
+    int mt = rows <= 16 ? 1 : rows <= 32 ? 2 : 4;
+    while (mt > 1 && LatentSmem(mt, p.dim).bytes > kSmemLimit) mt /= 2;
+    const int smem = LatentSmem(mt, p.dim).bytes;
+    auto kernel = mt == 4 ? pick_mma<4>(p.out_dim) : mt == 2 ? pick_mma<2>(p.out_dim) : pick_mma<1>(p.out_dim);
+    INGOT_CUDA_TRY(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
+    // Shares of the keys: CTAs run in rounds of as many as fit the GPU; a share costs about 64 keys' time besides its keys. A share is
+    // whole tiles, and no more pages than the kernel's table holds.
+    const int row_tiles = (rows + 16 * mt - 1) / (16 * mt), max_pages = p.max_blocks + 3;
+    const int keys = p.map.window > 0 ? std::min(p.max_blocks * kBlockTokens, p.map.window + p.st.max_len) : p.max_blocks * kBlockTokens;
+    const long long ctas = (long long)row_tiles * p.st.n_seq;
+    const int slots = kv->num_sms * std::max(1, std::min(4, kSmemLimit / (smem + 1024)));
+    long long best = -1;
+    for (int n = 1; n <= kMaxSplits; n++) {
+        const int share = ((keys + n - 1) / n + kTileKeys - 1) / kTileKeys * kTileKeys;
+        if (n > 1 && share < 2 * kTileKeys) break;
+        const long long cost = (ctas * n + slots - 1) / slots * (share + 64 + (n > 1 ? 2 * n : 0));
+        if (best < 0 || cost < best) { best = cost; p.n_splits = n; }
+    }
+    p.n_splits = std::max(p.n_splits, (max_pages + kMaxSharePages - 8) / (kMaxSharePages - 7));
+    if (p.n_splits > kMaxSplits) return launch_shared_kv_plain(p, INGOT_F16, s);
+    if (p.n_splits > 1) {
+        const size_t need = (size_t)p.st.n_tok * p.n_head * p.n_splits * (p.out_dim + 2);
+        if (need > kv->part_floats) {
+            float* fresh = nullptr;
+            INGOT_CUDA_TRY(cudaMalloc(&fresh, need * sizeof(float)));
+            if (kv->part) kv->retired.push_back(kv->part);  // a captured graph may still point into it
+            kv->part = fresh;
+            kv->part_floats = need;
+        }
+        p.part = kv->part;
+    }
+    INGOT_CUDA_TRY(ingot_launch_pdl(kernel, dim3(row_tiles, p.n_splits, p.st.n_seq), dim3(kLatThreads), size_t(smem), s, p));
+    if (p.n_splits > 1) INGOT_CUDA_TRY(ingot_launch_pdl(latent_merge_kernel, dim3(p.n_head, p.st.n_tok), dim3(kMergeThreads), 0, s, p));
+    return INGOT_OK;
+}
+
+bool step_ok(const ingot_step* st) {
+    return st && st->n_tok >= 1 && st->n_seq >= 1 && st->n_seq <= 65535 && st->max_len >= 1 && st->row_seq && st->row_start && st->len && st->pos0;
+}
+
+}  // namespace
+
+extern "C" {
+
+int ingot_latent_append(ingot_skv* kv, int layer, const ingot_step* step, const float* proj_dev, int proj_ld, int q_off, int latent_off,
+                        const ingot_latent_shape* shape, const float* norm_dev, float eps, const double* turns_dev, const ingot_act_out* q_plain,
+                        void* q_rows_dev, const int32_t* tables_dev, const int32_t* first_page_dev, int max_blocks, void* stream) {
+    INGOT_REQUIRE(kv && step_ok(step) && shape, "ingot_latent_append: null handle or bad step");
+    INGOT_REQUIRE_DEVICE(kv);
+    INGOT_REQUIRE(layer >= 0 && layer < kv->n_layer, "ingot_latent_append: layer out of range");
+    INGOT_REQUIRE(proj_dev && norm_dev && q_plain && tables_dev && max_blocks >= 1 && (turns_dev || shape->rot_dims == 0), "ingot_latent_append: null argument");
+    const ingot_latent_shape& sh = *shape;
+    INGOT_REQUIRE(sh.n_head >= 1 && sh.dim >= 0 && sh.dim % 4 == 0 && sh.rank >= 1 && sh.rank_count >= 1 && sh.rank_count <= sh.rank && sh.rot >= 0 &&
+                      sh.rot_dims >= 0 && sh.rot_dims % 2 == 0 && sh.rot_dims <= sh.rot && sh.rank + sh.rot <= kv->dim,
+                  "ingot_latent_append: bad shape");
+    INGOT_REQUIRE(proj_ld % 4 == 0 && q_off % 4 == 0 && (sh.dim + sh.rot) % 4 == 0 && q_plain->ld % 2 == 0, "ingot_latent_append: rows and offsets must be multiples of 4 floats");
+    if (sh.rot_dims > kMaxRot || kv->n_head_kv != 1 || kv->inv_rms) {
+        ingot_set_error("ingot_latent_append: needs a window-form cache with one row per token and at most " + std::to_string(kMaxRot) + " rotated values");
+        return INGOT_ERR_UNSUPPORTED;
+    }
+    const size_t esz = kv->dtype == INGOT_F32 ? 4 : 2;
+    AppendParams p = {*step, proj_dev, proj_ld, q_off, latent_off, sh, norm_dev, eps, turns_dev,
+                      SharedOut{q_plain->f32, static_cast<__nv_bfloat16*>(q_plain->hi), static_cast<__nv_bfloat16*>(q_plain->lo), q_plain->ld, 1.0f}, q_rows_dev,
+                      static_cast<char*>(kv->rows) + kv->layer_elems * layer * esz, kv->dim, tables_dev, first_page_dev, max_blocks, kv->n_blocks, page_map(kv),
+                      kv->status_dev};
+    auto kernel = kv->dtype == INGOT_F32 ? latent_append_kernel<float> : latent_append_kernel<__half>;
+    INGOT_CUDA_TRY(ingot_launch_pdl(kernel, dim3(step->n_tok), dim3(kAppendThreads), 0, static_cast<cudaStream_t>(stream), p));
+    return INGOT_OK;
+}
+
+int ingot_latent_queries(const ingot_skv* kv, const float* q_dev, int n_tok, int n_head, int rank, void* q_rows_dev, void* stream) {
+    INGOT_REQUIRE(kv && q_dev && q_rows_dev && n_tok >= 1 && n_head >= 1, "ingot_latent_queries: null argument");
+    INGOT_REQUIRE(rank >= 4 && rank % 4 == 0 && rank <= kv->dim, "ingot_latent_queries: bad latent length");
+    const size_t n4 = (size_t)n_tok * n_head * rank / 4;
+    const dim3 grid((unsigned)((n4 + 255) / 256));
+    cudaStream_t s = static_cast<cudaStream_t>(stream);
+    if (kv->dtype == INGOT_F32) INGOT_CUDA_TRY(ingot_launch_pdl(latent_queries_kernel<float>, grid, dim3(256), 0, s, static_cast<float*>(q_rows_dev), q_dev, rank, kv->dim, n4));
+    else INGOT_CUDA_TRY(ingot_launch_pdl(latent_queries_kernel<__half>, grid, dim3(256), 0, s, static_cast<__half*>(q_rows_dev), q_dev, rank, kv->dim, n4));
+    return INGOT_OK;
+}
+
+int ingot_latent_attend(ingot_skv* kv, int layer, const ingot_step* step, const void* q_rows_dev, int n_head, int rank, float scale, const float* sink_dev,
+                        const ingot_act_out* out, const int32_t* tables_dev, const int32_t* first_page_dev, int max_blocks, int skip_len, int impl, void* stream) {
+    INGOT_REQUIRE(kv && step_ok(step), "ingot_latent_attend: null handle or bad step");
+    INGOT_REQUIRE_DEVICE(kv);
+    INGOT_REQUIRE(layer >= 0 && layer < kv->n_layer, "ingot_latent_attend: layer out of range");
+    INGOT_REQUIRE(q_rows_dev && out && tables_dev && max_blocks >= 1 && n_head >= 1, "ingot_latent_attend: null argument");
+    INGOT_REQUIRE(rank >= 1 && rank <= kv->dim && kv->n_head_kv == 1 && !kv->inv_rms, "ingot_latent_attend: bad rows");
+    const size_t esz = kv->dtype == INGOT_F32 ? 4 : 2;
+    AttendParams p = {*step, q_rows_dev, static_cast<const char*>(kv->rows) + kv->layer_elems * layer * esz, nullptr, tables_dev, first_page_dev, max_blocks,
+                      kv->n_blocks, n_head, 1, kv->dim, rank, page_map(kv), scale,
+                      SharedOut{out->f32, static_cast<__nv_bfloat16*>(out->hi), static_cast<__nv_bfloat16*>(out->lo), out->ld, 1.0f}, kv->status_dev, 1, nullptr,
+                      sink_dev, skip_len > 0 ? skip_len : 0x7fffffff};
+    cudaStream_t s = static_cast<cudaStream_t>(stream);
+    if (kv->dtype == INGOT_F16 && impl != 1 && mma_takes(kv->dim, rank) && out->ld % 2 == 0) return launch_mma(kv, p, s);
+    if (impl == 2) {
+        ingot_set_error("ingot_latent_attend: the tensor-core kernel does not take this row length");
+        return INGOT_ERR_UNSUPPORTED;
+    }
+    return launch_shared_kv_plain(p, kv->dtype, s);
+}
+
+}  // extern "C"

@@ -108,7 +108,7 @@ __global__ void __launch_bounds__(kAppendThreads) shared_kv_append_kernel(const 
     if (threadIdx.x == 0) p.inv_rms[(size_t)blk * kBlockTokens + slot] = ik;
 }
 
-// ---- plain form: f32 arithmetic on the FMA pipes, any row length up to 512, f32 or f16 rows -------------------------
+// ---- plain form: f32 arithmetic on the FMA pipes, any row length up to 1024, f32 or f16 rows -------------------------
 // A CTA owns 16 (token, head) rows of one KV head - 4 per warp - and walks the visible keys 32 at a time through shared
 // memory: lane = key for the scores, lane = dims for the weighted sum.
 constexpr int kRows = 16, kKeys = 32;
@@ -120,7 +120,7 @@ __global__ void __launch_bounds__(128) shared_kv_attend_kernel(const AttendParam
     const int seq = blockIdx.z, kvh = blockIdx.y;
     const int group = p.n_head / p.n_head_kv, len = p.st.len[seq];
     const int row0 = blockIdx.x * kRows, n_rows = len * group;
-    if (row0 >= n_rows) return;
+    if (row0 >= n_rows || len >= p.skip_len) return;
     const int dim = p.dim, ldk = kD * 32 + 1;
     float* sq = smem;                       // [16][kD * 32]
     float* sk = sq + kRows * kD * 32;       // [32][kD * 32 + 1]
@@ -163,7 +163,7 @@ __global__ void __launch_bounds__(128) shared_kv_attend_kernel(const AttendParam
             }
             const T* src = static_cast<const T*>(p.rows) + (((size_t)max(blk, 0) * p.n_head_kv + kvh) * kBlockTokens + slot) * dim;
             for (int d = part; d < kD * 32; d += 4) sk[key * ldk + d] = blk >= 0 && d < dim ? widen(src[d]) : 0.f;
-            if (part == 0) sr[key] = blk >= 0 ? p.inv_rms[(size_t)blk * kBlockTokens + slot] * p.scale : 0.f;
+            if (part == 0) sr[key] = blk < 0 ? 0.f : p.inv_rms ? p.inv_rms[(size_t)blk * kBlockTokens + slot] * p.scale : p.scale;
         }
         __syncthreads();
         const int j = j0 + lane;
@@ -198,7 +198,11 @@ __global__ void __launch_bounds__(128) shared_kv_attend_kernel(const AttendParam
     for (int r = 0; r < 4; r++) {
         const int rr = row0 + warp * 4 + r;
         if (rr >= n_rows) continue;
-        const float inv = 1.0f / l[r];
+        float inv = 1.0f / l[r];
+        if (p.sink) {
+            const float sink = p.sink[kvh * group + rr % group], top = fmaxf(m[r], sink), mine = expf(m[r] - top);
+            inv = mine / (l[r] * mine + expf(sink - top));
+        }
 #pragma unroll
         for (int i = 0; i < kD; i++) {
             const int d = lane + 32 * i;
@@ -212,10 +216,11 @@ int launch_plain(const AttendParams& p, cudaStream_t s) {
     const int group = p.n_head / p.n_head_kv;
     const dim3 grid((unsigned)(((size_t)p.st.max_len * group + kRows - 1) / kRows), p.n_head_kv, p.st.n_seq);
     const int units = (p.dim + 31) / 32;
-    const int kd = units <= 1 ? 1 : units <= 2 ? 2 : units <= 4 ? 4 : units <= 8 ? 8 : 16;
+    const int kd = units <= 1 ? 1 : units <= 2 ? 2 : units <= 4 ? 4 : units <= 8 ? 8 : units <= 16 ? 16 : units <= 20 ? 20 : 32;
     const size_t smem = ((size_t)kRows * kd * 32 + (size_t)kKeys * (kd * 32 + 1) + kKeys) * sizeof(float);
     auto kernel = kd == 1 ? shared_kv_attend_kernel<T, 1> : kd == 2 ? shared_kv_attend_kernel<T, 2> : kd == 4 ? shared_kv_attend_kernel<T, 4>
-                : kd == 8 ? shared_kv_attend_kernel<T, 8> : shared_kv_attend_kernel<T, 16>;
+                : kd == 8 ? shared_kv_attend_kernel<T, 8> : kd == 16 ? shared_kv_attend_kernel<T, 16> : kd == 20 ? shared_kv_attend_kernel<T, 20>
+                : shared_kv_attend_kernel<T, 32>;
     if (smem > 48 * 1024) INGOT_CUDA_TRY(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, int(smem)));
     INGOT_CUDA_TRY(ingot_launch_pdl(kernel, grid, dim3(128), smem, s, p));
     return INGOT_OK;
@@ -674,41 +679,55 @@ int launch_mma(ingot_skv* kv, AttendParams p, cudaStream_t s) {
     return INGOT_OK;
 }
 
+int create(ingot_skv** out, int n_layer, int n_head_kv, int head_dim, int dtype, int chunk, int window, int n_blocks, bool scales, const char* who) {
+    *out = nullptr;
+    INGOT_REQUIRE(n_layer >= 1 && n_head_kv >= 1 && n_blocks >= 1 && chunk >= 0 && window >= 0, std::string(who) + ": bad sizes");
+    INGOT_REQUIRE(dtype == INGOT_F32 || dtype == INGOT_F16, std::string(who) + ": rows are f32 or f16");
+    const int longest = scales ? 512 : 1024;
+    if (head_dim < 4 || head_dim > longest || head_dim % 4 != 0) {
+        ingot_set_error(std::string(who) + ": row length must be a multiple of 4 and at most " + std::to_string(longest));
+        return INGOT_ERR_UNSUPPORTED;
+    }
+    ingot_skv* kv = new (std::nothrow) ingot_skv();
+    if (!kv) return INGOT_ERR_NOMEM;
+    kv->n_layer = n_layer; kv->n_head_kv = n_head_kv; kv->dim = head_dim; kv->dtype = dtype; kv->chunk = chunk; kv->window = window; kv->n_blocks = n_blocks;
+    kv->layer_elems = (size_t)n_blocks * n_head_kv * kBlockTokens * head_dim;
+    const size_t bytes = kv->layer_elems * n_layer * (dtype == INGOT_F32 ? 4 : 2), scale_bytes = (size_t)n_layer * n_blocks * kBlockTokens * 4;
+    cudaError_t e;
+    // zero-filled: rows that were never written stay finite, so a masked key cannot inject NaN through 0 * garbage
+    if ((e = cudaGetDevice(&kv->device)) != cudaSuccess || (e = cudaDeviceGetAttribute(&kv->num_sms, cudaDevAttrMultiProcessorCount, kv->device)) != cudaSuccess ||
+        (e = cudaMalloc(&kv->rows, bytes)) != cudaSuccess || (e = cudaMalloc(&kv->status_dev, sizeof(int))) != cudaSuccess ||
+        (e = cudaMemset(kv->rows, 0, bytes)) != cudaSuccess || (e = cudaMemset(kv->status_dev, 0, sizeof(int))) != cudaSuccess ||
+        (scales && ((e = cudaMalloc(&kv->inv_rms, scale_bytes)) != cudaSuccess || (e = cudaMemset(kv->inv_rms, 0, scale_bytes)) != cudaSuccess)) ||
+        (e = cudaDeviceSynchronize()) != cudaSuccess) {
+        const int rc = ingot_cuda_fail(e, who);
+        ingot_skv_destroy(kv);
+        return rc;
+    }
+    *out = kv;
+    return INGOT_OK;
+}
+
 bool step_ok(const ingot_step* st) {
     return st && st->n_tok >= 1 && st->n_seq >= 1 && st->n_seq <= 65535 && st->max_len >= 1 && st->row_seq && st->row_start && st->len && st->pos0;
 }
 
 }  // namespace
 
+int launch_shared_kv_plain(const AttendParams& p, int dtype, cudaStream_t stream) {
+    return dtype == INGOT_F32 ? launch_plain<float>(p, stream) : launch_plain<__half>(p, stream);
+}
+
 extern "C" {
 
 int ingot_skv_create(ingot_skv** out, int n_layer, int n_head_kv, int head_dim, int dtype, int chunk, int n_blocks) {
     INGOT_REQUIRE(out != nullptr, "ingot_skv_create: out is null");
-    *out = nullptr;
-    INGOT_REQUIRE(n_layer >= 1 && n_head_kv >= 1 && n_blocks >= 1 && chunk >= 0, "ingot_skv_create: bad sizes");
-    INGOT_REQUIRE(dtype == INGOT_F32 || dtype == INGOT_F16, "ingot_skv_create: rows are f32 or f16");
-    if (head_dim < 4 || head_dim > 512 || head_dim % 4 != 0) {
-        ingot_set_error("ingot_skv_create: row length must be a multiple of 4 and at most 512");
-        return INGOT_ERR_UNSUPPORTED;
-    }
-    ingot_skv* kv = new (std::nothrow) ingot_skv();
-    if (!kv) return INGOT_ERR_NOMEM;
-    kv->n_layer = n_layer; kv->n_head_kv = n_head_kv; kv->dim = head_dim; kv->dtype = dtype; kv->chunk = chunk; kv->n_blocks = n_blocks;
-    kv->layer_elems = (size_t)n_blocks * n_head_kv * kBlockTokens * head_dim;
-    const size_t bytes = kv->layer_elems * n_layer * (dtype == INGOT_F32 ? 4 : 2), scale_bytes = (size_t)n_layer * n_blocks * kBlockTokens * 4;
-    cudaError_t e;
-    // zero-filled: rows that were never written stay finite, so a masked key cannot inject NaN through 0 * garbage
-    if ((e = cudaGetDevice(&kv->device)) != cudaSuccess || (e = cudaDeviceGetAttribute(&kv->num_sms, cudaDevAttrMultiProcessorCount, kv->device)) != cudaSuccess ||
-        (e = cudaMalloc(&kv->rows, bytes)) != cudaSuccess || (e = cudaMalloc(&kv->inv_rms, scale_bytes)) != cudaSuccess ||
-        (e = cudaMalloc(&kv->status_dev, sizeof(int))) != cudaSuccess || (e = cudaMemset(kv->rows, 0, bytes)) != cudaSuccess ||
-        (e = cudaMemset(kv->inv_rms, 0, scale_bytes)) != cudaSuccess || (e = cudaMemset(kv->status_dev, 0, sizeof(int))) != cudaSuccess ||
-        (e = cudaDeviceSynchronize()) != cudaSuccess) {
-        const int rc = ingot_cuda_fail(e, "ingot_skv_create");
-        ingot_skv_destroy(kv);
-        return rc;
-    }
-    *out = kv;
-    return INGOT_OK;
+    return create(out, n_layer, n_head_kv, head_dim, dtype, chunk, 0, n_blocks, true, "ingot_skv_create");
+}
+
+int ingot_skv_create_window(ingot_skv** out, int n_layer, int n_head_kv, int row_length, int dtype, int window, int n_blocks) {
+    INGOT_REQUIRE(out != nullptr, "ingot_skv_create_window: out is null");
+    return create(out, n_layer, n_head_kv, row_length, dtype, 0, window, n_blocks, false, "ingot_skv_create_window");
 }
 
 void ingot_skv_destroy(ingot_skv* kv) {
@@ -723,7 +742,7 @@ void ingot_skv_destroy(ingot_skv* kv) {
 
 int ingot_skv_pages(int chunk, int n_positions) {
     if (n_positions < 1 || chunk < 0) return 0;
-    const PageMap map = {chunk, (chunk + kBlockTokens - 1) / kBlockTokens};
+    const PageMap map = {chunk, (chunk + kBlockTokens - 1) / kBlockTokens, 0};
     return map.page(n_positions - 1) + 1;
 }
 
@@ -749,6 +768,7 @@ int ingot_skv_append(ingot_skv* kv, int layer, const ingot_step* step, const flo
                      int n_head, int head_size, const float* q_norm_dev, const float* k_norm_dev, float eps, void* q_out_dev,
                      const int32_t* tables_dev, const int32_t* first_page_dev, int max_blocks, void* stream) {
     INGOT_REQUIRE(kv && step_ok(step), "ingot_skv_append: null handle or bad step");
+    INGOT_REQUIRE(kv->inv_rms, "ingot_skv_append: the cache was created for rows without scales");
     INGOT_REQUIRE_DEVICE(kv);
     INGOT_REQUIRE(layer >= 0 && layer < kv->n_layer, "ingot_skv_append: layer out of range");
     INGOT_REQUIRE(proj_dev && q_norm_dev && k_norm_dev && q_out_dev && tables_dev && max_blocks >= 1, "ingot_skv_append: null argument");
@@ -759,7 +779,7 @@ int ingot_skv_append(ingot_skv* kv, int layer, const ingot_step* step, const flo
     AppendParams p = {*step, proj_dev, proj_ld, q_off, k_off, n_head, kv->n_head_kv, kv->dim, n_head * head_size, kv->n_head_kv * head_size,
                       q_norm_dev, k_norm_dev, eps, q_out_dev, static_cast<char*>(kv->rows) + kv->layer_elems * layer * esz,
                       kv->inv_rms + (size_t)layer * kv->n_blocks * kBlockTokens, tables_dev, first_page_dev, max_blocks, kv->n_blocks,
-                      PageMap{kv->chunk, (kv->chunk + kBlockTokens - 1) / kBlockTokens}, kv->status_dev};
+                      page_map(kv), kv->status_dev};
     auto kernel = kv->dtype == INGOT_F32 ? shared_kv_append_kernel<float> : shared_kv_append_kernel<__half>;
     INGOT_CUDA_TRY(ingot_launch_pdl(kernel, dim3(step->n_tok), dim3(kAppendThreads), 0, static_cast<cudaStream_t>(stream), p));
     return INGOT_OK;
@@ -768,6 +788,7 @@ int ingot_skv_append(ingot_skv* kv, int layer, const ingot_step* step, const flo
 int ingot_skv_attend(ingot_skv* kv, int layer, const ingot_step* step, const void* q_dev, int n_head, int out_dim, float scale,
                      float out_scale, const ingot_act_out* out, const int32_t* tables_dev, const int32_t* first_page_dev, int max_blocks, int impl, void* stream) {
     INGOT_REQUIRE(kv && step_ok(step), "ingot_skv_attend: null handle or bad step");
+    INGOT_REQUIRE(kv->inv_rms, "ingot_skv_attend: the cache was created for rows without scales");
     INGOT_REQUIRE_DEVICE(kv);
     INGOT_REQUIRE(layer >= 0 && layer < kv->n_layer, "ingot_skv_attend: layer out of range");
     INGOT_REQUIRE(q_dev && out && tables_dev && max_blocks >= 1, "ingot_skv_attend: null argument");
@@ -776,7 +797,7 @@ int ingot_skv_attend(ingot_skv* kv, int layer, const ingot_step* step, const voi
     const size_t esz = kv->dtype == INGOT_F32 ? 4 : 2;
     AttendParams p = {*step, q_dev, static_cast<const char*>(kv->rows) + kv->layer_elems * layer * esz,
                       kv->inv_rms + (size_t)layer * kv->n_blocks * kBlockTokens, tables_dev, first_page_dev, max_blocks, kv->n_blocks, n_head, kv->n_head_kv,
-                      kv->dim, out_dim, PageMap{kv->chunk, (kv->chunk + kBlockTokens - 1) / kBlockTokens}, scale,
+                      kv->dim, out_dim, page_map(kv), scale,
                       SharedOut{out->f32, static_cast<__nv_bfloat16*>(out->hi), static_cast<__nv_bfloat16*>(out->lo), out->ld, out_scale}, kv->status_dev, 1, nullptr};
     cudaStream_t s = static_cast<cudaStream_t>(stream);
     if (kv->dtype == INGOT_F32) return launch_plain<float>(p, s);

@@ -10,10 +10,10 @@
 struct ingot_skv {
     int device = 0, num_sms = 0;
     int n_layer = 0, n_head_kv = 0, dim = 0;  // dim: row length (padded head size)
-    int dtype = INGOT_F32, chunk = 0, n_blocks = 0;
+    int dtype = INGOT_F32, chunk = 0, window = 0, n_blocks = 0;
     size_t layer_elems = 0;
     void* rows = nullptr;
-    float* inv_rms = nullptr;  // [layer][block][16]
+    float* inv_rms = nullptr;  // [layer][block][16]; null in caches whose rows are the keys as they are (window form)
     int* status_dev = nullptr;
     float* part = nullptr;  // split-key partials of decoded tokens, grown on demand
     size_t part_floats = 0;
@@ -21,12 +21,18 @@ struct ingot_skv {
     std::vector<CUtensorMap> tmaps;  // per layer, 128-value f16 rows only: [page * kv head][16][128] in boxes of 16 x 64
 };
 
+// Which keys a position sees and which page holds it: the whole past, its own chunk, or a window that slides along.
 struct PageMap {
     int chunk, pages_per_chunk;  // chunk 0: one chunk of unlimited length
+    int window = 0;              // > 0 (chunk is 0 then): position i sees i - window + 1 .. i
     __host__ __device__ __forceinline__ int page(int pos) const { return chunk > 0 ? (pos / chunk) * pages_per_chunk + (pos % chunk) / kBlockTokens : pos / kBlockTokens; }
     __host__ __device__ __forceinline__ int slot(int pos) const { return (chunk > 0 ? pos % chunk : pos) % kBlockTokens; }
-    __host__ __device__ __forceinline__ int first_visible(int pos) const { return chunk > 0 ? pos / chunk * chunk : 0; }
+    __host__ __device__ __forceinline__ int first_visible(int pos) const {
+        if (chunk > 0) return pos / chunk * chunk;
+        return window > 0 && pos >= window ? pos - window + 1 : 0;
+    }
 };
+inline PageMap page_map(const ingot_skv* kv) { return PageMap{kv->chunk, (kv->chunk + kBlockTokens - 1) / kBlockTokens, kv->window}; }
 
 struct SharedOut {
     float* f32;
@@ -40,6 +46,18 @@ struct SharedOut {
             const __nv_bfloat16 h = __float2bfloat16_rn(v * scale);
             hi[i] = h;
             if (lo) lo[i] = __float2bfloat16_rn(v * scale - __bfloat162float(h));
+        }
+    }
+    // Two neighbouring columns, c and ld even.
+    __device__ __forceinline__ void store2(size_t row, int c, float a, float b) const {
+        const size_t i = row * ld + c;
+        a *= scale;
+        b *= scale;
+        if (f32) *reinterpret_cast<float2*>(f32 + i) = make_float2(a, b);
+        if (hi) {
+            const __nv_bfloat162 h = __floats2bfloat162_rn(a, b);
+            *reinterpret_cast<__nv_bfloat162*>(hi + i) = h;
+            if (lo) *reinterpret_cast<__nv_bfloat162*>(lo + i) = __floats2bfloat162_rn(a - __low2float(h), b - __high2float(h));
         }
     }
 };
@@ -57,7 +75,7 @@ struct AttendParams {
     ingot_step st;
     const void* q;
     const void* rows;
-    const float* inv_rms;
+    const float* inv_rms;  // null: keys have no scale of their own
     const int32_t *tables, *first_page;
     int max_blocks, n_blocks, n_head, n_head_kv, dim, out_dim;
     PageMap map;
@@ -66,7 +84,12 @@ struct AttendParams {
     int* status;
     int n_splits;   // decoding: CTAs per (token, KV head) over the keys
     float* part;    // [token][head][split][dim + 2]
+    const float* sink = nullptr;  // per head: one more term exp(sink) of the denominator (null: none)
+    int skip_len = 0x7fffffff;    // sequences of the step with this many tokens or more are left to another launch
 };
+
+// The plain kernel (f32 arithmetic, any row length up to 1024, window, chunk and sink); dtype of rows and queries.
+int launch_shared_kv_plain(const AttendParams& p, int dtype, cudaStream_t stream);
 
 // tcgen05 form for portions of prompts over rows of 128 values (attn_shared_kv_sm100.cu); INGOT_ERR_UNSUPPORTED if the driver
 // cannot encode its tensor map.

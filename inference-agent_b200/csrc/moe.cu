@@ -1,0 +1,237 @@
+// Mixture of experts: routing, and the plain form of the experts' products (the tensor-core form is the grouped product of
+// backend/linear_sm100.cu). No counterpart in the reference, whose feed-forwards are dense.
+//
+// A token's pairs are its `top` experts; pair p = token * top + k. The experts work on ROWS: the pairs sorted by expert, in token
+// order within one, so that an expert's rows are a run [group_start[e], group_start[e + 1]) and the order is the same in every run.
+#include "ingot_internal.cuh"
+
+namespace {
+
+__device__ __forceinline__ float warp_sum(float v) {
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
+    return v;
+}
+
+// One warp per token: its `top` largest logits, larger first, the lower expert of equal ones; the weight is the logit's sigmoid.
+// The k-th choice is the largest (logit, -expert) below the one before, so nothing has to be marked as taken.
+__global__ void __launch_bounds__(128) moe_select_kernel(const float* logits, int ld, int n_tok, int n_expert, int top, int32_t* expert_of, float* weight_of) {
+    INGOT_PDL_TRIGGER();
+    INGOT_PDL_WAIT();
+    const int t = blockIdx.x * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+    if (t >= n_tok) return;
+    const float* z = logits + (size_t)t * ld;
+    float last = INFINITY;
+    int last_e = -1;
+    for (int k = 0; k < top; k++) {
+        float best = -INFINITY;
+        int best_e = n_expert;
+        for (int e = lane; e < n_expert; e += 32) {
+            float v = z[e];
+            if (!(v == v)) v = -INFINITY;
+            if ((v < last || (v == last && e > last_e)) && (v > best || best_e == n_expert)) { best = v; best_e = e; }
+        }
+#pragma unroll
+        for (int o = 16; o > 0; o >>= 1) {
+            const float v = __shfl_xor_sync(0xffffffffu, best, o);
+            const int e = __shfl_xor_sync(0xffffffffu, best_e, o);
+            if (e < n_expert && (best_e == n_expert || v > best || (v == best && e < best_e))) { best = v; best_e = e; }
+        }
+        if (lane == 0) {
+            expert_of[(size_t)t * top + k] = best_e;
+            weight_of[(size_t)t * top + k] = 1.0f / (1.0f + expf(-best));
+        }
+        last = best;
+        last_e = best_e;
+    }
+}
+
+// One CTA per expert: where its rows start (pairs of lower experts), then its pairs in order.
+constexpr int kSortThreads = 512;
+__global__ void __launch_bounds__(kSortThreads) moe_sort_kernel(const int32_t* expert_of, const float* weight_of, int n_pairs, int n_expert, int32_t* group_start,
+                                                                int32_t* row_of, int32_t* pair_of, float* row_weight) {
+    INGOT_PDL_TRIGGER();
+    INGOT_PDL_WAIT();
+    __shared__ int s_warp[kSortThreads / 32];
+    __shared__ int s_base;
+    const int e = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    int lower = 0;
+    for (int i = threadIdx.x; i < n_pairs; i += kSortThreads) lower += expert_of[i] < e;
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) lower += __shfl_xor_sync(0xffffffffu, lower, o);
+    if (lane == 0) s_warp[warp] = lower;
+    __syncthreads();
+    if (threadIdx.x == 0) {
+        int sum = 0;
+        for (int w = 0; w < kSortThreads / 32; w++) sum += s_warp[w];
+        s_base = sum;
+        group_start[e] = sum;
+        if (e == n_expert - 1) group_start[n_expert] = n_pairs;
+    }
+    __syncthreads();
+    for (int i0 = 0; i0 < n_pairs; i0 += kSortThreads) {
+        const int i = i0 + threadIdx.x;
+        const bool mine = i < n_pairs && expert_of[i] == e;
+        const unsigned votes = __ballot_sync(0xffffffffu, mine);
+        if (lane == 0) s_warp[warp] = __popc(votes);
+        __syncthreads();
+        int before = s_base, all = 0;
+        for (int w = 0; w < kSortThreads / 32; w++) {
+            if (w < warp) before += s_warp[w];
+            all += s_warp[w];
+        }
+        if (mine) {
+            const int r = before + __popc(votes & ((1u << lane) - 1));
+            row_of[i] = r;
+            pair_of[r] = i;
+            row_weight[r] = weight_of[i];
+        }
+        __syncthreads();
+        if (threadIdx.x == 0) s_base += all;
+        __syncthreads();
+    }
+}
+
+// bf16 planes of the rows: row r is its token's row.
+__global__ void __launch_bounds__(128) moe_gather_kernel(uint4* hi, uint4* lo, const uint4* src_hi, const uint4* src_lo, const int32_t* pair_of, int top, int n8) {
+    INGOT_PDL_TRIGGER();
+    INGOT_PDL_WAIT();
+    const size_t r = blockIdx.x, t = size_t(pair_of[r] / top);
+    for (int i = threadIdx.x; i < n8; i += 128) {
+        hi[r * n8 + i] = src_hi[t * n8 + i];
+        if (lo) lo[r * n8 + i] = src_lo[t * n8 + i];
+    }
+}
+
+// Plain products: out[row][o] = act(row_weight * W_e[o] . x[source(row)]), f32 arithmetic on bf16 weights. A warp owns one output of
+// up to kRowTile rows of one expert; grid.y counts row tiles, expert after expert.
+constexpr int kRowTile = 8;
+__global__ void __launch_bounds__(256) moe_linear_kernel(float* out, const __nv_bfloat16* w, const float* x, int x_ld, int n_in, int n_out, int n_expert,
+                                                         const int32_t* group_start, const int32_t* pair_of, int top, const float* row_weight, int act) {
+    INGOT_PDL_TRIGGER();
+    INGOT_PDL_WAIT();
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    // which expert's which tile: 32 experts at a time
+    int tile = blockIdx.y, e = -1, r0 = 0, r1 = 0;
+    for (int e0 = 0; e0 < n_expert && e < 0; e0 += 32) {
+        const int mine = e0 + lane;
+        const int a = mine < n_expert ? group_start[mine] : 0, b = mine < n_expert ? group_start[mine + 1] : 0;
+        const int n = (b - a + kRowTile - 1) / kRowTile;
+        int upto = n;
+#pragma unroll
+        for (int o = 1; o < 32; o <<= 1) {
+            const int v = __shfl_up_sync(0xffffffffu, upto, o);
+            if (lane >= o) upto += v;
+        }
+        const unsigned hit = __ballot_sync(0xffffffffu, tile < upto);
+        if (hit) {
+            const int src = __ffs(hit) - 1;
+            const int local = tile - (__shfl_sync(0xffffffffu, upto, src) - __shfl_sync(0xffffffffu, n, src));
+            e = e0 + src;
+            r0 = __shfl_sync(0xffffffffu, a, src) + local * kRowTile;
+            r1 = min(__shfl_sync(0xffffffffu, b, src), r0 + kRowTile);
+        } else {
+            tile -= __shfl_sync(0xffffffffu, upto, 31);
+        }
+    }
+    if (e < 0) return;
+    const int o = blockIdx.x * 8 + warp;
+    if (o >= n_out) return;
+    const __nv_bfloat16* wr = w + ((size_t)e * n_out + o) * n_in;
+    const float* xr[kRowTile];
+#pragma unroll
+    for (int i = 0; i < kRowTile; i++) {
+        const int r = min(r0 + i, r1 - 1);
+        xr[i] = x + (size_t)(pair_of ? pair_of[r] / top : r) * x_ld;
+    }
+    float acc[kRowTile];
+#pragma unroll
+    for (int i = 0; i < kRowTile; i++) acc[i] = 0.f;
+    for (int c = lane * 8; c < n_in; c += 256) {
+        const uint4 raw = *reinterpret_cast<const uint4*>(wr + c);
+        const uint32_t u[4] = {raw.x, raw.y, raw.z, raw.w};
+        float wv[8];
+#pragma unroll
+        for (int i = 0; i < 4; i++) {
+            wv[2 * i] = __uint_as_float(u[i] << 16);
+            wv[2 * i + 1] = __uint_as_float(u[i] & 0xffff0000u);
+        }
+#pragma unroll
+        for (int i = 0; i < kRowTile; i++) {
+            if (r0 + i >= r1) break;
+            const float4 a = *reinterpret_cast<const float4*>(xr[i] + c), b = *reinterpret_cast<const float4*>(xr[i] + c + 4);
+            acc[i] = fmaf(wv[0], a.x, acc[i]); acc[i] = fmaf(wv[1], a.y, acc[i]);
+            acc[i] = fmaf(wv[2], a.z, acc[i]); acc[i] = fmaf(wv[3], a.w, acc[i]);
+            acc[i] = fmaf(wv[4], b.x, acc[i]); acc[i] = fmaf(wv[5], b.y, acc[i]);
+            acc[i] = fmaf(wv[6], b.z, acc[i]); acc[i] = fmaf(wv[7], b.w, acc[i]);
+        }
+    }
+#pragma unroll
+    for (int i = 0; i < kRowTile; i++) {
+        if (r0 + i >= r1) break;
+        float v = warp_sum(acc[i]);
+        if (lane == 0) {
+            if (row_weight) v *= row_weight[r0 + i];
+            if (act == INGOT_ACT_RELU2) v = v > 0.f ? v * v : 0.f;
+            out[(size_t)(r0 + i) * n_out + o] = v;
+        }
+    }
+}
+
+// x[t] += sum over the token's pairs of rows[row_of[pair]]; row_of null: rows[t]
+__global__ void moe_add_kernel(float* x, const float* rows, const int32_t* row_of, int top, int n4) {
+    INGOT_PDL_TRIGGER();
+    INGOT_PDL_WAIT();
+    const int i = blockIdx.x * blockDim.x + threadIdx.x;
+    if (i >= n4) return;
+    const size_t t = blockIdx.y;
+    float4 v = reinterpret_cast<const float4*>(x)[t * n4 + i];
+    for (int k = 0; k < top; k++) {
+        const float4 a = reinterpret_cast<const float4*>(rows)[(row_of ? (size_t)row_of[t * top + k] : t) * n4 + i];
+        v.x += a.x; v.y += a.y; v.z += a.z; v.w += a.w;
+    }
+    reinterpret_cast<float4*>(x)[t * n4 + i] = v;
+}
+
+}  // namespace
+
+extern "C" {
+
+int ingot_moe_route(const float* logits_dev, int ld, int n_tok, int n_expert, int top, int32_t* expert_of_dev, float* weight_of_dev, int32_t* group_start_dev,
+                    int32_t* row_of_dev, int32_t* pair_of_dev, float* row_weight_dev, void* stream) {
+    INGOT_REQUIRE(logits_dev && expert_of_dev && weight_of_dev && group_start_dev && row_of_dev && pair_of_dev && row_weight_dev, "ingot_moe_route: null argument");
+    INGOT_REQUIRE(n_tok >= 1 && n_expert >= 1 && top >= 1 && top <= n_expert && ld >= n_expert && (long long)n_tok * top < (1ll << 30), "ingot_moe_route: bad sizes");
+    cudaStream_t s = static_cast<cudaStream_t>(stream);
+    INGOT_CUDA_TRY(ingot_launch_pdl(moe_select_kernel, dim3((n_tok + 3) / 4), dim3(128), 0, s, logits_dev, ld, n_tok, n_expert, top, expert_of_dev, weight_of_dev));
+    INGOT_CUDA_TRY(ingot_launch_pdl(moe_sort_kernel, dim3(n_expert), dim3(kSortThreads), 0, s, (const int32_t*)expert_of_dev, (const float*)weight_of_dev, n_tok * top, n_expert,
+                                    group_start_dev, row_of_dev, pair_of_dev, row_weight_dev));
+    return INGOT_OK;
+}
+
+int ingot_moe_gather(void* hi_dev, void* lo_dev, const void* src_hi_dev, const void* src_lo_dev, const int32_t* pair_of_dev, int n_rows, int top, int n, void* stream) {
+    INGOT_REQUIRE(hi_dev && src_hi_dev && pair_of_dev && (!lo_dev || src_lo_dev), "ingot_moe_gather: null argument");
+    INGOT_REQUIRE(n_rows >= 1 && top >= 1 && n >= 8 && n % 8 == 0, "ingot_moe_gather: bad sizes");
+    INGOT_CUDA_TRY(ingot_launch_pdl(moe_gather_kernel, dim3(n_rows), dim3(128), 0, static_cast<cudaStream_t>(stream), static_cast<uint4*>(hi_dev), static_cast<uint4*>(lo_dev),
+                                    static_cast<const uint4*>(src_hi_dev), static_cast<const uint4*>(src_lo_dev), pair_of_dev, top, n / 8));
+    return INGOT_OK;
+}
+
+int ingot_moe_linear(float* out_dev, const void* w_dev, const float* x_dev, int x_ld, int n_in, int n_out, int n_expert, int n_rows, const int32_t* group_start_dev,
+                     const int32_t* pair_of_dev, int top, const float* row_weight_dev, int act, void* stream) {
+    INGOT_REQUIRE(out_dev && w_dev && x_dev && group_start_dev, "ingot_moe_linear: null argument");
+    INGOT_REQUIRE(n_in >= 8 && n_in % 8 == 0 && x_ld % 4 == 0 && n_out >= 1 && n_expert >= 1 && n_rows >= 1 && top >= 1, "ingot_moe_linear: bad sizes");
+    const int tiles = n_rows / kRowTile + (n_rows < n_expert ? n_rows : n_expert);  // at least as many as there can be
+    INGOT_REQUIRE(tiles <= 65535, "ingot_moe_linear: too many rows");
+    INGOT_CUDA_TRY(ingot_launch_pdl(moe_linear_kernel, dim3((n_out + 7) / 8, tiles), dim3(256), 0, static_cast<cudaStream_t>(stream), out_dev,
+                                    static_cast<const __nv_bfloat16*>(w_dev), x_dev, x_ld, n_in, n_out, n_expert, group_start_dev, pair_of_dev, top, row_weight_dev, act));
+    return INGOT_OK;
+}
+
+int ingot_moe_add(float* x_dev, const float* rows_dev, const int32_t* row_of_dev, int n_tok, int top, int n, void* stream) {
+    INGOT_REQUIRE(x_dev && rows_dev, "ingot_moe_add: null argument");
+    INGOT_REQUIRE(n_tok >= 1 && top >= 1 && (row_of_dev || top == 1) && n >= 4 && n % 4 == 0, "ingot_moe_add: bad sizes");
+    INGOT_CUDA_TRY(ingot_launch_pdl(moe_add_kernel, dim3((n / 4 + 127) / 128, n_tok), dim3(128), 0, static_cast<cudaStream_t>(stream), x_dev, rows_dev, row_of_dev, top, n / 4));
+    return INGOT_OK;
+}
+
+}  // extern "C"

@@ -57,12 +57,20 @@ ABI = {
     "ingot_selective_scan": (_I, [_P, _P, _P, _I, _P, _I, _P, _P, _I, _I, _I, _P, _I, _P, _P, _P, _I, _I, _I, _P, _P]),
     "ingot_gated_lru": (_I, [_P, _P, _P, _I, _P, _I, _I, _P, _P, _P, _P, _I, _P, _P, _I, C.c_float, _I, _P, _P]),
     "ingot_skv_create": (_I, [C.POINTER(_P), _I, _I, _I, _I, _I, _I]),
+    "ingot_skv_create_window": (_I, [C.POINTER(_P), _I, _I, _I, _I, _I, _I]),
     "ingot_skv_destroy": (None, [_P]),
     "ingot_skv_pages": (_I, [_I, _I]),
     "ingot_skv_row_length": (_I, [_I]),
     "ingot_skv_status_dev": (_P, [_P]),
     "ingot_skv_status": (_I, [_P, _P, C.POINTER(_I)]),
     "ingot_skv_append": (_I, [_P, _I, _P, _P, _I, _I, _I, _I, _I, _P, _P, C.c_float, _P, _P, _P, _I, _P]),
+    "ingot_latent_append": (_I, [_P, _I, _P, _P, _I, _I, _I, _P, _P, C.c_float, _P, _P, _P, _P, _P, _I, _P]),
+    "ingot_latent_queries": (_I, [_P, _P, _I, _I, _I, _P, _P]),
+    "ingot_latent_attend": (_I, [_P, _I, _P, _P, _I, _I, C.c_float, _P, _P, _P, _P, _I, _I, _I, _P]),
+    "ingot_moe_route": (_I, [_P, _I, _I, _I, _I, _P, _P, _P, _P, _P, _P, _P]),
+    "ingot_moe_gather": (_I, [_P, _P, _P, _P, _P, _I, _I, _I, _P]),
+    "ingot_moe_linear": (_I, [_P, _P, _P, _I, _I, _I, _I, _I, _P, _P, _I, _P, _I, _P]),
+    "ingot_moe_add": (_I, [_P, _P, _P, _I, _I, _I, _P]),
     "ingot_skv_attend": (_I, [_P, _I, _P, _P, _I, _I, C.c_float, C.c_float, _P, _P, _P, _I, _I, _P]),
     "ingot_hbm_read_probe": (_I, [_SZ, _I, C.POINTER(C.c_double), _P]),
 }
