@@ -379,19 +379,40 @@ typedef struct ingot_latent_shape {
 /* Columns q_off.. of proj_dev's rows: n_head x [dim | rot]; columns latent_off..: [rank | rot], the latent not yet normalised.
  * Writes the cache rows of the step's positions, the rotated query parts into q_rows_dev [n_tok][n_head][row length] (cache type;
  * may be null) and the unrotated query parts to q_plain [n_tok][n_head * dim]. turns_dev [rot_dims / 2]: turns per position
- * (base^(-2 i / rot_dims) / 2 pi). norm_dev [rank], zero in the padding. Tables as for ingot_skv_append. */
+ * (base^(-2 i / rot_dims) / 2 pi). norm_dev [rank], zero in the padding. Tables as for ingot_skv_append.
+ * From token long_from on the queries go to q_long_dev instead, f16 [n_tok][n_head][long_dim | long_rot], both parts zero-padded (the
+ * operand of ingot_latent_attend_expanded; f16 caches only); null: no token does. */
 int ingot_latent_append(ingot_skv* kv, int layer, const ingot_step* step, const float* proj_dev, int proj_ld, int q_off, int latent_off,
                         const ingot_latent_shape* shape, const float* norm_dev, float eps, const double* turns_dev, const ingot_act_out* q_plain,
-                        void* q_rows_dev, const int32_t* tables_dev, const int32_t* first_page_dev, int max_blocks, void* stream);
+                        void* q_rows_dev, void* q_long_dev, int long_from, int long_dim, int long_rot, const int32_t* tables_dev,
+                        const int32_t* first_page_dev, int max_blocks, void* stream);
 /* Latent queries f32 [n_tok][n_head * rank] into the first rank columns of the query rows. */
 int ingot_latent_queries(const ingot_skv* kv, const float* q_dev, int n_tok, int n_head, int rank, void* q_rows_dev, void* stream);
 /* out [n_tok][n_head * rank]: sum over the visible keys of softmax(q_row . row * scale) times the first rank columns of the row;
- * sink_dev [n_head] (may be null): the denominator also holds exp(sink). skip_len > 0: sequences of the step with that many tokens
- * or more are left out. impl: 0 = library's choice, 1 = the plain f32-arithmetic kernel, 2 = the tensor-core kernel (f16 rows, row
- * length a multiple of 32, rank a multiple of 16 and at most 512). */
+ * sink_dev [n_head] (may be null): the denominator also holds exp(sink). impl: 0 = library's choice, 1 = the plain f32-arithmetic
+ * kernel, 2 = the tensor-core kernel (f16 rows, row length a multiple of 32, rank a multiple of 16 and at most 512). */
 int ingot_latent_attend(ingot_skv* kv, int layer, const ingot_step* step, const void* q_rows_dev, int n_head, int rank, float scale,
                         const float* sink_dev, const ingot_act_out* out, const int32_t* tables_dev, const int32_t* first_page_dev, int max_blocks,
-                        int skip_len, int impl, void* stream);
+                        int impl, void* stream);
+
+/* The same for long portions, on keys and values computed from the cached latents (f16, tcgen05). For each sequence of the step
+ * the keys it sees - positions key_pos .. the portion's last - are rows key0, key0 + 1, .. of two buffers.
+ * ingot_latent_gather fetches them from the cache: latents [key][rank], rotated parts [key][rot_ld] (zero-padded); max_keys: the
+ * most any sequence of the step has. The expansion of the latents is a product (ingot_linear_tc_run_f16 of the backend). */
+int ingot_latent_gather(ingot_skv* kv, int layer, const ingot_step* step, const int32_t* key0_dev, const int32_t* key_pos_dev,
+                        int max_keys, int rank, int rot, void* latent_dev, void* rotated_dev, int rot_ld, const int32_t* tables_dev,
+                        const int32_t* first_page_dev, int max_blocks, void* stream);
+typedef struct ingot_latent_expansion {
+    const void* q;              /* f16 [q_rows][n_head][dim | rot], row t = token t of the step */
+    const void* kv;             /* f16 [key_rows][n_head][dim | v]: unrotated keys and values */
+    const void* rotated;        /* f16 [key_rows][rot] */
+    long long q_rows, key_rows; /* rows of the buffers (all of them hold finite numbers) */
+    int n_head, dim, rot, v;    /* padded parts: multiples of 64, dim + rot <= 256, v <= 128 */
+    const int32_t *key0, *key_pos; /* device, per sequence */
+} ingot_latent_expansion;
+/* out [n_tok][n_head * out_dim], out_dim <= v. */
+int ingot_latent_attend_expanded(ingot_skv* kv, const ingot_step* step, const ingot_latent_expansion* x, float scale,
+                                 const float* sink_dev, int out_dim, const ingot_act_out* out, void* stream);
 
 /* ---- Mixture of experts -----------------------------------------------------------------------------
  * Pair p = token * top + k is a token's k-th expert; rows are the pairs sorted by expert, in token order within one. */

@@ -308,7 +308,18 @@ private:
         return std::max(32, round_up((n_tok + chunks - 1) / chunks, 16));
     }
 
-    StepCtx upload_step(const StepEntry* entries, int n, Step& step) {
+    StepCtx upload_step(const StepEntry* asked, int n, Step& step) {
+        // Sequences run in ascending order of their portions, so that decoded tokens and short portions are the first rows and a
+        // mixer can treat them apart from long ones.
+        std::vector<int> order(static_cast<size_t>(n));
+        for (int i = 0; i < n; i++) order[size_t(i)] = i;
+        std::stable_sort(order.begin(), order.end(), [&](int a, int b) { return asked[a].n_tokens < asked[b].n_tokens; });
+        std::vector<StepEntry> entries;
+        std::vector<int> place(static_cast<size_t>(n));
+        for (int i = 0; i < n; i++) {
+            entries.push_back(asked[order[size_t(i)]]);
+            place[size_t(order[size_t(i)])] = i;
+        }
         std::vector<int32_t>& m = meta_;
         m.clear();
         auto mark = [&] { while (m.size() % 4) m.push_back(0); return m.size(); };
@@ -334,7 +345,11 @@ private:
         for (int i = 0; i < n; i++) m.push_back(entries[i].seq_id);
         const size_t o_want = mark();
         for (int i = 0; i < n; i++)
-            for (int w = 0; w < entries[i].n_want; w++) m.push_back(m[o_start + size_t(i)] + entries[i].want[w]);
+            for (int w = 0; w < asked[i].n_want; w++) m.push_back(m[o_start + size_t(place[size_t(i)])] + asked[i].want[w]);
+        rows_asked_.clear();
+        for (int i = 0; i < n; i++)
+            for (int t = 0; t < asked[i].n_tokens; t++) rows_asked_.push_back(m[o_start + size_t(place[size_t(i)])] + t);
+        lens_sorted_.assign(m.begin() + long(o_len), m.begin() + long(o_len) + n);
         step.first_want = step.n_want ? m[o_want] : 0;
         struct PlanAt { size_t seq, t0, len, first; int n_chunks, max_chunks; };
         auto plan = [&](int threads) {
@@ -359,7 +374,8 @@ private:
             return p;
         };
         const PlanAt scan = plan(scan_threads_), lru = plan(lru_threads_);
-        std::vector<std::pair<size_t, size_t>> table_at;
+        struct TableAt { size_t first, table, key0, key_pos; };
+        std::vector<TableAt> table_at;
         for (auto& g : ops_.caches) {
             const size_t o_first = mark();
             int width = 1;
@@ -376,7 +392,16 @@ private:
                 for (int k = 0; k < width; k++) m.push_back(first + k < g->pool.pages_per_seq() ? row[first + k] : -1);
             }
             g->width = width;
-            table_at.emplace_back(o_first, o_table);
+            const size_t o_key0 = mark();
+            plan_expansions(*g, entries);
+            for (int i = 0, row = 0, b = 0; i < n; i++) {  // key rows count from 0 in each run of sequences that are expanded together
+                if (i >= g->first_long && g->expansions[size_t(b)].seq0 + g->expansions[size_t(b)].n_seq <= i) { b++; row = 0; }
+                m.push_back(row);
+                if (i >= g->first_long) row += keys_seen(*g, entries[size_t(i)]);
+            }
+            const size_t o_key_pos = mark();
+            for (int i = 0; i < n; i++) m.push_back(g->first_visible(entries[size_t(i)].pos0));
+            table_at.push_back({o_first, o_table, o_key0, o_key_pos});
         }
         mark();
         if (m.size() > meta_cap_) {
@@ -400,6 +425,7 @@ private:
         s.st.len = meta_dev_ + o_len;
         s.st.pos0 = meta_dev_ + o_pos;
         s.st.slot = meta_dev_ + o_slot;
+        s.lens = lens_sorted_.data();
         step.tokens = meta_dev_ + o_tok;
         step.bigrams = meta_dev_ + o_bigram;
         step.want_rows = meta_dev_ + o_want;
@@ -426,11 +452,36 @@ private:
         fill(s.lru, lru, lru_scratch_, &lru_scratch_dev_, &lru_cap_);
         for (size_t i = 0; i < ops_.caches.size(); i++) {
             ops_.caches[i]->first_page = meta_dev_ + table_at[i].first;
-            ops_.caches[i]->tables = meta_dev_ + table_at[i].second;
+            ops_.caches[i]->tables = meta_dev_ + table_at[i].table;
+            ops_.caches[i]->key0 = meta_dev_ + table_at[i].key0;
+            ops_.caches[i]->key_pos = meta_dev_ + table_at[i].key_pos;
         }
         s.tc = ops_.ws != nullptr && step.n_tok >= kMinTcTokens;
         s.planes = s.tc && step.n_tok <= kPairTokens ? 2 : 1;
         return s;
+    }
+
+    static int keys_seen(const CacheGroup& g, const StepEntry& e) { return e.pos0 + e.n_tokens - g.first_visible(e.pos0); }
+    // Which sequences of the step (in ascending order of their portions) run on expanded keys, and how many at a time.
+    void plan_expansions(CacheGroup& g, const std::vector<StepEntry>& entries) const {
+        const int n = int(entries.size());
+        g.first_long = n;
+        g.expansions.clear();
+        if (g.expand_from <= 0 || !ops_.ws) return;
+        while (g.first_long > 0 && entries[size_t(g.first_long) - 1].n_tokens >= g.expand_from) g.first_long--;
+        for (int i = g.first_long; i < n; i++) {
+            const int keys = keys_seen(g, entries[size_t(i)]);
+            if (keys > g.key_rows) {  // more than there is room for: this step stays on the rows
+                g.first_long = n;
+                g.expansions.clear();
+                return;
+            }
+            if (g.expansions.empty() || g.expansions.back().n_keys + keys > g.key_rows) g.expansions.push_back({i, 0, 0, 0});
+            CacheGroup::Expansion& e = g.expansions.back();
+            e.n_seq++;
+            e.n_keys += keys;
+            e.most_keys = std::max(e.most_keys, keys);
+        }
     }
 
     int32_t bigram_row(int64_t prev, int64_t cur) const {
@@ -511,7 +562,10 @@ private:
         std::vector<float> rows(size_t(n_tok) * ld);
         cuda_check(cudaStreamSynchronize(ops_.stream), "tap");
         cuda_check(cudaMemcpy(rows.data(), ops_.x, rows.size() * 4, cudaMemcpyDeviceToHost), "tap");
-        for (int t = 0; t < n_tok; t++) tap_->insert(tap_->end(), rows.begin() + size_t(t) * ld, rows.begin() + size_t(t) * ld + w);
+        for (int t = 0; t < n_tok; t++) {
+            const auto row = rows.begin() + long(size_t(rows_asked_[size_t(t)]) * ld);
+            tap_->insert(tap_->end(), row, row + w);
+        }
     }
 
     const Design design_;
@@ -536,6 +590,7 @@ private:
     std::vector<int> lens_;            // tokens each sequence has run = position of its next one
     std::vector<int32_t> last_token_;  // of each sequence: part of its state where embeddings look at pairs of tokens
     std::vector<int32_t> meta_;
+    std::vector<int32_t> lens_sorted_, rows_asked_;  // of the current step: portions in the order they run; row of each token as asked
     int32_t *meta_dev_ = nullptr, *meta_host_ = nullptr;
     size_t meta_cap_ = 0;
     float *logits_dev_ = nullptr, *logits_ = nullptr;

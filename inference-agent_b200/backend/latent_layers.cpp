@@ -1,11 +1,19 @@
 // Latent attention of the model-folder backend (kernels: csrc/attn_latent.cu).
+#include <cuda_fp16.h>
+
+#include <cstdlib>
+
 #include "layer_ops.h"
 
 namespace {
 
 // q = W_q h, [c' | k'] = W_dkv h; c = rmsnorm(c'), k = rot(k') shared by all heads; head i scores (q_i . U_i c + rot(q_i') . k) * scale
 // under a softmax with a sink and averages V_i c; W_o over the heads side by side. W_q and W_dkv are one product. The cache holds
-// [c | k] per token; here the attention runs on those rows: U_i^T takes the query into the latent space, V_i follows once per token.
+// [c | k] per token. Two ways to the same result, chosen per sequence of a step:
+//   decoded tokens, short portions   on the cached rows: U_i^T takes the query into the latent space, V_i follows once per token
+//   long portions (16-bit form)      on keys and values expanded from the rows the portion sees
+// From how many tokens on expanding pays: it costs keys * rank * (dim + vdim) products and saves, per pair of tokens, the difference
+// between 2 rank + rot and dim + rot + vdim of them. INGOT_LATENT_EXPAND sets the number (0: never).
 class LatentAttentionMixer : public Mixer {
 public:
     LatentAttentionMixer(LayerOps& ops, const Json& c, const std::string& p) {
@@ -49,6 +57,7 @@ public:
         }
         w_value_ = ops.matrix(v.width(), latent.padded, {Part{p + "uv", {v.count(), rank}, v, latent}}, v.padded);
         w_o_ = ops.matrix(p + "o", in, v);
+        plan_expansion(ops, p, rank, rot, vdim, window);
         std::vector<double> turns;
         for (int i = 0; i < rot_dims / 2; i++) turns.push_back(std::pow(base, -2.0 * i / rot_dims) / (2 * 3.14159265358979323846));
         turns_ = static_cast<double*>(ops.alloc(turns.size() * sizeof(double)));
@@ -64,14 +73,39 @@ public:
         ops.need(kValue, value_ld_);
     }
     void run(LayerOps& ops, const StepCtx& s, const float* norm, const float* next_norm) override {
-        float *proj = ops.buf(kProj), *latent = ops.buf(kLatent), *value = ops.buf(kValue);
-        void* rows = ops.buf(kQuery);
+        float *proj = ops.buf(kProj), *value = ops.buf(kValue);
         const CacheGroup& g = *cache_;
-        const int layer = cache_layer_ + ops.pass;
+        const int layer = cache_layer_ + ops.pass, n_seq = s.st.n_seq;
+        const int from = expands_ && s.tc ? std::min(g.first_long, n_seq) : n_seq;  // sequences from here on are long
+        StepCtx head = s;  // the others: the first rows of the step
+        head.st.n_seq = from;
+        head.st.n_tok = 0;
+        for (int i = 0; i < from; i++) head.st.n_tok += s.lens[i];
+        head.st.max_len = from > 0 ? s.lens[from - 1] : 0;
+        if (from < n_seq) head.planes = head.st.n_tok <= kPairTokens ? 2 : 1;
+
         ops.norm_project(s, proj, w_in_, norm);
-        const ingot_act_out plain = ops.operand(s, ops.buf(kQueryPlain), plain_ld_, false);
-        ingot_check(ingot_latent_append(g.kv, layer, &s.st, proj, proj_ld_, 0, latent_off_, &shape_, norm_, ops.eps, turns_, &plain, rows, g.tables, g.first_page,
-                                        g.width, ops.stream));
+        const ingot_act_out plain = ops.operand(head, ops.buf(kQueryPlain), plain_ld_, false);
+        ingot_check(ingot_latent_append(g.kv, layer, &s.st, proj, proj_ld_, 0, latent_off_, &shape_, norm_, ops.eps, turns_, &plain, ops.buf(kQuery),
+                                        from < n_seq ? ops.buf(kQueryLong) : nullptr, head.st.n_tok, long_dim_, long_rot_, g.tables, g.first_page, g.width, ops.stream));
+        if (from > 0) on_rows(ops, head, layer);
+        if (from < n_seq) {
+            const ingot_act_out out = ops.operand(s, value, value_ld_, false);
+            for (const auto& e : g.expansions) on_expansion(ops, s, e, layer, out);
+        }
+        if (s.tc) {
+            if (from > 0) ops.prepare_rows(head, value, value_ld_, value_ld_);
+            ops.operand_ready(s, value_ld_);
+        }
+        ops.project_residual(s, w_o_, value, next_norm);
+    }
+
+private:
+    // kValue = V (attention on the rows) of the step's rows
+    void on_rows(LayerOps& ops, const StepCtx& s, int layer) {
+        const CacheGroup& g = *cache_;
+        float* latent = ops.buf(kLatent);
+        void* rows = ops.buf(kQuery);
         ops.operand_ready(s, plain_ld_);
         if (s.tc) {
             cuda_check(ingot_linear_tc_run_half(ops.ws, rows, heads_ * row_, row_, w_query_.data, w_query_.n_in, w_query_.n_out, shape_.rank, ops.stream), "latent queries");
@@ -80,15 +114,75 @@ public:
             ingot_check(ingot_latent_queries(g.kv, latent, s.st.n_tok, heads_, shape_.rank, rows, ops.stream));
         }
         const ingot_act_out mixed = ops.operand(s, latent, latent_ld_, false);
-        ingot_check(ingot_latent_attend(g.kv, layer, &s.st, rows, heads_, shape_.rank, scale_, sink_, &mixed, g.tables, g.first_page, g.width, 0, 0, ops.stream));
+        ingot_check(ingot_latent_attend(g.kv, layer, &s.st, rows, heads_, shape_.rank, scale_, sink_, &mixed, g.tables, g.first_page, g.width, 0, ops.stream));
         ops.operand_ready(s, latent_ld_);
-        ops.project(s, value, w_value_, latent, latent_ld_);
-        if (s.tc) ops.prepare_rows(s, value, value_ld_, value_ld_);
-        ops.project_residual(s, w_o_, value, next_norm);
+        ops.project(s, ops.buf(kValue), w_value_, latent, latent_ld_);
+    }
+    // The rows of one run of long sequences of `out`, through keys and values of their own.
+    void on_expansion(LayerOps& ops, const StepCtx& s, const CacheGroup::Expansion& e, int layer, const ingot_act_out& out) {
+        const CacheGroup& g = *cache_;
+        ingot_step st = s.st;
+        st.n_seq = e.n_seq;
+        st.max_len = s.lens[e.seq0 + e.n_seq - 1];
+        st.row_start += e.seq0;
+        st.len += e.seq0;
+        st.pos0 += e.seq0;
+        st.slot += e.seq0;
+        const int32_t *key0 = g.key0 + e.seq0, *key_pos = g.key_pos + e.seq0;
+        ingot_check(ingot_latent_gather(g.kv, layer, &st, key0, key_pos, e.most_keys, shape_.rank, shape_.rot, ops.keys(0), ops.keys(1), long_rot_,
+                                        g.tables + size_t(e.seq0) * g.width, g.first_page + e.seq0, g.width, ops.stream));
+        const int expanded = heads_ * (long_dim_ + long_v_);
+        cuda_check(ingot_linear_tc_run_f16(ops.ws, ops.keys(2), expanded, ops.keys(0), g.key_rows, e.n_keys, w_expand_, shape_.rank, expanded, ops.stream), "expansion");
+        ingot_latent_expansion x = {};
+        x.q = ops.buf(kQueryLong);
+        x.kv = ops.keys(2);
+        x.rotated = ops.keys(1);
+        x.q_rows = ops.max_step;
+        x.key_rows = g.key_rows;
+        x.n_head = heads_;
+        x.dim = long_dim_;
+        x.rot = long_rot_;
+        x.v = long_v_;
+        x.key0 = key0;
+        x.key_pos = key_pos;
+        ingot_check(ingot_latent_attend_expanded(g.kv, &st, &x, scale_, sink_, value_ld_ / heads_, &out, ops.stream));
+    }
+    void plan_expansion(LayerOps& ops, const std::string& p, int rank, int rot, int vdim, int window) {
+        long_dim_ = round_up(dim_, 64);
+        long_rot_ = round_up(rot, 64);
+        long_v_ = round_up(vdim, 64);
+        const int saved = 2 * rank + rot - (dim_ + rot + vdim);
+        int least = saved > 0 ? std::max(64, std::min(512, rank * (dim_ + vdim) / saved)) : 0;
+        if (const char* e = getenv("INGOT_LATENT_EXPAND")) least = std::max(0, atoi(e));
+        expands_ = !ops.opt.f32 && least > 0 && least <= ops.max_step && long_dim_ + long_rot_ <= 256 && long_v_ <= 128 && scale_ > 0;
+        if (!expands_) return;
+        CacheGroup& g = *cache_;
+        g.expand_from = g.expand_from > 0 ? std::min(g.expand_from, least) : least;
+        // a portion and what its first token sees; without a window, a context of some length besides
+        g.key_rows = int(std::min<long long>(ops.opt.max_tokens, (long long)ops.max_step + (window > 0 ? window : 32768)));
+        const int expanded = heads_ * (long_dim_ + long_v_);
+        ops.need_keys(size_t(g.key_rows) * shape_.rank * 2, size_t(g.key_rows) * long_rot_ * 2, size_t(g.key_rows) * expanded * 2);
+        ops.need(kQueryLong, heads_ * (long_dim_ + long_rot_) / 2);
+        // f16 like the latents: a bf16 weight is an f16 number too unless it is tiny (below 2^-14 it loses bits of its own 8)
+        std::vector<uint16_t> host(size_t(expanded) * shape_.rank, 0);
+        auto fill = [&](const std::string& name, int size, int at) {
+            const std::vector<float> w = tensor_f32(ops.bf16(name, {heads_ * size, rank}));
+            for (int h = 0; h < heads_; h++)
+                for (int k = 0; k < size; k++)
+                    for (int r = 0; r < rank; r++) {
+                        const __half v = __float2half_rn(std::min(std::max(w[(size_t(h) * size + k) * rank + r], -65504.f), 65504.f));
+                        memcpy(&host[(size_t(h) * (long_dim_ + long_v_) + at + k) * shape_.rank + r], &v, 2);
+                    }
+        };
+        fill(p + "uk", dim_, 0);
+        fill(p + "uv", vdim, long_dim_);
+        w_expand_ = ops.matrix(host, expanded, shape_.rank, 0, true).data;
     }
 
-private:
     int heads_, dim_, row_, latent_off_, proj_ld_, plain_ld_, latent_ld_, value_ld_, cache_layer_ = 0;
+    int long_dim_ = 0, long_rot_ = 0, long_v_ = 0;
+    bool expands_ = false;
+    void* w_expand_ = nullptr;
     ingot_latent_shape shape_ = {};
     float scale_;
     CacheGroup* cache_;

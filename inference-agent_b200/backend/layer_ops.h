@@ -54,6 +54,8 @@ cudaError_t ingot_linear_tc_run_blocks(ingot_linear_ws* ws, float* out, const vo
 cudaError_t ingot_linear_tc_run_partial(ingot_linear_ws* ws, const void* w, int n_in, int n_out, int slot, cudaStream_t s);
 cudaError_t ingot_linear_tc_run_half(ingot_linear_ws* ws, void* out, int out_ld, int out_block, const void* w, int n_in, int n_out, int rows_per_block,
                                      cudaStream_t s);
+cudaError_t ingot_linear_tc_run_f16(ingot_linear_ws* ws, void* out, int out_ld, const void* a, int a_rows, int n_tok, const void* w, int n_in, int n_out,
+                                    cudaStream_t s);
 cudaError_t ingot_linear_tc_finish_residual_norm_bf16(ingot_linear_ws* ws, float* x, const float* norm_w, float eps, int n_mean, int planes,
                                                       const float* pair_rows, const int32_t* row_of, int top, cudaStream_t s);
 cudaError_t ingot_linear_tc_finish_gated_bf16(ingot_linear_ws* ws, int act, int planes, cudaStream_t s);
@@ -98,13 +100,14 @@ struct Part {
     int r0 = 0, c0 = 0, src_row0 = 0, src_stride = 0;
 };
 
-enum Buf { kProj, kConv, kStateIn, kDt, kGates, kMix, kGateUp, kMid, kNormed, kQuery, kQueryPlain, kLatent, kValue, kRouter, kExpertIn, kExpertMid, kExpertOut,
+enum Buf { kProj, kConv, kStateIn, kDt, kGates, kMix, kGateUp, kMid, kNormed, kQuery, kQueryPlain, kQueryLong, kLatent, kValue, kRouter, kExpertIn, kExpertMid, kExpertOut,
            kBranch, kConcat, kBufCount };
 
 // The step as the launches see it.
 struct StepCtx {
     ingot_step st = {};
     ingot_scan_plan scan = {}, lru = {};
+    const int32_t* lens = nullptr;  // host copy of st.len; sequences come in ascending order of it
     bool tc = false;  // products on the tensor cores (16-bit form, more than one token)
     int planes = 1;   // bf16 planes an activation is given as there
 };
@@ -119,6 +122,12 @@ struct CacheGroup {
     int pages_per_chunk = 0;
     const int32_t *tables = nullptr, *first_page = nullptr;  // device, of the current step
     int width = 0;
+    // Portions that run on keys expanded per head (latent attention): from how many tokens on (0: none), how many keys at a time, and
+    // of the current step the first sequence that does, the runs of sequences that are expanded together, and where their keys go.
+    int expand_from = 0, key_rows = 0, first_long = 0;
+    struct Expansion { int seq0, n_seq, n_keys, most_keys; };
+    std::vector<Expansion> expansions;
+    const int32_t *key0 = nullptr, *key_pos = nullptr;       // device, per sequence
     int page(int pos) const { return ingot_skv_pages(chunk, pos + 1) - 1; }
     int first_visible(int pos) const { return chunk > 0 ? pos / chunk * chunk : window > 0 && pos >= window ? pos - window + 1 : 0; }
     bool forgets() const { return chunk > 0 || window > 0; }  // pages fall out of sight for good
@@ -153,9 +162,14 @@ public:
         return p;
     }
     void need(Buf b, int columns) { columns_[b] = std::max(columns_[b], columns); }
+    void need_keys(size_t latents, size_t rotated, size_t expanded) {
+        const size_t bytes[3] = {latents, rotated, expanded};
+        for (int i = 0; i < 3; i++) key_bytes_[i] = std::max(key_bytes_[i], bytes[i]);
+    }
     void tc_shape(int n_in, int n_out) { tc_in_ = std::max(tc_in_, n_in); tc_out_ = std::max(tc_out_, n_out); }
     void allocate() {
         for (int b = 0; b < kBufCount; b++) bufs_[b] = columns_[b] ? static_cast<float*>(alloc(size_t(max_step) * columns_[b] * 4, true)) : nullptr;
+        for (int i = 0; i < 3; i++) keys_[i] = key_bytes_[i] ? alloc(key_bytes_[i], true) : nullptr;
         if (!opt.f32 && max_step >= kMinTcTokens) cuda_check(ingot_linear_ws_create_bf16(&ws, max_step, tc_in_, tc_out_), "linear workspace");
         loader_.finish();
         cuda_check(cudaDeviceSynchronize(), "model upload");
@@ -220,6 +234,7 @@ public:
 
     // ---- the step ----
     float* buf(Buf b) const { return bufs_[b]; }
+    void* keys(int i) const { return keys_[i]; }  // 0 latents, 1 rotated parts, 2 expanded keys and values
     // Output of a kernel that feeds a product: the operand planes on the tensor-core path (and f32 rows if `keep`), else f32.
     ingot_act_out operand(const StepCtx& s, float* f32, int ld, bool keep, int planes = 0) const {
         ingot_act_out o = {};
@@ -366,6 +381,8 @@ private:
     int columns_[kBufCount] = {};
     float* bufs_[kBufCount] = {};
     int tc_in_ = 8, tc_out_ = 8;
+    size_t key_bytes_[3] = {0, 0, 0};
+    void* keys_[3] = {nullptr, nullptr, nullptr};
     Branch branch_;
     const float* norm_ready_ = nullptr;  // the norm weights x has been prepared with
 };

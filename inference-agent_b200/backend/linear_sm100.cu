@@ -818,6 +818,45 @@ cudaError_t ingot_linear_tc_run_half(ingot_linear_ws* ws, void* out, int out_ld,
     return launch_gemm(ws, nullptr, &w, n_in, &n_out, 1, 0, 0, false, false, s, rows_per_block, static_cast<__half*>(out), out_ld, out_block);
 }
 
+// The map of an activation or weight buffer, made once.
+static const CUtensorMap* map_of(ingot_linear_ws* ws, const void* base, int rows, int cols, int box, bool bf16) {
+    const auto key = std::make_tuple(base, rows, cols, box);
+    auto it = ws->w_maps.find(key);
+    if (it == ws->w_maps.end()) {
+        CUtensorMap tm;
+        if (!make_map(&tm, base, rows, cols, box, bf16)) return nullptr;
+        it = ws->w_maps.emplace(key, tm).first;
+    }
+    return &it->second;
+}
+
+// out f16 [n_tok][out_ld] = a W^T, both operands f16: a [a_rows][n_in] with n_tok <= a_rows, W [n_out][n_in]. Lengths are multiples of 8.
+cudaError_t ingot_linear_tc_run_f16(ingot_linear_ws* ws, void* out, int out_ld, const void* a, int a_rows, int n_tok, const void* w, int n_in, int n_out, cudaStream_t s) {
+    if (n_in % 8 != 0 || n_out % 8 != 0 || out_ld % 8 != 0 || n_tok < 1 || n_tok > a_rows) return cudaErrorInvalidValue;
+    GemmParams p = {};
+    p.tiles_m = (n_tok + kBM - 1) / kBM;
+    const long long waves128 = ((long long)((n_out + 127) / 128) * p.tiles_m + ws->num_sms - 1) / ws->num_sms;
+    const long long waves256 = ((long long)((n_out + 255) / 256) * p.tiles_m + ws->num_sms - 1) / ws->num_sms;
+    const int kBN = waves128 > 1 && 3 * waves256 < 2 * waves128 ? 256 : 128;
+    if (ws->w_maps.size() > 65536) ws->w_maps.clear();
+    const CUtensorMap *ma = map_of(ws, a, a_rows, n_in, 128, false), *mw = map_of(ws, w, n_out, n_in, kBN, false);
+    if (!ma || !mw) return cudaErrorUnknown;
+    p.tiles_n = (n_out + kBN - 1) / kBN;
+    for (int m = 0; m < 3; m++) { p.n_out[m] = n_out; p.tile_end[m] = p.tiles_n; }
+    p.status = ws->status;
+    p.n_tok = n_tok;
+    p.k_steps = (n_in + kBK - 1) / kBK;
+    p.n_split = 1;
+    p.a_bytes = kBoxBytes;
+    p.idesc = idesc_f16(kBN);
+    p.out_half = static_cast<__half*>(out);
+    p.half_ld = out_ld;
+    auto run = [&](auto kernel, int smem) {
+        return launch_pdl(kernel, dim3(p.tiles_n * p.tiles_m), dim3(kThreads), (size_t)smem, s, *ma, *ma, *mw, *mw, *mw, p);
+    };
+    return kBN == 256 ? run(linear_sm100_kernel<1, 256, false>, Ring<1, 256>::kSmemBytes) : run(linear_sm100_kernel<1, 128, false>, Ring<1, 128>::kSmemBytes);
+}
+
 cudaError_t ingot_grouped_tc_run(ingot_linear_ws* ws, const ingot_grouped_gemm* g, cudaStream_t s) {
     if (!ws->bf16 || g->n_in % 8 != 0 || g->n_out % 8 != 0 || g->n_rows < 1 || g->n_groups < 1 || g->rows_per_group < 1) return cudaErrorInvalidValue;
     const int planes = g->a_lo ? 2 : 1, box_rows = g->rows_per_group >= 128 ? 128 : (g->rows_per_group + 7) / 8 * 8;
@@ -831,20 +870,10 @@ cudaError_t ingot_grouped_tc_run(ingot_linear_ws* ws, const ingot_grouped_gemm* 
         const long long waves256 = ((long long)((g->n_out + 255) / 256) * likely + ws->num_sms - 1) / ws->num_sms;
         if (waves128 > 1 && 3 * waves256 < 2 * waves128) kBN = 256;
     }
-    auto map_of = [&](const void* base, int rows, int cols, int box) -> const CUtensorMap* {
-        const auto key = std::make_tuple(base, rows, cols, box);
-        auto it = ws->w_maps.find(key);
-        if (it == ws->w_maps.end()) {
-            CUtensorMap tm;
-            if (!make_map(&tm, base, rows, cols, box, true)) return nullptr;
-            if (ws->w_maps.size() > 65536) ws->w_maps.clear();
-            it = ws->w_maps.emplace(key, tm).first;
-        }
-        return &it->second;
-    };
-    const CUtensorMap* hi = map_of(g->a_hi, g->n_rows, g->n_in, box_rows);
-    const CUtensorMap* lo = planes > 1 ? map_of(g->a_lo, g->n_rows, g->n_in, box_rows) : hi;
-    const CUtensorMap* w = map_of(g->w, g->n_groups * g->n_out, g->n_in, kBN);
+    if (ws->w_maps.size() > 65536) ws->w_maps.clear();
+    const CUtensorMap* hi = map_of(ws, g->a_hi, g->n_rows, g->n_in, box_rows, true);
+    const CUtensorMap* lo = planes > 1 ? map_of(ws, g->a_lo, g->n_rows, g->n_in, box_rows, true) : hi;
+    const CUtensorMap* w = map_of(ws, g->w, g->n_groups * g->n_out, g->n_in, kBN, true);
     if (!hi || !lo || !w) return cudaErrorUnknown;
     p.tiles_n = (g->n_out + kBN - 1) / kBN;
     for (int m = 0; m < 3; m++) { p.n_out[m] = g->n_out; p.tile_end[m] = p.tiles_n; }

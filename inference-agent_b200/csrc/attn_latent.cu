@@ -42,6 +42,8 @@ struct AppendParams {
     const double* turns;  // [rot_dims / 2] turns per position
     SharedOut plain;      // [n_tok][n_head * dim]
     void* q_rows;         // [n_tok][n_head][row]; the rotated part is written
+    __half* q_long;       // [n_tok][n_head][long_dim | long_rot] of the tokens from long_from on, instead of the two above
+    int long_from, long_dim, long_rot;
     void* rows;
     int row;
     const int32_t *tables, *first_page;
@@ -88,6 +90,21 @@ __global__ void __launch_bounds__(kAppendThreads) latent_append_kernel(const App
         for (int i = threadIdx.x; i < p.sh.rot; i += kAppendThreads) put(dst + p.sh.rank + i, rotated(c + p.sh.rank, i));
     }
     const int per = p.sh.dim + p.sh.rot;
+    if (tok >= p.long_from) {
+        const int width = p.long_dim + p.long_rot;
+        __half* dst = p.q_long + (size_t)tok * p.sh.n_head * width;
+        for (int i = threadIdx.x * 2; i < p.sh.n_head * width; i += kAppendThreads * 2) {
+            const int h = i / width, d = i - h * width;
+            float v[2];
+#pragma unroll
+            for (int e = 0; e < 2; e++) {
+                const int k = d + e - p.long_dim;
+                v[e] = k < 0 ? (d + e < p.sh.dim ? q[h * per + d + e] : 0.f) : k < p.sh.rot ? rotated(q + h * per + p.sh.dim, k) : 0.f;
+            }
+            *reinterpret_cast<__half2*>(dst + i) = __floats2half2_rn(fminf(fmaxf(v[0], -65504.f), 65504.f), fminf(fmaxf(v[1], -65504.f), 65504.f));
+        }
+        return;
+    }
     if (p.plain.f32 || p.plain.hi) {
         const int n4 = p.sh.n_head * p.sh.dim / 4, d4 = p.sh.dim / 4;
         for (int i = threadIdx.x; i < n4; i += kAppendThreads) {
@@ -157,7 +174,7 @@ __global__ void __launch_bounds__(kLatThreads) latent_mma_kernel(const AttendPar
     INGOT_PDL_WAIT();
     const int seq = blockIdx.z, len = p.st.len[seq], H = p.n_head, n_rows = len * H;
     const int split = blockIdx.y, row0 = ((int)gridDim.x - 1 - (int)blockIdx.x) * 16 * kMT;  // later rows see more keys, they go first
-    if (row0 >= n_rows || len >= p.skip_len) return;
+    if (row0 >= n_rows) return;
     const LatentSmem L(kMT, p.dim);
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, j = lane & 3;
     const int mi = warp % kMT, kg = warp / kMT;
@@ -383,8 +400,7 @@ __global__ void __launch_bounds__(kMergeThreads) latent_merge_kernel(const Atten
     INGOT_PDL_TRIGGER();
     INGOT_PDL_WAIT();
     __shared__ float s_f[kMaxSplits];
-    const int h = blockIdx.x, seq = p.st.row_seq[blockIdx.y];
-    if (p.st.len[seq] >= p.skip_len) return;
+    const int h = blockIdx.x;
     const size_t tok = blockIdx.y;
     const int ld = p.out_dim + 2;
     const float* part = p.part + (tok * p.n_head + h) * p.n_splits * ld;
@@ -420,7 +436,7 @@ constexpr int kSmemLimit = 227 * 1024;
 bool mma_takes(int dim, int dv) { return dim % 32 == 0 && dv % 16 == 0 && dv <= 512 && LatentSmem(1, dim).bytes <= kSmemLimit; }
 
 int launch_mma(ingot_skv* kv, AttendParams p, cudaStream_t s) {
-    const int rows = std::min(p.st.max_len, p.skip_len) * p.n_head;
+    const int rows = p.st.max_len * p.n_head;
     int mt = rows <= 16 ? 1 : rows <= 32 ? 2 : 4;
     while (mt > 1 && LatentSmem(mt, p.dim).bytes > kSmemLimit) mt /= 2;
     const int smem = LatentSmem(mt, p.dim).bytes;
@@ -467,7 +483,8 @@ extern "C" {
 
 int ingot_latent_append(ingot_skv* kv, int layer, const ingot_step* step, const float* proj_dev, int proj_ld, int q_off, int latent_off,
                         const ingot_latent_shape* shape, const float* norm_dev, float eps, const double* turns_dev, const ingot_act_out* q_plain,
-                        void* q_rows_dev, const int32_t* tables_dev, const int32_t* first_page_dev, int max_blocks, void* stream) {
+                        void* q_rows_dev, void* q_long_dev, int long_from, int long_dim, int long_rot, const int32_t* tables_dev,
+                        const int32_t* first_page_dev, int max_blocks, void* stream) {
     INGOT_REQUIRE(kv && step_ok(step) && shape, "ingot_latent_append: null handle or bad step");
     INGOT_REQUIRE_DEVICE(kv);
     INGOT_REQUIRE(layer >= 0 && layer < kv->n_layer, "ingot_latent_append: layer out of range");
@@ -481,9 +498,12 @@ int ingot_latent_append(ingot_skv* kv, int layer, const ingot_step* step, const 
         ingot_set_error("ingot_latent_append: needs a window-form cache with one row per token and at most " + std::to_string(kMaxRot) + " rotated values");
         return INGOT_ERR_UNSUPPORTED;
     }
+    INGOT_REQUIRE(!q_long_dev || (kv->dtype == INGOT_F16 && long_from >= 0 && long_dim % 2 == 0 && long_rot % 2 == 0 && long_dim >= sh.dim && long_rot >= sh.rot),
+                  "ingot_latent_append: bad long queries");
     const size_t esz = kv->dtype == INGOT_F32 ? 4 : 2;
     AppendParams p = {*step, proj_dev, proj_ld, q_off, latent_off, sh, norm_dev, eps, turns_dev,
                       SharedOut{q_plain->f32, static_cast<__nv_bfloat16*>(q_plain->hi), static_cast<__nv_bfloat16*>(q_plain->lo), q_plain->ld, 1.0f}, q_rows_dev,
+                      static_cast<__half*>(q_long_dev), q_long_dev ? long_from : 0x7fffffff, long_dim, long_rot,
                       static_cast<char*>(kv->rows) + kv->layer_elems * layer * esz, kv->dim, tables_dev, first_page_dev, max_blocks, kv->n_blocks, page_map(kv),
                       kv->status_dev};
     auto kernel = kv->dtype == INGOT_F32 ? latent_append_kernel<float> : latent_append_kernel<__half>;
@@ -503,7 +523,7 @@ int ingot_latent_queries(const ingot_skv* kv, const float* q_dev, int n_tok, int
 }
 
 int ingot_latent_attend(ingot_skv* kv, int layer, const ingot_step* step, const void* q_rows_dev, int n_head, int rank, float scale, const float* sink_dev,
-                        const ingot_act_out* out, const int32_t* tables_dev, const int32_t* first_page_dev, int max_blocks, int skip_len, int impl, void* stream) {
+                        const ingot_act_out* out, const int32_t* tables_dev, const int32_t* first_page_dev, int max_blocks, int impl, void* stream) {
     INGOT_REQUIRE(kv && step_ok(step), "ingot_latent_attend: null handle or bad step");
     INGOT_REQUIRE_DEVICE(kv);
     INGOT_REQUIRE(layer >= 0 && layer < kv->n_layer, "ingot_latent_attend: layer out of range");
@@ -513,7 +533,7 @@ int ingot_latent_attend(ingot_skv* kv, int layer, const ingot_step* step, const 
     AttendParams p = {*step, q_rows_dev, static_cast<const char*>(kv->rows) + kv->layer_elems * layer * esz, nullptr, tables_dev, first_page_dev, max_blocks,
                       kv->n_blocks, n_head, 1, kv->dim, rank, page_map(kv), scale,
                       SharedOut{out->f32, static_cast<__nv_bfloat16*>(out->hi), static_cast<__nv_bfloat16*>(out->lo), out->ld, 1.0f}, kv->status_dev, 1, nullptr,
-                      sink_dev, skip_len > 0 ? skip_len : 0x7fffffff};
+                      sink_dev};
     cudaStream_t s = static_cast<cudaStream_t>(stream);
     if (kv->dtype == INGOT_F16 && impl != 1 && mma_takes(kv->dim, rank) && out->ld % 2 == 0) return launch_mma(kv, p, s);
     if (impl == 2) {

@@ -1,0 +1,487 @@
+// Latent attention of long portions on the expansion (attn_latent.cu has the mechanism): keys and values of each head computed from
+// the cached latents for the positions the portion sees, then attention per head on the sm_100a tensor cores - the tcgen05 / TMA /
+// tensor-memory pipeline of attn_shared_kv_sm100.cu with keys and values of unequal lengths, a window and a sink.
+//
+// Operands, all f16, laid out by their producers so that every TMA box is 128 rows x 64 columns (a unit, 16 KB):
+//   queries   [token][head][dim | rot]   unrotated and rotated part, each padded to 64 columns
+//   expanded  [key][head][dim | value]   U_h c and V_h c, likewise
+//   rotated   [key][rot]                 one part shared by all heads
+// The keys of a sequence are consecutive rows, from the first one its portion sees to the portion's last token, so position and row
+// differ by a constant; rows past the end belong to other sequences and are masked by their position.
+//
+// One CTA = one head x 256 tokens (two tiles of 128 rows) of one sequence; it walks the keys 128 at a time. Score operands are 2 to 4
+// units deep, values 1 or 2. One ring of units serves both, in the order K0 | V0 K1 | V1 K2 | ..; a value tile of two units whose slots
+// are not adjacent (the ring wraps) is multiplied unit by unit.
+// Roles: warp 0 TMA, warp 1 MMA issue, warps 4-7 and 8-11 softmax of the two row tiles, one thread per row.
+// Tensor memory: S0 S1 (128 columns each), O0 O1 (up to 128 each); P (f16) overwrites the first half of its S. MMA order:
+//   QK(0,0) QK(1,0) | PV(0,j) QK(0,j+1) PV(1,j) QK(1,j+1) | ...
+// Every mbarrier wait is bounded: on expiry all roles leave, copies in flight are drained, tensor memory is freed and the cache's
+// status word gets its bit.
+#include <map>
+#include <mutex>
+#include <tuple>
+
+#include "attn_shared_kv.cuh"
+#include "sm100_ptx.cuh"
+
+namespace {
+
+using namespace ingot_sm100;
+
+constexpr int kTileRows = 128, kTileKeys = 128, kUnit = 128 * 64 * 2;
+constexpr int kAllUnits = 14;  // of shared memory: two query tiles and the ring
+constexpr int kMaxRing = kAllUnits - 4;
+constexpr int kThreads = 384;
+constexpr uint32_t kTmemCols = 512;
+constexpr float kRescaleThreshold = 8.0f;  // log2 units
+constexpr unsigned long long kWaitLimitNs = 2000000000ull;
+constexpr int kOffBar = kAllUnits * kUnit;
+constexpr int kSmemBytes = kOffBar + 256 + 1024;  // + alignment slack
+
+struct Bars {
+    uint64_t full[kMaxRing];
+    uint64_t empty[kMaxRing];
+    uint64_t q_ready;
+    uint64_t s_ready[2];
+    uint64_t p_ready[2];
+    uint64_t o_final[2];
+    uint32_t tmem_base;
+    uint32_t abort_flag;
+};
+static_assert(sizeof(Bars) <= 256, "barriers");
+
+struct Params {
+    ingot_step st;
+    const int32_t *key0, *key_pos;  // per sequence: first key row, and its position
+    PageMap map;
+    int n_head, dim_units, rot_units, v_units, out_dim;
+    float scale;                    // of the scores, times log2 e
+    const float* sink;
+    SharedOut out;
+    int* status;
+};
+
+__device__ __forceinline__ float ex2(float x) {
+    float y;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+    return y;
+}
+__device__ __forceinline__ void ffma2(float& d0, float& d1, float a0, float a1, float b, float c) {
+    asm("{\n.reg .b64 ra, rb, rc, rd;\n"
+        "mov.b64 ra, {%2, %3};\nmov.b64 rb, {%4, %4};\nmov.b64 rc, {%5, %5};\n"
+        "fma.rn.f32x2 rd, ra, rb, rc;\nmov.b64 {%0, %1}, rd;\n}\n"
+        : "=f"(d0), "=f"(d1) : "f"(a0), "f"(a1), "f"(b), "f"(c));
+}
+__device__ __forceinline__ void fadd2(float& d0, float& d1, float a0, float a1, float b0, float b1) {
+    asm("{\n.reg .b64 ra, rb, rd;\n"
+        "mov.b64 ra, {%2, %3};\nmov.b64 rb, {%4, %5};\n"
+        "add.rn.f32x2 rd, ra, rb;\nmov.b64 {%0, %1}, rd;\n}\n"
+        : "=f"(d0), "=f"(d1) : "f"(a0), "f"(a1), "f"(b0), "f"(b1));
+}
+
+// Instruction descriptors, kind::f16: f16 A and B, f32 accumulate, M = 128; scores: A and B K-major, N = 128; values: B MN-major
+constexpr uint32_t kIdescQK = (1u << 4) | ((128u >> 3) << 17) | ((128u >> 4) << 24);
+__device__ __forceinline__ uint32_t idesc_pv(int n) { return (1u << 4) | (1u << 16) | ((uint32_t)(n >> 3) << 17) | ((128u >> 4) << 24); }
+
+__global__ void __launch_bounds__(kThreads, 1)
+latent_sm100_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_kv, const __grid_constant__ CUtensorMap map_rot,
+                    const __grid_constant__ Params p) {
+    extern __shared__ unsigned char smem_dyn[];
+    INGOT_PDL_TRIGGER();
+    const uint32_t smem_base = (smem_u32(smem_dyn) + 1023u) & ~1023u;
+    unsigned char* smem_al = smem_dyn + (smem_base - smem_u32(smem_dyn));
+    Bars* bars = reinterpret_cast<Bars*>(smem_al + kOffBar);
+    volatile uint32_t* abort_flag = &bars->abort_flag;
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int warp_u = __shfl_sync(0xffffffffu, warp, 0);
+
+    const int seq = blockIdx.z, head = blockIdx.y, len = p.st.len[seq];
+    const int row_base = ((int)gridDim.x - 1 - (int)blockIdx.x) * 2 * kTileRows;  // later rows may see more keys, they go first
+    if (row_base >= len) {
+        INGOT_PDL_WAIT();
+        return;
+    }
+    const int pos0 = p.st.pos0[seq], tok0 = p.st.row_start[seq];
+    const int first_key = p.map.first_visible(pos0 + row_base);  // position of the first key this CTA fetches
+    const int key_row0 = p.key0[seq] + first_key - p.key_pos[seq];
+    const int n_it = (pos0 + min(row_base + 2 * kTileRows, len) - 1 - first_key) / kTileKeys + 1;
+    const int nq = p.dim_units + p.rot_units, nv = p.v_units, ring = kAllUnits - 2 * nq;
+    const uint32_t ring_base = smem_base + 2 * nq * kUnit;
+
+    if (threadIdx.x == 0) {
+        for (int s = 0; s < ring; s++) { mbar_init(smem_u32(&bars->full[s]), 1); mbar_init(smem_u32(&bars->empty[s]), 1); }
+        mbar_init(smem_u32(&bars->q_ready), 1);
+        for (int q = 0; q < 2; q++) {
+            mbar_init(smem_u32(&bars->s_ready[q]), 1);
+            mbar_init(smem_u32(&bars->p_ready[q]), 4);
+            mbar_init(smem_u32(&bars->o_final[q]), 1);
+        }
+        bars->abort_flag = 0;
+        asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
+    }
+    if (warp == 1) {
+        asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;" ::"r"(smem_u32(&bars->tmem_base)), "r"(kTmemCols) : "memory");
+        asm volatile("tcgen05.relinquish_alloc_permit.cta_group::1.sync.aligned;" ::: "memory");
+    }
+    INGOT_PDL_WAIT();  // the operands come from the kernels before
+    tc_fence_before();
+    __syncthreads();
+    tc_fence_after();
+    const uint32_t tmem = bars->tmem_base;
+
+    if (warp_u < 4) {
+        asm volatile("setmaxnreg.dec.sync.aligned.u32 56;");
+        if (warp_u == 0) {
+            // ---------------- TMA producer: one lane ----------------
+            if (lane == 0) {
+                const int q_x = head * nq * 64, kv_x = head * (p.dim_units + nv) * 64;
+                const uint32_t q_ready = smem_u32(&bars->q_ready);
+                mbar_expect_tx(q_ready, 2 * nq * kUnit);
+                for (int q = 0; q < 2; q++)
+                    for (int u = 0; u < nq; u++)
+                        tma_load_2d(smem_base + (q * nq + u) * kUnit, &map_q, q_x + u * 64, tok0 + row_base + q * kTileRows, q_ready);
+                int slot = 0, round = 0, armed = 0;
+                bool ok = true;
+                auto unit = [&](const CUtensorMap* map, int x, int y) {
+                    if (!ok) return;
+                    ok = mbar_wait(smem_u32(&bars->empty[slot]), (uint32_t)((round & 1) ^ 1), abort_flag, kWaitLimitNs);
+                    if (!ok) return;
+                    const uint32_t full = smem_u32(&bars->full[slot]);
+                    mbar_expect_tx(full, kUnit);
+                    tma_load_2d(ring_base + slot * kUnit, map, x, y, full);
+                    armed++;
+                    if (++slot == ring) { slot = 0; round++; }
+                };
+                for (int it = 0; it <= n_it && ok; it++) {
+                    if (it > 0)
+                        for (int u = 0; u < nv; u++) unit(&map_kv, kv_x + (p.dim_units + u) * 64, key_row0 + (it - 1) * kTileKeys);
+                    if (it < n_it) {
+                        for (int u = 0; u < p.dim_units; u++) unit(&map_kv, kv_x + u * 64, key_row0 + it * kTileKeys);
+                        for (int u = 0; u < p.rot_units; u++) unit(&map_rot, u * 64, key_row0 + it * kTileKeys);
+                    }
+                }
+                if (!ok) {
+                    // copies already issued must land before the CTA's shared memory is released
+                    for (int i = max(0, armed - ring); i < armed; i++) {
+                        const uint64_t t0 = globaltimer_ns();
+                        while (!mbar_try_wait(smem_u32(&bars->full[i % ring]), (uint32_t)((i / ring) & 1)) && globaltimer_ns() - t0 < 100000000ull) {}
+                    }
+                    const uint64_t t0 = globaltimer_ns();
+                    while (!mbar_try_wait(q_ready, 0) && globaltimer_ns() - t0 < 100000000ull) {}
+                }
+            }
+        } else if (warp_u == 1) {
+            // ---------------- MMA issuer: the whole warp walks the loop, one elected lane issues ----------------
+            int slot = 0, round = 0;  // of the next unit to be consumed
+            bool ok = __all_sync(0xffffffffu, mbar_wait(smem_u32(&bars->q_ready), 0, abort_flag, kWaitLimitNs)) != 0;
+            auto wait_units = [&](int n) {  // the n units from the current place on have landed
+                int s = slot, r = round;
+                for (int u = 0; u < n && ok; u++) {
+                    ok = __all_sync(0xffffffffu, mbar_wait(smem_u32(&bars->full[s]), (uint32_t)(r & 1), abort_flag, kWaitLimitNs)) != 0;
+                    if (++s == ring) { s = 0; r++; }
+                }
+            };
+            auto advance = [&](int n) {
+                slot += n;
+                if (slot >= ring) { slot -= ring; round++; }
+            };
+            auto wrap = [&](int s) { return s >= ring ? s - ring : s; };
+            auto issue_qk = [&](int q, int first) {
+                for (int u = 0; u < nq; u++) {
+                    const uint32_t a = smem_base + (q * nq + u) * kUnit, b = ring_base + wrap(first + u) * kUnit;
+#pragma unroll
+                    for (int ks = 0; ks < 4; ks++)
+                        tc_mma_ss(tmem + q * 128, make_desc(a + ks * 32, 16, 1024), make_desc(b + ks * 32, 16, 1024), kIdescQK, (u > 0 || ks > 0) ? 1u : 0u);
+                }
+                tc_commit(smem_u32(&bars->s_ready[q]));
+            };
+            auto issue_pv = [&](int q, int first, bool fresh) {
+                const int step = first + nv <= ring ? nv : 1;  // units per instruction
+                for (int u = 0; u < nv; u += step) {
+                    const uint32_t v = ring_base + wrap(first + u) * kUnit;
+#pragma unroll
+                    for (int ks = 0; ks < 8; ks++)
+                        tc_mma_ts(tmem + 256 + q * 128 + u * 64, tmem + q * 128 + ks * 8, make_desc(v + ks * 2048, kUnit, 1024), idesc_pv(step * 64),
+                                  (!fresh || ks > 0) ? 1u : 0u);
+                }
+            };
+            auto release = [&](int first, int n) {
+                for (int u = 0; u < n; u++) tc_commit(smem_u32(&bars->empty[wrap(first + u)]));
+            };
+            wait_units(nq);
+            if (ok) {
+                tc_fence_after();
+                if (elect_one()) {
+                    issue_qk(0, slot);
+                    issue_qk(1, slot);
+                    release(slot, nq);
+                }
+                __syncwarp();
+                advance(nq);
+            }
+            for (int j = 0; j < n_it && ok; j++) {
+                const bool more = j + 1 < n_it;
+                wait_units(more ? nv + nq : nv);
+                if (!ok) break;
+                const int v_slot = slot, k_slot = wrap(slot + nv);
+#pragma unroll
+                for (int q = 0; q < 2; q++) {
+                    ok = __all_sync(0xffffffffu, mbar_wait(smem_u32(&bars->p_ready[q]), (uint32_t)(j & 1), abort_flag, kWaitLimitNs)) != 0;
+                    if (!ok) break;
+                    tc_fence_after();
+                    if (elect_one()) {
+                        issue_pv(q, v_slot, j == 0);
+                        if (q == 1) release(v_slot, nv);
+                        if (more) {
+                            issue_qk(q, k_slot);
+                            if (q == 1) release(k_slot, nq);
+                        } else {
+                            tc_commit(smem_u32(&bars->o_final[q]));
+                        }
+                    }
+                    __syncwarp();
+                }
+                advance(more ? nv + nq : nv);
+            }
+        }
+    } else {
+        asm volatile("setmaxnreg.inc.sync.aligned.u32 224;");
+        // ---------------- softmax warps: one thread per row ----------------
+        const int q = (warp - 4) >> 2, row_in_tile = ((warp & 3) << 5) | lane;
+        const int R = row_base + q * kTileRows + row_in_tile;
+        const bool valid = R < len;
+        const int pos = pos0 + (valid ? R : len - 1), vis = p.map.first_visible(pos);  // rows past the end behave like the last row
+        const uint32_t lane_sel = (uint32_t)((warp & 3) << 5) << 16;
+        const uint32_t s_tmem = tmem + q * 128 + lane_sel, o_tmem = tmem + 256 + q * 128 + lane_sel;
+        float m_ref = 0.f, l = 0.f;
+        bool ok = true;
+        const int pos_min = __shfl_sync(0xffffffffu, pos, 0), vis_max = __shfl_sync(0xffffffffu, vis, 31);  // rows ascend with the lane
+        for (int j = 0; j < n_it; j++) {
+            ok = mbar_wait(smem_u32(&bars->s_ready[q]), (uint32_t)(j & 1), abort_flag, kWaitLimitNs);
+            ok = __all_sync(0xffffffffu, ok) != 0;
+            if (!ok) break;
+            tc_fence_after();
+            float s[128];
+#pragma unroll
+            for (int c = 0; c < 4; c++) tmem_ld32(s_tmem + c * 32, *reinterpret_cast<float(*)[32]>(&s[c * 32]));
+            tmem_wait_ld();
+            const int kp = first_key + j * kTileKeys;  // position of the tile's first key
+            if (kp < vis_max || kp + kTileKeys - 1 > pos_min) {  // warp-uniform: some row of this warp needs the mask
+                const int lo = vis - kp, hi = pos - kp;
+#pragma unroll
+                for (int i = 0; i < 128; i++)
+                    if (i < lo || i > hi) s[i] = -INFINITY;
+            }
+            float mxa = fmaxf(s[0], s[1]), mxb = fmaxf(s[2], s[3]), mxc = fmaxf(s[4], s[5]), mxd = fmaxf(s[6], s[7]);
+#pragma unroll
+            for (int i = 8; i < 128; i += 8) {
+                mxa = fmaxf(mxa, fmaxf(s[i], s[i + 1]));
+                mxb = fmaxf(mxb, fmaxf(s[i + 2], s[i + 3]));
+                mxc = fmaxf(mxc, fmaxf(s[i + 4], s[i + 5]));
+                mxd = fmaxf(mxd, fmaxf(s[i + 6], s[i + 7]));
+            }
+            const float mx = fmaxf(fmaxf(mxa, mxb), fmaxf(mxc, mxd)) * p.scale;
+            // Lazy rescale: the reference maximum moves only when the row's grew by more than 2^8. A row that has seen only masked
+            // keys keeps -inf; its first finite maximum "grows" from there with a rescale factor of exactly 0.
+            const bool grow = j == 0 || mx > m_ref + kRescaleThreshold;
+            if (j == 0) {
+                m_ref = mx;
+            } else if (__any_sync(0xffffffffu, grow)) {
+                const float alpha = grow ? ex2(m_ref - mx) : 1.0f;
+                if (grow) { m_ref = mx; l *= alpha; }
+                for (int c = 0; c < nv * 2; c++) {
+                    float o[32];
+                    tmem_ld32(o_tmem + c * 32, o);
+                    tmem_wait_ld();
+                    uint32_t ob[32];
+#pragma unroll
+                    for (int i = 0; i < 32; i++) ob[i] = __float_as_uint(o[i] * alpha);
+                    tmem_st32(o_tmem + c * 32, ob);
+                }
+            }
+            const float neg_m = m_ref == -INFINITY ? 0.f : -m_ref;
+            float sum0 = 0.f, sum1 = 0.f;
+#pragma unroll
+            for (int c = 0; c < 2; c++) {
+                uint32_t pk[32];
+#pragma unroll
+                for (int i = 0; i < 32; i++) {
+                    float x0, x1;
+                    ffma2(x0, x1, s[c * 64 + 2 * i], s[c * 64 + 2 * i + 1], p.scale, neg_m);
+                    const float p0 = ex2(x0), p1 = ex2(x1);
+                    fadd2(sum0, sum1, sum0, sum1, p0, p1);
+                    pk[i] = pack_half2_rn(p0, p1);
+                }
+                tmem_st32(s_tmem + c * 32, pk);
+            }
+            l += sum0 + sum1;
+            tmem_wait_st();
+            tc_fence_before();
+            __syncwarp();
+            if (lane == 0) mbar_arrive(smem_u32(&bars->p_ready[q]));
+        }
+        // ---------------- epilogue: O / l through the tile's Q buffer, row-contiguous stores ----------------
+        if (ok) {
+            ok = mbar_wait(smem_u32(&bars->o_final[q]), 0, abort_flag, kWaitLimitNs);
+            ok = __all_sync(0xffffffffu, ok) != 0;
+        }
+        if (ok) {
+            tc_fence_after();
+            if (p.sink) l += exp2f(p.sink[head] * 1.44269504f - m_ref);
+            const float inv = 1.0f / l;
+            unsigned char* stage = smem_al + q * nq * kUnit;  // [128 rows][64 f32], 16-byte pieces XOR-swizzled by row
+            const int warp_row0 = (warp & 3) << 5, piece = lane & 15;
+            const int rows_here = min(32, len - (row_base + q * kTileRows + warp_row0));  // of this warp (may be negative)
+            for (int ps = 0; ps < nv; ps++) {
+                if (ps) __syncwarp();
+                unsigned char* my = stage + row_in_tile * 256;
+#pragma unroll
+                for (int c = 0; c < 2; c++) {
+                    float o[32];
+                    tmem_ld32(o_tmem + ps * 64 + c * 32, o);
+                    tmem_wait_ld();
+#pragma unroll
+                    for (int i = 0; i < 8; i++)
+                        *reinterpret_cast<float4*>(my + (((c * 8 + i) ^ (row_in_tile & 7)) << 4)) =
+                            make_float4(o[4 * i] * inv, o[4 * i + 1] * inv, o[4 * i + 2] * inv, o[4 * i + 3] * inv);
+                }
+                __syncwarp();
+                const int d = ps * 64 + piece * 4;
+#pragma unroll 4
+                for (int it = 0; it < 16; it++) {
+                    const int owner = it * 2 + (lane >> 4);
+                    if (owner >= rows_here || d >= p.out_dim) continue;
+                    const int r = warp_row0 + owner;
+                    const float4 v = *reinterpret_cast<const float4*>(stage + r * 256 + ((piece ^ (r & 7)) << 4));
+                    const size_t row = (size_t)tok0 + row_base + q * kTileRows + r;
+                    p.out.store2(row, head * p.out_dim + d, v.x, v.y);  // out_dim is a multiple of 4
+                    p.out.store2(row, head * p.out_dim + d + 2, v.z, v.w);
+                }
+            }
+        }
+    }
+    // ---------------- teardown ----------------
+    tc_fence_before();
+    __syncthreads();
+    if (threadIdx.x == 0 && *abort_flag) atomicOr(p.status, kDevErrBarrierTimeout);
+    if (warp == 1) {
+        tc_fence_after();
+        asm volatile("tcgen05.dealloc.cta_group::1.sync.aligned.b32 %0, %1;" ::"r"(tmem), "r"(kTmemCols) : "memory");
+    }
+}
+
+// Cached rows of the keys a portion sees, one after the other: latents [key][rank], rotated parts [key][rot_ld]. One warp per key.
+struct GatherParams {
+    ingot_step st;
+    const int32_t *key0, *key_pos;
+    const __half* rows;
+    int row, rank, rot, rot_ld;
+    const int32_t *tables, *first_page;
+    int max_blocks, n_blocks;
+    PageMap map;
+    int* status;
+    __half *latent, *rotated;
+};
+__global__ void __launch_bounds__(256) latent_gather_kernel(const GatherParams p) {
+    INGOT_PDL_TRIGGER();
+    INGOT_PDL_WAIT();
+    const int seq = blockIdx.y, i = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+    const int len = p.st.len[seq];
+    if (i >= p.st.pos0[seq] + len - p.key_pos[seq]) return;
+    const int pos = p.key_pos[seq] + i;
+    const int blk = table_block(p.tables, p.first_page, p.max_blocks, p.n_blocks, seq, p.map.page(pos), p.status);
+    const size_t at = (size_t)p.key0[seq] + i;
+    const uint4* src = reinterpret_cast<const uint4*>(p.rows + ((size_t)max(blk, 0) * kBlockTokens + p.map.slot(pos)) * p.row);
+    const uint4 zero = make_uint4(0, 0, 0, 0);
+    for (int c = lane; c < p.rank / 8; c += 32) reinterpret_cast<uint4*>(p.latent + at * p.rank)[c] = blk >= 0 ? src[c] : zero;
+    for (int c = lane; c < p.rot_ld / 8; c += 32) reinterpret_cast<uint4*>(p.rotated + at * p.rot_ld)[c] = blk >= 0 && c < p.rot / 8 ? src[p.rank / 8 + c] : zero;
+}
+
+typedef CUresult (*EncodeTiledFn)(CUtensorMap*, CUtensorMapDataType, cuuint32_t, void*, const cuuint64_t*, const cuuint64_t*,
+                                  const cuuint32_t*, const cuuint32_t*, CUtensorMapInterleave, CUtensorMapSwizzle,
+                                  CUtensorMapL2promotion, CUtensorMapFloatOOBfill);
+EncodeTiledFn encode_fn() {
+    static EncodeTiledFn fn = nullptr;
+    static std::once_flag once;
+    std::call_once(once, [] {
+        void* sym = nullptr;
+        cudaDriverEntryPointQueryResult qres;
+        if (cudaGetDriverEntryPoint("cuTensorMapEncodeTiled", &sym, cudaEnableDefault, &qres) == cudaSuccess &&
+            qres == cudaDriverEntryPointSuccess)
+            fn = reinterpret_cast<EncodeTiledFn>(sym);
+    });
+    return fn;
+}
+// f16 [rows][cols], boxes of 128 rows x 64 columns, 128-byte swizzle, zeros outside
+bool unit_map(CUtensorMap* map, const void* base, long long rows, int cols) {
+    const cuuint64_t dims[2] = {(cuuint64_t)cols, (cuuint64_t)rows};
+    const cuuint64_t strides[1] = {(cuuint64_t)cols * 2};
+    const cuuint32_t box[2] = {64, 128}, estr[2] = {1, 1};
+    return encode_fn() && encode_fn()(map, CU_TENSOR_MAP_DATA_TYPE_FLOAT16, 2, const_cast<void*>(base), dims, strides, box, estr, CU_TENSOR_MAP_INTERLEAVE_NONE,
+                                      CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) == CUDA_SUCCESS;
+}
+
+bool step_ok(const ingot_step* st) {
+    return st && st->n_tok >= 1 && st->n_seq >= 1 && st->n_seq <= 65535 && st->max_len >= 1 && st->row_start && st->len && st->pos0;
+}
+
+}  // namespace
+
+extern "C" {
+
+int ingot_latent_gather(ingot_skv* kv, int layer, const ingot_step* step, const int32_t* key0_dev, const int32_t* key_pos_dev, int max_keys,
+                        int rank, int rot, void* latent_dev, void* rotated_dev, int rot_ld, const int32_t* tables_dev, const int32_t* first_page_dev, int max_blocks,
+                        void* stream) {
+    INGOT_REQUIRE(kv && step_ok(step), "ingot_latent_gather: null handle or bad step");
+    INGOT_REQUIRE_DEVICE(kv);
+    INGOT_REQUIRE(layer >= 0 && layer < kv->n_layer, "ingot_latent_gather: layer out of range");
+    INGOT_REQUIRE(key0_dev && key_pos_dev && latent_dev && rotated_dev && tables_dev && max_blocks >= 1 && max_keys >= 1, "ingot_latent_gather: null argument");
+    INGOT_REQUIRE(kv->dtype == INGOT_F16 && kv->n_head_kv == 1 && kv->dim % 8 == 0 && rank % 8 == 0 && rot % 8 == 0 && rank + rot <= kv->dim && rot_ld % 8 == 0 &&
+                      rot_ld >= rot, "ingot_latent_gather: bad rows");
+    const GatherParams p = {*step, key0_dev, key_pos_dev, static_cast<const __half*>(kv->rows) + kv->layer_elems * layer, kv->dim, rank, rot, rot_ld,
+                            tables_dev, first_page_dev, max_blocks, kv->n_blocks, page_map(kv), kv->status_dev, static_cast<__half*>(latent_dev),
+                            static_cast<__half*>(rotated_dev)};
+    INGOT_CUDA_TRY(ingot_launch_pdl(latent_gather_kernel, dim3((max_keys + 7) / 8, step->n_seq), dim3(256), 0, static_cast<cudaStream_t>(stream), p));
+    return INGOT_OK;
+}
+
+int ingot_latent_attend_expanded(ingot_skv* kv, const ingot_step* step, const ingot_latent_expansion* x, float scale, const float* sink_dev,
+                                 int out_dim, const ingot_act_out* out, void* stream) {
+    INGOT_REQUIRE(kv && step_ok(step) && x && out, "ingot_latent_attend_expanded: null handle or bad step");
+    INGOT_REQUIRE_DEVICE(kv);
+    INGOT_REQUIRE(x->q && x->kv && x->rotated && x->key0 && x->key_pos && x->n_head >= 1 && x->q_rows >= 1 && x->key_rows >= 1, "ingot_latent_attend_expanded: null argument");
+    INGOT_REQUIRE(out_dim >= 4 && out_dim % 4 == 0 && out_dim <= x->v && out->ld % 4 == 0, "ingot_latent_attend_expanded: bad output");
+    if (x->dim < 64 || x->dim % 64 || x->rot < 64 || x->rot % 64 || x->dim + x->rot > 256 || (x->v != 64 && x->v != 128)) {
+        ingot_set_error("ingot_latent_attend_expanded: parts are multiples of 64 columns, 256 for scores and 128 for values at most");
+        return INGOT_ERR_UNSUPPORTED;
+    }
+    static std::mutex lock;
+    static std::map<std::tuple<int, const void*, long long, int>, CUtensorMap> maps;  // per device, buffer and shape
+    CUtensorMap m[3];
+    {
+        std::lock_guard<std::mutex> hold(lock);
+        const std::tuple<int, const void*, long long, int> keys[3] = {
+            {kv->device, x->q, x->q_rows, x->n_head * (x->dim + x->rot)}, {kv->device, x->kv, x->key_rows, x->n_head * (x->dim + x->v)}, {kv->device, x->rotated, x->key_rows, x->rot}};
+        if (maps.size() > 4096) maps.clear();
+        for (int i = 0; i < 3; i++) {
+            auto it = maps.find(keys[i]);
+            if (it == maps.end()) {
+                CUtensorMap fresh;
+                if (!unit_map(&fresh, std::get<1>(keys[i]), std::get<2>(keys[i]), std::get<3>(keys[i]))) {
+                    ingot_set_error("ingot_latent_attend_expanded: the driver cannot encode the tensor map");
+                    return INGOT_ERR_UNSUPPORTED;
+                }
+                it = maps.emplace(keys[i], fresh).first;
+            }
+            m[i] = it->second;
+        }
+    }
+    const Params p = {*step, x->key0, x->key_pos, page_map(kv), x->n_head, x->dim / 64, x->rot / 64, x->v / 64, out_dim, scale * 1.44269504f, sink_dev,
+                      SharedOut{out->f32, static_cast<__nv_bfloat16*>(out->hi), static_cast<__nv_bfloat16*>(out->lo), out->ld, 1.0f}, kv->status_dev};
+    INGOT_CUDA_TRY(cudaFuncSetAttribute(latent_sm100_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, kSmemBytes));
+    const dim3 grid((step->max_len + 2 * kTileRows - 1) / (2 * kTileRows), x->n_head, step->n_seq);
+    INGOT_CUDA_TRY(ingot_launch_pdl(latent_sm100_kernel, grid, dim3(kThreads), size_t(kSmemBytes), static_cast<cudaStream_t>(stream), m[0], m[1], m[2], p));
+    return INGOT_OK;
+}
+
+}  // extern "C"

@@ -120,7 +120,7 @@ __global__ void __launch_bounds__(128) shared_kv_attend_kernel(const AttendParam
     const int seq = blockIdx.z, kvh = blockIdx.y;
     const int group = p.n_head / p.n_head_kv, len = p.st.len[seq];
     const int row0 = blockIdx.x * kRows, n_rows = len * group;
-    if (row0 >= n_rows || len >= p.skip_len) return;
+    if (row0 >= n_rows) return;
     const int dim = p.dim, ldk = kD * 32 + 1;
     float* sq = smem;                       // [16][kD * 32]
     float* sk = sq + kRows * kD * 32;       // [32][kD * 32 + 1]

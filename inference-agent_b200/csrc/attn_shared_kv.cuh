@@ -85,7 +85,6 @@ struct AttendParams {
     int n_splits;   // decoding: CTAs per (token, KV head) over the keys
     float* part;    // [token][head][split][dim + 2]
     const float* sink = nullptr;  // per head: one more term exp(sink) of the denominator (null: none)
-    int skip_len = 0x7fffffff;    // sequences of the step with this many tokens or more are left to another launch
 };
 
 // The plain kernel (f32 arithmetic, any row length up to 1024, window, chunk and sink); dtype of rows and queries.

@@ -64,9 +64,11 @@ ABI = {
     "ingot_skv_status_dev": (_P, [_P]),
     "ingot_skv_status": (_I, [_P, _P, C.POINTER(_I)]),
     "ingot_skv_append": (_I, [_P, _I, _P, _P, _I, _I, _I, _I, _I, _P, _P, C.c_float, _P, _P, _P, _I, _P]),
-    "ingot_latent_append": (_I, [_P, _I, _P, _P, _I, _I, _I, _P, _P, C.c_float, _P, _P, _P, _P, _P, _I, _P]),
+    "ingot_latent_append": (_I, [_P, _I, _P, _P, _I, _I, _I, _P, _P, C.c_float, _P, _P, _P, _P, _I, _I, _I, _P, _P, _I, _P]),
+    "ingot_latent_gather": (_I, [_P, _I, _P, _P, _P, _I, _I, _I, _P, _P, _I, _P, _P, _I, _P]),
+    "ingot_latent_attend_expanded": (_I, [_P, _P, _P, C.c_float, _P, _I, _P, _P]),
     "ingot_latent_queries": (_I, [_P, _P, _I, _I, _I, _P, _P]),
-    "ingot_latent_attend": (_I, [_P, _I, _P, _P, _I, _I, C.c_float, _P, _P, _P, _P, _I, _I, _I, _P]),
+    "ingot_latent_attend": (_I, [_P, _I, _P, _P, _I, _I, C.c_float, _P, _P, _P, _P, _I, _I, _P]),
     "ingot_moe_route": (_I, [_P, _I, _I, _I, _I, _P, _P, _P, _P, _P, _P, _P]),
     "ingot_moe_gather": (_I, [_P, _P, _P, _P, _P, _I, _I, _I, _P]),
     "ingot_moe_linear": (_I, [_P, _P, _P, _I, _I, _I, _I, _I, _P, _P, _I, _P, _I, _P]),

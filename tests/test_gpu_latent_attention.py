@@ -1,0 +1,344 @@
+"""Latent attention (csrc/attn_latent.cu) through the C ABI against latent_moe_reference.py: both cache types, every kernel, lengths
+that need padding, pages in random order that leave with the window, single keys that stand out at every edge, sinks."""
+import ctypes as C
+
+import numpy as np
+import pytest
+
+import latent_moe_reference as R
+from hybrid_step import Step, act_out, dev, lib
+
+pytestmark = pytest.mark.gpu
+F32, F16 = 0, 1
+EPS, BASE = 1e-5, 300.0
+
+
+class CShape(C.Structure):
+    _fields_ = [(n, C.c_int) for n in ("n_head", "dim", "rot", "rank", "rank_count", "rot_dims")]
+
+
+class Shape:
+    def __init__(self, heads, dim, rot, rank, window, rot_dims=None):
+        self.heads, self.dim, self.rot, self.rank, self.window = heads, dim, rot, rank, window
+        self.rot_dims = rot if rot_dims is None else rot_dims
+        up = lambda v, q: (v + q - 1) // q * q
+        self.dim_p, self.rot_p, self.rank_p = up(dim, 8), up(rot, 8), up(rank, 16)
+        self.row = up(self.rank_p + self.rot_p, 32)
+        self.c = CShape(heads, self.dim_p, self.rot_p, self.rank_p, rank, self.rot_dims)
+        self.scale = 1.3 / (dim + rot) ** 0.5
+
+
+def reference(s, q, kv, norm, U, sink):
+    """q [n, heads, dim + rot], kv [n, rank + rot] before normalisation and rotation, U [heads, dim, rank]: the mixed latents."""
+    n = q.shape[0]
+    c = R.rms(kv[:, :s.rank], EPS) * norm
+    kr = R.rotate(kv[:, s.rank:], range(n), s.rot_dims, BASE)
+    qr = R.rotate(q[:, :, s.dim:], range(n), s.rot_dims, BASE)
+    out = np.zeros((n, s.heads, s.rank))
+    for h in range(s.heads):
+        score = (q[:, h, :s.dim] @ U[h] @ c.T + qr[:, h] @ kr.T) * s.scale
+        score = np.where(R.window_visible(n, s.window), score, -np.inf)
+        out[:, h] = R.softmax_with_sink(score, -np.inf if sink is None else sink[h]) @ c
+    return out
+
+
+def run(s, seqs, cuts, norm, U, sink, dtype, impl, seed=0, tables_seen_only=True):
+    """seqs: [(q, kv)]; cuts: portion lengths per sequence (repeated). Pages behind the window are not in the tables."""
+    import torch
+    rng = np.random.default_rng(seed)
+    pages = [(q.shape[0] + 15) // 16 for q, _ in seqs]
+    order = rng.permutation(sum(pages) + 3).astype(np.int32)
+    tables = np.split(order[:sum(pages)], np.cumsum(pages)[:-1])
+    h = C.c_void_p()
+    lib(lib().ingot_skv_create_window(C.byref(h), 2, 1, s.row, dtype, s.window, len(order)))
+    turns = dev(np.array([BASE ** (-2.0 * i / s.rot_dims) / (2 * np.pi) for i in range(s.rot_dims // 2)]), np.float64)
+    norm_d = dev(np.pad(norm, (0, s.rank_p - s.rank)))
+    sink_d = None if sink is None else dev(sink)
+    outs = [np.zeros((q.shape[0], s.heads, s.rank)) for q, _ in seqs]
+    done, k = [0] * len(seqs), 0
+    try:
+        while any(d < q.shape[0] for d, (q, _) in zip(done, seqs)):
+            live = [i for i, (q, _) in enumerate(seqs) if done[i] < q.shape[0]]
+            part = [min(cuts[i][k % len(cuts[i])], seqs[i][0].shape[0] - done[i]) for i in live]
+            st = Step(part, [done[i] for i in live], [0] * len(live))
+            q = np.concatenate([seqs[i][0][done[i]:done[i] + n] for i, n in zip(live, part)])
+            kv = np.concatenate([seqs[i][1][done[i]:done[i] + n] for i, n in zip(live, part)])
+            n_tok = st.n_tok
+            heads = np.zeros((n_tok, s.heads, s.dim_p + s.rot_p))
+            heads[:, :, :s.dim], heads[:, :, s.dim_p:s.dim_p + s.rot] = q[:, :, :s.dim], q[:, :, s.dim:]
+            lat = np.zeros((n_tok, s.rank_p + s.rot_p))
+            lat[:, :s.rank], lat[:, s.rank_p:s.rank_p + s.rot] = kv[:, :s.rank], kv[:, s.rank:]
+            proj = dev(np.concatenate([heads.reshape(n_tok, -1), lat], axis=1))
+            first = [max(0, done[i] - s.window + 1) // 16 if s.window and tables_seen_only else 0 for i in live]
+            width = max((done[i] + n + 15) // 16 - f for i, n, f in zip(live, part, first))
+            tab = np.full((len(live), width), -1, np.int32)
+            for r, (i, n, f) in enumerate(zip(live, part, first)):
+                tab[r, :(done[i] + n + 15) // 16 - f] = tables[i][f:(done[i] + n + 15) // 16]
+            td, fd = dev(tab, np.int32), dev(first, np.int32)
+            plain = torch.zeros(n_tok, s.heads * s.dim_p, device="cuda")
+            rows = torch.zeros(n_tok, s.heads, s.row, device="cuda", dtype=torch.float32 if dtype == F32 else torch.float16)
+            out = torch.zeros(n_tok, s.heads * s.rank_p, device="cuda")
+            hi, lo = (torch.zeros(n_tok, s.heads * s.rank_p, device="cuda", dtype=torch.bfloat16) for _ in range(2))
+            po, oo = act_out(plain), act_out(out, hi, lo)
+            for layer in (1, 0):
+                lib(lib().ingot_latent_append(h, layer, C.byref(st.c), proj.data_ptr(), proj.shape[1], 0, s.heads * (s.dim_p + s.rot_p), C.byref(s.c),
+                                              norm_d.data_ptr(), EPS, turns.data_ptr(), C.byref(po), rows.data_ptr(), None, 0, 0, 0, td.data_ptr(), fd.data_ptr(), width, None))
+            torch.cuda.synchronize()
+            got_plain = plain.cpu().numpy().reshape(n_tok, s.heads, s.dim_p)
+            assert np.array_equal(got_plain[:, :, :s.dim], q[:, :, :s.dim].astype(np.float32))
+            ql = np.zeros((n_tok, s.heads, s.rank_p))
+            ql[:, :, :s.rank] = np.einsum("nhd,hdr->nhr", q[:, :, :s.dim], U)
+            qd = dev(ql.reshape(n_tok, -1))
+            lib(lib().ingot_latent_queries(h, qd.data_ptr(), n_tok, s.heads, s.rank_p, rows.data_ptr(), None))
+            lib(lib().ingot_latent_attend(h, 0, C.byref(st.c), rows.data_ptr(), s.heads, s.rank_p, s.scale, None if sink is None else sink_d.data_ptr(),
+                                          C.byref(oo), td.data_ptr(), fd.data_ptr(), width, impl, None))
+            torch.cuda.synchronize()
+            status = C.c_int(-1)
+            lib(lib().ingot_skv_status(h, None, C.byref(status)))
+            assert status.value == 0
+            assert ((hi.float() + lo.float() - out).abs().max() <= 1e-4 * out.abs().max()).item()  # the bf16 pair is the f32 result
+            res = out.cpu().numpy().reshape(n_tok, s.heads, s.rank_p)
+            assert not res[:, :, s.rank:].any()
+            r = 0
+            for i, n in zip(live, part):
+                outs[i][done[i]:done[i] + n] = res[r:r + n, :, :s.rank]
+                r += n
+                done[i] += n
+            k += 1
+    finally:
+        lib().ingot_skv_destroy(h)
+    return outs
+
+
+class CExpansion(C.Structure):
+    _fields_ = [("q", C.c_void_p), ("kv", C.c_void_p), ("rotated", C.c_void_p), ("q_rows", C.c_longlong), ("key_rows", C.c_longlong), ("n_head", C.c_int),
+                ("dim", C.c_int), ("rot", C.c_int), ("v", C.c_int), ("key0", C.c_void_p), ("key_pos", C.c_void_p)]
+
+
+def run_expanded(s, seqs, starts, norm, U, V, sink, seed=0):
+    """The tokens from starts[i] on as one portion of sequence i, on expanded keys and values (V [heads, vdim, rank]); what comes before is
+    only appended. Returns [len, heads, vdim] per sequence."""
+    import torch
+    rng = np.random.default_rng(seed)
+    up = lambda v: (v + 63) // 64 * 64
+    vdim = V.shape[1]
+    D, Rt, Dv = up(s.dim), up(s.rot), up(vdim)
+    pages = [(q.shape[0] + 15) // 16 for q, _ in seqs]
+    order = rng.permutation(sum(pages) + 3).astype(np.int32)
+    tables = np.split(order[:sum(pages)], np.cumsum(pages)[:-1])
+    h = C.c_void_p()
+    lib(lib().ingot_skv_create_window(C.byref(h), 1, 1, s.row, F16, s.window, len(order)))
+    turns = dev(np.array([BASE ** (-2.0 * i / s.rot_dims) / (2 * np.pi) for i in range(s.rot_dims // 2)]), np.float64)
+    norm_d, sink_d = dev(np.pad(norm, (0, s.rank_p - s.rank))), None if sink is None else dev(sink)
+    width = max(pages)
+    tab = np.full((len(seqs), width), -1, np.int32)
+    for r, t in enumerate(tables):
+        tab[r, :len(t)] = t
+    td = dev(tab, np.int32)
+    try:
+        for before in (True, False):
+            who = [i for i in range(len(seqs)) if not before or starts[i] > 0]
+            if not who:
+                continue
+            lens, pos = ([starts[i] for i in who], [0] * len(who)) if before else ([seqs[i][0].shape[0] - starts[i] for i in who], starts)
+            st = Step(lens, pos, [0] * len(who))
+            cut = lambda a, i, k: a[:starts[i]] if before else a[starts[i]:]
+            q, kv = (np.concatenate([cut(seqs[i][k], i, k) for i in who]) for k in (0, 1))
+            n_tok = st.n_tok
+            heads, lat = np.zeros((n_tok, s.heads, s.dim_p + s.rot_p)), np.zeros((n_tok, s.rank_p + s.rot_p))
+            heads[:, :, :s.dim], heads[:, :, s.dim_p:s.dim_p + s.rot] = q[:, :, :s.dim], q[:, :, s.dim:]
+            lat[:, :s.rank], lat[:, s.rank_p:s.rank_p + s.rot] = kv[:, :s.rank], kv[:, s.rank:]
+            proj = dev(np.concatenate([heads.reshape(n_tok, -1), lat], axis=1))
+            long = torch.full((n_tok, s.heads, D + Rt), np.nan, device="cuda", dtype=torch.float16)
+            mine = dev(tab[who], np.int32)
+            lib(lib().ingot_latent_append(h, 0, C.byref(st.c), proj.data_ptr(), proj.shape[1], 0, s.heads * (s.dim_p + s.rot_p), C.byref(s.c), norm_d.data_ptr(), EPS,
+                                          turns.data_ptr(), C.byref(act_out(torch.zeros(1, 4, device="cuda"))), None, long.data_ptr(), 0, D, Rt, mine.data_ptr(), None,
+                                          width, None))
+        first = [max(0, p - s.window + 1) if s.window else 0 for p in starts]
+        count = [q.shape[0] - f for (q, _), f in zip(seqs, first)]
+        key0, key_pos = np.concatenate([[0], np.cumsum(count)[:-1]]) + 5, np.array(first)
+        rows = sum(count) + 9
+        latent = torch.zeros(rows, s.rank_p, device="cuda", dtype=torch.float16)
+        rotated = torch.zeros(rows, Rt, device="cuda", dtype=torch.float16)
+        kd, pd = dev(key0, np.int32), dev(key_pos, np.int32)
+        lib(lib().ingot_latent_gather(h, 0, C.byref(st.c), kd.data_ptr(), pd.data_ptr(), max(count), s.rank_p, s.rot_p, latent.data_ptr(), rotated.data_ptr(), Rt,
+                                      td.data_ptr(), None, width, None))
+        kv = torch.zeros(rows, s.heads, D + Dv, device="cuda", dtype=torch.float16)
+        c = latent[:, :s.rank].double()
+        kv[:, :, :s.dim] = torch.einsum("nr,hdr->nhd", c, torch.from_numpy(U).cuda()).half()
+        kv[:, :, D:D + vdim] = torch.einsum("nr,hdr->nhd", c, torch.from_numpy(V).cuda()).half()
+        vp = (vdim + 3) // 4 * 4
+        out = torch.full((n_tok, s.heads * vp), np.nan, device="cuda")
+        hi, lo = (torch.full((n_tok, s.heads * vp), np.nan, device="cuda", dtype=torch.bfloat16) for _ in range(2))
+        x = CExpansion(long.data_ptr(), kv.data_ptr(), rotated.data_ptr(), n_tok, rows, s.heads, D, Rt, Dv, kd.data_ptr(), pd.data_ptr())
+        lib(lib().ingot_latent_attend_expanded(h, C.byref(st.c), C.byref(x), s.scale, None if sink is None else sink_d.data_ptr(), vp, C.byref(act_out(out, hi, lo)), None))
+        torch.cuda.synchronize()
+        status = C.c_int(-1)
+        lib(lib().ingot_skv_status(h, None, C.byref(status)))
+        assert status.value == 0
+        assert ((hi.float() + lo.float() - out).abs().max() <= 1e-4 * out.abs().max()).item()
+        res = out.cpu().numpy().reshape(n_tok, s.heads, vp)[:, :, :vdim]
+        return np.split(res, np.cumsum([q.shape[0] - p for (q, _), p in zip(seqs, starts)])[:-1])
+    finally:
+        lib().ingot_skv_destroy(h)
+
+
+def random_case(s, lens, seed):
+    rng = np.random.default_rng(seed)
+    seqs = [(rng.standard_normal((n, s.heads, s.dim + s.rot)), 2 * rng.standard_normal((n, s.rank + s.rot))) for n in lens]
+    return seqs, 1 + 0.3 * rng.standard_normal(s.rank), rng.standard_normal((s.heads, s.dim, s.rank)) / s.rank ** 0.5, rng.standard_normal(s.heads) + 1
+
+
+SHAPES = [(3, 10, 6, 21, 19), (16, 16, 16, 48, 40), (20, 8, 4, 64, 0), (5, 24, 40, 130, 33), (32, 16, 32, 256, 64), (7, 12, 2, 500, 100), (1, 8, 8, 16, 1),
+          (70, 8, 64, 512, 48)]
+CUTS = {"whole": [[10 ** 9]] * 3, "portions": [[70, 2, 33, 16], [5, 64], [2]], "single": [[1]] * 3}
+FORMS = [(F32, 0), (F16, 1), (F16, 2)]
+TOL = {F32: 2e-5, F16: 1e-2}
+
+
+@pytest.mark.parametrize("cut", CUTS)
+@pytest.mark.parametrize("shape", SHAPES, ids=str)
+@pytest.mark.parametrize("dtype,impl", FORMS)
+def test_against_plain_attention(shape, cut, dtype, impl):
+    s = Shape(*shape)
+    lens = (137, 67, 3) if cut != "single" else (70, 37, 3)
+    seqs, norm, U, sink = random_case(s, lens, s.rank)
+    got = run(s, seqs, CUTS[cut], norm, U, sink, dtype, impl)
+    for (q, kv), g in zip(seqs, got):
+        want = reference(s, q, kv, norm, U, sink)
+        assert np.abs(g - want).max() < TOL[dtype] * max(1, np.abs(want).max()), np.abs(g - want).max()
+
+
+@pytest.mark.parametrize("dtype,impl", FORMS)
+def test_parts_that_pass_unrotated_and_no_sink(dtype, impl):
+    s = Shape(4, 8, 12, 40, 30, rot_dims=6)
+    seqs, norm, U, _ = random_case(s, (90, 20), 3)
+    got = run(s, seqs, [[40, 1, 7], [3]], norm, U, None, dtype, impl)
+    for (q, kv), g in zip(seqs, got):
+        assert np.abs(g - reference(s, q, kv, norm, U, None)).max() < TOL[dtype] * 3
+
+
+@pytest.mark.parametrize("decoded", [False, True])
+@pytest.mark.parametrize("dtype,impl", FORMS)
+def test_a_key_that_stands_out_is_seen_up_to_the_windows_edge_and_not_beyond(dtype, impl, decoded):
+    """One query matches one key so strongly that it takes all the weight if it is visible: at page borders, just inside and just
+    outside the window, in the first tokens. Through the latent part and through the rotated part."""
+    n, window = 130, 40
+    s = Shape(4, 32, 8, 32, window)
+    U = np.tile(np.eye(32), (4, 1, 1))
+    rng = np.random.default_rng(5)
+    for key, query in [(0, 0), (0, 39), (0, 40), (15, 54), (15, 55), (16, 55), (16, 56), (47, 86), (48, 87), (48, 88), (90, 129), (89, 129), (31, 32), (60, 100)]:
+        for rotated in (False, True):
+            q = 0.02 * rng.standard_normal((n, 4, 40))
+            kv = np.concatenate([np.eye(32)[rng.integers(1, 32, n)], 0.02 * rng.standard_normal((n, 8))], axis=1)
+            kv[key, :32] = np.eye(32)[0]
+            if rotated:  # the query's rotated part is the key's turned by their distance, so that the score is its full length
+                kv[key, 32:] = 12 * np.array([1, 1, 1, 1, 0, 0, 0, 0])
+                q[query, :, 32:] = R.rotate(kv[key:key + 1, 32:], [key - query], 8, BASE)[0]
+            else:
+                q[query, :, 0] = 60
+            want = reference(s, q, kv, np.ones(32), U, np.zeros(4))
+            cuts = [[query, 1, 10 ** 9]] if decoded and query else [[10 ** 9]]
+            got = run(s, [(q, kv)], cuts, np.ones(32), U, np.zeros(4), dtype, impl)[0]
+            seen = query - key < window
+            assert (got[query, 0, 0] > 0.9 * np.sqrt(32)) == seen, (key, query, rotated)
+            assert np.abs(got - want).max() < (2e-5 if dtype == F32 else 2e-2)
+
+
+@pytest.mark.parametrize("dtype,impl", FORMS)
+@pytest.mark.parametrize("strength", [-200.0, 3.0, 40.0, 200.0])
+def test_the_sink_takes_its_share_once(dtype, impl, strength):
+    """From nothing to all of the weight, with keys in one share or in several (long prompts split their keys)."""
+    s = Shape(2, 16, 8, 32, 0)
+    seqs, norm, U, _ = random_case(s, (900,), 2)
+    sink = np.array([strength, -200.0])
+    q, kv = seqs[0]
+    got = run(s, seqs, [[898, 1, 1]], norm, U, sink, dtype, impl)[0]
+    want = reference(s, q, kv, norm, U, sink)
+    assert np.abs(got - want).max() < TOL[dtype] * 2
+    if strength > 100:
+        assert np.abs(got[:, 0]).max() < 1e-20
+
+
+@pytest.mark.parametrize("shape,n", [((16, 8, 16, 64, 0), 1500), ((7, 8, 8, 256, 900), 2000), ((32, 16, 64, 512, 700), 1100), ((128, 8, 8, 96, 300), 500)], ids=str)
+def test_decoding_over_many_keys(shape, n):
+    s = Shape(*shape)
+    seqs, norm, U, sink = random_case(s, (n, n // 3, 9), n)
+    got = run(s, seqs, [[n - 3, 1, 1, 1], [n // 3 - 3, 1, 1, 1], [6, 1, 1, 1]], norm, U, sink, F16, 0)
+    for (q, kv), g in zip(seqs, got):
+        want = reference(s, q, kv, norm, U, sink)
+        assert np.abs(g[-3:] - want[-3:]).max() < 1e-2 * max(1, np.abs(want).max())
+
+
+EXPANDED = [((3, 10, 6, 21, 19), 14), ((4, 128, 64, 512, 300), 128), ((2, 64, 64, 64, 0), 64), ((5, 100, 72, 48, 128), 80), ((2, 150, 30, 40, 1000), 100), ((7, 32, 32, 96, 72), 32),
+            ((1, 64, 8, 32, 1), 8)]
+
+
+@pytest.mark.parametrize("shape,vdim", EXPANDED, ids=str)
+@pytest.mark.parametrize("starts", [(0, 0, 0), (130, 1, 2), (650, 299, 0)], ids=str)
+def test_expanded_keys_on_tcgen05(shape, vdim, starts):
+    """Long portions on keys and values of their own: several row tiles, unequal sequences, portions that start anywhere in a window."""
+    s = Shape(*shape)
+    seqs, norm, U, sink = random_case(s, (700, 300, 5), vdim)
+    V = np.random.default_rng(1).standard_normal((s.heads, vdim, s.rank)) / s.rank ** 0.5
+    got = run_expanded(s, seqs, list(starts), norm, U, V, sink)
+    for (q, kv), p, g in zip(seqs, starts, got):
+        want = np.einsum("nhr,hvr->nhv", reference(s, q, kv, norm, U, sink), V)[p:]
+        assert np.abs(g - want).max() < 1.5e-2 * max(1, np.abs(want).max()), np.abs(g - want).max()
+
+
+@pytest.mark.parametrize("strength", [-200.0, 3.0, 200.0])
+def test_edges_and_sinks_on_expanded_keys(strength):
+    """Keys that stand out just inside and just outside the window, at tile borders, with sinks from nothing to everything."""
+    n, window = 420, 150
+    s = Shape(2, 32, 8, 32, window)
+    U = V = np.tile(np.eye(32), (2, 1, 1))
+    rng = np.random.default_rng(5)
+    pairs = [(0, 149), (1, 151), (127, 276), (128, 278), (130, 279), (255, 256), (256, 405), (100, 250), (269, 419), (17, 17)]
+    q = 0.02 * rng.standard_normal((n, 2, 40))
+    kv = np.concatenate([np.eye(32)[rng.integers(20, 32, n)], 0.02 * rng.standard_normal((n, 8))], axis=1)
+    for i, (key, query) in enumerate(pairs):  # every pair has a direction of its own
+        kv[key, :32] = np.eye(32)[i]
+        q[query, :, i] = 60
+    sink = np.array([strength, 0.0])
+    for start in (0, 16):
+        got = run_expanded(s, [(q, kv)], [start], np.ones(32), U, V, sink)[0]
+        want = reference(s, q, kv, np.ones(32), U, sink)[start:]
+        assert np.abs(got - want).max() < 2e-2
+        for i, (key, query) in enumerate(pairs):
+            if query >= start:
+                assert (got[query - start, 1, i] > 0.9 * np.sqrt(32)) == (query - key < window), (key, query)
+    if strength > 100:
+        assert np.abs(got[:, 0]).max() < 1e-20
+
+
+def test_angles_far_along():
+    """Positions in the hundred thousands: the angle is exact to a fraction of a turn, not to 32-bit turns."""
+    import torch
+    s = Shape(1, 8, 8, 16, 16)
+    pos, kv = 765432, np.concatenate([np.ones(16), np.arange(1.0, 9.0)])
+    h = C.c_void_p()
+    lib(lib().ingot_skv_create_window(C.byref(h), 1, 1, s.row, F32, 16, 2))
+    turns = dev(np.array([BASE ** (-2.0 * i / 8) / (2 * np.pi) for i in range(4)]), np.float64)
+    st, norm = Step([1], [pos], [0]), dev(np.ones(16))
+    proj = dev(np.concatenate([np.zeros(8), np.arange(1.0, 9.0), kv])[None])
+    rows, plain, tab, first = torch.zeros(1, s.row, device="cuda"), torch.zeros(1, 8, device="cuda"), dev([[1]], np.int32), dev([pos // 16], np.int32)
+    lib(lib().ingot_latent_append(h, 0, C.byref(st.c), proj.data_ptr(), proj.shape[1], 0, 16, C.byref(s.c), norm.data_ptr(), EPS, turns.data_ptr(),
+                                  C.byref(act_out(plain)), rows.data_ptr(), None, 0, 0, 0, tab.data_ptr(), first.data_ptr(), 1, None))
+    torch.cuda.synchronize()
+    want = R.rotate(np.arange(1.0, 9.0)[None], [pos], 8, BASE)[0]
+    assert np.abs(rows.cpu().numpy()[0, 16:24] - want).max() < 5e-6
+    lib().ingot_skv_destroy(h)
+
+
+def test_refusals():
+    h = C.c_void_p()
+    assert lib().ingot_skv_create_window(C.byref(h), 1, 1, 1028, F16, 8, 4) == 3
+    assert lib().ingot_skv_create_window(C.byref(h), 1, 1, 32, F16, -1, 4) == 1
+    lib(lib().ingot_skv_create_window(C.byref(h), 1, 1, 32, F16, 8, 4))
+    st, w = Step([1], [0], [0]), dev(np.zeros(64))
+    sh = CShape(1, 8, 8, 32, 32, 8)  # 32 + 8 does not fit a row of 32
+    assert lib().ingot_latent_append(h, 0, C.byref(st.c), w.data_ptr(), 64, 0, 16, C.byref(sh), w.data_ptr(), EPS, w.data_ptr(), C.byref(act_out(w)), None,
+                                     None, 0, 0, 0, w.data_ptr(), None, 1, None) == 1
+    assert lib().ingot_skv_append(h, 0, C.byref(st.c), w.data_ptr(), 64, 0, 32, 1, 32, w.data_ptr(), w.data_ptr(), EPS, w.data_ptr(), w.data_ptr(), None, 1, None) == 1
+    lib().ingot_skv_destroy(h)
