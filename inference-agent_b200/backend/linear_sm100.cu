@@ -411,8 +411,20 @@ __global__ void rmsnorm_split_kernel(__half* hi, __half* lo, const float* x, con
     LINEAR_PDL_WAIT();
     __shared__ float red[32];
     const float* xr = x + (size_t)blockIdx.x * n;
+    constexpr int kKeep = 4;  // float4s of the row a thread keeps between the two passes
+    float4 kept[kKeep];
     float ss = 0.f;
-    for (int i = threadIdx.x; i < n; i += blockDim.x) ss += xr[i] * xr[i];
+#pragma unroll
+    for (int k = 0; k < kKeep; k++) {
+        const int i = (threadIdx.x + k * blockDim.x) * 4;
+        kept[k] = i < n ? *reinterpret_cast<const float4*>(xr + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+    }
+#pragma unroll
+    for (int k = 0; k < kKeep; k++) { ss += kept[k].x * kept[k].x; ss += kept[k].y * kept[k].y; ss += kept[k].z * kept[k].z; ss += kept[k].w * kept[k].w; }
+    for (int i = (threadIdx.x + kKeep * blockDim.x) * 4; i < n; i += blockDim.x * 4) {
+        const float4 v = *reinterpret_cast<const float4*>(xr + i);
+        ss += v.x * v.x; ss += v.y * v.y; ss += v.z * v.z; ss += v.w * v.w;
+    }
 #pragma unroll
     for (int o = 16; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
     if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = ss;
@@ -425,11 +437,17 @@ __global__ void rmsnorm_split_kernel(__half* hi, __half* lo, const float* x, con
     }
     __syncthreads();
     const float scale = red[0];
-    for (int i = threadIdx.x * 4; i < n; i += blockDim.x * 4) {
-        const float4 v = *reinterpret_cast<const float4*>(xr + i), g = *reinterpret_cast<const float4*>(w + i);
+    auto put = [&](int i, const float4& v) {
+        const float4 g = *reinterpret_cast<const float4*>(w + i);
         const float f[4] = {v.x * scale * g.x, v.y * scale * g.y, v.z * scale * g.z, v.w * scale * g.w};
         store_split4<kAct>(hi, lo, (size_t)blockIdx.x * n + i, f);
+    };
+#pragma unroll
+    for (int k = 0; k < kKeep; k++) {
+        const int i = (threadIdx.x + k * blockDim.x) * 4;
+        if (i < n) put(i, kept[k]);
     }
+    for (int i = (threadIdx.x + kKeep * blockDim.x) * 4; i < n; i += blockDim.x * 4) put(i, *reinterpret_cast<const float4*>(xr + i));
 }
 
 // Consumers of k-slice partials [n_split][n_tok][n_out]: the sum over slices (always in slice order) is folded into

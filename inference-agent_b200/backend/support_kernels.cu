@@ -53,15 +53,37 @@ __global__ void rmsnorm_rows_kernel(float* out, const float* x, const float* w, 
     __shared__ float red[32];
     const float* xr = x + (size_t)(rows ? rows[blockIdx.x] : (int)blockIdx.x) * n;
     float* orow = out + (size_t)blockIdx.x * n;
+    constexpr int kKeep = 8;  // float4s of the row a thread keeps between the two passes
+    const int n4 = n % 4 == 0 ? n / 4 : 0;
+    float4 v[kKeep];
     float ss = 0.f;
-    for (int i = threadIdx.x; i < n; i += blockDim.x) ss += xr[i] * xr[i];
+    if (n4) {
+#pragma unroll
+        for (int k = 0; k < kKeep; k++) {
+            const int i = threadIdx.x + k * blockDim.x;
+            v[k] = i < n4 ? reinterpret_cast<const float4*>(xr)[i] : make_float4(0.f, 0.f, 0.f, 0.f);
+        }
+#pragma unroll
+        for (int k = 0; k < kKeep; k++) { ss += v[k].x * v[k].x; ss += v[k].y * v[k].y; ss += v[k].z * v[k].z; ss += v[k].w * v[k].w; }
+    }
+    const int kept = n4 ? min(n, kKeep * 4 * (int)blockDim.x) : 0;
+    for (int i = kept + threadIdx.x; i < n; i += blockDim.x) ss += xr[i] * xr[i];
     ss = warp_sum(ss);
     if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = ss;
     __syncthreads();
     float t = 0.f;
     for (int i = 0; i < (int)(blockDim.x >> 5); i++) t += red[i];
     const float scale = 1.0f / sqrtf(t / float(n_mean) + eps);
-    for (int i = threadIdx.x; i < n; i += blockDim.x) orow[i] = xr[i] * scale * w[i];
+    if (n4) {
+#pragma unroll
+        for (int k = 0; k < kKeep; k++) {
+            const int i = threadIdx.x + k * blockDim.x;
+            if (i >= n4) break;
+            const float4 g = reinterpret_cast<const float4*>(w)[i];
+            reinterpret_cast<float4*>(orow)[i] = make_float4(v[k].x * scale * g.x, v[k].y * scale * g.y, v[k].z * scale * g.z, v[k].w * scale * g.w);
+        }
+    }
+    for (int i = kept + threadIdx.x; i < n; i += blockDim.x) orow[i] = xr[i] * scale * w[i];
 }
 
 // Activation of gated feed-forwards: 0 silu, 1 the tanh form of gelu.

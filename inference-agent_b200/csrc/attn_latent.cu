@@ -30,7 +30,7 @@ __device__ __forceinline__ void put(__half* p, float v) { *p = __float2half_rn(f
 
 constexpr int kMaxRot = 512;  // rotated values per head
 
-// One CTA per token: the token's cache row, the rotated part of its query rows, and the unrotated query as operand of the
+// Per token one CTA for its cache row and one for every few heads: the rotated part of its query rows, and the unrotated query as operand of the
 // product that takes it into the latent space.
 struct AppendParams {
     ingot_step st;
@@ -43,7 +43,7 @@ struct AppendParams {
     SharedOut plain;      // [n_tok][n_head * dim]
     void* q_rows;         // [n_tok][n_head][row]; the rotated part is written
     __half* q_long;       // [n_tok][n_head][long_dim | long_rot] of the tokens from long_from on, instead of the two above
-    int long_from, long_dim, long_rot;
+    int long_from, long_dim, long_rot, heads_per_cta;
     void* rows;
     int row;
     const int32_t *tables, *first_page;
@@ -67,58 +67,65 @@ __global__ void __launch_bounds__(kAppendThreads) latent_append_kernel(const App
     INGOT_PDL_WAIT();
     const float* q = p.proj + (size_t)tok * p.proj_ld + p.q_off;
     const float* c = p.proj + (size_t)tok * p.proj_ld + p.latent_off;
-    float ss = 0.f;
-    for (int i = threadIdx.x; i < p.sh.rank; i += kAppendThreads) ss = fmaf(c[i], c[i], ss);
-    ss = warp_sum(ss);
-    const int warp = threadIdx.x >> 5;
-    if ((threadIdx.x & 31) == 0) red[warp] = ss;
-    __syncthreads();
-    ss = 0.f;
-#pragma unroll
-    for (int w = 0; w < kAppendThreads / 32; w++) ss += red[w];
-    const float inv = 1.0f / sqrtf(ss / float(p.sh.rank_count) + p.eps);
     // value i of a rotated part that starts at v
     auto rotated = [&](const float* v, int i) {
         if (i < half) return v[i] * s_cos[i] - v[i + half] * s_sin[i];
         if (i < 2 * half) return v[i] * s_cos[i - half] + v[i - half] * s_sin[i - half];
         return v[i];
     };
-    const int blk = table_block(p.tables, p.first_page, p.max_blocks, p.n_blocks, seq, p.map.page(pos), p.status);
-    if (blk >= 0) {
+    if (blockIdx.y == 0) {  // the cache row
+        float ss = 0.f;
+        for (int i = threadIdx.x; i < p.sh.rank; i += kAppendThreads) ss = fmaf(c[i], c[i], ss);
+        ss = warp_sum(ss);
+        const int warp = threadIdx.x >> 5;
+        if ((threadIdx.x & 31) == 0) red[warp] = ss;
+        __syncthreads();
+        ss = 0.f;
+#pragma unroll
+        for (int w = 0; w < kAppendThreads / 32; w++) ss += red[w];
+        const float inv = 1.0f / sqrtf(ss / float(p.sh.rank_count) + p.eps);
+        const int blk = table_block(p.tables, p.first_page, p.max_blocks, p.n_blocks, seq, p.map.page(pos), p.status);
+        if (blk < 0) return;
         T* dst = static_cast<T*>(p.rows) + ((size_t)blk * kBlockTokens + p.map.slot(pos)) * p.row;
         for (int i = threadIdx.x; i < p.sh.rank; i += kAppendThreads) put(dst + i, c[i] * inv * p.norm_w[i]);
         for (int i = threadIdx.x; i < p.sh.rot; i += kAppendThreads) put(dst + p.sh.rank + i, rotated(c + p.sh.rank, i));
+        return;
     }
-    const int per = p.sh.dim + p.sh.rot;
+    __syncthreads();  // the angles
+    // heads h0..h1-1, four values at a time
+    const int per = p.sh.dim + p.sh.rot, h0 = ((int)blockIdx.y - 1) * p.heads_per_cta, h1 = min(h0 + p.heads_per_cta, p.sh.n_head);
     if (tok >= p.long_from) {
-        const int width = p.long_dim + p.long_rot;
+        const int width = p.long_dim + p.long_rot, w4 = width / 4;
         __half* dst = p.q_long + (size_t)tok * p.sh.n_head * width;
-        for (int i = threadIdx.x * 2; i < p.sh.n_head * width; i += kAppendThreads * 2) {
-            const int h = i / width, d = i - h * width;
-            float v[2];
+        for (int i = threadIdx.x; i < (h1 - h0) * w4; i += kAppendThreads) {
+            const int h = h0 + i / w4, d = (i % w4) * 4, k = d - p.long_dim;
+            float v[4] = {0.f, 0.f, 0.f, 0.f};
+            if (k < 0) {
+                if (d < p.sh.dim) *reinterpret_cast<float4*>(v) = *reinterpret_cast<const float4*>(q + h * per + d);
+            } else if (k < p.sh.rot) {
 #pragma unroll
-            for (int e = 0; e < 2; e++) {
-                const int k = d + e - p.long_dim;
-                v[e] = k < 0 ? (d + e < p.sh.dim ? q[h * per + d + e] : 0.f) : k < p.sh.rot ? rotated(q + h * per + p.sh.dim, k) : 0.f;
+                for (int e = 0; e < 4; e++) v[e] = rotated(q + h * per + p.sh.dim, k + e);
             }
-            *reinterpret_cast<__half2*>(dst + i) = __floats2half2_rn(fminf(fmaxf(v[0], -65504.f), 65504.f), fminf(fmaxf(v[1], -65504.f), 65504.f));
+            __half o[4];
+#pragma unroll
+            for (int e = 0; e < 4; e++) put(o + e, v[e]);
+            *reinterpret_cast<uint2*>(dst + h * width + d) = *reinterpret_cast<const uint2*>(o);
         }
         return;
     }
-    if (p.plain.f32 || p.plain.hi) {
-        const int n4 = p.sh.n_head * p.sh.dim / 4, d4 = p.sh.dim / 4;
-        for (int i = threadIdx.x; i < n4; i += kAppendThreads) {
-            const int h = i / d4, d = (i - h * d4) * 4;
+    const int w4 = per / 4;
+    for (int i = threadIdx.x; i < (h1 - h0) * w4; i += kAppendThreads) {
+        const int h = h0 + i / w4, d = (i % w4) * 4, k = d - p.sh.dim;
+        if (k < 0) {
             const float4 v = *reinterpret_cast<const float4*>(q + h * per + d);
             p.plain.store2(tok, h * p.sh.dim + d, v.x, v.y);
             p.plain.store2(tok, h * p.sh.dim + d + 2, v.z, v.w);
+        } else if (p.q_rows) {
+            T* dst = static_cast<T*>(p.q_rows) + ((size_t)tok * p.sh.n_head + h) * p.row + p.sh.rank + k;
+#pragma unroll
+            for (int e = 0; e < 4; e++) put(dst + e, rotated(q + h * per + p.sh.dim, k + e));
         }
     }
-    if (p.q_rows)
-        for (int i = threadIdx.x; i < p.sh.n_head * p.sh.rot; i += kAppendThreads) {
-            const int h = i / p.sh.rot, d = i - h * p.sh.rot;
-            put(static_cast<T*>(p.q_rows) + ((size_t)tok * p.sh.n_head + h) * p.row + p.sh.rank + d, rotated(q + h * per + p.sh.dim, d));
-        }
 }
 
 // Latent queries f32 [n_tok][n_head * rank] into the query rows.
@@ -237,29 +244,55 @@ __global__ void __launch_bounds__(kLatThreads) latent_mma_kernel(const AttendPar
         for (int n = 0; n < kMT; n++) s[n][0] = s[n][1] = s[n][2] = s[n][3] = 0.f;
         {
             const uint32_t a_addr = s_base + L.q + (mi * 16 + (lane & 15)) * stride + (lane >> 4) * 16;
-            if (kMT == 1) {  // one 8-key tile: a load covers two k-steps
-                const uint32_t b_addr = tile + (kg * 8 + (lane & 7)) * stride + (lane >> 3) * 16;
-                for (int ks = 0; ks < p.dim / 16; ks += 2) {
-                    uint32_t a0[4], a1[4], b[4];
-                    ldmatrix4(a0, a_addr + ks * 32);
-                    ldmatrix4(a1, a_addr + ks * 32 + 32);
-                    ldmatrix4(b, b_addr + ks * 32);
-                    mma_16816(s[0], a0[0], a0[1], a0[2], a0[3], b[0], b[1]);
-                    mma_16816(s[0], a1[0], a1[1], a1[2], a1[3], b[2], b[3]);
-                }
-            } else {
-                const uint32_t b_addr = tile + (kg * 8 * kMT + (lane & 7) + ((lane >> 4) & 1) * 8) * stride + ((lane >> 3) & 1) * 16;
-                for (int ks = 0; ks < p.dim / 16; ks++) {
-                    uint32_t a[4];
-                    ldmatrix4(a, a_addr + ks * 32);
+            // Pairs of k-steps (the row length is a multiple of 32), the next pair's operands requested before this one is multiplied.
+            // With few score tiles per warp the two steps of a pair go to accumulators of their own: shorter chains of MMAs.
+            constexpr int kB = kMT == 1 ? 1 : kMT;  // operand loads per pair
+            const uint32_t b_addr = kMT == 1 ? tile + (kg * 8 + (lane & 7)) * stride + (lane >> 3) * 16
+                                             : tile + (kg * 8 * kMT + (lane & 7) + ((lane >> 4) & 1) * 8) * stride + ((lane >> 3) & 1) * 16;
+            auto load = [&](uint32_t (&a)[2][4], uint32_t (&b)[kB][4], int ks) {
+                ldmatrix4(a[0], a_addr + ks * 32);
+                ldmatrix4(a[1], a_addr + ks * 32 + 32);
+                if (kMT == 1) {  // one 8-key tile: a load covers both steps
+                    ldmatrix4(b[0], b_addr + ks * 32);
+                } else {
 #pragma unroll
-                    for (int n = 0; n + 1 < kMT; n += 2) {
-                        uint32_t b[4];
-                        ldmatrix4(b, b_addr + n * 8 * stride + ks * 32);
-                        mma_16816(s[n], a[0], a[1], a[2], a[3], b[0], b[1]);
-                        mma_16816(s[n + 1], a[0], a[1], a[2], a[3], b[2], b[3]);
+                    for (int n = 0; n < kMT / 2; n++) {
+                        ldmatrix4(b[2 * n], b_addr + n * 16 * stride + ks * 32);
+                        ldmatrix4(b[kB > 1 ? 2 * n + 1 : 0], b_addr + n * 16 * stride + ks * 32 + 32);
                     }
                 }
+            };
+            float s2[kMT <= 2 ? kMT : 1][4];
+#pragma unroll
+            for (int n = 0; n < (kMT <= 2 ? kMT : 1); n++) s2[n][0] = s2[n][1] = s2[n][2] = s2[n][3] = 0.f;
+            auto multiply = [&](const uint32_t (&a)[2][4], const uint32_t (&b)[kB][4]) {
+                if (kMT == 1) {
+                    mma_16816(s[0], a[0][0], a[0][1], a[0][2], a[0][3], b[0][0], b[0][1]);
+                    mma_16816(s2[0], a[1][0], a[1][1], a[1][2], a[1][3], b[0][2], b[0][3]);
+                } else {
+#pragma unroll
+                    for (int h = 0; h < 2; h++)
+#pragma unroll
+                        for (int n = 0; n < kMT; n++) {
+                            const uint32_t* t = b[kB > 1 ? (n & ~1) + h : 0];
+                            mma_16816(kMT == 2 && h ? s2[kMT == 2 ? n : 0] : s[n], a[h][0], a[h][1], a[h][2], a[h][3], t[(n & 1) * 2], t[(n & 1) * 2 + 1]);
+                        }
+                }
+            };
+            uint32_t a0[2][4], b0[kB][4], a1[2][4], b1[kB][4];
+            const int steps = p.dim / 16;
+            load(a0, b0, 0);
+            for (int ks = 0; ks < steps; ks += 4) {
+                if (ks + 2 < steps) load(a1, b1, ks + 2);
+                multiply(a0, b0);
+                if (ks + 4 < steps) load(a0, b0, ks + 4);
+                if (ks + 2 < steps) multiply(a1, b1);
+            }
+            if (kMT <= 2) {
+#pragma unroll
+                for (int n = 0; n < (kMT <= 2 ? kMT : 1); n++)
+#pragma unroll
+                    for (int e = 0; e < 4; e++) s[n][e] += s2[n][e];
             }
         }
         float mx_lo = -INFINITY, mx_hi = -INFINITY;
@@ -395,28 +428,32 @@ __global__ void __launch_bounds__(kLatThreads) latent_mma_kernel(const AttendPar
 }
 
 // out = sum_s o_s 2^(m_s - M) / (sum_s l_s 2^(m_s - M) + 2^(sink - M)) over the splits of one (token, head)
-constexpr int kMergeThreads = 128, kMaxSplits = 64;
+constexpr int kMergeThreads = 256, kMaxSplits = 64;
 __global__ void __launch_bounds__(kMergeThreads) latent_merge_kernel(const AttendParams p) {
     INGOT_PDL_TRIGGER();
     INGOT_PDL_WAIT();
-    __shared__ float s_f[kMaxSplits];
+    __shared__ float s_f[kMaxSplits], s_m[kMaxSplits], s_l[kMaxSplits];
     const int h = blockIdx.x;
     const size_t tok = blockIdx.y;
     const int ld = p.out_dim + 2;
     const float* part = p.part + (tok * p.n_head + h) * p.n_splits * ld;
-    float top = p.sink ? p.sink[h] * 1.44269504f : -INFINITY;
-    const float sink = top;
-    for (int s = 0; s < p.n_splits; s++) top = fmaxf(top, part[s * ld + p.out_dim]);
-    float l = p.sink ? exp2f(sink - top) : 0.f;
-    for (int s = 0; s < p.n_splits; s++) {
-        const float f = exp2f(part[s * ld + p.out_dim] - top);
-        l = fmaf(f, part[s * ld + p.out_dim + 1], l);
-        if (threadIdx.x == 0) s_f[s] = f;
+    const float sink = p.sink ? p.sink[h] * 1.44269504f : -INFINITY;
+    if (threadIdx.x < p.n_splits) {
+        const float2 ml = *reinterpret_cast<const float2*>(part + threadIdx.x * ld + p.out_dim);
+        s_m[threadIdx.x] = ml.x;
+        s_l[threadIdx.x] = ml.y;
     }
     __syncthreads();
+    float top = sink;
+    for (int s = 0; s < p.n_splits; s++) top = fmaxf(top, s_m[s]);
+    if (threadIdx.x < p.n_splits) s_f[threadIdx.x] = exp2f(s_m[threadIdx.x] - top);
+    __syncthreads();
+    float l = p.sink ? exp2f(sink - top) : 0.f;
+    for (int s = 0; s < p.n_splits; s++) l = fmaf(s_f[s], s_l[s], l);
     const float inv = 1.0f / l;
     for (int d = threadIdx.x * 2; d < p.out_dim; d += kMergeThreads * 2) {
         float a = 0.f, b = 0.f;
+#pragma unroll 8
         for (int s = 0; s < p.n_splits; s++) {
             const float2 v = *reinterpret_cast<const float2*>(part + s * ld + d);
             a = fmaf(s_f[s], v.x, a);
@@ -490,24 +527,25 @@ int ingot_latent_append(ingot_skv* kv, int layer, const ingot_step* step, const 
     INGOT_REQUIRE(layer >= 0 && layer < kv->n_layer, "ingot_latent_append: layer out of range");
     INGOT_REQUIRE(proj_dev && norm_dev && q_plain && tables_dev && max_blocks >= 1 && (turns_dev || shape->rot_dims == 0), "ingot_latent_append: null argument");
     const ingot_latent_shape& sh = *shape;
-    INGOT_REQUIRE(sh.n_head >= 1 && sh.dim >= 0 && sh.dim % 4 == 0 && sh.rank >= 1 && sh.rank_count >= 1 && sh.rank_count <= sh.rank && sh.rot >= 0 &&
+    INGOT_REQUIRE(sh.n_head >= 1 && sh.dim >= 0 && sh.dim % 4 == 0 && sh.rot % 4 == 0 && sh.rank >= 1 && sh.rank_count >= 1 && sh.rank_count <= sh.rank && sh.rot >= 0 &&
                       sh.rot_dims >= 0 && sh.rot_dims % 2 == 0 && sh.rot_dims <= sh.rot && sh.rank + sh.rot <= kv->dim,
                   "ingot_latent_append: bad shape");
-    INGOT_REQUIRE(proj_ld % 4 == 0 && q_off % 4 == 0 && (sh.dim + sh.rot) % 4 == 0 && q_plain->ld % 2 == 0, "ingot_latent_append: rows and offsets must be multiples of 4 floats");
+    INGOT_REQUIRE(proj_ld % 4 == 0 && q_off % 4 == 0 && q_plain->ld % 2 == 0, "ingot_latent_append: rows and offsets must be multiples of 4 floats");
     if (sh.rot_dims > kMaxRot || kv->n_head_kv != 1 || kv->inv_rms) {
         ingot_set_error("ingot_latent_append: needs a window-form cache with one row per token and at most " + std::to_string(kMaxRot) + " rotated values");
         return INGOT_ERR_UNSUPPORTED;
     }
-    INGOT_REQUIRE(!q_long_dev || (kv->dtype == INGOT_F16 && long_from >= 0 && long_dim % 2 == 0 && long_rot % 2 == 0 && long_dim >= sh.dim && long_rot >= sh.rot),
+    INGOT_REQUIRE(!q_long_dev || (kv->dtype == INGOT_F16 && long_from >= 0 && long_dim % 4 == 0 && long_rot % 4 == 0 && long_dim >= sh.dim && long_rot >= sh.rot),
                   "ingot_latent_append: bad long queries");
     const size_t esz = kv->dtype == INGOT_F32 ? 4 : 2;
+    const int heads_per_cta = step->n_tok >= 512 ? 16 : 8;
     AppendParams p = {*step, proj_dev, proj_ld, q_off, latent_off, sh, norm_dev, eps, turns_dev,
                       SharedOut{q_plain->f32, static_cast<__nv_bfloat16*>(q_plain->hi), static_cast<__nv_bfloat16*>(q_plain->lo), q_plain->ld, 1.0f}, q_rows_dev,
-                      static_cast<__half*>(q_long_dev), q_long_dev ? long_from : 0x7fffffff, long_dim, long_rot,
+                      static_cast<__half*>(q_long_dev), q_long_dev ? long_from : 0x7fffffff, long_dim, long_rot, heads_per_cta,
                       static_cast<char*>(kv->rows) + kv->layer_elems * layer * esz, kv->dim, tables_dev, first_page_dev, max_blocks, kv->n_blocks, page_map(kv),
                       kv->status_dev};
     auto kernel = kv->dtype == INGOT_F32 ? latent_append_kernel<float> : latent_append_kernel<__half>;
-    INGOT_CUDA_TRY(ingot_launch_pdl(kernel, dim3(step->n_tok), dim3(kAppendThreads), 0, static_cast<cudaStream_t>(stream), p));
+    INGOT_CUDA_TRY(ingot_launch_pdl(kernel, dim3(step->n_tok, 1 + (sh.n_head + heads_per_cta - 1) / heads_per_cta), dim3(kAppendThreads), 0, static_cast<cudaStream_t>(stream), p));
     return INGOT_OK;
 }
 

@@ -46,50 +46,58 @@ __global__ void __launch_bounds__(128) moe_select_kernel(const float* logits, in
     }
 }
 
-// One CTA per expert: where its rows start (pairs of lower experts), then its pairs in order.
-constexpr int kSortThreads = 512;
+// One CTA per expert: where its rows start (pairs of lower experts), then its pairs in order. A thread owns a run of pairs, so one scan
+// over the threads' counts places them all.
+constexpr int kSortThreads = 1024;
 __global__ void __launch_bounds__(kSortThreads) moe_sort_kernel(const int32_t* expert_of, const float* weight_of, int n_pairs, int n_expert, int32_t* group_start,
                                                                 int32_t* row_of, int32_t* pair_of, float* row_weight) {
     INGOT_PDL_TRIGGER();
     INGOT_PDL_WAIT();
-    __shared__ int s_warp[kSortThreads / 32];
-    __shared__ int s_base;
+    __shared__ int s_lower[kSortThreads / 32], s_mine[kSortThreads / 32];
     const int e = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    int lower = 0;
-    for (int i = threadIdx.x; i < n_pairs; i += kSortThreads) lower += expert_of[i] < e;
+    const int run = ((n_pairs + kSortThreads - 1) / kSortThreads + 3) / 4 * 4, first = min((int)threadIdx.x * run, n_pairs), last = min(first + run, n_pairs);
+    int lower = 0, mine = 0;
+    for (int i = first; i < last; i += 4) {
+        int v[4];
+        if (i + 4 <= last) {
+            *reinterpret_cast<int4*>(v) = *reinterpret_cast<const int4*>(expert_of + i);
+        } else {
+            for (int k = 0; k < 4; k++) v[k] = i + k < last ? expert_of[i + k] : 0x7fffffff;
+        }
+#pragma unroll
+        for (int k = 0; k < 4; k++) {
+            lower += v[k] < e;
+            mine += v[k] == e;
+        }
+    }
+    int upto = mine;  // within the warp, then over the warps
+#pragma unroll
+    for (int o = 1; o < 32; o <<= 1) {
+        const int v = __shfl_up_sync(0xffffffffu, upto, o);
+        if (lane >= o) upto += v;
+    }
 #pragma unroll
     for (int o = 16; o > 0; o >>= 1) lower += __shfl_xor_sync(0xffffffffu, lower, o);
-    if (lane == 0) s_warp[warp] = lower;
+    if (lane == 31) s_mine[warp] = upto;
+    if (lane == 0) s_lower[warp] = lower;
     __syncthreads();
+    int row = upto - mine;
+    for (int w = 0; w < kSortThreads / 32; w++) {
+        row += s_lower[w];
+        if (w < warp) row += s_mine[w];
+    }
     if (threadIdx.x == 0) {
-        int sum = 0;
-        for (int w = 0; w < kSortThreads / 32; w++) sum += s_warp[w];
-        s_base = sum;
-        group_start[e] = sum;
+        group_start[e] = row;
         if (e == n_expert - 1) group_start[n_expert] = n_pairs;
     }
-    __syncthreads();
-    for (int i0 = 0; i0 < n_pairs; i0 += kSortThreads) {
-        const int i = i0 + threadIdx.x;
-        const bool mine = i < n_pairs && expert_of[i] == e;
-        const unsigned votes = __ballot_sync(0xffffffffu, mine);
-        if (lane == 0) s_warp[warp] = __popc(votes);
-        __syncthreads();
-        int before = s_base, all = 0;
-        for (int w = 0; w < kSortThreads / 32; w++) {
-            if (w < warp) before += s_warp[w];
-            all += s_warp[w];
+    if (mine == 0) return;
+    for (int i = first; i < last; i++)
+        if (expert_of[i] == e) {
+            row_of[i] = row;
+            pair_of[row] = i;
+            row_weight[row] = weight_of[i];
+            row++;
         }
-        if (mine) {
-            const int r = before + __popc(votes & ((1u << lane) - 1));
-            row_of[i] = r;
-            pair_of[r] = i;
-            row_weight[r] = weight_of[i];
-        }
-        __syncthreads();
-        if (threadIdx.x == 0) s_base += all;
-        __syncthreads();
-    }
 }
 
 // bf16 planes of the rows: row r is its token's row.
@@ -178,6 +186,76 @@ __global__ void __launch_bounds__(256) moe_linear_kernel(float* out, const __nv_
     }
 }
 
+// The same for the few rows of one token, bound by streaming the weights: a warp owns two outputs of one row and keeps eight 16-byte
+// weight loads in flight while it multiplies the eight before; the row's x is read once for both.
+constexpr int kGemvLoads = 4;
+__global__ void __launch_bounds__(256) moe_gemv_kernel(float* out, const __nv_bfloat16* w, const float* x, int x_ld, int n_in, int n_out, const int32_t* group_start,
+                                                       int n_expert, const int32_t* pair_of, int top, const float* row_weight, int act) {
+    INGOT_PDL_TRIGGER();
+    INGOT_PDL_WAIT();
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, row = blockIdx.y;
+    int e = 0;  // the expert whose run holds this row: runs start in ascending order
+    for (int e0 = 0; e0 < n_expert; e0 += 32) {
+        const bool past = e0 + lane < n_expert && group_start[e0 + lane + 1] <= row;
+        e += __popc(__ballot_sync(0xffffffffu, past));
+    }
+    const int o = (blockIdx.x * 8 + warp) * 2;
+    if (o >= n_out || e >= n_expert) return;
+    const bool two = o + 1 < n_out;
+    const uint4* wa = reinterpret_cast<const uint4*>(w + ((size_t)e * n_out + o) * n_in);
+    const uint4* wb = two ? wa + n_in / 8 : wa;
+    const float* xr = x + (size_t)(pair_of ? pair_of[row] / top : row) * x_ld;
+    const int n8 = n_in / 8;
+    const uint4 zero = make_uint4(0, 0, 0, 0);
+    uint4 a[2][kGemvLoads], b[2][kGemvLoads];
+    auto request = [&](uint4 (&u)[kGemvLoads], uint4 (&v)[kGemvLoads], int c0) {
+#pragma unroll
+        for (int k = 0; k < kGemvLoads; k++) {
+            const int c = c0 + k * 32 + lane;
+            u[k] = c < n8 ? __ldcs(wa + c) : zero;
+            v[k] = c < n8 ? __ldcs(wb + c) : zero;
+        }
+    };
+    float acc_a = 0.f, acc_b = 0.f;
+    auto dot = [](const uint4& raw, const float4& p, const float4& q, float acc) {
+        acc = fmaf(__uint_as_float(raw.x << 16), p.x, acc); acc = fmaf(__uint_as_float(raw.x & 0xffff0000u), p.y, acc);
+        acc = fmaf(__uint_as_float(raw.y << 16), p.z, acc); acc = fmaf(__uint_as_float(raw.y & 0xffff0000u), p.w, acc);
+        acc = fmaf(__uint_as_float(raw.z << 16), q.x, acc); acc = fmaf(__uint_as_float(raw.z & 0xffff0000u), q.y, acc);
+        acc = fmaf(__uint_as_float(raw.w << 16), q.z, acc); return fmaf(__uint_as_float(raw.w & 0xffff0000u), q.w, acc);
+    };
+    auto consume = [&](const uint4 (&u)[kGemvLoads], const uint4 (&v)[kGemvLoads], int c0) {
+#pragma unroll
+        for (int k = 0; k < kGemvLoads; k++) {
+            const int c = c0 + k * 32 + lane;
+            if (c >= n8) break;
+            const float4 p = *reinterpret_cast<const float4*>(xr + c * 8), q = *reinterpret_cast<const float4*>(xr + c * 8 + 4);
+            acc_a = dot(u[k], p, q, acc_a);
+            acc_b = dot(v[k], p, q, acc_b);
+        }
+    };
+    constexpr int kStep = kGemvLoads * 32;
+    request(a[0], b[0], 0);
+    for (int c = 0; c < n8; c += 2 * kStep) {
+        request(a[1], b[1], c + kStep);
+        consume(a[0], b[0], c);
+        request(a[0], b[0], c + 2 * kStep);
+        consume(a[1], b[1], c + kStep);
+    }
+    acc_a = warp_sum(acc_a);
+    acc_b = warp_sum(acc_b);
+    if (lane == 0) {
+        const float f = row_weight ? row_weight[row] : 1.0f;
+        acc_a *= f;
+        acc_b *= f;
+        if (act == INGOT_ACT_RELU2) {
+            acc_a = acc_a > 0.f ? acc_a * acc_a : 0.f;
+            acc_b = acc_b > 0.f ? acc_b * acc_b : 0.f;
+        }
+        out[(size_t)row * n_out + o] = acc_a;
+        if (two) out[(size_t)row * n_out + o + 1] = acc_b;
+    }
+}
+
 // x[t] += sum over the token's pairs of rows[row_of[pair]]; row_of null: rows[t]
 __global__ void moe_add_kernel(float* x, const float* rows, const int32_t* row_of, int top, int n4) {
     INGOT_PDL_TRIGGER();
@@ -220,6 +298,11 @@ int ingot_moe_linear(float* out_dev, const void* w_dev, const float* x_dev, int 
                      const int32_t* pair_of_dev, int top, const float* row_weight_dev, int act, void* stream) {
     INGOT_REQUIRE(out_dev && w_dev && x_dev && group_start_dev, "ingot_moe_linear: null argument");
     INGOT_REQUIRE(n_in >= 8 && n_in % 8 == 0 && x_ld % 4 == 0 && n_out >= 1 && n_expert >= 1 && n_rows >= 1 && top >= 1, "ingot_moe_linear: bad sizes");
+    if (n_rows <= 2 * top) {  // one token (or two): a row per expert, as good as always
+        INGOT_CUDA_TRY(ingot_launch_pdl(moe_gemv_kernel, dim3((n_out + 15) / 16, n_rows), dim3(256), 0, static_cast<cudaStream_t>(stream), out_dev,
+                                        static_cast<const __nv_bfloat16*>(w_dev), x_dev, x_ld, n_in, n_out, group_start_dev, n_expert, pair_of_dev, top, row_weight_dev, act));
+        return INGOT_OK;
+    }
     const int tiles = n_rows / kRowTile + (n_rows < n_expert ? n_rows : n_expert);  // at least as many as there can be
     INGOT_REQUIRE(tiles <= 65535, "ingot_moe_linear: too many rows");
     INGOT_CUDA_TRY(ingot_launch_pdl(moe_linear_kernel, dim3((n_out + 7) / 8, tiles), dim3(256), 0, static_cast<cudaStream_t>(stream), out_dev,

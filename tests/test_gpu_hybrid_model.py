@@ -29,7 +29,7 @@ CONFIGS = {
                        vocab=103, width=46, loop=(1, 3, 2), bigram=(37, 31, 7)),
     # every expert is chosen (nothing hangs on a close choice), one head, a window of one page, a loop over all layers, no bigrams
     "latent_all": L.config([L.layer(1, 24, 16, 40, 64, 16, experts=2, top=2, ff=40), L.layer(20, 16, 2, 8, 40, 100, scale=0.15, experts=1, top=1, ff=8)],
-                           vocab=90, width=64, loop=(0, 2, 3), softcap=4.0),
+                           vocab=90, width=64, loop=(0, 2, 2), softcap=5.0),
     # rows longer than a tensor-core tile, no loop, many experts, some of them idle
     "latent_long": L.config([L.layer(4, 64, 32, 48, 150, 70, scale=0.1, experts=40, top=6, ff=33), L.layer(33, 8, 8, 8, 72, 1, experts=33, top=2, ff=16)],
                             vocab=130, width=130, bigram=(64, 3, 1)),
