@@ -32,7 +32,9 @@ public:
         shape_.rank = latent.padded;
         shape_.rank_count = rank;
         shape_.rot_dims = rot_dims;
-        row_ = round_up(shape_.rank + shape_.rot, 32);
+        // rows of whole 64-column units that hold the latent in whole blocks of 128 suit the tcgen05 kernel of decoded tokens
+        const int least = shape_.rank + shape_.rot, wide = round_up(std::max(least, round_up(rank, 128)), 64);
+        row_ = !ops.opt.f32 && rank <= 512 && wide * 3 <= least * 4 ? wide : round_up(least, 32);
         if (row_ > 1024) throw std::runtime_error("model config: latent rows of more than 1024 values are not supported");
         cache_ = ops.cache_group(1, row_, 0, window, false, &cache_layer_);
 

@@ -143,7 +143,7 @@ __global__ void latent_queries_kernel(T* q_rows, const float* q, int rank, int r
     put(o, v.x); put(o + 1, v.y); put(o + 2, v.z); put(o + 3, v.w);
 }
 
-// ---- tensor-core form on the rows: f16, m16n8k16 MMAs -------------------------------------------------------------------
+// ---- tensor-core form on the rows: f16, m16n8k16 MMAs; single tokens have a tcgen05 form (attn_latent_decode_sm100.cu) -------------------------------------------------------------------
 // A CTA owns 16 kMT rows - (token, head) pairs, token-major - of one sequence and one share of the keys they see, in tiles of 64
 // keys = 4 pages. The rows are long (a latent and a rotated part), so neither the queries nor the result of a tile of rows fits one
 // warp's registers; the 8 warps therefore share the work in two ways:
@@ -472,6 +472,24 @@ constexpr int kSmemLimit = 227 * 1024;
 
 bool mma_takes(int dim, int dv) { return dim % 32 == 0 && dv % 16 == 0 && dv <= 512 && LatentSmem(1, dim).bytes <= kSmemLimit; }
 
+int make_room(ingot_skv* kv, AttendParams& p) {  // for the partial results of several shares
+    if (p.n_splits <= 1) return INGOT_OK;
+    const size_t need = (size_t)p.st.n_tok * p.n_head * p.n_splits * (p.out_dim + 2);
+    if (need > kv->part_floats) {
+        float* fresh = nullptr;
+        INGOT_CUDA_TRY(cudaMalloc(&fresh, need * sizeof(float)));
+        if (kv->part) kv->retired.push_back(kv->part);  // a captured graph may still point into it
+        kv->part = fresh;
+        kv->part_floats = need;
+    }
+    p.part = kv->part;
+    return INGOT_OK;
+}
+int merge(const AttendParams& p, cudaStream_t s) {
+    if (p.n_splits > 1) INGOT_CUDA_TRY(ingot_launch_pdl(latent_merge_kernel, dim3(p.n_head, p.st.n_tok), dim3(kMergeThreads), 0, s, p));
+    return INGOT_OK;
+}
+
 int launch_mma(ingot_skv* kv, AttendParams p, cudaStream_t s) {
     const int rows = p.st.max_len * p.n_head;
     int mt = rows <= 16 ? 1 : rows <= 32 ? 2 : 4;
@@ -494,20 +512,25 @@ int launch_mma(ingot_skv* kv, AttendParams p, cudaStream_t s) {
     }
     p.n_splits = std::max(p.n_splits, (max_pages + kMaxSharePages - 8) / (kMaxSharePages - 7));
     if (p.n_splits > kMaxSplits) return launch_shared_kv_plain(p, INGOT_F16, s);
-    if (p.n_splits > 1) {
-        const size_t need = (size_t)p.st.n_tok * p.n_head * p.n_splits * (p.out_dim + 2);
-        if (need > kv->part_floats) {
-            float* fresh = nullptr;
-            INGOT_CUDA_TRY(cudaMalloc(&fresh, need * sizeof(float)));
-            if (kv->part) kv->retired.push_back(kv->part);  // a captured graph may still point into it
-            kv->part = fresh;
-            kv->part_floats = need;
-        }
-        p.part = kv->part;
-    }
+    if (const int rc = make_room(kv, p)) return rc;
     INGOT_CUDA_TRY(ingot_launch_pdl(kernel, dim3(row_tiles, p.n_splits, p.st.n_seq), dim3(kLatThreads), size_t(smem), s, p));
-    if (p.n_splits > 1) INGOT_CUDA_TRY(ingot_launch_pdl(latent_merge_kernel, dim3(p.n_head, p.st.n_tok), dim3(kMergeThreads), 0, s, p));
-    return INGOT_OK;
+    return merge(p, s);
+}
+
+// Single tokens on tcgen05. A share of the keys costs its tiles and about one tile more; several shares cost a merge.
+int launch_decode(ingot_skv* kv, int layer, AttendParams p, cudaStream_t s) {
+    constexpr int kDecodeTile = 128;
+    const int keys = p.map.window > 0 ? std::min(p.max_blocks * kBlockTokens, p.map.window + kBlockTokens) : p.max_blocks * kBlockTokens;
+    const int tiles = (keys + kDecodeTile - 1) / kDecodeTile, heads = latent_decode_heads(p.n_head);
+    const long long ctas = (long long)((p.n_head + heads - 1) / heads) * p.st.n_seq;
+    long long best = -1;
+    for (int n = 1; n <= std::min(kMaxSplits, tiles); n++) {
+        const long long cost = (ctas * n + kv->num_sms - 1) / kv->num_sms * ((tiles + n - 1) / n + 1) * 32 + (n > 1 ? 24 + n : 0);
+        if (best < 0 || cost < best) { best = cost; p.n_splits = n; }
+    }
+    if (const int rc = make_room(kv, p)) return rc;
+    if (const int rc = launch_latent_decode_sm100(kv, layer, p, s)) return rc;
+    return merge(p, s);
 }
 
 bool step_ok(const ingot_step* st) {
@@ -573,9 +596,13 @@ int ingot_latent_attend(ingot_skv* kv, int layer, const ingot_step* step, const 
                       SharedOut{out->f32, static_cast<__nv_bfloat16*>(out->hi), static_cast<__nv_bfloat16*>(out->lo), out->ld, 1.0f}, kv->status_dev, 1, nullptr,
                       sink_dev};
     cudaStream_t s = static_cast<cudaStream_t>(stream);
-    if (kv->dtype == INGOT_F16 && impl != 1 && mma_takes(kv->dim, rank) && out->ld % 2 == 0) return launch_mma(kv, p, s);
-    if (impl == 2) {
-        ingot_set_error("ingot_latent_attend: the tensor-core kernel does not take this row length");
+    if (kv->dtype == INGOT_F16 && (impl == 0 || impl == 3) && step->max_len == 1 && latent_decode_takes(kv->dim, rank)) {
+        const int rc = launch_decode(kv, layer, p, s);
+        if (rc != INGOT_ERR_UNSUPPORTED || impl == 3) return rc;
+    }
+    if (kv->dtype == INGOT_F16 && impl != 1 && impl != 3 && mma_takes(kv->dim, rank) && out->ld % 2 == 0) return launch_mma(kv, p, s);
+    if (impl == 2 || impl == 3) {
+        ingot_set_error("ingot_latent_attend: the tensor-core kernel does not take this row length, latent or step");
         return INGOT_ERR_UNSUPPORTED;
     }
     return launch_shared_kv_plain(p, kv->dtype, s);

@@ -90,6 +90,12 @@ struct AttendParams {
 // The plain kernel (f32 arithmetic, any row length up to 1024, window, chunk and sink); dtype of rows and queries.
 int launch_shared_kv_plain(const AttendParams& p, int dtype, cudaStream_t stream);
 
+// Latent attention of decoded tokens on tcgen05 (attn_latent_decode_sm100.cu): which rows it takes, heads per CTA, and the launch for
+// a step of single tokens (p.n_splits and p.part set).
+bool latent_decode_takes(int row, int rank);
+int latent_decode_heads(int n_head);
+int launch_latent_decode_sm100(ingot_skv* kv, int layer, const AttendParams& p, cudaStream_t stream);
+
 // tcgen05 form for portions of prompts over rows of 128 values (attn_shared_kv_sm100.cu); INGOT_ERR_UNSUPPORTED if the driver
 // cannot encode its tensor map.
 int launch_shared_kv_sm100(ingot_skv* kv, int layer, const AttendParams& p, cudaStream_t stream);

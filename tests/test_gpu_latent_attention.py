@@ -18,12 +18,12 @@ class CShape(C.Structure):
 
 
 class Shape:
-    def __init__(self, heads, dim, rot, rank, window, rot_dims=None):
+    def __init__(self, heads, dim, rot, rank, window, rot_dims=None, wide=False):
         self.heads, self.dim, self.rot, self.rank, self.window = heads, dim, rot, rank, window
         self.rot_dims = rot if rot_dims is None else rot_dims
         up = lambda v, q: (v + q - 1) // q * q
         self.dim_p, self.rot_p, self.rank_p = up(dim, 8), up(rot, 8), up(rank, 16)
-        self.row = up(self.rank_p + self.rot_p, 32)
+        self.row = up(max(self.rank_p + self.rot_p, up(rank, 128)), 64) if wide else up(self.rank_p + self.rot_p, 32)
         self.c = CShape(heads, self.dim_p, self.rot_p, self.rank_p, rank, self.rot_dims)
         self.scale = 1.3 / (dim + rot) ** 0.5
 
@@ -91,7 +91,7 @@ def run(s, seqs, cuts, norm, U, sink, dtype, impl, seed=0, tables_seen_only=True
             qd = dev(ql.reshape(n_tok, -1))
             lib(lib().ingot_latent_queries(h, qd.data_ptr(), n_tok, s.heads, s.rank_p, rows.data_ptr(), None))
             lib(lib().ingot_latent_attend(h, 0, C.byref(st.c), rows.data_ptr(), s.heads, s.rank_p, s.scale, None if sink is None else sink_d.data_ptr(),
-                                          C.byref(oo), td.data_ptr(), fd.data_ptr(), width, impl, None))
+                                          C.byref(oo), td.data_ptr(), fd.data_ptr(), width, impl if impl != 3 or max(part) == 1 else 2, None))
             torch.cuda.synchronize()
             status = C.c_int(-1)
             lib(lib().ingot_skv_status(h, None, C.byref(status)))
@@ -193,6 +193,7 @@ SHAPES = [(3, 10, 6, 21, 19), (16, 16, 16, 48, 40), (20, 8, 4, 64, 0), (5, 24, 4
           (70, 8, 64, 512, 48)]
 CUTS = {"whole": [[10 ** 9]] * 3, "portions": [[70, 2, 33, 16], [5, 64], [2]], "single": [[1]] * 3}
 FORMS = [(F32, 0), (F16, 1), (F16, 2)]
+ALL_FORMS = FORMS + [(F16, 3)]  # 3: tcgen05, single tokens only
 TOL = {F32: 2e-5, F16: 1e-2}
 
 
@@ -209,6 +210,17 @@ def test_against_plain_attention(shape, cut, dtype, impl):
         assert np.abs(g - want).max() < TOL[dtype] * max(1, np.abs(want).max()), np.abs(g - want).max()
 
 
+@pytest.mark.parametrize("shape", SHAPES, ids=str)
+def test_single_tokens_on_tcgen05(shape):
+    """Token by token, unequal sequences: every length of the last tile and page, from the first token on."""
+    s = Shape(*shape, wide=True)
+    seqs, norm, U, sink = random_case(s, (300, 150, 40), s.rank + 1)
+    got = run(s, seqs, [[1], [30, 1, 1, 1, 1, 1], [1]], norm, U, sink, F16, 3)
+    for (q, kv), g in zip(seqs, got):
+        want = reference(s, q, kv, norm, U, sink)
+        assert np.abs(g - want).max() < TOL[F16] * max(1, np.abs(want).max()), np.abs(g - want).max()
+
+
 @pytest.mark.parametrize("dtype,impl", FORMS)
 def test_parts_that_pass_unrotated_and_no_sink(dtype, impl):
     s = Shape(4, 8, 12, 40, 30, rot_dims=6)
@@ -219,12 +231,12 @@ def test_parts_that_pass_unrotated_and_no_sink(dtype, impl):
 
 
 @pytest.mark.parametrize("decoded", [False, True])
-@pytest.mark.parametrize("dtype,impl", FORMS)
+@pytest.mark.parametrize("dtype,impl", ALL_FORMS)
 def test_a_key_that_stands_out_is_seen_up_to_the_windows_edge_and_not_beyond(dtype, impl, decoded):
     """One query matches one key so strongly that it takes all the weight if it is visible: at page borders, just inside and just
     outside the window, in the first tokens. Through the latent part and through the rotated part."""
     n, window = 130, 40
-    s = Shape(4, 32, 8, 32, window)
+    s = Shape(4, 32, 8, 32, window, wide=impl == 3)
     U = np.tile(np.eye(32), (4, 1, 1))
     rng = np.random.default_rng(5)
     for key, query in [(0, 0), (0, 39), (0, 40), (15, 54), (15, 55), (16, 55), (16, 56), (47, 86), (48, 87), (48, 88), (90, 129), (89, 129), (31, 32), (60, 100)]:
@@ -245,11 +257,11 @@ def test_a_key_that_stands_out_is_seen_up_to_the_windows_edge_and_not_beyond(dty
             assert np.abs(got - want).max() < (2e-5 if dtype == F32 else 2e-2)
 
 
-@pytest.mark.parametrize("dtype,impl", FORMS)
+@pytest.mark.parametrize("dtype,impl", ALL_FORMS)
 @pytest.mark.parametrize("strength", [-200.0, 3.0, 40.0, 200.0])
 def test_the_sink_takes_its_share_once(dtype, impl, strength):
     """From nothing to all of the weight, with keys in one share or in several (long prompts split their keys)."""
-    s = Shape(2, 16, 8, 32, 0)
+    s = Shape(2, 16, 8, 32, 0, wide=impl == 3)
     seqs, norm, U, _ = random_case(s, (900,), 2)
     sink = np.array([strength, -200.0])
     q, kv = seqs[0]
@@ -261,10 +273,12 @@ def test_the_sink_takes_its_share_once(dtype, impl, strength):
 
 
 @pytest.mark.parametrize("shape,n", [((16, 8, 16, 64, 0), 1500), ((7, 8, 8, 256, 900), 2000), ((32, 16, 64, 512, 700), 1100), ((128, 8, 8, 96, 300), 500)], ids=str)
-def test_decoding_over_many_keys(shape, n):
-    s = Shape(*shape)
+@pytest.mark.parametrize("impl", [2, 3])
+def test_decoding_over_many_keys(shape, n, impl):
+    """Keys in several shares, from one row tile of heads to several."""
+    s = Shape(*shape, wide=True)
     seqs, norm, U, sink = random_case(s, (n, n // 3, 9), n)
-    got = run(s, seqs, [[n - 3, 1, 1, 1], [n // 3 - 3, 1, 1, 1], [6, 1, 1, 1]], norm, U, sink, F16, 0)
+    got = run(s, seqs, [[n - 3, 1, 1, 1], [n // 3 - 3, 1, 1, 1], [6, 1, 1, 1]], norm, U, sink, F16, impl)
     for (q, kv), g in zip(seqs, got):
         want = reference(s, q, kv, norm, U, sink)
         assert np.abs(g[-3:] - want[-3:]).max() < 1e-2 * max(1, np.abs(want).max())
