@@ -517,15 +517,15 @@ int launch_mma(ingot_skv* kv, AttendParams p, cudaStream_t s) {
     return merge(p, s);
 }
 
-// Single tokens on tcgen05. A share of the keys costs its tiles and about one tile more; several shares cost a merge.
+// Single tokens on tcgen05. A share of the keys costs its tiles and about three tiles more; several shares cost a merge.
 int launch_decode(ingot_skv* kv, int layer, AttendParams p, cudaStream_t s) {
-    constexpr int kDecodeTile = 128;
+    constexpr int kDecodeTile = 64;
     const int keys = p.map.window > 0 ? std::min(p.max_blocks * kBlockTokens, p.map.window + kBlockTokens) : p.max_blocks * kBlockTokens;
     const int tiles = (keys + kDecodeTile - 1) / kDecodeTile, heads = latent_decode_heads(p.n_head);
     const long long ctas = (long long)((p.n_head + heads - 1) / heads) * p.st.n_seq;
     long long best = -1;
     for (int n = 1; n <= std::min(kMaxSplits, tiles); n++) {
-        const long long cost = (ctas * n + kv->num_sms - 1) / kv->num_sms * ((tiles + n - 1) / n + 1) * 32 + (n > 1 ? 24 + n : 0);
+        const long long cost = (ctas * n + kv->num_sms - 1) / kv->num_sms * ((tiles + n - 1) / n + 3) * 16 + (n > 1 ? 24 + n : 0);
         if (best < 0 || cost < best) { best = cost; p.n_splits = n; }
     }
     if (const int rc = make_room(kv, p)) return rc;

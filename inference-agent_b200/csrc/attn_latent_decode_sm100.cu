@@ -1,15 +1,17 @@
 // Latent attention of decoded tokens on the sm_100a tensor cores (attn_latent.cu has the mechanism). One token's heads are few and the
 // cached rows long, so the products are turned round: keys, then latent columns, are the 128 rows of the MMAs, the heads their columns.
-//     S^T [128 keys][heads]      = rows . q^T      A: the key tile as it lies in memory (K-major), B: the query rows
+//     S^T [keys][heads]          = rows . q^T      A: the key tile as it lies in memory (K-major), B: the query rows
 //     O^T [128 columns][heads] += rows^T . p^T     A: the same tile read along its other dimension (MN-major), B: the weights
 // Nothing is padded but the heads (to 16 or 32), one tile of shared memory serves both products, and the whole result of 512 latent
 // columns and 32 heads takes 128 columns of tensor memory. The kernel is bound by reading the rows.
 //
-// One CTA = up to 32 heads of one token x one share of its visible pages, in tiles of 128 keys = 8 pages. A tile is row / 64 units of
-// 128 keys x 64 columns (16 KB, TMA, one box per page); as many tiles as fit make the ring, and each unit is given back on its own: the
-// last ones (rotated part) after the scores, a pair of the others after its block of latent columns.
+// One CTA = up to 32 heads of one token x one share of its visible pages, in tiles of 64 keys = 4 pages, so that two tiles of the
+// longest rows fit shared memory and one loads while the other is multiplied. (The score MMAs still have 128 rows: the upper 64 read
+// whatever follows the unit and their results are not looked at.) A tile is row / 64 units of 64 keys x 64 columns (8 KB, TMA, one box
+// per page); each unit is given back on its own: the last ones (rotated part) after the scores, a pair of the others after its block
+// of latent columns.
 // Roles: warp 0 TMA, warp 1 MMA issue, warps 2-5 softmax. The scores come out of tensor memory with a key per thread, go through shared
-// memory to a quarter of the heads per warp (four keys per lane), and back as f16 weights, the B operand of the second product.
+// memory to a quarter of the heads per warp (two keys per lane), and back as f16 weights, the B operand of the second product.
 // Every mbarrier wait is bounded: on expiry all roles leave, copies in flight are drained, tensor memory is freed and the cache's
 // status word gets its bit.
 #include <mutex>
@@ -21,9 +23,9 @@ namespace {
 
 using namespace ingot_sm100;
 
-constexpr int kKeys = 128, kPages = kKeys / kBlockTokens, kUnit = kKeys * 128;
+constexpr int kKeys = 64, kPages = kKeys / kBlockTokens, kUnit = kKeys * 128;
 constexpr int kThreads = 192;
-constexpr int kMaxUnits = 12;
+constexpr int kMaxUnits = 24;
 constexpr float kRescaleThreshold = 8.0f;  // log2 units
 constexpr unsigned long long kWaitLimitNs = 2000000000ull;
 constexpr int kSmemLimit = 227 * 1024;
@@ -42,18 +44,20 @@ struct Bars {
 
 template <int kN>  // heads per CTA
 struct Layout {
-    static constexpr int kP = kN * 256;         // weights: two blocks [heads][64 keys]
+    static constexpr int kP = kN * 128;         // weights [heads][64 keys]
     static constexpr int kS = kN * kKeys * 4;   // scores [heads][keys]
     int units, stages, off_ring, off_p, off_s, off_vec, off_bar, bytes;
+    // behind the ring: weights and scores, and at least a unit, which the score MMAs of the last one read as their upper rows
+    __host__ __device__ static constexpr int after_ring() { return kP + kS > kUnit ? kP + kS : kUnit; }
     __host__ __device__ explicit Layout(int row) {
         units = row / 64;
-        const int fixed = units * kN * 128 + kP + kS + 2 * kN * 4 + int(sizeof(Bars)) + 1024 + 64;
+        const int fixed = units * kN * 128 + 1024 + after_ring() + 2 * kN * 4 + int(sizeof(Bars)) + 1024 + 64;
         stages = (kSmemLimit - fixed) / (units * kUnit);
         if (stages * units > kMaxUnits) stages = kMaxUnits / units;
         off_ring = (units * kN * 128 + 1023) / 1024 * 1024;
         off_p = off_ring + stages * units * kUnit;
         off_s = off_p + kP;
-        off_vec = off_s + kS;
+        off_vec = off_p + after_ring();
         off_bar = (off_vec + 2 * kN * 4 + 15) / 16 * 16;
         bytes = off_bar + int(sizeof(Bars)) + 1024;
     }
@@ -209,8 +213,8 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap map_rows, const __grid_
                     const int s = (it % stages) * units + 2 * b;
                     const uint32_t a = smem_base + L.off_ring + s * kUnit, w = smem_base + L.off_p;
 #pragma unroll
-                    for (int ks = 0; ks < 8; ks++)
-                        tc_mma_ss(tmem + (2 + b) * kN, make_desc(a + ks * 2048, kUnit, 1024), make_desc(w + (ks >> 2) * kN * 128 + (ks & 3) * 32, 16, 1024), kIdescV<kN>,
+                    for (int ks = 0; ks < kKeys / 16; ks++)
+                        tc_mma_ss(tmem + (2 + b) * kN, make_desc(a + ks * 2048, kUnit, 1024), make_desc(w + ks * 32, 16, 1024), kIdescV<kN>,
                                   (it > 0 || ks > 0) ? 1u : 0u);
                     tc_commit(smem_u32(&bars->empty[s]));
                     tc_commit(smem_u32(&bars->empty[s + 1]));
@@ -235,7 +239,7 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap map_rows, const __grid_
         for (int it = 0; it < n_it; it++) {
             ok = mbar_wait(smem_u32(&bars->s_ready[it & 1]), (uint32_t)((it >> 1) & 1), abort_flag, kWaitLimitNs);
             ok = __all_sync(0xffffffffu, ok) != 0;
-            if (ok) {
+            if (ok && quarter < 2) {  // the tile's keys are the lower half of the lanes
                 float s[kN];
                 tc_fence_after();
                 tmem_ld<kN>(tmem + (it & 1) * kN + lane_sel, s);
@@ -247,13 +251,13 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap map_rows, const __grid_
             }
             ok = softmax_all(ok);
             if (!ok) break;  // all four warps together
-            // this warp's heads, four keys per lane
-            float4 v[kHeadsPerWarp];
+            // this warp's heads, two keys per lane
+            float2 v[kHeadsPerWarp];
             bool grows = false;
 #pragma unroll
             for (int h = 0; h < kHeadsPerWarp; h++) {
-                v[h] = *reinterpret_cast<const float4*>(s_score + (quarter * kHeadsPerWarp + h) * kKeys + lane * 4);
-                grows = grows || fmaxf(fmaxf(v[h].x, v[h].y), fmaxf(v[h].z, v[h].w)) > m_ref[h] + kRescaleThreshold;
+                v[h] = *reinterpret_cast<const float2*>(s_score + (quarter * kHeadsPerWarp + h) * kKeys + lane * 2);
+                grows = grows || fmaxf(v[h].x, v[h].y) > m_ref[h] + kRescaleThreshold;
             }
             // Lazy rescale: a head's reference maximum moves only when its maximum grew by more than 2^8 (always at the first tile,
             // every one of which holds a visible key).
@@ -263,7 +267,7 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap map_rows, const __grid_
             if (__any_sync(0xffffffffu, grows)) {
 #pragma unroll
                 for (int h = 0; h < kHeadsPerWarp; h++) {
-                    float mx = fmaxf(fmaxf(v[h].x, v[h].y), fmaxf(v[h].z, v[h].w));
+                    float mx = fmaxf(v[h].x, v[h].y);
 #pragma unroll
                     for (int o = 16; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
                     if (mx > m_ref[h] + kRescaleThreshold) {
@@ -285,13 +289,10 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap map_rows, const __grid_
 #pragma unroll
             for (int h = 0; h < kHeadsPerWarp; h++) {
                 const float ref = m_ref[h] == -INFINITY ? 0.f : m_ref[h];
-                const float p0 = ex2(v[h].x - ref), p1 = ex2(v[h].y - ref), p2 = ex2(v[h].z - ref), p3 = ex2(v[h].w - ref);
-                l[h] += (p0 + p1) + (p2 + p3);
-                const int head = quarter * kHeadsPerWarp + h;
-                // row `head` of the block of keys 0-63 or 64-127, 16-byte pieces XOR-swizzled by row
-                unsigned char* row = smem_al + L.off_p + (lane >> 4) * kN * 128 + head * 128;
-                const int piece = (lane & 15) >> 1;
-                *reinterpret_cast<uint2*>(row + ((piece ^ (head & 7)) << 4) + (lane & 1) * 8) = make_uint2(pack_half2_rn(p0, p1), pack_half2_rn(p2, p3));
+                const float p0 = ex2(v[h].x - ref), p1 = ex2(v[h].y - ref);
+                l[h] += p0 + p1;
+                const int head = quarter * kHeadsPerWarp + h;  // 16-byte pieces of its row XOR-swizzled
+                *reinterpret_cast<uint32_t*>(smem_al + L.off_p + head * 128 + (((lane >> 2) ^ (head & 7)) << 4) + (lane & 3) * 4) = pack_half2_rn(p0, p1);
             }
             asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
             ok = softmax_all(ok);  // scores are read, factors and weights are in
