@@ -46,6 +46,7 @@ struct AppendParams {
     int long_from, long_dim, long_rot, heads_per_cta;
     void* rows;
     int row;
+    bool tiled;
     const int32_t *tables, *first_page;
     int max_blocks, n_blocks;
     PageMap map;
@@ -86,9 +87,10 @@ __global__ void __launch_bounds__(kAppendThreads) latent_append_kernel(const App
         const float inv = 1.0f / sqrtf(ss / float(p.sh.rank_count) + p.eps);
         const int blk = table_block(p.tables, p.first_page, p.max_blocks, p.n_blocks, seq, p.map.page(pos), p.status);
         if (blk < 0) return;
-        T* dst = static_cast<T*>(p.rows) + ((size_t)blk * kBlockTokens + p.map.slot(pos)) * p.row;
-        for (int i = threadIdx.x; i < p.sh.rank; i += kAppendThreads) put(dst + i, c[i] * inv * p.norm_w[i]);
-        for (int i = threadIdx.x; i < p.sh.rot; i += kAppendThreads) put(dst + p.sh.rank + i, rotated(c + p.sh.rank, i));
+        T* dst = static_cast<T*>(p.rows) + (size_t)blk * kBlockTokens * p.row;
+        const int slot = p.map.slot(pos);
+        for (int i = threadIdx.x; i < p.sh.rank; i += kAppendThreads) put(dst + page_elem(p.tiled, p.row, slot, i), c[i] * inv * p.norm_w[i]);
+        for (int i = threadIdx.x; i < p.sh.rot; i += kAppendThreads) put(dst + page_elem(p.tiled, p.row, slot, p.sh.rank + i), rotated(c + p.sh.rank, i));
         return;
     }
     __syncthreads();  // the angles
@@ -213,7 +215,7 @@ __global__ void __launch_bounds__(kLatThreads) latent_mma_kernel(const AttendPar
         const uint32_t dst = s_base + L.k + (t & 1) * kTileKeys * stride;
         for (int i = threadIdx.x; i < kTileKeys * pieces; i += kLatThreads) {
             const int key = i / pieces, c = i - key * pieces, blk = s_blk[t * 4 + (key >> 4)];
-            cp16(dst + key * stride + c * 16, static_cast<const __half*>(p.rows) + ((size_t)max(blk, 0) * kBlockTokens + (key & 15)) * p.dim + c * 8, blk >= 0);
+            cp16(dst + key * stride + c * 16, static_cast<const __half*>(p.rows) + (size_t)max(blk, 0) * kBlockTokens * p.dim + page_elem(p.tiled, p.dim, key & 15, c * 8), blk >= 0);
         }
         asm volatile("cp.async.commit_group;" ::: "memory");
     };
@@ -518,7 +520,7 @@ int launch_mma(ingot_skv* kv, AttendParams p, cudaStream_t s) {
 }
 
 // Single tokens on tcgen05. A share of the keys costs its tiles and about three tiles more; several shares cost a merge.
-int launch_decode(ingot_skv* kv, int layer, AttendParams p, cudaStream_t s) {
+int launch_decode(ingot_skv* kv, AttendParams p, cudaStream_t s) {
     constexpr int kDecodeTile = 64;
     const int keys = p.map.window > 0 ? std::min(p.max_blocks * kBlockTokens, p.map.window + kBlockTokens) : p.max_blocks * kBlockTokens;
     const int tiles = (keys + kDecodeTile - 1) / kDecodeTile, heads = latent_decode_heads(p.n_head);
@@ -529,7 +531,7 @@ int launch_decode(ingot_skv* kv, int layer, AttendParams p, cudaStream_t s) {
         if (best < 0 || cost < best) { best = cost; p.n_splits = n; }
     }
     if (const int rc = make_room(kv, p)) return rc;
-    if (const int rc = launch_latent_decode_sm100(kv, layer, p, s)) return rc;
+    if (const int rc = launch_latent_decode_sm100(kv, p, s)) return rc;
     return merge(p, s);
 }
 
@@ -565,7 +567,7 @@ int ingot_latent_append(ingot_skv* kv, int layer, const ingot_step* step, const 
     AppendParams p = {*step, proj_dev, proj_ld, q_off, latent_off, sh, norm_dev, eps, turns_dev,
                       SharedOut{q_plain->f32, static_cast<__nv_bfloat16*>(q_plain->hi), static_cast<__nv_bfloat16*>(q_plain->lo), q_plain->ld, 1.0f}, q_rows_dev,
                       static_cast<__half*>(q_long_dev), q_long_dev ? long_from : 0x7fffffff, long_dim, long_rot, heads_per_cta,
-                      static_cast<char*>(kv->rows) + kv->layer_elems * layer * esz, kv->dim, tables_dev, first_page_dev, max_blocks, kv->n_blocks, page_map(kv),
+                      static_cast<char*>(kv->rows) + kv->layer_elems * layer * esz, kv->dim, kv->tiled, tables_dev, first_page_dev, max_blocks, kv->n_blocks, page_map(kv),
                       kv->status_dev};
     auto kernel = kv->dtype == INGOT_F32 ? latent_append_kernel<float> : latent_append_kernel<__half>;
     INGOT_CUDA_TRY(ingot_launch_pdl(kernel, dim3(step->n_tok, 1 + (sh.n_head + heads_per_cta - 1) / heads_per_cta), dim3(kAppendThreads), 0, static_cast<cudaStream_t>(stream), p));
@@ -594,10 +596,10 @@ int ingot_latent_attend(ingot_skv* kv, int layer, const ingot_step* step, const 
     AttendParams p = {*step, q_rows_dev, static_cast<const char*>(kv->rows) + kv->layer_elems * layer * esz, nullptr, tables_dev, first_page_dev, max_blocks,
                       kv->n_blocks, n_head, 1, kv->dim, rank, page_map(kv), scale,
                       SharedOut{out->f32, static_cast<__nv_bfloat16*>(out->hi), static_cast<__nv_bfloat16*>(out->lo), out->ld, 1.0f}, kv->status_dev, 1, nullptr,
-                      sink_dev};
+                      kv->tiled, sink_dev};
     cudaStream_t s = static_cast<cudaStream_t>(stream);
-    if (kv->dtype == INGOT_F16 && (impl == 0 || impl == 3) && step->max_len == 1 && latent_decode_takes(kv->dim, rank)) {
-        const int rc = launch_decode(kv, layer, p, s);
+    if (kv->tiled && (impl == 0 || impl == 3) && step->max_len == 1 && latent_decode_takes(kv->dim, rank)) {
+        const int rc = launch_decode(kv, p, s);
         if (rc != INGOT_ERR_UNSUPPORTED || impl == 3) return rc;
     }
     if (kv->dtype == INGOT_F16 && impl != 1 && impl != 3 && mma_takes(kv->dim, rank) && out->ld % 2 == 0) return launch_mma(kv, p, s);

@@ -6,10 +6,9 @@
 // columns and 32 heads takes 128 columns of tensor memory. The kernel is bound by reading the rows.
 //
 // One CTA = up to 32 heads of one token x one share of its visible pages, in tiles of 64 keys = 4 pages, so that two tiles of the
-// longest rows fit shared memory and one loads while the other is multiplied. (The score MMAs still have 128 rows: the upper 64 read
-// whatever follows the unit and their results are not looked at.) A tile is row / 64 units of 64 keys x 64 columns (8 KB, TMA, one box
-// per page); each unit is given back on its own: the last ones (rotated part) after the scores, a pair of the others after its block
-// of latent columns.
+// longest rows fit shared memory and one loads while the other is multiplied. Pages lie in memory as the MMAs want them (tiled order,
+// page_elem): a page is one contiguous copy, the 8-key groups of a tile follow each other units * 1024 bytes apart, whatever the page.
+// (The score MMAs still have 128 rows: the upper 64 read what follows the tile in shared memory and their results are not looked at.)
 // Roles: warp 0 TMA, warp 1 MMA issue, warps 2-5 softmax. The scores come out of tensor memory with a key per thread, go through shared
 // memory to a quarter of the heads per warp (two keys per lane), and back as f16 weights, the B operand of the second product.
 // Every mbarrier wait is bounded: on expiry all roles leave, copies in flight are drained, tensor memory is freed and the cache's
@@ -23,16 +22,16 @@ namespace {
 
 using namespace ingot_sm100;
 
-constexpr int kKeys = 64, kPages = kKeys / kBlockTokens, kUnit = kKeys * 128;
+constexpr int kKeys = 64, kPages = kKeys / kBlockTokens;
 constexpr int kThreads = 192;
-constexpr int kMaxUnits = 24;
+constexpr int kMaxStages = 8;
 constexpr float kRescaleThreshold = 8.0f;  // log2 units
 constexpr unsigned long long kWaitLimitNs = 2000000000ull;
 constexpr int kSmemLimit = 227 * 1024;
 
 struct Bars {
-    uint64_t full[kMaxUnits];
-    uint64_t empty[kMaxUnits];
+    uint64_t full[kMaxStages];
+    uint64_t empty[kMaxStages];
     uint64_t q_ready;
     uint64_t s_ready[2];
     uint64_t p_ready;
@@ -46,20 +45,22 @@ template <int kN>  // heads per CTA
 struct Layout {
     static constexpr int kP = kN * 128;         // weights [heads][64 keys]
     static constexpr int kS = kN * kKeys * 4;   // scores [heads][keys]
-    int units, stages, off_ring, off_p, off_s, off_vec, off_bar, bytes;
-    // behind the ring: weights and scores, and at least a unit, which the score MMAs of the last one read as their upper rows
-    __host__ __device__ static constexpr int after_ring() { return kP + kS > kUnit ? kP + kS : kUnit; }
+    int units, tile, stages, off_q, off_p, off_s, off_vec, off_bar, bytes;
+    // The ring comes first, and the whole is at least a tile longer than it: the upper rows of the score MMAs stay inside.
     __host__ __device__ explicit Layout(int row) {
         units = row / 64;
-        const int fixed = units * kN * 128 + 1024 + after_ring() + 2 * kN * 4 + int(sizeof(Bars)) + 1024 + 64;
-        stages = (kSmemLimit - fixed) / (units * kUnit);
-        if (stages * units > kMaxUnits) stages = kMaxUnits / units;
-        off_ring = (units * kN * 128 + 1023) / 1024 * 1024;
-        off_p = off_ring + stages * units * kUnit;
+        tile = kKeys * row * 2;
+        const int fixed = units * kN * 128 + kP + kS + 2 * kN * 4 + int(sizeof(Bars)) + 64, limit = kSmemLimit - 1024;
+        stages = 0;
+        while (stages < kMaxStages && (stages + 1) * tile + fixed <= limit && (stages + 2) * tile <= limit) stages++;
+        off_q = stages * tile;
+        off_p = off_q + units * kN * 128;
         off_s = off_p + kP;
-        off_vec = off_p + after_ring();
+        off_vec = off_s + kS;
         off_bar = (off_vec + 2 * kN * 4 + 15) / 16 * 16;
-        bytes = off_bar + int(sizeof(Bars)) + 1024;
+        bytes = off_bar + int(sizeof(Bars));
+        if (bytes < (stages + 1) * tile) bytes = (stages + 1) * tile;
+        bytes += 1024;
     }
 };
 
@@ -105,7 +106,7 @@ template <int kN> constexpr uint32_t kIdescV = kIdescS<kN> | (1u << 15);
 
 template <int kN>
 __global__ void __launch_bounds__(kThreads, 1)
-latent_decode_kernel(const __grid_constant__ CUtensorMap map_rows, const __grid_constant__ CUtensorMap map_q, const __grid_constant__ AttendParams p) {
+latent_decode_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ AttendParams p) {
     constexpr int kHeadsPerWarp = kN / 4;
     extern __shared__ unsigned char smem_dyn[];
     INGOT_PDL_TRIGGER();
@@ -126,7 +127,7 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap map_rows, const __grid_
     const int units = L.units, stages = L.stages, blocks = (p.out_dim + 127) / 128;
 
     if (threadIdx.x == 0) {
-        for (int s = 0; s < stages * units; s++) { mbar_init(smem_u32(&bars->full[s]), 1); mbar_init(smem_u32(&bars->empty[s]), 1); }
+        for (int s = 0; s < stages; s++) { mbar_init(smem_u32(&bars->full[s]), 1); mbar_init(smem_u32(&bars->empty[s]), 1); }
         mbar_init(smem_u32(&bars->q_ready), 1);
         mbar_init(smem_u32(&bars->s_ready[0]), 1);
         mbar_init(smem_u32(&bars->s_ready[1]), 1);
@@ -148,81 +149,86 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap map_rows, const __grid_
     const uint32_t tmem = bars->tmem_base;  // S0 S1 | O, one column per head each
 
     if (warp_u == 0) {
-        // ---------------- TMA producer: lanes 0-7 fetch one page each ----------------
+        // ---------------- producer: lanes 0-3 fetch one page each ----------------
         int armed = 0;
         bool ok = true;
-        if (lane == 0 && n_it > 0) {
-            mbar_expect_tx(smem_u32(&bars->q_ready), units * kN * 128);
-            for (int u = 0; u < units; u++) tma_load_2d(smem_base + u * kN * 128, &map_q, u * 64, (int)tok * p.n_head + h0, smem_u32(&bars->q_ready));
-        }
-        for (int it = 0; it < n_it && ok; it++) {
+        const uint32_t page_bytes = kBlockTokens * p.dim * 2;
+        for (int it = 0; it < n_it; it++) {
             // pages past the last one, or without a valid block, are replaced by block 0: their keys are masked
-            const int page = page0 + it * kPages + lane;
+            const int page = page0 + it * kPages + lane, s = it % stages;
             const int blk = lane < kPages && page <= page_b ? max(table_block(p.tables, p.first_page, p.max_blocks, p.n_blocks, seq, page, p.status), 0) : 0;
-            for (int u = 0; u < units; u++) {
-                const int s = (it % stages) * units + u;
-                const uint32_t full = smem_u32(&bars->full[s]);
-                if (lane == 0) {
-                    ok = mbar_wait(smem_u32(&bars->empty[s]), (uint32_t)(((it / stages) & 1) ^ 1), abort_flag, kWaitLimitNs);
-                    if (ok) mbar_expect_tx(full, kUnit);
-                }
-                ok = __shfl_sync(0xffffffffu, ok, 0);
-                if (!ok) break;
-                if (lane < kPages) tma_load_3d(smem_base + L.off_ring + s * kUnit + lane * (kBlockTokens * 128), &map_rows, u * 64, 0, blk, full);
-                armed++;
+            const uint32_t full = smem_u32(&bars->full[s]);
+            if (lane == 0) {
+                ok = mbar_wait(smem_u32(&bars->empty[s]), (uint32_t)(((it / stages) & 1) ^ 1), abort_flag, kWaitLimitNs);
+                if (ok) mbar_expect_tx(full, L.tile);
+            }
+            ok = __shfl_sync(0xffffffffu, ok, 0);
+            if (!ok) break;
+            if (lane < kPages)
+                bulk_load(smem_base + s * L.tile + lane * page_bytes, static_cast<const __half*>(p.rows) + (size_t)blk * kBlockTokens * p.dim, page_bytes, full);
+            armed = it + 1;
+            if (it == 0 && lane == 0) {
+                mbar_expect_tx(smem_u32(&bars->q_ready), units * kN * 128);
+                for (int u = 0; u < units; u++) tma_load_2d(smem_base + L.off_q + u * kN * 128, &map_q, u * 64, (int)tok * p.n_head + h0, smem_u32(&bars->q_ready));
             }
         }
         if (!ok && lane == 0) {
             // copies already issued must land before the CTA's shared memory is released
-            for (int i = max(0, armed - stages * units); i < armed; i++) {
-                const int it = i / units, s = (it % stages) * units + i % units;
+            for (int it = max(0, armed - stages); it < armed; it++) {
                 const uint64_t t0 = globaltimer_ns();
-                while (!mbar_try_wait(smem_u32(&bars->full[s]), (uint32_t)((it / stages) & 1)) && globaltimer_ns() - t0 < 100000000ull) {}
+                while (!mbar_try_wait(smem_u32(&bars->full[it % stages]), (uint32_t)((it / stages) & 1)) && globaltimer_ns() - t0 < 100000000ull) {}
             }
             const uint64_t t0 = globaltimer_ns();
-            while (!mbar_try_wait(smem_u32(&bars->q_ready), 0) && globaltimer_ns() - t0 < 100000000ull) {}
+            while (armed > 0 && !mbar_try_wait(smem_u32(&bars->q_ready), 0) && globaltimer_ns() - t0 < 100000000ull) {}
         }
     } else if (warp_u == 1) {
         // ---------------- MMA issuer: the whole warp walks the loop, one elected lane issues ----------------
         bool ok = n_it == 0 || __all_sync(0xffffffffu, mbar_wait(smem_u32(&bars->q_ready), 0, abort_flag, kWaitLimitNs)) != 0;
+        const uint32_t group = units * 1024;  // bytes from one group of 8 keys to the next
         auto scores = [&](int it) {
-            for (int u = 0; u < units && ok; u++) {
-                const int s = (it % stages) * units + u;
-                ok = __all_sync(0xffffffffu, mbar_wait(smem_u32(&bars->full[s]), (uint32_t)((it / stages) & 1), abort_flag, kWaitLimitNs)) != 0;
-                if (!ok) break;
-                tc_fence_after();
-                if (elect_one()) {
-                    const uint32_t a = smem_base + L.off_ring + s * kUnit, b = smem_base + u * kN * 128;
+            ok = __all_sync(0xffffffffu, mbar_wait(smem_u32(&bars->full[it % stages]), (uint32_t)((it / stages) & 1), abort_flag, kWaitLimitNs)) != 0;
+            if (!ok) return;
+            tc_fence_after();
+            if (elect_one()) {
+                for (int u = 0; u < units; u++) {
+                    const uint32_t a = smem_base + (it % stages) * L.tile + u * 1024, b = smem_base + L.off_q + u * kN * 128;
 #pragma unroll
                     for (int ks = 0; ks < 4; ks++)
-                        tc_mma_ss(tmem + (it & 1) * kN, make_desc(a + ks * 32, 16, 1024), make_desc(b + ks * 32, 16, 1024), kIdescS<kN>, (u > 0 || ks > 0) ? 1u : 0u);
-                    if (u >= 2 * blocks) tc_commit(smem_u32(&bars->empty[s]));  // no part of the values
-                    if (u == units - 1) tc_commit(smem_u32(&bars->s_ready[it & 1]));
+                        tc_mma_ss(tmem + (it & 1) * kN, make_desc(a + ks * 32, 16, group), make_desc(b + ks * 32, 16, 1024), kIdescS<kN>, (u > 0 || ks > 0) ? 1u : 0u);
                 }
-                __syncwarp();
+                tc_commit(smem_u32(&bars->s_ready[it & 1]));
             }
+            __syncwarp();
         };
         if (n_it > 0 && ok) scores(0);
         for (int it = 0; it < n_it && ok; it++) {
-            if (stages > 1 && it + 1 < n_it) scores(it + 1);  // with one stage the next tile only comes in as this one is given back
+            // The next tile's scores go first if it is there before this one's weights are - but this one is given back without
+            // waiting for it, so that two tiles are on their way at a time.
+            const bool more = it + 1 < n_it;
+            bool ahead = false;
+            for (int spin = 0; more && stages > 1 && ok && spin < (1 << 20); spin++) {
+                if (__any_sync(0xffffffffu, mbar_test(smem_u32(&bars->p_ready), (uint32_t)(it & 1)))) break;
+                if (__all_sync(0xffffffffu, mbar_test(smem_u32(&bars->full[(it + 1) % stages]), (uint32_t)(((it + 1) / stages) & 1)))) {
+                    scores(it + 1);
+                    ahead = true;
+                    break;
+                }
+            }
             ok = ok && __all_sync(0xffffffffu, mbar_wait(smem_u32(&bars->p_ready), (uint32_t)(it & 1), abort_flag, kWaitLimitNs)) != 0;
             if (!ok) break;
             tc_fence_after();
             if (elect_one()) {
                 for (int b = 0; b < blocks; b++) {
-                    const int s = (it % stages) * units + 2 * b;
-                    const uint32_t a = smem_base + L.off_ring + s * kUnit, w = smem_base + L.off_p;
+                    const uint32_t a = smem_base + (it % stages) * L.tile + b * 2048, w = smem_base + L.off_p;
 #pragma unroll
                     for (int ks = 0; ks < kKeys / 16; ks++)
-                        tc_mma_ss(tmem + (2 + b) * kN, make_desc(a + ks * 2048, kUnit, 1024), make_desc(w + ks * 32, 16, 1024), kIdescV<kN>,
-                                  (it > 0 || ks > 0) ? 1u : 0u);
-                    tc_commit(smem_u32(&bars->empty[s]));
-                    tc_commit(smem_u32(&bars->empty[s + 1]));
+                        tc_mma_ss(tmem + (2 + b) * kN, make_desc(a + ks * 2 * group, 1024, group), make_desc(w + ks * 32, 16, 1024), kIdescV<kN>, (it > 0 || ks > 0) ? 1u : 0u);
                 }
+                tc_commit(smem_u32(&bars->empty[it % stages]));
                 tc_commit(smem_u32(&bars->pv_done));
             }
             __syncwarp();
-            if (stages == 1 && it + 1 < n_it) scores(it + 1);
+            if (more && !ahead) scores(it + 1);
         }
     } else {
         // ---------------- softmax warps ----------------
@@ -355,13 +361,17 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap map_rows, const __grid_
                     tmem_wait_ld();
                 }
                 const int d = b * 128 + quarter * 32 + lane;
-                if (d < p.out_dim) {
+                if (d >= p.out_dim) continue;
+                if (p.n_splits == 1) {
 #pragma unroll
-                    for (int h = 0; h < kN; h++) {
-                        if (h >= heads) break;
-                        if (p.n_splits == 1) p.out.store(tok, (h0 + h) * p.out_dim + d, o[h] * s_max[h]);
-                        else p.part[((tok * p.n_head + h0 + h) * p.n_splits + split) * (p.out_dim + 2) + d] = n_it > 0 ? o[h] : 0.f;
-                    }
+                    for (int h = 0; h < kN; h++)
+                        if (h < heads) p.out.store(tok, (h0 + h) * p.out_dim + d, o[h] * s_max[h]);
+                } else {
+                    float* part = p.part + ((tok * p.n_head + h0) * p.n_splits + split) * (p.out_dim + 2) + d;
+                    const size_t next = (size_t)p.n_splits * (p.out_dim + 2);
+#pragma unroll
+                    for (int h = 0; h < kN; h++)
+                        if (h < heads) part[h * next] = n_it > 0 ? o[h] : 0.f;
                 }
             }
         }
@@ -397,34 +407,20 @@ EncodeTiledFn encode_fn() {
 // Row lengths the kernel takes: whole units, the latent's blocks of 128 columns inside the row, at least one tile in shared memory.
 bool latent_decode_takes(int row, int rank) {
     const int blocks = (rank + 127) / 128;
-    return row % 64 == 0 && blocks * 128 <= row && row / 64 <= kMaxUnits && blocks <= 4 && Layout<32>(row).stages >= 1 && encode_fn() != nullptr;
+    return row % 64 == 0 && blocks * 128 <= row && blocks <= 4 && Layout<32>(row).stages >= 1 && encode_fn() != nullptr;
 }
 int latent_decode_heads(int n_head) { return n_head <= 16 ? 16 : 32; }
 
 // Decoded tokens (every sequence of the step has one); n_splits and part are set. q_rows: rows of the query buffer.
-int launch_latent_decode_sm100(ingot_skv* kv, int layer, const AttendParams& p, cudaStream_t stream) {
-    EncodeTiledFn encode = encode_fn();
-    const cuuint32_t e3[3] = {1, 1, 1};
-    if (kv->tmaps.empty()) {
-        std::vector<CUtensorMap> maps(kv->n_layer);
-        for (int i = 0; i < kv->n_layer; i++) {
-            const cuuint64_t dims[3] = {(cuuint64_t)kv->dim, kBlockTokens, (cuuint64_t)kv->n_blocks};
-            const cuuint64_t strides[2] = {(cuuint64_t)kv->dim * 2, (cuuint64_t)kBlockTokens * kv->dim * 2};
-            const cuuint32_t box[3] = {64, kBlockTokens, 1};
-            if (encode(&maps[i], CU_TENSOR_MAP_DATA_TYPE_FLOAT16, 3, static_cast<__half*>(kv->rows) + (size_t)i * kv->layer_elems, dims, strides, box, e3,
-                       CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
-                       CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) != CUDA_SUCCESS)
-                return INGOT_ERR_UNSUPPORTED;
-        }
-        kv->tmaps = std::move(maps);
-    }
+int launch_latent_decode_sm100(const ingot_skv* kv, const AttendParams& p, cudaStream_t stream) {
+    if (!kv->tiled) return INGOT_ERR_UNSUPPORTED;
     const int n = latent_decode_heads(p.n_head);
     CUtensorMap map_q;
     {
         const cuuint64_t dims[2] = {(cuuint64_t)kv->dim, (cuuint64_t)p.st.n_tok * p.n_head};
         const cuuint64_t strides[1] = {(cuuint64_t)kv->dim * 2};
-        const cuuint32_t box[2] = {64, (cuuint32_t)n};
-        if (encode(&map_q, CU_TENSOR_MAP_DATA_TYPE_FLOAT16, 2, const_cast<void*>(p.q), dims, strides, box, e3, CU_TENSOR_MAP_INTERLEAVE_NONE,
+        const cuuint32_t box[2] = {64, (cuuint32_t)n}, estr[2] = {1, 1};
+        if (encode_fn()(&map_q, CU_TENSOR_MAP_DATA_TYPE_FLOAT16, 2, const_cast<void*>(p.q), dims, strides, box, estr, CU_TENSOR_MAP_INTERLEAVE_NONE,
                    CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_128B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) != CUDA_SUCCESS)
             return INGOT_ERR_UNSUPPORTED;
     }
@@ -432,11 +428,11 @@ int launch_latent_decode_sm100(ingot_skv* kv, int layer, const AttendParams& p, 
     if (n == 16) {
         const int smem = Layout<16>(kv->dim).bytes;
         INGOT_CUDA_TRY(cudaFuncSetAttribute(latent_decode_kernel<16>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
-        INGOT_CUDA_TRY(ingot_launch_pdl(latent_decode_kernel<16>, grid, dim3(kThreads), size_t(smem), stream, kv->tmaps[layer], map_q, p));
+        INGOT_CUDA_TRY(ingot_launch_pdl(latent_decode_kernel<16>, grid, dim3(kThreads), size_t(smem), stream, map_q, p));
     } else {
         const int smem = Layout<32>(kv->dim).bytes;
         INGOT_CUDA_TRY(cudaFuncSetAttribute(latent_decode_kernel<32>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
-        INGOT_CUDA_TRY(ingot_launch_pdl(latent_decode_kernel<32>, grid, dim3(kThreads), size_t(smem), stream, kv->tmaps[layer], map_q, p));
+        INGOT_CUDA_TRY(ingot_launch_pdl(latent_decode_kernel<32>, grid, dim3(kThreads), size_t(smem), stream, map_q, p));
     }
     return INGOT_OK;
 }

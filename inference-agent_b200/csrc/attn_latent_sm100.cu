@@ -375,6 +375,7 @@ struct GatherParams {
     ingot_step st;
     const int32_t *key0, *key_pos;
     const __half* rows;
+    bool tiled;
     int row, rank, rot, rot_ld;
     const int32_t *tables, *first_page;
     int max_blocks, n_blocks;
@@ -391,10 +392,12 @@ __global__ void __launch_bounds__(256) latent_gather_kernel(const GatherParams p
     const int pos = p.key_pos[seq] + i;
     const int blk = table_block(p.tables, p.first_page, p.max_blocks, p.n_blocks, seq, p.map.page(pos), p.status);
     const size_t at = (size_t)p.key0[seq] + i;
-    const uint4* src = reinterpret_cast<const uint4*>(p.rows + ((size_t)max(blk, 0) * kBlockTokens + p.map.slot(pos)) * p.row);
+    const __half* page = p.rows + (size_t)max(blk, 0) * kBlockTokens * p.row;
+    const int slot = p.map.slot(pos);
+    auto piece = [&](int c) { return *reinterpret_cast<const uint4*>(page + page_elem(p.tiled, p.row, slot, c * 8)); };
     const uint4 zero = make_uint4(0, 0, 0, 0);
-    for (int c = lane; c < p.rank / 8; c += 32) reinterpret_cast<uint4*>(p.latent + at * p.rank)[c] = blk >= 0 ? src[c] : zero;
-    for (int c = lane; c < p.rot_ld / 8; c += 32) reinterpret_cast<uint4*>(p.rotated + at * p.rot_ld)[c] = blk >= 0 && c < p.rot / 8 ? src[p.rank / 8 + c] : zero;
+    for (int c = lane; c < p.rank / 8; c += 32) reinterpret_cast<uint4*>(p.latent + at * p.rank)[c] = blk >= 0 ? piece(c) : zero;
+    for (int c = lane; c < p.rot_ld / 8; c += 32) reinterpret_cast<uint4*>(p.rotated + at * p.rot_ld)[c] = blk >= 0 && c < p.rot / 8 ? piece(p.rank / 8 + c) : zero;
 }
 
 typedef CUresult (*EncodeTiledFn)(CUtensorMap*, CUtensorMapDataType, cuuint32_t, void*, const cuuint64_t*, const cuuint64_t*,
@@ -438,7 +441,7 @@ int ingot_latent_gather(ingot_skv* kv, int layer, const ingot_step* step, const 
     INGOT_REQUIRE(key0_dev && key_pos_dev && latent_dev && rotated_dev && tables_dev && max_blocks >= 1 && max_keys >= 1, "ingot_latent_gather: null argument");
     INGOT_REQUIRE(kv->dtype == INGOT_F16 && kv->n_head_kv == 1 && kv->dim % 8 == 0 && rank % 8 == 0 && rot % 8 == 0 && rank + rot <= kv->dim && rot_ld % 8 == 0 &&
                       rot_ld >= rot, "ingot_latent_gather: bad rows");
-    const GatherParams p = {*step, key0_dev, key_pos_dev, static_cast<const __half*>(kv->rows) + kv->layer_elems * layer, kv->dim, rank, rot, rot_ld,
+    const GatherParams p = {*step, key0_dev, key_pos_dev, static_cast<const __half*>(kv->rows) + kv->layer_elems * layer, kv->tiled, kv->dim, rank, rot, rot_ld,
                             tables_dev, first_page_dev, max_blocks, kv->n_blocks, page_map(kv), kv->status_dev, static_cast<__half*>(latent_dev),
                             static_cast<__half*>(rotated_dev)};
     INGOT_CUDA_TRY(ingot_launch_pdl(latent_gather_kernel, dim3((max_keys + 7) / 8, step->n_seq), dim3(256), 0, static_cast<cudaStream_t>(stream), p));

@@ -161,8 +161,8 @@ __global__ void __launch_bounds__(128) shared_kv_attend_kernel(const AttendParam
                 slot = p.map.slot(j);
                 blk = table_block(p.tables, p.first_page, p.max_blocks, p.n_blocks, seq, p.map.page(j), p.status);
             }
-            const T* src = static_cast<const T*>(p.rows) + (((size_t)max(blk, 0) * p.n_head_kv + kvh) * kBlockTokens + slot) * dim;
-            for (int d = part; d < kD * 32; d += 4) sk[key * ldk + d] = blk >= 0 && d < dim ? widen(src[d]) : 0.f;
+            const T* src = static_cast<const T*>(p.rows) + ((size_t)max(blk, 0) * p.n_head_kv + kvh) * kBlockTokens * dim;
+            for (int d = part; d < kD * 32; d += 4) sk[key * ldk + d] = blk >= 0 && d < dim ? widen(src[page_elem(p.tiled, dim, slot, d)]) : 0.f;
             if (part == 0) sr[key] = blk < 0 ? 0.f : p.inv_rms ? p.inv_rms[(size_t)blk * kBlockTokens + slot] * p.scale : p.scale;
         }
         __syncthreads();
@@ -691,6 +691,7 @@ int create(ingot_skv** out, int n_layer, int n_head_kv, int head_dim, int dtype,
     ingot_skv* kv = new (std::nothrow) ingot_skv();
     if (!kv) return INGOT_ERR_NOMEM;
     kv->n_layer = n_layer; kv->n_head_kv = n_head_kv; kv->dim = head_dim; kv->dtype = dtype; kv->chunk = chunk; kv->window = window; kv->n_blocks = n_blocks;
+    kv->tiled = !scales && dtype == INGOT_F16 && head_dim % 64 == 0;
     kv->layer_elems = (size_t)n_blocks * n_head_kv * kBlockTokens * head_dim;
     const size_t bytes = kv->layer_elems * n_layer * (dtype == INGOT_F32 ? 4 : 2), scale_bytes = (size_t)n_layer * n_blocks * kBlockTokens * 4;
     cudaError_t e;

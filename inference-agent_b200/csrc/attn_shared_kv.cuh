@@ -11,6 +11,7 @@ struct ingot_skv {
     int device = 0, num_sms = 0;
     int n_layer = 0, n_head_kv = 0, dim = 0;  // dim: row length (padded head size)
     int dtype = INGOT_F32, chunk = 0, window = 0, n_blocks = 0;
+    bool tiled = false;  // pages in the order of page_elem()
     size_t layer_elems = 0;
     void* rows = nullptr;
     float* inv_rms = nullptr;  // [layer][block][16]; null in caches whose rows are the keys as they are (window form)
@@ -33,6 +34,14 @@ struct PageMap {
     }
 };
 inline PageMap page_map(const ingot_skv* kv) { return PageMap{kv->chunk, (kv->chunk + kBlockTokens - 1) / kBlockTokens, kv->window}; }
+
+// Element of a page of one KV head that holds column `col` of slot `slot`. Plain: row after row. Tiled (f16 rows of whole 64-column
+// units): [8-slot half][unit][8 slots][64 columns] with the 16-byte pieces of a slot XOR-swizzled by it - the shared-memory image the
+// tcgen05 kernels multiply, so that a page comes in as one contiguous copy; the 8 values of a piece stay together.
+__host__ __device__ __forceinline__ int page_elem(bool tiled, int row, int slot, int col) {
+    if (!tiled) return slot * row + col;
+    return (((slot >> 3) * (row >> 6) + (col >> 6)) * 8 + (slot & 7)) * 64 + ((((col >> 3) & 7) ^ (slot & 7)) << 3) + (col & 7);
+}
 
 struct SharedOut {
     float* f32;
@@ -84,6 +93,7 @@ struct AttendParams {
     int* status;
     int n_splits;   // decoding: CTAs per (token, KV head) over the keys
     float* part;    // [token][head][split][dim + 2]
+    bool tiled = false;           // order of the pages
     const float* sink = nullptr;  // per head: one more term exp(sink) of the denominator (null: none)
 };
 
@@ -94,7 +104,7 @@ int launch_shared_kv_plain(const AttendParams& p, int dtype, cudaStream_t stream
 // a step of single tokens (p.n_splits and p.part set).
 bool latent_decode_takes(int row, int rank);
 int latent_decode_heads(int n_head);
-int launch_latent_decode_sm100(ingot_skv* kv, int layer, const AttendParams& p, cudaStream_t stream);
+int launch_latent_decode_sm100(const ingot_skv* kv, const AttendParams& p, cudaStream_t stream);
 
 // tcgen05 form for portions of prompts over rows of 128 values (attn_shared_kv_sm100.cu); INGOT_ERR_UNSUPPORTED if the driver
 // cannot encode its tensor map.
