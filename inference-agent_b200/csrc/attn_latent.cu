@@ -455,7 +455,7 @@ __global__ void __launch_bounds__(kMergeThreads) latent_merge_kernel(const Atten
     const float inv = 1.0f / l;
     for (int d = threadIdx.x * 2; d < p.out_dim; d += kMergeThreads * 2) {
         float a = 0.f, b = 0.f;
-#pragma unroll 8
+#pragma unroll 16
         for (int s = 0; s < p.n_splits; s++) {
             const float2 v = *reinterpret_cast<const float2*>(part + s * ld + d);
             a = fmaf(s_f[s], v.x, a);
