@@ -389,7 +389,7 @@ int ingot_latent_append(ingot_skv* kv, int layer, const ingot_step* step, const 
 /* Latent queries f32 [n_tok][n_head * rank] into the first rank columns of the query rows. */
 int ingot_latent_queries(const ingot_skv* kv, const float* q_dev, int n_tok, int n_head, int rank, void* q_rows_dev, void* stream);
 /* out [n_tok][n_head * rank]: sum over the visible keys of softmax(q_row . row * scale) times the first rank columns of the row;
- * sink_dev [n_head] (may be null): the denominator also holds exp(sink). impl: 0 = library's choice, 1 = the plain f32-arithmetic
+ * sink_dev [n_head] (may be null): one more term of each head's softmax sum, exp(sink), without a value. impl: 0 = library's choice, 1 = the plain f32-arithmetic
  * kernel, 2 = the warp-level tensor-core kernel (f16 rows, row length a multiple of 32, rank a multiple of 16 and at most 512), 3 =
  * the tcgen05 kernel (single tokens; f16 rows, row length a multiple of 64 and at least rank rounded up to 128, rank at most 512). */
 int ingot_latent_attend(ingot_skv* kv, int layer, const ingot_step* step, const void* q_rows_dev, int n_head, int rank, float scale,

@@ -3,7 +3,7 @@
 //
 // The mechanism, per head h:
 //     score(i, j) = (q_i . U_h c_j + rot(q_i') . rot(k_j')) * scale,      output_i = sum_j a_ij V_h c_j
-// with a_ij the softmax over the visible keys whose denominator may hold one more term exp(sink_h). Two equal ways to compute it:
+// with a_ij the softmax over the visible keys, its sum taken with one more term exp(sink_h) where there are sinks. Two equal ways to compute it:
 //   on the rows       q_i . U_h c_j = (U_h^T q_i) . c_j and sum_j a_ij V_h c_j = V_h (sum_j a_ij c_j): the query is taken into the
 //                     latent space once, the cached row [c | rot] is the key and its first part the value of every head, V_h
 //                     follows once per token. Reads each cached row once for all heads: decoded tokens and short portions.

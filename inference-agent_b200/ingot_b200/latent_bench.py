@@ -27,7 +27,7 @@ def config(size):
              "mixer": {"heads": heads, "dim": dim, "rot_dim": rot, "vdim": vdim, "kv_rank": rank, "scale": (dim + rot) ** -0.5, "rot": {"base": 500000.0, "dims": rot},
                        "mask": {"size": window}}}
     return {"architecture": "Banevik", "layers": [layer] * 3, "loop": {"start": 1, "stop": 2, "times": 2}, "norm": {"eps": 1e-6}, "vocab": VOCAB, "width": width,
-            "logit_softcap": 30.0, "embedding": {"bigram": {"buckets": 65521, "mul_prev": 31, "mul_cur": 17}}}
+            "logit_softcap": 30.0, "embedding": {"bigram": {"buckets": 65521, "mul_prev": 1009, "mul_cur": 8191}}}
 
 
 def weight_shapes(cfg):

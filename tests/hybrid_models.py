@@ -1,5 +1,5 @@
 """Small random models for the tests of the model-folder backend: configurations and weights of the hybrid recurrent design (the latent
-design's are in latent_moe_models.py), folders, and the checker's logits of either."""
+design's are in latent_moe_models.py), folders, and the plain implementations' logits."""
 import json
 import os
 

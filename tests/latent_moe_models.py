@@ -1,5 +1,5 @@
-"""Small random models of the looped latent-attention / mixture-of-experts design for the tests: configurations, weights, and the
-checker's logits (folders are written by hybrid_models.write)."""
+"""Small random models of the looped latent-attention / mixture-of-experts design for the tests: configurations, weights, and
+the plain implementation's logits (folders are written by hybrid_models.write)."""
 import numpy as np
 
 import latent_moe_reference as R

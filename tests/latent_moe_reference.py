@@ -1,4 +1,4 @@
-"""Plain NumPy statement of the looped latent-attention / mixture-of-experts decoder ("Banevik"), used as the checker of the CUDA path.
+"""Plain NumPy statement of the looped latent-attention / mixture-of-experts decoder ("Banevik"): what the CUDA path is tested against.
 
 The slow textbook form in float64 (or whatever dtype the weights have): one function per mechanism, loops over tokens, heads and
 experts, no code shared with the product. A model is a dict of weights (name -> ndarray) and the parsed config.json.
@@ -7,7 +7,7 @@ import numpy as np
 
 
 def rms(x, eps):
-    """x divided by its root mean square over the last axis; eps inside the root."""
+    """x / sqrt(mean(x^2) + eps) over the last axis."""
     return x / np.sqrt(np.mean(np.square(x), axis=-1, keepdims=True) + eps)
 
 
@@ -17,7 +17,7 @@ def offset_norm(x, w, eps):
 
 
 def bigram_rows(tokens, buckets, mul_prev, mul_cur):
-    """Table row of every token from it and the one before; a sequence's first token has the last row to itself."""
+    """Table row of every token, hashed from the pair it ends; the row behind the hashed ones stands for having no predecessor."""
     rows = [buckets]
     for a, b in zip(tokens[:-1], tokens[1:]):
         rows.append((int(a) * mul_prev + int(b) * mul_cur) % buckets)
@@ -46,7 +46,7 @@ def rotate(x, positions, dims, base):
 
 
 def window_visible(n, size):
-    """[n, n] bool: query i sees itself and the size - 1 tokens before it (size 0: all of them)."""
+    """[n, n] bool: query i sees keys i - size + 1 .. i (size 0: 0 .. i)."""
     i, j = np.arange(n)[:, None], np.arange(n)[None, :]
     return (j <= i) & ((i - j < size) | (size == 0))
 
@@ -81,7 +81,7 @@ def latent_attention(h, W, p, m, eps):
 
 
 def route(h, w_router, top):
-    """(chosen experts [n, top], their sigmoid scores [n, top]): the largest scores, as they are."""
+    """(experts [n, top], weights [n, top]): the top sigmoid scores, larger first; nothing is normalised."""
     s = 1.0 / (1.0 + np.exp(-(h @ w_router.T)))
     best = np.argsort(-s, axis=1, kind="stable")[:, :top]
     return best, np.take_along_axis(s, best, axis=1)

@@ -284,7 +284,7 @@ def test_decoding_over_many_keys(shape, n, impl):
         assert np.abs(g[-3:] - want[-3:]).max() < 1e-2 * max(1, np.abs(want).max())
 
 
-EXPANDED = [((3, 10, 6, 21, 19), 14), ((4, 128, 64, 512, 300), 128), ((2, 64, 64, 64, 0), 64), ((5, 100, 72, 48, 128), 80), ((2, 150, 30, 40, 1000), 100), ((7, 32, 32, 96, 72), 32),
+EXPANDED = [((3, 10, 6, 21, 19), 14), ((4, 128, 64, 512, 300), 128), ((2, 64, 64, 64, 0), 64), ((5, 100, 72, 48, 128), 80), ((2, 150, 30, 40, 1000), 100), ((7, 48, 24, 112, 90), 40),
             ((1, 64, 8, 32, 1), 8)]
 
 
