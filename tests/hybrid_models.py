@@ -107,9 +107,9 @@ def error(got, want):
 
 def off(got, want, clear=None):
     """The largest error; where some positions hang on a close choice of an expert (`clear` False), which rounding can turn, the
-    largest but for those and one in twenty others (their neighbours see their values)."""
+    largest but for those and one in ten others (their neighbours see their values)."""
     e = error(got, want)
     if clear is None or clear.all():
         return e.max()
     e = np.sort(e[clear])
-    return e[:len(e) - len(e) // 20 - 1].max() if len(e) > 1 else 0.0
+    return e[:len(e) - len(e) // 10 - 1].max() if len(e) > 1 else 0.0

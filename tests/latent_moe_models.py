@@ -69,7 +69,7 @@ def reference_logits(cfg, weights, tokens, residuals=None):
     return R.forward(tokens, {k: v.astype(np.float64) for k, v in weights.items()}, cfg, residuals)
 
 
-def clear_choices(cfg, weights, tokens, gap=0.08):
+def clear_choices(cfg, weights, tokens, gap=0.2):
     """[n] bool: positions at which every router's choice is clear (the best expert left out is `gap` behind, in logits)."""
     W = {k: v.astype(np.float64) for k, v in weights.items()}
     eps = cfg["norm"]["eps"]

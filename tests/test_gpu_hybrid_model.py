@@ -26,7 +26,7 @@ CONFIGS = {
     # latent attention and mixtures: nothing a multiple of anything, windows that differ, a loop in the middle, unequal layers
     "latent": L.config([L.layer(3, 10, 6, 14, 21, 19, experts=5, top=2, ff=20), L.layer(5, 12, 4, 9, 30, 33, base=500.0, experts=3, top=3, ff=13),
                         L.layer(2, 7, 8, 11, 17, 50), L.layer(3, 10, 6, 14, 21, 19, experts=4, top=1, ff=30)],
-                       vocab=103, width=46, loop=(1, 3, 2), bigram=(37, 29, 7)),
+                       vocab=103, width=46, loop=(1, 3, 2), bigram=(37, 19, 7)),
     # every expert is chosen (nothing hangs on a close choice), one head, a window of one page, a loop over all layers, no bigrams
     "latent_all": L.config([L.layer(1, 24, 16, 40, 64, 16, experts=2, top=2, ff=40), L.layer(20, 16, 2, 8, 40, 100, scale=0.15, experts=1, top=1, ff=8)],
                            vocab=90, width=64, loop=(0, 2, 2), softcap=5.0),
