@@ -415,18 +415,65 @@ typedef struct ingot_latent_expansion {
 int ingot_latent_attend_expanded(ingot_skv* kv, const ingot_step* step, const ingot_latent_expansion* x, float scale,
                                  const float* sink_dev, int out_dim, const ingot_act_out* out, void* stream);
 
+/* ---- Grouped-query attention over joined rows -------------------------------------------------------
+ * A window-form cache whose rows are [key | value] of one token and KV head side by side, in plain page order. */
+int ingot_skv_create_joined(ingot_skv** out, int n_layer, int n_head_kv, int row_length, int dtype, int window, int n_blocks);
+/* RMS norm of queries and keys before rotation: none, over each head with one weight [dim] for all, or over the whole projection with a
+ * weight [heads][dim]. Weights are zero in the padding. */
+enum { INGOT_QK_NORM_NONE = 0, INGOT_QK_NORM_HEAD = 1, INGOT_QK_NORM_ALL = 2 };
+typedef struct ingot_gqa_shape {
+    int n_head, n_head_kv;
+    int dim, vdim;   /* stored columns of a query / key and of a value head, zero-padded; dim + vdim is the row length */
+    int dim_count;   /* true size of a query / key head */
+    int rot_dims;    /* rotated values of a head, even: pairs (2 i, 2 i + 1); the rest passes unchanged */
+    int norm;        /* INGOT_QK_NORM_* */
+} ingot_gqa_shape;
+/* Columns q_off.. (n_head * dim), k_off.. (n_head_kv * dim) and v_off.. (n_head_kv * vdim) of proj_dev's rows. Writes the cache rows of the
+ * step's positions and the queries, q_out_dev [n_tok][n_head][dim] in the cache's type. turns_dev [rot_dims / 2]: turns per position;
+ * cosine and sine are multiplied by rot_gain. first_values_dev [n_tok][n_head_kv * vdim] (null: nothing is mixed): store_first != 0
+ * stores the values there, else they become (1 - mix) v + mix * stored before they are cached. Tables as for ingot_skv_append. */
+int ingot_gqa_append(ingot_skv* kv, int layer, const ingot_step* step, const float* proj_dev, int proj_ld, int q_off, int k_off, int v_off,
+                     const ingot_gqa_shape* shape, const float* q_norm_dev, const float* k_norm_dev, float eps, const double* turns_dev, float rot_gain,
+                     float* first_values_dev, int store_first, float mix, void* q_out_dev, const int32_t* tables_dev, const int32_t* first_page_dev,
+                     int max_blocks, void* stream);
+/* out [n_tok][n_head * vdim]: the softmax average of the visible values, scores q . k * scale. sink_dev [n_head] (may be null): one more
+ * term exp(sink) of a head's softmax sum. gate_dev (may be null): the result times sigmoid(z), z at gate_dev[t * gate_ld + ...], one per
+ * head or one per result column. impl: 0 = library's choice, 1 = the plain f32-arithmetic kernel, 2 = the warp-level tensor-core kernel
+ * with split keys (f16, sizes that are multiples of 16 and at most 256), 3 = the tcgen05 kernel (f16, sizes that are multiples of 16,
+ * keys at most 256, values at most 128, scale > 0), which 0 takes from INGOT_GQA_LONG_ROWS (token, head) rows per KV head on. The step may
+ * be some sequences of a larger one: n_seq and the per-sequence arrays are theirs, n_tok and the rows those of the whole. */
+#define INGOT_GQA_LONG_ROWS 128
+int ingot_gqa_attend(ingot_skv* kv, int layer, const ingot_step* step, const void* q_dev, const ingot_gqa_shape* shape, float scale, const float* sink_dev,
+                     const float* gate_dev, int gate_ld, int gate_per_head, const ingot_act_out* out, const int32_t* tables_dev, const int32_t* first_page_dev,
+                     int max_blocks, int impl, void* stream);
+
 /* ---- Mixture of experts -----------------------------------------------------------------------------
  * Pair p = token * top + k is a token's k-th expert; rows are the pairs sorted by expert, in token order within one. */
-enum { INGOT_ACT_NONE = 0, INGOT_ACT_RELU2 = 1 };  /* RELU2: the square of relu */
+enum { INGOT_ACT_NONE = 0, INGOT_ACT_RELU2 = 1, INGOT_ACT_SILU_GATED = 2 };  /* RELU2: the square of relu; SILU_GATED: silu(gate) * up */
 /* The top experts of each token by logit (the lower index of equal ones) with sigmoid(logit) as weight, and their sorting:
  * expert_of, weight_of, row_of [n_tok * top] by pair, pair_of, row_weight [n_tok * top] by row, group_start [n_expert + 1]. */
 int ingot_moe_route(const float* logits_dev, int ld, int n_tok, int n_expert, int top, int32_t* expert_of_dev, float* weight_of_dev,
                     int32_t* group_start_dev, int32_t* row_of_dev, int32_t* pair_of_dev, float* row_weight_dev, void* stream);
-/* bf16 planes [n_rows][n] of the rows from planes [n_tok][n] of the tokens (lo may be null). n a multiple of 8. */
+/* Routers over n_expert experts and n_identity identity experts behind them (whose output is the token's own input): scores are the softmax
+ * of all the logits, choices the `top` largest of score + correction within the `keep` best of `groups` equal runs of neighbours (a run is
+ * as good as its best choice), weights the scores of the chosen over their sum (+ 1e-20), times scale. At most 1024 outputs. */
+typedef struct ingot_moe_router {
+    int n_expert, n_identity, top, groups, keep;
+    float scale;
+    const float* correction;  /* device, [n_expert + n_identity]; may be null */
+} ingot_moe_router;
+/* As ingot_moe_route. Pairs of identity experts have no row: row_of is -1, their weights add up in self_gain_dev [n_tok], and only the
+ * first group_start[n_expert] rows exist. shared_gain_dev [n_tok] (may be null): sigmoid of the logit behind the router's. */
+int ingot_moe_route_grouped(const ingot_moe_router* router, const float* logits_dev, int ld, int n_tok, int32_t* expert_of_dev, float* weight_of_dev,
+                            int32_t* group_start_dev, int32_t* row_of_dev, int32_t* pair_of_dev, float* row_weight_dev, float* self_gain_dev,
+                            float* shared_gain_dev, void* stream);
+/* bf16 planes [n_rows][n] of the rows from planes [n_tok][n] of the tokens (lo may be null). n a multiple of 8. n_rows_dev (may be null):
+ * how many of the n_rows rows exist. */
 int ingot_moe_gather(void* hi_dev, void* lo_dev, const void* src_hi_dev, const void* src_lo_dev, const int32_t* pair_of_dev, int n_rows,
-                     int top, int n, void* stream);
+                     const int32_t* n_rows_dev, int top, int n, void* stream);
 /* out[row] = act(row_weight[row] * W_e x), W bf16 [n_expert][n_out][n_in], f32 arithmetic. x row of a row: its token's
- * (pair_of_dev given) or its own; row_weight_dev may be null. */
+ * (pair_of_dev given) or its own; row_weight_dev may be null. SILU_GATED: out[row] = row_weight[row] * silu(gate) * up, n_out a multiple of
+ * 32, W [n_expert][2 n_out][n_in] with each 32 gate rows followed by the 32 up rows of the same outputs. */
 int ingot_moe_linear(float* out_dev, const void* w_dev, const float* x_dev, int x_ld, int n_in, int n_out, int n_expert, int n_rows,
                      const int32_t* group_start_dev, const int32_t* pair_of_dev, int top, const float* row_weight_dev, int act, void* stream);
 /* x [n_tok][n] += the sum of each token's rows of [n_tok * top][n] (row_of_dev null, top 1: its own). */

@@ -1,0 +1,140 @@
+// Grouped-query attention of the model-folder backend (kernels: csrc/attn_gqa.cu, attn_gqa_sm100.cu).
+#include "layer_ops.h"
+
+namespace {
+
+// Frequencies of rotated pairs, in turns per position, and the factor of their sines and cosines. With "scaling" (YaRN): pairs that turn
+// more often than `fast` times within the `original` positions keep their frequency, those that turn less often than `slow` times have it
+// divided by `factor`, and those between are blended linearly by their index.
+struct Rotation {
+    std::vector<double> turns;
+    float gain = 1.f;
+    explicit Rotation(const Json& c) {
+        const int dims = get_int(c, "dims", 0);
+        if (dims % 2 != 0) throw std::runtime_error("model config: \"rot.dims\" must be even");
+        const double base = c.at("base").number(), two_pi = 2 * 3.14159265358979323846;
+        for (int i = 0; i < dims / 2; i++) turns.push_back(std::pow(base, -2.0 * i / dims) / two_pi);
+        if (!has(c, "scaling")) return;
+        const Json& s = c.at("scaling");
+        const double factor = s.at("factor").number(), original = s.at("original").number();
+        auto pair_that_turns = [&](double times) { return dims * std::log(original / (two_pi * times)) / (2 * std::log(base)); };
+        const double lo = std::max(std::floor(pair_that_turns(s.at("fast").number())), 0.0);
+        const double hi = std::min(std::ceil(pair_that_turns(s.at("slow").number())), double(dims - 1));
+        for (int i = 0; i < dims / 2; i++) {
+            const double slowed = std::min(std::max((i - lo) / std::max(hi - lo, 0.001), 0.0), 1.0);
+            turns[size_t(i)] *= slowed / factor + (1 - slowed);
+        }
+        gain = float(0.1 * std::log(factor) + 1.0);
+    }
+};
+
+// q, k, v and the output gate's logits are one product of the normed input; queries and keys are normed and rotated, values mixed with the
+// first mixing layer's, and keys and values cached side by side. Decoded tokens and short portions take the split-key kernel, portions of
+// many rows the tcgen05 one, each over its sequences of the step; the gate is applied where the result is stored as W_o's operand.
+class GroupedAttentionMixer : public Mixer {
+public:
+    GroupedAttentionMixer(LayerOps& ops, const AttentionKind& kind, const Json& c, const std::string& p) : gate_(kind.gate) {
+        const int heads = get_int(c, "heads"), kv_heads = get_int(c, "kv_heads"), dim = get_int(c, "dim"), vdim = get_int(c, "vdim"), d = ops.width;
+        if (heads % kv_heads != 0) throw std::runtime_error("model config: \"heads\" is not a multiple of \"kv_heads\"");
+        scale_ = get_float(c, "scale");
+        shape_.n_head = heads;
+        shape_.n_head_kv = kv_heads;
+        shape_.dim = round_up(dim, 16);
+        shape_.vdim = round_up(vdim, 16);
+        shape_.dim_count = dim;
+        shape_.norm = kind.qk_norm;
+        if (shape_.dim + shape_.vdim > 1024) throw std::runtime_error("model config: a key and a value of more than 1024 values together are not supported");
+        if (has(c, "rot")) {
+            const Rotation rot(c.at("rot"));
+            shape_.rot_dims = int(rot.turns.size()) * 2;
+            if (shape_.rot_dims > dim) throw std::runtime_error("model config: \"rot.dims\" is more than \"dim\"");
+            rot_gain_ = rot.gain;
+            turns_ = static_cast<double*>(ops.alloc(rot.turns.size() * sizeof(double)));
+            cuda_check(cudaMemcpy(turns_, rot.turns.data(), rot.turns.size() * sizeof(double), cudaMemcpyHostToDevice), "cudaMemcpy");
+        }
+        const int window = has(c, "mask") ? get_int(c.at("mask"), "size") : 0;
+        cache_ = ops.cache_group(kv_heads, shape_.dim + shape_.vdim, 0, window, CacheGroup::joined, &cache_layer_);
+
+        const Groups in = flat(d), q = {heads, dim, shape_.dim}, k = {kv_heads, dim, shape_.dim}, v = {kv_heads, vdim, shape_.vdim}, out = {heads, vdim, shape_.vdim};
+        const Groups g = gate_ == OutputGate::per_head ? flat(heads) : out;
+        k_off_ = q.width();
+        v_off_ = k_off_ + k.width();
+        gate_off_ = v_off_ + v.width();
+        proj_ld_ = gate_off_ + (gate_ == OutputGate::none ? 0 : g.width());
+        out_ld_ = out.width();
+        std::vector<Part> parts = {Part{p + "q", {q.count(), d}, q, in, 0}, Part{p + "k", {k.count(), d}, k, in, k_off_}, Part{p + "v", {v.count(), d}, v, in, v_off_}};
+        if (gate_ != OutputGate::none) parts.push_back(Part{p + "g", {g.count(), d}, g, in, gate_off_});
+        w_in_ = ops.matrix(proj_ld_, in.padded, parts);
+        w_o_ = ops.matrix(p + "o", in, out);
+        if (shape_.norm == INGOT_QK_NORM_HEAD) {
+            q_norm_ = ops.vector(p + "q.norm", {dim}, {1, dim, shape_.dim});
+            k_norm_ = ops.vector(p + "k.norm", {dim}, {1, dim, shape_.dim});
+        } else if (shape_.norm == INGOT_QK_NORM_ALL) {
+            q_norm_ = ops.vector(p + "q.norm", {q.count()}, q);
+            k_norm_ = ops.vector(p + "k.norm", {k.count()}, k);
+        }
+        if (kind.sink) sink_ = ops.vector(p + "sink", {heads}, {1, heads, heads});
+        if (has(c, "v_mix") && c.at("v_mix").boolean()) {
+            mixes_ = true;
+            first_ = ops.mixed_values == 0;
+            if (first_) ops.mixed_values = v.width();
+            else if (ops.mixed_values != v.width()) throw std::runtime_error("model config: layers that mix values need equal \"kv_heads\" and \"vdim\"");
+            if (!first_) mix_ = ops.scalar(p + "vmix");
+            ops.need(kFirstValue, v.width());
+        }
+        ops.need(kProj, proj_ld_);
+        ops.need(kQuery, ops.opt.f32 ? q.width() : q.width() / 2);
+        ops.need(kMix, out_ld_);
+        ops.need(kBranch, in.padded);
+    }
+    void run(LayerOps& ops, const StepCtx& s, const Norms& n) override {
+        float *proj = ops.buf(kProj), *mix = ops.buf(kMix);
+        const CacheGroup& g = *cache_;
+        const int layer = cache_layer_ + ops.pass, n_seq = s.st.n_seq;
+        ops.norm_project(s, proj, w_in_, n.in);
+        ingot_check(ingot_gqa_append(g.kv, layer, &s.st, proj, proj_ld_, 0, k_off_, v_off_, &shape_, q_norm_, k_norm_, ops.eps, turns_, rot_gain_,
+                                     mixes_ ? ops.buf(kFirstValue) : nullptr, first_, mix_, ops.buf(kQuery), g.tables, g.first_page, g.width, ops.stream));
+        const ingot_act_out out = ops.operand(s, mix, out_ld_, false);
+        // sequences come in ascending order of their portions: the long ones are the last
+        int from = n_seq;
+        if (!ops.opt.f32)
+            while (from > 0 && (long long)s.lens[from - 1] * (shape_.n_head / shape_.n_head_kv) >= INGOT_GQA_LONG_ROWS) from--;
+        attend(ops, s, layer, 0, from, out);
+        attend(ops, s, layer, from, n_seq, out);
+        ops.operand_ready(s, out_ld_);
+        ops.project_residual(s, w_o_, mix, n);
+    }
+
+private:
+    // The sequences first..last-1 of the step.
+    void attend(LayerOps& ops, const StepCtx& s, int layer, int first, int last, const ingot_act_out& out) {
+        if (first == last) return;
+        const CacheGroup& g = *cache_;
+        ingot_step st = s.st;
+        st.n_seq = last - first;
+        st.max_len = s.lens[last - 1];
+        st.row_start += first;
+        st.len += first;
+        st.pos0 += first;
+        st.slot += first;
+        const float* gate = gate_ == OutputGate::none ? nullptr : ops.buf(kProj) + gate_off_;
+        ingot_check(ingot_gqa_attend(g.kv, layer, &st, ops.buf(kQuery), &shape_, scale_, sink_, gate, proj_ld_, gate_ == OutputGate::per_head, &out,
+                                     g.tables + size_t(first) * g.width, g.first_page + first, g.width, 0, ops.stream));
+    }
+
+    const OutputGate gate_;
+    ingot_gqa_shape shape_ = {};
+    int k_off_, v_off_, gate_off_, proj_ld_, out_ld_, cache_layer_ = 0;
+    float scale_, rot_gain_ = 1.f, mix_ = 0.f;
+    bool mixes_ = false, first_ = false;
+    CacheGroup* cache_;
+    Matrix w_in_, w_o_;
+    float *q_norm_ = nullptr, *k_norm_ = nullptr, *sink_ = nullptr;
+    double* turns_ = nullptr;
+};
+
+}  // namespace
+
+std::unique_ptr<Mixer> make_grouped_attention(LayerOps& ops, const AttentionKind& kind, const Json& config, const std::string& prefix) {
+    return std::make_unique<GroupedAttentionMixer>(ops, kind, config, prefix);
+}

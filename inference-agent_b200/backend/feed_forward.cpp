@@ -3,7 +3,7 @@
 
 namespace {
 
-// Gated feed-forward: W_down (gelu(W_gate h) * (W_up h)).
+// Gated feed-forward: W_down (act(W_gate h) * (W_up h)), act the design's.
 class GatedFeedForward : public FeedForward {
 public:
     GatedFeedForward(LayerOps& ops, const Json& c, const std::string& p) {
@@ -15,11 +15,16 @@ public:
         ops.need(kBranch, d.padded);
         ops.tc_shape(ff.padded, 2 * ff.padded);
     }
-    void run(LayerOps& ops, const StepCtx& s, const float* norm, const float* next_norm) override {
-        ops.gated_project(s, w_gu_, norm);
-        ops.project_residual(s, w_down_, ops.buf(kMid), next_norm);
+    void run(LayerOps& ops, const StepCtx& s, const Norms& n) override {
+        ops.gated_project(s, w_gu_, n.in);
+        ops.project_residual(s, w_down_, ops.buf(kMid), n);
     }
-    void branch(LayerOps& ops, const StepCtx& s, const float* norm) override {
+    // The result for h = norm(x) in the planes or kNormed, as the product of a residual sum.
+    void product(LayerOps& ops, const StepCtx& s, const Norm& norm, ingot_residual_norm& r) {
+        ops.gated_project_normed(s, w_gu_, norm);
+        ops.product(s, w_down_, ops.buf(kMid), r);
+    }
+    void branch(LayerOps& ops, const StepCtx& s, const Norm& norm) override {
         ops.gated_project(s, w_gu_, norm);
         ops.project(s, ops.buf(kBranch), w_down_, ops.buf(kMid), w_down_.n_in);
         ops.set_branch(Branch{ops.buf(kBranch), nullptr, 1});
@@ -29,41 +34,101 @@ private:
     Matrix w_gu_, w_down_;
 };
 
-// Mixture of experts: router scores sigmoid(W_router h), the `top` experts with the largest; expert e on w h, w its score:
-// W_down,e relu(W_up,e (w h))^2. The weight is applied to the product W_up h, which is the same and keeps h in one copy. Tensor-core
-// path: rows gathered by expert, two grouped products with the activation in the first one's epilogue; the rows of the second go into
-// the residual sum where the mixer's output does.
+// Mixture of experts. Tensor-core path: rows gathered by expert, two grouped products with the activation in the first one's epilogue; the
+// rows of the second go into the residual sum. Two forms, by the design:
+//   squared relu   router scores sigmoid(W_router h), the `top` largest; expert e on w h, w its score: W_down,e relu(W_up,e (w h))^2. The
+//                  weight is applied to the product W_up h, which is the same and keeps h in one copy.
+//   gated          softmax scores with a correction that counts for the choice only, groups of experts, weights that sum to router.scale,
+//                  identity experts (ingot_moe_route_grouped); expert e: W_down,e (silu(W_gate,e h) * (W_up,e h)), the weight on the
+//                  product's operand; gate and up rows of a stack alternate in runs of 32. A shared expert for every token with a gate of
+//                  its own, whose row is the last of the router's matrix. The residual sum takes the routed rows, the shared expert's
+//                  product with its gate, and h itself times the identity experts' weights.
 class MixtureFeedForward : public FeedForward {
 public:
-    MixtureFeedForward(LayerOps& ops, const Json& c, const std::string& p) {
-        experts_ = get_int(c.at("router"), "experts", 1, 1 << 16);
-        top_ = get_int(c.at("router"), "top", 1, experts_);
-        const Groups ff = flat(get_int(c.at("expert"), "ff")), d = flat(ops.width), e = flat(experts_);
-        std::vector<Part> up, down;
+    MixtureFeedForward(LayerOps& ops, const Json& c, const std::string& p) : gated_(ops.design.gated_experts) {
+        const Json& r = c.at("router");
+        experts_ = get_int(r, "experts", 1, 1 << 16);
+        const int identity = gated_ && has(r, "identity") ? get_int(r, "identity", 0, 1 << 16) : 0, outputs = experts_ + identity;
+        top_ = get_int(r, "top", 1, outputs);
+        const Groups ff = gated_ ? Groups{1, get_int(c.at("expert"), "ff"), round_up(get_int(c.at("expert"), "ff"), 32)} : flat(get_int(c.at("expert"), "ff")), d = flat(ops.width);
+        const bool shared = gated_ && has(c, "shared");
+        const Groups e = flat(outputs + shared);
+        std::vector<Part> up, down, router = {Part{p + "router", {outputs, d.count()}, {1, outputs, e.padded}, d}};
         for (int i = 0; i < experts_; i++) {
             const std::string q = p + "e" + std::to_string(i) + ".";
-            up.push_back(Part{q + "up", {ff.count(), d.count()}, ff, d, i * ff.padded});
+            if (gated_) {  // runs of 32 rows: gate, up, gate, ..
+                for (int run = 0; run * 32 < ff.size; run++) {
+                    const Groups rows = {1, std::min(32, ff.size - run * 32), 32};
+                    const int at = i * 2 * ff.padded + run * 64;
+                    up.push_back(Part{q + "gate", {ff.count(), d.count()}, rows, d, at, 0, run * 32});
+                    up.push_back(Part{q + "up", {ff.count(), d.count()}, rows, d, at + 32, 0, run * 32});
+                }
+            } else {
+                up.push_back(Part{q + "up", {ff.count(), d.count()}, ff, d, i * ff.padded});
+            }
             down.push_back(Part{q + "down", {d.count(), ff.count()}, d, ff, i * d.padded});
         }
-        w_router_ = ops.matrix(p + "router", e, d);
-        w_up_ = ops.matrix(experts_ * ff.padded, d.padded, up, 0, true);
+        if (shared) {
+            router.push_back(Part{p + "shared.sg", {1, d.count()}, {1, 1, 1}, d, outputs});
+            shared_ = std::make_unique<GatedFeedForward>(ops, c.at("shared"), p + "shared.");
+        }
+        up_rows_ = (gated_ ? 2 : 1) * ff.padded;
+        w_router_ = ops.matrix(e.padded, d.padded, router);
+        w_up_ = ops.matrix(experts_ * up_rows_, d.padded, up, 0, true);
         w_down_ = ops.matrix(experts_ * d.padded, ff.padded, down, 0, true);
         ff_ = ff.padded;
         d_ = d.padded;
         const size_t pairs = size_t(ops.max_step) * top_;
         auto ints = [&](size_t n) { return static_cast<int32_t*>(ops.alloc(n * 4, true)); };
+        auto floats = [&](size_t n) { return static_cast<float*>(ops.alloc(n * 4, true)); };
         expert_of_ = ints(pairs);
         row_of_ = ints(pairs);
         pair_of_ = ints(pairs);
         start_ = ints(size_t(experts_) + 1);
-        weight_of_ = static_cast<float*>(ops.alloc(pairs * 4, true));
-        row_weight_ = static_cast<float*>(ops.alloc(pairs * 4, true));
+        weight_of_ = floats(pairs);
+        row_weight_ = floats(pairs);
+        if (gated_) {
+            route_ = {experts_, identity, top_, 1, 1, get_float(r, "scale"), ops.vector(p + "correction", {outputs}, {1, outputs, outputs})};
+            if (has(r, "groups")) {
+                route_.groups = get_int(r.at("groups"), "count", 1, outputs);
+                route_.keep = get_int(r.at("groups"), "keep", 1, route_.groups);
+                if (outputs % route_.groups != 0) throw std::runtime_error("model config: the router's outputs do not form equal groups");
+            }
+            if (top_ > outputs / route_.groups * route_.keep) throw std::runtime_error("model config: \"top\" is more than the kept groups hold");
+            if (identity > 0) self_gain_ = floats(size_t(ops.max_step));
+            if (shared) shared_gain_ = floats(size_t(ops.max_step));
+        }
         ops.need(kRouter, e.padded);
         ops.need(kExpertMid, top_ * ff_);   // f32, or two bf16 planes
         ops.need(kExpertOut, top_ * d_);
         if (!ops.opt.f32) ops.need(kExpertIn, top_ * d_);
     }
-    void branch(LayerOps& ops, const StepCtx& s, const float* norm) override {
+    void branch(LayerOps& ops, const StepCtx& s, const Norm& norm) override {
+        if (gated_) throw std::runtime_error("model: gated experts have no form beside the mixer");
+        route_and_run(ops, s, norm);
+        ops.set_branch(Branch{ops.buf(kExpertOut), row_of_, top_});
+    }
+    void run(LayerOps& ops, const StepCtx& s, const Norms& n) override {
+        route_and_run(ops, s, n.in);
+        ingot_residual_norm r = {};
+        if (shared_) shared_->product(ops, s, n.in, r);
+        if (!gated_ && !n.post && !n.next.b) {
+            ops.set_branch(Branch{ops.buf(kExpertOut), row_of_, top_});
+            ops.add_branch(s);
+            return;
+        }
+        r.gain = shared_gain_;
+        r.branch = ops.buf(kExpertOut);
+        r.row_of = row_of_;
+        r.top = top_;
+        r.self_gain = self_gain_;
+        r.self = n.in;
+        ops.finish(s, r, n);
+    }
+
+private:
+    // kExpertOut: the experts' results, pair by pair (row_of_), for h = norm(x); h stays in the planes or kNormed.
+    void route_and_run(LayerOps& ops, const StepCtx& s, const Norm& norm) {
         const int rows = s.st.n_tok * top_;
         float *mid = ops.buf(kExpertMid), *out = ops.buf(kExpertOut), *z = ops.buf(kRouter);
         if (s.tc) {
@@ -73,41 +138,43 @@ public:
             ops.norm_rows(s, norm);
             ops.project(s, z, w_router_, ops.buf(kNormed), d_);
         }
-        ingot_check(ingot_moe_route(z, w_router_.n_out, s.st.n_tok, experts_, top_, expert_of_, weight_of_, start_, row_of_, pair_of_, row_weight_, ops.stream));
+        if (gated_)
+            ingot_check(ingot_moe_route_grouped(&route_, z, w_router_.n_out, s.st.n_tok, expert_of_, weight_of_, start_, row_of_, pair_of_, row_weight_, self_gain_, shared_gain_,
+                                                ops.stream));
+        else
+            ingot_check(ingot_moe_route(z, w_router_.n_out, s.st.n_tok, experts_, top_, expert_of_, weight_of_, start_, row_of_, pair_of_, row_weight_, ops.stream));
+        const int act = gated_ ? INGOT_ACT_SILU_GATED : INGOT_ACT_RELU2;
         if (s.tc) {
             void *h_hi, *h_lo;
             ingot_linear_ws_planes(ops.ws, &h_hi, &h_lo);
             const bool pair = s.planes > 1;
             char *in_hi = reinterpret_cast<char*>(ops.buf(kExpertIn)), *mid_hi = reinterpret_cast<char*>(mid);
             void *in_lo = pair ? in_hi + size_t(rows) * d_ * 2 : nullptr, *mid_lo = pair ? mid_hi + size_t(rows) * ff_ * 2 : nullptr;
-            ingot_check(ingot_moe_gather(in_hi, in_lo, h_hi, h_lo, pair_of_, rows, top_, d_, ops.stream));
+            ingot_check(ingot_moe_gather(in_hi, in_lo, h_hi, h_lo, pair_of_, rows, start_ + experts_, top_, d_, ops.stream));
             ingot_grouped_gemm g = {};
             g.n_rows = rows;
             g.rows_per_group = s.st.n_tok;
             g.n_groups = experts_;
             g.group_start = start_;
-            g.a_hi = in_hi; g.a_lo = in_lo; g.w = w_up_.data; g.n_in = d_; g.n_out = ff_;
-            g.row_scale = row_weight_; g.act = INGOT_ACT_RELU2; g.out_hi = mid_hi; g.out_lo = mid_lo;
+            g.a_hi = in_hi; g.a_lo = in_lo; g.w = w_up_.data; g.n_in = d_; g.n_out = up_rows_;
+            g.row_scale = row_weight_; g.act = act; g.out_hi = mid_hi; g.out_lo = mid_lo;
             cuda_check(ingot_grouped_tc_run(ops.ws, &g, ops.stream), "experts");
             g.a_hi = mid_hi; g.a_lo = mid_lo; g.w = w_down_.data; g.n_in = ff_; g.n_out = d_;
             g.row_scale = nullptr; g.act = INGOT_ACT_NONE; g.out_hi = g.out_lo = nullptr; g.out = out;
             cuda_check(ingot_grouped_tc_run(ops.ws, &g, ops.stream), "experts");
         } else {
-            ingot_check(ingot_moe_linear(mid, w_up_.data, ops.buf(kNormed), d_, d_, ff_, experts_, rows, start_, pair_of_, top_, row_weight_, INGOT_ACT_RELU2, ops.stream));
+            ingot_check(ingot_moe_linear(mid, w_up_.data, ops.buf(kNormed), d_, d_, ff_, experts_, rows, start_, pair_of_, top_, row_weight_, act, ops.stream));
             ingot_check(ingot_moe_linear(out, w_down_.data, mid, ff_, ff_, d_, experts_, rows, start_, nullptr, top_, nullptr, INGOT_ACT_NONE, ops.stream));
         }
-        ops.set_branch(Branch{out, row_of_, top_});
-    }
-    void run(LayerOps& ops, const StepCtx& s, const float* norm, const float*) override {
-        branch(ops, s, norm);
-        ops.add_branch(s);
     }
 
-private:
-    int experts_, top_, ff_, d_;
+    const bool gated_;
+    int experts_, top_, ff_, d_, up_rows_;
     Matrix w_router_, w_up_, w_down_;
+    std::unique_ptr<GatedFeedForward> shared_;
+    ingot_moe_router route_ = {};
     int32_t *expert_of_, *row_of_, *pair_of_, *start_;
-    float *weight_of_, *row_weight_;
+    float *weight_of_, *row_weight_, *self_gain_ = nullptr, *shared_gain_ = nullptr;
 };
 
 }  // namespace

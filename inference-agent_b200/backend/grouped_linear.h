@@ -13,7 +13,8 @@ struct ingot_grouped_gemm {
     int n_in, n_out, n_groups;     // lengths are multiples of 8
     const int32_t* group_start;    // device, [n_groups + 1]
     const float* row_scale;        // device, [n_rows]: multiplies the accumulator (null: none), then
-    int act;                       // INGOT_ACT_*
+    int act;                       // INGOT_ACT_*; SILU_GATED: n_out counts gate and up columns (runs of 32 of each), the result is half as wide
+                                   // and the factor follows the activation
     float* out;                    // f32 [n_rows][n_out], or
     void *out_hi, *out_lo;         // bf16 plane(s) of the same shape (out_hi non-null)
 };

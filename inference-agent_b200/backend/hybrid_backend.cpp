@@ -1,12 +1,12 @@
 // Decoder-only models whose layers are listed one by one in their configuration, each with a mixer of its own kind - recurrent,
-// attention, or several side by side - and an optional feed-forward ("Besudra", "Banevik" and designs like them).
+// attention, or several side by side - and an optional feed-forward ("Besudra", "Banevik", "Silevik" and designs like them).
 //
 // Reading guide.
 //   layer_ops.h     what layers are written in (LayerOps), and the interfaces Mixer and FeedForward: weights, per-sequence state and
 //                   launches of one kind each. LayerOps picks the kernel by the number of tokens: weight-streaming GEMV for one
 //                   token, tcgen05 GEMM for more (f32 kernels in the 32-bit form).
-//   recurrent_layers.cpp, latent_layers.cpp, feed_forward.cpp   the kinds. A new one is a class there plus a line in make_mixer()
-//                   or make_feed_forward().
+//   recurrent_layers.cpp, latent_layers.cpp, attention_layers.cpp, feed_forward.cpp   the kinds. A new one is a class there plus a line
+//                   in make_mixer() or make_feed_forward().
 //   HybridBackend   the step: one ragged batch of portions of several sequences, state slots and cache pages, the loop over layers
 //                   (some of which may run several times, each pass with a state of its own), logits. A Design is what a model
 //                   family fixes; everything else comes from its configuration.
@@ -22,6 +22,8 @@ std::unique_ptr<Mixer> make_mixer(const std::string& type, LayerOps& ops, const 
     if (type == "mamba1") return make_selective_scan(ops, config, prefix);
     if (type == "parallel") return make_parallel(ops, config, prefix);
     if (type == "latent_attention") return make_latent_attention(ops, config, prefix);
+    for (const AttentionKind& kind : ops.design.attention)
+        if (type == kind.type) return make_grouped_attention(ops, kind, config, prefix);
     throw std::runtime_error("model config: unknown layer type \"" + type + "\"");
 }
 
@@ -34,17 +36,10 @@ std::unique_ptr<FeedForward> make_feed_forward(LayerOps& ops, const Json& config
 
 // ---- the model -------------------------------------------------------------------------------------------------------
 
-// What a design fixes and its configuration does not say.
-struct Design {
-    float norm_offset;     // the norms' weights are stored around this: x / rms(x) * (norm_offset + w)
-    bool parallel;         // a layer adds mixer(norm1 x) + ff(norm2 x), both of the same x, instead of one after the other
-    bool tied_head;        // the output matrix is the embedding table
-};
-
 class HybridBackend : public ModelBackend {
 public:
     HybridBackend(const ModelDir& dir, const EngineOptions& opt, const Design& design)
-        : design_(design), ops_(dir, opt, opt.max_step_tokens > 0 ? opt.max_step_tokens : opt.max_tokens), max_seqs_(opt.max_seqs), max_ctx_(opt.max_tokens) {
+        : design_(design), ops_(dir, opt, design, opt.max_step_tokens > 0 ? opt.max_step_tokens : opt.max_tokens), max_seqs_(opt.max_seqs), max_ctx_(opt.max_tokens) {
         if (opt.max_tokens < 1 || opt.max_seqs < 1) throw std::runtime_error("engine: needs at least one token and one sequence");
         int device = 0;
         cuda_check(cudaGetDevice(&device), "cudaGetDevice");
@@ -53,12 +48,12 @@ public:
         n_vocab_ = get_int(c, "vocab");
         ops_.width = get_int(c, "width");
         ops_.eps = get_float(c.at("norm"), "eps");
-        ops_.norm_offset = design.norm_offset;
         const Groups d = flat(ops_.width);
         ops_.x = static_cast<float*>(ops_.alloc(size_t(ops_.max_step) * d.padded * 4, true));
         ops_.need(kNormed, d.padded);
         ops_.tc_shape(d.padded, round_up(n_vocab_, 8));
         embed_ = ops_.matrix("embed", flat(n_vocab_), d);
+        if (has(c, "embedding") && has(c.at("embedding"), "scale")) embed_scale_ = get_float(c.at("embedding"), "scale");
         if (has(c, "embedding") && has(c.at("embedding"), "bigram")) {
             const Json& b = c.at("embedding").at("bigram");
             bigram_buckets_ = get_int(b, "buckets");
@@ -85,10 +80,12 @@ public:
             Layer L;
             L.type = layers[i].at("type").str();
             ops_.passes = in_loop(i) ? loop_times_ : 1;
-            L.norm1 = ops_.norm_vector(p + "norm1");
+            L.norm1 = ops_.norm(p + "norm1");
+            if (design.sandwich) L.norm1b = ops_.norm(p + "norm1b");
             L.mixer = make_mixer(L.type, ops_, layers[i].at("mixer"), p + "mix.");
             if (layers[i].has("mlp") && !layers[i].at("mlp").is_null()) {
-                L.norm2 = ops_.norm_vector(p + "norm2");
+                L.norm2 = ops_.norm(p + "norm2");
+                if (design.sandwich) L.norm2b = ops_.norm(p + "norm2b");
                 L.mlp = make_feed_forward(ops_, layers[i].at("mlp"), p + "mlp.");
             }
             scan_threads_ = std::max(scan_threads_, L.mixer->scan_threads());
@@ -97,7 +94,8 @@ public:
             lru_scratch_ = std::max(lru_scratch_, L.mixer->lru_scratch_per_chunk());
             layers_.push_back(std::move(L));
         }
-        final_norm_ = ops_.norm_vector("final.norm");
+        // a factor of the logits rides on the norm before them
+        final_norm_ = ops_.norm("final.norm", has(c, "logit_scale") ? get_float(c, "logit_scale") : 1.f);
         if (design.tied_head) {
             head_ = embed_;
             table_bytes -= size_t(embed_.n_out) * embed_.n_in * 2;
@@ -123,9 +121,10 @@ public:
             if (g->window > 0) blocks = std::min(pages, (long long)max_seqs_ * (g->pages_seen() + 2) + ops_.max_step / INGOT_BLOCK_TOKENS);
             if (blocks > (1 << 26)) throw std::runtime_error("engine: cache pool too large");
             const int dtype = opt.f32 ? INGOT_F32 : INGOT_F16;
-            if (g->scales && g->window > 0) throw std::runtime_error("engine: no cache form for scaled rows behind a window");
-            ingot_check(g->scales ? ingot_skv_create(&g->kv, g->n_layer, g->kv_heads, g->dim, dtype, g->chunk, int(blocks))
-                                  : ingot_skv_create_window(&g->kv, g->n_layer, g->kv_heads, g->dim, dtype, g->window, int(blocks)));
+            if (g->form == CacheGroup::scaled && g->window > 0) throw std::runtime_error("engine: no cache form for scaled rows behind a window");
+            ingot_check(g->form == CacheGroup::scaled  ? ingot_skv_create(&g->kv, g->n_layer, g->kv_heads, g->dim, dtype, g->chunk, int(blocks))
+                        : g->form == CacheGroup::plain ? ingot_skv_create_window(&g->kv, g->n_layer, g->kv_heads, g->dim, dtype, g->window, int(blocks))
+                                                       : ingot_skv_create_joined(&g->kv, g->n_layer, g->kv_heads, g->dim, dtype, g->window, int(blocks)));
             g->pool = BlockPool(int(blocks), max_seqs_, ingot_skv_pages(g->chunk, max_ctx_));
         }
         embed_status_ = static_cast<int*>(ops_.alloc(sizeof(int), true));
@@ -241,7 +240,7 @@ public:
 private:
     struct Layer {
         std::string type;
-        float *norm1 = nullptr, *norm2 = nullptr;
+        Norm norm1, norm1b, norm2, norm2b;  // before and after the mixer, before and after the feed-forward
         std::unique_ptr<Mixer> mixer;
         std::unique_ptr<FeedForward> mlp;
     };
@@ -265,7 +264,6 @@ private:
     };
     static constexpr size_t kMaxStatus = 64;
 
-    static bool has(const Json& j, const char* key) { return j.has(key) && !j.at(key).is_null(); }
     bool in_loop(size_t i) const { return loop_times_ > 0 && i >= loop_start_ && i < loop_stop_; }
 
     Step check(const StepEntry* entries, int n) const {
@@ -515,36 +513,51 @@ private:
     void encode(const StepCtx& s, const Step& step) {
         if (bigram_.data || x0_)
             cuda_check(ingot_support_embed_sum_bf16(ops_.x, x0_, embed_.data, n_vocab_, step.tokens, bigram_.data, bigram_buckets_ + 1, step.bigrams, embed_.n_in,
-                                                    s.st.n_tok, embed_status_, ops_.stream), "embedding rows");
+                                                    s.st.n_tok, embed_scale_, embed_status_, ops_.stream), "embedding rows");
         else
-            cuda_check(ingot_support_embed_rows_bf16(ops_.x, embed_.data, embed_.n_in, n_vocab_, step.tokens, s.st.n_tok, embed_status_, ops_.stream), "embedding rows");
+            cuda_check(ingot_support_embed_rows_bf16(ops_.x, embed_.data, embed_.n_in, n_vocab_, step.tokens, s.st.n_tok, embed_scale_, embed_status_, ops_.stream), "embedding rows");
         ops_.begin();
         for (size_t i = 0; i < runs_.size(); i++) {
             const Layer& L = layers_[runs_[i].layer];
             // the norm that is read next, unless something else happens to x first
             const bool more = i + 1 < runs_.size() && !runs_[i + 1].entry;
-            const float* following = more ? first_norm(layers_[runs_[i + 1].layer]) : nullptr;
+            const Norm following = more ? first_norm(layers_[runs_[i + 1].layer]) : Norm();
             ops_.pass = runs_[i].pass;
             if (runs_[i].entry) ops_.project_concat(s, loop_in_, x0_);
             if (design_.parallel) {
                 if (L.mlp) L.mlp->branch(ops_, s, L.norm2);
-                L.mixer->run(ops_, s, L.norm1, following);
+                L.mixer->run(ops_, s, {L.norm1, L.norm1b, following});
             } else {
-                L.mixer->run(ops_, s, L.norm1, L.mlp ? L.norm2 : following);
-                if (L.mlp) L.mlp->run(ops_, s, L.norm2, following);
+                L.mixer->run(ops_, s, {L.norm1, L.norm1b, L.mlp ? L.norm2 : following});
+                if (L.mlp) L.mlp->run(ops_, s, {L.norm2, L.norm2b, following});
             }
             if (tap_) tap(s.st.n_tok);
         }
         if (!step.n_want) return;
         const int ld = embed_.n_in;
-        if (step.n_want == 1 && LayerOps::streams(head_)) {
-            cuda_check(ingot_support_gemv_bf16(logits_dev_, head_.data, head_.n_out, head_.n_in, ops_.x + size_t(step.first_want) * ld, final_norm_, ops_.eps,
+        if (step.n_want == 1 && LayerOps::streams(head_) && !final_norm_.b) {
+            cuda_check(ingot_support_gemv_bf16(logits_dev_, head_.data, head_.n_out, head_.n_in, ops_.x + size_t(step.first_want) * ld, final_norm_.w, ops_.eps,
                                                ops_.width, 0, 0, 0, ops_.stream), "logits");
             cap_logits(step);
             return;
         }
-        cuda_check(ingot_support_rmsnorm_rows(ops_.buf(kNormed), ops_.x, final_norm_, step.want_rows, step.n_want, ld, ops_.width, ops_.eps, ops_.stream), "final norm");
-        if (ops_.ws && step.n_want >= kMinTcTokens) {
+        if (final_norm_.b) {
+            ingot_residual_norm r = {};
+            r.x = ops_.x;
+            r.n = ld;
+            r.n_mean = ops_.width;
+            r.n_rows = step.n_want;
+            r.eps = ops_.eps;
+            r.rows = step.want_rows;
+            r.next = final_norm_;
+            r.out = ops_.buf(kNormed);
+            cuda_check(ingot_residual_norm_run(&r, ops_.stream), "final norm");
+        } else {
+            cuda_check(ingot_support_rmsnorm_rows(ops_.buf(kNormed), ops_.x, final_norm_.w, step.want_rows, step.n_want, ld, ops_.width, ops_.eps, ops_.stream), "final norm");
+        }
+        if (step.n_want == 1 && LayerOps::streams(head_)) {
+            cuda_check(ingot_support_gemv_bf16(logits_dev_, head_.data, head_.n_out, head_.n_in, ops_.buf(kNormed), nullptr, 0.f, ld, 0, 0, 0, ops_.stream), "logits");
+        } else if (ops_.ws && step.n_want >= kMinTcTokens) {
             cuda_check(ingot_linear_tc_prepare_bf16(ops_.ws, ops_.buf(kNormed), ld, ld, step.n_want, step.n_want <= kPairTokens ? 2 : 1, ops_.stream), "final norm");
             cuda_check(ingot_linear_tc_run(ops_.ws, logits_dev_, head_.data, head_.n_in, head_.n_out, 0, ops_.stream), "logits");
         } else {
@@ -555,7 +568,7 @@ private:
     void cap_logits(const Step& step) {
         if (softcap_ > 0) cuda_check(ingot_support_softcap(logits_dev_, size_t(step.n_want) * head_.n_out, softcap_, ops_.stream), "softcap");
     }
-    const float* first_norm(const Layer& L) const { return design_.parallel && L.mlp ? L.norm2 : L.norm1; }
+    Norm first_norm(const Layer& L) const { return design_.parallel && L.mlp ? L.norm2 : L.norm1; }
 
     void tap(int n_tok) {
         const int ld = embed_.n_in, w = ops_.width;
@@ -579,8 +592,8 @@ private:
     size_t loop_start_ = 0, loop_stop_ = 0;
     int loop_times_ = 0;
     float* x0_ = nullptr;              // the embedding output, kept for the loop
-    float softcap_ = 0.f;
-    float* final_norm_ = nullptr;
+    float softcap_ = 0.f, embed_scale_ = 1.f;
+    Norm final_norm_;
     int* embed_status_ = nullptr;
     size_t weight_bytes_ = 0;
     int scan_threads_ = 0, lru_threads_ = 0;
@@ -605,11 +618,34 @@ private:
     float last_ms_ = 0.f;
 };
 
-const RegisterModel kBesudra("Besudra", [](const ModelDir& dir, const EngineOptions& opt) -> std::unique_ptr<ModelBackend> {
-    return std::make_unique<HybridBackend>(dir, opt, Design{0.f, false, false});
-});
-const RegisterModel kBanevik("Banevik", [](const ModelDir& dir, const EngineOptions& opt) -> std::unique_ptr<ModelBackend> {
-    return std::make_unique<HybridBackend>(dir, opt, Design{1.f, true, true});
-});
+// Selective scans, attention beside a gated recurrent unit; gelu feed-forwards.
+Design besudra() { return Design{}; }
+// Looped latent attention in parallel with squared-relu experts.
+Design banevik() {
+    Design d;
+    d.norm_offset = 1.f;
+    d.parallel = d.tied_head = true;
+    return d;
+}
+// Three kinds of grouped-query attention - windowed, without positions, with sinks - between layer norms before and after each part; silu
+// feed-forwards and gated experts.
+Design silevik() {
+    Design d;
+    d.centred = d.sandwich = true;
+    d.act = 0;
+    d.gated_experts = true;
+    d.attention = {{"attention", INGOT_QK_NORM_NONE, false, OutputGate::per_value},
+                   {"attention_2", INGOT_QK_NORM_HEAD, false, OutputGate::per_head},
+                   {"attention_3", INGOT_QK_NORM_ALL, true, OutputGate::none}};
+    return d;
+}
+
+template <Design (*kDesign)()>
+std::unique_ptr<ModelBackend> open_design(const ModelDir& dir, const EngineOptions& opt) {
+    return std::make_unique<HybridBackend>(dir, opt, kDesign());
+}
+const RegisterModel kBesudra("Besudra", open_design<besudra>);
+const RegisterModel kBanevik("Banevik", open_design<banevik>);
+const RegisterModel kSilevik("Silevik", open_design<silevik>);
 
 }  // namespace

@@ -36,7 +36,7 @@ public:
         const int least = shape_.rank + shape_.rot, wide = round_up(std::max(least, round_up(rank, 128)), 64);
         row_ = !ops.opt.f32 && rank <= 512 && wide * 3 <= least * 4 ? wide : round_up(least, 32);
         if (row_ > 1024) throw std::runtime_error("model config: latent rows of more than 1024 values are not supported");
-        cache_ = ops.cache_group(1, row_, 0, window, false, &cache_layer_);
+        cache_ = ops.cache_group(1, row_, 0, window, CacheGroup::plain, &cache_layer_);
 
         const int per = shape_.dim + shape_.rot;
         latent_off_ = heads_ * per;
@@ -74,7 +74,7 @@ public:
         ops.need(kLatent, latent_ld_);
         ops.need(kValue, value_ld_);
     }
-    void run(LayerOps& ops, const StepCtx& s, const float* norm, const float* next_norm) override {
+    void run(LayerOps& ops, const StepCtx& s, const Norms& n) override {
         float *proj = ops.buf(kProj), *value = ops.buf(kValue);
         const CacheGroup& g = *cache_;
         const int layer = cache_layer_ + ops.pass, n_seq = s.st.n_seq;
@@ -86,7 +86,7 @@ public:
         head.st.max_len = from > 0 ? s.lens[from - 1] : 0;
         if (from < n_seq) head.planes = head.st.n_tok <= kPairTokens ? 2 : 1;
 
-        ops.norm_project(s, proj, w_in_, norm);
+        ops.norm_project(s, proj, w_in_, n.in);
         const ingot_act_out plain = ops.operand(head, ops.buf(kQueryPlain), plain_ld_, false);
         ingot_check(ingot_latent_append(g.kv, layer, &s.st, proj, proj_ld_, 0, latent_off_, &shape_, norm_, ops.eps, turns_, &plain, ops.buf(kQuery),
                                         from < n_seq ? ops.buf(kQueryLong) : nullptr, head.st.n_tok, long_dim_, long_rot_, g.tables, g.first_page, g.width, ops.stream));
@@ -99,7 +99,7 @@ public:
             if (from > 0) ops.prepare_rows(head, value, value_ld_, value_ld_);
             ops.operand_ready(s, value_ld_);
         }
-        ops.project_residual(s, w_o_, value, next_norm);
+        ops.project_residual(s, w_o_, value, n);
     }
 
 private:

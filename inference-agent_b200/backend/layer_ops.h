@@ -1,4 +1,4 @@
-// What the layers of a model folder are written in: projections (with the RMS norm of their input or the residual add of their
+// What the layers of a model folder are written in: projections (with the norm of their input or the residual add of their
 // output folded in), scratch activations, weight upload, state and cache groups; and the interfaces of a layer's two parts.
 //
 // Precision. Weights are bf16. In the 16-bit form the tensor-core products take bf16 activations (a hi + lo pair where the
@@ -24,13 +24,14 @@
 #include "grouped_linear.h"
 #include "ingot_cuda.h"
 #include "model_registry.h"
+#include "residual_norm.h"
 #include "weight_streamer.h"
 
 extern "C" {
 cudaError_t ingot_support_embed_rows_bf16(float* out, const void* table, int n_in, int n_rows_table, const int32_t* rows_dev, int n_rows,
-                                          int* status_dev, cudaStream_t s);
+                                          float scale, int* status_dev, cudaStream_t s);
 cudaError_t ingot_support_embed_sum_bf16(float* out, float* copy, const void* table, int n_rows_table, const int32_t* rows_dev, const void* table2,
-                                         int n_rows_table2, const int32_t* rows2_dev, int n_in, int n_rows, int* status_dev, cudaStream_t s);
+                                         int n_rows_table2, const int32_t* rows2_dev, int n_in, int n_rows, float scale, int* status_dev, cudaStream_t s);
 cudaError_t ingot_support_concat_rows(float* f32, void* hi, void* lo, const float* a, const float* b, int n, int n_rows, cudaStream_t s);
 cudaError_t ingot_support_softcap(float* x, size_t n, float cap, cudaStream_t s);
 cudaError_t ingot_support_rmsnorm_rows(float* out, const float* x, const float* w, const int32_t* rows_dev, int n_rows, int n, int n_mean,
@@ -44,6 +45,7 @@ struct ingot_linear_ws;
 cudaError_t ingot_linear_ws_create_bf16(ingot_linear_ws** out, int max_tok, int max_in, int max_out);
 void ingot_linear_ws_destroy(ingot_linear_ws* ws);
 int* ingot_linear_ws_status_dev(ingot_linear_ws* ws);
+const float* ingot_linear_ws_slices(const ingot_linear_ws* ws, int slot, int* n_slices);
 void ingot_linear_ws_planes(ingot_linear_ws* ws, void** hi, void** lo);
 cudaError_t ingot_linear_tc_prepared(ingot_linear_ws* ws, int n_in, int n_tok, int planes);
 cudaError_t ingot_linear_tc_prepare_bf16(ingot_linear_ws* ws, const float* x, int x_ld, int n_in, int n_tok, int planes, cudaStream_t s);
@@ -75,6 +77,39 @@ inline int get_int(const Json& j, const char* key, int lo = 1, int hi = 1 << 28)
     return int(v);
 }
 inline float get_float(const Json& j, const char* key) { return float(j.at(key).number()); }
+inline bool has(const Json& j, const char* key) { return j.has(key) && !j.at(key).is_null(); }
+
+// A kind of grouped-query attention layer: what the design fixes about it; its sizes, rotation, window and value mixing come from the
+// configuration.
+enum class OutputGate { none, per_head, per_value };
+struct AttentionKind {
+    const char* type;  // name in the configuration
+    int qk_norm;       // INGOT_QK_NORM_*
+    bool sink;
+    OutputGate gate;
+};
+
+// What a design fixes and its configuration does not say.
+struct Design {
+    float norm_offset = 0.f;     // the norms' weights are stored around this: x / rms(x) * (norm_offset + w)
+    bool centred = false;        // norms over the residual are layer norms with a bias (tensor NAME.b) instead of RMS norms
+    bool sandwich = false;       // a part's result is normed too before the residual sum (tensors norm1b, norm2b)
+    bool parallel = false;       // a layer adds mixer(norm1 x) + ff(norm2 x), both of the same x, instead of one after the other
+    bool tied_head = false;      // the output matrix is the embedding table
+    int act = 1;                 // of gated feed-forwards: 0 silu, 1 the tanh form of gelu
+    bool gated_experts = false;  // experts are gated (silu) and weighed by a softmax router, instead of squared-relu ones by sigmoid scores
+    std::vector<AttentionKind> attention = {};
+};
+
+// A norm over the residual's length as it is uploaded: RMS, or centred if it has a bias.
+struct Norm : ingot_norm {
+    Norm() : ingot_norm{nullptr, nullptr} {}
+    explicit operator bool() const { return w != nullptr; }
+    bool operator==(const Norm& o) const { return w == o.w; }
+};
+// The norms around one part of a layer: of its input, of its result before the residual sum (may be none), and the one that reads the
+// residual stream next (none: something else happens to it first).
+struct Norms { Norm in, post, next; };
 
 // A dimension of n groups of `size` values, each stored with `padded` places.
 struct Groups {
@@ -101,7 +136,7 @@ struct Part {
 };
 
 enum Buf { kProj, kConv, kStateIn, kDt, kGates, kMix, kGateUp, kMid, kNormed, kQuery, kQueryPlain, kQueryLong, kLatent, kValue, kRouter, kExpertIn, kExpertMid, kExpertOut,
-           kBranch, kConcat, kBufCount };
+           kBranch, kConcat, kFirstValue, kBufCount };
 
 // The step as the launches see it.
 struct StepCtx {
@@ -115,7 +150,7 @@ struct StepCtx {
 // Shared-row attention caches of equal shape and visibility live in one handle with one page pool.
 struct CacheGroup {
     int kv_heads, dim, chunk, window;  // visibility: own chunk, sliding window (one of them 0), or the whole past
-    bool scales;                       // rows with a key scale of their own (ingot_skv_create) or without (ingot_skv_create_window)
+    enum Form { scaled, plain, joined } form;  // rows with a key scale of their own (ingot_skv_create), without (ingot_skv_create_window), [key | value]
     int n_layer = 0;
     ingot_skv* kv = nullptr;
     BlockPool pool;
@@ -143,7 +178,7 @@ struct Branch {
 
 class LayerOps {
 public:
-    LayerOps(const ModelDir& dir, const EngineOptions& opt, int max_step) : dir(dir), opt(opt), max_step(max_step) {
+    LayerOps(const ModelDir& dir, const EngineOptions& opt, const Design& design, int max_step) : dir(dir), opt(opt), design(design), max_step(max_step) {
         cuda_check(cudaStreamCreateWithFlags(&stream, cudaStreamNonBlocking), "cudaStreamCreate");
     }
     ~LayerOps() {
@@ -189,12 +224,19 @@ public:
     }
     float* vector(const std::string& name, const std::vector<int64_t>& shape, Groups g) { return upload(host_vector(name, shape, g)); }
     float* vector(const std::string& name, int n) { return vector(name, {n}, flat(n)); }
-    // The weight of an RMS norm over the residual stream, as the design stores it (around norm_offset).
-    float* norm_vector(const std::string& name) {
-        std::vector<float> v = host_vector(name, {width}, flat(width));
-        for (int i = 0; i < width; i++) v[size_t(i)] += norm_offset;
-        return upload(v);
+    // A norm over the residual stream as the design stores it (RMS weights around norm_offset, or weight and bias); its result times `gain`.
+    Norm norm(const std::string& name, float gain = 1.f) {
+        Norm n;
+        auto load = [&](const std::string& tensor, float offset) {
+            std::vector<float> v = host_vector(tensor, {width}, flat(width));
+            for (int i = 0; i < width; i++) v[size_t(i)] = (v[size_t(i)] + offset) * gain;
+            return upload(v);
+        };
+        n.w = load(name, design.norm_offset);
+        if (design.centred) n.b = load(name + ".b", 0.f);
+        return n;
     }
+    float scalar(const std::string& name) { return tensor_f32(dir.tensor(name, {}))[0]; }
     const TensorView& bf16(const std::string& name, const std::vector<int64_t>& shape) const {
         const TensorView& t = dir.tensor(name, shape);
         if (t.dtype != "BF16") throw std::runtime_error("model: tensor " + name + " has type " + t.dtype + ", expected BF16");
@@ -251,16 +293,16 @@ public:
     }
     static bool streams(const Matrix& w) { return w.n_in % 256 == 0 && w.n_in <= 12032 && w.rows_per_block == 0; }
 
-    // out [n_tok][w.n_out] = W rmsnorm(x)
-    void norm_project(const StepCtx& s, float* out, const Matrix& w, const float* norm) {
+    // out [n_tok][w.n_out] = W norm(x)
+    void norm_project(const StepCtx& s, float* out, const Matrix& w, const Norm& norm) {
         if (s.tc) {
             prepare_norm(s, w, norm);
             cuda_check(ingot_linear_tc_run(ws, out, w.data, w.n_in, w.n_out, 0, stream), "projection");
-        } else if (s.st.n_tok == 1 && streams(w)) {
-            cuda_check(ingot_support_gemv_bf16(out, w.data, w.n_out, w.n_in, x, norm, eps, width, 0, 0, 0, stream), "projection");
+        } else if (s.st.n_tok == 1 && streams(w) && !norm.b) {
+            cuda_check(ingot_support_gemv_bf16(out, w.data, w.n_out, w.n_in, x, norm.w, eps, width, 0, 0, 0, stream), "projection");
         } else {
             norm_rows(s, norm);
-            cuda_check(ingot_support_linear_bf16(out, w.data, buf(kNormed), w.n_in, w.n_in, w.n_out, 0, s.st.n_tok, 0, stream), "projection");
+            project(s, out, w, buf(kNormed), w.n_in);
         }
     }
     // out = W in. Tensor-core path: the operand planes must hold `in` (operand_ready).
@@ -283,13 +325,20 @@ public:
         if (s.tc) prepare_rows(s, in, in_ld, w.n_in, planes);
         project(s, out, w, in, in_ld);
     }
-    // x += W in; next_norm: the norm that the following product reads x through (null: none), folded into the same kernel.
-    void project_residual(const StepCtx& s, const Matrix& w, const float* in, const float* next_norm) {
-        norm_ready_ = nullptr;
+    // x += post(W in); n.next: the norm that the following product reads x through, folded into the same kernel.
+    void project_residual(const StepCtx& s, const Matrix& w, const float* in, const Norms& n) {
+        if (n.post || n.next.b) {
+            ingot_residual_norm r = {};
+            product(s, w, in, r);
+            finish(s, r, n);
+            add_branch(s);
+            return;
+        }
+        norm_ready_ = Norm();
         if (s.tc) {
             cuda_check(ingot_linear_tc_run_partial(ws, w.data, w.n_in, w.n_out, 0, stream), "output projection");
-            cuda_check(ingot_linear_tc_finish_residual_norm_bf16(ws, x, next_norm, eps, width, s.planes, branch_.rows, branch_.row_of, branch_.top, stream), "residual");
-            norm_ready_ = next_norm;
+            cuda_check(ingot_linear_tc_finish_residual_norm_bf16(ws, x, n.next.w, eps, width, s.planes, branch_.rows, branch_.row_of, branch_.top, stream), "residual");
+            norm_ready_ = n.next;
             branch_ = Branch();
             return;
         }
@@ -300,6 +349,40 @@ public:
         }
         add_branch(s);
     }
+    // W in as the product of a residual sum (finish): slices in the workspace, or rows of kBranch.
+    void product(const StepCtx& s, const Matrix& w, const float* in, ingot_residual_norm& r) {
+        if (s.tc) {
+            cuda_check(ingot_linear_tc_run_partial(ws, w.data, w.n_in, w.n_out, 0, stream), "output projection");
+            r.product = ingot_linear_ws_slices(ws, 0, &r.n_slices);
+        } else {
+            project(s, buf(kBranch), w, in, w.n_in);
+            r.product = buf(kBranch);
+            r.n_slices = 1;
+        }
+    }
+    // x += post(the terms of r), and next(x) for the part that follows.
+    void finish(const StepCtx& s, ingot_residual_norm& r, const Norms& n) {
+        norm_ready_ = Norm();
+        r.post = n.post;
+        if (n.next.b) r.next = n.next;  // RMS norms are folded into the products that read through them
+        residual_norm(s, r);
+        if (n.next.b) norm_ready_ = n.next;
+    }
+    void residual_norm(const StepCtx& s, ingot_residual_norm& r) {
+        r.x = x;
+        r.n = round_up(width, 8);
+        r.n_mean = width;
+        r.n_rows = s.st.n_tok;
+        r.eps = eps;
+        if (r.next.w) {
+            const ingot_act_out o = operand(s, buf(kNormed), r.n, false);
+            r.out = o.f32;
+            r.hi = o.hi;
+            r.lo = o.lo;
+        }
+        cuda_check(ingot_residual_norm_run(&r, stream), "residual");
+        if (r.next.w) operand_ready(s, r.n);
+    }
     // A feed-forward that runs beside the mixer leaves its result here; the mixer's project_residual takes it in.
     void set_branch(const Branch& b) { branch_ = b; }
     // The same without a mixer to join: x += branch.
@@ -307,7 +390,7 @@ public:
         if (!branch_.rows) return;
         ingot_check(ingot_moe_add(x, branch_.rows, branch_.row_of, s.st.n_tok, branch_.top, round_up(width, 8), stream));
         branch_ = Branch();
-        norm_ready_ = nullptr;
+        norm_ready_ = Norm();
     }
     // x = W [x; x0], two residual-length rows side by side
     void project_concat(const StepCtx& s, const Matrix& w, const float* x0) {
@@ -316,56 +399,80 @@ public:
         cuda_check(ingot_support_concat_rows(o.f32, o.hi, o.lo, x, x0, n, s.st.n_tok, stream), "concatenation");
         operand_ready(s, 2 * n);
         project(s, x, w, buf(kConcat), 2 * n);
-        norm_ready_ = nullptr;
+        norm_ready_ = Norm();
     }
-    // kMid (or the operand planes) = gelu(W_gate h) * (W_up h), h = rmsnorm(x); w holds the gate rows and then the up rows
-    void gated_project(const StepCtx& s, const Matrix& w, const float* norm) {
+    // kMid (or the operand planes) = act(W_gate h) * (W_up h), h = norm(x); w holds the gate rows and then the up rows
+    void gated_project(const StepCtx& s, const Matrix& w, const Norm& norm) {
+        if (s.tc) prepare_norm(s, w, norm);
+        else if (norm.b || !(s.st.n_tok == 1 && streams(w))) norm_rows(s, norm);
+        gated_project_normed(s, w, norm);
+    }
+    // The same when the planes, or kNormed, hold h (single tokens read x through an RMS norm themselves).
+    void gated_project_normed(const StepCtx& s, const Matrix& w, const Norm& norm) {
         const int ff = w.n_out / 2;
         if (s.tc) {
-            prepare_norm(s, w, norm);
             cuda_check(ingot_linear_tc_run_partial(ws, w.data, w.n_in, w.n_out, 0, stream), "gate / up");
-            cuda_check(ingot_linear_tc_finish_gated_bf16(ws, 1, s.planes, stream), "gate");
+            cuda_check(ingot_linear_tc_finish_gated_bf16(ws, design.act, s.planes, stream), "gate");
         } else if (s.st.n_tok == 1 && streams(w)) {
-            cuda_check(ingot_support_gemv_bf16(buf(kMid), w.data, ff, w.n_in, x, norm, eps, width, 1, 1, 0, stream), "gate / up");
+            cuda_check(ingot_support_gemv_bf16(buf(kMid), w.data, ff, w.n_in, norm.b ? buf(kNormed) : x, norm.b ? nullptr : norm.w, eps, width, 1, design.act, 0, stream), "gate / up");
         } else {
-            norm_rows(s, norm);
             cuda_check(ingot_support_linear_bf16(buf(kGateUp), w.data, buf(kNormed), w.n_in, w.n_in, w.n_out, 0, s.st.n_tok, 0, stream), "gate / up");
-            cuda_check(ingot_support_gated_act(buf(kMid), buf(kGateUp), s.st.n_tok, ff, 1, stream), "gate");
+            cuda_check(ingot_support_gated_act(buf(kMid), buf(kGateUp), s.st.n_tok, ff, design.act, stream), "gate");
         }
     }
-    void begin() { norm_ready_ = nullptr; branch_ = Branch(); }
-    void norm_rows(const StepCtx& s, const float* norm) {
-        cuda_check(ingot_support_rmsnorm_rows(buf(kNormed), x, norm, nullptr, s.st.n_tok, round_up(width, 8), width, eps, stream), "rmsnorm");
+    void begin() { norm_ready_ = Norm(); branch_ = Branch(); }
+    // Without tensor cores: kNormed = norm(x).
+    void norm_rows(const StepCtx& s, const Norm& norm) {
+        if (norm.b) {
+            norm_now(s, norm);
+            return;
+        }
+        cuda_check(ingot_support_rmsnorm_rows(buf(kNormed), x, norm.w, nullptr, s.st.n_tok, round_up(width, 8), width, eps, stream), "rmsnorm");
     }
-    // Tensor-core path: the planes hold rmsnorm(x; norm).
-    void prepare_norm(const StepCtx& s, const Matrix& w, const float* norm) {
+    // Tensor-core path: the planes hold norm(x).
+    void prepare_norm(const StepCtx& s, const Matrix& w, const Norm& norm) {
+        if (norm.b) {
+            norm_now(s, norm);
+            return;
+        }
         const bool ready = norm_ready_ == norm && norm;  // the kernel that finished x already normalised it for this product
-        norm_ready_ = nullptr;
-        if (!ready) cuda_check(ingot_linear_tc_prepare_norm_bf16(ws, x, norm, eps, w.n_in, width, s.st.n_tok, s.planes, stream), "rmsnorm");
+        norm_ready_ = Norm();
+        if (!ready) cuda_check(ingot_linear_tc_prepare_norm_bf16(ws, x, norm.w, eps, w.n_in, width, s.st.n_tok, s.planes, stream), "rmsnorm");
+    }
+    // A centred norm, unless the kernel that finished x took it.
+    void norm_now(const StepCtx& s, const Norm& norm) {
+        const bool ready = norm_ready_ == norm;
+        norm_ready_ = Norm();
+        if (ready) return;
+        ingot_residual_norm r = {};
+        r.next = norm;
+        residual_norm(s, r);
     }
 
     const ModelDir& dir;
     const EngineOptions opt;
+    const Design design;
     const int max_step;
     cudaStream_t stream = nullptr;
     ingot_linear_ws* ws = nullptr;
     float* x = nullptr;  // residual stream [n_tok][round_up(width, 8)]
     int width = 0;
-    float eps = 0.f, norm_offset = 0.f;
+    float eps = 0.f;
     int passes = 1;  // of the layer under construction: each pass of a loop has a state and a cache of its own
     int pass = 0;    // the one that runs
     size_t weight_bytes = 0;
     std::vector<std::unique_ptr<CacheGroup>> caches;
+    int mixed_values = 0;  // length of the values that layers mix with the first such layer's (kFirstValue); 0: none so far
 
     // The group a layer's caches belong to; *layer: the first of its `passes` caches there.
-    CacheGroup* cache_group(int kv_heads, int dim, int chunk, int window, bool scales, int* layer) {
+    CacheGroup* cache_group(int kv_heads, int dim, int chunk, int window, CacheGroup::Form form, int* layer) {
         CacheGroup* g = nullptr;
         for (auto& c : caches)
-            if (c->kv_heads == kv_heads && c->dim == dim && c->chunk == chunk && c->window == window && c->scales == scales) g = c.get();
+            if (c->kv_heads == kv_heads && c->dim == dim && c->chunk == chunk && c->window == window && c->form == form) g = c.get();
         if (!g) {
             caches.push_back(std::make_unique<CacheGroup>());
             g = caches.back().get();
-            g->kv_heads = kv_heads; g->dim = dim; g->chunk = chunk; g->window = window; g->scales = scales;
+            g->kv_heads = kv_heads; g->dim = dim; g->chunk = chunk; g->window = window; g->form = form;
         }
         *layer = g->n_layer;
         g->n_layer += passes;
@@ -384,7 +491,7 @@ private:
     size_t key_bytes_[3] = {0, 0, 0};
     void* keys_[3] = {nullptr, nullptr, nullptr};
     Branch branch_;
-    const float* norm_ready_ = nullptr;  // the norm weights x has been prepared with
+    Norm norm_ready_;  // the norm x has been prepared with
 };
 
 // ---- layers ----------------------------------------------------------------------------------------------------------
@@ -392,8 +499,8 @@ private:
 class Mixer {
 public:
     virtual ~Mixer() = default;
-    // x += mixer(rmsnorm(x; norm)) + the branch set beside it; next_norm as in LayerOps::project_residual.
-    virtual void run(LayerOps& ops, const StepCtx& s, const float* norm, const float* next_norm) = 0;
+    // x += post(mixer(in(x))) + the branch set beside it; norms as in LayerOps::project_residual.
+    virtual void run(LayerOps& ops, const StepCtx& s, const Norms& n) = 0;
     // Threads one time chunk of a recurrence of this mixer occupies (0: none); sizes the chunks of a step.
     virtual int scan_threads() const { return 0; }
     virtual int lru_threads() const { return 0; }
@@ -404,10 +511,10 @@ public:
 class FeedForward {
 public:
     virtual ~FeedForward() = default;
-    // x += ff(rmsnorm(x; norm)), after the mixer
-    virtual void run(LayerOps& ops, const StepCtx& s, const float* norm, const float* next_norm) = 0;
-    // ff(rmsnorm(x; norm)) as a branch beside the mixer (LayerOps::set_branch); runs before the mixer does
-    virtual void branch(LayerOps& ops, const StepCtx& s, const float* norm) = 0;
+    // x += post(ff(in(x))), after the mixer
+    virtual void run(LayerOps& ops, const StepCtx& s, const Norms& n) = 0;
+    // ff(norm(x)) as a branch beside the mixer (LayerOps::set_branch); runs before the mixer does
+    virtual void branch(LayerOps& ops, const StepCtx& s, const Norm& norm) = 0;
 };
 
 // One function per kind; a further kind is a class in a file of its own and a line in make_mixer / make_feed_forward
@@ -415,5 +522,6 @@ public:
 std::unique_ptr<Mixer> make_selective_scan(LayerOps& ops, const Json& config, const std::string& prefix);
 std::unique_ptr<Mixer> make_parallel(LayerOps& ops, const Json& config, const std::string& prefix);
 std::unique_ptr<Mixer> make_latent_attention(LayerOps& ops, const Json& config, const std::string& prefix);
+std::unique_ptr<Mixer> make_grouped_attention(LayerOps& ops, const AttentionKind& kind, const Json& config, const std::string& prefix);
 std::unique_ptr<FeedForward> make_gated_feed_forward(LayerOps& ops, const Json& config, const std::string& prefix);
 std::unique_ptr<FeedForward> make_mixture(LayerOps& ops, const Json& config, const std::string& prefix);

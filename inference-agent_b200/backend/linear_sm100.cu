@@ -111,7 +111,7 @@ struct GemmParams {
     const int32_t* group_start;
     int n_groups;
     const float* row_scale;                // epilogue: accumulator * row_scale[row] (null: none), then act
-    int act;                               // 1: square of relu
+    int act;                               // 1: square of relu, 2: silu(gate) * up (INGOT_ACT_*)
     __nv_bfloat16 *out_hi, *out_lo;        // bf16 plane(s) [rows][n_out] instead of f32
     __half* out_half;                      // f16 instead of f32: row stride half_ld, block b's columns from b * half_block on
     int half_ld, half_block;
@@ -283,57 +283,84 @@ linear_sm100_kernel(const __grid_constant__ CUtensorMap map_hi, const __grid_con
             float* dst = (split_k ? mat_partial + (size_t)split * p.n_tok * mat_n_out : p.out) + (size_t)row * mat_n_out + n0;
             const bool add = !split_k && p.accumulate;
             const float scale = p.row_scale && row < row_end ? p.row_scale[row] : 1.0f;
+            if (kGrouped && p.act == 2) {
+                // Runs of 32 gate columns, each followed by the 32 up columns of the same outputs: scale * silu(gate) * up, half as wide.
+                const int half_out = mat_n_out / 2;
 #pragma unroll
-            for (int c = 0; c < kBN / 32; c++) {
-                float v[32];
-                tmem_ld32(tmem + ((uint32_t)(lg * 32) << 16) + c * 32, v);
-                tmem_wait_ld();
-                if (row < row_end) {
-                    if (kGrouped && (p.row_scale || p.act)) {
+                for (int c = 0; c < kBN / 64; c++) {
+                    float g[32], u[32];
+                    tmem_ld32(tmem + ((uint32_t)(lg * 32) << 16) + c * 64, g);
+                    tmem_ld32(tmem + ((uint32_t)(lg * 32) << 16) + c * 64 + 32, u);
+                    tmem_wait_ld();
+                    if (row >= row_end || n0 + c * 64 >= mat_n_out) continue;
+                    const size_t at = (size_t)row * half_out + n0 / 2 + c * 32;
 #pragma unroll
-                        for (int i = 0; i < 32; i++) {
-                            v[i] *= scale;
-                            if (p.act == 1) v[i] = v[i] > 0.f ? v[i] * v[i] : 0.f;
+                    for (int i = 0; i < 32; i += 8) {
+                        __nv_bfloat162 h[4], l[4];
+#pragma unroll
+                        for (int e = 0; e < 4; e++) {
+                            const float a = g[i + 2 * e], b = g[i + 2 * e + 1];
+                            const float x = a / (1.0f + expf(-a)) * u[i + 2 * e] * scale, y = b / (1.0f + expf(-b)) * u[i + 2 * e + 1] * scale;
+                            h[e] = __floats2bfloat162_rn(x, y);
+                            l[e] = __floats2bfloat162_rn(x - __low2float(h[e]), y - __high2float(h[e]));
                         }
+                        *reinterpret_cast<uint4*>(p.out_hi + at + i) = *reinterpret_cast<const uint4*>(h);
+                        if (p.out_lo) *reinterpret_cast<uint4*>(p.out_lo + at + i) = *reinterpret_cast<const uint4*>(l);
                     }
-                    if (kGrouped && p.out_hi) {  // n_out is a multiple of 8
+                }
+            } else {
 #pragma unroll
-                        for (int i = 0; i < 32; i += 8) {
-                            const int col = n0 + c * 32 + i;
-                            if (col >= col_end) break;
-                            const size_t at = (size_t)row * mat_n_out + col;
-                            __nv_bfloat162 h[4], l[4];
+                for (int c = 0; c < kBN / 32; c++) {
+                    float v[32];
+                    tmem_ld32(tmem + ((uint32_t)(lg * 32) << 16) + c * 32, v);
+                    tmem_wait_ld();
+                    if (row < row_end) {
+                        if (kGrouped && (p.row_scale || p.act)) {
 #pragma unroll
-                            for (int e = 0; e < 4; e++) {
-                                h[e] = __floats2bfloat162_rn(v[i + 2 * e], v[i + 2 * e + 1]);
-                                l[e] = __floats2bfloat162_rn(v[i + 2 * e] - __low2float(h[e]), v[i + 2 * e + 1] - __high2float(h[e]));
+                            for (int i = 0; i < 32; i++) {
+                                v[i] *= scale;
+                                if (p.act == 1) v[i] = v[i] > 0.f ? v[i] * v[i] : 0.f;
                             }
-                            *reinterpret_cast<uint4*>(p.out_hi + at) = *reinterpret_cast<const uint4*>(h);
-                            if (p.out_lo) *reinterpret_cast<uint4*>(p.out_lo + at) = *reinterpret_cast<const uint4*>(l);
                         }
-                    } else if (!kGrouped && p.out_half) {  // n_out and the blocks are multiples of 8
+                        if (kGrouped && p.out_hi) {  // n_out is a multiple of 8
 #pragma unroll
-                        for (int i = 0; i < 32; i += 8) {
-                            const int col = n0 + c * 32 + i;
-                            if (col >= col_end) break;
-                            __half2 h[4];
+                            for (int i = 0; i < 32; i += 8) {
+                                const int col = n0 + c * 32 + i;
+                                if (col >= col_end) break;
+                                const size_t at = (size_t)row * mat_n_out + col;
+                                __nv_bfloat162 h[4], l[4];
 #pragma unroll
-                            for (int e = 0; e < 4; e++)
-                                h[e] = __floats2half2_rn(fminf(fmaxf(v[i + 2 * e], -65504.f), 65504.f), fminf(fmaxf(v[i + 2 * e + 1], -65504.f), 65504.f));
-                            *reinterpret_cast<uint4*>(p.out_half + (size_t)row * p.half_ld + blk * p.half_block + (col - blk * p.rows_per_block)) = *reinterpret_cast<const uint4*>(h);
-                        }
-                    } else {
+                                for (int e = 0; e < 4; e++) {
+                                    h[e] = __floats2bfloat162_rn(v[i + 2 * e], v[i + 2 * e + 1]);
+                                    l[e] = __floats2bfloat162_rn(v[i + 2 * e] - __low2float(h[e]), v[i + 2 * e + 1] - __high2float(h[e]));
+                                }
+                                *reinterpret_cast<uint4*>(p.out_hi + at) = *reinterpret_cast<const uint4*>(h);
+                                if (p.out_lo) *reinterpret_cast<uint4*>(p.out_lo + at) = *reinterpret_cast<const uint4*>(l);
+                            }
+                        } else if (!kGrouped && p.out_half) {  // n_out and the blocks are multiples of 8
 #pragma unroll
-                        for (int i = 0; i < 32; i += 4) {
-                            const int col = n0 + c * 32 + i;
-                            if (col + 3 < col_end) {
-                                float4* d4 = reinterpret_cast<float4*>(dst + c * 32 + i);
-                                float4 o = make_float4(v[i], v[i + 1], v[i + 2], v[i + 3]);
-                                if (add) { const float4 old = *d4; o.x += old.x; o.y += old.y; o.z += old.z; o.w += old.w; }
-                                *d4 = o;
-                            } else {
+                            for (int i = 0; i < 32; i += 8) {
+                                const int col = n0 + c * 32 + i;
+                                if (col >= col_end) break;
+                                __half2 h[4];
+#pragma unroll
                                 for (int e = 0; e < 4; e++)
-                                    if (col + e < col_end) dst[c * 32 + i + e] = add ? dst[c * 32 + i + e] + v[i + e] : v[i + e];
+                                    h[e] = __floats2half2_rn(fminf(fmaxf(v[i + 2 * e], -65504.f), 65504.f), fminf(fmaxf(v[i + 2 * e + 1], -65504.f), 65504.f));
+                                *reinterpret_cast<uint4*>(p.out_half + (size_t)row * p.half_ld + blk * p.half_block + (col - blk * p.rows_per_block)) = *reinterpret_cast<const uint4*>(h);
+                            }
+                        } else {
+#pragma unroll
+                            for (int i = 0; i < 32; i += 4) {
+                                const int col = n0 + c * 32 + i;
+                                if (col + 3 < col_end) {
+                                    float4* d4 = reinterpret_cast<float4*>(dst + c * 32 + i);
+                                    float4 o = make_float4(v[i], v[i + 1], v[i + 2], v[i + 3]);
+                                    if (add) { const float4 old = *d4; o.x += old.x; o.y += old.y; o.z += old.z; o.w += old.w; }
+                                    *d4 = o;
+                                } else {
+                                    for (int e = 0; e < 4; e++)
+                                        if (col + e < col_end) dst[c * 32 + i + e] = add ? dst[c * 32 + i + e] + v[i + e] : v[i + e];
+                                }
                             }
                         }
                     }
@@ -876,6 +903,7 @@ cudaError_t ingot_linear_tc_run_f16(ingot_linear_ws* ws, void* out, int out_ld, 
 }
 
 cudaError_t ingot_grouped_tc_run(ingot_linear_ws* ws, const ingot_grouped_gemm* g, cudaStream_t s) {
+    if (g->act == 2 && (g->n_out % 64 != 0 || !g->out_hi)) return cudaErrorInvalidValue;
     if (!ws->bf16 || g->n_in % 8 != 0 || g->n_out % 8 != 0 || g->n_rows < 1 || g->n_groups < 1 || g->rows_per_group < 1) return cudaErrorInvalidValue;
     const int planes = g->a_lo ? 2 : 1, box_rows = g->rows_per_group >= 128 ? 128 : (g->rows_per_group + 7) / 8 * 8;
     GemmParams p = {};
@@ -927,6 +955,12 @@ cudaError_t ingot_linear_tc_run_partial(ingot_linear_ws* ws, const void* w, int 
 cudaError_t ingot_linear_tc_run_partial_group(ingot_linear_ws* ws, const void* const* w, int n_in, const int* n_out, int count,
                                               int first_slot, int append, cudaStream_t s) {
     return launch_gemm(ws, nullptr, w, n_in, n_out, count, 0, first_slot, true, append != 0, s);
+}
+
+// The product left in `slot`: *n_slices matrices [prepared tokens][n_out] f32 to be summed in order.
+const float* ingot_linear_ws_slices(const ingot_linear_ws* ws, int slot, int* n_slices) {
+    *n_slices = ws->slot_split[slot];
+    return ws->partial + (size_t)slot * ws->partial_floats;
 }
 
 static Slices slices_of(const ingot_linear_ws* ws, int slot) {

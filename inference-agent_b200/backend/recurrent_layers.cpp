@@ -44,10 +44,10 @@ public:
         ops.need(kDt, ip_);
         ops.need(kMix, ip_);
     }
-    void run(LayerOps& ops, const StepCtx& s, const float* norm, const float* next_norm) override {
+    void run(LayerOps& ops, const StepCtx& s, const Norms& n) override {
         float *xz = ops.buf(kProj), *xc = ops.buf(kConv), *dbc = ops.buf(kStateIn), *dt = ops.buf(kDt);
         const int ld_bc = rank_p_ + 2 * np_;
-        ops.norm_project(s, xz, w_in_, norm);
+        ops.norm_project(s, xz, w_in_, n.in);
         const ingot_act_out conv = ops.operand(s, xc, ip_, true);
         ingot_check(ingot_causal_conv(&s.st, xz, 2 * ip_, nullptr, conv_w_, conv_b_, taps_, ip_, ops.opt.f32 ? 1 : 2, ops.at_pass(conv_state_, size_t(taps_ - 1) * ip_), &conv, ops.stream));
         ops.operand_ready(s, ip_);
@@ -57,7 +57,7 @@ public:
         ingot_check(ingot_selective_scan(&s.st, &s.scan, xc, ip_, dt, ip_, dt_b_, dbc, ld_bc, rank_p_, rank_p_ + np_, xz + ip_, 2 * ip_, a2_, d_,
                                          ops.at_pass(state_, size_t(ip_) * np_), ip_, states_, ops.opt.f32 ? 1 : 0, &y, ops.stream));
         ops.operand_ready(s, ip_);
-        ops.project_residual(s, w_o_, ops.buf(kMix), next_norm);
+        ops.project_residual(s, w_o_, ops.buf(kMix), n);
     }
     int scan_threads() const override { return ip_ * 2; }
     size_t scan_scratch_per_chunk() const override { return size_t(ip_) * (np_ + 1); }
@@ -90,7 +90,7 @@ public:
         const int row = ops.opt.f32 ? round_up(dim_, 8) : ingot_skv_row_length(dim_);
         if (row < 2 || row > 512) throw std::runtime_error("model config: heads of more than 512 values are not supported");
         row_ = row;
-        cache_ = ops.cache_group(kv_heads_, row, chunk, 0, true, &cache_layer_);
+        cache_ = ops.cache_group(kv_heads_, row, chunk, 0, CacheGroup::scaled, &cache_layer_);
 
         width_ = get_int(r, "width");
         const int blocks = get_int(r, "blocks");
@@ -135,10 +135,10 @@ public:
         ops.need(kMix, mix_ld_);
         ops.need(kQuery, q.width());
     }
-    void run(LayerOps& ops, const StepCtx& s, const float* norm, const float* next_norm) override {
+    void run(LayerOps& ops, const StepCtx& s, const Norms& n) override {
         float *proj = ops.buf(kProj), *u = ops.buf(kConv), *gates = ops.buf(kGates), *mix = ops.buf(kMix);
         const CacheGroup& g = *cache_;
-        ops.norm_project(s, proj, w_in_, norm);
+        ops.norm_project(s, proj, w_in_, n.in);
         const ingot_act_out conv = ops.operand(s, u, wp_, true, 2);
         ingot_check(ingot_causal_conv(&s.st, proj + x_off_, proj_ld_, x_b_, conv_w_, conv_b_, taps_, wp_, 0, ops.at_pass(conv_state_, size_t(taps_ - 1) * wp_), &conv, ops.stream));
         ops.operand_ready(s, wp_, 2);
@@ -156,7 +156,7 @@ public:
         ingot_check(ingot_gated_lru(&s.st, &s.lru, u, wp_, gates, 2 * wp_, block_, r_b_, i_b_, softplus_lam_, proj + y_off_, proj_ld_, y_b_, ops.at_pass(state_, size_t(wp_)), wp_,
                                     right_scale_, ops.opt.f32 ? 1 : 0, &right, ops.stream));
         ops.operand_ready(s, mix_ld_);
-        ops.project_residual(s, w_o_, mix, next_norm);
+        ops.project_residual(s, w_o_, mix, n);
     }
     int lru_threads() const override { return wp_; }
     size_t lru_scratch_per_chunk() const override { return 2 * size_t(wp_); }

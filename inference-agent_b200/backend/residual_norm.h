@@ -1,0 +1,31 @@
+// What happens to the residual stream between two parts of a layer, one launch (residual_norm.cu).
+#pragma once
+
+#include <cuda_runtime.h>
+#include <stdint.h>
+
+// A norm over the residual's length: x / rms(x) * w, or with a bias the centred one, (x - mean) / sqrt(variance + eps) * w + b.
+struct ingot_norm {
+    const float *w, *b;  // w null: none
+};
+
+// Per row:  y = gain * product + sum of its branch rows + self_gain * self(x);  x += post(y);  out = next(x).
+// Every term is optional; without any, x is only read. Rows hold n floats of which the first n_mean count; weights are zero beyond.
+struct ingot_residual_norm {
+    float* x;
+    int n, n_mean, n_rows;
+    float eps;
+    const int32_t* rows;        // row of x each row of the launch is (null: the same)
+    const float* product;       // [n_slices][n_rows][n], summed in order
+    int n_slices;
+    const float* gain;          // [n_rows] (null: 1)
+    const float* branch;        // rows of another part, row r's at row_of[r * top + k]; a negative entry is none
+    const int32_t* row_of;
+    int top;
+    const float* self_gain;     // [n_rows]
+    ingot_norm self, post, next;
+    float* out;                 // next(x) as f32 rows and / or bf16 planes
+    void *hi, *lo;
+};
+
+extern "C" cudaError_t ingot_residual_norm_run(const ingot_residual_norm* r, cudaStream_t s);

@@ -573,7 +573,7 @@ __device__ __forceinline__ float embed_to_f32(__nv_bfloat16 v) { return __bfloat
 // ops::dequant_row on the host). A row index outside the table gives zeros and raises *status.
 template <typename W>
 __global__ void embed_rows_kernel(float* out, const W* __restrict__ table, int n_in, int n_rows_table, const int32_t* __restrict__ rows,
-                                  int* status) {
+                                  int* status, float scale) {
     const int row = rows[blockIdx.x];
     float* o = out + (size_t)blockIdx.x * n_in;
     if (row < 0 || row >= n_rows_table) {
@@ -582,18 +582,19 @@ __global__ void embed_rows_kernel(float* out, const W* __restrict__ table, int n
         return;
     }
     const W* src = table + (size_t)row * n_in;
-    for (int i = threadIdx.x; i < n_in; i += blockDim.x) o[i] = embed_to_f32(src[i]);
+    for (int i = threadIdx.x; i < n_in; i += blockDim.x) o[i] = embed_to_f32(src[i]) * scale;
 }
 
 // The same from two tables, added; `copy` (may be null) receives the rows too. A row index outside its table gives zeros and raises *status.
 __global__ void embed_sum_kernel(float* out, float* copy, const __nv_bfloat16* __restrict__ table, int n_table, const int32_t* __restrict__ rows,
-                                 const __nv_bfloat16* __restrict__ table2, int n_table2, const int32_t* __restrict__ rows2, int n, int* status) {
+                                 const __nv_bfloat16* __restrict__ table2, int n_table2, const int32_t* __restrict__ rows2, int n, float scale, int* status) {
     const int a = rows[blockIdx.x], b = table2 ? rows2[blockIdx.x] : 0;
     const bool ok = a >= 0 && a < n_table && (!table2 || (b >= 0 && b < n_table2));
     if (!ok && threadIdx.x == 0) atomicOr(status, 1);
     for (int i = threadIdx.x; i < n; i += blockDim.x) {
         float v = ok ? __bfloat162float(table[(size_t)a * n + i]) : 0.f;
         if (ok && table2) v += __bfloat162float(table2[(size_t)b * n + i]);
+        v *= scale;
         out[(size_t)blockIdx.x * n + i] = v;
         if (copy) copy[(size_t)blockIdx.x * n + i] = v;
     }
@@ -635,8 +636,8 @@ extern "C" {
 cudaError_t ingot_support_embed_rows(float* out, const void* table, int is_f16, int n_in, int n_rows_table, const int32_t* rows_dev,
                                      int n_rows, int* status_dev, cudaStream_t s) {
     if (n_rows < 1 || n_in < 1) return cudaErrorInvalidValue;
-    if (is_f16) embed_rows_kernel<__half><<<n_rows, 256, 0, s>>>(out, static_cast<const __half*>(table), n_in, n_rows_table, rows_dev, status_dev);
-    else embed_rows_kernel<float><<<n_rows, 256, 0, s>>>(out, static_cast<const float*>(table), n_in, n_rows_table, rows_dev, status_dev);
+    if (is_f16) embed_rows_kernel<__half><<<n_rows, 256, 0, s>>>(out, static_cast<const __half*>(table), n_in, n_rows_table, rows_dev, status_dev, 1.0f);
+    else embed_rows_kernel<float><<<n_rows, 256, 0, s>>>(out, static_cast<const float*>(table), n_in, n_rows_table, rows_dev, status_dev, 1.0f);
     return cudaGetLastError();
 }
 
@@ -661,7 +662,7 @@ static cudaError_t gemv_group(float* const* outs, const void* const* ws, const v
     const bool plain = fmt == kFmtF16 || fmt == kFmtBF16;
     const int chunk = plain ? 256 : fmt == kFmtQ8_0 ? 512 : 1024;
     if (fmt < 0 || fmt > 3 || n_mat < 1 || n_mat > 3 || n_in % chunk != 0 || n_in > kGemvMaxIn ||
-        (swiglu && (n_mat != 2 || n_out[0] != n_out[1] || !norm_w)) || (!plain && !scales))
+        (swiglu && (n_mat != 2 || n_out[0] != n_out[1] || (!norm_w && fmt != kFmtBF16))) || (!plain && !scales))
         return cudaErrorInvalidValue;
     GemvGroup g = {};
     int total = 0;
@@ -681,6 +682,8 @@ static cudaError_t gemv_group(float* const* outs, const void* const* ws, const v
     typedef void (*Kernel)(GemvGroup, const float*, const float*, float, int, int, int, int, int, int);
     auto pick = [&](auto fmt_tag) -> Kernel {
         constexpr int F = decltype(fmt_tag)::value;
+        if constexpr (F == kFmtBF16)
+            if (swiglu && !norm_w) return short_rows ? gemv_stream_kernel<false, true, 6, F> : gemv_stream_kernel<false, true, 4, F>;
         return short_rows ? (swiglu ? gemv_stream_kernel<true, true, 6, F> : norm_w ? gemv_stream_kernel<true, false, 6, F> : gemv_stream_kernel<false, false, 6, F>)
                           : (swiglu ? gemv_stream_kernel<true, true, 4, F> : norm_w ? gemv_stream_kernel<true, false, 4, F> : gemv_stream_kernel<false, false, 4, F>);
     };
@@ -734,7 +737,7 @@ cudaError_t ingot_support_gemv_group(float* const* outs, const void* const* ws, 
 }
 
 // The same streaming kernel for one bf16 matrix [n_out][n_in] (n_in a multiple of 256): out (+)= W x', x' = rmsnorm(x) with the mean
-// over n_mean floats if norm_w is given. gated: W holds a gate and an up half of n_out rows each, out = act(gate) * up.
+// over n_mean floats if norm_w is given, else x itself. gated: W holds a gate and an up half of n_out rows each, out = act(gate) * up.
 cudaError_t ingot_support_gemv_bf16(float* out, const void* w, int n_out, int n_in, const float* x, const float* norm_w, float eps, int n_mean,
                                     int gated, int act, int accumulate, cudaStream_t s) {
     float* outs[2] = {out, out};
@@ -805,11 +808,11 @@ cudaError_t ingot_support_linear_bf16(float* out, const void* w, const float* x,
     return launch_linear<__nv_bfloat16>(out, w, x, x_ld, n_in, n_out, rows_per_block, n_tok, accumulate, s);
 }
 
-// Embedding rows of a bf16 table, widened to f32 (table rows n_in apart).
+// Embedding rows of a bf16 table, widened to f32 and scaled (table rows n_in apart).
 cudaError_t ingot_support_embed_rows_bf16(float* out, const void* table, int n_in, int n_rows_table, const int32_t* rows_dev, int n_rows,
-                                          int* status_dev, cudaStream_t s) {
+                                          float scale, int* status_dev, cudaStream_t s) {
     if (n_rows < 1 || n_in < 1) return cudaErrorInvalidValue;
-    embed_rows_kernel<__nv_bfloat16><<<n_rows, 256, 0, s>>>(out, static_cast<const __nv_bfloat16*>(table), n_in, n_rows_table, rows_dev, status_dev);
+    embed_rows_kernel<__nv_bfloat16><<<n_rows, 256, 0, s>>>(out, static_cast<const __nv_bfloat16*>(table), n_in, n_rows_table, rows_dev, status_dev, scale);
     return cudaGetLastError();
 }
 
@@ -826,12 +829,12 @@ cudaError_t ingot_support_gated_act(float* out, const float* in, int n_rows, int
     return support_launch(gated_act_kernel, dim3(unsigned((total + 255) / 256)), dim3(256), 0, s, out, in, n, total, act);
 }
 
-// out[r] (and copy[r], may be null) = table[rows[r]] + table2[rows2[r]] (table2 may be null); rows of n_in values.
+// out[r] (and copy[r], may be null) = scale * (table[rows[r]] + table2[rows2[r]]) (table2 may be null); rows of n_in values.
 cudaError_t ingot_support_embed_sum_bf16(float* out, float* copy, const void* table, int n_rows_table, const int32_t* rows_dev, const void* table2,
-                                         int n_rows_table2, const int32_t* rows2_dev, int n_in, int n_rows, int* status_dev, cudaStream_t s) {
+                                         int n_rows_table2, const int32_t* rows2_dev, int n_in, int n_rows, float scale, int* status_dev, cudaStream_t s) {
     if (n_rows < 1 || n_in < 1 || (table2 && !rows2_dev) || !status_dev) return cudaErrorInvalidValue;
     embed_sum_kernel<<<n_rows, 256, 0, s>>>(out, copy, static_cast<const __nv_bfloat16*>(table), n_rows_table, rows_dev,
-                                            static_cast<const __nv_bfloat16*>(table2), n_rows_table2, rows2_dev, n_in, status_dev);
+                                            static_cast<const __nv_bfloat16*>(table2), n_rows_table2, rows2_dev, n_in, scale, status_dev);
     return cudaGetLastError();
 }
 

@@ -109,6 +109,7 @@ __global__ void __launch_bounds__(kAppendThreads) shared_kv_append_kernel(const 
 }
 
 // ---- plain form: f32 arithmetic on the FMA pipes, any row length up to 1024, f32 or f16 rows -------------------------
+// The key is the row or its first q_dim columns, the value its out_dim columns from v_off on.
 // A CTA owns 16 (token, head) rows of one KV head - 4 per warp - and walks the visible keys 32 at a time through shared
 // memory: lane = key for the scores, lane = dims for the weighted sum.
 constexpr int kRows = 16, kKeys = 32;
@@ -121,7 +122,7 @@ __global__ void __launch_bounds__(128) shared_kv_attend_kernel(const AttendParam
     const int group = p.n_head / p.n_head_kv, len = p.st.len[seq];
     const int row0 = blockIdx.x * kRows, n_rows = len * group;
     if (row0 >= n_rows) return;
-    const int dim = p.dim, ldk = kD * 32 + 1;
+    const int dim = p.dim, ldk = kD * 32 + 1, q_dim = p.q_dim > 0 ? p.q_dim : dim;
     float* sq = smem;                       // [16][kD * 32]
     float* sk = sq + kRows * kD * 32;       // [32][kD * 32 + 1]
     float* sr = sk + kKeys * ldk;           // [32] 1/rms * scale
@@ -133,7 +134,7 @@ __global__ void __launch_bounds__(128) shared_kv_attend_kernel(const AttendParam
         const int r = i / (kD * 32), d = i - r * (kD * 32);
         const int rr = row0 + r;
         float v = 0.f;
-        if (rr < n_rows && d < dim) v = widen(static_cast<const T*>(p.q)[((tok0 + rr / group) * p.n_head + kvh * group + rr % group) * dim + d]);
+        if (rr < n_rows && d < q_dim) v = widen(static_cast<const T*>(p.q)[((tok0 + rr / group) * p.n_head + kvh * group + rr % group) * q_dim + d]);
         sq[i] = v;
     }
     int lo[4], hi[4];  // visible keys lo..hi of this warp's rows (none: hi < lo)
@@ -173,7 +174,7 @@ __global__ void __launch_bounds__(128) shared_kv_attend_kernel(const AttendParam
             const float* qr = sq + (warp * 4 + r) * kD * 32;
             const float* kr = sk + lane * ldk;
             float s0 = 0.f, s1 = 0.f;
-            for (int d = 0; d < dim; d += 2) {
+            for (int d = 0; d < q_dim; d += 2) {
                 s0 = fmaf(qr[d], kr[d], s0);
                 s1 = fmaf(qr[d + 1], kr[d + 1], s1);
             }
@@ -190,7 +191,8 @@ __global__ void __launch_bounds__(128) shared_kv_attend_kernel(const AttendParam
                 const float pk = __shfl_sync(0xffffffffu, e, k);
                 if (pk == 0.f) continue;  // warp-uniform
 #pragma unroll
-                for (int i = 0; i < kD; i++) acc[r][i] = fmaf(pk, sk[k * ldk + lane + 32 * i], acc[r][i]);
+                for (int i = 0; i < kD; i++)
+                    if (p.v_off + 32 * i < kD * 32) acc[r][i] = fmaf(pk, sk[k * ldk + p.v_off + lane + 32 * i], acc[r][i]);
             }
         }
     }
@@ -206,7 +208,9 @@ __global__ void __launch_bounds__(128) shared_kv_attend_kernel(const AttendParam
 #pragma unroll
         for (int i = 0; i < kD; i++) {
             const int d = lane + 32 * i;
-            if (d < p.out_dim) p.out.store(tok0 + rr / group, (kvh * group + rr % group) * p.out_dim + d, acc[r][i] * inv);
+            const size_t row = tok0 + rr / group;
+            const int h = kvh * group + rr % group;
+            if (d < p.out_dim) p.out.store(row, h * p.out_dim + d, acc[r][i] * inv * p.gate.at(row, h, p.out_dim, d));
         }
     }
 }
@@ -679,7 +683,7 @@ int launch_mma(ingot_skv* kv, AttendParams p, cudaStream_t s) {
     return INGOT_OK;
 }
 
-int create(ingot_skv** out, int n_layer, int n_head_kv, int head_dim, int dtype, int chunk, int window, int n_blocks, bool scales, const char* who) {
+int create(ingot_skv** out, int n_layer, int n_head_kv, int head_dim, int dtype, int chunk, int window, int n_blocks, bool scales, bool tiles, const char* who) {
     *out = nullptr;
     INGOT_REQUIRE(n_layer >= 1 && n_head_kv >= 1 && n_blocks >= 1 && chunk >= 0 && window >= 0, std::string(who) + ": bad sizes");
     INGOT_REQUIRE(dtype == INGOT_F32 || dtype == INGOT_F16, std::string(who) + ": rows are f32 or f16");
@@ -691,7 +695,7 @@ int create(ingot_skv** out, int n_layer, int n_head_kv, int head_dim, int dtype,
     ingot_skv* kv = new (std::nothrow) ingot_skv();
     if (!kv) return INGOT_ERR_NOMEM;
     kv->n_layer = n_layer; kv->n_head_kv = n_head_kv; kv->dim = head_dim; kv->dtype = dtype; kv->chunk = chunk; kv->window = window; kv->n_blocks = n_blocks;
-    kv->tiled = !scales && dtype == INGOT_F16 && head_dim % 64 == 0;
+    kv->tiled = tiles && dtype == INGOT_F16 && head_dim % 64 == 0;
     kv->layer_elems = (size_t)n_blocks * n_head_kv * kBlockTokens * head_dim;
     const size_t bytes = kv->layer_elems * n_layer * (dtype == INGOT_F32 ? 4 : 2), scale_bytes = (size_t)n_layer * n_blocks * kBlockTokens * 4;
     cudaError_t e;
@@ -723,12 +727,17 @@ extern "C" {
 
 int ingot_skv_create(ingot_skv** out, int n_layer, int n_head_kv, int head_dim, int dtype, int chunk, int n_blocks) {
     INGOT_REQUIRE(out != nullptr, "ingot_skv_create: out is null");
-    return create(out, n_layer, n_head_kv, head_dim, dtype, chunk, 0, n_blocks, true, "ingot_skv_create");
+    return create(out, n_layer, n_head_kv, head_dim, dtype, chunk, 0, n_blocks, true, false, "ingot_skv_create");
 }
 
 int ingot_skv_create_window(ingot_skv** out, int n_layer, int n_head_kv, int row_length, int dtype, int window, int n_blocks) {
     INGOT_REQUIRE(out != nullptr, "ingot_skv_create_window: out is null");
-    return create(out, n_layer, n_head_kv, row_length, dtype, 0, window, n_blocks, false, "ingot_skv_create_window");
+    return create(out, n_layer, n_head_kv, row_length, dtype, 0, window, n_blocks, false, true, "ingot_skv_create_window");
+}
+
+int ingot_skv_create_joined(ingot_skv** out, int n_layer, int n_head_kv, int row_length, int dtype, int window, int n_blocks) {
+    INGOT_REQUIRE(out != nullptr, "ingot_skv_create_joined: out is null");
+    return create(out, n_layer, n_head_kv, row_length, dtype, 0, window, n_blocks, false, false, "ingot_skv_create_joined");
 }
 
 void ingot_skv_destroy(ingot_skv* kv) {

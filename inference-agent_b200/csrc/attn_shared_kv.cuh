@@ -19,7 +19,7 @@ struct ingot_skv {
     float* part = nullptr;  // split-key partials of decoded tokens, grown on demand
     size_t part_floats = 0;
     std::vector<void*> retired;
-    std::vector<CUtensorMap> tmaps;  // per layer, 128-value f16 rows only: [page * kv head][16][128] in boxes of 16 x 64
+    std::vector<CUtensorMap> tmaps;  // per layer, f16 rows in plain order: [page * kv head][16][row] in boxes of 16 x 64
 };
 
 // Which keys a position sees and which page holds it: the whole past, its own chunk, or a window that slides along.
@@ -71,6 +71,27 @@ struct SharedOut {
     }
 };
 
+// A factor sigmoid(z) of the result: z one number per (token, head) or one per value (null: none).
+struct OutGate {
+    const float* z = nullptr;
+    int ld = 0, per_head = 0;
+    __device__ __forceinline__ static float sigmoid(float v) { return 1.0f / (1.0f + expf(-v)); }
+    __device__ __forceinline__ float at(size_t row, int head, int out_dim, int d) const {
+        if (!z) return 1.0f;
+        return sigmoid(z[row * ld + (per_head ? head : head * out_dim + d)]);
+    }
+    // Columns d..d+3 of a head; rows, heads and d start on 16 bytes.
+    __device__ __forceinline__ float4 at4(size_t row, int head, int out_dim, int d) const {
+        if (!z) return make_float4(1.f, 1.f, 1.f, 1.f);
+        if (per_head) {
+            const float g = sigmoid(z[row * ld + head]);
+            return make_float4(g, g, g, g);
+        }
+        const float4 v = *reinterpret_cast<const float4*>(z + row * ld + head * out_dim + d);
+        return make_float4(sigmoid(v.x), sigmoid(v.y), sigmoid(v.z), sigmoid(v.w));
+    }
+};
+
 // Block of a page of sequence `seq` (index within the step), or -1 with the status bit raised if the table has none.
 __device__ __forceinline__ int table_block(const int32_t* tables, const int32_t* first_page, int max_blocks, int n_blocks, int seq, int page, int* status) {
     const int i = page - (first_page ? first_page[seq] : 0);
@@ -95,6 +116,9 @@ struct AttendParams {
     float* part;    // [token][head][split][dim + 2]
     bool tiled = false;           // order of the pages
     const float* sink = nullptr;  // per head: one more term exp(sink) of the denominator (null: none)
+    int q_dim = 0;                // columns of the row that are the key (0: all of them), and the first one of the value
+    int v_off = 0;
+    OutGate gate = {};
 };
 
 // The plain kernel (f32 arithmetic, any row length up to 1024, window, chunk and sink); dtype of rows and queries.
@@ -105,6 +129,10 @@ int launch_shared_kv_plain(const AttendParams& p, int dtype, cudaStream_t stream
 bool latent_decode_takes(int row, int rank);
 int latent_decode_heads(int n_head);
 int launch_latent_decode_sm100(const ingot_skv* kv, const AttendParams& p, cudaStream_t stream);
+
+// Attention over joined [key | value] rows for portions of prompts on tcgen05 (attn_gqa_sm100.cu): which sizes it takes, and the launch.
+bool gqa_sm100_takes(int dim, int vdim, float scale);
+int launch_gqa_sm100(ingot_skv* kv, int layer, const AttendParams& p, cudaStream_t stream);
 
 // tcgen05 form for portions of prompts over rows of 128 values (attn_shared_kv_sm100.cu); INGOT_ERR_UNSUPPORTED if the driver
 // cannot encode its tensor map.

@@ -46,6 +46,102 @@ __global__ void __launch_bounds__(128) moe_select_kernel(const float* logits, in
     }
 }
 
+// Routers that choose by softmax score plus a correction, within the best groups of neighbouring outputs, and weigh by the score alone.
+// One warp per token; the outputs behind the experts' are identity experts (the input itself) and, if asked for, one gate.
+struct GroupedRouter {
+    ingot_moe_router r;
+    const float* logits;
+    int ld, n_tok;
+    int32_t* expert_of;
+    float* weight_of;
+    int32_t* row_of;
+    float *self_gain, *shared_gain;
+};
+// The largest of get(0..n-1) below (last, -last_i) in the order of (value, lower index first); -1 if there is none.
+template <class F>
+__device__ __forceinline__ int warp_next_largest(int n, float last, int last_i, float* value, F&& get) {
+    const int lane = threadIdx.x & 31;
+    float best = -INFINITY;
+    int best_i = n;
+    for (int i = lane; i < n; i += 32) {
+        const float v = get(i);
+        if ((v < last || (v == last && i > last_i)) && (v > best || best_i == n)) { best = v; best_i = i; }
+    }
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) {
+        const float v = __shfl_xor_sync(0xffffffffu, best, o);
+        const int i = __shfl_xor_sync(0xffffffffu, best_i, o);
+        if (i < n && (best_i == n || v > best || (v == best && i < best_i))) { best = v; best_i = i; }
+    }
+    *value = best;
+    return best_i < n ? best_i : -1;
+}
+constexpr int kRouterOutputs = 1024, kRouterWarps = 4;  // most outputs of a router (experts and identity experts)
+__global__ void __launch_bounds__(kRouterWarps * 32) moe_select_grouped_kernel(const GroupedRouter p) {
+    extern __shared__ float s_choice_all[];  // per warp: choice scores [n], group scores [count], weights [top]
+    INGOT_PDL_TRIGGER();
+    INGOT_PDL_WAIT();
+    const int t = blockIdx.x * kRouterWarps + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+    if (t >= p.n_tok) return;
+    const int n = p.r.n_expert + p.r.n_identity, top = p.r.top, count = p.r.groups, per = n / count;
+    float* choice = s_choice_all + (threadIdx.x >> 5) * (n + count + top);
+    float *group = choice + n, *weight = group + count;
+    const float* z = p.logits + (size_t)t * p.ld;
+    float most = -INFINITY;
+    for (int e = lane; e < n; e += 32) most = fmaxf(most, z[e]);
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) most = fmaxf(most, __shfl_xor_sync(0xffffffffu, most, o));
+    float sum = 0.f;
+    for (int e = lane; e < n; e += 32) sum += expf(z[e] - most);
+    const float inv = 1.0f / warp_sum(sum);
+    for (int e = lane; e < n; e += 32) {
+        const float c = expf(z[e] - most) * inv + (p.r.correction ? p.r.correction[e] : 0.f);
+        choice[e] = c == c ? c : -INFINITY;
+    }
+    __syncwarp();
+    if (p.r.keep < count) {
+        for (int g = lane; g < count; g += 32) {
+            float best = -INFINITY;
+            for (int i = 0; i < per; i++) best = fmaxf(best, choice[g * per + i]);
+            group[g] = best;
+        }
+        __syncwarp();
+        // groups at and above the keep-th best are open
+        float last = INFINITY;
+        int last_g = -1;
+        for (int k = 0; k < p.r.keep; k++) last_g = warp_next_largest(count, last, last_g, &last, [&](int g) { return group[g]; });
+        __syncwarp();
+        for (int e = lane; e < n; e += 32) {
+            const int g = e / per;
+            if (group[g] < last || (group[g] == last && g > last_g)) choice[e] = -INFINITY;
+        }
+        __syncwarp();
+    }
+    float last = INFINITY, total = 0.f;
+    int last_e = -1;
+    for (int k = 0; k < top; k++) {
+        last_e = warp_next_largest(n, last, last_e, &last, [&](int e) { return choice[e]; });
+        const float s = expf(z[last_e] - most) * inv;
+        total += s;
+        if (lane == 0) {
+            weight[k] = s;
+            p.expert_of[(size_t)t * top + k] = last_e;
+        }
+    }
+    if (lane == 0) {
+        const float f = p.r.scale / (total + 1e-20f);
+        float self = 0.f;
+        for (int k = 0; k < top; k++) {
+            const float w = weight[k] * f;
+            const size_t pair = (size_t)t * top + k;
+            p.weight_of[pair] = w;
+            if (p.expert_of[pair] >= p.r.n_expert) { self += w; p.row_of[pair] = -1; }
+        }
+        if (p.self_gain) p.self_gain[t] = self;
+        if (p.shared_gain) p.shared_gain[t] = 1.0f / (1.0f + expf(-z[n]));
+    }
+}
+
 // One CTA per expert: where its rows start (pairs of lower experts), then its pairs in order. A thread owns a run of pairs, so one scan
 // over the threads' counts places them all.
 constexpr int kSortThreads = 1024;
@@ -88,7 +184,11 @@ __global__ void __launch_bounds__(kSortThreads) moe_sort_kernel(const int32_t* e
     }
     if (threadIdx.x == 0) {
         group_start[e] = row;
-        if (e == n_expert - 1) group_start[n_expert] = n_pairs;
+        if (e == n_expert - 1) {  // pairs of what lies behind the experts have no rows
+            int all = row;
+            for (int w = 0; w < kSortThreads / 32; w++) all += s_mine[w];
+            group_start[n_expert] = all;
+        }
     }
     if (mine == 0) return;
     for (int i = first; i < last; i++)
@@ -100,10 +200,12 @@ __global__ void __launch_bounds__(kSortThreads) moe_sort_kernel(const int32_t* e
         }
 }
 
-// bf16 planes of the rows: row r is its token's row.
-__global__ void __launch_bounds__(128) moe_gather_kernel(uint4* hi, uint4* lo, const uint4* src_hi, const uint4* src_lo, const int32_t* pair_of, int top, int n8) {
+// bf16 planes of the rows: row r is its token's row. n_rows (device, may be null): how many of the launch's rows there are.
+__global__ void __launch_bounds__(128) moe_gather_kernel(uint4* hi, uint4* lo, const uint4* src_hi, const uint4* src_lo, const int32_t* pair_of, int top, int n8,
+                                                         const int32_t* n_rows) {
     INGOT_PDL_TRIGGER();
     INGOT_PDL_WAIT();
+    if (n_rows && (int)blockIdx.x >= *n_rows) return;
     const size_t r = blockIdx.x, t = size_t(pair_of[r] / top);
     for (int i = threadIdx.x; i < n8; i += 128) {
         hi[r * n8 + i] = src_hi[t * n8 + i];
@@ -113,7 +215,11 @@ __global__ void __launch_bounds__(128) moe_gather_kernel(uint4* hi, uint4* lo, c
 
 // Plain products: out[row][o] = act(row_weight * W_e[o] . x[source(row)]), f32 arithmetic on bf16 weights. A warp owns one output of
 // up to kRowTile rows of one expert; grid.y counts row tiles, expert after expert.
+// kGated: the matrices hold gate and up rows interleaved (gate_row), an output is row_weight * silu(gate) * up.
 constexpr int kRowTile = 8;
+__device__ __forceinline__ int gate_row(int o) { return o / 32 * 64 + o % 32; }  // the up row is 32 further on
+__device__ __forceinline__ float silu(float v) { return v / (1.0f + expf(-v)); }
+template <bool kGated>
 __global__ void __launch_bounds__(256) moe_linear_kernel(float* out, const __nv_bfloat16* w, const float* x, int x_ld, int n_in, int n_out, int n_expert,
                                                          const int32_t* group_start, const int32_t* pair_of, int top, const float* row_weight, int act) {
     INGOT_PDL_TRIGGER();
@@ -145,39 +251,47 @@ __global__ void __launch_bounds__(256) moe_linear_kernel(float* out, const __nv_
     if (e < 0) return;
     const int o = blockIdx.x * 8 + warp;
     if (o >= n_out) return;
-    const __nv_bfloat16* wr = w + ((size_t)e * n_out + o) * n_in;
+    const __nv_bfloat16* wr = w + (kGated ? (size_t)e * 2 * n_out + gate_row(o) : (size_t)e * n_out + o) * n_in;
     const float* xr[kRowTile];
 #pragma unroll
     for (int i = 0; i < kRowTile; i++) {
         const int r = min(r0 + i, r1 - 1);
         xr[i] = x + (size_t)(pair_of ? pair_of[r] / top : r) * x_ld;
     }
-    float acc[kRowTile];
+    float acc[kRowTile], up[kRowTile];
 #pragma unroll
-    for (int i = 0; i < kRowTile; i++) acc[i] = 0.f;
-    for (int c = lane * 8; c < n_in; c += 256) {
-        const uint4 raw = *reinterpret_cast<const uint4*>(wr + c);
+    for (int i = 0; i < kRowTile; i++) acc[i] = up[i] = 0.f;
+    auto widen = [](const uint4& raw, float (&wv)[8]) {
         const uint32_t u[4] = {raw.x, raw.y, raw.z, raw.w};
-        float wv[8];
 #pragma unroll
         for (int i = 0; i < 4; i++) {
             wv[2 * i] = __uint_as_float(u[i] << 16);
             wv[2 * i + 1] = __uint_as_float(u[i] & 0xffff0000u);
         }
+    };
+    auto dot = [](const float (&wv)[8], const float4& a, const float4& b, float v) {
+        v = fmaf(wv[0], a.x, v); v = fmaf(wv[1], a.y, v);
+        v = fmaf(wv[2], a.z, v); v = fmaf(wv[3], a.w, v);
+        v = fmaf(wv[4], b.x, v); v = fmaf(wv[5], b.y, v);
+        v = fmaf(wv[6], b.z, v); return fmaf(wv[7], b.w, v);
+    };
+    for (int c = lane * 8; c < n_in; c += 256) {
+        float wv[8], uv[8];
+        widen(*reinterpret_cast<const uint4*>(wr + c), wv);
+        if (kGated) widen(*reinterpret_cast<const uint4*>(wr + (size_t)32 * n_in + c), uv);
 #pragma unroll
         for (int i = 0; i < kRowTile; i++) {
             if (r0 + i >= r1) break;
             const float4 a = *reinterpret_cast<const float4*>(xr[i] + c), b = *reinterpret_cast<const float4*>(xr[i] + c + 4);
-            acc[i] = fmaf(wv[0], a.x, acc[i]); acc[i] = fmaf(wv[1], a.y, acc[i]);
-            acc[i] = fmaf(wv[2], a.z, acc[i]); acc[i] = fmaf(wv[3], a.w, acc[i]);
-            acc[i] = fmaf(wv[4], b.x, acc[i]); acc[i] = fmaf(wv[5], b.y, acc[i]);
-            acc[i] = fmaf(wv[6], b.z, acc[i]); acc[i] = fmaf(wv[7], b.w, acc[i]);
+            acc[i] = dot(wv, a, b, acc[i]);
+            if (kGated) up[i] = dot(uv, a, b, up[i]);
         }
     }
 #pragma unroll
     for (int i = 0; i < kRowTile; i++) {
         if (r0 + i >= r1) break;
         float v = warp_sum(acc[i]);
+        if (kGated) v = silu(v) * warp_sum(up[i]);
         if (lane == 0) {
             if (row_weight) v *= row_weight[r0 + i];
             if (act == INGOT_ACT_RELU2) v = v > 0.f ? v * v : 0.f;
@@ -187,8 +301,10 @@ __global__ void __launch_bounds__(256) moe_linear_kernel(float* out, const __nv_
 }
 
 // The same for the few rows of one token, bound by streaming the weights: a warp owns two outputs of one row and keeps eight 16-byte
-// weight loads in flight while it multiplies the eight before; the row's x is read once for both.
+// weight loads in flight while it multiplies the eight before; the row's x is read once for both. kGated: the two are the gate and the
+// up row of one output.
 constexpr int kGemvLoads = 4;
+template <bool kGated>
 __global__ void __launch_bounds__(256) moe_gemv_kernel(float* out, const __nv_bfloat16* w, const float* x, int x_ld, int n_in, int n_out, const int32_t* group_start,
                                                        int n_expert, const int32_t* pair_of, int top, const float* row_weight, int act) {
     INGOT_PDL_TRIGGER();
@@ -199,11 +315,11 @@ __global__ void __launch_bounds__(256) moe_gemv_kernel(float* out, const __nv_bf
         const bool past = e0 + lane < n_expert && group_start[e0 + lane + 1] <= row;
         e += __popc(__ballot_sync(0xffffffffu, past));
     }
-    const int o = (blockIdx.x * 8 + warp) * 2;
+    const int o = (blockIdx.x * 8 + warp) * (kGated ? 1 : 2);
     if (o >= n_out || e >= n_expert) return;
-    const bool two = o + 1 < n_out;
-    const uint4* wa = reinterpret_cast<const uint4*>(w + ((size_t)e * n_out + o) * n_in);
-    const uint4* wb = two ? wa + n_in / 8 : wa;
+    const bool two = !kGated && o + 1 < n_out;
+    const uint4* wa = reinterpret_cast<const uint4*>(w + (kGated ? (size_t)e * 2 * n_out + gate_row(o) : (size_t)e * n_out + o) * n_in);
+    const uint4* wb = kGated ? wa + (size_t)32 * (n_in / 8) : two ? wa + n_in / 8 : wa;
     const float* xr = x + (size_t)(pair_of ? pair_of[row] / top : row) * x_ld;
     const int n8 = n_in / 8;
     const uint4 zero = make_uint4(0, 0, 0, 0);
@@ -245,6 +361,7 @@ __global__ void __launch_bounds__(256) moe_gemv_kernel(float* out, const __nv_bf
     acc_b = warp_sum(acc_b);
     if (lane == 0) {
         const float f = row_weight ? row_weight[row] : 1.0f;
+        if (kGated) acc_a = silu(acc_a) * acc_b;
         acc_a *= f;
         acc_b *= f;
         if (act == INGOT_ACT_RELU2) {
@@ -286,11 +403,35 @@ int ingot_moe_route(const float* logits_dev, int ld, int n_tok, int n_expert, in
     return INGOT_OK;
 }
 
-int ingot_moe_gather(void* hi_dev, void* lo_dev, const void* src_hi_dev, const void* src_lo_dev, const int32_t* pair_of_dev, int n_rows, int top, int n, void* stream) {
+int ingot_moe_route_grouped(const ingot_moe_router* router, const float* logits_dev, int ld, int n_tok, int32_t* expert_of_dev, float* weight_of_dev,
+                            int32_t* group_start_dev, int32_t* row_of_dev, int32_t* pair_of_dev, float* row_weight_dev, float* self_gain_dev, float* shared_gain_dev,
+                            void* stream) {
+    INGOT_REQUIRE(router && logits_dev && expert_of_dev && weight_of_dev && group_start_dev && row_of_dev && pair_of_dev && row_weight_dev,
+                  "ingot_moe_route_grouped: null argument");
+    const ingot_moe_router& r = *router;
+    const int n = r.n_expert + r.n_identity;
+    INGOT_REQUIRE(n_tok >= 1 && r.n_expert >= 1 && r.n_identity >= 0 && r.groups >= 1 && n % r.groups == 0 && r.keep >= 1 && r.keep <= r.groups && r.top >= 1 &&
+                      r.top <= n / r.groups * r.keep && ld >= n + (shared_gain_dev ? 1 : 0) && (long long)n_tok * r.top < (1ll << 30) &&
+                      (r.n_identity == 0 || self_gain_dev), "ingot_moe_route_grouped: bad sizes");
+    if (n > kRouterOutputs) {
+        ingot_set_error("ingot_moe_route_grouped: at most " + std::to_string(kRouterOutputs) + " experts");
+        return INGOT_ERR_UNSUPPORTED;
+    }
+    cudaStream_t s = static_cast<cudaStream_t>(stream);
+    const GroupedRouter p = {r, logits_dev, ld, n_tok, expert_of_dev, weight_of_dev, row_of_dev, self_gain_dev, shared_gain_dev};
+    const size_t smem = size_t(kRouterWarps) * (n + r.groups + r.top) * sizeof(float);
+    INGOT_CUDA_TRY(ingot_launch_pdl(moe_select_grouped_kernel, dim3((n_tok + kRouterWarps - 1) / kRouterWarps), dim3(kRouterWarps * 32), smem, s, p));
+    INGOT_CUDA_TRY(ingot_launch_pdl(moe_sort_kernel, dim3(r.n_expert), dim3(kSortThreads), 0, s, (const int32_t*)expert_of_dev, (const float*)weight_of_dev, n_tok * r.top,
+                                    r.n_expert, group_start_dev, row_of_dev, pair_of_dev, row_weight_dev));
+    return INGOT_OK;
+}
+
+int ingot_moe_gather(void* hi_dev, void* lo_dev, const void* src_hi_dev, const void* src_lo_dev, const int32_t* pair_of_dev, int n_rows, const int32_t* n_rows_dev, int top,
+                     int n, void* stream) {
     INGOT_REQUIRE(hi_dev && src_hi_dev && pair_of_dev && (!lo_dev || src_lo_dev), "ingot_moe_gather: null argument");
     INGOT_REQUIRE(n_rows >= 1 && top >= 1 && n >= 8 && n % 8 == 0, "ingot_moe_gather: bad sizes");
     INGOT_CUDA_TRY(ingot_launch_pdl(moe_gather_kernel, dim3(n_rows), dim3(128), 0, static_cast<cudaStream_t>(stream), static_cast<uint4*>(hi_dev), static_cast<uint4*>(lo_dev),
-                                    static_cast<const uint4*>(src_hi_dev), static_cast<const uint4*>(src_lo_dev), pair_of_dev, top, n / 8));
+                                    static_cast<const uint4*>(src_hi_dev), static_cast<const uint4*>(src_lo_dev), pair_of_dev, top, n / 8, n_rows_dev));
     return INGOT_OK;
 }
 
@@ -298,15 +439,22 @@ int ingot_moe_linear(float* out_dev, const void* w_dev, const float* x_dev, int 
                      const int32_t* pair_of_dev, int top, const float* row_weight_dev, int act, void* stream) {
     INGOT_REQUIRE(out_dev && w_dev && x_dev && group_start_dev, "ingot_moe_linear: null argument");
     INGOT_REQUIRE(n_in >= 8 && n_in % 8 == 0 && x_ld % 4 == 0 && n_out >= 1 && n_expert >= 1 && n_rows >= 1 && top >= 1, "ingot_moe_linear: bad sizes");
+    const bool gated = act == INGOT_ACT_SILU_GATED;
+    INGOT_REQUIRE(!gated || n_out % 32 == 0, "ingot_moe_linear: gated outputs come in runs of 32");
+    cudaStream_t s = static_cast<cudaStream_t>(stream);
+    const __nv_bfloat16* w = static_cast<const __nv_bfloat16*>(w_dev);
     if (n_rows <= 2 * top) {  // one token (or two): a row per expert, as good as always
-        INGOT_CUDA_TRY(ingot_launch_pdl(moe_gemv_kernel, dim3((n_out + 15) / 16, n_rows), dim3(256), 0, static_cast<cudaStream_t>(stream), out_dev,
-                                        static_cast<const __nv_bfloat16*>(w_dev), x_dev, x_ld, n_in, n_out, group_start_dev, n_expert, pair_of_dev, top, row_weight_dev, act));
+        auto kernel = gated ? moe_gemv_kernel<true> : moe_gemv_kernel<false>;
+        const int per = gated ? 8 : 16;
+        INGOT_CUDA_TRY(ingot_launch_pdl(kernel, dim3((n_out + per - 1) / per, n_rows), dim3(256), 0, s, out_dev, w, x_dev, x_ld, n_in, n_out, group_start_dev, n_expert, pair_of_dev,
+                                        top, row_weight_dev, act));
         return INGOT_OK;
     }
     const int tiles = n_rows / kRowTile + (n_rows < n_expert ? n_rows : n_expert);  // at least as many as there can be
     INGOT_REQUIRE(tiles <= 65535, "ingot_moe_linear: too many rows");
-    INGOT_CUDA_TRY(ingot_launch_pdl(moe_linear_kernel, dim3((n_out + 7) / 8, tiles), dim3(256), 0, static_cast<cudaStream_t>(stream), out_dev,
-                                    static_cast<const __nv_bfloat16*>(w_dev), x_dev, x_ld, n_in, n_out, n_expert, group_start_dev, pair_of_dev, top, row_weight_dev, act));
+    auto kernel = gated ? moe_linear_kernel<true> : moe_linear_kernel<false>;
+    INGOT_CUDA_TRY(ingot_launch_pdl(kernel, dim3((n_out + 7) / 8, tiles), dim3(256), 0, s, out_dev, w, x_dev, x_ld, n_in, n_out, n_expert, group_start_dev, pair_of_dev, top,
+                                    row_weight_dev, act));
     return INGOT_OK;
 }
 

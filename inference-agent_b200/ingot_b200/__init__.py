@@ -58,6 +58,9 @@ ABI = {
     "ingot_gated_lru": (_I, [_P, _P, _P, _I, _P, _I, _I, _P, _P, _P, _P, _I, _P, _P, _I, C.c_float, _I, _P, _P]),
     "ingot_skv_create": (_I, [C.POINTER(_P), _I, _I, _I, _I, _I, _I]),
     "ingot_skv_create_window": (_I, [C.POINTER(_P), _I, _I, _I, _I, _I, _I]),
+    "ingot_skv_create_joined": (_I, [C.POINTER(_P), _I, _I, _I, _I, _I, _I]),
+    "ingot_gqa_append": (_I, [_P, _I, _P, _P, _I, _I, _I, _I, _P, _P, _P, C.c_float, _P, C.c_float, _P, _I, C.c_float, _P, _P, _P, _I, _P]),
+    "ingot_gqa_attend": (_I, [_P, _I, _P, _P, _P, C.c_float, _P, _P, _I, _I, _P, _P, _P, _I, _I, _P]),
     "ingot_skv_destroy": (None, [_P]),
     "ingot_skv_pages": (_I, [_I, _I]),
     "ingot_skv_row_length": (_I, [_I]),
@@ -70,7 +73,8 @@ ABI = {
     "ingot_latent_queries": (_I, [_P, _P, _I, _I, _I, _P, _P]),
     "ingot_latent_attend": (_I, [_P, _I, _P, _P, _I, _I, C.c_float, _P, _P, _P, _P, _I, _I, _P]),
     "ingot_moe_route": (_I, [_P, _I, _I, _I, _I, _P, _P, _P, _P, _P, _P, _P]),
-    "ingot_moe_gather": (_I, [_P, _P, _P, _P, _P, _I, _I, _I, _P]),
+    "ingot_moe_route_grouped": (_I, [_P, _P, _I, _I, _P, _P, _P, _P, _P, _P, _P, _P, _P]),
+    "ingot_moe_gather": (_I, [_P, _P, _P, _P, _P, _I, _P, _I, _I, _P]),
     "ingot_moe_linear": (_I, [_P, _P, _P, _I, _I, _I, _I, _I, _P, _P, _I, _P, _I, _P]),
     "ingot_moe_add": (_I, [_P, _P, _P, _I, _I, _I, _P]),
     "ingot_skv_attend": (_I, [_P, _I, _P, _P, _I, _I, C.c_float, C.c_float, _P, _P, _P, _I, _I, _P]),

@@ -120,6 +120,6 @@ def test_plain_experts_against_the_mixture(n, experts, top, d, ff):
     assert np.abs(xd.cpu().numpy() - want).max() < 1e-4
     planes = bf16(h)
     gathered = torch.zeros(n * top, d, device="cuda", dtype=torch.bfloat16)
-    lib(lib().ingot_moe_gather(p(gathered), None, p(planes), None, p(pd), n * top, top, d, None))
+    lib(lib().ingot_moe_gather(p(gathered), None, p(planes), None, p(pd), n * top, None, top, d, None))
     torch.cuda.synchronize()
     assert torch.equal(gathered, planes[torch.from_numpy(pair // top).cuda().long()])
