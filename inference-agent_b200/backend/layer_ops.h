@@ -236,7 +236,11 @@ public:
         if (design.centred) n.b = load(name + ".b", 0.f);
         return n;
     }
-    float scalar(const std::string& name) { return tensor_f32(dir.tensor(name, {}))[0]; }
+    float scalar(const std::string& name) {
+        const TensorView& t = dir.tensor(name);
+        if (t.elems() != 1) throw std::runtime_error("model: tensor " + name + " is not one number");
+        return tensor_f32(t)[0];
+    }
     const TensorView& bf16(const std::string& name, const std::vector<int64_t>& shape) const {
         const TensorView& t = dir.tensor(name, shape);
         if (t.dtype != "BF16") throw std::runtime_error("model: tensor " + name + " has type " + t.dtype + ", expected BF16");

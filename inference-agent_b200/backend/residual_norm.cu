@@ -56,8 +56,8 @@ __device__ __forceinline__ float4 apply(float4 v, float2 m, const ingot_norm& n,
     return o;
 }
 
-template <int kKeep>
-__global__ void residual_norm_kernel(const ingot_residual_norm p) {
+template <int kKeep, int kThreads>
+__global__ void __launch_bounds__(kThreads) residual_norm_kernel(const ingot_residual_norm p) {
     __shared__ float red[32];
     INGOT_PDL_TRIGGER();
     INGOT_PDL_WAIT();
@@ -150,9 +150,11 @@ extern "C" cudaError_t ingot_residual_norm_run(const ingot_residual_norm* r, cud
         (r->top > 0 && (!r->branch || !r->row_of)) || (r->self_gain && !r->self.w) || (r->next.w && !r->out && !r->hi))
         return cudaErrorInvalidValue;
     auto run = [&](auto kernel, int threads) { return ingot_launch_pdl(kernel, dim3(r->n_rows), dim3(threads), 0, s, *r); };
-    if (r->n <= 1024) return run(residual_norm_kernel<1>, (r->n / 4 + 31) / 32 * 32);
-    if (r->n <= 4096) return run(residual_norm_kernel<4>, (r->n / 16 + 31) / 32 * 32);
-    if (r->n <= 8192) return run(residual_norm_kernel<8>, 256);
-    if (r->n <= 32768) return run(residual_norm_kernel<8>, 1024);
+    const int quads = r->n / 4;
+    auto warps = [&](int keep) { return (quads + 32 * keep - 1) / (32 * keep) * 32; };  // threads that hold a row of `keep` quads each
+    if (quads <= 256) return run(residual_norm_kernel<1, 256>, warps(1));
+    if (quads <= 1024) return run(residual_norm_kernel<4, 256>, warps(4));
+    if (quads <= 2048) return run(residual_norm_kernel<8, 256>, 256);
+    if (quads <= 8192) return run(residual_norm_kernel<8, 1024>, 1024);
     return cudaErrorInvalidValue;
 }

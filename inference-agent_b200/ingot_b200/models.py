@@ -136,7 +136,7 @@ def write_safetensors(path, tensors):
 def to_bf16(x):
     """float array -> bf16 bits (uint16), round to nearest even."""
     u = np.ascontiguousarray(x, dtype=np.float32).view(np.uint32)
-    return ((u + 0x7FFF + ((u >> 16) & 1)) >> 16).astype(np.uint16)
+    return ((u + 0x7FFF + ((u >> 16) & 1)) >> 16).astype(np.uint16).reshape(np.shape(x))
 
 
 def from_bf16(bits):

@@ -1,5 +1,5 @@
-"""Small random models for the tests of the model-folder backend: configurations and weights of the hybrid recurrent design (the latent
-design's are in latent_moe_models.py), folders, and the plain implementations' logits."""
+"""Small random models for the tests of the model-folder backend: configurations and weights of the hybrid recurrent design (the others'
+are in latent_moe_models.py and silevik_models.py), folders, and the plain implementations' logits."""
 import json
 import os
 
@@ -7,7 +7,11 @@ import numpy as np
 
 import hybrid_reference as R
 import latent_moe_models as L
+import silevik_models as S
 from ingot_b200 import models as M
+
+
+OTHERS = {"Banevik": L, "Silevik": S}
 
 
 def mamba(inner, state, dt_rank, conv, ff=None):
@@ -54,8 +58,8 @@ def shapes(cfg):
 def random_weights(cfg, seed=0, qk_gain=2.5):
     """bf16-representable float32 weights. Decays are slow (long memory) and the scores are sharp, so that a lost state or a
     key on the wrong side of an edge moves the logits."""
-    if cfg["architecture"] == "Banevik":
-        return L.random_weights(cfg, seed)
+    if cfg["architecture"] in OTHERS:
+        return OTHERS[cfg["architecture"]].random_weights(cfg, seed)
     rng = np.random.default_rng(seed)
     w = {}
     for name, shape in shapes(cfg).items():
@@ -93,9 +97,14 @@ def write(folder, cfg, weights):
 
 
 def reference_logits(cfg, weights, tokens):
-    if cfg["architecture"] == "Banevik":
-        return L.reference_logits(cfg, weights, tokens)
+    if cfg["architecture"] in OTHERS:
+        return OTHERS[cfg["architecture"]].reference_logits(cfg, weights, tokens)
     return R.forward(tokens, {k: v.astype(np.float64) for k, v in weights.items()}, cfg)
+
+
+def clear_choices(cfg, weights, tokens):
+    """Positions at which no router's choice is close, or None for designs without routers."""
+    return OTHERS[cfg["architecture"]].clear_choices(cfg, weights, tokens) if cfg["architecture"] in OTHERS else None
 
 
 def error(got, want):

@@ -1,5 +1,5 @@
 """Whole models of the designs the model-folder backend serves through the framework's step function, scheduler and command line, against the plain
-implementations in hybrid_reference.py and latent_moe_reference.py. Sizes are deliberately uneven; none needs to be a multiple of anything."""
+implementations in hybrid_reference.py, latent_moe_reference.py and silevik_reference.py. Sizes are deliberately uneven; none needs to be a multiple of anything."""
 import json
 import os
 import subprocess
@@ -9,6 +9,7 @@ import pytest
 
 import hybrid_models as H
 import latent_moe_models as L
+import silevik_models as S
 from ingot_b200 import models as M
 
 pytestmark = pytest.mark.gpu
@@ -33,6 +34,20 @@ CONFIGS = {
     # rows longer than a tensor-core tile, no loop, many experts, some of them idle
     "latent_long": L.config([L.layer(4, 64, 32, 48, 150, 70, scale=0.1, experts=40, top=6, ff=33), L.layer(33, 8, 8, 8, 72, 1, experts=33, top=2, ff=16)],
                             vocab=130, width=130, bigram=(64, 3, 1)),
+    # sandwich norms: uneven heads of every kind, keys and values of unequal lengths, scaled rotation, groups with identity experts, a layer
+    # without a feed-forward, values mixed in some layers only
+    "sandwich": S.config([S.layer("attention", 6, 3, 20, 12, 19, rot=8, base=500.0, v_mix=False, mlp=S.dense(37)),
+                          S.layer("attention_3", 3, 3, 18, 11, rot=14, scaling=(4.0, 64, 8.0, 1.0), mlp=S.moe(5, 3, 3, (4, 2), 20, 13)),
+                          S.layer("attention_2", 4, 1, 25, 40, v_mix=False),
+                          S.layer("attention", 6, 3, 10, 11, 33, rot=10, mlp=S.moe(6, 0, 2, (3, 2), 33, 40, scale=0.7)),
+                          S.layer("attention_2", 9, 3, 8, 11, mlp=S.dense(16))], vocab=103, width=46),
+    # every output is chosen (nothing hangs on a close choice), one head, one KV head for many, a window of one token, no groups
+    "sandwich_all": S.config([S.layer("attention_2", 12, 1, 32, 24, mlp=S.moe(3, 2, 5, None, 40, 32)), S.layer("attention", 1, 1, 48, 24, 1, rot=48, mlp=S.moe(2, 0, 2, None, 8, None)),
+                              S.layer("attention_3", 8, 1, 16, 24, 50, rot=2, mlp=S.moe(1, 1, 2, None, 64, 8))], vocab=90, width=64, logit_scale=1.0, embedding_scale=1.0),
+    # keys and values past the sizes the tcgen05 kernel takes, many experts, some of them idle, width past a tile
+    "sandwich_long": S.config([S.layer("attention_3", 4, 2, 200, 72, rot=64, scaling=(8.0, 32, 4.0, 0.5), scale=0.06, mlp=S.moe(36, 12, 6, (8, 3), 33, 24)),
+                               S.layer("attention", 33, 3, 72, 136, 70, rot=24, scale=0.1, v_mix=False, mlp=S.dense(100)),
+                               S.layer("attention_2", 10, 2, 96, 72, scale=0.1, mlp=S.moe(9, 3, 2, (3, 1), 70, 40))], vocab=130, width=130),
 }
 TOL = {True: 3e-5, False: 4e-2}
 
@@ -44,7 +59,7 @@ def case(request, tmp_path_factory):
     folder = H.write(tmp_path_factory.mktemp(request.param), cfg, w)
     rng = np.random.default_rng(9)
     tokens = [rng.integers(0, cfg["vocab"], n).tolist() for n in (231, 90, 41, 3, 130)]
-    want = [Want(H.reference_logits(cfg, w, t), L.clear_choices(cfg, w, t) if cfg["architecture"] == "Banevik" else None) for t in tokens]
+    want = [Want(H.reference_logits(cfg, w, t), H.clear_choices(cfg, w, t)) for t in tokens]
     return cfg, folder, tokens, want
 
 
@@ -152,7 +167,7 @@ def test_long_decoding(case):
     rng = np.random.default_rng(17)
     t = rng.integers(0, cfg["vocab"], 420).tolist()
     w = H.random_weights(cfg, seed=[len(k) for k, v in CONFIGS.items() if v is cfg][0])
-    want = Want(H.reference_logits(cfg, w, t), L.clear_choices(cfg, w, t) if cfg["architecture"] == "Banevik" else None)
+    want = Want(H.reference_logits(cfg, w, t), H.clear_choices(cfg, w, t))
     for f32 in (True, False):
         with M.Model(folder, f32=f32, max_tokens=448, max_seqs=2) as m:
             first = m.step([(1, 0, t[:9], list(range(9)))])

@@ -5,6 +5,7 @@ import numpy as np
 import pytest
 
 import latent_moe_reference as R
+import silevik_reference as S
 from hybrid_step import dev, lib
 from ingot_b200 import models as M
 
@@ -41,6 +42,62 @@ def test_routing_of_ties_and_values_that_are_not_numbers():
     z = np.array([[1, 2, 2, 1], [np.nan] * 4, [np.nan, 0, np.nan, -5], [-np.inf] * 4], np.float32)
     expert = route(z, 4, 3)[0].reshape(4, 3)
     assert expert.tolist() == [[1, 2, 0], [0, 1, 2], [1, 3, 0], [0, 1, 2]]
+
+
+class CRouter(C.Structure):
+    _fields_ = [(n, C.c_int) for n in ("n_expert", "n_identity", "top", "groups", "keep")] + [("scale", C.c_float), ("correction", C.c_void_p)]
+
+
+def route_grouped(z, experts, identity, top, groups, keep, scale, correction, shared):
+    import torch
+    n = z.shape[0]
+    zd, cd = dev(z), None if correction is None else dev(correction)
+    i = lambda k: torch.full((k,), -7, device="cuda", dtype=torch.int32)
+    f = lambda k: torch.full((k,), -3.0, device="cuda")
+    out = [i(n * top), f(n * top), i(experts + 1), i(n * top), i(n * top), f(n * top), f(n), f(n)]
+    r = CRouter(experts, identity, top, groups, keep, scale, None if cd is None else cd.data_ptr())
+    ptr = [t.data_ptr() for t in out]
+    lib(lib().ingot_moe_route_grouped(C.byref(r), zd.data_ptr(), z.shape[1], n, *ptr[:6], ptr[6], ptr[7] if shared else None, None))
+    torch.cuda.synchronize()
+    return [t.cpu().numpy() for t in out]
+
+
+GROUPED = [(1, 5, 3, 2, 4, 2), (40, 12, 0, 3, 3, 1), (7, 3, 1, 4, 1, 1), (300, 60, 4, 6, 8, 3), (65, 10, 30, 5, 10, 9), (33, 1, 1, 1, 2, 1), (9, 300, 20, 8, 20, 20), (2050, 8, 4, 2, 4, 2)]
+
+
+@pytest.mark.parametrize("n,experts,identity,top,groups,keep", GROUPED)
+def test_grouped_routing(n, experts, identity, top, groups, keep):
+    rng = np.random.default_rng(n + experts)
+    outputs, total = experts + identity, experts + identity + 3
+    z = np.full((n, total), 1e9, np.float32)  # columns behind the router's are the shared gate and padding
+    z[:, :outputs] = rng.standard_normal((n, outputs)) * 2
+    z[:, outputs] = rng.standard_normal(n)
+    c = (rng.standard_normal(outputs) - 1.0).astype(np.float32)  # choice scores of both signs
+    expert, weight, start, row, pair, row_w, self_gain, shared = route_grouped(z, experts, identity, top, groups, keep, 1.7, c, True)
+    chosen, want = S.route(z[:, :outputs].astype(np.float64), np.eye(outputs), c.astype(np.float64), top, groups, keep, 1.7)
+    same = np.array([set(a) == set(b) for a, b in zip(expert.reshape(n, top), chosen)])
+    assert same.mean() > 0.99  # 32-bit and 64-bit scores may order a close pair differently
+    ok = np.repeat((expert.reshape(n, top) == chosen).all(axis=1), top)
+    assert np.abs(weight - want.reshape(-1))[ok].max() < 1e-5 and ok.mean() > 0.98
+    assert np.allclose(weight.reshape(n, top).sum(axis=1), 1.7, atol=1e-5)
+    real = expert < experts
+    assert np.allclose(self_gain, np.where(real, 0, weight).reshape(n, top).sum(axis=1), atol=1e-6)
+    assert np.allclose(shared, 1 / (1 + np.exp(-z[:, outputs])), atol=1e-6)
+    order = np.argsort(expert, kind="stable")[:real.sum()]
+    assert np.array_equal(pair[:real.sum()], order) and np.array_equal(row_w[:real.sum()], weight[order])
+    assert np.array_equal(row[order], np.arange(real.sum())) and (row[~real] == -1).all()
+    assert np.array_equal(start, np.searchsorted(np.sort(expert), np.arange(experts + 1)))
+
+
+def test_grouped_routing_with_negative_choices_and_ties():
+    """What is closed counts as minus infinity, not 0; equal choices go to the lower index, equal groups to the lower group."""
+    z = np.zeros((1, 6), np.float32)
+    expert = route_grouped(z, 6, 0, 2, 3, 1, 1.0, np.array([-9, -8, -3, -4, -7, -3], np.float32), False)[0]
+    assert expert.tolist() == [2, 3]
+    expert, weight = route_grouped(z, 4, 2, 3, 3, 2, 1.0, None, False)[:2]
+    assert expert.tolist() == [0, 1, 2] and np.allclose(weight, 1 / 3)
+    nan = np.full((1, 6), np.nan, np.float32)
+    assert route_grouped(nan, 6, 0, 2, 1, 1, 1.0, None, False)[0].tolist() == [0, 1]
 
 
 class CGrouped(C.Structure):
@@ -93,8 +150,49 @@ def test_grouped_product(counts, n_in, n_out, planes):
         torch.cuda.synchronize()
         act = np.square(np.maximum(want * scale[:, None], 0))
         assert np.abs((o_hi.double() + o_lo.double()).cpu().numpy() - act).max() < 1e-4 * max(1, act.max())
+        if n_out % 32 == 0:  # the columns as runs of 32 gate and 32 up ones, taken together
+            wide = n_out // 32 * 32 // 64 * 64
+            if wide:
+                w2 = wd[:, :wide].contiguous()
+                g.w, g.n_out, g.act = w2.data_ptr(), wide, 2
+                o_hi, o_lo = (torch.full((rows, wide // 2), np.nan, device="cuda", dtype=torch.bfloat16) for _ in range(2))
+                g.out_hi, g.out_lo = o_hi.data_ptr(), o_lo.data_ptr()
+                assert L.ingot_grouped_tc_run(ws, C.byref(g), None) == 0
+                torch.cuda.synchronize()
+                runs = want[:, :wide].reshape(rows, -1, 2, 32)
+                act = (S.silu(runs[:, :, 0]) * runs[:, :, 1]).reshape(rows, -1) * scale[:, None]
+                assert np.abs((o_hi.double() + o_lo.double()).cpu().numpy() - act).max() < 1e-4 * max(1, np.abs(act).max())
     finally:
         L.ingot_linear_ws_destroy(ws)
+
+
+@pytest.mark.parametrize("n,experts,identity,top,d,ff", [(1, 4, 0, 2, 40, 32), (1, 3, 2, 4, 256, 64), (2, 5, 1, 3, 64, 32), (9, 5, 3, 5, 64, 96), (130, 12, 4, 3, 48, 64)])
+def test_plain_gated_experts_and_identity_experts(n, experts, identity, top, d, ff):
+    """Routing, both products in f32 arithmetic, and the residual sum that takes the identity experts and the shared expert in."""
+    import torch
+    import residual_norm as N
+    rng = np.random.default_rng(d + n)
+    W = {"router": rng.standard_normal((experts + identity, d)) / d ** 0.5, "correction": rng.standard_normal(experts + identity) * 0.3}
+    gate, up = (bf16(rng.standard_normal((experts, ff, d)) / d ** 0.5) for _ in range(2))
+    down = bf16(rng.standard_normal((experts, d, ff)) / ff ** 0.5)
+    stack = torch.stack([gate.view(experts, ff // 32, 32, d), up.view(experts, ff // 32, 32, d)], dim=2).reshape(experts, 2 * ff, d).contiguous()
+    for e in range(experts):
+        W[f"e{e}.gate"], W[f"e{e}.up"], W[f"e{e}.down"] = (t[e].double().cpu().numpy() for t in (gate, up, down))
+    x = rng.standard_normal((n, d)).astype(np.float32)
+    norm, post = ((rng.standard_normal(d) + 2, rng.standard_normal(d)) for _ in range(2))
+    shared, z_shared = rng.standard_normal((n, d)), rng.standard_normal(n)
+    h = S.layer_norm(x.astype(np.float64), *norm, 1e-5)
+    mlp = {"router": {"experts": experts, "top": top, "scale": 1.3}}
+    want = x + S.layer_norm(S.mixture(h, W, "", mlp) + S.sigmoid(z_shared)[:, None] * shared, *post, 1e-5)
+    z = np.concatenate([h @ W["router"].T, z_shared[:, None]], axis=1)
+    _, _, start, row, pair, row_w, self_gain, shared_gain = route_grouped(z.astype(np.float32), experts, identity, top, 1, 1, 1.3, W["correction"].astype(np.float32), True)
+    hd, xd, sd, rd, pd, wd = dev(h), dev(x), dev(start, np.int32), dev(row, np.int32), dev(pair, np.int32), dev(row_w)
+    mid, out = torch.zeros(n * top, ff, device="cuda"), torch.full((n * top, d), float("nan"), device="cuda")  # rows of identity experts are never written
+    p = lambda t: t.data_ptr()
+    lib(lib().ingot_moe_linear(p(mid), p(stack), p(hd), d, d, ff, experts, n * top, p(sd), p(pd), top, p(wd), 2, None))
+    lib(lib().ingot_moe_linear(p(out), p(down), p(mid), ff, ff, d, experts, n * top, p(sd), None, top, None, 0, None))
+    N.run(xd, eps=1e-5, product=dev(shared)[None], gain=dev(shared_gain), branch=out, row_of=rd, top=top, self_gain=dev(self_gain) if identity else None, self_norm=norm, post=post)
+    assert np.abs(xd.cpu().numpy() - want).max() < 2e-4
 
 
 @pytest.mark.parametrize("n,experts,top,d,ff", [(1, 4, 2, 40, 24), (9, 5, 5, 64, 16), (130, 12, 3, 48, 72), (600, 3, 1, 16, 8)])

@@ -1,0 +1,63 @@
+"""The residual sum with norms before and after it (backend/residual_norm.cu) against the plain statement, at lengths on both sides of every
+launch shape, padded or not."""
+import numpy as np
+import pytest
+
+import residual_norm as N
+import silevik_reference as R
+from hybrid_step import dev
+
+pytestmark = pytest.mark.gpu
+EPS = 1e-5
+SIZES = [(8, 5), (48, 48), (1024, 1021), (1032, 1030), (4096, 4096), (4104, 4100), (8192, 8191), (9000, 8999)]
+
+
+def plain(x, pair):
+    return R.rms_norm(x, pair[0], EPS) if pair[1] is None else R.layer_norm(x, *pair, EPS)
+
+
+@pytest.mark.parametrize("centred", [True, False])
+@pytest.mark.parametrize("n,count", SIZES)
+def test_every_term(n, count, centred):
+    import torch
+    rng = np.random.default_rng(n)
+    rows, slices, top = 5, 3, 2
+    pad = lambda a: np.pad(a, [(0, 0)] * (a.ndim - 1) + [(0, n - count)])
+    x, product, branch = 40 + rng.standard_normal((rows, count)), rng.standard_normal((slices, rows, count)), rng.standard_normal((7, count))
+    pairs = [(rng.standard_normal(count) + 1, rng.standard_normal(count) if centred else None) for _ in range(3)]
+    gain, self_gain = rng.random(rows), rng.standard_normal(rows)
+    self_gain[2] = 0.0
+    row_of = np.array([[0, 6], [-1, 3], [2, -1], [-1, -1], [5, 1]])
+    y = product.sum(axis=0) * gain[:, None] + self_gain[:, None] * plain(x, pairs[0])
+    for r, t in zip(range(rows), row_of):
+        y[r] += sum(branch[i] for i in t if i >= 0)
+    want = x + plain(y, pairs[1])
+    read = plain(want, pairs[2])
+    xd = dev(pad(x))
+    out = torch.full((rows, n), float("nan"), device="cuda")
+    hi, lo = (torch.full((rows, n), float("nan"), device="cuda", dtype=torch.bfloat16) for _ in range(2))
+    N.run(xd, EPS, count, product=dev(pad(product)), gain=dev(gain), branch=dev(pad(branch)), row_of=dev(row_of, np.int32), top=top, self_gain=dev(self_gain), self_norm=pairs[0],
+          post=pairs[1], next_norm=pairs[2], out=out, hi=hi, lo=lo)
+    assert np.abs(xd.cpu().numpy()[:, :count] - want).max() < 2e-4 and not xd.cpu().numpy()[:, count:].any()
+    got = out.cpu().numpy()
+    assert np.abs(got[:, :count] - read).max() < (3e-4 if centred else 2e-5) * np.abs(read).max() and not got[:, count:].any()
+    assert ((hi.float() + lo.float() - out).abs().max() <= 1e-4 * out.abs().max()).item()
+
+
+def test_a_norm_alone_of_chosen_rows():
+    import torch
+    rng = np.random.default_rng(0)
+    x, pair = rng.standard_normal((9, 64)), (rng.standard_normal(64), rng.standard_normal(64))
+    xd, out = dev(x), torch.zeros(3, 64, device="cuda")
+    N.run(xd, EPS, rows=dev([7, 0, 7], np.int32), next_norm=pair, out=out)
+    assert np.abs(out.cpu().numpy() - R.layer_norm(x[[7, 0, 7]], *pair, EPS)).max() < 1e-5
+    assert np.array_equal(xd.cpu().numpy(), x.astype(np.float32))  # x is only read
+
+
+def test_the_variance_is_taken_around_the_mean():
+    """Values with a mean a thousand times their spread: squares would lose it."""
+    import torch
+    x = 3000.0 + np.arange(256.0)[None] % 7
+    xd, out = dev(x), torch.zeros(1, 256, device="cuda")
+    N.run(xd, EPS, next_norm=(np.ones(256), np.zeros(256)), out=out)
+    assert np.abs(out.cpu().numpy() - R.layer_norm(x, 1.0, 0.0, EPS)).max() < 1e-3
