@@ -1,7 +1,7 @@
 #!/usr/bin/env python
 """Benchmark of the B200 attention path: decode KV-cache HBM GB/s and causal-prefill TFLOP/s.
 
-    python bench.py --gpus N --steps K --warmup W [--workload decode_c2|prefill_c5|c1_prefill128|c3_chunked|c4_batched|e2e_model|hybrid_layers|latent_layers]
+    python bench.py --gpus N --steps K --warmup W [--workload decode_c2|prefill_c5|c1_prefill128|c3_chunked|c4_batched|e2e_model|hybrid_layers|latent_layers|grouped_layers]
                     [--impl reference]
 
 Headline (`metric`/`value`): single-token decode attention at 4096 keys, 24 query / 8 KV heads,
@@ -880,6 +880,33 @@ def run_latent_layers(args):
                          "llama_decode_weight_stream_frac": round(llama["decode"][1]["weight_gb_s"] / peaks["hbm_gbs"], 4)}}
 
 
+def run_grouped_layers(args):
+    """Prefill and decode throughput of the sandwich-normed grouped-query attention / grouped-mixture design (model folders,
+    backend/attention_layers.cpp, feed_forward.cpp) at sizes of real layers with random weights, beside this framework's Llama-shaped
+    layers of equal width and heads. Device time per step through the library's own step function; weights exceed the L2."""
+    import torch
+    from ingot_b200 import grouped_bench as GB
+    from ingot_b200 import hybrid_bench as HB
+    torch.cuda.set_device(0)
+    reps = max(args.steps // 5, 5)
+    grouped = GB.run_grouped(args.grouped_size, reps=reps, work=os.environ.get("INGOT_E2E_DIR", "/tmp"))
+    llama = HB.run_llama(args.grouped_size, reps=reps)
+    peaks = measured_peaks()
+    top = grouped["prefill"][2048]
+    layers = GB.config(args.grouped_size)["layers"]
+    return {"metric": "grouped-attention layers, 2048-token prefill tokens/s", "value": top["tok_s"], "unit": "tok/s", "n_gpus": 1, "steps": reps,
+            "warmup": 3, "ms_per_step": top["ms"], "higher_is_better": True, "scaling": "weak", "vs_baseline": None,
+            "dtype": "bf16 weights, bf16 products with f32 accumulation, f32 residual, norms, scores and routers", "data": "synthetic",
+            "config": {"workload": f"{args.grouped_size}: {layers[0]}, {layers[1]}, the first again, {layers[3]['type']} with scaled rotation and sinks; "
+                                   f"vocabulary {GB.VOCAB}; decode at 1024 tokens of context", "l2": "weights of a step exceed the L2"},
+            "grouped": grouped, "llama_layers": llama,
+            "roofline": {"bound": "tensor", "unit": "TFLOP/s", "peak": peaks["tflops_burst"], "achieved": top["tflops"],
+                         "frac": round(top["tflops"] / peaks["tflops_burst"], 4),
+                         "decode_weight_stream_frac": round(grouped["decode"][1]["weight_gb_s"] / peaks["hbm_gbs"], 4),
+                         "llama_prefill_frac": round(llama["prefill"][2048]["tflops"] / peaks["tflops_burst"], 4),
+                         "llama_decode_weight_stream_frac": round(llama["decode"][1]["weight_gb_s"] / peaks["hbm_gbs"], 4)}}
+
+
 # ------------------------------------------------------------------------------------------------
 # CPU reference legs
 # ------------------------------------------------------------------------------------------------
@@ -982,9 +1009,10 @@ def main():
     ap.add_argument("--steps", type=int, default=50)
     ap.add_argument("--warmup", type=int, default=5)
     ap.add_argument("--impl", default="ingot", choices=["ingot", "reference"])
-    ap.add_argument("--workload", default="decode_c2", choices=["decode_c2", "prefill_c5", "c1_prefill128", "c3_chunked", "c4_batched", "e2e_model", "hybrid_layers", "latent_layers"])
+    ap.add_argument("--workload", default="decode_c2", choices=["decode_c2", "prefill_c5", "c1_prefill128", "c3_chunked", "c4_batched", "e2e_model", "hybrid_layers", "latent_layers", "grouped_layers"])
     ap.add_argument("--hybrid-size", default="w4096", choices=["w2048", "w4096"], help="hybrid_layers: width of the layers")
     ap.add_argument("--latent-size", default="w4096", choices=["w2048", "w4096"], help="latent_layers: width of the layers")
+    ap.add_argument("--grouped-size", default="w4096", choices=["w2048", "w4096"], help="grouped_layers: width of the layers")
     ap.add_argument("--small-model", action="store_true", help="e2e_model: 2 layers and a 32064-token vocabulary")
     ap.add_argument("--wtype", default="F16", choices=["F16", "Q8_0", "Q4_0", "Q4_1", "Q6_K"], help="e2e_model: weight type of the GGUF")
     ap.add_argument("--output-type", default=None, choices=["F16", "Q8_0", "Q4_0", "Q4_1", "Q6_K"],
@@ -1020,6 +1048,9 @@ def main():
         return
     if args.workload == "latent_layers":
         print(json.dumps(run_latent_layers(args)), flush=True)
+        return
+    if args.workload == "grouped_layers":
+        print(json.dumps(run_grouped_layers(args)), flush=True)
         return
 
     start_watchdog(int(os.environ.get("WORLD_SIZE", "1")))  # before the process group comes up: its set-up can stall too

@@ -440,9 +440,10 @@ int ingot_gqa_append(ingot_skv* kv, int layer, const ingot_step* step, const flo
  * term exp(sink) of a head's softmax sum. gate_dev (may be null): the result times sigmoid(z), z at gate_dev[t * gate_ld + ...], one per
  * head or one per result column. impl: 0 = library's choice, 1 = the plain f32-arithmetic kernel, 2 = the warp-level tensor-core kernel
  * with split keys (f16, sizes that are multiples of 16 and at most 256), 3 = the tcgen05 kernel (f16, sizes that are multiples of 16,
- * keys at most 256, values at most 128, scale > 0), which 0 takes from INGOT_GQA_LONG_ROWS (token, head) rows per KV head on. The step may
- * be some sequences of a larger one: n_seq and the per-sequence arrays are theirs, n_tok and the rows those of the whole. */
-#define INGOT_GQA_LONG_ROWS 128
+ * keys at most 256, values at most 128, scale > 0), which 0 takes for portions of several tokens when the step's sequences, each as long
+ * as the longest, have INGOT_GQA_LONG_ROWS (token, head) pairs. The step may be some sequences of a larger one: n_seq and the per-sequence
+ * arrays are theirs, n_tok and the rows those of the whole. */
+#define INGOT_GQA_LONG_ROWS 2560
 int ingot_gqa_attend(ingot_skv* kv, int layer, const ingot_step* step, const void* q_dev, const ingot_gqa_shape* shape, float scale, const float* sink_dev,
                      const float* gate_dev, int gate_ld, int gate_per_head, const ingot_act_out* out, const int32_t* tables_dev, const int32_t* first_page_dev,
                      int max_blocks, int impl, void* stream);

@@ -29,8 +29,8 @@ struct Rotation {
 };
 
 // q, k, v and the output gate's logits are one product of the normed input; queries and keys are normed and rotated, values mixed with the
-// first mixing layer's, and keys and values cached side by side. Decoded tokens and short portions take the split-key kernel, portions of
-// many rows the tcgen05 one, each over its sequences of the step; the gate is applied where the result is stored as W_o's operand.
+// first mixing layer's, and keys and values cached side by side. Single tokens and portions of several are two calls, each over its
+// sequences of the step: the split-key kernel, and that or the tcgen05 one (ingot_gqa_attend chooses by the number of rows); the gate is applied where the result is stored as W_o's operand.
 class GroupedAttentionMixer : public Mixer {
 public:
     GroupedAttentionMixer(LayerOps& ops, const AttentionKind& kind, const Json& c, const std::string& p) : gate_(kind.gate) {
@@ -76,9 +76,9 @@ public:
         if (kind.sink) sink_ = ops.vector(p + "sink", {heads}, {1, heads, heads});
         if (has(c, "v_mix") && c.at("v_mix").boolean()) {
             mixes_ = true;
-            first_ = ops.mixed_values == 0;
-            if (first_) ops.mixed_values = v.width();
-            else if (ops.mixed_values != v.width()) throw std::runtime_error("model config: layers that mix values need equal \"kv_heads\" and \"vdim\"");
+            first_ = ops.mixed_values.n == 0;
+            if (first_) ops.mixed_values = v;
+            else if (ops.mixed_values.n != kv_heads || ops.mixed_values.size != vdim) throw std::runtime_error("model config: layers that mix values need equal \"kv_heads\" and \"vdim\"");
             if (!first_) mix_ = ops.scalar(p + "vmix");
             ops.need(kFirstValue, v.width());
         }
@@ -95,10 +95,10 @@ public:
         ingot_check(ingot_gqa_append(g.kv, layer, &s.st, proj, proj_ld_, 0, k_off_, v_off_, &shape_, q_norm_, k_norm_, ops.eps, turns_, rot_gain_,
                                      mixes_ ? ops.buf(kFirstValue) : nullptr, first_, mix_, ops.buf(kQuery), g.tables, g.first_page, g.width, ops.stream));
         const ingot_act_out out = ops.operand(s, mix, out_ld_, false);
-        // sequences come in ascending order of their portions: the long ones are the last
+        // sequences come in ascending order of their portions: single tokens first
         int from = n_seq;
         if (!ops.opt.f32)
-            while (from > 0 && (long long)s.lens[from - 1] * (shape_.n_head / shape_.n_head_kv) >= INGOT_GQA_LONG_ROWS) from--;
+            while (from > 0 && s.lens[from - 1] > 1) from--;
         attend(ops, s, layer, 0, from, out);
         attend(ops, s, layer, from, n_seq, out);
         ops.operand_ready(s, out_ld_);

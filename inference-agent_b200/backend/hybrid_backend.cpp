@@ -168,12 +168,13 @@ public:
         const StepCtx s = upload_step(entries, n, step);
         reserve_logits(step.n_want);
         // Steps of single decoded tokens are the same launches every time but for what the metadata says: captured once per
-        // batch size and replayed. The first such step of a size runs eagerly.
+        // batch size and reach (Step::reach) and replayed. The first such step of a size runs eagerly.
         const bool replay = step.decode && !tap_ && use_graphs_;
+        const std::pair<int, int> key(n, step.reach);
         cuda_check(cudaEventRecord(ev0_, ops_.stream), "cudaEventRecord");
-        if (replay && graphs_.count(n) && graphs_[n].exec) {
-            cuda_check(cudaGraphLaunch(graphs_[n].exec, ops_.stream), "cudaGraphLaunch");
-        } else if (replay && graphs_[n].seen++ > 0) {
+        if (replay && graphs_.count(key) && graphs_[key].exec) {
+            cuda_check(cudaGraphLaunch(graphs_[key].exec, ops_.stream), "cudaGraphLaunch");
+        } else if (replay && graphs_[key].seen++ > 0) {
             cuda_check(cudaStreamBeginCapture(ops_.stream, cudaStreamCaptureModeThreadLocal), "cudaStreamBeginCapture");
             try {
                 encode(s, step);
@@ -183,9 +184,9 @@ public:
                 if (dead) cudaGraphDestroy(dead);
                 throw;
             }
-            cuda_check(cudaStreamEndCapture(ops_.stream, &graphs_[n].graph), "cudaStreamEndCapture");
-            cuda_check(cudaGraphInstantiate(&graphs_[n].exec, graphs_[n].graph, 0), "cudaGraphInstantiate");
-            cuda_check(cudaGraphLaunch(graphs_[n].exec, ops_.stream), "cudaGraphLaunch");
+            cuda_check(cudaStreamEndCapture(ops_.stream, &graphs_[key].graph), "cudaStreamEndCapture");
+            cuda_check(cudaGraphInstantiate(&graphs_[key].exec, graphs_[key].graph, 0), "cudaGraphInstantiate");
+            cuda_check(cudaGraphLaunch(graphs_[key].exec, ops_.stream), "cudaGraphLaunch");
         } else {
             encode(s, step);
         }
@@ -252,6 +253,7 @@ private:
     struct Step {
         int n_tok = 0, max_len = 0, n_want = 0;
         bool decode = true;           // one token of every sequence, its logits wanted
+        int reach = 0;                // decoding: pages of the longest sequence, rounded up to a power of two (block tables are this wide)
         const int32_t* want_rows = nullptr;  // device
         const int32_t* tokens = nullptr;     // device
         const int32_t* bigrams = nullptr;    // device: rows of the bigram table
@@ -286,6 +288,7 @@ private:
             step.max_len = std::max(step.max_len, e.n_tokens);
             step.n_want += e.n_want;
             step.decode = step.decode && e.n_tokens == 1 && e.n_want == 1;
+            while (step.reach * INGOT_BLOCK_TOKENS < e.pos0 + e.n_tokens) step.reach = std::max(8, step.reach * 2);
         }
         if (step.n_tok > ops_.max_step) throw std::runtime_error("engine: more tokens than a step may carry");
         return step;
@@ -382,7 +385,8 @@ private:
                 width = std::max(width, g->page(entries[i].pos0 + entries[i].n_tokens - 1) - first + 1);
                 m.push_back(first);
             }
-            if (step.decode) width = g->forgets() ? std::min(g->pages_seen(), g->pool.pages_per_seq()) : g->pool.pages_per_seq();  // the same at every step
+            // the same at every step that replays the same launches
+            if (step.decode) width = std::min({g->forgets() ? g->pages_seen() : step.reach, step.reach, g->pool.pages_per_seq()});
             const size_t o_table = mark();
             for (int i = 0; i < n; i++) {
                 const int first = m[o_first + size_t(i)];
@@ -610,7 +614,7 @@ private:
     int logit_rows_ = 0;
     std::vector<int*> status_words_;
     int* status_host_ = nullptr;
-    std::map<int, Graph> graphs_;      // by batch size
+    std::map<std::pair<int, int>, Graph> graphs_;  // by batch size and reach
     const bool use_graphs_ = !(getenv("INGOT_DECODE_GRAPH") && atoi(getenv("INGOT_DECODE_GRAPH")) == 0);
     const int scan_threads_per_sm_ = getenv("INGOT_SCAN_THREADS") ? std::max(1, atoi(getenv("INGOT_SCAN_THREADS"))) : 1024;
     std::vector<float>* tap_ = nullptr;

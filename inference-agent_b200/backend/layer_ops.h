@@ -466,7 +466,7 @@ public:
     int pass = 0;    // the one that runs
     size_t weight_bytes = 0;
     std::vector<std::unique_ptr<CacheGroup>> caches;
-    int mixed_values = 0;  // length of the values that layers mix with the first such layer's (kFirstValue); 0: none so far
+    Groups mixed_values = {0, 0, 0};  // the values that layers mix with the first such layer's (kFirstValue): heads and sizes; none so far
 
     // The group a layer's caches belong to; *layer: the first of its `passes` caches there.
     CacheGroup* cache_group(int kv_heads, int dim, int chunk, int window, CacheGroup::Form form, int* layer) {

@@ -1,6 +1,6 @@
 // Residual sum with norms before and after it: the sum of a product's slices, of routed rows and of the part's own input, the norm of that
 // result, the residual add, and the norm the next part reads x through, as f32 rows or as the bf16 operand of its products. One CTA per
-// row, which stays in registers throughout; variances are means of squared deviations, taken in a second pass over the registers.
+// row, which stays in registers throughout.
 #include "residual_norm.h"
 
 #include <cuda_bf16.h>
@@ -9,10 +9,15 @@
 
 namespace {
 
+template <int kKeep>
+struct Row {
+    float4 v[kKeep];
+};
+
+// Sum over the block. red: a float per warp that no other exchange of the kernel uses.
 __device__ __forceinline__ float block_sum(float v, float* red) {
 #pragma unroll
     for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
-    __syncthreads();  // red is free again
     if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = v;
     __syncthreads();
     float t = 0.f;
@@ -20,48 +25,61 @@ __device__ __forceinline__ float block_sum(float v, float* red) {
     return t;
 }
 
+// (mean, 1 / deviation) of the first n_mean values of the row the block holds, the deviation around the mean in a second pass over the
+// registers; the mean is 0 for norms that do not centre.
 template <int kKeep>
-struct Row {
-    float4 v[kKeep];
-};
-
-// (mean, 1 / deviation) of the first n_mean values; the mean is 0 for norms that do not centre.
-template <int kKeep>
-__device__ __forceinline__ float2 moments(const Row<kKeep>& r, int n_mean, bool centred, float eps, float* red) {
-    float mean = 0.f;
-    if (centred) {  // the padding holds zeros
-        float s = 0.f;
+__device__ __forceinline__ float2 moments(const Row<kKeep>& r, int n_mean, bool centred, float inv_n, float eps, float* red, int red_ld) {
+    float mean = 0.f, sq = 0.f;
+    if (centred) {
+        float sum = 0.f;  // the padding holds zeros
 #pragma unroll
-        for (int k = 0; k < kKeep; k++) s += (r.v[k].x + r.v[k].y) + (r.v[k].z + r.v[k].w);
-        mean = block_sum(s, red) / float(n_mean);
+        for (int k = 0; k < kKeep; k++) sum += (r.v[k].x + r.v[k].y) + (r.v[k].z + r.v[k].w);
+        mean = block_sum(sum, red) * inv_n;
     }
-    float ss = 0.f;
 #pragma unroll
     for (int k = 0; k < kKeep; k++) {
-        const int i = (threadIdx.x + k * blockDim.x) * 4;
+        const int left = n_mean - int(threadIdx.x + k * blockDim.x) * 4;
         const float d[4] = {r.v[k].x - mean, r.v[k].y - mean, r.v[k].z - mean, r.v[k].w - mean};
+        if (left >= 4) {
+            sq = fmaf(d[0], d[0], sq); sq = fmaf(d[1], d[1], sq); sq = fmaf(d[2], d[2], sq); sq = fmaf(d[3], d[3], sq);
+        } else {
 #pragma unroll
-        for (int e = 0; e < 4; e++)
-            if (i + e < n_mean) ss = fmaf(d[e], d[e], ss);
+            for (int e = 0; e < 3; e++)
+                if (e < left) sq = fmaf(d[e], d[e], sq);
+        }
     }
-    return make_float2(mean, 1.0f / sqrtf(block_sum(ss, red) / float(n_mean) + eps));
-}
-__device__ __forceinline__ float4 apply(float4 v, float2 m, const ingot_norm& n, int i) {
-    const float4 w = *reinterpret_cast<const float4*>(n.w + i);
-    float4 o = make_float4((v.x - m.x) * m.y * w.x, (v.y - m.x) * m.y * w.y, (v.z - m.x) * m.y * w.z, (v.w - m.x) * m.y * w.w);
-    if (n.b) {
-        const float4 b = *reinterpret_cast<const float4*>(n.b + i);
-        o.x += b.x; o.y += b.y; o.z += b.z; o.w += b.w;
-    }
-    return o;
+    return make_float2(mean, rsqrtf(fmaf(block_sum(sq, red + red_ld), inv_n, eps)));
 }
 
-template <int kKeep, int kThreads>
-__global__ void __launch_bounds__(kThreads) residual_norm_kernel(const ingot_residual_norm p) {
-    __shared__ float red[32];
+// The part of a norm's weights that belongs to this thread's values, requested ahead of the moments.
+template <int kKeep>
+struct Weights {
+    Row<kKeep> w, b;
+    __device__ __forceinline__ void load(const ingot_norm& n, int len, int step) {
+#pragma unroll
+        for (int k = 0; k < kKeep; k++) {
+            const int i = threadIdx.x * 4 + k * step;
+            w.v[k] = n.w && i < len ? *reinterpret_cast<const float4*>(n.w + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+            b.v[k] = n.b && i < len ? *reinterpret_cast<const float4*>(n.b + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+        }
+    }
+    __device__ __forceinline__ float4 apply(float4 v, float2 m, int k) const {
+        return make_float4(fmaf((v.x - m.x) * m.y, w.v[k].x, b.v[k].x), fmaf((v.y - m.x) * m.y, w.v[k].y, b.v[k].y),
+                           fmaf((v.z - m.x) * m.y, w.v[k].z, b.v[k].z), fmaf((v.w - m.x) * m.y, w.v[k].w, b.v[k].w));
+    }
+};
+__device__ __forceinline__ void add(float4& a, const float4& b) { a.x += b.x; a.y += b.y; a.z += b.z; a.w += b.w; }
+
+template <int kKeep, int kThreads, int kBlocks>
+__global__ void __launch_bounds__(kThreads, kBlocks) residual_norm_kernel(const ingot_residual_norm p, float inv_n) {
+    constexpr int kWarps = kThreads / 32;
+    __shared__ float red[3][2 * kWarps];  // of the three norms
     INGOT_PDL_TRIGGER();
-    INGOT_PDL_WAIT();
     const int row = blockIdx.x, step = blockDim.x * 4;
+    const bool sum = p.n_slices > 0 || p.top > 0 || p.self_gain;
+    Weights<kKeep> w;  // weights do not depend on the kernel before
+    w.load(sum && p.post.w ? p.post : p.next, p.n, step);
+    INGOT_PDL_WAIT();
     float* xr = p.x + (size_t)(p.rows ? p.rows[row] : row) * p.n;
     Row<kKeep> x;
 #pragma unroll
@@ -69,66 +87,67 @@ __global__ void __launch_bounds__(kThreads) residual_norm_kernel(const ingot_res
         const int i = threadIdx.x * 4 + k * step;
         x.v[k] = i < p.n ? *reinterpret_cast<const float4*>(xr + i) : make_float4(0.f, 0.f, 0.f, 0.f);
     }
-    if (p.n_slices > 0 || p.top > 0 || p.self_gain) {
+    if (sum) {
         Row<kKeep> y;
-        const float gain = p.gain ? p.gain[row] : 1.0f;
-        const size_t slice = (size_t)p.n_rows * p.n;
 #pragma unroll
-        for (int k = 0; k < kKeep; k++) {
-            const int i = threadIdx.x * 4 + k * step;
-            y.v[k] = make_float4(0.f, 0.f, 0.f, 0.f);
-            if (i >= p.n) continue;
-            for (int s = 0; s < p.n_slices; s++) {
-                const float4 a = *reinterpret_cast<const float4*>(p.product + s * slice + (size_t)row * p.n + i);
-                y.v[k].x += a.x; y.v[k].y += a.y; y.v[k].z += a.z; y.v[k].w += a.w;
-            }
-            y.v[k].x *= gain; y.v[k].y *= gain; y.v[k].z *= gain; y.v[k].w *= gain;
-        }
-        for (int t = 0; t < p.top; t++) {
-            const int r = p.row_of[(size_t)row * p.top + t];
-            if (r < 0) continue;
+        for (int k = 0; k < kKeep; k++) y.v[k] = make_float4(0.f, 0.f, 0.f, 0.f);
+        const size_t slice = (size_t)p.n_rows * p.n;
+        auto take = [&](const float* from) {  // all of the thread's pieces of a row in flight together
 #pragma unroll
             for (int k = 0; k < kKeep; k++) {
                 const int i = threadIdx.x * 4 + k * step;
-                if (i >= p.n) continue;
-                const float4 a = *reinterpret_cast<const float4*>(p.branch + (size_t)r * p.n + i);
-                y.v[k].x += a.x; y.v[k].y += a.y; y.v[k].z += a.z; y.v[k].w += a.w;
+                if (i < p.n) add(y.v[k], *reinterpret_cast<const float4*>(from + i));
             }
+        };
+        for (int s = 0; s < p.n_slices; s++) take(p.product + s * slice + (size_t)row * p.n);
+        if (p.gain) {
+            const float gain = p.gain[row];
+#pragma unroll
+            for (int k = 0; k < kKeep; k++) { y.v[k].x *= gain; y.v[k].y *= gain; y.v[k].z *= gain; y.v[k].w *= gain; }
+        }
+        for (int t0 = 0; t0 < p.top; t0 += 4) {
+            int r[4];
+#pragma unroll
+            for (int t = 0; t < 4; t++) r[t] = t0 + t < p.top ? p.row_of[(size_t)row * p.top + t0 + t] : -1;
+#pragma unroll
+            for (int t = 0; t < 4; t++)
+                if (r[t] >= 0) take(p.branch + (size_t)r[t] * p.n);
         }
         const float self = p.self_gain ? p.self_gain[row] : 0.f;
         if (self != 0.f) {  // block-uniform
-            const float2 m = moments(x, p.n_mean, p.self.b != nullptr, p.eps, red);
+            const float2 m = moments(x, p.n_mean, p.self.b != nullptr, inv_n, p.eps, red[0], kWarps);
 #pragma unroll
             for (int k = 0; k < kKeep; k++) {
                 const int i = threadIdx.x * 4 + k * step;
                 if (i >= p.n) continue;
-                const float4 h = apply(x.v[k], m, p.self, i);
-                y.v[k].x = fmaf(self, h.x, y.v[k].x); y.v[k].y = fmaf(self, h.y, y.v[k].y);
-                y.v[k].z = fmaf(self, h.z, y.v[k].z); y.v[k].w = fmaf(self, h.w, y.v[k].w);
+                const float4 g = *reinterpret_cast<const float4*>(p.self.w + i);
+                const float4 b = p.self.b ? *reinterpret_cast<const float4*>(p.self.b + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+                y.v[k].x = fmaf(self, fmaf((x.v[k].x - m.x) * m.y, g.x, b.x), y.v[k].x);
+                y.v[k].y = fmaf(self, fmaf((x.v[k].y - m.x) * m.y, g.y, b.y), y.v[k].y);
+                y.v[k].z = fmaf(self, fmaf((x.v[k].z - m.x) * m.y, g.z, b.z), y.v[k].z);
+                y.v[k].w = fmaf(self, fmaf((x.v[k].w - m.x) * m.y, g.w, b.w), y.v[k].w);
             }
         }
         if (p.post.w) {
-            const float2 m = moments(y, p.n_mean, p.post.b != nullptr, p.eps, red);
+            const float2 m = moments(y, p.n_mean, p.post.b != nullptr, inv_n, p.eps, red[1], kWarps);
 #pragma unroll
-            for (int k = 0; k < kKeep; k++) {
-                const int i = threadIdx.x * 4 + k * step;
-                if (i < p.n) y.v[k] = apply(y.v[k], m, p.post, i);
-            }
+            for (int k = 0; k < kKeep; k++) y.v[k] = w.apply(y.v[k], m, k);
+            if (p.next.w) w.load(p.next, p.n, step);
         }
 #pragma unroll
         for (int k = 0; k < kKeep; k++) {
             const int i = threadIdx.x * 4 + k * step;
-            x.v[k].x += y.v[k].x; x.v[k].y += y.v[k].y; x.v[k].z += y.v[k].z; x.v[k].w += y.v[k].w;
+            add(x.v[k], y.v[k]);
             if (i < p.n) *reinterpret_cast<float4*>(xr + i) = x.v[k];
         }
     }
     if (!p.next.w) return;
-    const float2 m = moments(x, p.n_mean, p.next.b != nullptr, p.eps, red);
+    const float2 m = moments(x, p.n_mean, p.next.b != nullptr, inv_n, p.eps, red[2], kWarps);
 #pragma unroll
     for (int k = 0; k < kKeep; k++) {
         const int i = threadIdx.x * 4 + k * step;
         if (i >= p.n) continue;
-        const float4 v = apply(x.v[k], m, p.next, i);
+        const float4 v = w.apply(x.v[k], m, k);
         const size_t at = (size_t)row * p.n + i;
         if (p.out) *reinterpret_cast<float4*>(p.out + at) = v;
         if (p.hi) {
@@ -149,12 +168,12 @@ extern "C" cudaError_t ingot_residual_norm_run(const ingot_residual_norm* r, cud
     if (!r->x || r->n < 4 || r->n % 4 != 0 || r->n_mean < 1 || r->n_mean > r->n || r->n_rows < 1 || (r->n_slices > 0 && !r->product) ||
         (r->top > 0 && (!r->branch || !r->row_of)) || (r->self_gain && !r->self.w) || (r->next.w && !r->out && !r->hi))
         return cudaErrorInvalidValue;
-    auto run = [&](auto kernel, int threads) { return ingot_launch_pdl(kernel, dim3(r->n_rows), dim3(threads), 0, s, *r); };
+    auto run = [&](auto kernel, int threads) { return ingot_launch_pdl(kernel, dim3(r->n_rows), dim3(threads), 0, s, *r, 1.0f / float(r->n_mean)); };
     const int quads = r->n / 4;
     auto warps = [&](int keep) { return (quads + 32 * keep - 1) / (32 * keep) * 32; };  // threads that hold a row of `keep` quads each
-    if (quads <= 256) return run(residual_norm_kernel<1, 256>, warps(1));
-    if (quads <= 1024) return run(residual_norm_kernel<4, 256>, warps(4));
-    if (quads <= 2048) return run(residual_norm_kernel<8, 256>, 256);
-    if (quads <= 8192) return run(residual_norm_kernel<8, 1024>, 1024);
+    if (quads <= 256) return run(residual_norm_kernel<1, 256, 2>, warps(1));
+    if (quads <= 1024) return run(residual_norm_kernel<4, 256, 2>, warps(4));
+    if (quads <= 2048) return run(residual_norm_kernel<4, 512, 1>, warps(4));
+    if (quads <= 8192) return run(residual_norm_kernel<8, 1024, 1>, 1024);
     return cudaErrorInvalidValue;
 }

@@ -14,10 +14,14 @@
 // of prompts on tcgen05 (attn_gqa_sm100.cu); decoded tokens and short portions on warp-level MMAs, the keys split over CTAs (here); any
 // size in f32 arithmetic (the plain kernel of attn_shared_kv.cu).
 #include <algorithm>
+#include <cstdlib>
 
 #include "attn_shared_kv.cuh"
+#include "sm100_ptx.cuh"
 
 namespace {
+
+using namespace ingot_sm100;
 
 __device__ __forceinline__ float warp_sum(float v) {
 #pragma unroll
@@ -37,7 +41,7 @@ __device__ __forceinline__ float dot4(float4 v, float acc) {
 constexpr int kMaxRot = 1024;  // rotated values per head
 constexpr int kAppendThreads = 256;
 
-// One CTA per token, a warp per head: queries out, keys and values into the cache.
+// A warp per head, one CTA or a few per token: queries out, keys and values into the cache.
 struct AppendParams {
     ingot_step st;
     const float* proj;
@@ -95,7 +99,7 @@ __global__ void __launch_bounds__(kAppendThreads) gqa_append_kernel(const Append
     const int blk = table_block(p.tables, p.first_page, p.max_blocks, p.n_blocks, seq, p.map.page(pos), p.status);
     T* page = static_cast<T*>(p.rows) + ((size_t)max(blk, 0) * G * kBlockTokens + p.map.slot(pos)) * (dim + vdim);  // of KV head 0
     const size_t head_stride = (size_t)kBlockTokens * (dim + vdim);
-    for (int h = warp; h < H + G; h += kAppendThreads / 32) {
+    for (int h = blockIdx.y * (kAppendThreads / 32) + warp; h < H + G; h += gridDim.y * (kAppendThreads / 32)) {
         const bool is_q = h < H;
         const float* src = row + (is_q ? p.q_off + h * dim : p.k_off + (h - H) * dim);
         const float* w = is_q ? p.q_norm : p.k_norm;
@@ -129,7 +133,7 @@ __global__ void __launch_bounds__(kAppendThreads) gqa_append_kernel(const Append
         }
     }
     const float keep = 1.0f - p.mix;
-    for (int i = threadIdx.x * 4; i < G * vdim; i += kAppendThreads * 4) {
+    for (int i = (blockIdx.y * kAppendThreads + threadIdx.x) * 4; i < G * vdim; i += gridDim.y * kAppendThreads * 4) {
         float4 v = *reinterpret_cast<const float4*>(row + p.v_off + i);
         if (p.first_values) {
             float4* f = reinterpret_cast<float4*>(p.first_values + (size_t)tok * G * vdim + i);
@@ -146,19 +150,23 @@ __global__ void __launch_bounds__(kAppendThreads) gqa_append_kernel(const Append
 
 // ---- decoded tokens and short portions: f16, m16n8k16 MMAs, the keys split over CTAs ---------------------------------------------------
 // A CTA serves 16 (token, head) rows of one KV head of one sequence over one share of the pages they see. Its four warps take every fourth
-// page each through a cp.async ring of their own - no barrier in the key loop - the block table of the share is in shared memory first, so
-// that no copy waits for an address. The warps' states are merged through shared memory; several shares are merged by a second launch.
-// kMax: most columns of a key or a value; the loops over 16-column steps stop at the true sizes.
-constexpr int kRing = 3, kWarps = 4, kMaxSharePages = 1024, kMaxSplits = 64, kSplitKeysMin = 128;
+// page each through a ring of bulk copies of their own - a lane fetches a slot's row, no barrier in the key loop - the block table of the
+// share is in shared memory first, so that no copy waits for an address. The warps' states are merged through shared memory; several shares
+// are merged by a second launch. kMax: most columns of a key or a value; the loops over 16-column steps stop at the true sizes.
+// Waits for copies are bounded: a warp that gives up waits, again bounded, for those in flight and raises the status word.
+constexpr unsigned long long kWaitLimitNs = 2000000000ull;
+constexpr int kMaxRing = 3, kWarps = 4, kMaxSharePages = 1024, kMaxSplits = 64, kSplitKeysMin = 128;
 constexpr int kSmemLimit = 227 * 1024;
 struct GqaSmem {
     int stride, page_bytes, blocks, bytes;  // stride: halves between rows, 16 bytes past the row so that ldmatrix has no bank conflicts
+    int ring;                             // pages per warp: three, or two where that lets two CTAs share an SM
     __host__ __device__ GqaSmem(int row, int vdim, int share_pages) {
         stride = row + 8;
         page_bytes = kBlockTokens * stride * 2;
-        blocks = kWarps * kRing * page_bytes;
-        const int ring = blocks + share_pages * 4, merge = kWarps * 16 * (vdim + 2) * 4;
-        bytes = ring > merge ? ring : merge;
+        ring = kWarps * kMaxRing * page_bytes <= 104 * 1024 ? kMaxRing : 2;
+        blocks = kWarps * ring * page_bytes;
+        const int loop = blocks + share_pages * 4, merge = kWarps * 16 * (vdim + 2) * 4;
+        bytes = loop > merge ? loop : merge;
     }
 };
 __device__ __forceinline__ void ldmatrix4(uint32_t (&r)[4], uint32_t addr) {
@@ -167,20 +175,25 @@ __device__ __forceinline__ void ldmatrix4(uint32_t (&r)[4], uint32_t addr) {
 __device__ __forceinline__ void ldmatrix4_trans(uint32_t (&r)[4], uint32_t addr) {
     asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
 }
-__device__ __forceinline__ void cp16(uint32_t dst, const void* src, bool on) {
-    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(on ? 16 : 0) : "memory");
+__device__ __forceinline__ float ex2(float x) {
+    float y;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+    return y;
 }
 
 template <int kMax>
 __global__ void __launch_bounds__(kWarps * 32) gqa_mma_kernel(const AttendParams p, int share_pages) {
     constexpr int kK = kMax / 16, kN = kMax / 8;
     extern __shared__ __align__(16) unsigned char smem[];
+    __shared__ uint64_t s_full[kWarps][kMaxRing];
+    __shared__ uint32_t s_abort;
     INGOT_PDL_TRIGGER();
     INGOT_PDL_WAIT();
     const int seq = blockIdx.z, kvh = blockIdx.y, group = p.n_head / p.n_head_kv, n_rows = p.st.len[seq] * group;
     const int split = blockIdx.x % p.n_splits, row0 = blockIdx.x / p.n_splits * 16;
     if (row0 >= n_rows) return;
     const GqaSmem L(p.dim, p.out_dim, share_pages);
+    const int ring = L.ring;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, j = lane & 3;
     const int pos0 = p.st.pos0[seq], n_k = p.q_dim / 16, n_v = p.out_dim / 16;
     const size_t tok0 = p.st.row_start[seq];
@@ -188,28 +201,25 @@ __global__ void __launch_bounds__(kWarps * 32) gqa_mma_kernel(const AttendParams
     const int page_a = p.map.page(p.map.first_visible(pos_first)), n_pages = p.map.page(pos_last) - page_a + 1;
     const int per = (n_pages + p.n_splits - 1) / p.n_splits, first = split * per, count = max(0, min(min(per, share_pages), n_pages - first));
     const __half* rows = static_cast<const __half*>(p.rows);
-    const uint32_t s_ring = (uint32_t)__cvta_generic_to_shared(smem) + warp * kRing * L.page_bytes;
+    const uint32_t s_ring = (uint32_t)__cvta_generic_to_shared(smem) + warp * ring * L.page_bytes;
     int* s_blk = reinterpret_cast<int*>(smem + L.blocks);
     for (int i = threadIdx.x; i < count; i += kWarps * 32)
         s_blk[i] = table_block(p.tables, p.first_page, p.max_blocks, p.n_blocks, seq, page_a + first + i, p.status);
+    if (threadIdx.x == 0) s_abort = 0;
+    if (lane < ring) mbar_init(smem_u32(&s_full[warp][lane]), 1);
+    asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
     __syncthreads();
 
-    const int pieces = p.dim / 8;  // 16-byte pieces of a row
-    auto stage = [&](int i, int buf) {  // page i of the share
-        if (i < count) {
-            const int blk = s_blk[i];
-            const __half* src = rows + ((size_t)max(blk, 0) * p.n_head_kv + kvh) * kBlockTokens * p.dim;
-            const uint32_t dst = s_ring + buf * L.page_bytes;
-            int slot = lane / pieces, c = lane - slot * pieces;
-            for (int k = lane; k < kBlockTokens * pieces; k += 32) {
-                cp16(dst + (slot * L.stride + c * 8) * 2, src + k * 8, blk >= 0);
-                for (c += 32; c >= pieces; c -= pieces) slot++;
-            }
-        }
-        asm volatile("cp.async.commit_group;" ::: "memory");
+    const uint32_t row_bytes = p.dim * 2;
+    auto stage = [&](int i, int buf) {  // page i of the share; one without a block comes from block 0 and is masked
+        if (i >= count) return;
+        const uint32_t full = smem_u32(&s_full[warp][buf]);
+        if (lane == 0) mbar_expect_tx(full, kBlockTokens * row_bytes);
+        __syncwarp();
+        if (lane < kBlockTokens)
+            bulk_load(s_ring + buf * L.page_bytes + lane * L.stride * 2, rows + (((size_t)max(s_blk[i], 0) * p.n_head_kv + kvh) * kBlockTokens + lane) * p.dim, row_bytes, full);
     };
-#pragma unroll
-    for (int k = 0; k < kRing - 1; k++) stage(warp + k * kWarps, k);
+    for (int k = 0; k < ring - 1; k++) stage(warp + k * kWarps, k);
 
     const int r_lo = row0 + g, r_hi = r_lo + 8;
     const int pos_lo = pos0 + min(r_lo, n_rows - 1) / group, pos_hi = pos0 + min(r_hi, n_rows - 1) / group;
@@ -234,38 +244,55 @@ __global__ void __launch_bounds__(kWarps * 32) gqa_mma_kernel(const AttendParams
     for (int i = 0; i < kN; i++) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
     const float scale = p.scale * 1.44269504f;
 
-    int buf = 0;
+    const int vis_max = p.map.first_visible(pos_last);
+    int buf = 0, round = 0;
     for (int i = warp; i < count; i += kWarps) {
-        asm volatile("cp.async.wait_group %0;" ::"n"(kRing - 2) : "memory");
-        __syncwarp();  // the page is in, and every lane is done with the buffer that is staged next
-        stage(i + (kRing - 1) * kWarps, buf == 0 ? kRing - 1 : buf - 1);
+        const bool ok = mbar_wait(smem_u32(&s_full[warp][buf]), round & 1, &s_abort, kWaitLimitNs);
+        if (!__all_sync(0xffffffffu, ok)) {
+            for (int k = i, b = buf, r = round; k < min(count, i + (ring - 1) * kWarps); k += kWarps) {  // what is in flight must land first
+                const uint64_t t0 = globaltimer_ns();
+                while (!mbar_try_wait(smem_u32(&s_full[warp][b]), r & 1) && globaltimer_ns() - t0 < 100000000ull) {}
+                if (++b == ring) { b = 0; r++; }
+            }
+            break;
+        }
+        // every lane is done with the buffer that is staged next: the votes above came after its last use
+        stage(i + (ring - 1) * kWarps, buf == 0 ? ring - 1 : buf - 1);
         const uint32_t page = s_ring + buf * L.page_bytes;
-        float s[2][4];
+        float s[2][4], s2[2][4];
 #pragma unroll
-        for (int e = 0; e < 4; e++) s[0][e] = s[1][e] = 0.f;
+        for (int e = 0; e < 4; e++) s[0][e] = s[1][e] = s2[0][e] = s2[1][e] = 0.f;
         const uint32_t a = page + (((lane & 7) + ((lane >> 4) & 1) * 8) * L.stride + ((lane >> 3) & 1) * 8) * 2;
 #pragma unroll
-        for (int k = 0; k < kK; k++) {
+        for (int k = 0; k < kK; k += 2) {  // even and odd steps in sums of their own: shorter chains
             if (k >= n_k) break;
             uint32_t b[4];
             ldmatrix4(b, a + k * 32);
             mma_16816(s[0], qf[k][0], qf[k][1], qf[k][2], qf[k][3], b[0], b[1]);
             mma_16816(s[1], qf[k][0], qf[k][1], qf[k][2], qf[k][3], b[2], b[3]);
+            if (k + 1 >= n_k) break;
+            ldmatrix4(b, a + k * 32 + 32);
+            mma_16816(s2[0], qf[k + 1][0], qf[k + 1][1], qf[k + 1][2], qf[k + 1][3], b[0], b[1]);
+            mma_16816(s2[1], qf[k + 1][0], qf[k + 1][1], qf[k + 1][2], qf[k + 1][3], b[2], b[3]);
         }
-        const int key0 = (page_a + first + i) * kBlockTokens + 2 * j;
-        const bool held = s_blk[i] >= 0;
-        float mx_lo = -INFINITY, mx_hi = -INFINITY;
 #pragma unroll
-        for (int nt = 0; nt < 2; nt++) {
-#pragma unroll
-            for (int e = 0; e < 2; e++) {
-                const int key = key0 + nt * 8 + e;
-                s[nt][e] = held && key >= vis_lo && key <= pos_lo ? s[nt][e] * scale : -INFINITY;
-                s[nt][2 + e] = held && key >= vis_hi && key <= pos_hi ? s[nt][2 + e] * scale : -INFINITY;
-            }
-            mx_lo = fmaxf(mx_lo, fmaxf(s[nt][0], s[nt][1]));
-            mx_hi = fmaxf(mx_hi, fmaxf(s[nt][2], s[nt][3]));
+        for (int e = 0; e < 4; e++) {
+            s[0][e] = (s[0][e] + s2[0][e]) * scale;
+            s[1][e] = (s[1][e] + s2[1][e]) * scale;
         }
+        const int key_first = (page_a + first + i) * kBlockTokens;
+        if (key_first < vis_max || key_first + kBlockTokens - 1 > pos_first || s_blk[i] < 0) {  // some row does not see all of the page
+            const bool held = s_blk[i] >= 0;
+#pragma unroll
+            for (int nt = 0; nt < 2; nt++)
+#pragma unroll
+                for (int e = 0; e < 2; e++) {
+                    const int key = key_first + 2 * j + nt * 8 + e;
+                    if (!held || key < vis_lo || key > pos_lo) s[nt][e] = -INFINITY;
+                    if (!held || key < vis_hi || key > pos_hi) s[nt][2 + e] = -INFINITY;
+                }
+        }
+        float mx_lo = fmaxf(fmaxf(s[0][0], s[0][1]), fmaxf(s[1][0], s[1][1])), mx_hi = fmaxf(fmaxf(s[0][2], s[0][3]), fmaxf(s[1][2], s[1][3]));
         mx_lo = fmaxf(mx_lo, __shfl_xor_sync(0xffffffffu, mx_lo, 1));
         mx_lo = fmaxf(mx_lo, __shfl_xor_sync(0xffffffffu, mx_lo, 2));
         mx_hi = fmaxf(mx_hi, __shfl_xor_sync(0xffffffffu, mx_hi, 1));
@@ -273,14 +300,14 @@ __global__ void __launch_bounds__(kWarps * 32) gqa_mma_kernel(const AttendParams
         const float mn_lo = fmaxf(m_lo, mx_lo), mn_hi = fmaxf(m_hi, mx_hi);
         // a row that has not seen a key yet keeps -inf; 0 stands in for it in the exponents
         const float rf_lo = mn_lo == -INFINITY ? 0.f : mn_lo, rf_hi = mn_hi == -INFINITY ? 0.f : mn_hi;
-        const float a_lo = exp2f(m_lo - rf_lo), a_hi = exp2f(m_hi - rf_hi);
+        const float a_lo = ex2(m_lo - rf_lo), a_hi = ex2(m_hi - rf_hi);
         m_lo = mn_lo;
         m_hi = mn_hi;
         uint32_t pa[4];
         float sum_lo = 0.f, sum_hi = 0.f;
 #pragma unroll
         for (int nt = 0; nt < 2; nt++) {
-            const float p0 = exp2f(s[nt][0] - rf_lo), p1 = exp2f(s[nt][1] - rf_lo), p2 = exp2f(s[nt][2] - rf_hi), p3 = exp2f(s[nt][3] - rf_hi);
+            const float p0 = ex2(s[nt][0] - rf_lo), p1 = ex2(s[nt][1] - rf_lo), p2 = ex2(s[nt][2] - rf_hi), p3 = ex2(s[nt][3] - rf_hi);
             sum_lo += p0 + p1;
             sum_hi += p2 + p3;
             pa[nt * 2] = pack_half2_rn(p0, p1);
@@ -301,7 +328,7 @@ __global__ void __launch_bounds__(kWarps * 32) gqa_mma_kernel(const AttendParams
             mma_16816(o[2 * d], pa[0], pa[1], pa[2], pa[3], b[0], b[1]);
             mma_16816(o[2 * d + 1], pa[0], pa[1], pa[2], pa[3], b[2], b[3]);
         }
-        buf = buf + 1 == kRing ? 0 : buf + 1;
+        if (++buf == ring) { buf = 0; round++; }
     }
 
     l_lo += __shfl_xor_sync(0xffffffffu, l_lo, 1);
@@ -310,8 +337,8 @@ __global__ void __launch_bounds__(kWarps * 32) gqa_mma_kernel(const AttendParams
     l_hi += __shfl_xor_sync(0xffffffffu, l_hi, 2);
 
     // merge the warps' states: [warp][16 rows][out_dim] and (m, l)
-    asm volatile("cp.async.wait_group 0;" ::: "memory");
     __syncthreads();
+    if (threadIdx.x == 0 && s_abort) atomicOr(p.status, kDevErrBarrierTimeout);
     const int dv = p.out_dim;
     float* so = reinterpret_cast<float*>(smem);
     float* sml = so + kWarps * 16 * dv;
@@ -465,7 +492,9 @@ int ingot_gqa_append(ingot_skv* kv, int layer, const ingot_step* step, const flo
                       q_out_dev, static_cast<char*>(kv->rows) + kv->layer_elems * layer * esz, tables_dev, first_page_dev, max_blocks, kv->n_blocks, page_map(kv),
                       kv->status_dev};
     auto kernel = kv->dtype == INGOT_F32 ? gqa_append_kernel<float> : gqa_append_kernel<__half>;
-    INGOT_CUDA_TRY(ingot_launch_pdl(kernel, dim3(step->n_tok), dim3(kAppendThreads), 0, static_cast<cudaStream_t>(stream), p));
+    // few tokens: a CTA per eight heads, so that no warp has several in a row
+    const int heads = shape->n_head + shape->n_head_kv, parts = step->n_tok <= 64 ? std::min(8, (heads + 7) / 8) : 1;
+    INGOT_CUDA_TRY(ingot_launch_pdl(kernel, dim3(step->n_tok, parts), dim3(kAppendThreads), 0, static_cast<cudaStream_t>(stream), p));
     return INGOT_OK;
 }
 
@@ -485,8 +514,11 @@ int ingot_gqa_attend(ingot_skv* kv, int layer, const ingot_step* step, const voi
                       false, sink_dev, shape->dim, shape->dim, OutGate{gate_dev, gate_ld, gate_per_head}};
     cudaStream_t s = static_cast<cudaStream_t>(stream);
     if (kv->dtype == INGOT_F16) {
-        const long long rows = (long long)step->max_len * (shape->n_head / shape->n_head_kv);
-        if ((impl == 3 || (impl == 0 && rows >= INGOT_GQA_LONG_ROWS)) && gqa_sm100_takes(shape->dim, shape->vdim, scale) && out->ld % 4 == 0) {
+        // The split-key kernel fills the GPU with any number of rows and reads the keys once per 16 of a KV head, the tcgen05 one walks them
+        // in one CTA per 256: it wins when there are rows for many CTAs. INGOT_GQA_LONG sets the number.
+        const char* env = getenv("INGOT_GQA_LONG");
+        const long long least = env ? atoll(env) : INGOT_GQA_LONG_ROWS, rows = (long long)step->n_seq * step->max_len * shape->n_head;
+        if ((impl == 3 || (impl == 0 && step->max_len > 1 && rows >= least)) && gqa_sm100_takes(shape->dim, shape->vdim, scale) && out->ld % 4 == 0) {
             const int rc = launch_gqa_sm100(kv, layer, p, s);
             if (rc != INGOT_ERR_UNSUPPORTED || impl == 3) return rc;
         }

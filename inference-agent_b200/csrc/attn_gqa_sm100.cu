@@ -49,6 +49,7 @@ __device__ __forceinline__ float ex2(float x) {
     asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
     return y;
 }
+__device__ __forceinline__ float sigmoid(float z) { return __fdividef(1.0f, 1.0f + ex2(-1.44269504f * z)); }  // z -> -inf: 1 / inf
 __device__ __forceinline__ void ffma2(float& d0, float& d1, float a0, float a1, float b, float c) {
     asm("{\n.reg .b64 ra, rb, rc, rd;\n"
         "mov.b64 ra, {%2, %3};\nmov.b64 rb, {%4, %4};\nmov.b64 rc, {%5, %5};\n"
@@ -329,6 +330,21 @@ gqa_sm100_kernel(const __grid_constant__ CUtensorMap map_rows, const __grid_cons
             if (lane == 0) mbar_arrive(smem_u32(&bars->p_ready[q]));
         }
         // ---------------- epilogue: O / l through the tile's Q buffer, row-contiguous stores ----------------
+        const int my_row = valid ? (int)(tok0 + tok) : -1, warp_row0 = (warp & 3) << 5, piece = lane & 7;
+        float4 gates[8];  // of the rows and columns this lane stores in a pass, requested ahead of the result
+        auto load_gates = [&](int ps) {
+            if (!p.gate.z) return;
+            const int d = ps * 32 + piece * 4;
+#pragma unroll
+            for (int it = 0; it < 8; it++) {
+                const int owner = it * 4 + (lane >> 3);
+                const int row = __shfl_sync(0xffffffffu, my_row, owner), h = __shfl_sync(0xffffffffu, head, owner);
+                if (row < 0 || d >= p.out_dim) continue;
+                const float* z = p.gate.z + (size_t)row * p.gate.ld;
+                gates[it] = p.gate.per_head ? make_float4(z[h], z[h], z[h], z[h]) : *reinterpret_cast<const float4*>(z + h * p.out_dim + d);
+            }
+        };
+        load_gates(0);
         if (ok) {
             ok = mbar_wait(smem_u32(&bars->o_final[q]), 0, abort_flag, kWaitLimitNs);
             ok = __all_sync(0xffffffffu, ok) != 0;
@@ -343,9 +359,11 @@ gqa_sm100_kernel(const __grid_constant__ CUtensorMap map_rows, const __grid_cons
                 inv = 1.0f / l;
             }
             unsigned char* stage = smem_al + q * nq * kUnit;  // [128 rows][32 f32], 16-byte pieces XOR-swizzled by row
-            const int my_row = valid ? (int)(tok0 + tok) : -1, warp_row0 = (warp & 3) << 5, piece = lane & 7;
             for (int ps = 0; ps < 2 * nv && ps * 32 < p.out_dim; ps++) {
-                if (ps) __syncwarp();
+                if (ps) {
+                    load_gates(ps);
+                    __syncwarp();
+                }
                 unsigned char* my = stage + row_in_tile * 128;
                 float o[32];
                 tmem_ld32(o_tmem + ps * 32, o);
@@ -355,16 +373,24 @@ gqa_sm100_kernel(const __grid_constant__ CUtensorMap map_rows, const __grid_cons
                     *reinterpret_cast<float4*>(my + ((i ^ (row_in_tile & 7)) << 4)) = make_float4(o[4 * i] * inv, o[4 * i + 1] * inv, o[4 * i + 2] * inv, o[4 * i + 3] * inv);
                 __syncwarp();
                 const int d = ps * 32 + piece * 4;
-#pragma unroll 4
+#pragma unroll
                 for (int it = 0; it < 8; it++) {
                     const int owner = it * 4 + (lane >> 3);
                     const int row = __shfl_sync(0xffffffffu, my_row, owner), h = __shfl_sync(0xffffffffu, head, owner);
                     if (row < 0 || d >= p.out_dim) continue;
                     const int r = warp_row0 + owner;
-                    const float4 v = *reinterpret_cast<const float4*>(stage + r * 128 + ((piece ^ (r & 7)) << 4));
-                    const float4 z = p.gate.at4(row, h, p.out_dim, d);
-                    p.out.store2(row, h * p.out_dim + d, v.x * z.x, v.y * z.y);  // out_dim is a multiple of 16
-                    p.out.store2(row, h * p.out_dim + d + 2, v.z * z.z, v.w * z.w);
+                    float4 v = *reinterpret_cast<const float4*>(stage + r * 128 + ((piece ^ (r & 7)) << 4));
+                    if (p.gate.z) { v.x *= sigmoid(gates[it].x); v.y *= sigmoid(gates[it].y); v.z *= sigmoid(gates[it].z); v.w *= sigmoid(gates[it].w); }
+                    const size_t e = (size_t)row * p.out.ld + h * p.out_dim + d;  // out_dim is a multiple of 16
+                    if (p.out.f32) *reinterpret_cast<float4*>(p.out.f32 + e) = v;
+                    if (p.out.hi) {
+                        const __nv_bfloat162 a = __floats2bfloat162_rn(v.x, v.y), b = __floats2bfloat162_rn(v.z, v.w);
+                        *reinterpret_cast<uint2*>(p.out.hi + e) = make_uint2(*reinterpret_cast<const uint32_t*>(&a), *reinterpret_cast<const uint32_t*>(&b));
+                        if (p.out.lo) {
+                            const __nv_bfloat162 c = __floats2bfloat162_rn(v.x - __low2float(a), v.y - __high2float(a)), f = __floats2bfloat162_rn(v.z - __low2float(b), v.w - __high2float(b));
+                            *reinterpret_cast<uint2*>(p.out.lo + e) = make_uint2(*reinterpret_cast<const uint32_t*>(&c), *reinterpret_cast<const uint32_t*>(&f));
+                        }
+                    }
                 }
             }
         }

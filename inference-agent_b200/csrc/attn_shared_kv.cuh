@@ -80,16 +80,6 @@ struct OutGate {
         if (!z) return 1.0f;
         return sigmoid(z[row * ld + (per_head ? head : head * out_dim + d)]);
     }
-    // Columns d..d+3 of a head; rows, heads and d start on 16 bytes.
-    __device__ __forceinline__ float4 at4(size_t row, int head, int out_dim, int d) const {
-        if (!z) return make_float4(1.f, 1.f, 1.f, 1.f);
-        if (per_head) {
-            const float g = sigmoid(z[row * ld + head]);
-            return make_float4(g, g, g, g);
-        }
-        const float4 v = *reinterpret_cast<const float4*>(z + row * ld + head * out_dim + d);
-        return make_float4(sigmoid(v.x), sigmoid(v.y), sigmoid(v.z), sigmoid(v.w));
-    }
 };
 
 // Block of a page of sequence `seq` (index within the step), or -1 with the status bit raised if the table has none.

@@ -62,6 +62,37 @@ def test_reach_of_a_window(tmp_path, window, f32, decoded):
             assert (moved[j:j + window] > 1e-6).all()
 
 
+@pytest.mark.parametrize("least", ["1", "300", "1000000"])
+def test_the_kernel_a_portion_takes_does_not_show(tmp_path, monkeypatch, least):
+    """Portions of all sizes of several sequences beside single tokens, on either kernel or on both in turn, against the plain implementation."""
+    monkeypatch.setenv("INGOT_GQA_LONG", least)
+    cfg = S.config([S.layer("attention", 6, 2, 40, 24, 90, rot=20, scale=0.15, mlp=S.dense(40)), S.layer("attention_2", 3, 1, 72, 48, scale=0.1, v_mix=False),
+                    S.layer("attention_3", 4, 2, 16, 24, rot=8, mlp=S.moe(3, 2, 5, None, 24, 16))], vocab=40, width=44)
+    w = S.random_weights(cfg, 4)
+    rng = np.random.default_rng(0)
+    tokens = [rng.integers(0, 40, n).tolist() for n in (600, 330, 150)]
+    want = [S.reference_logits(cfg, w, t) for t in tokens]
+    with open_model(tmp_path, cfg, w, max_tokens=1152, max_seqs=3, max_step_tokens=320) as m:
+        at, got = [0, 0, 0], [[], [], []]
+        cuts = [[150, 2, 100, 1, 180, 3, 64], [40, 1, 39, 130, 120], [1, 2, 41, 100, 6]]
+        for k in range(40):
+            step = []
+            for s in range(3):
+                n = min(cuts[s][k % len(cuts[s])], len(tokens[s]) - at[s])
+                if n > 0:
+                    step.append((s, at[s], tokens[s][at[s]:at[s] + n], list(range(n))))
+            if not step:
+                break
+            rows, r = m.step(step), 0
+            for s, p, t, _ in step:
+                got[s].append(rows[r:r + len(t)])
+                r += len(t)
+                at[s] += len(t)
+        assert at == [600, 330, 150]
+        for s in range(3):
+            assert H.error(np.concatenate(got[s]), want[s]).max() < 4e-2, s
+
+
 def test_a_far_key_decides(tmp_path):
     """Layers that see everything: one token hundreds of positions back has a score far above all others, for a portion and for decoded
     tokens; taking it away shows."""
@@ -186,6 +217,6 @@ def test_refusals(tmp_path):
     missing = {k: v for k, v in w.items() if k != "l2.mix.sink"}
     with pytest.raises(M.ModelError, match="sink is missing"):
         open_model(tmp_path / "h", cfg, missing)
-    two = S.config([S.layer("attention_2", 2, 2, 8, 12), S.layer("attention_2", 2, 1, 8, 12)], vocab=20, width=16)
+    two = S.config([S.layer("attention_2", 2, 2, 8, 12), S.layer("attention_2", 2, 1, 8, 24)], vocab=20, width=16)
     with pytest.raises(M.ModelError, match="mix values"):
         open_model(tmp_path / "i", two, S.random_weights(two))
